@@ -16,7 +16,7 @@ from typing import Optional
 
 import torch
 
-from ..models.qwen3 import Qwen3ForCausalLM, load_target
+from ..models import is_model, load_target
 from ..sampling import SamplingParams, sample
 from ..tree import build_ancestor_matrix, get_algorithm, gpu_tree_accept, tree_accept
 from ..utils.timing import PhaseTimer
@@ -43,7 +43,7 @@ def decode_text(tokenizer, ids) -> str:
 class LLM:
     def __init__(self, model_name_or_path, device: str = "cuda", dtype: torch.dtype = torch.bfloat16,
                  attn_implementation: str = "sdpa", tokenizer=None):
-        if isinstance(model_name_or_path, Qwen3ForCausalLM):
+        if is_model(model_name_or_path):
             self.model = model_name_or_path.to(device=device, dtype=dtype)
             self.tokenizer = tokenizer
         else:

@@ -14,7 +14,8 @@ import torch
 
 
 class DenseKVCache:
-    """Contiguous ``(Hkv, capacity, D)`` K and V per layer with a shared length."""
+    """Contiguous ``(Hkv, capacity, D)`` K and V per layer with a shared length; a latent-attention model's latent rows
+    are held as ``k`` with one head (and no ``v``)."""
 
     def __init__(self, cfg, device, dtype, capacity: int = 512):
         self.cfg, self.device, self.dtype = cfg, device, dtype
@@ -25,12 +26,16 @@ class DenseKVCache:
         self._grow(capacity)
 
     def _grow(self, cap: int) -> None:
-        L, Hkv, D = self.cfg.num_hidden_layers, self.cfg.num_key_value_heads, self.cfg.head_dim
-        nk = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
-        nv = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
-        for i in range(len(self.k)):
-            nk[i][:, : self.length] = self.k[i][:, : self.length]
-            nv[i][:, : self.length] = self.v[i][:, : self.length]
+        widths = self.cfg.latent_widths()
+        if widths is not None:
+            nk, nv = [torch.zeros(1, cap, w, dtype=self.dtype, device=self.device) for w in widths], []
+        else:
+            L, Hkv, D = self.cfg.num_hidden_layers, self.cfg.num_key_value_heads, self.cfg.head_dim
+            nk = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
+            nv = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
+        for new, old in ((nk, self.k), (nv, self.v)):
+            for n, o in zip(new, old):
+                n[:, : self.length] = o[:, : self.length]
         self.k, self.v, self.capacity = nk, nv, cap
 
     def ensure(self, n: int) -> None:
@@ -51,7 +56,7 @@ class DenseKVCache:
         (reference: ``_select_kv_cache``, ``jetspec/core/llm.py:86-112``).
         """
         n = len(keep_tree_indices)
-        if (n and n <= 64 and self.k[0].is_cuda and self.k[0].dtype == torch.bfloat16 and self.k[0].shape[-1] == 128
+        if (n and n <= 64 and self.v and self.k[0].is_cuda and self.k[0].dtype == torch.bfloat16 and self.k[0].shape[-1] == 128
                 and self.k[0].is_contiguous()):
             from ..ops import cuda_ext as X                   # compaction kernel (rows staged in shared memory)
             keep = torch.as_tensor(keep_tree_indices, dtype=torch.int32).to(self.device)
@@ -62,7 +67,8 @@ class DenseKVCache:
         idx = torch.as_tensor(keep_tree_indices, dtype=torch.long, device=self.device) + past_len
         for i in range(len(self.k)):
             self.k[i][:, past_len:past_len + n] = self.k[i][:, idx]
-            self.v[i][:, past_len:past_len + n] = self.v[i][:, idx]
+            if self.v:
+                self.v[i][:, past_len:past_len + n] = self.v[i][:, idx]
         self.length = past_len + n
 
 
@@ -74,6 +80,8 @@ class ModelRunner:
     def _kernel_attention_ok(self, ids: torch.Tensor, T: int, ancestor) -> bool:
         cfg = self.cfg
         w = self.model.lm_head.weight
+        if cfg.latent_widths() is not None:
+            return False
         if not (ids.is_cuda and w.dtype == torch.bfloat16 and cfg.head_dim == 128):
             return False
         if cfg.sliding_window and any(t == "sliding_attention" for t in (cfg.layer_types or [])):
@@ -123,9 +131,6 @@ class ModelRunner:
         cache.ensure(past + T)
         pos = (position_ids.reshape(-1) if position_ids is not None
                else torch.arange(past, past + T, device=ids.device))
-        Hq, Hkv, D = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
-        g = Hq // Hkv
-        scale = 1.0 / math.sqrt(D)
         vis = torch.ones(T, past + T, dtype=torch.bool, device=ids.device)
         vis[:, past:] = (ancestor.to(ids.device) if ancestor is not None
                          else torch.tril(torch.ones(T, T, dtype=torch.bool, device=ids.device)))
@@ -134,6 +139,22 @@ class ModelRunner:
         use_kernel = bool(attn_kernel) and self._kernel_attention_ok(ids, T, ancestor)
         if use_kernel:
             kern = self._kernel_attention_args(cache, past, T, ancestor, ids.device)
+
+        latent_cache = cfg.latent_widths() is not None
+        if not latent_cache:
+            Hq, Hkv, D = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
+            g = Hq // Hkv
+            scale = 1.0 / math.sqrt(D)
+
+        def latent(layer: int, mixer, q, c):
+            """Latent attention as the plain formula over the contiguous cache: keys and values are expanded."""
+            cache.k[layer][0, past:past + T] = c
+            C, m = cache.k[layer][0, :past + T].float(), mixer.cfg
+            K = (C @ mixer.k_up.weight.float().t()).view(past + T, m.heads, m.dim)
+            V = (C @ mixer.v_up.weight.float().t()).view(past + T, m.heads, m.vdim)
+            s = torch.einsum("nhd,lhd->hnl", q.float(), K) * m.scale
+            p = torch.softmax(s.masked_fill(~vis[None], float("-inf")), -1)
+            return torch.einsum("hnl,lhv->nhv", p, V).reshape(T, m.heads * m.vdim).to(q.dtype)
 
         def attn(layer: int, q, k, v):
             cache.k[layer][:, past:past + T] = k.transpose(0, 1)
@@ -156,6 +177,7 @@ class ModelRunner:
             p = torch.softmax(s, -1)
             return torch.einsum("hgnl,hld->nhgd", p, V).reshape(T, Hq * D).to(q.dtype)
 
+        attn.latent = latent
         taps = list(target_layer_ids) if (output_hidden_states or target_layer_ids is not None) and target_layer_ids else None
         rows = slice(T - 1, T) if last_position_logits_only else None
         logits, hidden = self.model(ids, pos, attn, tap_layers=taps, logits_rows=rows)

@@ -30,8 +30,8 @@ import torch
 
 from .. import ops
 from ..core.llm import decode_text, resolve_eos
-from ..models.qwen3 import Qwen3ForCausalLM, load_target
-from ..runtime import PagedKVPool, Scheduler, SequenceRequest, build_attn_metadata
+from ..models import is_model, load_target
+from ..runtime import PagedAttention, PagedKVPool, Scheduler, SequenceRequest, build_attn_metadata
 from ..sampling import SamplingParams, sample
 from ..tree import (build_from_topk, get_algorithm, gpu_tree_accept, should_extend, splice_extension,
                     tree_accept)
@@ -104,7 +104,7 @@ class JetSpecEngine:
                  expert_parallel=None):
         if attn_backend not in _BACKEND_ALIASES:
             raise ValueError(f"unknown attn_backend {attn_backend!r}; expected one of {sorted(_BACKEND_ALIASES)}")
-        if isinstance(model_name_or_path, Qwen3ForCausalLM):
+        if is_model(model_name_or_path):
             self.model = model_name_or_path.to(device=device, dtype=dtype)
             self.tokenizer = tokenizer
         else:
@@ -160,10 +160,21 @@ class JetSpecEngine:
             # frozen but idle and outside a session: the graphs captured against the old pool are dropped with it
             # (self._fast below) and captured again on demand
         world = self.tp.world if getattr(self, "tp", None) is not None else 1
-        self.pool = PagedKVPool(self.cfg.num_hidden_layers, self.cfg.num_key_value_heads // world, self.cfg.head_dim,
-                                max(want_pages, 2), page_size=self.block_size,
-                                max_seqs=max(self._max_seqs, seqs), max_seq_len=max_len,
-                                device=self.device, dtype=self.dtype)
+        self.pool = PagedKVPool.for_model(self.cfg, max(want_pages, 2), world=world, page_size=self.block_size,
+                                          max_seqs=max(self._max_seqs, seqs), max_seq_len=max_len,
+                                          device=self.device, dtype=self.dtype)
+        self._fast = None
+        return self.pool
+
+    def reserve_pool(self, max_tokens: int, max_seqs: int) -> PagedKVPool:
+        """A fresh pool of exactly ``max_tokens`` positions (rounded up to whole pages) and ``max_seqs`` sequences, for
+        callers that drive :meth:`step` themselves.  Nothing may be resident."""
+        if self.pool is not None and self.pool.resident():
+            raise RuntimeError("cannot replace the KV pool while sequences are resident")
+        pages = (int(max_tokens) + self.block_size - 1) // self.block_size
+        self._num_pages, self._max_seqs, self._max_seq_len = pages, int(max_seqs), pages * self.block_size
+        self.pool = PagedKVPool.for_model(self.cfg, pages, page_size=self.block_size, max_seqs=int(max_seqs),
+                                          max_seq_len=pages * self.block_size, device=self.device, dtype=self.dtype)
         self._fast = None
         return self.pool
 
@@ -191,16 +202,47 @@ class JetSpecEngine:
                                    num_query_nodes=None if trees is not None else [int(t.numel()) for t in token_rows],
                                    device=self.device)
         ids = torch.cat([t.reshape(-1) for t in token_rows]).to(self.device)
-        scale = 1.0 / math.sqrt(self.cfg.head_dim)
-
-        def attn(layer, q, k, v):
-            kp, vp = pool.layer(layer)
-            ops.kv_scatter(k, v, kp, vp, meta.slots)
-            return ops.paged_tree_attention(q, kp, vp, pool.slot_map, meta.seq_rows, meta.cu_q, meta.past_lens,
-                                            meta.mask_bits, scale, causal=meta.causal, max_q=meta.max_q)
-
+        if self.ragged_kernels:
+            from .fast_round import FastRound
+            logits, hidden = FastRound.get(self).ragged_forward(ids, meta, past_lens, taps, logits_rows)
+            return logits, hidden, meta
+        head_dim = getattr(self.cfg, "head_dim", None)          # latent attention carries its own scale
+        attn = PagedAttention(pool, meta, 1.0 / math.sqrt(head_dim) if head_dim else 1.0)
         logits, hidden = self.model(ids, meta.positions.long(), attn, tap_layers=taps, logits_rows=logits_rows)
         return logits, hidden, meta
+
+    @property
+    def ragged_kernels(self) -> bool:
+        """Whether ragged forwards (portions of prompts beside decoded tokens) run on the fused kernel stack; K/V models
+        run theirs through the module path's kernels."""
+        return self.use_kernels and self.cfg.latent_widths() is not None and self.cfg.kernel_path_ok()
+
+    @torch.inference_mode()
+    def step(self, entries):
+        """Run the next tokens of several sequences as ONE ragged batch, from the cache earlier steps left.
+
+        ``entries``: ``[(seq_id, tokens, want), ...]``, ``tokens`` a list of ids and ``want`` the places among them
+        whose logits are returned.  Portions may be cut anywhere and stand beside single decoded tokens.  The cache
+        positions are reserved here; a sequence's length advances by its tokens.  Returns the wanted logits
+        ``(sum of wants, vocab)`` in the order of the entries (``None`` when nothing is wanted)."""
+        pool = self.pool
+        order = sorted(range(len(entries)), key=lambda i: len(entries[i][1]))    # short portions first: see FastRound
+        seqs, rows, past, start, first = [], [], [], {}, 0
+        for i in order:
+            sid, toks, _ = entries[i]
+            have = pool.state(sid).length if pool.has(sid) else 0
+            pool.reserve(sid, have + len(toks))
+            seqs.append(sid)
+            rows.append(torch.tensor(toks, dtype=torch.long, device=self.device))
+            past.append(have)
+            start[i] = first
+            first += len(toks)
+        want = [start[i] + int(k) for i, (_, _, w) in enumerate(entries) for k in w]
+        logits, _, _ = self._forward(seqs, rows, past, logits_rows=torch.tensor(want, dtype=torch.long, device=self.device))
+        for sid, have, toks in zip(seqs, past, rows):
+            pool.state(sid).length = have + int(toks.numel())
+            pool.touch(sid)
+        return logits if want else None
 
     def _prefill(self, seq_id: int, ids: torch.Tensor, taps=None, reserve: int = 0):
         """Causal prefill of one sequence; returns ``(last-row logits, tap hidden (T, taps*H))``."""
@@ -218,7 +260,7 @@ class JetSpecEngine:
         if self.tp is not None and temperature > 0.0:
             raise NotImplementedError("tensor-parallel batches decode greedily")
         kernel_path = self.tp is not None
-        if not kernel_path and self.use_kernels and temperature <= 0.0 and self.cfg.head_dim == 128:
+        if not kernel_path and self.use_kernels and temperature <= 0.0 and self.cfg.kernel_path_ok():
             from .fast_round import FastRound
             kernel_path = FastRound.get(self)._kernel_prefill_ok()      # the same prompt path as single requests
         if kernel_path:
@@ -456,12 +498,14 @@ class JetSpecEngine:
 
     @torch.inference_mode()
     def generate_batch(self, prompts: list, sampling_params: SamplingParams = None,
-                       max_batch_size: Optional[int] = None) -> list:
+                       max_batch_size: Optional[int] = None, prefill_chunk: Optional[int] = None) -> list:
         """Continuous-batching AR decode.  Returns ``[{"token_ids","text"}, …]`` in prompt order.
 
         Requests are queued with the scheduler; each iteration prefills newly admitted
         requests, runs ONE ragged decode forward over all running sequences, and retires
-        finished ones so that waiting requests take their pages.
+        finished ones so that waiting requests take their pages.  With ``prefill_chunk`` prompts are fed in portions
+        of at most that many tokens, each portion in one batch with the other requests' decode tokens
+        (:meth:`step`), so a long prompt never holds the running requests up.
         """
         sp = sampling_params or SamplingParams()
         id_rows = [self._ids(p)[0] for p in prompts]
@@ -484,6 +528,9 @@ class JetSpecEngine:
             self.last_stats["evictions"] += len(out.evicted)
             for v in out.evicted:
                 sched.restore_sequence(v.seq_id)
+            if prefill_chunk:
+                self._chunked_step(sched, int(prefill_chunk), sp.temperature, results, reqs)
+                continue
             for req in out.admitted:
                 toks = torch.tensor(req.input_ids, device=self.device)
                 first, _ = self._prefill_batch_member(req.seq_id, toks, None, sp.temperature)
@@ -503,7 +550,7 @@ class JetSpecEngine:
             self.last_stats["steps"] += 1
             self.last_stats["max_batch"] = max(self.last_stats["max_batch"], len(ready))
             past = [self.pool.state(r.seq_id).length for r in ready]
-            if self.use_kernels and sp.temperature <= 0.0 and self.cfg.head_dim == 128 \
+            if self.use_kernels and sp.temperature <= 0.0 and self.cfg.kernel_path_ok() \
                     and (env_flag("JETSPEC_BATCH_GRAPH", True) or self.tp is not None):
                 # one graph replay per decode step: every sequence contributes a one-node "tree"
                 from .fast_round import FastRound
@@ -519,6 +566,33 @@ class JetSpecEngine:
                 self.pool.touch(r.seq_id)
                 self._record_token(sched, r, int(t), results, reqs)
         return results
+
+    def _chunked_step(self, sched, chunk: int, temperature: float, results, reqs) -> None:
+        """One mixed batch: the next portion of every prompt still being fed, beside one token of every other
+        running request; requests whose last prompt token ran (or that decoded) get their next token."""
+        if self.tp is not None:
+            raise NotImplementedError("tensor-parallel batches prefill whole prompts")
+        if not sched.running:
+            raise RuntimeError("scheduler stalled: a waiting request does not fit in an empty pool")
+        entries, takers = [], []
+        for r in list(sched.running.values()):
+            if r.seq_id not in sched.running:
+                continue                                   # evicted by an earlier request's _ensure_room
+            have = self.pool.state(r.seq_id).length if self.pool.has(r.seq_id) else 0
+            toks = r.input_ids[have:have + chunk] if r.is_prefill else r.input_ids[-1:]
+            self._ensure_room(sched, r, have + len(toks))
+            last = not r.is_prefill or have + len(toks) == r.prompt_len
+            entries.append((r.seq_id, toks, [len(toks) - 1] if last else []))
+            takers.append(r if last else None)
+        keep = [i for i, e in enumerate(entries) if e[0] in sched.running]
+        entries, takers = [entries[i] for i in keep], [takers[i] for i in keep]
+        logits = self.step(entries)
+        self.last_stats["steps"] += 1
+        self.last_stats["max_batch"] = max(self.last_stats["max_batch"], len(entries))
+        if logits is None:
+            return
+        for r, t in zip([r for r in takers if r is not None], sample(logits, temperature).tolist()):
+            self._record_token(sched, r, int(t), results, reqs)
 
     def _record_token(self, sched, req, tok, results, reqs):
         sched.mark_decode_step(req.seq_id, tok)
@@ -563,7 +637,7 @@ class JetSpecEngine:
         # when the graph path is certain to take every tree, trees are built as host lists only (no device tensors)
         if self.tp is not None:
             batch_graph = True         # the sharded stack exists on the kernel path only
-        graph_ok = bool(batch_graph and self.use_kernels and sp.temperature <= 0.0 and self.cfg.head_dim == 128
+        graph_ok = bool(batch_graph and self.use_kernels and sp.temperature <= 0.0 and self.cfg.kernel_path_ok()
                         and n_max <= 256)
         for i, row in enumerate(id_rows):
             r = SequenceRequest(seq_id=self._new_seq_id(), input_ids=row.tolist(), max_new_tokens=sp.max_new_tokens,

@@ -1,8 +1,12 @@
-"""Model configuration read from a Hugging Face ``config.json``.
+"""Model configurations read from ``config.json``: Qwen3 (Hugging Face layout) and Karuzen.
 
 Only the fields the decoder actually uses are kept.  The draft head adds
 ``block_size``, ``num_target_layers`` and ``dflash_config`` on top of the Qwen3
 fields (reference: ``jetspec/models/draft_head.py:317-337``).
+
+What the engines, the cache and the kernel path ask of a configuration, whatever the family: ``vocab_size``,
+``hidden_size``, ``num_hidden_layers`` (layer RUNS, i.e. cache layers), ``eos_token_id``, ``latent_widths()`` (``None``
+for a K/V cache) and ``kernel_path_ok()``.
 """
 from __future__ import annotations
 
@@ -66,6 +70,14 @@ class Qwen3Config:
             return False
         return (layer_idx + 1) % max(1, self.decoder_sparse_step) == 0
 
+    def latent_widths(self) -> Optional[list]:
+        """Widths of the latent rows a cache layer holds, or ``None`` when it holds K and V heads."""
+        return None
+
+    def kernel_path_ok(self) -> bool:
+        """Whether the graph-captured kernel path covers this geometry."""
+        return self.head_dim == 128
+
     # -- io -------------------------------------------------------------------
     @classmethod
     def from_dict(cls, d: dict) -> "Qwen3Config":
@@ -117,6 +129,133 @@ def _merge_eos(a, b) -> list:
     return out
 
 
+@dataclass
+class LatentAttentionConfig:
+    """Sizes of a latent attention: queries through a latent of ``q_rank``, keys and values from one of ``kv_rank``."""
+    heads: int
+    dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+
+
+@dataclass
+class RoutedExpertsConfig:
+    """Sizes of a sigmoid-routed expert layer; ``shared_ff`` is 0 without a shared expert."""
+    experts: int
+    top: int
+    scale: float
+    ff: int
+    shared_ff: int = 0
+
+
+@dataclass
+class KaruzenLayerConfig:
+    mixer: LatentAttentionConfig
+    dense_ff: int = 0                               # > 0: a dense feed-forward of this width
+    moe: Optional[RoutedExpertsConfig] = None       # a layer with neither has no feed-forward
+
+
+@dataclass
+class KaruzenConfig:
+    """Karuzen: parallel blocks (latent attention beside a dense or routed feed-forward) under one Dynamic Tanh norm
+    each, a range of layers run several times with shared weights, tied embeddings."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 1
+    norm_eps: float = 1e-5
+    eos_token_id: Any = None
+    model_type: str = "karuzen"
+
+    def layer_runs(self) -> list:
+        """``[(layer index, add the embedding output before it), ...]`` in execution order.  Every run has its own
+        cache layer; the layers of the loop appear once per pass."""
+        n, a, b = len(self.layers), self.loop_start, self.loop_stop
+        if b <= a:
+            return [(i, False) for i in range(n)]
+        runs = [(i, False) for i in range(a)]
+        for times in range(self.loop_times):
+            runs += [(i, times > 0 and i == a) for i in range(a, b)]
+        return runs + [(i, False) for i in range(b, n)]
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layer_runs())
+
+    @property
+    def is_moe(self) -> bool:
+        return any(l.moe is not None for l in self.layers)
+
+    def latent_widths(self) -> list:
+        return [self.layers[i].mixer.kv_rank for i, _ in self.layer_runs()]
+
+    def kernel_path_ok(self) -> bool:
+        return all(l.moe is None or (l.moe.experts <= 1024 and l.moe.top <= 32) for l in self.layers)
+
+    # -- io -------------------------------------------------------------------
+    @classmethod
+    def from_dict(cls, d: dict) -> "KaruzenConfig":
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            if e["type"] != "latent_attention":
+                raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
+            m, f = e["mixer"], e.get("mlp")
+            lc = KaruzenLayerConfig(LatentAttentionConfig(
+                heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), q_rank=int(m["q_rank"]),
+                kv_rank=int(m["kv_rank"]), scale=float(m["scale"])))
+            if f is not None and f["kind"] == "dense":
+                lc.dense_ff = int(f["ff"])
+            elif f is not None and f["kind"] == "moe":
+                r, sh = f["router"], f.get("shared")
+                lc.moe = RoutedExpertsConfig(experts=int(r["experts"]), top=int(r["top"]), scale=float(r["scale"]),
+                                             ff=int(f["expert"]["ff"]), shared_ff=int(sh["ff"]) if sh else 0)
+            elif f is not None:
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            layers.append(lc)
+        loop = d.get("loop") or {}
+        cfg = cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                  loop_start=int(loop.get("start", 0)), loop_stop=int(loop.get("stop", 0)),
+                  loop_times=int(loop.get("times", 1)), norm_eps=float(d["norm"]["eps"]),
+                  eos_token_id=d.get("eos_token_id"))
+        if not 0 <= cfg.loop_start <= max(cfg.loop_start, cfg.loop_stop) <= len(layers):
+            raise ValueError(f"loop {loop} does not fit {len(layers)} layers")
+        return cfg
+
+    @classmethod
+    def from_pretrained(cls, path: str, subfolder: str = "") -> "KaruzenConfig":
+        with open(os.path.join(path, subfolder, "config.json") if subfolder else os.path.join(path, "config.json")) as f:
+            return cls.from_dict(json.load(f))
+
+    def to_dict(self) -> dict:
+        layers = []
+        for l in self.layers:
+            mlp = None
+            if l.dense_ff:
+                mlp = {"kind": "dense", "ff": l.dense_ff}
+            elif l.moe is not None:
+                mlp = {"kind": "moe", "expert": {"ff": l.moe.ff},
+                       "router": {"experts": l.moe.experts, "top": l.moe.top, "scale": l.moe.scale}}
+                if l.moe.shared_ff:
+                    mlp["shared"] = {"ff": l.moe.shared_ff}
+            layers.append({"type": "latent_attention", "mixer": asdict(l.mixer), "mlp": mlp})
+        d = {"architecture": "Karuzen", "vocab": self.vocab_size, "width": self.hidden_size, "layers": layers,
+             "norm": {"eps": self.norm_eps}}
+        if self.loop_stop > self.loop_start:
+            d["loop"] = {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times}
+        if self.eos_token_id is not None:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    def save_pretrained(self, path: str) -> None:
+        os.makedirs(path, exist_ok=True)
+        with open(os.path.join(path, "config.json"), "w") as f:
+            json.dump(self.to_dict(), f, indent=1)
+
+
 # Geometry presets used by the tests and the benchmarks (random-init weights).
 def tiny_config(**over) -> Qwen3Config:
     """2 layers, hidden 256, 4 q / 2 kv heads, head_dim 64, SwiGLU 512, vocab 1024."""
@@ -141,6 +280,27 @@ def qwen3_30b_a3b_config(**over) -> Qwen3Config:
               norm_topk_prob=True, model_type="qwen3_moe")
     kw.update(over)
     return Qwen3Config(**kw)
+
+
+def karuzen_tiny_config(**over) -> KaruzenConfig:
+    """4 layers (dense, routed, routed, no feed-forward), the middle two run three times; width 192, 3 heads."""
+    mix = LatentAttentionConfig(heads=3, dim=40, vdim=24, q_rank=56, kv_rank=72, scale=0.2)
+    moe = RoutedExpertsConfig(experts=6, top=2, scale=1.3, ff=48, shared_ff=80)
+    kw = dict(vocab_size=320, hidden_size=192, norm_eps=1e-5, loop_start=1, loop_stop=3, loop_times=3,
+              layers=[KaruzenLayerConfig(mix, dense_ff=160), KaruzenLayerConfig(mix, moe=moe),
+                      KaruzenLayerConfig(mix, moe=moe), KaruzenLayerConfig(mix)])
+    kw.update(over)
+    return KaruzenConfig(**kw)
+
+
+def karuzen_bench_config(layers: int = 16, moe: bool = False, **over) -> KaruzenConfig:
+    """Width 4096, 32 heads of 128, latents of 1536 and 512, feed-forward 12288 (or 64 experts of 1536, 8 a token)."""
+    mix = LatentAttentionConfig(heads=32, dim=128, vdim=128, q_rank=1536, kv_rank=512, scale=128 ** -0.5)
+    ex = RoutedExpertsConfig(experts=64, top=8, scale=2.5, ff=1536, shared_ff=1536)
+    kw = dict(vocab_size=151936, hidden_size=4096, layers=[
+        KaruzenLayerConfig(mix, moe=ex) if moe else KaruzenLayerConfig(mix, dense_ff=12288) for _ in range(layers)])
+    kw.update(over)
+    return KaruzenConfig(**kw)
 
 
 def draft_head_config(target: Qwen3Config, num_layers: int = 1, block_size: int = 16,

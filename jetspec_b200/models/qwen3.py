@@ -15,8 +15,6 @@ what the grouped GEMM consumes (reference stacks them the same way at patch time
 """
 from __future__ import annotations
 
-import json
-import os
 from typing import Callable, Optional, Sequence
 
 import torch
@@ -24,6 +22,7 @@ import torch.nn as nn
 
 from .. import ops
 from .config import Qwen3Config
+from .registry import load_target, load_tokenizer, register_family  # noqa: F401  (re-exported)
 
 
 class RMSNorm(nn.Module):
@@ -290,23 +289,5 @@ def _moe_key_remap(cfg: Qwen3Config):
     return remap
 
 
-def load_target(model_name_or_path, device="cuda", dtype=torch.bfloat16, attn_implementation: str = "auto",
-                **_unused):
-    """Load a target LM and its tokenizer from a local Hugging Face directory.
-
-    Counterpart of the reference's ``load_target`` (``jetspec/models/qwen3.py:38-71``).
-    ``attn_implementation`` is accepted for signature compatibility; attention is
-    always this framework's own backend.  The tokenizer is ``None`` when the
-    directory has no tokenizer files (token-id prompts still work).
-    """
-    model = Qwen3ForCausalLM.from_pretrained(model_name_or_path, dtype=dtype, device=device)
-    return model, load_tokenizer(model_name_or_path)
-
-
-def load_tokenizer(path: str):
-    has_tok = any(os.path.exists(os.path.join(path, f))
-                  for f in ("tokenizer.json", "tokenizer_config.json", "vocab.json"))
-    if not has_tok:
-        return None
-    from transformers import AutoTokenizer
-    return AutoTokenizer.from_pretrained(path)
+register_family("qwen3", Qwen3Config, Qwen3ForCausalLM, aliases=(
+    "qwen3_moe", "Qwen3ForCausalLM", "Qwen3MoeForCausalLM"))

@@ -63,6 +63,49 @@ def silu_mul(gate_up):
     return ref.silu_mul(gate_up)
 
 
+def _kern_any(x: torch.Tensor) -> bool:
+    """Ops whose kernels exist in bf16 and in fp32."""
+    return x.is_cuda and x.dtype in (torch.bfloat16, torch.float32)
+
+
+def dynamic_tanh(x, alpha, weight, bias, out_dtype):
+    if x.is_cuda and x.dtype == torch.float32 and out_dtype in (torch.bfloat16, torch.float32):
+        return _ext().dynamic_tanh(x, alpha, weight, bias, out_dtype)
+    return ref.dynamic_tanh(x, alpha, weight, bias, out_dtype)
+
+
+def gelu_tanh_mul(gate, up):
+    if _kern_any(gate):
+        return _ext().gelu_tanh_mul(gate, up)
+    return ref.gelu_tanh_mul(gate, up)
+
+
+def relu_squared(x):
+    if _kern_any(x):
+        return _ext().relu_squared(x)
+    return ref.relu_squared(x)
+
+
+def latent_scatter(c, pool, slots):
+    if _kern_any(c):
+        return _ext().latent_scatter(c, pool, slots)
+    return ref.latent_scatter(c, pool, slots)
+
+
+def latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal: bool = False):
+    if _kern_any(q):
+        return _ext().latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits,
+                                       float(scale), bool(causal))
+    return ref.latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal)
+
+
+def sigmoid_moe(x, router_w, correction, w_up, w_down, top, scale):
+    if _kern_any(x):
+        wts, idx = _ext().sigmoid_route(ref.linear(x.float(), router_w.float()), correction, top, scale)
+        return ref.experts_relu_squared(x, wts, idx.long(), w_up, w_down)
+    return ref.sigmoid_moe(x, router_w, correction, w_up, w_down, top, scale)
+
+
 def qkv_postprocess(qkv, q_norm_w, k_norm_w, positions, num_q_heads, num_kv_heads, head_dim, theta, eps):
     if _kern(qkv) and head_dim == 128:
         ext = _ext()
@@ -116,5 +159,6 @@ def moe_forward(x, gate_w, w_gate_up, w_down, top_k, renorm, router_logits=None)
 __all__ = [
     "rmsnorm", "add_rmsnorm", "linear", "silu_mul", "qkv_postprocess", "kv_scatter",
     "paged_tree_attention", "lm_head_argmax", "lm_head_topk_logprobs", "moe_forward",
+    "dynamic_tanh", "gelu_tanh_mul", "relu_squared", "latent_scatter", "latent_attention", "sigmoid_moe",
     "pack_ancestor_bits", "unpack_ancestor_bits", "rope_cos_sin", "apply_rope", "moe_route", "sample",
 ]

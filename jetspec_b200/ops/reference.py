@@ -59,6 +59,21 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return (F.silu(g) * u).to(gate_up.dtype)
 
 
+def dynamic_tanh(x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out_dtype) -> torch.Tensor:
+    """``tanh(alpha x) * weight + bias`` in fp32, result in ``out_dtype``."""
+    return (torch.tanh(alpha.float() * x.float()) * weight.float() + bias.float()).to(out_dtype)
+
+
+def gelu_tanh_mul(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """``gelu_tanh(gate) * up``, fp32 inside."""
+    return (F.gelu(gate.float(), approximate="tanh") * up.float()).to(gate.dtype)
+
+
+def relu_squared(x: torch.Tensor) -> torch.Tensor:
+    r = torch.relu(x.float())
+    return (r * r).to(x.dtype)
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``x (M, K) @ w (N, K)^T``; the weight layout of ``nn.Linear``."""
     return F.linear(x, w, bias)
@@ -156,6 +171,42 @@ def paged_tree_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Te
     return out
 
 
+def latent_attention(q: torch.Tensor, w_uk: torch.Tensor, w_uv: torch.Tensor, pool: torch.Tensor,
+                     slot_map: torch.Tensor, seq_rows: torch.Tensor, cu_q: torch.Tensor, past_lens: torch.Tensor,
+                     mask_bits: Optional[torch.Tensor], scale: float, causal: bool = False) -> torch.Tensor:
+    """Attention over slot-addressed latent rows, keys and values expanded from them.
+
+    ``q (T, H, D)``; ``pool (S, >= R)`` holds one latent row per slot; ``w_uk (H*D, R)`` and ``w_uv (H*V, R)`` give
+    head ``h`` of a cached row ``c`` the key ``w_uk[h] c`` and the value ``w_uv[h] c``.  Sequences, visibility and
+    masks as in :func:`paged_tree_attention`; softmax in fp32.  Returns ``(T, H*V)`` in ``q.dtype``.
+    """
+    T, H, D = q.shape
+    R, V = w_uk.shape[1], w_uv.shape[0] // H
+    wk, wv = w_uk.float().view(H, D, R), w_uv.float().view(H, V, R)
+    out = torch.empty(T, H * V, dtype=q.dtype, device=q.device)
+    cu, pl, rows = cu_q.tolist(), past_lens.tolist(), seq_rows.tolist()
+    for b in range(len(cu) - 1):
+        s, e = cu[b], cu[b + 1]
+        n = e - s
+        if n == 0:
+            continue
+        L = pl[b] + n
+        c = pool[slot_map[rows[b], :L].long(), :R].float()
+        k, v = torch.einsum("lr,hdr->hld", c, wk), torch.einsum("lr,hvr->hlv", c, wv)
+        vis = torch.ones(n, L, dtype=torch.bool, device=q.device)
+        vis[:, pl[b]:] = (torch.tril(torch.ones(n, n, dtype=torch.bool, device=q.device)) if causal
+                          else unpack_ancestor_bits(mask_bits[s:e], n))
+        sc = torch.einsum("nhd,hld->hnl", q[s:e].float(), k) * scale
+        p = torch.nan_to_num(torch.softmax(sc.masked_fill(~vis[None], float("-inf")), dim=-1), nan=0.0)
+        out[s:e] = torch.einsum("hnl,hlv->nhv", p, v).reshape(n, H * V).to(q.dtype)
+    return out
+
+
+def latent_scatter(c: torch.Tensor, pool: torch.Tensor, slots: torch.Tensor) -> None:
+    """Write ``c (T, R)`` into the first ``R`` columns of ``pool (S, >= R)`` at ``slots (T,)``."""
+    pool[slots.long(), :c.shape[1]] = c.to(pool.dtype)
+
+
 def kv_scatter(k: torch.Tensor, v: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                slots: torch.Tensor) -> None:
     """Write ``k, v (T, Hkv, D)`` into ``(Hkv, S, D)`` pools at ``slots (T,)``."""
@@ -225,6 +276,32 @@ def moe_forward(x: torch.Tensor, gate_w: torch.Tensor, w_gate_up: torch.Tensor, 
         y = F.linear(h, w_down[e]).float()
         out.index_add_(0, tok, y * flat_w[sel, None])
     return out.to(x.dtype)
+
+
+def sigmoid_route(logits: torch.Tensor, correction: torch.Tensor, top: int, scale: float):
+    """fp32 scores ``s = sigmoid(logits)``; the ``top`` largest ``s + correction`` are chosen and weighted by
+    ``s / (sum of the chosen s + 1e-20) * scale``.  Returns ``(weights, experts)``, largest choice score first."""
+    s = torch.sigmoid(logits.float())
+    idx = torch.topk(s + correction.float(), top, dim=-1).indices
+    w = s.gather(-1, idx)
+    return w / (w.sum(-1, keepdim=True) + 1e-20) * scale, idx
+
+
+def sigmoid_moe(x: torch.Tensor, router_w: torch.Tensor, correction: torch.Tensor, w_up: torch.Tensor,
+                w_down: torch.Tensor, top: int, scale: float) -> torch.Tensor:
+    """Routed experts ``w_down[e] relu(w_up[e] x)^2`` with sigmoid routing; fp32 ``(T, H)``."""
+    wts, idx = sigmoid_route(F.linear(x.float(), router_w.float()), correction, top, scale)
+    return experts_relu_squared(x, wts, idx, w_up, w_down)
+
+
+def experts_relu_squared(x, wts, idx, w_up, w_down) -> torch.Tensor:
+    """``sum_j wts[:, j] * (w_down[idx_j] relu(w_up[idx_j] x)^2)``, summed in fp32."""
+    out = torch.zeros(x.shape[0], w_down.shape[1], dtype=torch.float32, device=x.device)
+    for e in idx.unique().tolist():
+        tok, j = (idx == e).nonzero(as_tuple=True)
+        y = F.linear(relu_squared(F.linear(x[tok], w_up[e])), w_down[e]).float()
+        out.index_add_(0, tok, y * wts[tok, j].unsqueeze(-1))
+    return out
 
 
 # --------------------------------------------------------------------------

@@ -5,6 +5,13 @@ One pool serves every layer and every sequence::
     k_pool, v_pool : (L, Hkv, S, D)       S = num_pages * page_size slots
     slot_map       : (max_seqs, max_len)  int32, on the device
 
+A model whose attention caches one latent row per token instead of K and V heads gets, per cache layer, a pool of
+rows of that layer's own width (rounded up to 64 elements, the rest stays zero)::
+
+    latent_pools : list of (S, width)
+
+Everything below the buffers (pages, slot maps, admission, eviction, commit) is the same for both kinds.
+
 A *page* (``page_size`` consecutive slots) is the unit of allocation and is shared
 by all layers (one page id addresses the same slots in each layer's slice), so a
 sequence of ``n`` tokens owns ``ceil(n / page_size)`` ids, not ``L`` times that.
@@ -40,6 +47,11 @@ class EvictionFailed(RuntimeError):
     """No sequence can be evicted (nothing else is resident)."""
 
 
+def latent_row_width(width: int) -> int:
+    """Elements a cached latent row takes: ``width`` rounded up to 64 (one 128-byte line of bf16)."""
+    return (int(width) + 63) // 64 * 64
+
+
 @dataclass
 class SeqState:
     seq_id: int
@@ -53,14 +65,18 @@ class SeqState:
 class PagedKVPool:
     def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, num_pages: int,
                  page_size: int = 16, max_seqs: int = 64, max_seq_len: int = 4096,
-                 device="cpu", dtype=torch.float32):
+                 device="cpu", dtype=torch.float32, latent_widths: Optional[list] = None):
         self.num_layers, self.num_kv_heads, self.head_dim = num_layers, num_kv_heads, head_dim
         self.page_size, self.num_pages = int(page_size), int(num_pages)
         self.max_seqs, self.max_seq_len = int(max_seqs), int(max_seq_len)
         self.device, self.dtype = torch.device(device), dtype
         S = self.num_pages * self.page_size
-        self.k_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
-        self.v_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
+        self.k_pool = self.v_pool = self.latent_pools = None
+        if latent_widths is not None:
+            self.latent_pools = [torch.zeros(S, latent_row_width(w), dtype=dtype, device=device) for w in latent_widths]
+        else:
+            self.k_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
+            self.v_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
         self.slot_map = torch.zeros(self.max_seqs, self.max_seq_len, dtype=torch.int32, device=device)
         self._free_pages: deque = deque(range(self.num_pages))
         self._refcount = [0] * self.num_pages
@@ -71,8 +87,12 @@ class PagedKVPool:
 
     # -- sizing ---------------------------------------------------------------
     @classmethod
-    def for_model(cls, cfg, num_pages: int, **kw) -> "PagedKVPool":
-        return cls(cfg.num_hidden_layers, cfg.num_key_value_heads, cfg.head_dim, num_pages, **kw)
+    def for_model(cls, cfg, num_pages: int, world: int = 1, **kw) -> "PagedKVPool":
+        """A pool of the shape ``cfg``'s attention caches (``world``: ranks the K/V heads are sharded over)."""
+        widths = cfg.latent_widths()
+        if widths is not None:
+            return cls(len(widths), 0, 0, num_pages, latent_widths=widths, **kw)
+        return cls(cfg.num_hidden_layers, cfg.num_key_value_heads // world, cfg.head_dim, num_pages, **kw)
 
     @property
     def num_slots(self) -> int:
@@ -90,6 +110,9 @@ class PagedKVPool:
 
     def layer(self, li: int):
         return self.k_pool[li], self.v_pool[li]
+
+    def latent(self, li: int) -> torch.Tensor:
+        return self.latent_pools[li]
 
     # -- sequences ------------------------------------------------------------
     def has(self, seq_id: int) -> bool:
