@@ -41,7 +41,9 @@ constexpr int UMMA_K = 16;
 constexpr int kGemmThreads = 192;
 constexpr int kTopK = 8;
 
-enum GemmEpi : int { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_ARGMAX = 2, EPI_TOPK = 3, EPI_STORE_F32 = 4, EPI_ALLREDUCE = 5, EPI_EP_COMBINE = 6 };
+enum GemmEpi : int { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_ARGMAX = 2, EPI_TOPK = 3, EPI_STORE_F32 = 4, EPI_ALLREDUCE = 5, EPI_EP_COMBINE = 6,
+                    EPI_INPROJ = 7, EPI_RELU2 = 8, EPI_RESID32 = 9 };
+enum GemmAct : int { ACT_GELU_GLU = 0, ACT_RELU2 = 1 };
 
 struct GemmParams {
   int M, N, K;
@@ -87,6 +89,27 @@ struct GemmParams {
   // 128-row box would make the activations half of every stage's bytes although almost none of its rows are used;
   // the accumulator rows beyond the box read stale shared memory and are never stored.
   int a_small_rows;
+  // EPI_INPROJ (fused input projections of a parallel block): columns below n_raw (a multiple of 128) are stored as
+  // fp32 to C; the rest pass through `act` and go to C2 as bf16.  ACT_GELU_GLU: every 128 weight rows hold 64 gate rows
+  // and the 64 up rows of the same outputs; ACT_RELU2: relu(.)^2 of each column.
+  __nv_bfloat16* C2;
+  int ldc2;
+  int n_raw;
+  int act;
+  // EPI_RESID32: C (fp32) = res32 + A W^T (+ emb); with norm_w, C2 = bf16(tanh(norm_alpha C) norm_w + norm_b), the
+  // next layer's Dynamic Tanh.  res32 may be C.
+  const float* res32;
+  const __nv_bfloat16* emb;
+  int ld_emb;
+  const float* norm_w;
+  const float* norm_b;
+  float norm_alpha;
+  // Batched mode: blockIdx.z is the batch element; its K columns of A start at z * a_batch_k, its weights are rows
+  // z*N .. (z+1)*N of W, its output starts at C + z * c_batch_stride.  A box that reaches past the element's own K
+  // columns meets zero-filled weights.  No K split in this mode.
+  int batch;
+  int a_batch_k;
+  long long c_batch_stride;
 };
 
 JS_DEVICE void red_release_sys_add(int* addr, int v) {
@@ -163,7 +186,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   // this CTA may still be streaming, so it normally sits behind the stages; only when both do
   // not fit (deep pipeline) it ALIASES them, guarded by one more cluster barrier after the main loop.
   const bool grouped = p.group_off != nullptr;
-  const int recv_total = recv_bytes(grouped ? 1 : gridDim.z, BN, EPI == EPI_SWIGLU);
+  const bool zbatch = grouped || p.batch > 0;     // blockIdx.z counts experts or batch elements, not K splits
+  const int recv_total = recv_bytes(zbatch ? 1 : gridDim.z, BN, EPI == EPI_SWIGLU || EPI == EPI_INPROJ);
   const bool alias = recv_aliases_stages(S::kTiles, recv_total);
   const int data_bytes = alias ? (S::kTiles > recv_total ? S::kTiles : recv_total) : S::kTiles + recv_total;
   uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + data_bytes);
@@ -174,9 +198,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
-  const int split = grouped ? 1 : gridDim.z;
-  const int z = grouped ? 0 : blockIdx.z;    // == rank in the (1,1,split) cluster
-  const int expert = grouped ? blockIdx.z : 0;
+  const int split = zbatch ? 1 : gridDim.z;
+  const int z = zbatch ? 0 : blockIdx.z;     // == rank in the (1,1,split) cluster
+  const int expert = zbatch ? blockIdx.z : 0;
+  const int ax0 = p.a_batch_k * expert;      // first A column of this batch element (0 in every other mode)
   int bx = blockIdx.x, by = blockIdx.y;        // column tile, row tile
   if (!grouped && p.m_fast) {
     const int lin = blockIdx.y * gridDim.x + blockIdx.x;
@@ -257,11 +282,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       pdl_wait();
       for (int i = 0; i < pre; ++i) {
         if (small0) {
-          tma_load_2d(smem + i * S::kStage, &tmA2, &full_bar[i], (kb_begin + i) * kXStep, m0);
+          tma_load_2d(smem + i * S::kStage, &tmA2, &full_bar[i], ax0 + (kb_begin + i) * kXStep, m0);
         } else {
 #pragma unroll
           for (int mt = 0; mt < MT; ++mt)
-            tma_load_2d(smem + i * S::kStage + mt * (BM * BK * 2), &tmA, &full_bar[i], (kb_begin + i) * kXStep, m0 + mt * BM);
+            tma_load_2d(smem + i * S::kStage + mt * (BM * BK * 2), &tmA, &full_bar[i], ax0 + (kb_begin + i) * kXStep, m0 + mt * BM);
         }
         load_sfa(i, kb_begin + i);
       }
@@ -279,11 +304,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           mbar_expect_tx(&full_bar[s], stage_bytes(small));
           tma_load_2d(smem + s * S::kStage + S::kStageA, &tmW, &full_bar[s], (kb_begin + i) * kXStep, wn0);
           if (small) {
-            tma_load_2d(smem + s * S::kStage, &tmA2, &full_bar[s], (kb_begin + i) * kXStep, m_tile);
+            tma_load_2d(smem + s * S::kStage, &tmA2, &full_bar[s], ax0 + (kb_begin + i) * kXStep, m_tile);
           } else {
 #pragma unroll
             for (int mt = 0; mt < MT; ++mt)
-              tma_load_2d(smem + s * S::kStage + mt * (BM * BK * 2), &tmA, &full_bar[s], (kb_begin + i) * kXStep, m_tile + mt * BM);
+              tma_load_2d(smem + s * S::kStage + mt * (BM * BK * 2), &tmA, &full_bar[s], ax0 + (kb_begin + i) * kXStep, m_tile + mt * BM);
           }
           load_sfw(s, kb_begin + i);
           load_sfa(s, kb_begin + i);
@@ -350,7 +375,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
   const int row = quad * 32 + lane;              // row of the tile owned by this thread
   uint32_t t_row = tmem_base + (static_cast<uint32_t>(quad * 32) << 16);
   // split-K: this CTA's receive area (after the pipeline stages) and the chunk -> owner mapping
-  constexpr bool kSwiglu = (EPI == EPI_SWIGLU);
+  constexpr bool kSwiglu = (EPI == EPI_SWIGLU || EPI == EPI_INPROJ);
   constexpr int kHC = (kSwiglu ? BN / 2 : BN) / 32;          // owned-chunk index space
   const int per_owner = (kHC + split - 1) / split;
   const int slots_per_src = kSwiglu ? 2 * per_owner : per_owner;
@@ -624,7 +649,101 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       epi_barrier();
       if (threadIdx.x == 64 && landed && !p.ar_push_only) p.peer_flags[p.rank][fidx] = 0;   // ready for this buffer's next turn
       }
-    } else if constexpr (EPI == EPI_STORE || EPI == EPI_STORE_F32) {
+    } else if constexpr (EPI == EPI_INPROJ) {
+      // every 128-column block is handled as two 64-column halves (gate | up, or simply neighbours)
+      auto store_bf16 = [&](__nv_bfloat16* out, const float* v) {
+#pragma unroll
+        for (int j = 0; j < 32; j += 8) {
+          uint4 ov;
+          __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
+#pragma unroll
+          for (int t = 0; t < 4; ++t) o2[t] = __floats2bfloat162_rn(v[j + 2 * t], v[j + 2 * t + 1]);
+          *reinterpret_cast<uint4*>(out + j) = ov;
+        }
+      };
+      for (int c0 = z * 32; c0 < BN / 2; c0 += split * 32) {
+        const int blk = c0 >> 6, cb = c0 & 63;
+        const int nb = n0 + blk * 128;
+        float g[32], u[32];
+        load_chunk(blk * 128 + cb, g);
+        load_chunk(blk * 128 + 64 + cb, u);
+        if (grow >= m_end || nb >= p.N) continue;
+        if (nb < p.n_raw) {
+          float* out = reinterpret_cast<float*>(p.C) + static_cast<size_t>(grow) * p.ldc + nb + cb;
+#pragma unroll
+          for (int j = 0; j < 32; j += 4) {
+            *reinterpret_cast<float4*>(out + j) = make_float4(g[j], g[j + 1], g[j + 2], g[j + 3]);
+            *reinterpret_cast<float4*>(out + 64 + j) = make_float4(u[j], u[j + 1], u[j + 2], u[j + 3]);
+          }
+          continue;
+        }
+        __nv_bfloat16* out2 = p.C2 + static_cast<size_t>(grow) * p.ldc2;
+        if (p.act == ACT_GELU_GLU) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float a = g[j];
+            g[j] = 0.5f * a * (1.f + tanhf(0.7978845608028654f * (a + 0.044715f * a * a * a))) * u[j];   // sqrt(2 / pi)
+          }
+          store_bf16(out2 + (nb - p.n_raw) / 2 + cb, g);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            g[j] = fmaxf(g[j], 0.f);
+            g[j] *= g[j];
+            u[j] = fmaxf(u[j], 0.f);
+            u[j] *= u[j];
+          }
+          store_bf16(out2 + nb - p.n_raw + cb, g);
+          store_bf16(out2 + nb - p.n_raw + 64 + cb, u);
+        }
+      }
+    } else if constexpr (EPI == EPI_RESID32) {
+      for (int c0 = z * 32; c0 < BN; c0 += split * 32) {
+        float v[32];
+        load_chunk(c0, v);
+        const int gc = n0 + c0;
+        if (grow >= m_end || gc >= p.N) continue;
+        float* out = reinterpret_cast<float*>(p.C) + static_cast<size_t>(grow) * p.ldc + gc;
+        const float* res = p.res32 + static_cast<size_t>(grow) * p.ldc + gc;
+        const __nv_bfloat16* emb = p.emb ? p.emb + static_cast<size_t>(grow) * p.ld_emb + gc : nullptr;
+#pragma unroll
+        for (int j = 0; j < 32; j += 8) {
+          if (gc + j >= p.N) break;
+#pragma unroll
+          for (int t = 0; t < 8; t += 4) {
+            const float4 rv = *reinterpret_cast<const float4*>(res + j + t);
+            v[j + t] += rv.x;
+            v[j + t + 1] += rv.y;
+            v[j + t + 2] += rv.z;
+            v[j + t + 3] += rv.w;
+          }
+          if (emb != nullptr) {
+            const uint4 ev = *reinterpret_cast<const uint4*>(emb + j);
+            const __nv_bfloat162* e2 = reinterpret_cast<const __nv_bfloat162*>(&ev);
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+              const float2 f = __bfloat1622float2(e2[t]);
+              v[j + 2 * t] += f.x;
+              v[j + 2 * t + 1] += f.y;
+            }
+          }
+          *reinterpret_cast<float4*>(out + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+          *reinterpret_cast<float4*>(out + j + 4) = make_float4(v[j + 4], v[j + 5], v[j + 6], v[j + 7]);
+          if (p.norm_w != nullptr) {
+            uint4 ov;
+            __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&ov);
+#pragma unroll
+            for (int t = 0; t < 4; ++t) {
+              const float2 w2 = __ldg(reinterpret_cast<const float2*>(p.norm_w + gc + j + 2 * t));
+              const float2 b2 = __ldg(reinterpret_cast<const float2*>(p.norm_b + gc + j + 2 * t));
+              o2[t] = __floats2bfloat162_rn(tanhf(p.norm_alpha * v[j + 2 * t]) * w2.x + b2.x,
+                                            tanhf(p.norm_alpha * v[j + 2 * t + 1]) * w2.y + b2.y);
+            }
+            *reinterpret_cast<uint4*>(p.C2 + static_cast<size_t>(grow) * p.ldc2 + gc + j) = ov;
+          }
+        }
+      }
+    } else if constexpr (EPI == EPI_STORE || EPI == EPI_STORE_F32 || EPI == EPI_RELU2) {
       // 32-column chunks are dealt round-robin to the CTAs of the K-split cluster
       for (int c0 = z * 32; c0 < BN; c0 += split * 32) {
         float v[32];
@@ -637,8 +756,16 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             for (int j = 0; j < 32; j += 4)
               if (gc + j < p.N) *reinterpret_cast<float4*>(out + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
           } else {
-            __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.C) + static_cast<size_t>(grow) * p.ldc + gc;
+            __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.C) + static_cast<size_t>(grow) * p.ldc + gc +
+                                 p.c_batch_stride * expert;
             const __nv_bfloat16* res = p.residual ? p.residual + static_cast<size_t>(grow) * p.ldc + gc : nullptr;
+            if constexpr (EPI == EPI_RELU2) {
+#pragma unroll
+              for (int j = 0; j < 32; ++j) {
+                v[j] = fmaxf(v[j], 0.f);
+                v[j] *= v[j];
+              }
+            }
 #pragma unroll
             for (int j = 0; j < 32; j += 8) {
               if (gc + j >= p.N) break;
@@ -939,7 +1066,7 @@ static int launch_gemm(const CUtensorMap& ta, const CUtensorMap& tw, const GemmP
   static int configured[kMaxDevicesCached] = {};
   auto kern = gemm_bf16_kernel<BN, EPI, BUDGET_KB, FP4, MT>;
   if (MT != 1 && (split != 1 || groups > 0)) return -19;
-  const int recv_total = recv_bytes(split, BN, EPI == EPI_SWIGLU);
+  const int recv_total = recv_bytes(split, BN, EPI == EPI_SWIGLU || EPI == EPI_INPROJ);
   const int data_bytes = recv_aliases_stages(S::kTiles, recv_total) ? (S::kTiles > recv_total ? S::kTiles : recv_total)
                                                                      : S::kTiles + recv_total;
   const int smem_bytes = data_bytes + 1024 /*align slack*/ + 256 /*barriers*/ + ((EPI == EPI_ALLREDUCE || EPI == EPI_EP_COMBINE) ? 8192 + 64 : 0);
@@ -1051,7 +1178,7 @@ extern "C" int js_gemm_bf16_allreduce(const void* A, const void* W, void* C, con
 // Grouped GEMM over `groups` experts in one launch.  A (total_rows, K) holds the rows sorted by expert,
 // expert e owning rows group_off[e] .. group_off[e+1] (device array, groups+1 entries); W is the stacked
 // (groups*N, K) weight; C (total_rows, N or N/2).  epi: 0 store, 1 swiglu (per-expert tile-interleaved
-// gate/up), 6 expert-parallel combine (weighted rows pushed to every rank's pair buffer).
+// gate/up), 8 relu(.)^2, 6 expert-parallel combine (weighted rows pushed to every rank's pair buffer).
 // max_rows_per_group bounds the row tiles launched per expert.
 extern "C" int js_gemm_bf16_grouped(const void* A, const void* W, void* C, int total_rows, int N, int K, int lda,
                                     int ldw, int ldc, int epi, int groups, const int* group_off,
@@ -1074,6 +1201,7 @@ extern "C" int js_gemm_bf16_grouped(const void* A, const void* W, void* C, int t
   if (m_tiles < 1) return 0;
   if (epi == EPI_STORE) return launch_gemm<128, EPI_STORE, 96>(ta, tw, p, 1, pdl != 0, stream, groups, m_tiles, &ta_small);
   if (epi == EPI_SWIGLU) return launch_gemm<128, EPI_SWIGLU, 96>(ta, tw, p, 1, pdl != 0, stream, groups, m_tiles, &ta_small);
+  if (epi == EPI_RELU2) return launch_gemm<128, EPI_RELU2, 96>(ta, tw, p, 1, pdl != 0, stream, groups, m_tiles, &ta_small);
   if (epi == EPI_EP_COMBINE) {
     if (!row_pair || !row_weight || !peer_pairs || !peer_cnt) return -22;
     return launch_gemm<128, EPI_EP_COMBINE, 96>(ta, tw, p, 1, pdl != 0, stream, groups, m_tiles, &ta_small);
@@ -1172,4 +1300,77 @@ extern "C" int js_gemm_nvfp4_allreduce(const void* Aq, const void* sfa, const fl
   p.row_scale = row_scale; p.w_scale = w_scale;
   p.ar_push_only = push_only;
   return launch_gemm<128, EPI_ALLREDUCE, 128, true>(ta, tw, p, split, pdl != 0, stream);
+}
+
+// Fused input projections of a parallel block: columns [0, n_raw) of A W^T as fp32 to C (T, ldc), the rest through `act`
+// (0: tanh-GELU gate * up, 64-row interleave; 1: relu^2) as bf16 to C2.  n_raw and N multiples of 128; bn 128 or 256.
+extern "C" int js_gemm_inproj(const void* A, const void* W, float* C, void* C2, int M, int N, int K, int lda, int ldw, int ldc,
+                              int ldc2, int n_raw, int act, int bn, int split, int deep, int* status, int pdl,
+                              cudaStream_t stream) {
+  using namespace js;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((K % 8) || (lda % 8) || (ldw % 8)) return -10;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) return -11;
+  if (split < 1 || split > 4 || split > (K + BK - 1) / BK || (bn != 128 && split != 1)) return -12;
+  if ((N % 128) || (n_raw % 128) || n_raw < 0 || n_raw > N || (ldc % 4) || (ldc2 % 8) || act < 0 || act > 1) return -15;
+  if ((n_raw > 0 && (C == nullptr || ldc < n_raw)) || (n_raw < N && C2 == nullptr)) return -22;
+  CUtensorMap ta, tw;
+  if (make_map(&ta, A, M, K, lda, BM) || make_map(&tw, W, N, K, ldw, bn)) return -16;
+  GemmParams p{};
+  p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.C = C; p.status = status; p.world = 1;
+  p.C2 = reinterpret_cast<__nv_bfloat16*>(C2); p.ldc2 = ldc2; p.n_raw = n_raw; p.act = act;
+  if (bn == 128)
+    return deep == 1   ? launch_gemm<128, EPI_INPROJ, 192>(ta, tw, p, split, pdl != 0, stream)
+           : deep == 2 ? launch_gemm<128, EPI_INPROJ, 128>(ta, tw, p, split, pdl != 0, stream)
+                       : launch_gemm<128, EPI_INPROJ, 96>(ta, tw, p, split, pdl != 0, stream);
+  if (bn == 256)
+    return deep ? launch_gemm<256, EPI_INPROJ, 192>(ta, tw, p, 1, pdl != 0, stream)
+                : launch_gemm<256, EPI_INPROJ, 96>(ta, tw, p, 1, pdl != 0, stream);
+  return -17;
+}
+
+// x_out (fp32) = x_in + A W^T (+ emb); with norm_w also h = bf16(tanh(alpha x_out) norm_w + norm_b).  N and the leading
+// dimensions multiples of 8.  bn 128 (split 1..4) or 256 (deep 1, or 3 = two row tiles per CTA).
+extern "C" int js_gemm_resid32(const void* A, const void* W, float* x_out, const float* x_in, int M, int N, int K, int lda, int ldw,
+                               int ldx, const void* emb, int ld_emb, void* h, int ldh, const float* norm_w, const float* norm_b,
+                               float norm_alpha, int bn, int split, int deep, int* status, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((K % 8) || (lda % 8) || (ldw % 8) || (N % 8) || (ldx % 4) || (ld_emb % 8) || (ldh % 8)) return -10;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) return -11;
+  if (split < 1 || split > 4 || split > (K + BK - 1) / BK || (bn != 128 && split != 1)) return -12;
+  if (norm_w != nullptr && (norm_b == nullptr || h == nullptr)) return -22;
+  CUtensorMap ta, tw;
+  if (make_map(&ta, A, M, K, lda, BM) || make_map(&tw, W, N, K, ldw, bn)) return -16;
+  GemmParams p{};
+  p.M = M; p.N = N; p.K = K; p.ldc = ldx; p.C = x_out; p.status = status; p.world = 1;
+  p.res32 = x_in; p.emb = reinterpret_cast<const __nv_bfloat16*>(emb); p.ld_emb = ld_emb;
+  p.C2 = reinterpret_cast<__nv_bfloat16*>(h); p.ldc2 = ldh; p.norm_w = norm_w; p.norm_b = norm_b; p.norm_alpha = norm_alpha;
+  if (bn == 128)
+    return deep == 1   ? launch_gemm<128, EPI_RESID32, 192>(ta, tw, p, split, pdl != 0, stream)
+           : deep == 2 ? launch_gemm<128, EPI_RESID32, 128>(ta, tw, p, split, pdl != 0, stream)
+                       : launch_gemm<128, EPI_RESID32, 96>(ta, tw, p, split, pdl != 0, stream);
+  if (bn == 256)
+    return deep == 3 ? launch_gemm<256, EPI_RESID32, 192, false, 2>(ta, tw, p, 1, pdl != 0, stream)
+                     : launch_gemm<256, EPI_RESID32, 192>(ta, tw, p, 1, pdl != 0, stream);
+  return -17;
+}
+
+// `batch` products C_z = A_z W_z^T in one launch: A_z = columns [z * a_batch_k, + K) of A (M, lda) (a_batch_k 0: the same A
+// for all), W_z = rows [z * N, + N) of W, C_z = C + z * c_batch_stride (M, ldc) bf16.  a_batch_k, N and ldc multiples of 8.
+extern "C" int js_gemm_bf16_batched(const void* A, const void* W, void* C, int M, int N, int K, int batch, int a_batch_k,
+                                    long long c_batch_stride, int lda, int ldw, int ldc, int* status, int pdl,
+                                    cudaStream_t stream) {
+  using namespace js;
+  if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return 0;
+  if ((K % 8) || (lda % 8) || (ldw % 8) || (N % 8) || (ldc % 8) || (a_batch_k % 8) || (c_batch_stride % 8)) return -10;
+  if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W) | reinterpret_cast<uintptr_t>(C)) & 15) return -11;
+  if (batch > 65535) return -12;
+  CUtensorMap ta, tw;
+  const uint64_t a_cols = a_batch_k > 0 ? static_cast<uint64_t>(batch - 1) * a_batch_k + K : K;
+  if (make_map(&ta, A, M, a_cols, lda, BM) || make_map(&tw, W, static_cast<uint64_t>(batch) * N, K, ldw, 128)) return -16;
+  GemmParams p{};
+  p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.C = C; p.status = status; p.world = 1;
+  p.batch = batch; p.a_batch_k = a_batch_k; p.c_batch_stride = c_batch_stride;
+  return launch_gemm<128, EPI_STORE, 96>(ta, tw, p, 1, pdl != 0, stream, batch, (M + BM - 1) / BM);
 }

@@ -72,7 +72,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int T, int E,
 __global__ void __launch_bounds__(kSortThreads)
 moe_sort_kernel(const int* __restrict__ idx, const float* __restrict__ wts, int P, int E, int first, int n_local,
                 int* __restrict__ order, float* __restrict__ row_weight, int* __restrict__ group_off,
-                int* __restrict__ counts_all, int k, int* __restrict__ token_of_row) {
+                int* __restrict__ counts_all, int k, int* __restrict__ token_of_row, int* __restrict__ inv) {
   extern __shared__ int sh[];
   int* key = sh;                       // P
   int* cnt = key + P;                  // n_local + 1
@@ -125,6 +125,7 @@ moe_sort_kernel(const int* __restrict__ idx, const float* __restrict__ wts, int 
         order[pos] = p;
         row_weight[pos] = wts[p];
         if (token_of_row != nullptr) token_of_row[pos] = p / k;
+        if (inv != nullptr) inv[p] = pos;
       }
       base += __popc(m);
     }
@@ -207,10 +208,11 @@ extern "C" int js_moe_route(const float* logits, int T, int E, int k, int renorm
 }
 
 // idx / wts (P = T*k) -> order (P), row_weight (P), group_off (n_local + 1), counts_all (E) and, when
-// token_of_row is given, the source token order[r] / k of every sorted row (the gather index of the dispatch).
-extern "C" int js_moe_sort(const int* idx, const float* wts, int P, int E, int first, int n_local, int* order,
-                           float* row_weight, int* group_off, int* counts_all, int k, int* token_of_row, int pdl,
-                           cudaStream_t stream) {
+// token_of_row is given, the source token order[r] / k of every sorted row (the gather index of the dispatch); inv
+// (optional, P) is the inverse permutation, inv[pair] = row.
+extern "C" int js_moe_sort_inv(const int* idx, const float* wts, int P, int E, int first, int n_local, int* order,
+                               float* row_weight, int* group_off, int* counts_all, int k, int* token_of_row, int* inv, int pdl,
+                               cudaStream_t stream) {
   if (P <= 0) return 0;
   if (k < 1) return -10;
   if (P > js::kSortMaxPairs || n_local < 1 || E < 1) return -10;
@@ -228,7 +230,14 @@ extern "C" int js_moe_sort(const int* idx, const float* wts, int P, int E, int f
   c.attrs = &a;
   c.numAttrs = pdl ? 1 : 0;
   return cudaLaunchKernelEx(&c, js::moe_sort_kernel, idx, wts, P, E, first, n_local, order, row_weight, group_off,
-                            counts_all, k, token_of_row) == cudaSuccess ? 0 : -4;
+                            counts_all, k, token_of_row, inv) == cudaSuccess ? 0 : -4;
+}
+
+extern "C" int js_moe_sort(const int* idx, const float* wts, int P, int E, int first, int n_local, int* order,
+                           float* row_weight, int* group_off, int* counts_all, int k, int* token_of_row, int pdl,
+                           cudaStream_t stream) {
+  return js_moe_sort_inv(idx, wts, P, E, first, n_local, order, row_weight, group_off, counts_all, k, token_of_row, nullptr, pdl,
+                         stream);
 }
 
 // ys (T*k, H) bf16 in expert-sorted row order -> out (T, H) bf16: each token's k expert outputs weighted and

@@ -327,19 +327,29 @@ class FastRound:
         X.load()
         m = engine.model
         self.embed_w, self.lm_head_w, self.final_norm = m.model.embed_tokens.weight, m.lm_head.weight, m.model.norm.weight
+        self.latent = None                 # launch sequence of a latent-attention decoder (replaces decoder_layers)
         self.tp = getattr(engine, "tp", None)
         self.ep = getattr(engine, "ep", None)
         if self.tp is not None and self.ep is not None:
             raise NotImplementedError("tensor parallelism and expert parallelism are separate plans here")
         world = self.tp.world if self.tp is not None else 1
-        self.lcfg = local_dims(self.cfg, world)
-        self.layers = kernel_layer_weights(m.model.layers, self.cfg, self.tp, self.ep)
+        if self.cfg.latent_widths() is not None:
+            if self.tp is not None or self.ep is not None:
+                raise NotImplementedError("latent-attention models run on one GPU")
+            from .latent_stack import LatentStack
+            self.latent = LatentStack(m, self.device)
+            self.lm_head_w = self.latent.table
+            self.lcfg, self.layers, self.freq = None, None, None
+        else:
+            self.lcfg = local_dims(self.cfg, world)
+            self.layers = kernel_layer_weights(m.model.layers, self.cfg, self.tp, self.ep)
+            self.freq = X.inv_freq(self.cfg.head_dim, self.cfg.rope_theta, self.device)
+        self.xn_cols = self.lm_head_w.shape[1]
         if self.tp is not None:
             from ..parallel.tp import shard_rows
             self.vocab_local = self.cfg.vocab_size // world
             self.lm_head_w = shard_rows(m.lm_head.weight, self.tp.rank, world)
-        self.freq = X.inv_freq(self.cfg.head_dim, self.cfg.rope_theta, self.device)
-        self.prefetcher = WeightPrefetcher(self.device) if _L2_PREFETCH else None
+        self.prefetcher = WeightPrefetcher(self.device) if _L2_PREFETCH and self.latent is None else None
         self.graphs: dict = {}
         self.draft_cache: dict = {}
         self.launches_per_round = 0
@@ -350,10 +360,57 @@ class FastRound:
         self.last_rounds = 0
         self._tp_graph_key = None
 
+    # ------------------------------------------------------------------ decoder stack (either model family)
+    def _new_stack(self, T: int, max_keys: int):
+        if self.latent is not None:
+            return self.latent.buffers(T, max_keys)
+        return _Stack(self.lcfg, T, self.device, max_keys)
+
+    def _run_stack(self, st, ids, seq_rows, cu_q, past, positions, slots, mask, causal: bool, max_q: int, xn, taps=None,
+                   tap_ids=None, pdl: bool = True, embed_pdl: bool = True, prefetch=None) -> int:
+        """Embedding, every layer run, final norm into ``xn``, and the tapped rows.  Returns the launch count."""
+        pool, cfg = self.eng.pool, self.cfg
+        if self.latent is not None:
+            batch = self.latent.uniform_batch(pool.slot_map, seq_rows, cu_q, past, slots, mask, causal, st.T, max_q, st.max_keys)
+            return self.latent.run(st, ids, pool.latent_pools, batch, xn, taps=taps, tap_ids=tap_ids, pdl=pdl)
+        X.embed(ids, self.embed_w, out=st.x, pdl=embed_pdl)
+        n = 1 + decoder_layers(self.lcfg, self.layers, st, pool.k_pool, pool.v_pool, pool.slot_map, seq_rows, cu_q, past,
+                               positions, slots, mask, causal, self.freq, taps=taps, tap_ids=tap_ids, pdl=pdl, tp=self.tp,
+                               prefetch=prefetch, then_prefetch=self.lm_head_w if prefetch is not None else None,
+                               final_norm=(self.final_norm, xn), ep=self.ep)
+        if taps is not None:
+            for j, t in enumerate(tap_ids):
+                if t == cfg.num_hidden_layers - 1:
+                    X.gather_rows(xn, None, taps, dst_col0=j * cfg.hidden_size, pdl=pdl)
+                    n += 1
+        return n
+
+    def ragged_forward(self, ids, meta, past_lens, taps=None, logits_rows=None):
+        """One ragged batch (portions of prompts, decoded tokens or trees) through the fused stack, launched eagerly.
+        Returns ``(fp32 logits of the wanted rows, tapped hidden rows or None)``."""
+        lat, pool, dev = self.latent, self.eng.pool, self.device
+        T = int(ids.numel())
+        taps = list(taps) if taps else None
+        counts = list(meta.counts)
+        st = lat.buffers(T, max(int(p) + n for p, n in zip(past_lens, counts)))
+        hidden = torch.empty(T, len(taps) * self.cfg.hidden_size, dtype=torch.bfloat16, device=dev) if taps else None
+        xn = torch.zeros(T, self.xn_cols, dtype=torch.bfloat16, device=dev)
+        batch = lat.ragged_batch(pool.slot_map, meta, counts, [int(p) for p in past_lens])
+        lat.run(st, ids.to(torch.int32), pool.latent_pools, batch, xn, taps=hidden, tap_ids=taps, pdl=_PDL)
+        rows = xn if logits_rows is None else xn[logits_rows].contiguous()
+        return self._logits(rows), hidden
+
+    def _logits(self, rows: torch.Tensor) -> torch.Tensor:
+        V = self.lm_head_w.shape[0]
+        out = torch.empty(rows.shape[0], (V + 3) // 4 * 4, dtype=torch.float32, device=self.device)
+        if rows.shape[0]:
+            X.gemm(rows, self.lm_head_w, out=out, epi=X.EPI_STORE_F32)
+        return out[:, :V]
+
     # ------------------------------------------------------------------ support matrix
     def supports_tree(self, drafter, algo_obj, block_size, tree_width, budget, extend_kwargs=None) -> bool:
         cfg = self.cfg
-        if cfg.head_dim != 128 or budget > 256 or tree_width > 8 or block_size - 1 > 48:
+        if not cfg.kernel_path_ok() or budget > 256 or tree_width > 8 or block_size - 1 > 48:
             return False
         if extend_kwargs:
             # the gated extension stays on the graph path for a draft head that runs inside the round, in chain mode
@@ -426,8 +483,8 @@ class FastRound:
         eos = sorted(self.eng.eos_token_ids)
         r["eos"] = torch.tensor(eos or [-1], dtype=torch.int32, device=dev)
         r["n_eos"] = len(eos)
-        r["stack"] = _Stack(self.lcfg, NB, dev, pool.max_seq_len)
-        r["xn"] = torch.zeros(NB, H, dtype=torch.bfloat16, device=dev)
+        r["stack"] = self._new_stack(NB, pool.max_seq_len)
+        r["xn"] = torch.zeros(NB, self.xn_cols, dtype=torch.bfloat16, device=dev)
         nt = X.n_tiles(self.lm_head_w.shape[0])
         r["am_ws"] = {"val": torch.zeros(NB, nt, dtype=torch.float32, device=dev),
                       "idx": torch.zeros(NB, nt, dtype=torch.int32, device=dev)}
@@ -446,7 +503,7 @@ class FastRound:
             # draws a token per node (inverse CDF, uniforms from the graph-registered generator), and acceptance
             # walks the tree against the SAMPLED tokens (reference: the graphed verify with the accept swapped,
             # jetspec/inference_engine/engine.py:1084-1109)
-            r["logits"] = torch.zeros(NB, self.lm_head_w.shape[0], dtype=torch.float32, device=dev)
+            r["logits"] = torch.zeros(NB, (self.lm_head_w.shape[0] + 3) // 4 * 4, dtype=torch.float32, device=dev)
             r["uniform"] = torch.zeros(NB, dtype=torch.float32, device=dev)
             r["sampled"] = torch.zeros(NB, dtype=torch.int64, device=dev)
         r["taps"] = torch.zeros(NB, len(tap_ids) * H, dtype=torch.bfloat16, device=dev) if tap_ids else None
@@ -675,23 +732,14 @@ class FastRound:
         pf = self.prefetcher
         if pf is not None:
             pf.ahead(self.layers[0]["qkv"])       # the first projection's weights arrive during the tree build
-        X.embed(r["tokens"], self.embed_w, out=st.x, pdl=pdl)
-        n += 1 + decoder_layers(self.lcfg, self.layers, st, pool.k_pool, pool.v_pool, pool.slot_map, r["seq_rows"],
-                                r["cu_q"], r["state"][ST_PAST:ST_PAST + 1], r["positions"], r["slots"], r["mask"],
-                                False, self.freq, taps=r["taps"], tap_ids=r["tap_ids"], pdl=pdl, tp=self.tp,
-                                prefetch=pf, then_prefetch=self.lm_head_w, final_norm=(self.final_norm, r["xn"]),
-                                ep=self.ep)
-        last = cfg.num_hidden_layers - 1
-        if r["taps"] is not None:
-            for j, t in enumerate(r["tap_ids"]):
-                if t == last:
-                    X.gather_rows(r["xn"], None, r["taps"], dst_col0=j * cfg.hidden_size, pdl=pdl)
-                    n += 1
+        n += self._run_stack(st, r["tokens"], r["seq_rows"], r["cu_q"], r["state"][ST_PAST:ST_PAST + 1], r["positions"],
+                             r["slots"], r["mask"], False, NB, r["xn"], taps=r["taps"], tap_ids=r["tap_ids"], pdl=pdl,
+                             embed_pdl=pdl, prefetch=pf)
         if r.get("temperature", 0.0) > 0.0:
             X.gemm(r["xn"], self.lm_head_w, out=r["logits"], epi=X.EPI_STORE_F32, bn=128, split=1, pdl=pdl)
             r["uniform"].uniform_()
             lib.js_sample_temperature.restype = ctypes.c_int
-            X._check(lib.js_sample_temperature(p(r["logits"]), 0, NB, r["logits"].shape[1], r["logits"].stride(0),
+            X._check(lib.js_sample_temperature(p(r["logits"]), 0, NB, self.lm_head_w.shape[0], r["logits"].stride(0),
                                                ctypes.c_float(r["temperature"]), p(r["uniform"]), p(r["sampled"]), s()),
                      "js_sample_temperature")
             r["greedy"].copy_(r["sampled"])
@@ -715,7 +763,7 @@ class FastRound:
     # ------------------------------------------------------------------ batched verify (continuous batching)
     def supports_batch_verify(self, trees, tap_ids) -> bool:
         cfg = self.cfg
-        if cfg.head_dim != 128 or not trees:
+        if not cfg.kernel_path_ok() or not trees:
             return False
         return all(t.host is not None and t.num_nodes <= 256 for t in trees)
 
@@ -758,8 +806,8 @@ class FastRound:
             r["ar"] = torch.arange(NB, dtype=torch.long, device=dev)
             r["greedy"] = _i32(T, dev)
             r["greedy_host"] = torch.zeros(T, dtype=torch.int32).pin_memory()
-            r["stack"] = _Stack(self.lcfg, T, dev, pool.max_seq_len)
-            r["xn"] = torch.zeros(T, H, dtype=torch.bfloat16, device=dev)
+            r["stack"] = self._new_stack(T, pool.max_seq_len)
+            r["xn"] = torch.zeros(T, self.xn_cols, dtype=torch.bfloat16, device=dev)
             nt = X.n_tiles(self.lm_head_w.shape[0])
             r["am_ws"] = {"val": torch.zeros(T, nt, dtype=torch.float32, device=dev),
                           "idx": torch.zeros(T, nt, dtype=torch.int32, device=dev)}
@@ -823,15 +871,8 @@ class FastRound:
         # KV slots of every sequence's tree window: slot_map[row_b, past_b + i]
         win = r["past"].long()[:, None] + r["ar"][None, :]
         r["slots"].copy_(pool.slot_map[r["seq_rows"].long()].gather(1, win).reshape(-1))
-        X.embed(r["tokens"], self.embed_w, out=st.x, pdl=False)
-        decoder_layers(self.lcfg, self.layers, st, pool.k_pool, pool.v_pool, pool.slot_map, r["seq_rows"], r["cu_q"],
-                       r["past"], r["positions"], r["slots"], r["mask"], False, self.freq, taps=r["taps"],
-                       tap_ids=r["tap_ids"], pdl=pdl, tp=self.tp, final_norm=(self.final_norm, r["xn"]))
-        last = cfg.num_hidden_layers - 1
-        if r["taps"] is not None:
-            for j, t in enumerate(r["tap_ids"]):
-                if t == last:
-                    X.gather_rows(r["xn"], None, r["taps"], dst_col0=j * cfg.hidden_size, pdl=pdl)
+        self._run_stack(st, r["tokens"], r["seq_rows"], r["cu_q"], r["past"], r["positions"], r["slots"], r["mask"], False,
+                        r["NB"], r["xn"], taps=r["taps"], tap_ids=r["tap_ids"], pdl=pdl, embed_pdl=False)
         if self.tp is None:
             X.lm_head_argmax(r["xn"], self.lm_head_w, ws=r["am_ws"], pdl=pdl, out_idx=r["greedy"], out_val=r["am_val"])
         else:
@@ -927,6 +968,8 @@ class FastRound:
         pool, dev, cfg = self.eng.pool, self.device, self.cfg
         T, H = ids.shape[1], cfg.hidden_size
         pool.reserve(sid, total)
+        if self.latent is not None:
+            return self._prefill_ragged(sid, ids, taps)
         row = pool.state(sid).row
         chunk = 512 if self.tp is None else min(512, self.tp.m_cap)
         if self.ep is not None:
@@ -985,6 +1028,22 @@ class FastRound:
         pool.state(sid).length = T
         self._tp_graph_key = None          # eager collectives ran: a batched-verify graph must re-synchronise first
         return int(out_idx.item()), hidden
+
+    def _prefill_ragged(self, sid: int, ids: torch.Tensor, taps, chunk: int = 2048):
+        """Prompt of one sequence through :meth:`ragged_forward` in portions of ``chunk`` tokens; same results as
+        :meth:`_prefill_kernels`."""
+        from ..runtime import build_attn_metadata
+        pool, T = self.eng.pool, ids.shape[1]
+        hidden, logits = [], None
+        for s0 in range(0, T, chunk):
+            n = min(chunk, T - s0)
+            meta = build_attn_metadata(pool, [sid], [s0], num_query_nodes=[n], device=self.device)
+            last = slice(n - 1, n) if s0 + n == T else slice(0, 0)
+            logits, hid = self.ragged_forward(ids[0, s0:s0 + n].to(self.device), meta, [s0], taps, last)
+            if hid is not None:
+                hidden.append(hid)
+            pool.state(sid).length = s0 + n
+        return int(logits[0].argmax()), (torch.cat(hidden) if hidden else None)
 
     # ------------------------------------------------------------------ public entry points
     @torch.inference_mode()
@@ -1137,7 +1196,7 @@ class FastRound:
     def generate_ar(self, sid, ids, sp: SamplingParams):
         """Autoregressive decode = rounds with a one-node tree (budget 1, no drafter)."""
         eng = self.eng
-        if sp.temperature > 0.0 or self.cfg.head_dim != 128:
+        if sp.temperature > 0.0 or not self.cfg.kernel_path_ok():
             logits, _ = eng._prefill(sid, ids[0], reserve=sp.max_new_tokens + 1)
             out = [int(sample(logits[-1], sp.temperature))]
             while len(out) < sp.max_new_tokens and out[-1] not in eng.eos_token_ids:

@@ -205,6 +205,7 @@ def inv_freq(head_dim: int, theta: float, device) -> torch.Tensor:
 
 # ------------------------------------------------------------------ GEMM
 EPI_STORE, EPI_SWIGLU, EPI_ARGMAX, EPI_TOPK, EPI_STORE_F32 = 0, 1, 2, 3, 4
+EPI_RELU2 = 8
 SM_COUNT = 148
 _DEEP = os.environ.get("JETSPEC_GEMM_DEEP", "0") == "1"
 _SPLIT_DEEP = os.environ.get("JETSPEC_SPLIT_DEEP")      # force the split-K pipeline: 1 = 192 KB, 2 = 128 KB, 0 = 96 KB
@@ -685,6 +686,178 @@ def kv_compact(k: torch.Tensor, v: torch.Tensor, past_len: int, keep: torch.Tens
     lib.js_kv_compact.restype = ctypes.c_int
     _check(lib.js_kv_compact(_p(k), _p(v), k.shape[0], k.shape[1], int(past_len), _p(keep), keep.numel(), _stream()),
            "js_kv_compact")
+
+
+# ------------------------------------------------------------------ latent attention, Dynamic Tanh, sigmoid routing
+def _is_bf16(t: torch.Tensor) -> int:
+    assert t.dtype in (torch.bfloat16, torch.float32), t.dtype
+    return int(t.dtype == torch.bfloat16)
+
+
+def dynamic_tanh(x: torch.Tensor, alpha, weight, bias, out_dtype) -> torch.Tensor:
+    """``tanh(alpha x) * weight + bias`` of fp32 rows ``x (T, W)``, result in ``out_dtype``."""
+    lib = load()
+    T, W = x.shape
+    assert x.dtype == torch.float32 and x.stride(1) == 1
+    out = torch.empty(T, W, dtype=out_dtype, device=x.device)
+    _check(lib.js_dynamic_tanh(_p(x), x.stride(0), _p(alpha), _p(weight), _p(bias), _is_bf16(weight), _p(out), W,
+                               _is_bf16(out), T, W, _stream()), "js_dynamic_tanh")
+    return out
+
+
+def gelu_tanh_mul(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    lib = load()
+    gate, up = gate.contiguous(), up.contiguous()
+    out = torch.empty_like(gate)
+    _check(lib.js_gelu_tanh_mul(_p(gate), _p(up), _p(out), ctypes.c_longlong(gate.numel()), _is_bf16(gate), _stream()),
+           "js_gelu_tanh_mul")
+    return out
+
+
+def relu_squared(x: torch.Tensor) -> torch.Tensor:
+    lib = load()
+    x = x.contiguous()
+    out = torch.empty_like(x)
+    _check(lib.js_relu_squared(_p(x), _p(out), ctypes.c_longlong(x.numel()), _is_bf16(x), _stream()), "js_relu_squared")
+    return out
+
+
+def latent_scatter(c: torch.Tensor, pool: torch.Tensor, slots: torch.Tensor) -> None:
+    """Rows ``c (T, R)`` into ``pool (S, Rp)`` at ``slots``; columns past ``R`` are zeroed."""
+    lib = load()
+    assert c.dtype == pool.dtype and c.stride(1) == 1 and pool.is_contiguous() and slots.dtype == torch.int32
+    _check(lib.js_latent_scatter(_p(c), c.stride(0), c.shape[1], _p(pool), pool.shape[1], pool.shape[0], _p(slots), c.shape[0],
+                                 _is_bf16(c), _p(status_word(c.device)), _stream()), "js_latent_scatter")
+
+
+LATENT_TC_MAX = 512        # widest latent row of the tensor-core kernel
+
+
+def latent_attn_splits(tiles: int, Rp: int, max_keys: int) -> int:
+    """Key splits of the tensor-core latent attention: one wave of CTAs, at least a couple of key tiles each."""
+    ctas = max(1, tiles * (2 if Rp > 256 else 1))
+    return max(1, min(SM_COUNT // ctas, (max_keys + 127) // 128, 16))
+
+
+def latent_attention_rows(qa: torch.Tensor, pool: torch.Tensor, heads: int, slot_map, seq_rows, cu_q, past_lens, mask_bits,
+                          scale: float, causal: bool, max_q: int, out: Optional[torch.Tensor] = None,
+                          splits: Optional[int] = None, ws: Optional[dict] = None, max_keys: Optional[int] = None,
+                          pdl: bool = False, impl: Optional[str] = None) -> torch.Tensor:
+    """Attention of absorbed query rows ``qa (T*heads, Rp)`` over the latent rows of ``pool (S, Rp)``; ``out`` has the
+    shape of ``qa``.  ``impl``: ``"tc"`` (bf16, Rp up to 512, masks up to 256 nodes) or ``"simt"``."""
+    lib = load()
+    rows, Rp = qa.shape
+    T, B = rows // heads, seq_rows.numel()
+    assert qa.is_contiguous() and pool.is_contiguous() and pool.shape[1] == Rp and qa.dtype == pool.dtype
+    if out is None:
+        out = torch.empty_like(qa)
+    W = mask_bits.shape[1] if mask_bits is not None else 0
+    if impl is None:
+        impl = "tc" if qa.dtype == torch.bfloat16 and Rp <= LATENT_TC_MAX and W <= 8 else "simt"
+    st = _p(status_word(qa.device))
+    if impl == "simt":
+        _check(lib.js_latent_attention_simt(_p(qa), _p(pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens),
+                                            _p(mask_bits), _p(out), B, T, heads, Rp, pool.shape[0], slot_map.shape[1], W,
+                                            int(causal), ctypes.c_float(scale), _is_bf16(qa), st, _stream()),
+               "js_latent_attention_simt")
+        return out
+    if splits is None:
+        splits = latent_attn_splits(rows // 128 + B, Rp, max_keys if max_keys is not None else slot_map.shape[1])
+    if splits > 1 and ws is None:
+        ws = {"o": torch.empty(splits, rows, Rp, dtype=torch.float32, device=qa.device),
+              "ml": torch.empty(splits, rows, 2, dtype=torch.float32, device=qa.device)}
+    _check(lib.js_latent_attention_tc(_p(qa), _p(pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), _p(mask_bits),
+                                      _p(out), _p(ws["o"] if splits > 1 else None), _p(ws["ml"] if splits > 1 else None), st,
+                                      B, T, heads, Rp, pool.shape[0], slot_map.shape[1], W, int(causal), int(splits),
+                                      int(max_q), ctypes.c_float(scale), int(pdl), _stream()), "js_latent_attention_tc")
+    return out
+
+
+def latent_attention(q: torch.Tensor, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float,
+                     causal: bool) -> torch.Tensor:
+    """Unfused form (see :func:`jetspec_b200.ops.reference.latent_attention`): the key expansion is moved onto the
+    query, the value expansion behind the attention, with library products around the attention kernel."""
+    T, H, D = q.shape
+    R, Rp = w_uk.shape[1], pool.shape[1]
+    V = w_uv.shape[0] // H
+    qa = torch.zeros(T, H, Rp, dtype=q.dtype, device=q.device)
+    qa[:, :, :R] = torch.bmm(q.transpose(0, 1), w_uk.view(H, D, R)).transpose(0, 1)
+    o = latent_attention_rows(qa.view(T * H, Rp), pool, H, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal, T)
+    o = o.view(T, H, Rp)[:, :, :R].transpose(0, 1)
+    return torch.bmm(o, w_uv.view(H, V, R).transpose(1, 2)).transpose(0, 1).reshape(T, H * V)
+
+
+def sigmoid_route(logits: torch.Tensor, correction: torch.Tensor, top: int, scale: float, gate_col: int = -1,
+                  act: Optional[torch.Tensor] = None, wts: Optional[torch.Tensor] = None, idx: Optional[torch.Tensor] = None,
+                  pdl: bool = False):
+    """``(weights (T, k) fp32, experts (T, k) int32)`` from fp32 router logits (a strided view may be wider than the
+    experts: the first ``correction.numel()`` columns count); with ``act`` its rows are scaled in place by
+    ``sigmoid(logits[:, gate_col])``."""
+    lib = load()
+    T, E = logits.shape[0], correction.numel()
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    correction = correction.float().contiguous()
+    if wts is None:
+        wts = torch.empty(T, top, dtype=torch.float32, device=logits.device)
+        idx = torch.empty(T, top, dtype=torch.int32, device=logits.device)
+    _check(lib.js_sigmoid_route(_p(logits), logits.stride(0), _p(correction), T, E, int(top), ctypes.c_float(scale), _p(wts),
+                                _p(idx), int(gate_col), _p(act), act.stride(0) if act is not None else 0,
+                                act.shape[1] if act is not None else 0, int(pdl), _stream()), "js_sigmoid_route")
+    return wts, idx
+
+
+def gemm_inproj(x, w, raw: Optional[torch.Tensor], n_raw: int, act_out: Optional[torch.Tensor], gelu: bool, pdl: bool = False,
+                bn: Optional[int] = None, split: Optional[int] = None, deep: Optional[int] = None) -> None:
+    """Fused input projections: ``x @ w.T`` whose first ``n_raw`` columns go to ``raw`` as fp32 and the rest through the
+    activation (tanh-GELU gate * up on 64-row interleaved weights, or relu^2) to ``act_out`` as bf16."""
+    lib = load()
+    M, K = x.shape
+    N = w.shape[0]
+    if bn is None:
+        tiles2 = ((M + 127) // 128) * (N // 256)
+        if M >= 512 and N % 256 == 0 and tiles2 >= 64:
+            bn, split, deep = 256, 1, 0
+        else:
+            bn, split, deep = pick_gemm_config(M, N, K, EPI_SWIGLU, 128)
+    _check(lib.js_gemm_inproj(_p(x), _p(w), _p(raw), _p(act_out), M, N, K, x.stride(0), w.stride(0),
+                              raw.stride(0) if raw is not None else 0, act_out.stride(0) if act_out is not None else 0,
+                              int(n_raw), 0 if gelu else 1, bn, split, int(deep), _p(status_word(x.device)), int(pdl),
+                              _stream()), f"js_gemm_inproj(M={M},N={N},K={K},bn={bn},split={split})")
+
+
+def gemm_resid32(a, w, x: torch.Tensor, norm=None, h: Optional[torch.Tensor] = None, emb: Optional[torch.Tensor] = None,
+                 pdl: bool = False, bn: Optional[int] = None, split: Optional[int] = None, deep: Optional[int] = None) -> None:
+    """``x += a @ w.T (+ emb)`` on the fp32 residual stream; ``norm = (weight fp32, bias fp32, alpha)`` also writes the
+    Dynamic Tanh of the new ``x`` to ``h``."""
+    lib = load()
+    M, K = a.shape
+    N = w.shape[0]
+    if bn is None:
+        bn, split, deep = pick_gemm_config(M, N, K, EPI_STORE)
+        if bn == 256 and deep != 3:
+            deep = 1
+    nw, nb, alpha = norm if norm is not None else (None, None, 0.0)
+    _check(lib.js_gemm_resid32(_p(a), _p(w), _p(x), _p(x), M, N, K, a.stride(0), w.stride(0), x.stride(0), _p(emb),
+                               emb.stride(0) if emb is not None else 0, _p(h), h.stride(0) if h is not None else 0, _p(nw),
+                               _p(nb), ctypes.c_float(alpha), bn, split, int(deep), _p(status_word(a.device)), int(pdl),
+                               _stream()), f"js_gemm_resid32(M={M},N={N},K={K},bn={bn},split={split})")
+
+
+def gemm_batched(a, w, out, batch: int, N: int, K: int, a_batch_k: int, c_batch_stride: int, ldc: int, pdl: bool = False) -> None:
+    """``batch`` products in one launch: columns ``[z * a_batch_k, + K)`` of ``a`` times rows ``[z * N, + N)`` of ``w``
+    (transposed), to ``out + z * c_batch_stride`` with leading dimension ``ldc``."""
+    lib = load()
+    _check(lib.js_gemm_bf16_batched(_p(a), _p(w), _p(out), a.shape[0], N, K, batch, a_batch_k, ctypes.c_longlong(c_batch_stride),
+                                    a.stride(0), w.stride(0), ldc, _p(status_word(a.device)), int(pdl), _stream()),
+           f"js_gemm_bf16_batched(M={a.shape[0]},N={N},K={K},batch={batch})")
+
+
+def gemm_grouped(a, w, out, total_rows: int, N: int, groups: int, group_off, cover: int, epi: int) -> None:
+    """Grouped GEMM over experts (rows of ``a`` sorted by expert, weights stacked)."""
+    lib = load()
+    _check(lib.js_gemm_bf16_grouped(_p(a), _p(w), _p(out), total_rows, N, a.shape[1], a.stride(0), w.stride(0), out.stride(0), epi,
+                                    groups, _p(group_off), cover, None, None, None, None, 1, _p(status_word(a.device)), 0,
+                                    _stream()), f"js_gemm_bf16_grouped(rows={total_rows},N={N},groups={groups},epi={epi})")
 
 
 # ------------------------------------------------------------------ MoE (grouped through the dense GEMM)

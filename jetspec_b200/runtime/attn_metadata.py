@@ -28,6 +28,7 @@ class AttnMeta:
     causal: bool
     max_q: int                  # largest per-sequence query count
     num_tokens: int
+    counts: Optional[list] = None      # query rows per sequence, as host integers
 
 
 def build_attn_metadata(pool, seq_ids: Sequence[int], past_lens: Sequence[int],
@@ -74,4 +75,4 @@ def build_attn_metadata(pool, seq_ids: Sequence[int], past_lens: Sequence[int],
         seq_rows=to(rows), cu_q=to(cu), past_lens=to(np.asarray(past_lens, dtype=np.int32)),
         positions=to(pos), slots=slots,
         mask_bits=(torch.from_numpy(bits.view(np.int32)).to(device) if bits is not None else None),
-        causal=causal, max_q=max(counts) if counts else 0, num_tokens=T)
+        causal=causal, max_q=max(counts) if counts else 0, num_tokens=T, counts=counts)
