@@ -479,8 +479,8 @@ class JetSpecEngine:
         return out
 
     # ------------------------------------------------------------ batching
-    def _make_scheduler(self, n_requests: int, max_batch_size: Optional[int]) -> Scheduler:
-        return Scheduler(self.pool, max_batch_size=max_batch_size or min(n_requests, self.pool.max_seqs),
+    def _make_scheduler(self, n_requests: int, max_batch_size: Optional[int], admission_evicts: bool = True) -> Scheduler:
+        return Scheduler(self.pool, admission_evicts=admission_evicts, max_batch_size=max_batch_size or min(n_requests, self.pool.max_seqs),
                          prefill_batch_size=max_batch_size or min(n_requests, self.pool.max_seqs))
 
     def _ensure_room(self, sched: Scheduler, req: SequenceRequest, tokens: int) -> bool:
@@ -514,7 +514,7 @@ class JetSpecEngine:
             self._ensure_pool(sum(int(r.numel()) + sp.max_new_tokens + 1 for r in id_rows), seqs=len(prompts))
         if self.pool.max_seq_len < longest:
             self._ensure_pool(longest * len(prompts), seqs=len(prompts))
-        sched = self._make_scheduler(len(prompts), max_batch_size)
+        sched = self._make_scheduler(len(prompts), max_batch_size, admission_evicts=not prefill_chunk)
         reqs = {}
         for i, row in enumerate(id_rows):
             r = SequenceRequest(seq_id=self._new_seq_id(), input_ids=row.tolist(), max_new_tokens=sp.max_new_tokens,

@@ -29,7 +29,8 @@ class TraceReplay:
         from ..runtime import Scheduler
         self.eng = engine
         pool = engine.reserve_pool(max_tokens, LIVE_REQUESTS)
-        self.sched = Scheduler(pool, max_batch_size=LIVE_REQUESTS, prefill_batch_size=LIVE_REQUESTS)
+        self.sched = Scheduler(pool, max_batch_size=LIVE_REQUESTS, prefill_batch_size=LIVE_REQUESTS,
+                               admission_evicts=False)
         self.live: dict = {}
 
     def admit(self, name: str, tokens: list) -> None:

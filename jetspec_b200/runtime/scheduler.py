@@ -66,13 +66,17 @@ class SchedulerOutput:
 
 class Scheduler:
     def __init__(self, cache: PagedKVPool, max_batch_size: int = 32, prefill_batch_size: int = 8,
-                 scheduling_policy: str = "fcfs", eviction_policy: str = "lru", max_queue: Optional[int] = None):
+                 scheduling_policy: str = "fcfs", eviction_policy: str = "lru", max_queue: Optional[int] = None,
+                 admission_evicts: bool = True):
         self.cache = cache
         self.max_batch_size = int(max_batch_size)
         self.prefill_batch_size = int(prefill_batch_size)
         self.policy = scheduling_policy
         self.evict_policy = eviction_policy
         self.max_queue = max_queue
+        # False: a waiting request is admitted only into free pages (prompts fed in portions need this: a request that
+        # is evicted before its last portion would start over, and two such requests could evict each other for ever)
+        self.admission_evicts = bool(admission_evicts)
         self.waiting_queue: deque = deque()
         self.running: dict = {}
         self.finished: dict = {}
@@ -99,6 +103,8 @@ class Scheduler:
             if not self._feasible_without(req.seq_id, want, protect):
                 # only the pages of requests admitted in this very step would make room, and those are never
                 # evicted: stop here instead of evicting every other sequence for nothing
+                break
+            if not self.admission_evicts and not self._fits_free(req.seq_id, want):
                 break
             ok = self._allocate_protecting(req.seq_id, want, protect)
             for sid in before - set(self.cache.resident()):
@@ -130,6 +136,11 @@ class Scheduler:
         evictable = sum(len(cache.state(sid).pages) for sid in self.running
                         if sid not in protect and sid != seq_id and cache.has(sid))
         return need <= cache.free_page_count + evictable
+
+    def _fits_free(self, seq_id: int, want: int) -> bool:
+        cache = self.cache
+        have = len(cache.state(seq_id).pages) if cache.has(seq_id) else 0
+        return cache.pages_for(want) - have <= cache.free_page_count
 
     def _allocate_protecting(self, seq_id: int, want: int, protect: list) -> bool:
         """Allocate, evicting policy-chosen victims; never evict a request admitted this step."""
