@@ -27,7 +27,7 @@ namespace js {
 constexpr int LROWS = 128;
 constexpr int LLOADERS = 256;
 constexpr int LTHREADS = 160 + LLOADERS;
-constexpr int LMAX_STAGES = 4;
+constexpr int LMAX_STAGES = 6;
 constexpr int kLatentSmemMax = 227 * 1024;
 
 struct LatentAttnParams {
@@ -232,8 +232,10 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
         for (int ch = 0; ch < nk; ++ch) lat_cp16(dst + ch * k_chunk, src + ch * 64, valid);
       }
       lat_commit();
-      lat_wait<2>();
-      publish_before(i - 1);
+      // all but the newest NST - 1 tiles have landed: publish as early as the ring allows
+      if (NST == 2) { lat_wait<1>(); publish_before(i); }
+      else if (NST == 3) { lat_wait<2>(); publish_before(i - 1); }
+      else { lat_wait<3>(); publish_before(i - 2); }
     }
     lat_wait<0>();                                      // on an error path too: no copy outlives the CTA
     if (ok) publish_before(nt);
@@ -254,11 +256,8 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
         umma_commit(&kv_empty[s]);
         umma_commit(&pv_done[pb]);
       };
-      for (int i = 0; i < nt && ok; ++i) {
+      auto issue_qk = [&](int i) {
         const int s = i % NST, sb = i & 1;
-        ok = lat_mbar_wait(&kv_full[s], (i / NST) & 1, p.status, kTimeoutFull);
-        if (!ok) break;
-        tc_fence_after();
         const uint32_t k_addr = smem_u32(sK + s * k_stage);
         for (int ch = 0; ch < nk; ++ch) {
           const uint64_t a = umma_desc_sw128(smem_u32(sQ) + ch * q_chunk), bd = umma_desc_sw128(k_addr + ch * k_chunk);
@@ -266,11 +265,28 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
           for (int kk = 0; kk < 4; ++kk) umma_f16(tmem_base + sb * 64, a + 2 * kk, bd + 2 * kk, idesc_qk, (ch | kk) != 0 ? 1u : 0u);
         }
         umma_commit(&s_full[sb]);
-        if (i >= 1) {
-          ok = lat_mbar_wait(&p_full[(i - 1) & 1], ((i - 1) >> 1) & 1, p.status, kTimeoutAccum);
-          if (!ok) break;
-          tc_fence_after();
-          issue_pv(i - 1);
+      };
+      for (int i = 0; i < nt && ok; ++i) {
+        // QK(i) needs tile i, PV(i-1) the probabilities of tile i-1; whichever is ready first goes first.  (With two
+        // stages tile i cannot even be loaded before PV(i-2) is done, so PV must never queue behind a tile in flight.)
+        bool qk = false, pv = i == 0;
+        for (uint32_t it = 0; ok && !(qk && pv); ++it) {
+          if (!qk && mbar_test_wait(&kv_full[i % NST], (i / NST) & 1)) {
+            tc_fence_after();
+            issue_qk(i);
+            qk = true;
+          }
+          if (!pv && mbar_test_wait(&p_full[(i - 1) & 1], ((i - 1) >> 1) & 1)) {
+            tc_fence_after();
+            issue_pv(i - 1);
+            pv = true;
+          }
+          if (qk && pv) break;
+          __nanosleep(20);
+          if (it >= kSpinLimit) {
+            report(p.status, qk ? kTimeoutAccum : kTimeoutFull);
+            ok = false;
+          }
         }
       }
       if (ok) {
@@ -432,35 +448,36 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
   }
 }
 
-// one warp per (token, head) row: merge the key splits
+// one CTA per (token, head) row: merge the key splits (at most 16; four columns per thread)
+constexpr int LMAX_SPLITS = 16;
 __global__ void __launch_bounds__(128)
 latent_attn_merge_kernel(const float* ws_o, const float* ws_ml, __nv_bfloat16* out, int rows, int Rp, int splits) {
   pdl_launch_dependents();
   pdl_wait();
-  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (row >= rows) return;
-  float m = -INFINITY;
-  for (int s = 0; s < splits; ++s) m = fmaxf(m, ws_ml[(static_cast<size_t>(s) * rows + row) * 2]);
-  float l = 0.f;
+  const int row = blockIdx.x, c = threadIdx.x * 4;
+  __shared__ float w[LMAX_SPLITS];
+  if (threadIdx.x < 32) {
+    const int s = threadIdx.x;
+    float2 ml = make_float2(-INFINITY, 0.f);
+    if (s < splits) ml = *reinterpret_cast<const float2*>(ws_ml + (static_cast<size_t>(s) * rows + row) * 2);
+    const float m = warp_max(ml.x);
+    const float f = ml.x == -INFINITY ? 0.f : exp2f(ml.x - m);
+    const float l = warp_sum(ml.y * f);
+    if (s < LMAX_SPLITS) w[s] = l > 0.f ? f / l : 0.f;
+  }
+  __syncthreads();
+  if (c >= Rp) return;
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
   for (int s = 0; s < splits; ++s) {
-    const float* ml = ws_ml + (static_cast<size_t>(s) * rows + row) * 2;
-    if (ml[0] != -INFINITY) l += ml[1] * exp2f(ml[0] - m);
+    const float f = w[s];
+    if (f == 0.f) continue;                          // that split saw no visible key (its O may be unwritten)
+    const float4 v = *reinterpret_cast<const float4*>(ws_o + (static_cast<size_t>(s) * rows + row) * Rp + c);
+    acc[0] += v.x * f; acc[1] += v.y * f; acc[2] += v.z * f; acc[3] += v.w * f;
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
-  for (int c = lane * 4; c < Rp; c += 128) {
-    float acc[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int s = 0; s < splits; ++s) {
-      const float ms = ws_ml[(static_cast<size_t>(s) * rows + row) * 2];
-      if (ms == -INFINITY) continue;                 // that split saw no visible key (its O may be unwritten)
-      const float w = exp2f(ms - m);
-      const float4 v = *reinterpret_cast<const float4*>(ws_o + (static_cast<size_t>(s) * rows + row) * Rp + c);
-      acc[0] += v.x * w; acc[1] += v.y * w; acc[2] += v.z * w; acc[3] += v.w * w;
-    }
-    __nv_bfloat162* dst = reinterpret_cast<__nv_bfloat162*>(out + static_cast<size_t>(row) * Rp + c);
-    dst[0] = __floats2bfloat162_rn(acc[0] * inv, acc[1] * inv);
-    dst[1] = __floats2bfloat162_rn(acc[2] * inv, acc[3] * inv);
-  }
+  __nv_bfloat162* dst = reinterpret_cast<__nv_bfloat162*>(out + static_cast<size_t>(row) * Rp + c);
+  dst[0] = __floats2bfloat162_rn(acc[0], acc[1]);
+  dst[1] = __floats2bfloat162_rn(acc[2], acc[3]);
 }
 
 template <int TK>
@@ -484,15 +501,15 @@ static int launch_latent(const LatentAttnParams& p, int q_tiles, int groups, int
 }  // namespace js
 
 // q, out (T*H, Rp) bf16, pool (S, Rp) bf16, Rp a multiple of 64 up to 512; max_q = most query tokens of one sequence;
-// masks of up to 8 words per token.  splits > 1 needs ws_o (splits, T*H, Rp) fp32 and ws_ml (splits, T*H, 2) fp32.
+// masks of up to 8 words per token; tk_want = keys per tile (32, or 64 where it fits; 0 picks).  splits > 1 needs ws_o (splits, T*H, Rp) fp32 and ws_ml (splits, T*H, 2) fp32.
 extern "C" int js_latent_attention_tc(const void* q, const void* pool, const int* slot_map, const int* seq_rows, const int* cu_q,
                                       const int* past_lens, const int* mask_bits, void* out, float* ws_o, float* ws_ml, int* status,
                                       int B, int T, int H, int Rp, int S, int max_len, int W, int causal, int splits, int max_q,
-                                      float scale, int pdl, cudaStream_t stream) {
+                                      float scale, int tk_want, int pdl, cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
   if (Rp % 64 || Rp < 64 || Rp > 512 || H < 1) return -10;
-  if (splits < 1) return -11;
+  if (splits < 1 || splits > LMAX_SPLITS) return -11;
   if (splits > 1 && (ws_o == nullptr || ws_ml == nullptr)) return -12;
   if (!causal && (mask_bits == nullptr || W < 1 || W > 8)) return -13;
   const int nk = Rp / 64;
@@ -500,7 +517,8 @@ extern "C" int js_latent_attention_tc(const void* q, const void* pool, const int
   const int rq = rows <= 32 ? 32 : rows <= 64 ? 64 : 128;
   const int budget = kLatentSmemMax - 1024 - 256;
   int tk = 64, stages = (budget - nk * rq * 128 - lat_p_bytes(64, rq)) / lat_stage_bytes(64, nk);
-  if (stages < 2) {
+  if (tk_want != 0 && tk_want != 32 && tk_want != 64) return -10;
+  if (stages < 2 || tk_want == 32) {
     tk = 32;
     stages = (budget - nk * rq * 128 - lat_p_bytes(32, rq)) / lat_stage_bytes(32, nk);
   }
@@ -520,7 +538,7 @@ extern "C" int js_latent_attention_tc(const void* q, const void* pool, const int
                           : launch_latent<32>(p, q_tiles, groups, smem, pdl != 0, stream);
   if (rc != 0 || splits == 1) return rc;
   cudaLaunchConfig_t c2 = {};
-  c2.gridDim = dim3((T * H + 3) / 4);
+  c2.gridDim = dim3(T * H);
   c2.blockDim = dim3(128);
   c2.stream = stream;
   cudaLaunchAttribute attr[1];

@@ -41,6 +41,7 @@ struct AttnParams {
   int* status;
   int B, T, Hq, Hkv, S, max_len, W, causal, splits;
   float scale_log2;            // softmax scale * log2(e)
+  int ldo;                     // merge kernel: elements between tokens of `out`
 };
 
 JS_DEVICE void cp_async16(void* smem, const void* gmem, bool valid) {
@@ -314,7 +315,7 @@ __global__ void attn_merge_kernel(AttnParams p) {
     acc[0] += v.x * w; acc[1] += v.y * w; acc[2] += v.z * w; acc[3] += v.w * w;
   }
   const float inv = l > 0.f ? 1.f / l : 0.f;
-  __nv_bfloat16* dst = p.out + static_cast<size_t>(row) * AD + lane * 4;
+  __nv_bfloat16* dst = p.out + static_cast<size_t>(row / p.Hq) * p.ldo + (row % p.Hq) * AD + lane * 4;
   *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(acc[0] * inv, acc[1] * inv);
   *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(acc[2] * inv, acc[3] * inv);
 }
@@ -368,7 +369,7 @@ extern "C" int js_paged_tree_attention(const void* q, const void* k_pool, const 
   AttnParams p{reinterpret_cast<const __nv_bfloat16*>(q), reinterpret_cast<const __nv_bfloat16*>(k_pool),
                reinterpret_cast<const __nv_bfloat16*>(v_pool), slot_map, seq_rows, cu_q, past_lens, mask_bits,
                reinterpret_cast<__nv_bfloat16*>(out), ws_o, ws_ml, status, B, T, Hq, Hkv, S, max_len, W, causal,
-               splits, scale * 1.4426950408889634f};
+               splits, scale * 1.4426950408889634f, Hq * AD};
   switch (G) {
     case 1: return launch_attn<1>(p, T + B, pdl != 0, stream);
     case 2: return launch_attn<2>(p, (T + 31) / 32 + B, pdl != 0, stream);
@@ -379,12 +380,13 @@ extern "C" int js_paged_tree_attention(const void* q, const void* k_pool, const 
   }
 }
 
-// Merge the key splits of a (splits, T, Hq, 128) fp32 workspace with its (max, sum) pairs into out (T, Hq*128).
-extern "C" int js_attn_merge(float* ws_o, float* ws_ml, void* out, int T, int Hq, int splits, int pdl, cudaStream_t stream) {
+// Merge the key splits of a (splits, T, Hq, 128) fp32 workspace with its (max, sum) pairs into out (T, Hq*128), ldo elements
+// between tokens.
+extern "C" int js_attn_merge(float* ws_o, float* ws_ml, void* out, int ldo, int T, int Hq, int splits, int pdl, cudaStream_t stream) {
   using namespace js;
   AttnParams p{};
   p.ws_o = ws_o; p.ws_ml = ws_ml; p.out = reinterpret_cast<__nv_bfloat16*>(out);
-  p.T = T; p.Hq = Hq; p.splits = splits;
+  p.T = T; p.Hq = Hq; p.splits = splits; p.ldo = ldo;
   cudaLaunchConfig_t c2 = {};
   c2.gridDim = dim3((T * Hq + 7) / 8);
   c2.blockDim = dim3(256);

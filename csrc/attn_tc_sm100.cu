@@ -56,6 +56,8 @@ struct AttnTcParams {
   int* status;
   int B, T, Hq, Hkv, S, max_len, W, causal, splits;
   float scale_log2;
+  long long kv_head, kv_slot;  // elements between heads / slots of the pools (S*128 and 128 for a (Hkv, S, 128) pool)
+  int ldo;                     // elements between tokens of `out`
   int cluster_merge;           // the key splits of a tile form a cluster and merge through distributed shared memory
 };
 
@@ -170,6 +172,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   const int node = node0 + row / G, head = h * G + row % G;
   const bool row_valid = node < n_b;
   const size_t out_row = static_cast<size_t>(q_begin + (row_valid ? node : 0)) * p.Hq + head;
+  __nv_bfloat16* out_ptr = p.out + static_cast<size_t>(q_begin + (row_valid ? node : 0)) * p.ldo + head * TD;
 
   const bool cmerge = p.cluster_merge != 0;
   float m_run = -INFINITY, l_run = 0.f;     // softmax threads: running (integer) maximum and sum of their row
@@ -263,7 +266,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         const bool valid = kp < L;
         int slot = slot_cur[j];
         if (slot < 0 || slot >= p.S) { report(p.status, kBadSlot); slot = 0; }
-        const size_t off = (static_cast<size_t>(h) * p.S + slot) * TD + ch * 8;
+        const size_t off = static_cast<size_t>(h) * p.kv_head + static_cast<size_t>(slot) * p.kv_slot + ch * 8;
         const uint32_t dst = (ch >> 3) * (TKEYS * 128) + r * 128 + (((ch & 7) ^ (r & 7)) << 4);
         cp_async16_tc(k_addr + dst, p.k_pool + off, valid);
         cp_async16_tc(k_addr + TKEYS * 256 + dst, p.v_pool + off, valid);
@@ -452,7 +455,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 #pragma unroll
           for (int j = 0; j < 16; ++j)
             o2[j] = __floats2bfloat162_rn(__uint_as_float(orr[2 * j]) * inv, __uint_as_float(orr[2 * j + 1]) * inv);
-          uint4* dst = reinterpret_cast<uint4*>(p.out + out_row * TD + c0);
+          uint4* dst = reinterpret_cast<uint4*>(out_ptr + c0);
 #pragma unroll
           for (int j = 0; j < 4; ++j) dst[j] = pk[j];
         } else {
@@ -535,7 +538,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(pk);
 #pragma unroll
         for (int j = 0; j < 16; ++j) o2[j] = __floats2bfloat162_rn(acc[2 * j] * inv, acc[2 * j + 1] * inv);
-        uint4* dst = reinterpret_cast<uint4*>(p.out + out_row * TD + c * 32);
+        uint4* dst = reinterpret_cast<uint4*>(out_ptr + c * 32);
 #pragma unroll
         for (int j = 0; j < 4; ++j) dst[j] = pk[j];
       }
@@ -588,7 +591,7 @@ extern "C" int js_attn_tc_set_trace(unsigned long long* buf) {
   return cudaMemcpyToSymbol(js::g_attn_trace, &buf, sizeof(buf)) == cudaSuccess ? 0 : -1;
 }
 
-extern "C" int js_attn_merge(float* ws_o, float* ws_ml, void* out, int T, int Hq, int splits, int pdl, cudaStream_t stream);
+extern "C" int js_attn_merge(float* ws_o, float* ws_ml, void* out, int ldo, int T, int Hq, int splits, int pdl, cudaStream_t stream);
 
 // How many clusters of `splits` CTAs of the kernel for GQA group size G can be resident at once on the current
 // device (a cluster lives inside one GPC, so this is less than SMs / splits); 0 or negative = cannot say.  The host
@@ -622,15 +625,18 @@ extern "C" int js_attn_tc_max_active_clusters(int G, int splits) {
   return n;
 }
 
-// Same arguments as js_paged_tree_attention.  Needs 128 % (Hq / Hkv) == 0 and W <= 8 (windows of up to 256 nodes).
-extern "C" int js_paged_tree_attention_tc(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
+// js_paged_tree_attention with the layout of the pools and the output spelled out: head h of slot s starts at
+// h * kv_head + s * kv_slot, token t of the output at t * ldo (all multiples of 8).  Needs 128 % (Hq / Hkv) == 0 and
+// W <= 8 (windows of up to 256 nodes).
+extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
                                           const int* seq_rows, const int* cu_q, const int* past_lens,
                                           const int* mask_bits, void* out, float* ws_o, float* ws_ml, int* status, int B,
                                           int T, int Hq, int Hkv, int S, int max_len, int W, int causal, int splits,
-                                          float scale, int pdl, cudaStream_t stream) {
+                                          float scale, long long kv_head, long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
   if (Hq % Hkv) return -10;
+  if ((kv_head % 8) || (kv_slot % 8) || (ldo % 8)) return -10;
   const int G = Hq / Hkv;
   if (splits < 1) return -11;
   if (splits > 1 && (ws_o == nullptr || ws_ml == nullptr)) return -12;
@@ -656,7 +662,7 @@ extern "C" int js_paged_tree_attention_tc(const void* q, const void* k_pool, con
   AttnTcParams p{reinterpret_cast<const __nv_bfloat16*>(q), reinterpret_cast<const __nv_bfloat16*>(k_pool),
                  reinterpret_cast<const __nv_bfloat16*>(v_pool), slot_map, seq_rows, cu_q, past_lens, mask_bits,
                  reinterpret_cast<__nv_bfloat16*>(out), ws_o, ws_ml, status, B, T, Hq, Hkv, S, max_len, W, causal,
-                 splits, scale * 1.4426950408889634f, in_cluster ? 1 : 0};
+                 splits, scale * 1.4426950408889634f, kv_head, kv_slot, ldo, in_cluster ? 1 : 0};
   int rc;
   switch (G) {
     case 1: rc = launch_attn_tc<1>(p, (T + 127) / 128 + B, pdl != 0, stream); break;
@@ -667,5 +673,16 @@ extern "C" int js_paged_tree_attention_tc(const void* q, const void* k_pool, con
     default: return -14;
   }
   if (rc != 0 || splits == 1 || p.cluster_merge) return rc;
-  return js_attn_merge(ws_o, ws_ml, out, T, Hq, splits, pdl, stream);
+  return js_attn_merge(ws_o, ws_ml, out, ldo, T, Hq, splits, pdl, stream);
+}
+
+// Same arguments as js_paged_tree_attention.
+extern "C" int js_paged_tree_attention_tc(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
+                                          const int* seq_rows, const int* cu_q, const int* past_lens,
+                                          const int* mask_bits, void* out, float* ws_o, float* ws_ml, int* status, int B,
+                                          int T, int Hq, int Hkv, int S, int max_len, int W, int causal, int splits,
+                                          float scale, int pdl, cudaStream_t stream) {
+  return js_paged_attention_tc_strided(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ws_o, ws_ml, status,
+                                       B, T, Hq, Hkv, S, max_len, W, causal, splits, scale,
+                                       static_cast<long long>(S) * js::TD, js::TD, Hq * js::TD, pdl, stream);
 }

@@ -96,26 +96,38 @@ latent_post_kernel(const float* proj, int ldp, int q_rank, int kv_rank, const __
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
-  const float* src = proj + static_cast<size_t>(t) * ldp;
-  if (blockIdx.y == 0) {
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < q_rank; i += blockDim.x) ss += src[i] * src[i];
-    const float inv = 1.f / sqrtf(block_sum(ss, red) / q_rank + eps);
-    for (int i = threadIdx.x; i < qp; i += blockDim.x)
-      cq[static_cast<size_t>(t) * qp + i] = __float2bfloat16_rn(i < q_rank ? src[i] * inv * __bfloat162float(qw[i]) : 0.f);
-    return;
+  const bool is_q = blockIdx.y == 0;
+  const int n = is_q ? q_rank : kv_rank, width = is_q ? qp : Rp;
+  const float* src = proj + static_cast<size_t>(t) * ldp + (is_q ? 0 : q_rank);
+  const __nv_bfloat16* w = is_q ? qw : kw;
+  size_t row = t;
+  if (!is_q) {
+    const int slot = slots[t];
+    if (slot < 0 || slot >= S) {
+      if (threadIdx.x == 0) report(status, kBadSlot);
+      return;
+    }
+    row = slot;
   }
-  src += q_rank;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < kv_rank; i += blockDim.x) ss += src[i] * src[i];
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / kv_rank + eps);
-  const int slot = slots[t];
-  if (slot < 0 || slot >= S) {
-    if (threadIdx.x == 0) report(status, kBadSlot);
-    return;
+  constexpr int KEEP = 8;                    // values a thread holds on to (latents up to 2048 wide); the rest is read twice
+  float v[KEEP], ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int i = threadIdx.x + j * 256;
+    v[j] = i < n ? src[i] : 0.f;
   }
-  for (int i = threadIdx.x; i < Rp; i += blockDim.x)
-    pool[static_cast<size_t>(slot) * Rp + i] = __float2bfloat16_rn(i < kv_rank ? src[i] * inv * __bfloat162float(kw[i]) : 0.f);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) ss += v[j] * v[j];
+  for (int i = threadIdx.x + KEEP * 256; i < n; i += 256) ss += src[i] * src[i];
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / n + eps);
+  __nv_bfloat16* dst = (is_q ? cq : pool) + row * width;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int i = threadIdx.x + j * 256;
+    if (i < width) dst[i] = __float2bfloat16_rn(i < n ? v[j] * inv * __bfloat162float(w[i]) : 0.f);
+  }
+  for (int i = threadIdx.x + KEEP * 256; i < width; i += 256)
+    dst[i] = __float2bfloat16_rn(i < n ? src[i] * inv * __bfloat162float(w[i]) : 0.f);
 }
 
 // Sigmoid routing, one warp per token: scores s = sigmoid(z), the k largest s + correction are chosen (ties: lower

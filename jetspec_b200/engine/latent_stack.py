@@ -60,7 +60,7 @@ class _LayerWeights:
         # the K/V kernel has 128-wide heads; padding narrower ones up to it pays from 64 on
         self.expand = 64 <= m.dim <= 128 and 64 <= m.vdim <= 128
         self.dp, self.vp = (128, 128) if self.expand else (_up(m.dim, 8), _up(m.vdim, 8))
-        self.norm = (layer.norm.weight.float(), layer.norm.bias.float(), float(layer.norm.alpha))
+        self.norm = (layer.norm.weight.float(), layer.norm.bias.float(), layer.norm.alpha.item())
         self.q_norm, self.kv_norm = mix.q_norm, mix.kv_norm
         raw = [mix.q_down.weight, mix.kv_down.weight]
         self.moe = None
@@ -96,7 +96,8 @@ class _LayerWeights:
         self.uk_t = _pad_heads(uk.view(m.heads, m.dim, m.kv_rank).transpose(1, 2).reshape(m.heads * m.kv_rank, m.dim),
                                m.heads, self.rp, self.dp)
         self.uv = _pad_heads(uv, m.heads, self.vp, self.rp)
-        self.uk = _pad_heads(uk, m.heads, self.dp, self.rp) if self.expand else None
+        # keys and values of every head from a latent row, one product: [heads * 128 keys | heads * 128 values]
+        self.ukv = torch.cat((_pad_heads(uk, m.heads, self.dp, self.rp), self.uv), 0) if self.expand else None
         attn_cols = m.heads * self.vp
         self.cat_cols = attn_cols + self.act_cols
         self.w_out = torch.zeros(wp, self.cat_cols, dtype=uk.dtype, device=uk.device)
@@ -118,7 +119,7 @@ class LatentStack:
         for L in self.layers:
             L.norm = self._pad_norm(*L.norm)
         fn = model.model.norm
-        self.final_norm = self._pad_norm(fn.weight.float(), fn.bias.float(), float(fn.alpha))
+        self.final_norm = self._pad_norm(fn.weight.float(), fn.bias.float(), fn.alpha.item())
         self.runs = cfg.layer_runs()
         table = model.model.embed_tokens.weight
         self.table = table if self.wp == self.width else _pad(table, table.shape[0], self.wp)
@@ -246,16 +247,12 @@ class LatentStack:
 
     def _expanded(self, st, L, pool, batch, part, q, cat, pdl) -> int:
         r0, r1, H, keys = part.r0, part.r1, L.heads, part.keys
-        c = st.get("c", L.rp, rows=keys)
-        kv = st.get("kv", H * 256, rows=keys).view(2, H, keys, 128)
+        c, kv = st.get("c", L.rp, rows=keys), st.get("kv", H * 256, rows=keys)
         X.gather_rows(pool, part.key_slots, c, pdl=pdl)
-        X.gemm_batched(c, L.uk, kv[0], H, 128, L.rp, 0, keys * 128, 128, pdl=pdl)
-        X.gemm_batched(c, L.uv, kv[1], H, 128, L.rp, 0, keys * 128, 128, pdl=pdl)
-        o = st.get("attn", H * 128)[r0:r1]
-        X.paged_tree_attention(q[r0:r1].view(r1 - r0, H, 128), kv[0], kv[1], part.key_map, part.key_base, part.cu_q, part.past, None,
-                               L.scale, True, part.max_q, out=o, max_keys=part.max_keys, pdl=pdl)
-        X.gather_rows(o, None, cat[r0:r1], pdl=pdl)
-        return 5
+        X.gemm(c, L.ukv, out=kv, pdl=pdl)
+        X.paged_attention_rows(q[r0:r1].view(r1 - r0, H, 128), kv[:, : H * 128], kv[:, H * 128:], part.key_map, part.key_base, part.cu_q,
+                               part.past, L.scale, part.max_q, cat[r0:r1], part.max_keys, pdl=pdl)
+        return 3
 
     def _experts(self, st, L, raw, act, pdl):
         """Route, sort by expert, run the two grouped GEMMs; the weighted rows stay behind for :meth:`_combine`."""

@@ -615,6 +615,27 @@ def paged_tree_attention(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens,
     return out
 
 
+def paged_attention_rows(q, k_rows, v_rows, slot_map, seq_rows, cu_q, past_lens, scale: float, max_q: int, out, max_keys: int,
+                         pdl: bool = False) -> torch.Tensor:
+    """Causal attention over keys and values stored row-major, ``k_rows, v_rows (keys, Hkv*128)`` (views of one wider
+    matrix are fine), on the tcgen05 kernel; ``out (T, >= Hq*128)`` may be a column block of a wider matrix."""
+    lib = load()
+    T, Hq, D = q.shape
+    Hkv = k_rows.shape[1] // 128
+    assert D == 128 and q.is_contiguous() and k_rows.stride(1) == 1 and v_rows.stride() == k_rows.stride()
+    splits = attn_splits_for(T, Hq, Hkv, max_keys)
+    ws_o = ws_ml = None
+    if splits > 1:
+        ws_o = torch.empty(splits, T, Hq, D, dtype=torch.float32, device=q.device)
+        ws_ml = torch.empty(splits, T, Hq, 2, dtype=torch.float32, device=q.device)
+    _check(lib.js_paged_attention_tc_strided(
+        _p(q), _p(k_rows), _p(v_rows), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), None, _p(out), _p(ws_o), _p(ws_ml),
+        _p(status_word(q.device)), seq_rows.numel(), T, Hq, Hkv, k_rows.shape[0], slot_map.shape[1], 0, 1, splits,
+        ctypes.c_float(scale), ctypes.c_longlong(128), ctypes.c_longlong(k_rows.stride(0)), out.stride(0), int(pdl), _stream()),
+        "js_paged_attention_tc_strided")
+    return out
+
+
 def l2_prefetch(t: torch.Tensor, max_bytes: Optional[int] = None, ctas: int = 8) -> None:
     """Ask the memory system to pull the first ``max_bytes`` of ``t`` into L2 (launch on the CURRENT stream;
     the kernel only issues ``cp.async.bulk.prefetch.L2`` requests and exits)."""
@@ -742,7 +763,7 @@ def latent_attn_splits(tiles: int, Rp: int, max_keys: int) -> int:
 def latent_attention_rows(qa: torch.Tensor, pool: torch.Tensor, heads: int, slot_map, seq_rows, cu_q, past_lens, mask_bits,
                           scale: float, causal: bool, max_q: int, out: Optional[torch.Tensor] = None,
                           splits: Optional[int] = None, ws: Optional[dict] = None, max_keys: Optional[int] = None,
-                          pdl: bool = False, impl: Optional[str] = None) -> torch.Tensor:
+                          pdl: bool = False, impl: Optional[str] = None, tile: int = 0) -> torch.Tensor:
     """Attention of absorbed query rows ``qa (T*heads, Rp)`` over the latent rows of ``pool (S, Rp)``; ``out`` has the
     shape of ``qa``.  ``impl``: ``"tc"`` (bf16, Rp up to 512, masks up to 256 nodes) or ``"simt"``."""
     lib = load()
@@ -769,7 +790,7 @@ def latent_attention_rows(qa: torch.Tensor, pool: torch.Tensor, heads: int, slot
     _check(lib.js_latent_attention_tc(_p(qa), _p(pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), _p(mask_bits),
                                       _p(out), _p(ws["o"] if splits > 1 else None), _p(ws["ml"] if splits > 1 else None), st,
                                       B, T, heads, Rp, pool.shape[0], slot_map.shape[1], W, int(causal), int(splits),
-                                      int(max_q), ctypes.c_float(scale), int(pdl), _stream()), "js_latent_attention_tc")
+                                      int(max_q), ctypes.c_float(scale), int(tile), int(pdl), _stream()), "js_latent_attention_tc")
     return out
 
 

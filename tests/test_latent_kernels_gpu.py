@@ -189,16 +189,18 @@ def test_sigmoid_routing_and_shared_gate(ext, T, E, k):
     assert torch.equal(act[:, 32:], before[:, 32:])
 
 
-def test_latent_norms_go_to_the_query_and_to_the_pool(ext):
-    T, qr, kr, eps = 9, 56, 72, 1e-3
+@pytest.mark.parametrize("qr,kr", [(56, 72), (2200, 40), (300, 2100)])
+def test_latent_norms_go_to_the_query_and_to_the_pool(ext, qr, kr):
+    T, eps, qp, Rp = 9, 1e-3, (qr + 15) // 8 * 8, (kr + 127) // 64 * 64
+    ld = qr + kr + 5
     g = torch.Generator().manual_seed(1)
-    proj = (torch.randn(T, 256, generator=g) * 0.05).to(DEV)
+    proj = (torch.randn(T, ld, generator=g) * 0.05).to(DEV)
     qw, kw = bf(qr, seed=2), bf(kr, seed=3)
-    cq = torch.full((T, 64), 5.0, dtype=torch.bfloat16, device=DEV)
-    pool = torch.full((40, 128), 5.0, dtype=torch.bfloat16, device=DEV)
+    cq = torch.full((T, qp), 5.0, dtype=torch.bfloat16, device=DEV)
+    pool = torch.full((40, Rp), 5.0, dtype=torch.bfloat16, device=DEV)
     slots = torch.randperm(40, generator=g)[:T].to(torch.int32).to(DEV)
     lib, p = ext.load(), ext._p
-    ext._check(lib.js_latent_post(p(proj), 256, qr, kr, p(qw), p(kw), ext.ctypes.c_float(eps), p(cq), 64, p(pool), 128, 40, p(slots), T,
+    ext._check(lib.js_latent_post(p(proj), ld, qr, kr, p(qw), p(kw), ext.ctypes.c_float(eps), p(cq), qp, p(pool), Rp, 40, p(slots), T,
                                   p(ext.status_word(DEV)), 0, ext._stream()), "js_latent_post")
     ext.check_status(DEV)
     rms = lambda x, w: x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps) * w.float()
