@@ -3,6 +3,8 @@
     python bench/kernel_cases.py gemm        # the four decoder GEMM shapes of Qwen3-8B at 128 rows
     python bench/kernel_cases.py gemm_rows2048   # the same shapes at 2048 rows (batched verify / prefill tiles)
     python bench/kernel_cases.py attention   # paged tree attention, 128 nodes over a 1.5k-token prefix
+    python bench/kernel_cases.py latent_attention # latent attention: 16 requests, one token x 32 heads, 2k cached rows of 512
+    python bench/kernel_cases.py parallel_block   # input / output GEMMs of a parallel block at 128 rows (fused epilogues)
     python bench/kernel_cases.py lm_head     # vocabulary GEMM with the argmax epilogue
     python bench/kernel_cases.py nvfp4       # activation quantiser + block-scaled GEMM on the same four shapes
     python bench/kernel_cases.py round_small # RMSNorm, norm+RoPE+KV scatter, draft top-k, tree build, accept+commit, KV compaction
@@ -98,6 +100,29 @@ def case_attention(reps: int = 2):
     torch.cuda.synchronize()
 
 
+def case_latent_attention(reps: int = 3):
+    H, R, B, ctx = 32, 512, 16, 2048
+    S = B * (ctx + 1) + 64
+    pool, qa = bf(S, R), bf(B * H, R)
+    smap = torch.randperm(S, device="cuda").to(torch.int32)[: B * (ctx + 1)].view(B, ctx + 1).contiguous()
+    i32 = dict(dtype=torch.int32, device="cuda")
+    rows, cu, past = torch.arange(B, **i32), torch.arange(B + 1, **i32), torch.full((B,), ctx, **i32)
+    for _ in range(reps):
+        X.latent_attention_rows(qa, pool, H, smap, rows, cu, past, None, 128 ** -0.5, True, 1, max_keys=ctx + 1)
+    torch.cuda.synchronize()
+
+
+def case_parallel_block(reps: int = 3):
+    T, W, lat, attn, ff = 128, 4096, 2048, 4096, 12288
+    h, w_in, w_out = bf(T, W), bf(lat + 2 * ff, W, scale=0.02), bf(W, attn + ff, scale=0.02)
+    raw, cat, x = torch.empty(T, lat, device="cuda"), bf(T, attn + ff), torch.randn(T, W, device="cuda")
+    norm = (torch.ones(W, device="cuda"), torch.zeros(W, device="cuda"), 0.5)
+    for _ in range(reps):
+        X.gemm_inproj(h, w_in, raw, lat, cat[:, attn:], True)
+        X.gemm_resid32(cat, w_out, x, norm=norm, h=h)
+    torch.cuda.synchronize()
+
+
 def case_round_small(reps: int = 2):
     """The small kernels of a decode round at Qwen3-8B sizes: RMSNorm, per-head norm + RoPE + KV scatter, the
     draft head's vocabulary top-k (GEMM epilogue + merge), device tree build, accept + commit, KV compaction."""
@@ -185,7 +210,8 @@ def case_collectives(reps: int = 3):
 
 if __name__ == "__main__":
     X.load()
-    {"gemm": case_gemm, "gemm_rows2048": case_gemm_rows2048, "lm_head": case_lm_head, "attention": case_attention, "nvfp4": case_nvfp4,
+    {"gemm": case_gemm, "gemm_rows2048": case_gemm_rows2048, "lm_head": case_lm_head, "attention": case_attention,
+     "latent_attention": case_latent_attention, "parallel_block": case_parallel_block, "nvfp4": case_nvfp4,
      "round_small": case_round_small, "collectives": case_collectives}[sys.argv[1]]()
     X.check_status("cuda")
     print("ok")

@@ -309,11 +309,16 @@ def draft_head_config(target: Qwen3Config, num_layers: int = 1, block_size: int 
     """Config of a causal-parallel draft head attached to ``target``."""
     from .draft_head import build_target_layer_ids
     ids = target_layer_ids or build_target_layer_ids(target.num_hidden_layers, num_taps)
+    if target.latent_widths() is not None:      # the head keeps its own K/V attention: 128-wide heads over the width
+        n = max(1, target.hidden_size // 128)
+        geometry = dict(intermediate_size=3 * target.hidden_size, num_attention_heads=n, num_key_value_heads=n, head_dim=128,
+                        rms_norm_eps=target.norm_eps)
+    else:
+        geometry = dict(intermediate_size=target.intermediate_size, num_attention_heads=target.num_attention_heads,
+                        num_key_value_heads=target.num_key_value_heads, head_dim=target.head_dim,
+                        rms_norm_eps=target.rms_norm_eps, rope_theta=target.rope_theta)
     return Qwen3Config(
-        vocab_size=target.vocab_size, hidden_size=target.hidden_size,
-        intermediate_size=target.intermediate_size, num_hidden_layers=num_layers,
-        num_attention_heads=target.num_attention_heads, num_key_value_heads=target.num_key_value_heads,
-        head_dim=target.head_dim, rms_norm_eps=target.rms_norm_eps, rope_theta=target.rope_theta,
+        vocab_size=target.vocab_size, hidden_size=target.hidden_size, num_hidden_layers=num_layers, **geometry,
         block_size=block_size, num_target_layers=target.num_hidden_layers,
         dflash_config={"causal_head": causal_head, "target_layer_ids": list(ids),
                        "target_hidden_size": target.hidden_size,

@@ -100,7 +100,7 @@ def latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, m
 
 
 def sigmoid_moe(x, router_w, correction, w_up, w_down, top, scale):
-    if _kern_any(x):
+    if _kern_any(x) and correction.numel() <= 1024 and top <= 32:      # what the routing kernel covers
         wts, idx = _ext().sigmoid_route(ref.linear(x.float(), router_w.float()), correction, top, scale)
         return ref.experts_relu_squared(x, wts, idx.long(), w_up, w_down)
     return ref.sigmoid_moe(x, router_w, correction, w_up, w_down, top, scale)

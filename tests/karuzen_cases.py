@@ -51,6 +51,8 @@ def cases():
         # a loop that runs once; nothing is a multiple of 8
         "ragged": config(100, 333, [(mixer(5, 18, 22, 30, 50), dense(36)), (mixer(5, 18, 22, 30, 50), moe(9, 2, 20, 2.0, shared=28))],
                          loop=(0, 1, 1)),
+        # a latent wider than the tensor-core attention takes, more experts than a warp has lanes
+        "broad": config(64, 120, [(mixer(2, 12, 12, 20, 520), moe(70, 6, 16, 1.1, shared=16)), (mixer(3, 8, 16, 24, 24), dense(48))]),
         # heads wide enough for the expanded form of long portions, a latent of five lines (two column groups)
         "wide": config(128, 200, [(wide, moe(6, 2, 64, 1.2, shared=64)), (wide, dense(96))], loop=(0, 1, 2)),
     }

@@ -145,7 +145,7 @@ def test_whole_prompt_and_residual_stream(arm, case):
 
 @pytest.mark.parametrize("arm", ARMS)
 @pytest.mark.parametrize("case,sizes", [("mixed", [1]), ("mixed", [2]), ("mixed", [5, 2, 17]), ("routed", [3]), ("plain", [16, 1, 15]),
-                                        ("ragged", [2, 31]), ("wide", [130, 1, 1, 2]), ("wide", [7])])
+                                        ("ragged", [2, 31]), ("broad", [9, 1]), ("wide", [130, 1, 1, 2]), ("wide", [7])])
 def test_portions_of_any_size_equal_the_whole(arm, case, sizes):
     """Prefill against token-by-token decoding and against portions cut inside and at the borders of pages."""
     cfg, w = CASES[case], WEIGHTS[case]
@@ -305,6 +305,38 @@ def test_sampling_follows_the_distribution(arm):
     top = set(probs.topk(20).indices.tolist())
     mass, hit = float(probs.topk(20).values.sum()), sum(t in top for t in draws) / n
     assert abs(hit - mass) < 4 * math.sqrt(mass * (1 - mass) / n) + 0.02
+
+
+@pytest.mark.parametrize("arm", ARMS)
+def test_draft_head_and_sampled_trees(arm):
+    """A draft head conditioned on tapped layer runs (inside the round graph on the GPU) stays lossless; sampled rounds run."""
+    from jetspec_b200 import DraftHeadTreeDrafter, RandomTreeDrafter, SamplingParams
+    from jetspec_b200.models import DraftHeadModel, draft_head_config
+    mix = mixer(3, 40, 24, 56, 72)
+    cfg = config(256, 211, [(mix, dense(160)), (mix, moe(6, 2, 48, 1.3, shared=40)), (mix, None)], loop=(0, 2, 2))
+    w = margin_weights(cfg, 21)
+    eng = engine_from(cfg, w, arm, max_seq_len=512)
+    p = prompt(21, cfg["vocab"])
+    want = K.greedy(p, w, cfg, 8)
+    head = DraftHeadModel.random_init(draft_head_config(eng.cfg, 1, 5, target_layer_ids=[0, 1, 4]), seed=1, dtype=arm[1], device=arm[0])
+    kw = dict(tree_depth=4, tree_width=2, budget=8)
+    d = DraftHeadTreeDrafter(head, eng.model, block_size=5)
+    t = torch.tensor([p])
+    assert eng.generate_tree(t, d, target_layer_ids=head.target_layer_ids, sampling_params=SamplingParams(0.0, 8), **kw)["token_ids"] == want
+    out = eng.generate_tree(t, RandomTreeDrafter(cfg["vocab"], seed=2), sampling_params=SamplingParams(1.0, 8), **kw)["token_ids"]
+    assert len(out) == 8 and all(0 <= x < cfg["vocab"] for x in out)
+
+
+@pytest.mark.gpu
+def test_experts_in_several_passes(monkeypatch):
+    """More (token, expert) pairs than one permutation launch takes: the tokens go through the experts in passes."""
+    from jetspec_b200.engine import latent_stack
+    monkeypatch.setattr(latent_stack, "MAX_SORT_PAIRS", 21)
+    cfg, w, arm = CASES["mixed"], WEIGHTS["mixed"], ("cuda", torch.bfloat16)
+    toks = prompt(37, cfg["vocab"])
+    eng = engine_from(cfg, w, arm)
+    eng.reserve_pool(64, 1)
+    assert_rows(replay(eng, [[("a", 37)]], {"a": toks})["a"], oracle_logits("mixed", cfg, w, toks), arm[1])
 
 
 def test_tree_visibility_matches_the_oracle():
