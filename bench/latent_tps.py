@@ -200,8 +200,7 @@ def kernel_table(T, context, n_seq):
                   H * R * 2, "qwen3 o GEMM + residual")
         gemm_case("karuzen W_uv behind the attention (batched over heads)", H * D, R, lambda w: X.gemm_batched(ol, w, cat, H, D, R, R, D, cat.stride(0)),
                   H * (R + D) * 2, "qwen3 o GEMM + residual")
-        tiles = min(T * H // 128 + n_seq, n_seq * ((per * H + 127) // 128))
-        sp = X.latent_attn_splits(tiles, R, context + per)
+        sp = X.latent_attn_splits(T, H, n_seq, per, R, context + per)
         add(f"karuzen latent attention ({sp} splits)", [lambda l=l: X.latent_attention_rows(
             qa.view(T * H, R), l, H, smap, srow, cu, past, None, D ** -0.5, True, per, out=ol.view(T * H, R), splits=sp) for l in lp],
             tot * R * 2 + T * H * R * 4, 4 * keys * H * R, 8, "qwen3 attention")

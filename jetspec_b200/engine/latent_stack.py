@@ -236,8 +236,7 @@ class LatentStack:
         X.gemm_batched(q[r0:r1], L.uk_t, qa, H, L.rp, L.dp, L.dp, L.rp, H * L.rp, pdl=pdl)
         rows = T * H
         tc = L.rp <= X.LATENT_TC_MAX and (batch.mask is None or batch.mask.shape[1] <= 8)
-        splits = X.latent_attn_splits(min(rows // 128 + part.seqs, part.seqs * ((part.max_q * H + 127) // 128)), L.rp,
-                                      part.max_keys) if tc else 1
+        splits = X.latent_attn_splits(T, H, part.seqs, part.max_q, L.rp, part.max_keys) if tc else 1
         X.latent_attention_rows(qa.view(rows, L.rp), pool, H, batch.slot_map, part.seq_rows, part.cu_q, part.past,
                                 None if batch.mask is None else batch.mask[r0:r1], L.scale, batch.causal, part.max_q,
                                 out=ol.view(rows, L.rp), splits=splits, ws=self._attn_ws(st, splits, rows, L.rp), pdl=pdl,

@@ -754,8 +754,10 @@ def latent_scatter(c: torch.Tensor, pool: torch.Tensor, slots: torch.Tensor) -> 
 LATENT_TC_MAX = 512        # widest latent row of the tensor-core kernel
 
 
-def latent_attn_splits(tiles: int, Rp: int, max_keys: int) -> int:
-    """Key splits of the tensor-core latent attention: one wave of CTAs, at least a couple of key tiles each."""
+def latent_attn_splits(T: int, heads: int, seqs: int, max_q: int, Rp: int, max_keys: int) -> int:
+    """Key splits of the tensor-core latent attention: one wave of CTAs (128 query rows of one sequence each, two column
+    groups for latents wider than 256), at least a couple of key tiles each."""
+    tiles = min(T * heads // 128 + seqs, seqs * ((max_q * heads + 127) // 128))
     ctas = max(1, tiles * (2 if Rp > 256 else 1))
     return max(1, min(SM_COUNT // ctas, (max_keys + 127) // 128, 16))
 
@@ -783,7 +785,7 @@ def latent_attention_rows(qa: torch.Tensor, pool: torch.Tensor, heads: int, slot
                "js_latent_attention_simt")
         return out
     if splits is None:
-        splits = latent_attn_splits(rows // 128 + B, Rp, max_keys if max_keys is not None else slot_map.shape[1])
+        splits = latent_attn_splits(T, heads, B, max_q, Rp, max_keys if max_keys is not None else slot_map.shape[1])
     if splits > 1 and ws is None:
         ws = {"o": torch.empty(splits, rows, Rp, dtype=torch.float32, device=qa.device),
               "ml": torch.empty(splits, rows, 2, dtype=torch.float32, device=qa.device)}
