@@ -19,7 +19,6 @@ import sys
 import torch
 
 LIVE_REQUESTS = 4        # slot-map rows of the replay's pool: no more requests are live at any time
-ROUND_TOKENS = 64        # a live request holds its tokens rounded up to this many
 
 
 class TraceReplay:

@@ -1,8 +1,8 @@
 """Karuzen decoder: parallel blocks, Dynamic Tanh norms, latent attention, looped layers, tied embeddings.
 
-One norm per layer; the mixer and the feed-forward read its output and both are added to the residual stream, which is
-kept in 32-bit.  A range of layers runs several times with the same weights: every run is a cache layer of its own, and
-the embedding output is added to the stream before each pass but the first.  ``forward`` has the contract of
+A block normalises the fp32 residual stream once, hands the result to its mixer and its feed-forward side by side and
+adds what both return.  A range of blocks can be traversed repeatedly with shared weights; each traversal writes cache
+layers of its own, and every later one starts by adding the token embeddings to the stream.  ``forward`` has the contract of
 :meth:`jetspec_b200.models.qwen3.Qwen3ForCausalLM.forward`, so the engines drive both families alike; layer numbers
 (taps, cache layers) count layer RUNS.
 """

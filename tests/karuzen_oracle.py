@@ -78,7 +78,7 @@ def moe_mlp(h, w, p, mlp):
 
 
 def layer(x, w, i, cfg, visible=None):
-    """Parallel block: one norm, both sublayers read its output, both are added."""
+    """``x + mixer(h) + ff(h)`` with ``h`` the block's single normalised input."""
     L, p = cfg["layers"][i], f"l{i}"
     h = dynamic_tanh(x, w[p + ".norm1.alpha"], w[p + ".norm1"], w[p + ".norm1.b"])
     y = latent_attention(h, w, p + ".mix", L["mixer"], cfg["norm"]["eps"], visible)

@@ -146,7 +146,7 @@ def latent_case(H, R, counts, pasts, tree, seed=0, dtype=torch.bfloat16, page=16
                 want=d(want).view(T * H, Rp), max_q=max(counts), max_keys=max(lens))
 
 
-CASES = [(4, 96, [1], [300]), (3, 72, [1, 1, 1, 1], [0, 63, 64, 200]), (5, 40, [130, 2, 33], [0, 65, 31]), (16, 320, [3, 1], [127, 500]),
+CASES = [(6, 104, [1], [300]), (3, 72, [1, 1, 1, 1], [0, 63, 64, 200]), (5, 40, [130, 2, 33], [0, 65, 31]), (16, 320, [3, 1], [127, 500]),
          (32, 512, [1, 1], [600, 15]), (12, 512, [40, 7], [100, 0]), (128, 256, [2, 1], [70, 129]), (1, 64, [200], [57]),
          (7, 192, [19], [1000])]
 
@@ -173,7 +173,7 @@ def test_latent_attention_plain_cores(ext, H, R, counts, pasts, dtype, tol, tree
     close(out, c["want"], tol)
 
 
-@pytest.mark.parametrize("T,E,k", [(5, 16, 4), (300, 6, 2), (9, 200, 8), (40, 700, 1), (3, 4, 4)])
+@pytest.mark.parametrize("T,E,k", [(5, 18, 3), (300, 6, 2), (9, 200, 8), (40, 700, 1), (3, 4, 4)])
 def test_sigmoid_routing_and_shared_gate(ext, T, E, k):
     from jetspec_b200.ops import reference as ref
     g = torch.Generator().manual_seed(T)
