@@ -1,12 +1,13 @@
-"""Model configurations read from ``config.json``: Qwen3 (Hugging Face layout) and Karuzen.
+"""Model configurations read from ``config.json``: Qwen3 (Hugging Face layout), Karuzen and Zasipel.
 
 Only the fields the decoder actually uses are kept.  The draft head adds
 ``block_size``, ``num_target_layers`` and ``dflash_config`` on top of the Qwen3
 fields (reference: ``jetspec/models/draft_head.py:317-337``).
 
 What the engines, the cache and the kernel path ask of a configuration, whatever the family: ``vocab_size``,
-``hidden_size``, ``num_hidden_layers`` (layer RUNS, i.e. cache layers), ``eos_token_id``, ``latent_widths()`` (``None``
-for a K/V cache) and ``kernel_path_ok()``.
+``hidden_size``, ``num_hidden_layers`` (layer RUNS, i.e. cache layers), ``eos_token_id``, ``kernel_path_ok()`` and what a
+cache layer holds: ``latent_widths()`` (``None`` unless every layer caches one latent row a token), ``kv_shapes()``
+(``None`` when all layers hold the same K and V heads) and ``state_shapes()`` (``None`` without recurrent layers).
 """
 from __future__ import annotations
 
@@ -72,6 +73,14 @@ class Qwen3Config:
 
     def latent_widths(self) -> Optional[list]:
         """Widths of the latent rows a cache layer holds, or ``None`` when it holds K and V heads."""
+        return None
+
+    def kv_shapes(self) -> Optional[list]:
+        """Per layer ``(kv_heads, dim, vdim)`` or ``None`` (nothing cached), when layers differ; else ``None``."""
+        return None
+
+    def state_shapes(self) -> Optional[list]:
+        """Per layer the :class:`DeltaConfig` whose state a sequence carries, or ``None``; ``None`` without any."""
         return None
 
     def kernel_path_ok(self) -> bool:
@@ -193,6 +202,12 @@ class KaruzenConfig:
     def latent_widths(self) -> list:
         return [self.layers[i].mixer.kv_rank for i, _ in self.layer_runs()]
 
+    def kv_shapes(self) -> None:
+        return None
+
+    def state_shapes(self) -> None:
+        return None
+
     def kernel_path_ok(self) -> bool:
         return all(l.moe is None or (l.moe.experts <= 1024 and l.moe.top <= 32) for l in self.layers)
 
@@ -256,6 +271,178 @@ class KaruzenConfig:
             json.dump(self.to_dict(), f, indent=1)
 
 
+
+@dataclass
+class WindowAttentionConfig:
+    """Sizes and constants of a sliding-window attention over grouped K/V heads: a token sees itself and the
+    ``window - 1`` tokens before it; the first ``rot_dims`` dimensions are rotated in neighbouring pairs."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    window: int
+    rot_dims: int
+    rot_base: float
+    scale: float
+    sink: bool = True                # a valueless key of score 0 takes part in the softmax
+    qk_norm: bool = True             # weightless RMS norm of q and k behind the rotation
+    bias: bool = True                # biases on all four projections
+
+
+@dataclass
+class DeltaConfig:
+    """Sizes of a gated delta rule.  ``decay``: one per ``"head"`` or per ``"channel"`` of the key; ``gate``: activation
+    of the output gate.  A rank of 0 makes that projection a single matrix, else it goes through that rank."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    taps: int
+    decay: str = "head"
+    gate: str = "silu"
+    decay_rank: int = 0
+    gate_rank: int = 0
+
+    @property
+    def channels(self) -> int:
+        """Channels of the short convolution: q, k and v side by side."""
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+    @property
+    def decays(self) -> int:
+        return self.heads * (self.dim if self.decay == "channel" else 1)
+
+
+@dataclass
+class TableExpertsConfig:
+    """Experts a table of token ids names, with equal weights; ``shared_ff`` is 0 without a shared expert."""
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0
+
+
+@dataclass
+class ZasipelLayerConfig:
+    """``window`` beside ``delta`` (a parallel layer), or ``delta`` alone."""
+    delta: DeltaConfig
+    window: Optional[WindowAttentionConfig] = None
+    moe: Optional[TableExpertsConfig] = None        # None: no feed-forward
+
+    @property
+    def mixer_type(self) -> str:
+        return "parallel" if self.window is not None else "channel_delta"
+
+
+@dataclass
+class ZasipelConfig:
+    """Zasipel: window attention and a gated delta rule side by side, or a channel-decay delta rule alone; experts chosen
+    by token id; norms on the sublayers' outputs only; untied head."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float = 1e-6
+    eos_token_id: Any = None
+    model_type: str = "zasipel"
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def is_moe(self) -> bool:
+        return any(l.moe is not None for l in self.layers)
+
+    def latent_widths(self) -> None:
+        return None
+
+    def kv_shapes(self) -> list:
+        return [(l.window.kv_heads, l.window.dim, l.window.vdim) if l.window is not None else None for l in self.layers]
+
+    def state_shapes(self) -> list:
+        return [l.delta for l in self.layers]
+
+    def kernel_path_ok(self) -> bool:
+        return all(l.delta.dim <= 256 and l.delta.vdim <= 256 and l.delta.taps <= 17
+                   and (l.window is None or (l.window.dim <= 512 and l.window.vdim <= 512))
+                   and (l.moe is None or l.moe.experts <= 1024) for l in self.layers)
+
+    # -- io -------------------------------------------------------------------
+    @classmethod
+    def from_dict(cls, d: dict, shape_of=None) -> "ZasipelConfig":
+        """``shape_of(tensor name)`` gives the two low ranks of a channel-decay layer, which only the weights tell
+        (without it: a quarter of the head size)."""
+        def delta(m, p, decay):
+            c = DeltaConfig(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                            taps=int(m["conv"]), decay=decay, gate="silu" if decay == "head" else "sigmoid")
+            if decay == "channel":
+                rank = lambda n, e: int(shape_of(p + n)[0]) if shape_of is not None else max(1, e // 4)
+                c.decay_rank, c.gate_rank = rank(".a1", c.dim), rank(".g1", c.vdim)
+            return c
+
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            m, f, p = e["mixer"], e.get("mlp"), f"l{i}.mix"
+            if e["type"] == "parallel":
+                a = m["left"]
+                lc = ZasipelLayerConfig(delta(m["right"], p + ".right", "head"), window=WindowAttentionConfig(
+                    heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]), vdim=int(a["vdim"]),
+                    window=int(a["mask"]["size"]), rot_dims=int(a["rot"]["dims"]), rot_base=float(a["rot"]["base"]),
+                    scale=float(a["scale"])))
+            elif e["type"] == "channel_delta":
+                lc = ZasipelLayerConfig(delta(m, p, "channel"))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {e['type']!r}")
+            for c in (lc.delta, lc.window):
+                if c is not None and c.heads % c.kv_heads:
+                    raise ValueError(f"layer {i}: {c.heads} heads do not divide over {c.kv_heads} key heads")
+            if f is not None:
+                if f["kind"] != "moe":
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+                r, sh = f["router"], f.get("shared")
+                lc.moe = TableExpertsConfig(experts=int(r["experts"]), top=int(r["top"]), ff=int(f["expert"]["ff"]),
+                                            shared_ff=int(sh["ff"]) if sh else 0)
+            layers.append(lc)
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers,
+                   norm_eps=float(d["norm"]["eps"]), eos_token_id=d.get("eos_token_id"))
+
+    @classmethod
+    def from_pretrained(cls, path: str, subfolder: str = "") -> "ZasipelConfig":
+        from .loader import tensor_shape
+        base = os.path.join(path, subfolder) if subfolder else path
+        with open(os.path.join(base, "config.json")) as f:
+            return cls.from_dict(json.load(f), shape_of=lambda name: tensor_shape(base, name))
+
+    def to_dict(self) -> dict:
+        def delta(c):
+            return {"heads": c.heads, "kv_heads": c.kv_heads, "dim": c.dim, "vdim": c.vdim, "conv": c.taps}
+
+        layers = []
+        for l in self.layers:
+            mixer = delta(l.delta)
+            if l.window is not None:
+                a = l.window
+                mixer = {"left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale,
+                                  "mask": {"size": a.window}, "rot": {"dims": a.rot_dims, "base": a.rot_base}},
+                         "right": mixer}
+            mlp = None
+            if l.moe is not None:
+                mlp = {"kind": "moe", "expert": {"ff": l.moe.ff}, "router": {"experts": l.moe.experts, "top": l.moe.top}}
+                if l.moe.shared_ff:
+                    mlp["shared"] = {"ff": l.moe.shared_ff}
+            layers.append({"type": l.mixer_type, "mixer": mixer, "mlp": mlp})
+        d = {"architecture": "Zasipel", "vocab": self.vocab_size, "width": self.hidden_size, "layers": layers,
+             "norm": {"eps": self.norm_eps}}
+        if self.eos_token_id is not None:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    def save_pretrained(self, path: str) -> None:
+        os.makedirs(path, exist_ok=True)
+        with open(os.path.join(path, "config.json"), "w") as f:
+            json.dump(self.to_dict(), f, indent=1)
+
+
 # Geometry presets used by the tests and the benchmarks (random-init weights).
 def tiny_config(**over) -> Qwen3Config:
     """2 layers, hidden 256, 4 q / 2 kv heads, head_dim 64, SwiGLU 512, vocab 1024."""
@@ -303,13 +490,25 @@ def karuzen_bench_config(layers: int = 16, moe: bool = False, **over) -> Karuzen
     return KaruzenConfig(**kw)
 
 
+def zasipel_tiny_config(**over) -> ZasipelConfig:
+    """3 layers (parallel, channel decay, parallel without a feed-forward); width 160."""
+    win = WindowAttentionConfig(heads=6, kv_heads=2, dim=24, vdim=40, window=21, rot_dims=12, rot_base=1e4, scale=0.3)
+    head = DeltaConfig(heads=4, kv_heads=2, dim=16, vdim=32, taps=4)
+    chan = DeltaConfig(heads=3, kv_heads=3, dim=24, vdim=16, taps=4, decay="channel", gate="sigmoid", decay_rank=10, gate_rank=6)
+    moe = TableExpertsConfig(experts=6, top=3, ff=40, shared_ff=56)
+    kw = dict(vocab_size=320, hidden_size=160, norm_eps=1e-5,
+              layers=[ZasipelLayerConfig(head, win, moe), ZasipelLayerConfig(chan, None, moe), ZasipelLayerConfig(head, win, None)])
+    kw.update(over)
+    return ZasipelConfig(**kw)
+
+
 def draft_head_config(target: Qwen3Config, num_layers: int = 1, block_size: int = 16,
                       target_layer_ids: Optional[list] = None, mask_token_id: Optional[int] = None,
                       num_taps: int = 5, causal_head: bool = True) -> Qwen3Config:
     """Config of a causal-parallel draft head attached to ``target``."""
     from .draft_head import build_target_layer_ids
     ids = target_layer_ids or build_target_layer_ids(target.num_hidden_layers, num_taps)
-    if target.latent_widths() is not None:      # the head keeps its own K/V attention: 128-wide heads over the width
+    if not hasattr(target, "head_dim"):         # the head keeps its own K/V attention: 128-wide heads over the width
         n = max(1, target.hidden_size // 128)
         geometry = dict(intermediate_size=3 * target.hidden_size, num_attention_heads=n, num_key_value_heads=n, head_dim=128,
                         rms_norm_eps=target.norm_eps)

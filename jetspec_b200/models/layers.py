@@ -1,9 +1,10 @@
-"""Building blocks that are not Qwen3's: Dynamic Tanh, latent attention, tanh-GELU MLP, sigmoid-routed experts.
+"""Building blocks that are not Qwen3's: Dynamic Tanh, latent attention, tanh-GELU MLP, sigmoid-routed experts; window
+attention with a sink, gated delta rules, two mixers side by side, table-routed experts.
 
 Each takes its sizes and constants as arguments, so a design can combine them freely; the Qwen3 twins (RMSNorm, grouped
 query attention, SwiGLU MLP, softmax-routed experts) are in :mod:`jetspec_b200.models.qwen3`.  ``forward`` is the
-unfused form on :mod:`jetspec_b200.ops`, in any dtype and on any device; the fused kernel form of a whole decoder made
-of these blocks is :mod:`jetspec_b200.engine.latent_stack`.
+unfused form on :mod:`jetspec_b200.ops`, in any dtype and on any device; the fused kernel forms of whole decoders made
+of these blocks are :mod:`jetspec_b200.engine.latent_stack` and :mod:`jetspec_b200.engine.hybrid_stack`.
 """
 from __future__ import annotations
 
@@ -11,7 +12,7 @@ import torch
 import torch.nn as nn
 
 from .. import ops
-from .config import LatentAttentionConfig, RoutedExpertsConfig
+from .config import DeltaConfig, LatentAttentionConfig, RoutedExpertsConfig, TableExpertsConfig, WindowAttentionConfig
 
 
 class DynamicTanh(nn.Module):
@@ -88,4 +89,117 @@ class SigmoidMoE(nn.Module):
             s = ops.linear(ops.relu_squared(ops.linear(h, self.shared_up.weight)), self.shared_down.weight)
             gate = torch.sigmoid(h.float() @ self.shared_gate.weight.float().t())
             y = y + gate * s.float()
+        return y
+
+
+class PlainRMSNorm(nn.Module):
+    """RMS norm of fp32 rows; 32-bit math and output."""
+
+    def __init__(self, dim: int, eps: float):
+        super().__init__()
+        self.eps = eps
+        self.weight = nn.Parameter(torch.ones(dim))
+
+    def forward(self, x):
+        return ops.rmsnorm_f32(x, self.weight, self.eps)
+
+
+class WindowAttention(nn.Module):
+    """Sliding-window attention over grouped K/V heads: rotation of the first dimensions in neighbouring pairs, optional
+    weightless norm of q and k behind it, optional valueless sink of score 0, optional biases.
+
+    ``forward(h, positions, attend)``: ``attend(q, k, v)`` stores the new K/V rows and returns the attention,
+    ``(T, heads * vdim)``."""
+
+    def __init__(self, cfg: WindowAttentionConfig, hidden: int, eps: float):
+        super().__init__()
+        self.cfg, self.eps = cfg, eps
+        lin = lambda i, o: nn.Linear(i, o, bias=cfg.bias)
+        self.q_proj, self.k_proj = lin(hidden, cfg.heads * cfg.dim), lin(hidden, cfg.kv_heads * cfg.dim)
+        self.v_proj, self.o_proj = lin(hidden, cfg.kv_heads * cfg.vdim), lin(cfg.heads * cfg.vdim, hidden)
+
+    def forward(self, h, positions, attend):
+        c, T = self.cfg, h.shape[0]
+        q, k, v = (ops.linear(h, p.weight, p.bias) for p in (self.q_proj, self.k_proj, self.v_proj))
+        q, k = (ops.rotate_norm(x.view(T, n, c.dim), positions, c.rot_dims, c.rot_base, self.eps if c.qk_norm else None)
+                for x, n in ((q, c.heads), (k, c.kv_heads)))
+        return ops.linear(attend(q, k, v.view(T, c.kv_heads, c.vdim)), self.o_proj.weight, self.o_proj.bias)
+
+
+class GatedDelta(nn.Module):
+    """Gated delta rule: short causal convolutions on q, k and v, unit-norm keys and queries, a decay per head or per key
+    channel, gated per-head norm of the read-outs.
+
+    ``forward(h, recur)``: ``recur(pre, z, b)`` advances the sequences' states by the un-convolved rows ``pre (T,
+    channels)``, the decay inputs ``z`` and the step-size inputs ``b`` and returns the read-outs, fp32 ``(T, heads, vdim)``."""
+
+    def __init__(self, cfg: DeltaConfig, hidden: int, eps: float):
+        super().__init__()
+        self.cfg, self.eps = cfg, eps
+        lin = lambda i, o: nn.Linear(i, o, bias=False)
+        kd, vd = cfg.kv_heads * cfg.dim, cfg.heads * cfg.vdim
+        self.q_proj, self.k_proj, self.v_proj = lin(hidden, kd), lin(hidden, kd), lin(hidden, vd)
+        self.q_conv, self.k_conv = nn.Parameter(torch.zeros(kd, cfg.taps)), nn.Parameter(torch.zeros(kd, cfg.taps))
+        self.v_conv = nn.Parameter(torch.zeros(vd, cfg.taps))
+        self.beta_proj = lin(hidden, cfg.heads)
+        self.A_log, self.dt_bias = nn.Parameter(torch.zeros(cfg.heads)), nn.Parameter(torch.zeros(cfg.decays))
+        if cfg.decay_rank:
+            self.decay_down, self.decay_up = lin(hidden, cfg.decay_rank), lin(cfg.decay_rank, cfg.decays)
+        else:
+            self.decay_proj = lin(hidden, cfg.decays)
+        if cfg.gate_rank:
+            self.gate_down, self.gate_up = lin(hidden, cfg.gate_rank), lin(cfg.gate_rank, vd)
+        else:
+            self.gate_proj = lin(hidden, vd)
+        self.o_norm = nn.Parameter(torch.ones(cfg.vdim))
+        self.o_proj = lin(vd, hidden)
+
+    def conv(self) -> torch.Tensor:
+        """Convolution taps of all channels, ``(channels, taps)``, in the order of ``pre``."""
+        return torch.cat((self.q_conv, self.k_conv, self.v_conv), 0)
+
+    def forward(self, h, recur):
+        c = self.cfg
+        lin = ops.linear
+        pre = torch.cat([lin(h, p.weight) for p in (self.q_proj, self.k_proj, self.v_proj)], -1)
+        b = ops.linear_f32(h, self.beta_proj.weight)
+        z = (ops.linear_f32(lin(h, self.decay_down.weight), self.decay_up.weight) if c.decay_rank
+             else ops.linear_f32(h, self.decay_proj.weight))
+        gate = lin(lin(h, self.gate_down.weight), self.gate_up.weight) if c.gate_rank else lin(h, self.gate_proj.weight)
+        y = ops.gated_head_norm(recur(pre, z, b), self.o_norm, gate, c.gate, self.eps)
+        return lin(y, self.o_proj.weight)
+
+
+class SideBySide(nn.Module):
+    """Window attention and a gated delta rule on the same input: half the sum of the two outputs, each RMS-normed over
+    the width first.  Returns fp32."""
+
+    def __init__(self, window: WindowAttentionConfig, delta: DeltaConfig, hidden: int, eps: float):
+        super().__init__()
+        self.left, self.right = WindowAttention(window, hidden, eps), GatedDelta(delta, hidden, eps)
+        self.left_norm, self.right_norm = PlainRMSNorm(hidden, eps), PlainRMSNorm(hidden, eps)
+
+    def forward(self, h, positions, attend, recur):
+        a = self.left_norm(self.left(h, positions, attend).float())
+        return 0.5 * (a + self.right_norm(self.right(h, recur).float()))
+
+
+class TableMoE(nn.Module):
+    """SwiGLU experts named by a table of token ids, equal weights, plus a SwiGLU shared expert.  Returns fp32."""
+
+    def __init__(self, cfg: TableExpertsConfig, hidden: int, vocab: int):
+        super().__init__()
+        self.cfg = cfg
+        self.w_gate, self.w_up = (nn.Parameter(torch.empty(cfg.experts, cfg.ff, hidden)) for _ in range(2))
+        self.w_down = nn.Parameter(torch.empty(cfg.experts, hidden, cfg.ff))
+        self.register_buffer("table", torch.zeros(vocab, cfg.top, dtype=torch.int32))
+        if cfg.shared_ff:
+            self.shared_gate, self.shared_up = (nn.Linear(hidden, cfg.shared_ff, bias=False) for _ in range(2))
+            self.shared_down = nn.Linear(cfg.shared_ff, hidden, bias=False)
+
+    def forward(self, h, ids):
+        y = ops.experts_swiglu(h, self.table[ids], self.w_gate, self.w_up, self.w_down)
+        if self.cfg.shared_ff:
+            a = torch.cat((ops.linear(h, self.shared_gate.weight), ops.linear(h, self.shared_up.weight)), -1)
+            y = y + ops.linear(ops.silu_mul(a), self.shared_down.weight).float()
         return y

@@ -33,6 +33,16 @@ def _checkpoint_files(path: str) -> list[str]:
     return [os.path.join(path, x) for x in files]
 
 
+def tensor_shape(path: str, name: str) -> tuple:
+    """Shape of one checkpoint tensor, from the file headers alone."""
+    from safetensors import safe_open
+    for fn in _checkpoint_files(path):
+        with safe_open(fn, framework="pt", device="cpu") as f:
+            if name in f.keys():
+                return tuple(f.get_slice(name).get_shape())
+    raise KeyError(f"no tensor {name!r} under {path}")
+
+
 @torch.no_grad()
 def load_state_into(module: torch.nn.Module, path: str, remap: Optional[Callable] = None,
                     strict: bool = True, prefix_strip: str = "") -> None:
@@ -71,7 +81,7 @@ def load_state_into(module: torch.nn.Module, path: str, remap: Optional[Callable
                 lost = sorted(want - got)[:4]
                 raise KeyError(f"stacked parameter {name!r} is missing {len(want - got)} of {len(want)} slices "
                                f"(first: {lost})")
-        missing = [n for n, p in module.named_parameters() if n not in seen]
+        missing = [n for n in module.state_dict() if n not in seen]
         # a tied lm_head is legitimately absent from the file
         missing = [n for n in missing if n != "lm_head.weight"]
         if missing:

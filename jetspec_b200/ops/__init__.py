@@ -106,6 +106,56 @@ def sigmoid_moe(x, router_w, correction, w_up, w_down, top, scale):
     return ref.sigmoid_moe(x, router_w, correction, w_up, w_down, top, scale)
 
 
+def rmsnorm_f32(x, weight, eps):
+    if x.is_cuda and x.dtype == torch.float32:
+        return _ext().rmsnorm_f32(x, weight, eps)
+    return ref.rmsnorm_f32(x, weight, eps)
+
+
+def linear_f32(x, w):
+    if _kern(x):
+        from . import cuda_ext
+        if cuda_ext.gemm_supported(x.shape[0], w.shape[0], x.shape[1]):
+            return cuda_ext.gemm(x.contiguous(), w, epi=cuda_ext.EPI_STORE_F32)
+    return ref.linear_f32(x, w)
+
+
+def rotate_norm(x, positions, dims, base, eps):
+    if _kern_any(x):
+        return _ext().rotate_norm(x, positions, dims, base, eps)
+    return ref.rotate_norm(x, positions, dims, base, eps)
+
+
+def window_scatter(k, v, k_pool, v_pool, slots):
+    return ref.window_scatter(k, v, k_pool, v_pool, slots)
+
+
+def window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, window, sink,
+                     causal: bool = False):
+    if _kern_any(q) and max(q.shape[-1], vdim) <= 512:
+        return _ext().window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, float(scale),
+                                       int(window), bool(sink), bool(causal))
+    return ref.window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, window, sink,
+                                causal)
+
+
+def delta_mix(pre, z, b, taps, A_log, dt_bias, cfg, state, conv, rows, cu_q, past_lens, mask_bits, causal: bool = True):
+    if _kern_any(pre) and cfg.dim <= 256 and cfg.taps <= 17:
+        return _ext().delta_mix(pre, z, b, taps, A_log, dt_bias, cfg, state, conv, rows, cu_q, past_lens, mask_bits,
+                                bool(causal))
+    return ref.delta_mix(pre, z, b, taps, A_log, dt_bias, cfg, state, conv, rows, cu_q, past_lens, mask_bits, causal)
+
+
+def gated_head_norm(o, weight, gate, kind, eps):
+    if _kern_any(gate):
+        return _ext().gated_head_norm(o, weight, gate, kind, eps)
+    return ref.gated_head_norm(o, weight, gate, kind, eps)
+
+
+def experts_swiglu(x, idx, w_gate, w_up, w_down):
+    return ref.experts_swiglu(x, idx, w_gate, w_up, w_down)
+
+
 def qkv_postprocess(qkv, q_norm_w, k_norm_w, positions, num_q_heads, num_kv_heads, head_dim, theta, eps):
     if _kern(qkv) and head_dim == 128:
         ext = _ext()
@@ -160,5 +210,7 @@ __all__ = [
     "rmsnorm", "add_rmsnorm", "linear", "silu_mul", "qkv_postprocess", "kv_scatter",
     "paged_tree_attention", "lm_head_argmax", "lm_head_topk_logprobs", "moe_forward",
     "dynamic_tanh", "gelu_tanh_mul", "relu_squared", "latent_scatter", "latent_attention", "sigmoid_moe",
+    "rmsnorm_f32", "linear_f32", "rotate_norm", "window_scatter", "window_attention", "delta_mix", "gated_head_norm",
+    "experts_swiglu",
     "pack_ancestor_bits", "unpack_ancestor_bits", "rope_cos_sin", "apply_rope", "moe_route", "sample",
 ]

@@ -317,3 +317,150 @@ def sample(logits: torch.Tensor, temperature: float = 0.0, generator=None) -> to
     probs = torch.softmax(logits.float() / temperature, dim=-1)
     flat = probs.reshape(-1, probs.shape[-1])
     return torch.multinomial(flat, 1, generator=generator).reshape(probs.shape[:-1])
+
+
+# --------------------------------------------------------------------------
+# window attention, gated delta rules, table-routed experts
+# --------------------------------------------------------------------------
+def rmsnorm_f32(x: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """RMS norm of fp32 rows, fp32 result."""
+    x = x.float()
+    return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+
+
+def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``x @ w.T`` with the product left in fp32."""
+    return F.linear(x.float(), w.float())
+
+
+def pair_freq(dims: int, base: float, device=None) -> torch.Tensor:
+    """``base^(-2i/dims)`` for the ``dims // 2`` rotated pairs, evaluated in double and rounded to fp32 once."""
+    return torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float32, device=device)
+
+
+def rotate_norm(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float, eps: Optional[float]) -> torch.Tensor:
+    """Rotate the pairs ``(2i, 2i+1)`` of the first ``dims`` entries of every head of ``x (T, heads, D)``; with ``eps``
+    every head is then divided by its root mean square.  fp32 math, result in ``x.dtype``."""
+    y = x.float().clone()
+    n = dims // 2
+    if n:
+        a = positions.to(torch.float32)[:, None] * pair_freq(dims, base, x.device)[None]
+        c, s = a.cos()[:, None], a.sin()[:, None]
+        u, v = y[..., 0:2 * n:2].clone(), y[..., 1:2 * n:2].clone()
+        y[..., 0:2 * n:2], y[..., 1:2 * n:2] = u * c - v * s, v * c + u * s
+    if eps is not None:
+        y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+    return y.to(x.dtype)
+
+
+def window_scatter(k: torch.Tensor, v: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, slots: torch.Tensor) -> None:
+    """:func:`kv_scatter` into pools whose rows may be wider than the heads."""
+    kv_scatter(k, v, k_pool[..., : k.shape[-1]], v_pool[..., : v.shape[-1]], slots)
+
+
+def window_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, vdim: int, slot_map: torch.Tensor,
+                     seq_rows: torch.Tensor, cu_q: torch.Tensor, past_lens: torch.Tensor, mask_bits: Optional[torch.Tensor],
+                     scale: float, window: int, sink: bool, causal: bool = False) -> torch.Tensor:
+    """:func:`paged_tree_attention` with a window, an optional valueless key of score 0, and heads narrower than the pools'
+    rows.  A row sees the last ``window`` tokens of its own path (itself included): in a tree a node's position is the
+    committed length plus its number of proper ancestors.  Returns ``(T, Hq*vdim)``."""
+    T, Hq, D = q.shape
+    Hkv = k_pool.shape[0]
+    g = Hq // Hkv
+    out = torch.empty(T, Hq * vdim, dtype=q.dtype, device=q.device)
+    cu, pl, rows = cu_q.tolist(), past_lens.tolist(), seq_rows.tolist()
+    for b in range(len(cu) - 1):
+        s, e = cu[b], cu[b + 1]
+        n, past = e - s, pl[b]
+        if n == 0:
+            continue
+        slots = slot_map[rows[b], :past + n].long()
+        k, v = k_pool[:, slots, :D].float(), v_pool[:, slots, :vdim].float()
+        anc = (torch.tril(torch.ones(n, n, dtype=torch.bool, device=q.device)) if causal else unpack_ancestor_bits(mask_bits[s:e], n))
+        pos = past + anc.sum(-1) - 1
+        key_pos = torch.cat((torch.arange(past, device=q.device), pos))
+        vis = torch.cat((torch.ones(n, past, dtype=torch.bool, device=q.device), anc), -1)
+        vis &= pos[:, None] - key_pos[None] < window
+        sc = torch.einsum("nhgd,hld->hgnl", q[s:e].float().view(n, Hkv, g, D), k) * scale
+        sc = sc.masked_fill(~vis[None, None], float("-inf"))
+        if sink:
+            sc = torch.cat((sc, torch.zeros_like(sc[..., :1])), -1)
+        p = torch.nan_to_num(torch.softmax(sc, dim=-1), nan=0.0)[..., : past + n]
+        out[s:e] = torch.einsum("hgnl,hlv->nhgv", p, v).reshape(n, Hq * vdim).to(q.dtype)
+    return out
+
+
+def delta_inputs(y: torch.Tensor, taps: torch.Tensor, z: torch.Tensor, b: torch.Tensor, A_log: torch.Tensor,
+                 dt_bias: torch.Tensor, cfg):
+    """One token's delta-rule inputs from its window ``y (taps, channels)`` of un-convolved rows (oldest first), decay
+    inputs ``z`` and step-size inputs ``b``: ``q, k (H, D)``, ``v (H, V)``, ``g (H, D or 1)``, ``beta (H,)``, fp32."""
+    H, G, D, V = cfg.heads, cfg.kv_heads, cfg.dim, cfg.vdim
+    c = F.silu((y.float() * taps.float().t()).sum(0))
+    q, k, v = c[: G * D].view(G, D), c[G * D: 2 * G * D].view(G, D), c[2 * G * D:].view(H, V)
+    unit = lambda x: x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)
+    q, k = (unit(x).repeat_interleave(H // G, 0) for x in (q, k))
+    g = torch.exp(-torch.exp(A_log.float())[:, None] * F.softplus(z.float() + dt_bias.float()).view(H, -1))
+    return q * D ** -0.5, k, v, g, torch.sigmoid(b.float())
+
+
+def delta_mix(pre: torch.Tensor, z: torch.Tensor, b: torch.Tensor, taps: torch.Tensor, A_log: torch.Tensor,
+              dt_bias: torch.Tensor, cfg, state: torch.Tensor, conv: torch.Tensor, rows: torch.Tensor, cu_q: torch.Tensor,
+              past_lens: torch.Tensor, mask_bits: Optional[torch.Tensor], causal: bool = True) -> torch.Tensor:
+    """Short convolutions and the gated delta rule over a ragged batch.
+
+    ``pre (T, channels)`` are un-convolved q | k | v rows; sequence ``i`` owns rows ``cu_q[i]:cu_q[i+1]``, its state is
+    ``state[rows[i]] (H, D, V)`` and its last convolution inputs ``conv[rows[i]] (taps - 1, channels)``, oldest first.
+    A sequence whose ``past_lens`` is 0 starts from zeros whatever its slot holds.  Causal: tokens follow one another and
+    the states advance.  With ``mask_bits`` (a token tree, parents before children) every node continues its parent's
+    state and the stored states stay as they are.  Per head ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q``.
+    Returns the read-outs, fp32 ``(T, H, V)``."""
+    n_old = taps.shape[1] - 1
+    out = torch.empty(pre.shape[0], cfg.heads, cfg.vdim, dtype=torch.float32, device=pre.device)
+    cu, pl, rl = cu_q.tolist(), past_lens.tolist(), rows.tolist()
+    for i in range(len(cu) - 1):
+        s, e, row = cu[i], cu[i + 1], rl[i]
+        n = e - s
+        if n == 0:
+            continue
+        S0, y0 = state[row].clone(), conv[row].to(pre.dtype)
+        if pl[i] == 0:
+            S0, y0 = torch.zeros_like(S0), torch.zeros_like(y0)
+        anc = None if causal else unpack_ancestor_bits(mask_bits[s:e], n).cpu()
+        kept = []                                       # per row: state behind it, un-convolved rows up to it
+        for t in range(n):
+            if causal:
+                parent = t - 1
+            else:
+                up = [j for j in range(t) if bool(anc[t, j])]
+                parent = up[-1] if up else -1
+            S, y = kept[parent] if parent >= 0 else (S0, y0)
+            y = torch.cat((y, pre[s + t: s + t + 1]), 0)
+            q, k, v, g, beta = delta_inputs(y[-(n_old + 1):], taps, z[s + t], b[s + t], A_log, dt_bias, cfg)
+            S = S * g[..., None]
+            u = beta[:, None] * (v - torch.einsum("hdv,hd->hv", S, k))
+            S = S + k[..., None] * u[:, None]
+            out[s + t] = torch.einsum("hdv,hd->hv", S, q)
+            kept.append((S, y[1:] if n_old else y[:0]))
+            if causal and t:
+                kept[t - 1] = None
+        if causal:
+            state[row], conv[row] = kept[-1][0], kept[-1][1].to(conv.dtype)
+    return out
+
+
+def gated_head_norm(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, kind: str, eps: float) -> torch.Tensor:
+    """``o (T, H, V)`` divided by its root mean square per head, times ``weight (V,)``, times ``silu`` or ``sigmoid`` of
+    ``gate (T, H*V)``; fp32 math, result in ``gate.dtype``."""
+    y = o.float() / torch.sqrt(o.float().pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+    a = F.silu(gate.float()) if kind == "silu" else torch.sigmoid(gate.float())
+    return (y.reshape(gate.shape) * a).to(gate.dtype)
+
+
+def experts_swiglu(x, idx, w_gate, w_up, w_down) -> torch.Tensor:
+    """Mean over the token's experts ``idx (T, top)`` of ``w_down[e] (silu(w_gate[e] x) * w_up[e] x)``, fp32 sums."""
+    out = torch.zeros(x.shape[0], w_down.shape[1], dtype=torch.float32, device=x.device)
+    for e in idx.unique().tolist():
+        tok = (idx == e).nonzero(as_tuple=True)[0]
+        a = silu_mul(torch.cat((F.linear(x[tok], w_gate[e]), F.linear(x[tok], w_up[e])), -1))
+        out.index_add_(0, tok, F.linear(a, w_down[e]).float())
+    return out / idx.shape[1]

@@ -1,8 +1,10 @@
 """Attention backend of the paged engine: owns cache placement and masking for one ragged forward.
 
-A decoder calls the backend once per layer run, ``backend(layer, q, k, v)`` for K/V attention or
-``backend.latent(layer, mixer, q, c)`` for latent attention; the backend writes the new rows into the pool at the
-step's slots and attends through the slot map.
+A decoder calls the backend once per layer run, ``backend(layer, q, k, v)`` for K/V attention,
+``backend.latent(layer, mixer, q, c)`` for latent attention or ``backend.window(layer, mixer, q, k, v)`` for window
+attention; the backend writes the new rows into the pool at the step's slots and attends through the slot map.
+``backend.delta(layer, mixer, pre, z, b)`` advances the recurrent states of the batch's sequences (or, for token trees,
+reads them and holds the nodes' inputs until a path is committed).
 """
 from __future__ import annotations
 
@@ -12,6 +14,8 @@ from .. import ops
 class PagedAttention:
     def __init__(self, pool, meta, scale: float = 1.0):
         self.pool, self.meta, self.scale = pool, meta, scale
+        if pool.states is not None and not meta.causal:
+            pool.states.begin_trees(meta.seq_rows.tolist(), meta.cu_q.tolist()[:-1])
 
     def __call__(self, layer, q, k, v):
         m = self.meta
@@ -25,3 +29,18 @@ class PagedAttention:
         ops.latent_scatter(c, pool, m.slots)
         return ops.latent_attention(q, mixer.k_up.weight, mixer.v_up.weight, pool, self.pool.slot_map, m.seq_rows,
                                     m.cu_q, m.past_lens, m.mask_bits, mixer.cfg.scale, causal=m.causal)
+
+    def window(self, layer, mixer, q, k, v):
+        m, c = self.meta, mixer.cfg
+        kp, vp = self.pool.layer(layer)
+        ops.window_scatter(k, v, kp, vp, m.slots)
+        return ops.window_attention(q, kp, vp, c.vdim, self.pool.slot_map, m.seq_rows, m.cu_q, m.past_lens, m.mask_bits, c.scale,
+                                    c.window, c.sink, causal=m.causal)
+
+    def delta(self, layer, mixer, pre, z, b):
+        m, states = self.meta, self.pool.states
+        weights = (mixer.conv(), mixer.A_log, mixer.dt_bias)
+        if not m.causal:
+            states.hold(layer, weights, pre, z, b)
+        state, conv = states.layer(layer)
+        return ops.delta_mix(pre, z, b, *weights, mixer.cfg, state, conv, m.seq_rows, m.cu_q, m.past_lens, m.mask_bits, m.causal)

@@ -10,7 +10,14 @@ rows of that layer's own width (rounded up to 64 elements, the rest stays zero):
 
     latent_pools : list of (S, width)
 
-Everything below the buffers (pages, slot maps, admission, eviction, commit) is the same for both kinds.
+A model whose layers differ gets its K and V pools per layer, ``(Hkv, S, width)`` (or nothing where a layer caches
+nothing), and one with recurrent layers also a :class:`~jetspec_b200.runtime.state_pool.StatePool`: a sequence's state
+slot is its slot-map row, so it is granted, given back, evicted and used again together with the row::
+
+    kv_layers : list of (k_pool, v_pool) or None
+    states    : StatePool or None
+
+Everything below the buffers (pages, slot maps, admission, eviction, commit) is the same for all kinds.
 
 A *page* (``page_size`` consecutive slots) is the unit of allocation and is shared
 by all layers (one page id addresses the same slots in each layer's slice), so a
@@ -38,6 +45,8 @@ from typing import Optional
 
 import torch
 
+from .state_pool import StatePool
+
 
 class EvictionRequired(RuntimeError):
     """The pool cannot serve the request without evicting another sequence."""
@@ -50,6 +59,11 @@ class EvictionFailed(RuntimeError):
 def latent_row_width(width: int) -> int:
     """Elements a cached latent row takes: ``width`` rounded up to 64 (one 128-byte line of bf16)."""
     return (int(width) + 63) // 64 * 64
+
+
+def window_row_width(dim: int, vdim: int, dtype: torch.dtype) -> tuple:
+    """Elements a K and a V row take: bf16 heads of up to 128 are padded to the tensor-core attention's 128."""
+    return (128, 128) if dtype == torch.bfloat16 and max(dim, vdim) <= 128 else (int(dim), int(vdim))
 
 
 @dataclass
@@ -65,18 +79,25 @@ class SeqState:
 class PagedKVPool:
     def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, num_pages: int,
                  page_size: int = 16, max_seqs: int = 64, max_seq_len: int = 4096,
-                 device="cpu", dtype=torch.float32, latent_widths: Optional[list] = None):
+                 device="cpu", dtype=torch.float32, latent_widths: Optional[list] = None,
+                 kv_shapes: Optional[list] = None, state_shapes: Optional[list] = None):
         self.num_layers, self.num_kv_heads, self.head_dim = num_layers, num_kv_heads, head_dim
         self.page_size, self.num_pages = int(page_size), int(num_pages)
         self.max_seqs, self.max_seq_len = int(max_seqs), int(max_seq_len)
         self.device, self.dtype = torch.device(device), dtype
         S = self.num_pages * self.page_size
-        self.k_pool = self.v_pool = self.latent_pools = None
-        if latent_widths is not None:
+        self.k_pool = self.v_pool = self.latent_pools = self.kv_layers = self.states = None
+        if kv_shapes is not None:
+            def pools(heads, dim, vdim):
+                return tuple(torch.zeros(heads, S, w, dtype=dtype, device=device) for w in window_row_width(dim, vdim, dtype))
+            self.kv_layers = [pools(*shape) if shape is not None else None for shape in kv_shapes]
+        elif latent_widths is not None:
             self.latent_pools = [torch.zeros(S, latent_row_width(w), dtype=dtype, device=device) for w in latent_widths]
         else:
             self.k_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
             self.v_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
+        if state_shapes is not None:
+            self.states = StatePool(state_shapes, self.max_seqs, device=device, dtype=dtype)
         self.slot_map = torch.zeros(self.max_seqs, self.max_seq_len, dtype=torch.int32, device=device)
         self._free_pages: deque = deque(range(self.num_pages))
         self._refcount = [0] * self.num_pages
@@ -92,6 +113,8 @@ class PagedKVPool:
         widths = cfg.latent_widths()
         if widths is not None:
             return cls(len(widths), 0, 0, num_pages, latent_widths=widths, **kw)
+        if cfg.kv_shapes() is not None:
+            return cls(cfg.num_hidden_layers, 0, 0, num_pages, kv_shapes=cfg.kv_shapes(), state_shapes=cfg.state_shapes(), **kw)
         return cls(cfg.num_hidden_layers, cfg.num_key_value_heads // world, cfg.head_dim, num_pages, **kw)
 
     @property
@@ -109,7 +132,7 @@ class PagedKVPool:
         return 1.0 - len(self._free_pages) / max(1, self.num_pages)
 
     def layer(self, li: int):
-        return self.k_pool[li], self.v_pool[li]
+        return self.kv_layers[li] if self.kv_layers is not None else (self.k_pool[li], self.v_pool[li])
 
     def latent(self, li: int) -> torch.Tensor:
         return self.latent_pools[li]
@@ -208,6 +231,8 @@ class PagedKVPool:
 
     def crop(self, seq_id: int, length: int) -> None:
         st = self._seqs[seq_id]
+        if self.states is not None and 0 < int(length) < st.length:
+            raise RuntimeError("a recurrent state cannot be cropped to an earlier position")
         st.length = min(st.length, int(length))
 
     def reset(self) -> None:
@@ -229,7 +254,7 @@ class PagedKVPool:
         ``path`` lists accepted node indices (root first).  The window
         ``slot_map[row, past:past+num_nodes]`` is permuted to ``path`` followed by the
         remaining nodes in index order, and the committed length becomes
-        ``past + len(path)``.  No KV bytes move.
+        ``past + len(path)``.  No KV bytes move; recurrent states advance along the path.
         """
         st = self._seqs[seq_id]
         if isinstance(path, (list, tuple)):      # host path: the permutation is built without a device read
@@ -243,6 +268,8 @@ class PagedKVPool:
             keep[p] = False
             order = torch.cat((p, torch.nonzero(keep, as_tuple=True)[0]))
             n_path = int(p.numel())
+        if self.states is not None:
+            self.states.commit(st.row, past, order[:n_path])
         win = self.slot_map[st.row, past:past + num_nodes]
         self.slot_map[st.row, past:past + num_nodes] = win[order]
         st.length = past + n_path

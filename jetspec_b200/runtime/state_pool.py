@@ -1,0 +1,63 @@
+"""Recurrent state of the sequences a pool serves.
+
+Per recurrent layer::
+
+    state : (slots + 1, heads, dim, vdim)      fp32
+    conv  : (slots + 1, taps - 1, channels)    the last inputs of the short convolutions, oldest first
+
+A sequence's slot is its slot-map row in the paged pool.  Nothing is cleared when a slot changes hands: a forward whose
+committed length is 0 starts from zeros whatever the slot holds.  The last slot belongs to no sequence; warm-up launches
+of captured graphs write there.
+
+A prompt portion or a decoded token advances the state in place.  A token tree does not, because most of its nodes are
+rejected: the forward *holds* every node's inputs of the recurrence, and :meth:`commit` advances the state along the
+accepted path from them.
+"""
+from __future__ import annotations
+
+import torch
+
+from .. import ops
+
+
+class StatePool:
+    def __init__(self, shapes: list, slots: int, device="cpu", dtype=torch.float32):
+        self.shapes, self.slots = list(shapes), int(slots)
+        self.device = torch.device(device)
+        self.state: list = []
+        self.conv: list = []
+        for c in self.shapes:
+            self.state.append(None if c is None else torch.zeros(slots + 1, c.heads, c.dim, c.vdim, dtype=torch.float32, device=device))
+            self.conv.append(None if c is None else torch.zeros(slots + 1, c.taps - 1, c.channels, dtype=dtype, device=device))
+        self._at: dict = {}          # state slot -> first row of its tree among the held rows
+        self._held: dict = {}        # layer -> (weights, pre, z, b) of every row of the last tree forward
+
+    @property
+    def scratch(self) -> int:
+        """The slot no sequence owns."""
+        return self.slots
+
+    def layer(self, i: int):
+        return self.state[i], self.conv[i]
+
+    def begin_trees(self, rows, starts) -> None:
+        """A tree forward begins: the tree of state slot ``rows[j]`` occupies the batch's rows from ``starts[j]`` on."""
+        self._at, self._held = {int(r): int(s) for r, s in zip(rows, starts)}, {}
+
+    def hold(self, layer: int, weights, pre, z, b) -> None:
+        """Keep a layer's recurrence inputs of a tree forward.  ``weights`` is ``(taps, A_log, dt_bias)``."""
+        self._held[layer] = (weights, pre, z, b)
+
+    def commit(self, row: int, past: int, path: torch.Tensor) -> None:
+        """Advance slot ``row`` (at committed length ``past``) along the accepted nodes ``path`` of its held tree."""
+        if row not in self._at:
+            raise RuntimeError("no tree forward is held for this sequence")
+        idx = path.to(self.device).long() + self._at.pop(row)
+        n = int(idx.numel())
+        if n == 0:
+            return
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=self.device)
+        rows, cu_q, past_t = i32([row]), i32([0, n]), i32([past])
+        for i, ((taps, A_log, dt_bias), pre, z, b) in self._held.items():
+            ops.delta_mix(pre[idx], z[idx], b[idx], taps, A_log, dt_bias, self.shapes[i], self.state[i], self.conv[i], rows, cu_q,
+                          past_t, None, True)
