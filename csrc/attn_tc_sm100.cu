@@ -58,6 +58,8 @@ struct AttnTcParams {
   float scale_log2;
   long long kv_head, kv_slot;  // elements between heads / slots of the pools (S*128 and 128 for a (Hkv, S, 128) pool)
   int ldo;                     // elements between tokens of `out`
+  int window;                  // > 0: a row sees the last `window` tokens of its own path only
+  int sink;                    // a valueless key of score 0 takes part in the softmax (counted by the last split)
   int cluster_merge;           // the key splits of a tile form a cluster and merge through distributed shared memory
 };
 
@@ -162,9 +164,11 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   const int* slots = p.slot_map + static_cast<size_t>(p.seq_rows[b]) * p.max_len;
   int L = past + n_b;
   if (p.causal) L = min(L, past + node0 + NPT);
-  const int n_tiles = (L + TKEYS - 1) / TKEYS;
-  const int t_begin = (n_tiles * split) / p.splits;
-  const int t_end = (n_tiles * (split + 1)) / p.splits;
+  // first key tile any row of this CTA can see (a tree's root sits at position `past`)
+  const int t_first = p.window > 0 ? max(0, past + (p.causal ? node0 : 0) - p.window + 1) / TKEYS : 0;
+  const int n_tiles = (L + TKEYS - 1) / TKEYS - t_first;
+  const int t_begin = t_first + (n_tiles * split) / p.splits;
+  const int t_end = t_first + (n_tiles * (split + 1)) / p.splits;
   const int nt = t_end - t_begin;
 
   // softmax thread's row
@@ -176,6 +180,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 
   const bool cmerge = p.cluster_merge != 0;
   float m_run = -INFINITY, l_run = 0.f;     // softmax threads: running (integer) maximum and sum of their row
+  if (p.sink && split == p.splits - 1) { m_run = 0.f; l_run = 1.f; }     // the last split always has a tile
   bool sm_ok = true;
   if (nt <= 0 && !cmerge) {   // more splits than key tiles: this split contributes nothing
     if (warp < 4 && row_valid && p.splits > 1) {
@@ -334,6 +339,21 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 #pragma unroll
     for (int w = 0; w < 8; ++w)
       mw[w] = (!p.causal && row_valid && w < p.W) ? p.mask_bits[static_cast<size_t>(q_begin + node) * p.W + w] : 0;
+    int cut = 0;                       // committed keys below it are out of the row's window
+    if (p.window > 0) {
+      if (p.causal) {
+        cut = past + node - p.window + 1;
+      } else {                         // a node's position is its number of proper ancestors behind the committed length
+        int cnt = 0;
+#pragma unroll
+        for (int w = 0; w < 8; ++w) cnt += __popc(static_cast<unsigned>(mw[w]));
+        cut = min(past, past + cnt - p.window);
+        int drop = cnt - p.window;     // ancestors out of the window are the lowest bits
+#pragma unroll
+        for (int w = 0; w < 8; ++w)
+          for (; drop > 0 && mw[w] != 0; --drop) mw[w] &= mw[w] - 1;
+      }
+    }
     bool ok = true;
     for (int i = 0; i < nt && ok; ++i) {
       const int sb = i & 1;
@@ -369,6 +389,8 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         }
         const int left = L - k0;                         // keys at or past L do not exist
         if (left < 64) vm &= (left <= 0) ? 0ull : ((1ull << left) - 1ull);
+        const int hidden = cut - k0;                     // this many of the tile's keys lie before the window
+        if (hidden > 0) vm = hidden >= 64 ? 0ull : vm & (~0ull << hidden);
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // four chains instead of one 64-deep
       if (vm == ~0ull) {              // the common case: every key of the tile is visible to this row
@@ -628,12 +650,14 @@ extern "C" int js_attn_tc_max_active_clusters(int G, int splits) {
 // js_paged_tree_attention with the layout of the pools and the output spelled out: head h of slot s starts at
 // h * kv_head + s * kv_slot, token t of the output at t * ldo (all multiples of 8).  Needs 128 % (Hq / Hkv) == 0 and
 // W <= 8 (windows of up to 256 nodes).
-extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
-                                          const int* seq_rows, const int* cu_q, const int* past_lens,
-                                          const int* mask_bits, void* out, float* ws_o, float* ws_ml, int* status, int B,
-                                          int T, int Hq, int Hkv, int S, int max_len, int W, int causal, int splits,
-                                          float scale, long long kv_head, long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
+// window > 0 limits a row to the last `window` tokens of its own path; sink adds a valueless key of score 0.
+extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
+                                      const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
+                                      float* ws_o, float* ws_ml, int* status, int B, int T, int Hq, int Hkv, int S, int max_len, int W,
+                                      int causal, int splits, float scale, int window, int sink, long long kv_head, long long kv_slot,
+                                      int ldo, int pdl, cudaStream_t stream) {
   using namespace js;
+  if (window < 0) return -10;
   if (T <= 0 || B <= 0) return 0;
   if (Hq % Hkv) return -10;
   if ((kv_head % 8) || (kv_slot % 8) || (ldo % 8)) return -10;
@@ -662,7 +686,7 @@ extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, 
   AttnTcParams p{reinterpret_cast<const __nv_bfloat16*>(q), reinterpret_cast<const __nv_bfloat16*>(k_pool),
                  reinterpret_cast<const __nv_bfloat16*>(v_pool), slot_map, seq_rows, cu_q, past_lens, mask_bits,
                  reinterpret_cast<__nv_bfloat16*>(out), ws_o, ws_ml, status, B, T, Hq, Hkv, S, max_len, W, causal,
-                 splits, scale * 1.4426950408889634f, kv_head, kv_slot, ldo, in_cluster ? 1 : 0};
+                 splits, scale * 1.4426950408889634f, kv_head, kv_slot, ldo, window, sink, in_cluster ? 1 : 0};
   int rc;
   switch (G) {
     case 1: rc = launch_attn_tc<1>(p, (T + 127) / 128 + B, pdl != 0, stream); break;
@@ -674,6 +698,15 @@ extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, 
   }
   if (rc != 0 || splits == 1 || p.cluster_merge) return rc;
   return js_attn_merge(ws_o, ws_ml, out, ldo, T, Hq, splits, pdl, stream);
+}
+
+extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
+                                          const int* seq_rows, const int* cu_q, const int* past_lens,
+                                          const int* mask_bits, void* out, float* ws_o, float* ws_ml, int* status, int B,
+                                          int T, int Hq, int Hkv, int S, int max_len, int W, int causal, int splits,
+                                          float scale, long long kv_head, long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
+  return js_window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ws_o, ws_ml, status, B, T, Hq,
+                                Hkv, S, max_len, W, causal, splits, scale, 0, 0, kv_head, kv_slot, ldo, pdl, stream);
 }
 
 // Same arguments as js_paged_tree_attention.

@@ -1,0 +1,511 @@
+// Kernels around window attention, post-norm sublayers and table-routed experts: rotation + norm of q and k with the
+// cache scatter, window attention on the plain cores (32-bit path, and heads the tensor-core kernel does not take), the
+// residual step behind a sublayer (norms of its output, sum of experts, next input, final norm), and the permutation of
+// (token, expert) pairs when a table of token ids names the experts.  Math is fp32; the residual stream is fp32.
+#include "common.cuh"
+
+#include <math.h>
+
+namespace js {
+
+JS_DEVICE float hk_ld(const float* p) { return *p; }
+JS_DEVICE float hk_ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+JS_DEVICE void hk_st(float* p, float v) { *p = v; }
+JS_DEVICE void hk_st(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+struct HybridLaunch {
+  cudaLaunchConfig_t c = {};
+  cudaLaunchAttribute a;
+  HybridLaunch(dim3 grid, dim3 block, cudaStream_t stream, int pdl, size_t smem = 0) {
+    c.gridDim = grid;
+    c.blockDim = block;
+    c.stream = stream;
+    c.dynamicSmemBytes = smem;
+    a.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    a.val.programmaticStreamSerializationAllowed = 1;
+    c.attrs = &a;
+    c.numAttrs = pdl ? 1 : 0;
+  }
+};
+
+// sum over a CTA of NT threads; every thread gets the result
+template <int NT>
+JS_DEVICE float cta_sum(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < NT / 32; ++i) s += red[i];
+  __syncthreads();
+  return s;
+}
+
+// ---------------------------------------------------------------- unfused forms
+template <typename TW>
+__global__ void __launch_bounds__(256) rmsnorm_f32_kernel(const float* x, int ldx, const TW* w, float* out, int W, float eps) {
+  __shared__ float red[8];
+  const float* xr = x + static_cast<size_t>(blockIdx.x) * ldx;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < W; c += 256) ss += xr[c] * xr[c];
+  const float r = 1.f / sqrtf(cta_sum<256>(ss, red) / W + eps);
+  for (int c = threadIdx.x; c < W; c += 256) out[static_cast<size_t>(blockIdx.x) * W + c] = xr[c] * r * hk_ld(w + c);
+}
+
+// One head vector per warp: rotate the pairs (2i, 2i+1) of the first `dims` entries, optionally divide by the root mean
+// square, store `width` entries (zeros past D).  Lane l holds the pairs l, l + 32, ...
+template <typename E, typename EB>
+JS_DEVICE void head_rotate_norm(const E* src, const EB* bias, E* dst, int D, int width, int dims, const float* freq, float pos,
+                                bool norm, float eps) {
+  constexpr int NP = 8;                // up to 512 entries
+  const int lane = threadIdx.x & 31;
+  float a[NP], b[NP], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int e = 2 * (lane + 32 * i);
+    a[i] = b[i] = 0.f;
+    if (e < D) a[i] = hk_ld(src + e) + (bias != nullptr ? hk_ld(bias + e) : 0.f);
+    if (e + 1 < D) b[i] = hk_ld(src + e + 1) + (bias != nullptr ? hk_ld(bias + e + 1) : 0.f);
+    if (e + 1 < dims) {
+      float sn, cs;
+      sincosf(pos * freq[e >> 1], &sn, &cs);
+      const float u = a[i], v = b[i];
+      a[i] = u * cs - v * sn;
+      b[i] = v * cs + u * sn;
+    }
+    ss += a[i] * a[i] + b[i] * b[i];
+  }
+  const float r = norm ? 1.f / sqrtf(warp_sum(ss) / D + eps) : 1.f;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int e = 2 * (lane + 32 * i);
+    if (e < width) hk_st(dst + e, a[i] * r);
+    if (e + 1 < width) hk_st(dst + e + 1, b[i] * r);
+  }
+}
+
+template <typename E>
+__global__ void __launch_bounds__(256)
+rotate_norm_kernel(const E* x, E* out, const int* positions, int T, int heads, int D, int dims, const float* freq, int norm, float eps) {
+  const int u = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (u >= T * heads) return;
+  head_rotate_norm<E, E>(x + static_cast<size_t>(u) * D, nullptr, out + static_cast<size_t>(u) * D, D, D, dims, freq,
+                         static_cast<float>(positions[u / heads]), norm != 0, eps);
+}
+
+// ---------------------------------------------------------------- fused: biases, rotation, norm, cache scatter
+// proj (T, ldp): [q heads | k heads | v heads]; q goes to qout (T, G, Gp, Dq) (each group of H/G heads padded to Gp heads,
+// which stay zero), k and v to their pool rows (G, S, Dp) and (G, S, Vp).
+__global__ void __launch_bounds__(256)
+window_post_kernel(const __nv_bfloat16* proj, int ldp, const float* bias, int H, int G, int Gp, int D, int V, int Dq, int Dp, int Vp, int dims,
+                   const float* freq, int norm, float eps, const int* positions, const int* slots, int S, __nv_bfloat16* qout,
+                   __nv_bfloat16* kpool, __nv_bfloat16* vpool, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, u = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (u >= H + 2 * G) return;
+  const __nv_bfloat16* row = proj + static_cast<size_t>(t) * ldp;
+  const float pos = static_cast<float>(positions[t]);
+  if (u < H) {
+    const int hp = (u / (H / G)) * Gp + u % (H / G);
+    head_rotate_norm<__nv_bfloat16, float>(row + u * D, bias != nullptr ? bias + u * D : nullptr,
+                                           qout + (static_cast<size_t>(t) * G * Gp + hp) * Dq, D, Dq, dims, freq, pos, norm != 0, eps);
+    return;
+  }
+  const int slot = slots[t];
+  if (slot < 0 || slot >= S) {
+    if (lane == 0) report(status, kBadSlot);
+    return;
+  }
+  if (u < H + G) {
+    const int c = u * D;
+    head_rotate_norm<__nv_bfloat16, float>(row + c, bias != nullptr ? bias + c : nullptr,
+                                           kpool + (static_cast<size_t>(u - H) * S + slot) * Dp, D, Dp, dims, freq, pos, norm != 0, eps);
+    return;
+  }
+  const int g = u - H - G, c = (H + G) * D + g * V;
+  __nv_bfloat16* dst = vpool + (static_cast<size_t>(g) * S + slot) * Vp;
+  for (int d = lane; d < Vp; d += 32)
+    dst[d] = __float2bfloat16_rn(d < V ? __bfloat162float(row[c + d]) + (bias != nullptr ? bias[c + d] : 0.f) : 0.f);
+}
+
+// ---------------------------------------------------------------- window attention on the plain cores
+// One CTA per (token, head); four warps take every fourth visible key each and merge at the end.  The row sees the last
+// `window` tokens of its own path; the sink is a key of score 0 without a value.
+template <typename E, int NPL>
+__global__ void __launch_bounds__(128)
+window_attn_simt_kernel(const E* q, long long q_tok, const E* kpool, const E* vpool, int Dp, int Vp, const int* slot_map, const int* seq_rows,
+                        const int* cu_q, const int* past_lens, const int* mask_bits, E* out, int ldo, int B, int H, int G, int D, int V,
+                        int S, int max_len, int W, int causal, float scale, int window, int sink, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, h = blockIdx.y, g = h / (H / G);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int lo = 0, hi = B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  const int i = t - cu_q[lo], past = past_lens[lo], n_b = cu_q[lo + 1] - cu_q[lo];
+  const int* slots = slot_map + static_cast<size_t>(seq_rows[lo]) * max_len;
+  const int* bits = causal ? nullptr : mask_bits + static_cast<size_t>(t) * W;
+  int pos = past + i;
+  if (!causal) {
+    int cnt = 0;
+    for (int w = 0; w < W; ++w) cnt += __popc(static_cast<unsigned>(bits[w]));
+    pos = past + cnt - 1;
+  }
+  const int first = max(0, pos - window + 1);
+  const int last = causal ? past + i : past + n_b - 1;
+  float qv[NPL], acc[NPL];
+#pragma unroll
+  for (int e = 0; e < NPL; ++e) {
+    const int c = lane + 32 * e;
+    qv[e] = c < D ? hk_ld(q + t * q_tok + static_cast<size_t>(h) * D + c) * scale : 0.f;
+    acc[e] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  if (sink && warp == 0) { m = 0.f; l = 1.f; }
+  for (int j = (causal ? first : min(first, past)) + warp; j <= last; j += 4) {
+    if (j < past) {
+      if (j < first) continue;
+    } else if (!causal) {
+      const int n = j - past;
+      if (!((bits[n >> 5] >> (n & 31)) & 1)) continue;
+      int depth = 0;                       // proper ancestors of node n, which are those of this row below n
+      for (int w = 0; w < (n >> 5); ++w) depth += __popc(static_cast<unsigned>(bits[w]));
+      depth += __popc(static_cast<unsigned>(bits[n >> 5]) & ((1u << (n & 31)) - 1u));
+      if (past + depth < first) continue;
+    }
+    int slot = slots[j];
+    if (slot < 0 || slot >= S) { if (lane == 0) report(status, kBadSlot); slot = 0; }
+    const E* kr = kpool + (static_cast<size_t>(g) * S + slot) * Dp;
+    const E* vr = vpool + (static_cast<size_t>(g) * S + slot) * Vp;
+    float d = 0.f;
+#pragma unroll
+    for (int e = 0; e < NPL; ++e) {
+      const int c = lane + 32 * e;
+      if (c < D) d += qv[e] * hk_ld(kr + c);
+    }
+    d = warp_sum(d);
+    const float mn = fmaxf(m, d), a = expf(m - mn), p = expf(d - mn);
+    l = l * a + p;
+#pragma unroll
+    for (int e = 0; e < NPL; ++e) {
+      const int c = lane + 32 * e;
+      acc[e] = acc[e] * a + (c < V ? p * hk_ld(vr + c) : 0.f);
+    }
+    m = mn;
+  }
+  __shared__ float sm[4], sl[4];
+  extern __shared__ float so[];            // 4 x V
+  if (lane == 0) { sm[warp] = m; sl[warp] = l; }
+#pragma unroll
+  for (int e = 0; e < NPL; ++e)
+    if (lane + 32 * e < V) so[warp * V + lane + 32 * e] = acc[e];
+  __syncthreads();
+  const float mm = fmaxf(fmaxf(sm[0], sm[1]), fmaxf(sm[2], sm[3]));
+  float f[4], tot = 0.f;
+#pragma unroll
+  for (int w2 = 0; w2 < 4; ++w2) {
+    f[w2] = sm[w2] == -INFINITY ? 0.f : expf(sm[w2] - mm);
+    tot += sl[w2] * f[w2];
+  }
+  const float inv = tot > 0.f ? 1.f / tot : 0.f;
+  for (int c = threadIdx.x; c < V; c += blockDim.x)
+    hk_st(out + static_cast<size_t>(t) * ldo + h * V + c, (so[c] * f[0] + so[V + c] * f[1] + so[2 * V + c] * f[2] + so[3 * V + c] * f[3]) * inv);
+}
+
+template <typename E>
+static int launch_window_simt(const void* q, long long q_tok, const void* kp, const void* vp, int Dp, int Vp, const int* slot_map,
+                              const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out, int ldo,
+                              int B, int T, int H, int G, int D, int V, int S, int max_len, int W, int causal, float scale, int window,
+                              int sink, int* status, int pdl, cudaStream_t stream) {
+  HybridLaunch l(dim3(T, H), dim3(128), stream, pdl, 4 * V * sizeof(float));
+  const int n = D > V ? D : V;
+  auto kern = n <= 64 ? window_attn_simt_kernel<E, 2> : n <= 128 ? window_attn_simt_kernel<E, 4>
+            : n <= 256 ? window_attn_simt_kernel<E, 8> : window_attn_simt_kernel<E, 16>;
+  return cudaLaunchKernelEx(&l.c, kern, (const E*)q, q_tok, (const E*)kp, (const E*)vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens,
+                            mask_bits, (E*)out, ldo, B, H, G, D, V, S, max_len, W, causal, scale, window, sink, status) == cudaSuccess ? 0 : -4;
+}
+
+// ---------------------------------------------------------------- the residual step behind a sublayer
+// y = one of
+//   pair    0.5 (a / rms(a) * wa + b / rms(b) * wb),  a = ya + bias
+//   single  ya + bias
+//   experts (sum_j ys[inv[t k + j]]) / k + sh
+// then x += y / rms(y) * w.  h = bf16(x), or with fw (the model's last norm) h = bf16(x / rms(x) * fw) and tap = bf16(x).
+struct ResidParams {
+  const __nv_bfloat16 *ya, *yb;
+  const float *bias, *wa, *wb;
+  int lda, ldb;
+  const __nv_bfloat16 *ys, *sh;
+  const int* inv;
+  int ldy, lds, k;
+  const float *w, *fw;
+  float eps;
+  float* x;
+  __nv_bfloat16 *h, *tap;
+  int ld, ldt, W;
+};
+
+constexpr int kResidThreads = 512;
+
+__global__ void __launch_bounds__(kResidThreads) resid_norm_kernel(ResidParams p) {
+  extern __shared__ float ry[];            // W
+  __shared__ float red[kResidThreads / 32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, W = p.W, tid = threadIdx.x;
+  float ss = 0.f;
+  if (p.ya == nullptr) {
+    const float wt = p.k > 0 ? 1.f / p.k : 0.f;
+    for (int c = tid * 2; c < W; c += kResidThreads * 2) {        // W even (padded): bf16 pairs
+      float2 acc = make_float2(0.f, 0.f);
+      for (int j = 0; j < p.k; ++j) {
+        const int r = p.inv[t * p.k + j];
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.ys + static_cast<size_t>(r) * p.ldy + c));
+        acc.x += f.x;
+        acc.y += f.y;
+      }
+      acc.x *= wt;
+      acc.y *= wt;
+      if (p.sh != nullptr) {
+        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.sh + static_cast<size_t>(t) * p.lds + c));
+        acc.x += f.x;
+        acc.y += f.y;
+      }
+      ry[c] = acc.x;
+      ss += acc.x * acc.x;
+      if (c + 1 < W) { ry[c + 1] = acc.y; ss += acc.y * acc.y; }
+    }
+  } else {
+    const __nv_bfloat16* a = p.ya + static_cast<size_t>(t) * p.lda;
+    const __nv_bfloat16* b = p.yb != nullptr ? p.yb + static_cast<size_t>(t) * p.ldb : nullptr;
+    auto load_a = [&](int c) {             // rows are padded to even length
+      float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a + c));
+      if (p.bias != nullptr) { v.x += p.bias[c]; v.y += c + 1 < W ? p.bias[c + 1] : 0.f; }
+      if (c + 1 >= W) v.y = 0.f;
+      return v;
+    };
+    auto put = [&](int c, float2 v) {
+      ry[c] = v.x;
+      if (c + 1 < W) ry[c + 1] = v.y;
+    };
+    if (b != nullptr) {
+      float sa = 0.f, sb = 0.f;
+      for (int c = tid * 2; c < W; c += kResidThreads * 2) {
+        const float2 v = load_a(c);
+        put(c, v);
+        sa += v.x * v.x + v.y * v.y;
+        const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(b + c));
+        sb += u.x * u.x + (c + 1 < W ? u.y * u.y : 0.f);
+      }
+      const float ra = 0.5f / sqrtf(cta_sum<kResidThreads>(sa, red) / W + p.eps);
+      const float rb = 0.5f / sqrtf(cta_sum<kResidThreads>(sb, red) / W + p.eps);
+      for (int c = tid * 2; c < W; c += kResidThreads * 2) {
+        const bool two = c + 1 < W;
+        const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(b + c));
+        const float2 v = make_float2(ry[c] * ra * p.wa[c] + u.x * rb * p.wb[c],
+                                     two ? ry[c + 1] * ra * p.wa[c + 1] + u.y * rb * p.wb[c + 1] : 0.f);
+        put(c, v);
+        ss += v.x * v.x + v.y * v.y;
+      }
+    } else {
+      for (int c = tid * 2; c < W; c += kResidThreads * 2) {
+        const float2 v = load_a(c);
+        put(c, v);
+        ss += v.x * v.x + v.y * v.y;
+      }
+    }
+  }
+  const float r = 1.f / sqrtf(cta_sum<kResidThreads>(ss, red) / W + p.eps);     // its barriers also publish ry
+  float* x = p.x + static_cast<size_t>(t) * p.ld;
+  __nv_bfloat16* h = p.h + static_cast<size_t>(t) * p.ld;
+  ss = 0.f;
+  for (int c = tid; c < W; c += kResidThreads) {
+    const float v = x[c] + ry[c] * r * p.w[c];
+    x[c] = v;
+    if (p.tap != nullptr) p.tap[static_cast<size_t>(t) * p.ldt + c] = __float2bfloat16_rn(v);
+    if (p.fw == nullptr) h[c] = __float2bfloat16_rn(v);
+    else { ry[c] = v; ss += v * v; }
+  }
+  if (p.fw == nullptr) return;
+  const float rf = 1.f / sqrtf(cta_sum<kResidThreads>(ss, red) / W + p.eps);
+  for (int c = tid; c < W; c += kResidThreads) h[c] = __float2bfloat16_rn(ry[c] * rf * p.fw[c]);
+}
+
+// x[t] = table[ids[t]] in fp32, h[t] the same in bf16
+__global__ void __launch_bounds__(256)
+embed_f32_kernel(const int* ids, const __nv_bfloat16* table, int V, int ldt, float* x, __nv_bfloat16* h, int ld, int W) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  int id = ids[t];
+  id = id < 0 ? 0 : (id >= V ? V - 1 : id);
+  for (int c = threadIdx.x; c < W; c += blockDim.x) {
+    const __nv_bfloat16 v = table[static_cast<size_t>(id) * ldt + c];
+    x[static_cast<size_t>(t) * ld + c] = __bfloat162float(v);
+    h[static_cast<size_t>(t) * ld + c] = v;
+  }
+}
+
+// ---------------------------------------------------------------- permutation of table-routed pairs
+// One CTA per (layer, pass): pairs (token, choice) of rows [t0, t0 + n) sorted by expert, stably.  All layers' permutations
+// depend on the token ids alone, so one launch at the start of a forward makes them all.
+struct TableLayer {
+  const int* table;      // (V, top)
+  int top, E;
+  int off_tok;           // where this layer's outputs start in `out`: per pass [tok | inv | group offsets]
+};
+
+constexpr int kTableThreads = 1024;
+
+__global__ void __launch_bounds__(kTableThreads)
+table_sort_kernel(const TableLayer* layers, const int* ids, int T, int rows_per_pass, int V, int* out) {
+  extern __shared__ int sh[];
+  pdl_launch_dependents();
+  pdl_wait();
+  const TableLayer L = layers[blockIdx.x];
+  const int t0 = blockIdx.y * rows_per_pass;
+  const int n = min(rows_per_pass, T - t0);
+  if (n <= 0) return;
+  const int P = n * L.top;
+  int* key = sh;                 // P
+  int* cnt = sh + P;             // E + 1
+  int* tok = out + L.off_tok + static_cast<size_t>(t0) * 2 * L.top + static_cast<size_t>(blockIdx.y) * (L.E + 1);
+  int* inv = tok + P;
+  int* goff = inv + P;
+  for (int i = threadIdx.x; i <= L.E; i += blockDim.x) cnt[i] = 0;
+  __syncthreads();
+  for (int p = threadIdx.x; p < P; p += blockDim.x) {
+    int id = ids[t0 + p / L.top];
+    id = id < 0 ? 0 : (id >= V ? V - 1 : id);
+    const int e = L.table[static_cast<size_t>(id) * L.top + p % L.top];
+    key[p] = e;
+    atomicAdd(&cnt[e], 1);
+  }
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (warp == 0) {               // exclusive scan
+    int run = 0;
+    for (int i0 = 0; i0 <= L.E; i0 += 32) {
+      const int i = i0 + lane, c = i < L.E ? cnt[i] : 0;
+      int inc = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, inc, o);
+        if (lane >= o) inc += v;
+      }
+      if (i <= L.E) { cnt[i] = run + inc - c; goff[i] = run + inc - c; }
+      run += __shfl_sync(0xffffffffu, inc, 31);
+    }
+  }
+  __syncthreads();
+  for (int e = warp; e < L.E; e += kTableThreads / 32) {
+    int base = cnt[e];
+    const int end = cnt[e + 1];
+    for (int p0 = 0; p0 < P && base < end; p0 += 32) {
+      const int p = p0 + lane;
+      const bool mine = p < P && key[p] == e;
+      const unsigned m = __ballot_sync(0xffffffffu, mine);
+      if (mine) {
+        const int pos = base + __popc(m & ((1u << lane) - 1u));
+        tok[pos] = t0 + p / L.top;
+        inv[p] = pos;
+      }
+      base += __popc(m);
+    }
+  }
+}
+
+}  // namespace js
+
+extern "C" int js_rmsnorm_f32(const float* x, int ldx, const void* w, int w_bf16, float* out, int T, int W, float eps, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0) return 0;
+  if (w_bf16) rmsnorm_f32_kernel<__nv_bfloat16><<<T, 256, 0, stream>>>(x, ldx, (const __nv_bfloat16*)w, out, W, eps);
+  else rmsnorm_f32_kernel<float><<<T, 256, 0, stream>>>(x, ldx, (const float*)w, out, W, eps);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// x, out (T, heads, D) contiguous; D at most 512, freq (dims / 2) fp32.
+extern "C" int js_rotate_norm(const void* x, void* out, const int* positions, int T, int heads, int D, int dims, const float* freq,
+                              int norm, float eps, int bf16, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0) return 0;
+  if (D > 512 || dims > D || (dims & 1)) return -10;
+  const int g = (T * heads + 7) / 8;
+  if (bf16) rotate_norm_kernel<__nv_bfloat16><<<g, 256, 0, stream>>>((const __nv_bfloat16*)x, (__nv_bfloat16*)out, positions, T, heads, D, dims, freq, norm, eps);
+  else rotate_norm_kernel<float><<<g, 256, 0, stream>>>((const float*)x, (float*)out, positions, T, heads, D, dims, freq, norm, eps);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+extern "C" int js_window_post(const void* proj, int ldp, const float* bias, int H, int G, int Gp, int D, int V, int Dq, int Dp, int Vp, int dims,
+                              const float* freq, int norm, float eps, const int* positions, const int* slots, int S, int T, void* qout,
+                              void* kpool, void* vpool, int* status, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0) return 0;
+  if (H % G || Dp > 512 || Dq > 512 || D > Dq || D > Dp || V > Vp || dims > D || (dims & 1) || Gp < H / G) return -10;
+  HybridLaunch l(dim3(T, (H + 2 * G + 7) / 8), dim3(256), stream, pdl);
+  using bf = __nv_bfloat16;
+  return cudaLaunchKernelEx(&l.c, window_post_kernel, (const bf*)proj, ldp, bias, H, G, Gp, D, V, Dq, Dp, Vp, dims, freq, norm, eps, positions,
+                            slots, S, (bf*)qout, (bf*)kpool, (bf*)vpool, status) == cudaSuccess ? 0 : -4;
+}
+
+// q: token t at t * q_tok, head h at h * D; pools (G, S, Dp) and (G, S, Vp); out (T, ldo), head h at h * V.  D, V at most 512.
+extern "C" int js_window_attention_simt(const void* q, long long q_tok, const void* kp, const void* vp, int Dp, int Vp, const int* slot_map,
+                                        const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
+                                        int ldo, int B, int T, int H, int G, int D, int V, int S, int max_len, int W, int causal,
+                                        float scale, int window, int sink, int bf16, int* status, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0 || B <= 0) return 0;
+  if (H % G || D > 512 || V > 512 || D > Dp || V > Vp || window < 1) return -10;
+  if (!causal && (mask_bits == nullptr || W < 1)) return -13;
+  return bf16 ? launch_window_simt<__nv_bfloat16>(q, q_tok, kp, vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ldo, B, T,
+                                                  H, G, D, V, S, max_len, W, causal, scale, window, sink, status, pdl, stream)
+              : launch_window_simt<float>(q, q_tok, kp, vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ldo, B, T, H, G,
+                                          D, V, S, max_len, W, causal, scale, window, sink, status, pdl, stream);
+}
+
+// Either ya (with yb, wa, wb for a pair; bias optional) or ys / inv / k and sh, all bf16 rows of even
+// length >= W.  W at most 24576.
+extern "C" int js_resid_norm(const void* ya, int lda, const float* bias, const float* wa, const void* yb, int ldb, const float* wb,
+                             const void* ys, int ldy, const int* inv, int k, const void* sh, int lds, const float* w, const float* fw,
+                             float eps, float* x, void* h, int ld, void* tap, int ldt, int T, int W, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0) return 0;
+  if (W < 1 || W > 24576 || ((lda | ldb | ldy | lds) & 1)) return -10;
+  if (ya == nullptr && ys == nullptr && sh == nullptr) return -13;
+  if (yb != nullptr && (wa == nullptr || wb == nullptr)) return -13;
+  using bf = __nv_bfloat16;
+  ResidParams p{(const bf*)ya, (const bf*)yb, bias, wa, wb, lda, ldb, (const bf*)ys, (const bf*)sh, inv, ldy, lds, ys != nullptr ? k : 0, w, fw, eps, x,
+                (bf*)h, (bf*)tap, ld, ldt, W};
+  const int smem = W * 4;
+  static int configured[kMaxDevicesCached] = {};
+  if (smem > 40 * 1024 && ensure_dyn_smem(resid_norm_kernel, smem, configured) != 0) return -3;
+  HybridLaunch l(dim3(T), dim3(kResidThreads), stream, pdl, smem);
+  return cudaLaunchKernelEx(&l.c, resid_norm_kernel, p) == cudaSuccess ? 0 : -4;
+}
+
+extern "C" int js_embed_f32(const int* ids, const void* table, int V, int ldt, float* x, void* h, int ld, int T, int W, int pdl,
+                            cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0) return 0;
+  HybridLaunch l(dim3(T), dim3(256), stream, pdl);
+  return cudaLaunchKernelEx(&l.c, embed_f32_kernel, ids, (const __nv_bfloat16*)table, V, ldt, x, (__nv_bfloat16*)h, ld, W) == cudaSuccess ? 0 : -4;
+}
+
+// layers: n_layers TableLayer records in device memory.  rows_per_pass * max_top at most 16384, max_E at most 1024.
+extern "C" int js_table_sort(const void* layers, int n_layers, const int* ids, int T, int rows_per_pass, int V, int max_top, int max_E,
+                             int* out, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0 || n_layers <= 0) return 0;
+  if (rows_per_pass < 1 || max_top < 1 || rows_per_pass * max_top > 16384 || max_E < 1 || max_E > 1024) return -10;
+  const int rows = T < rows_per_pass ? T : rows_per_pass;
+  const int smem = (rows * max_top + max_E + 1) * 4;
+  static int configured[kMaxDevicesCached] = {};
+  if (ensure_dyn_smem(table_sort_kernel, smem, configured) != 0) return -3;
+  HybridLaunch l(dim3(n_layers, (T + rows_per_pass - 1) / rows_per_pass), dim3(kTableThreads), stream, pdl, smem);
+  return cudaLaunchKernelEx(&l.c, table_sort_kernel, (const TableLayer*)layers, ids, T, rows_per_pass, V, out) == cudaSuccess ? 0 : -4;
+}

@@ -215,7 +215,8 @@ class JetSpecEngine:
     def ragged_kernels(self) -> bool:
         """Whether ragged forwards (portions of prompts beside decoded tokens) run on the fused kernel stack; K/V models
         run theirs through the module path's kernels."""
-        return self.use_kernels and self.cfg.latent_widths() is not None and self.cfg.kernel_path_ok()
+        fused = self.cfg.latent_widths() is not None or self.cfg.kv_shapes() is not None
+        return self.use_kernels and fused and self.cfg.kernel_path_ok()
 
     @torch.inference_mode()
     def step(self, entries):

@@ -327,18 +327,21 @@ class FastRound:
         X.load()
         m = engine.model
         self.embed_w, self.lm_head_w, self.final_norm = m.model.embed_tokens.weight, m.lm_head.weight, m.model.norm.weight
-        self.latent = None                 # launch sequence of a latent-attention decoder (replaces decoder_layers)
+        self.stack = None                  # fused launch sequence of a decoder decoder_layers does not cover
         self.tp = getattr(engine, "tp", None)
         self.ep = getattr(engine, "ep", None)
         if self.tp is not None and self.ep is not None:
             raise NotImplementedError("tensor parallelism and expert parallelism are separate plans here")
         world = self.tp.world if self.tp is not None else 1
-        if self.cfg.latent_widths() is not None:
+        if self.cfg.latent_widths() is not None or self.cfg.kv_shapes() is not None:
             if self.tp is not None or self.ep is not None:
-                raise NotImplementedError("latent-attention models run on one GPU")
-            from .latent_stack import LatentStack
-            self.latent = LatentStack(m, self.device)
-            self.lm_head_w = self.latent.table
+                raise NotImplementedError(f"{self.cfg.model_type} models run on one GPU")
+            if self.cfg.latent_widths() is not None:
+                from .latent_stack import LatentStack as Stack
+            else:
+                from .hybrid_stack import HybridStack as Stack
+            self.stack = Stack(m, self.device)
+            self.lm_head_w = self.stack.head
             self.lcfg, self.layers, self.freq = None, None, None
         else:
             self.lcfg = local_dims(self.cfg, world)
@@ -349,7 +352,7 @@ class FastRound:
             from ..parallel.tp import shard_rows
             self.vocab_local = self.cfg.vocab_size // world
             self.lm_head_w = shard_rows(m.lm_head.weight, self.tp.rank, world)
-        self.prefetcher = WeightPrefetcher(self.device) if _L2_PREFETCH and self.latent is None else None
+        self.prefetcher = WeightPrefetcher(self.device) if _L2_PREFETCH and self.stack is None else None
         self.graphs: dict = {}
         self.draft_cache: dict = {}
         self.launches_per_round = 0
@@ -362,17 +365,18 @@ class FastRound:
 
     # ------------------------------------------------------------------ decoder stack (either model family)
     def _new_stack(self, T: int, max_keys: int):
-        if self.latent is not None:
-            return self.latent.buffers(T, max_keys)
+        if self.stack is not None:
+            return self.stack.buffers(T, max_keys)
         return _Stack(self.lcfg, T, self.device, max_keys)
 
     def _run_stack(self, st, ids, seq_rows, cu_q, past, positions, slots, mask, causal: bool, max_q: int, xn, taps=None,
-                   tap_ids=None, pdl: bool = True, embed_pdl: bool = True, prefetch=None) -> int:
+                   tap_ids=None, pdl: bool = True, embed_pdl: bool = True, prefetch=None, state_rows=None) -> int:
         """Embedding, every layer run, final norm into ``xn``, and the tapped rows.  Returns the launch count."""
         pool, cfg = self.eng.pool, self.cfg
-        if self.latent is not None:
-            batch = self.latent.uniform_batch(pool.slot_map, seq_rows, cu_q, past, slots, mask, causal, st.T, max_q, st.max_keys)
-            return self.latent.run(st, ids, pool.latent_pools, batch, xn, taps=taps, tap_ids=tap_ids, pdl=pdl)
+        if self.stack is not None:
+            batch = self.stack.uniform_batch(pool.slot_map, seq_rows, cu_q, past, slots, mask, causal, st.T, max_q, st.max_keys,
+                                             positions=positions, state_rows=state_rows)
+            return self.stack.run(st, ids, self.stack.caches(pool), batch, xn, taps=taps, tap_ids=tap_ids, pdl=pdl)
         X.embed(ids, self.embed_w, out=st.x, pdl=embed_pdl)
         n = 1 + decoder_layers(self.lcfg, self.layers, st, pool.k_pool, pool.v_pool, pool.slot_map, seq_rows, cu_q, past,
                                positions, slots, mask, causal, self.freq, taps=taps, tap_ids=tap_ids, pdl=pdl, tp=self.tp,
@@ -388,15 +392,18 @@ class FastRound:
     def ragged_forward(self, ids, meta, past_lens, taps=None, logits_rows=None):
         """One ragged batch (portions of prompts, decoded tokens or trees) through the fused stack, launched eagerly.
         Returns ``(fp32 logits of the wanted rows, tapped hidden rows or None)``."""
-        lat, pool, dev = self.latent, self.eng.pool, self.device
+        stack, pool, dev = self.stack, self.eng.pool, self.device
         T = int(ids.numel())
         taps = list(taps) if taps else None
         counts = list(meta.counts)
-        st = lat.buffers(T, max(int(p) + n for p, n in zip(past_lens, counts)))
+        st = stack.buffers(T, max(int(p) + n for p, n in zip(past_lens, counts)))
         hidden = torch.empty(T, len(taps) * self.cfg.hidden_size, dtype=torch.bfloat16, device=dev) if taps else None
         xn = torch.zeros(T, self.xn_cols, dtype=torch.bfloat16, device=dev)
-        batch = lat.ragged_batch(pool.slot_map, meta, counts, [int(p) for p in past_lens])
-        lat.run(st, ids.to(torch.int32), pool.latent_pools, batch, xn, taps=hidden, tap_ids=taps, pdl=_PDL)
+        batch = stack.ragged_batch(pool.slot_map, meta, counts, [int(p) for p in past_lens])
+        stack.run(st, ids.to(torch.int32), stack.caches(pool), batch, xn, taps=hidden, tap_ids=taps, pdl=_PDL)
+        if pool.states is not None and not meta.causal:
+            starts = [sum(counts[:j]) for j in range(len(counts))]
+            stack.hold_trees(st, pool, meta.seq_rows.tolist(), starts, max(counts))
         rows = xn if logits_rows is None else xn[logits_rows].contiguous()
         return self._logits(rows), hidden
 
@@ -754,6 +761,9 @@ class FastRound:
                                            p(r["committed"]), r["committed"].numel(), p(r["eos"]), r["n_eos"],
                                            r["max_new"], p(r["path_idx"]), p(r["result"]), p(status), int(pdl), s()),
                  "js_tree_accept_commit")
+        if pool.states is not None and NB > 1:         # one row is a plain decode step: its states advanced in the forward
+            n += self.stack.commit(st, pool, r["seq_rows"], r["cu_q"], r["state"][ST_PAST:ST_PAST + 1], r["path_idx"],
+                                   r["state"][ST_NEW:ST_NEW + 1], pdl=pdl)
         if remote is not None:
             remote.target_push_header(r["state"], r["committed"], r["path_idx"], pdl)
             n += 4
@@ -793,14 +803,15 @@ class FastRound:
                                f"(m_cap={self.tp.m_cap}); construct TensorParallel with a larger m_cap")
         if fresh:
             H, T = cfg.hidden_size, B * NB
-            n_in = T * (2 + W) + 2 * B
+            n_in = T * (2 + W) + 3 * B
             r = {"B": B, "NB": NB, "W": W, "tap_ids": tap_ids}
             r["inp"] = _i32(n_in, dev)
             r["inp_host"] = torch.zeros(n_in, dtype=torch.int32).pin_memory()
             r["tokens"], r["positions"] = r["inp"][:T], r["inp"][T:2 * T]
             r["mask"] = r["inp"][2 * T:2 * T + T * W].view(T, W)
             r["seq_rows"] = r["inp"][2 * T + T * W:2 * T + T * W + B]
-            r["past"] = r["inp"][2 * T + T * W + B:]
+            r["past"] = r["inp"][2 * T + T * W + B:2 * T + T * W + 2 * B]
+            r["state_rows"] = r["inp"][2 * T + T * W + 2 * B:]
             r["slots"] = _i32(T, dev)
             r["cu_q"] = (torch.arange(B + 1, dtype=torch.int32, device=dev) * NB).contiguous()
             r["ar"] = torch.arange(NB, dtype=torch.long, device=dev)
@@ -817,7 +828,7 @@ class FastRound:
         h = r["inp_host"].numpy()
         tok, pos = h[:T].reshape(B, NB), h[T:2 * T].reshape(B, NB)
         bits = h[2 * T:2 * T + T * W].reshape(B, NB, W)
-        rows, pst = h[2 * T + T * W:2 * T + T * W + B], h[2 * T + T * W + B:]
+        rows, pst, srow = h[2 * T + T * W:].reshape(3, B)
         pad_bits = np.zeros((NB, W), dtype=np.uint32)                   # a pad row sees only itself
         idx = np.arange(NB)
         pad_bits[idx, idx >> 5] = np.uint32(1) << (idx & 31).astype(np.uint32)
@@ -836,6 +847,8 @@ class FastRound:
             bits[b, :n, :max(1, (n + 31) // 32)] = ancestor_bits_np(t_par, n, max(1, (n + 31) // 32)).view(np.int32)
             rows[b] = pool.state(sid).row
             pst[b] = p0
+        # recurrent states must not advance twice: the warm-up launch of a fresh graph works on the scratch slot
+        srow[:] = pool.states.scratch if fresh and pool.states is not None else rows
         r["inp"].copy_(r["inp_host"], non_blocking=True)
         if fresh:
             if self.tp is not None:
@@ -853,6 +866,8 @@ class FastRound:
             pool.frozen = True
             self.graphs[key] = r
             self._tp_graph_key = None
+            srow[:] = rows
+            r["inp"].copy_(r["inp_host"], non_blocking=True)
         if self.tp is not None and getattr(self, "_tp_graph_key", None) != key:
             # the graph's collectives restart their buffer cycle: every rank must have left the previous sequence
             # of collectives (eager prefill, another graph) before the first replay of this one
@@ -861,6 +876,8 @@ class FastRound:
             self._tp_graph_key = key
         r["graph"].replay()
         torch.cuda.current_stream().synchronize()
+        if pool.states is not None and NB > 1:
+            self.stack.hold_trees(r["stack"], pool, rows.tolist(), [b * NB for b in range(B)], NB)
         g_all = r["greedy_host"].numpy().reshape(B, NB)
         greedy = [g_all[b, :t.num_nodes].tolist() for b, t in enumerate(trees)]
         return greedy, r["taps"]
@@ -872,7 +889,8 @@ class FastRound:
         win = r["past"].long()[:, None] + r["ar"][None, :]
         r["slots"].copy_(pool.slot_map[r["seq_rows"].long()].gather(1, win).reshape(-1))
         self._run_stack(st, r["tokens"], r["seq_rows"], r["cu_q"], r["past"], r["positions"], r["slots"], r["mask"], False,
-                        r["NB"], r["xn"], taps=r["taps"], tap_ids=r["tap_ids"], pdl=pdl, embed_pdl=False)
+                        r["NB"], r["xn"], taps=r["taps"], tap_ids=r["tap_ids"], pdl=pdl, embed_pdl=False,
+                        state_rows=r["state_rows"])
         if self.tp is None:
             X.lm_head_argmax(r["xn"], self.lm_head_w, ws=r["am_ws"], pdl=pdl, out_idx=r["greedy"], out_val=r["am_val"])
         else:
@@ -968,7 +986,7 @@ class FastRound:
         pool, dev, cfg = self.eng.pool, self.device, self.cfg
         T, H = ids.shape[1], cfg.hidden_size
         pool.reserve(sid, total)
-        if self.latent is not None:
+        if self.stack is not None:
             return self._prefill_ragged(sid, ids, taps)
         row = pool.state(sid).row
         chunk = 512 if self.tp is None else min(512, self.tp.m_cap)

@@ -123,12 +123,18 @@ class LatentStack:
         self.runs = cfg.layer_runs()
         table = model.model.embed_tokens.weight
         self.table = table if self.wp == self.width else _pad(table, table.shape[0], self.wp)
+        self.head = self.table
         self.vocab = cfg.vocab_size
         self.loops = any(again for _, again in self.runs)
 
     def _pad_norm(self, w, b, alpha):
         p = lambda v: _pad(v.view(1, -1), 1, self.wp).view(-1)
         return p(w), p(b), alpha
+
+    @staticmethod
+    def caches(pool):
+        """What :meth:`run` needs of a pool."""
+        return pool.latent_pools
 
     # ------------------------------------------------------------------ buffers
     def buffers(self, T: int, max_keys: int) -> "types.SimpleNamespace":
@@ -286,7 +292,8 @@ class LatentStack:
         return types.SimpleNamespace(r0=r0, r1=r1, seq_rows=seq_rows, cu_q=cu_q, past=past, max_q=max_q, max_keys=max_keys,
                                      seqs=int(seq_rows.numel()), expand=expand, **kw)
 
-    def uniform_batch(self, slot_map, seq_rows, cu_q, past, slots, mask, causal, rows, max_q, max_keys):
+    def uniform_batch(self, slot_map, seq_rows, cu_q, past, slots, mask, causal, rows, max_q, max_keys, positions=None,
+                      state_rows=None):
         """A batch whose sequences all take the absorbed form (decode steps and token trees)."""
         return types.SimpleNamespace(slot_map=slot_map, slots=slots, mask=mask, causal=causal,
                                      parts=[self.part(0, rows, seq_rows, cu_q, past, max_q, max_keys)])

@@ -206,6 +206,7 @@ def inv_freq(head_dim: int, theta: float, device) -> torch.Tensor:
 # ------------------------------------------------------------------ GEMM
 EPI_STORE, EPI_SWIGLU, EPI_ARGMAX, EPI_TOPK, EPI_STORE_F32 = 0, 1, 2, 3, 4
 EPI_RELU2 = 8
+ACT_GELU_GLU, ACT_RELU2, ACT_NONE = 0, 1, 2
 SM_COUNT = 148
 _DEEP = os.environ.get("JETSPEC_GEMM_DEEP", "0") == "1"
 _SPLIT_DEEP = os.environ.get("JETSPEC_SPLIT_DEEP")      # force the split-K pipeline: 1 = 192 KB, 2 = 128 KB, 0 = 96 KB
@@ -830,9 +831,12 @@ def sigmoid_route(logits: torch.Tensor, correction: torch.Tensor, top: int, scal
 
 
 def gemm_inproj(x, w, raw: Optional[torch.Tensor], n_raw: int, act_out: Optional[torch.Tensor], gelu: bool, pdl: bool = False,
-                bn: Optional[int] = None, split: Optional[int] = None, deep: Optional[int] = None) -> None:
+                bn: Optional[int] = None, split: Optional[int] = None, deep: Optional[int] = None,
+                act: Optional[int] = None) -> None:
     """Fused input projections: ``x @ w.T`` whose first ``n_raw`` columns go to ``raw`` as fp32 and the rest through the
-    activation (tanh-GELU gate * up on 64-row interleaved weights, or relu^2) to ``act_out`` as bf16."""
+    activation (``gelu``: tanh-GELU gate * up on 64-row interleaved weights, else relu^2; ``act`` names any ``ACT_*``
+    instead) to ``act_out`` as bf16."""
+    act = act if act is not None else ACT_GELU_GLU if gelu else ACT_RELU2
     lib = load()
     M, K = x.shape
     N = w.shape[0]
@@ -844,7 +848,7 @@ def gemm_inproj(x, w, raw: Optional[torch.Tensor], n_raw: int, act_out: Optional
             bn, split, deep = pick_gemm_config(M, N, K, EPI_SWIGLU, 128)
     _check(lib.js_gemm_inproj(_p(x), _p(w), _p(raw), _p(act_out), M, N, K, x.stride(0), w.stride(0),
                               raw.stride(0) if raw is not None else 0, act_out.stride(0) if act_out is not None else 0,
-                              int(n_raw), 0 if gelu else 1, bn, split, int(deep), _p(status_word(x.device)), int(pdl),
+                              int(n_raw), int(act), bn, split, int(deep), _p(status_word(x.device)), int(pdl),
                               _stream()), f"js_gemm_inproj(M={M},N={N},K={K},bn={bn},split={split})")
 
 
@@ -881,6 +885,139 @@ def gemm_grouped(a, w, out, total_rows: int, N: int, groups: int, group_off, cov
     _check(lib.js_gemm_bf16_grouped(_p(a), _p(w), _p(out), total_rows, N, a.shape[1], a.stride(0), w.stride(0), out.stride(0), epi,
                                     groups, _p(group_off), cover, None, None, None, None, 1, _p(status_word(a.device)), 0,
                                     _stream()), f"js_gemm_bf16_grouped(rows={total_rows},N={N},groups={groups},epi={epi})")
+
+
+# ------------------------------------------------------------------ window attention, delta rules, post-norm steps
+_pair_freq: dict = {}
+
+
+def pair_freq(dims: int, base: float, device) -> torch.Tensor:
+    key = (dims, float(base), str(device))
+    if key not in _pair_freq:
+        from .reference import pair_freq as table
+        _pair_freq[key] = table(dims, base, device)
+    return _pair_freq[key]
+
+
+def rmsnorm_f32(x: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    lib = load()
+    assert x.dim() == 2 and x.dtype == torch.float32 and x.stride(1) == 1
+    out = torch.empty_like(x, memory_format=torch.contiguous_format)
+    assert w.is_contiguous()
+    _check(lib.js_rmsnorm_f32(_p(x), x.stride(0), _p(w), _is_bf16(w), _p(out), x.shape[0], x.shape[1], ctypes.c_float(eps),
+                              _stream()), "js_rmsnorm_f32")
+    return out
+
+
+def rotate_norm(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float, eps: Optional[float]) -> torch.Tensor:
+    lib = load()
+    T, heads, D = x.shape
+    x = x.contiguous()
+    out = torch.empty_like(x)
+    # named: a temporary would be freed, and its memory possibly handed out again, before the launch
+    pos, freq = positions.to(torch.int32), pair_freq(dims, base, x.device)
+    _check(lib.js_rotate_norm(_p(x), _p(out), _p(pos), T, heads, D, dims, _p(freq),
+                              int(eps is not None), ctypes.c_float(eps or 0.0), _is_bf16(x), _stream()), "js_rotate_norm")
+    return out
+
+
+def window_attention(q, k_pool, v_pool, vdim: int, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int,
+                     sink: bool, causal: bool, out: Optional[torch.Tensor] = None, pdl: bool = False) -> torch.Tensor:
+    """Window attention on the plain cores (bf16 or fp32, heads of up to 512); see the reference op for the contract."""
+    lib = load()
+    T, H, D = q.shape
+    assert q.stride(2) == 1 and q.stride(1) == D
+    G, S, Dp = k_pool.shape
+    if out is None:
+        out = torch.empty(T, H * vdim, dtype=q.dtype, device=q.device)
+    _check(lib.js_window_attention_simt(
+        _p(q), ctypes.c_longlong(q.stride(0)), _p(k_pool), _p(v_pool), Dp, v_pool.shape[2], _p(slot_map), _p(seq_rows), _p(cu_q),
+        _p(past_lens), _p(mask_bits), _p(out), out.stride(0), seq_rows.numel(), T, H, G, D, vdim, S, slot_map.shape[1],
+        mask_bits.shape[1] if mask_bits is not None else 0, int(causal), ctypes.c_float(scale), int(window), int(sink), _is_bf16(q),
+        _p(status_word(q.device)), int(pdl), _stream()), "js_window_attention_simt")
+    return out
+
+
+def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int) -> int:
+    """Key splits of the tensor-core kernel: a CTA's rows span at most the window and their own tokens."""
+    return attn_splits_for(T, Hq, Hkv, min(max_keys, window + 128 // (Hq // Hkv)))
+
+
+def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int, sink: bool,
+                        causal: bool, out: torch.Tensor, splits: int = 1, ws: Optional[dict] = None, pdl: bool = False) -> torch.Tensor:
+    """Window attention on the tcgen05 kernel: bf16, heads padded to 128, groups of 1, 2, 4, 8 or 16 query heads."""
+    lib = load()
+    T, Hq, D = q.shape
+    G, S, _ = k_pool.shape
+    assert D == 128 and q.is_contiguous() and k_pool.shape[2] == 128 and v_pool.shape[2] == 128
+    _check(lib.js_window_attention_tc(
+        _p(q), _p(k_pool), _p(v_pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), _p(mask_bits), _p(out),
+        _p(ws["o"] if splits > 1 else None), _p(ws["ml"] if splits > 1 else None), _p(status_word(q.device)), seq_rows.numel(), T, Hq,
+        G, S, slot_map.shape[1], mask_bits.shape[1] if mask_bits is not None else 0, int(causal), int(splits), ctypes.c_float(scale),
+        int(window), int(sink), ctypes.c_longlong(S * 128), ctypes.c_longlong(128), out.stride(0), int(pdl), _stream()),
+        "js_window_attention_tc")
+    return out
+
+
+def delta_buffers(T: int, cfg, device) -> dict:
+    """Prepared inputs of a delta rule for ``T`` rows and its read-outs, all fp32."""
+    f = lambda *n: torch.empty(T, *n, dtype=torch.float32, device=device)
+    return {"q": f(cfg.kv_heads * cfg.dim), "k": f(cfg.kv_heads * cfg.dim), "v": f(cfg.heads * cfg.vdim), "gl": f(cfg.decays),
+            "beta": f(cfg.heads), "o": f(cfg.heads, cfg.vdim)}
+
+
+def delta_prep(buf: dict, cfg, pre, z, b, taps, A_log, dt_bias, conv, rows, cu_q, past_lens, mask_bits, pdl: bool = False) -> None:
+    """Short convolutions, unit norms, decays and step sizes of every row into ``buf``."""
+    lib = load()
+    T = pre.shape[0]
+    assert pre.stride(1) == 1 and z.stride(1) == 1 and b.stride(1) == 1 and z.dtype == b.dtype == torch.float32
+    assert taps.dtype == pre.dtype == A_log.dtype == dt_bias.dtype == conv.dtype and taps.is_contiguous()
+    _check(lib.js_delta_prep(
+        cfg.heads, cfg.kv_heads, cfg.dim, cfg.vdim, cfg.taps, int(cfg.decay == "channel"), _p(pre), pre.stride(0), _p(z), z.stride(0),
+        _p(b), b.stride(0), _p(taps), _p(A_log), _p(dt_bias), _p(conv), _p(rows), _p(cu_q), _p(past_lens), _p(mask_bits),
+        mask_bits.shape[1] if mask_bits is not None else 0, rows.numel(), T, _p(buf["q"]), _p(buf["k"]), _p(buf["v"]), _p(buf["gl"]),
+        _p(buf["beta"]), _is_bf16(pre), int(pdl), _stream()), "js_delta_prep")
+
+
+def delta_seq(buf: dict, cfg, state, conv, pre, rows, cu_q, past_lens, mask_bits=None, path=None, path_len=None, pdl: bool = False) -> None:
+    """The recurrence over prepared rows: causal (states advance), over token trees (``mask_bits``: nothing is stored), or
+    along the rows ``path[:path_len]`` of one sequence (states advance, nothing is read out)."""
+    lib = load()
+    mode = 1 if mask_bits is not None else 2 if path is not None else 0
+    B = rows.numel()
+    W = mask_bits.shape[1] if mask_bits is not None else 0
+    # paths of a tree are walked by several CTAs: enough of them to fill the device, at most one per 4 nodes
+    groups = max(1, min(32 * W // 4, 4 * SM_COUNT // max(1, B * cfg.heads * ((cfg.vdim + 31) // 32)))) if W else 1
+    _check(lib.js_delta_seq(
+        mode, cfg.heads, cfg.kv_heads, cfg.dim, cfg.vdim, cfg.taps, int(cfg.decay == "channel"), _p(buf["q"]), _p(buf["k"]), _p(buf["v"]),
+        _p(buf["gl"]), _p(buf["beta"]), _p(state), _p(rows), _p(cu_q), _p(past_lens), B, _p(mask_bits), W, groups, _p(path), _p(path_len),
+        _p(buf["o"] if mode != 2 else None), _p(pre), pre.stride(0), _p(conv), _is_bf16(pre), int(pdl), _stream()), "js_delta_seq")
+
+
+def delta_mix(pre, z, b, taps, A_log, dt_bias, cfg, state, conv, rows, cu_q, past_lens, mask_bits, causal: bool) -> torch.Tensor:
+    """Unfused form of a delta rule; see the reference op for the contract."""
+    if not causal and mask_bits.shape[1] > 8:
+        from . import reference as ref
+        return ref.delta_mix(pre, z, b, taps, A_log, dt_bias, cfg, state, conv, rows, cu_q, past_lens, mask_bits, causal)
+    buf = delta_buffers(pre.shape[0], cfg, pre.device)
+    mask = None if causal else mask_bits
+    delta_prep(buf, cfg, pre, z, b, taps, A_log, dt_bias, conv, rows, cu_q, past_lens, mask)
+    delta_seq(buf, cfg, state, conv, pre, rows, cu_q, past_lens, mask)
+    return buf["o"]
+
+
+def gated_head_norm(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, kind: str, eps: float, out: Optional[torch.Tensor] = None,
+                    vp: Optional[int] = None, pdl: bool = False) -> torch.Tensor:
+    """``o (T, H, V)`` fp32 -> ``out (T, H * vp)`` in the gate's dtype; columns of a head past ``V`` are zero."""
+    lib = load()
+    T, H, V = o.shape
+    vp = vp or V
+    if out is None:
+        out = torch.empty(T, H * vp, dtype=gate.dtype, device=gate.device)
+    assert w.dtype == gate.dtype == out.dtype and gate.stride(1) == 1
+    _check(lib.js_gated_head_norm(_p(o), _p(w), _p(gate), gate.stride(0), _p(out), out.stride(0), T, H, V, vp, int(kind == "silu"),
+                                  ctypes.c_float(eps), _is_bf16(gate), int(pdl), _stream()), "js_gated_head_norm")
+    return out
 
 
 # ------------------------------------------------------------------ MoE (grouped through the dense GEMM)

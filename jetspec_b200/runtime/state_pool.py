@@ -15,6 +15,8 @@ accepted path from them.
 """
 from __future__ import annotations
 
+from typing import Callable, Optional
+
 import torch
 
 from .. import ops
@@ -30,6 +32,7 @@ class StatePool:
             self.state.append(None if c is None else torch.zeros(slots + 1, c.heads, c.dim, c.vdim, dtype=torch.float32, device=device))
             self.conv.append(None if c is None else torch.zeros(slots + 1, c.taps - 1, c.channels, dtype=dtype, device=device))
         self._at: dict = {}          # state slot -> first row of its tree among the held rows
+        self._advance = None
         self._held: dict = {}        # layer -> (weights, pre, z, b) of every row of the last tree forward
 
     @property
@@ -40,9 +43,10 @@ class StatePool:
     def layer(self, i: int):
         return self.state[i], self.conv[i]
 
-    def begin_trees(self, rows, starts) -> None:
-        """A tree forward begins: the tree of state slot ``rows[j]`` occupies the batch's rows from ``starts[j]`` on."""
-        self._at, self._held = {int(r): int(s) for r, s in zip(rows, starts)}, {}
+    def begin_trees(self, rows, starts, advance: Optional[Callable] = None) -> None:
+        """A tree forward: the tree of state slot ``rows[j]`` occupies the batch's rows from ``starts[j]`` on.  A caller
+        that holds the rows itself gives ``advance(row, past, start, path)``, which :meth:`commit` then calls."""
+        self._at, self._held, self._advance = {int(r): int(s) for r, s in zip(rows, starts)}, {}, advance
 
     def hold(self, layer: int, weights, pre, z, b) -> None:
         """Keep a layer's recurrence inputs of a tree forward.  ``weights`` is ``(taps, A_log, dt_bias)``."""
@@ -52,10 +56,12 @@ class StatePool:
         """Advance slot ``row`` (at committed length ``past``) along the accepted nodes ``path`` of its held tree."""
         if row not in self._at:
             raise RuntimeError("no tree forward is held for this sequence")
-        idx = path.to(self.device).long() + self._at.pop(row)
-        n = int(idx.numel())
+        start, n = self._at.pop(row), int(path.numel())
         if n == 0:
             return
+        if self._advance is not None:
+            return self._advance(row, past, start, path.to(self.device))
+        idx = path.to(self.device).long() + start
         i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=self.device)
         rows, cu_q, past_t = i32([row]), i32([0, n]), i32([past])
         for i, ((taps, A_log, dt_bias), pre, z, b) in self._held.items():
