@@ -15,7 +15,11 @@ import torch
 
 class DenseKVCache:
     """Contiguous ``(Hkv, capacity, D)`` K and V per layer with a shared length; a latent-attention model's latent rows
-    are held as ``k`` with one head (and no ``v``)."""
+    are held as ``k`` with one head (and no ``v``).
+
+    A recurrent layer holds the inputs of its recurrence as rows of the same kind (``rec``), which :meth:`crop` and
+    :meth:`select` handle like K and V, and its state at an earlier position (``folded`` positions are in it).  The next
+    forward first advances the state over the rows that are committed by then."""
 
     def __init__(self, cfg, device, dtype, capacity: int = 512):
         self.cfg, self.device, self.dtype = cfg, device, dtype
@@ -23,20 +27,34 @@ class DenseKVCache:
         self.capacity = 0
         self.k: list = []
         self.v: list = []
+        self.rec: list = []
+        self.folded = 0
+        self.states = None
+        if cfg.state_shapes() is not None:
+            from ..runtime.state_pool import StatePool
+            self.states = StatePool(cfg.state_shapes(), 1, device=device, dtype=dtype)
         self._grow(capacity)
 
     def _grow(self, cap: int) -> None:
-        widths = self.cfg.latent_widths()
-        if widths is not None:
+        widths, shapes = self.cfg.latent_widths(), self.cfg.kv_shapes()
+        if shapes is not None:
+            one = lambda i: [torch.zeros(s[0], cap, s[i], dtype=self.dtype, device=self.device) if s is not None else None for s in shapes]
+            nk, nv = one(1), one(2)
+        elif widths is not None:
             nk, nv = [torch.zeros(1, cap, w, dtype=self.dtype, device=self.device) for w in widths], []
         else:
             L, Hkv, D = self.cfg.num_hidden_layers, self.cfg.num_key_value_heads, self.cfg.head_dim
             nk = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
             nv = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
-        for new, old in ((nk, self.k), (nv, self.v)):
+        nr = []
+        if self.states is not None:     # (un-convolved rows, decay inputs, step-size inputs), each as one head
+            row = lambda w, dt: torch.zeros(1, cap, w, dtype=dt, device=self.device)
+            nr = [(row(c.channels, self.dtype), row(c.decays, torch.float32), row(c.heads, torch.float32)) for c in self.states.shapes]
+        for new, old in ((nk, self.k), (nv, self.v), ([x for r in nr for x in r], [x for r in self.rec for x in r])):
             for n, o in zip(new, old):
-                n[:, : self.length] = o[:, : self.length]
-        self.k, self.v, self.capacity = nk, nv, cap
+                if n is not None:
+                    n[:, : self.length] = o[:, : self.length]
+        self.k, self.v, self.rec, self.capacity = nk, nv, nr, cap
 
     def ensure(self, n: int) -> None:
         if n > self.capacity:
@@ -46,6 +64,8 @@ class DenseKVCache:
         return self.length
 
     def crop(self, length: int) -> None:
+        if self.folded > int(length):
+            raise RuntimeError("a recurrent state cannot be cropped to an earlier position")
         self.length = min(self.length, int(length))
 
     def select(self, past_len: int, keep_tree_indices) -> None:
@@ -56,7 +76,7 @@ class DenseKVCache:
         (reference: ``_select_kv_cache``, ``jetspec/core/llm.py:86-112``).
         """
         n = len(keep_tree_indices)
-        if (n and n <= 64 and self.v and self.k[0].is_cuda and self.k[0].dtype == torch.bfloat16 and self.k[0].shape[-1] == 128
+        if (n and n <= 64 and self.v and self.states is None and self.k[0].is_cuda and self.k[0].dtype == torch.bfloat16 and self.k[0].shape[-1] == 128
                 and self.k[0].is_contiguous()):
             from ..ops import cuda_ext as X                   # compaction kernel (rows staged in shared memory)
             keep = torch.as_tensor(keep_tree_indices, dtype=torch.int32).to(self.device)
@@ -65,11 +85,27 @@ class DenseKVCache:
             self.length = past_len + n
             return
         idx = torch.as_tensor(keep_tree_indices, dtype=torch.long, device=self.device) + past_len
-        for i in range(len(self.k)):
-            self.k[i][:, past_len:past_len + n] = self.k[i][:, idx]
-            if self.v:
-                self.v[i][:, past_len:past_len + n] = self.v[i][:, idx]
+        for t in (*self.k, *self.v, *(x for r in self.rec for x in r)):
+            if t is not None:
+                t[:, past_len:past_len + n] = t[:, idx]
         self.length = past_len + n
+
+    def delta(self, layer: int, mixer, pre, z, b, mask_bits):
+        """Delta rule of ``len(pre)`` new rows behind the cached ones.  The committed rows the state lacks are folded in
+        first; the new rows are read out from it without being stored, as a tree (``mask_bits``, ``None``: a chain)."""
+        from .. import ops
+        past, T = self.length, pre.shape[0]
+        i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device=self.device)
+        weights, cfg = (mixer.conv(), mixer.A_log, mixer.dt_bias), mixer.cfg
+        state, conv = self.states.layer(layer)
+        if past > self.folded:
+            rows = [x[0, self.folded:past] for x in self.rec[layer]]
+            ops.delta_mix(*rows, *weights, cfg, state, conv, i32(0), i32(0, past - self.folded), i32(self.folded), None, True)
+        for x, new in zip(self.rec[layer], (pre, z, b)):
+            x[0, past:past + T] = new
+        if mask_bits is None:                          # on copies: the rows may yet be cropped
+            state, conv = state[:1].clone(), conv[:1].clone()
+        return ops.delta_mix(pre, z, b, *weights, cfg, state, conv, i32(0), i32(0, T), i32(past), mask_bits, mask_bits is None)
 
 
 class ModelRunner:
@@ -80,7 +116,7 @@ class ModelRunner:
     def _kernel_attention_ok(self, ids: torch.Tensor, T: int, ancestor) -> bool:
         cfg = self.cfg
         w = self.model.lm_head.weight
-        if cfg.latent_widths() is not None:
+        if not hasattr(cfg, "head_dim"):
             return False
         if not (ids.is_cuda and w.dtype == torch.bfloat16 and cfg.head_dim == 128):
             return False
@@ -140,8 +176,7 @@ class ModelRunner:
         if use_kernel:
             kern = self._kernel_attention_args(cache, past, T, ancestor, ids.device)
 
-        latent_cache = cfg.latent_widths() is not None
-        if not latent_cache:
+        if hasattr(cfg, "head_dim"):
             Hq, Hkv, D = cfg.num_attention_heads, cfg.num_key_value_heads, cfg.head_dim
             g = Hq // Hkv
             scale = 1.0 / math.sqrt(D)
@@ -177,9 +212,31 @@ class ModelRunner:
             p = torch.softmax(s, -1)
             return torch.einsum("hgnl,hld->nhgd", p, V).reshape(T, Hq * D).to(q.dtype)
 
-        attn.latent = latent
+        bits = None
+        if ancestor is not None and cache.states is not None:
+            from ..tree.ancestor import pack_ancestor_bits
+            bits = pack_ancestor_bits(ancestor.to(ids.device))
+
+        def window(layer: int, mixer, q, k, v):
+            """Window attention as the plain formula over the contiguous cache."""
+            m = mixer.cfg
+            cache.k[layer][:, past:past + T] = k.transpose(0, 1)
+            cache.v[layer][:, past:past + T] = v.transpose(0, 1)
+            K, V = cache.k[layer][:, :past + T].float(), cache.v[layer][:, :past + T].float()
+            s = torch.einsum("nhgd,hld->hgnl", q.float().view(T, m.kv_heads, m.heads // m.kv_heads, m.dim), K) * m.scale
+            seen = vis & (pos[:, None] - key_pos[None, :] < m.window)
+            s = s.masked_fill(~seen[None, None], float("-inf"))
+            if m.sink:
+                s = torch.cat((s, torch.zeros_like(s[..., :1])), -1)
+            p = torch.softmax(s, -1)[..., : past + T]
+            return torch.einsum("hgnl,hlv->nhgv", p, V).reshape(T, m.heads * m.vdim).to(q.dtype)
+
+        attn.latent, attn.window = latent, window
+        attn.delta = lambda layer, mixer, pre, z, b: cache.delta(layer, mixer, pre, z, b, bits)
         taps = list(target_layer_ids) if (output_hidden_states or target_layer_ids is not None) and target_layer_ids else None
         rows = slice(T - 1, T) if last_position_logits_only else None
         logits, hidden = self.model(ids, pos, attn, tap_layers=taps, logits_rows=rows)
+        if cache.states is not None:
+            cache.folded = past
         cache.length = past + T
         return logits.unsqueeze(0), cache, (hidden.unsqueeze(0) if hidden is not None else None)

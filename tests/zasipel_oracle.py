@@ -179,3 +179,72 @@ def greedy(tokens, w, cfg, n):
     for _ in range(n):
         ids.append(int(forward(ids, w, cfg)[-1].argmax()))
     return ids[len(tokens):]
+
+
+# ------------------------------------------------------------------ random models for the tests
+def random_weights(cfg, ranks=(5, 7), seed=0, dtype=torch.float64):
+    """Weights of every tensor ``cfg`` implies, rounded to bf16 (what a checkpoint holds).  ``ranks``: the low ranks of
+    the decay and of the gate of channel-decay layers.  Decays spread from forgetting within a token to remembering
+    hundreds."""
+    g = torch.Generator().manual_seed(seed)
+    w, W, V = {}, cfg["width"], cfg["vocab"]
+    bf = lambda x: x.to(torch.bfloat16).to(dtype)
+
+    def mat(name, *shape, std=None):
+        w[name] = bf(torch.randn(*shape, generator=g) * (std if std is not None else 1.0 / math.sqrt(shape[-1])))
+
+    def vec(name, n, around, spread):
+        w[name] = bf(around + spread * torch.randn(n, generator=g))
+
+    def delta(p, m, channel):
+        kd, vd = m["kv_heads"] * m["dim"], m["heads"] * m["vdim"]
+        for n, c in (("q", kd), ("k", kd), ("v", vd)):
+            mat(f"{p}.{n}", c, W)
+            mat(f"{p}.{n}.conv", c, m["conv"], std=0.6)
+        mat(p + ".b", m["heads"], W)
+        w[p + ".A_log"] = bf(torch.linspace(-5.0, 1.5, m["heads"]))
+        vec(p + ".norm", m["vdim"], 1.0, 0.2)
+        if channel:
+            mat(p + ".a1", ranks[0], W)
+            mat(p + ".a2", m["heads"] * m["dim"], ranks[0])
+            vec(p + ".dt_bias", m["heads"] * m["dim"], -1.0, 1.5)
+            mat(p + ".g1", ranks[1], W)
+            mat(p + ".g2", vd, ranks[1])
+        else:
+            mat(p + ".a", m["heads"], W)
+            vec(p + ".dt_bias", m["heads"], -1.0, 1.0)
+            mat(p + ".g", vd, W)
+        mat(p + ".o", W, vd)
+
+    def experts(p, f):
+        for n, c in (("gate", f), ("up", f)):
+            mat(f"{p}.{n}", c, W)
+        mat(p + ".down", W, f)
+
+    mat("embed", V, W, std=1.0)
+    for i, L in enumerate(cfg["layers"]):
+        p, m, f = f"l{i}", L["mixer"], L["mlp"]
+        vec(p + ".norm1", W, 1.0, 0.2)
+        if L["type"] == "parallel":
+            a = m["left"]
+            for n, c, k in (("q", a["heads"] * a["dim"], W), ("k", a["kv_heads"] * a["dim"], W), ("v", a["kv_heads"] * a["vdim"], W),
+                            ("o", W, a["heads"] * a["vdim"])):
+                mat(f"{p}.mix.left.{n}", c, k)
+                vec(f"{p}.mix.left.{n}.b", c, 0.0, 0.5)
+            delta(p + ".mix.right", m["right"], False)
+            vec(p + ".mix.left.out", W, 1.0, 0.2)
+            vec(p + ".mix.right.out", W, 1.0, 0.2)
+        else:
+            delta(p + ".mix", m, True)
+        if f is None:
+            continue
+        vec(p + ".norm2", W, 1.0, 0.2)
+        for e in range(f["router"]["experts"]):
+            experts(f"{p}.mlp.e{e}", f["expert"]["ff"])
+        order = torch.rand(V, f["router"]["experts"], generator=g).argsort(-1)
+        w[p + ".mlp.table"] = order[:, : f["router"]["top"]].to(torch.int32)
+        if f.get("shared"):
+            experts(p + ".mlp.shared", f["shared"]["ff"])
+    vec("final.norm", W, 1.0, 0.2)
+    mat("head", V, W)
+    return w
