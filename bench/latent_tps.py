@@ -74,14 +74,16 @@ def throughput(name, cfg, prompt=2048, context=2048, batches=(1, 16)):
     from jetspec_b200 import JetSpecEngine
     from jetspec_b200.engine.engine import _OneNode
     from jetspec_b200.engine.fast_round import FastRound
-    from jetspec_b200.models import KaruzenForCausalLM, Qwen3ForCausalLM
-    cls = KaruzenForCausalLM if cfg.latent_widths() is not None else Qwen3ForCausalLM
-    model = cls.random_init(cfg, seed=0, dtype=torch.bfloat16, device="cuda")
+    from jetspec_b200.models import family_of
+    model = family_of({"model_type": cfg.model_type}).model_cls.random_init(cfg, seed=0, dtype=torch.bfloat16, device="cuda")
     eng = JetSpecEngine(model, device="cuda", dtype=torch.bfloat16, max_seq_len=max(prompt, context) + 64, max_seqs=max(batches))
     out = {"model": name, "family": cfg.model_type, "layer_runs": cfg.num_hidden_layers, "cache_bytes_per_token": 0}
     eng._ensure_pool((max(prompt, context) + 48) * max(batches), seqs=max(batches))
     pool, fast = eng.pool, FastRound.get(eng)
-    bufs = pool.latent_pools if pool.latent_pools is not None else [pool.k_pool, pool.v_pool]
+    bufs = (pool.latent_pools if pool.latent_pools is not None else [b for kv in pool.kv_layers if kv is not None for b in kv]
+            if pool.kv_layers is not None else [pool.k_pool, pool.v_pool])
+    if pool.states is not None:
+        out["state_bytes_per_sequence"] = sum(t[0].numel() * t.element_size() for t in (*pool.states.state, *pool.states.conv))
     out["cache_bytes_per_token"] = sum(b.numel() * b.element_size() for b in bufs) // pool.num_slots
     ids = torch.randint(0, cfg.vocab_size, (1, prompt), generator=torch.Generator().manual_seed(0)).cuda()
 

@@ -1,0 +1,576 @@
+// Fused forms of the gated delta rule (equations and state layout: delta_kernels.cu).
+//
+//   step   one row per sequence (decode): convolution, unit norms, decays, recurrence, per-head norm and gate in ONE kernel,
+//          the head's whole state in registers, read once and written once;
+//   block  prompt portions: rows go in blocks of 8.  With c the logarithms of the decays accumulated inside a block, c_N at its
+//          end, M_ij = beta_i sum_d k_i k_j e^(c_i - c_j) below the diagonal, P the same with q and the diagonal, T = (1 + M)^-1:
+//
+//              w_i = beta_i v_i - (beta_i e^(c_i) k_i)^T S          everything is read from the state BEFORE the block, so
+//              o_i = (e^(c_i) q_i)^T S + sum_m (P T)_im w_m         the only chain left is one matrix product per block
+//              S  <- e^(c_N) S + sum_m (sum_j T_jm e^(c_N - c_j) k_j) w_m^T
+//
+//          A first kernel makes the bracketed rows of all blocks in parallel (with the convolutions and norms); a second one
+//          walks the blocks.  No exponent is ever positive.  All of it is fp32 on the CUDA cores, like the row-by-row kernel.
+#include "common.cuh"
+
+#include <math.h>
+
+namespace js {
+
+JS_DEVICE float df_ld(const float* p) { return *p; }
+JS_DEVICE float df_ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+JS_DEVICE float df_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+JS_DEVICE float df_silu(float z) { return z / (1.f + expf(-z)); }
+JS_DEVICE float df_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+constexpr int kBlk = 8;
+constexpr int kBlkMaxTaps = 17;
+
+struct DeltaIn {
+  int H, G, D, V, taps, channel;
+  const __nv_bfloat16* pre;            // (T, ldp) un-convolved q | k | v
+  const float *z, *b;                  // (T, ldz), (T, ldb)
+  int ldp, ldz, ldb;
+  const __nv_bfloat16 *wt, *A_log, *dt_bias;     // taps (C, n), (H), (H or H*D)
+  __nv_bfloat16* conv;                 // (slots, taps, C) ring
+  const int *rows, *cu_q, *past_lens;
+  int B;
+};
+
+// silu of the convolution of channel c at local row i of a sequence (rows q0 .., committed length past, ring cs)
+JS_DEVICE float conv_at(const DeltaIn& p, const __nv_bfloat16* cs, int C, int q0, int past, int i, int c) {
+  float y = 0.f;
+  const __nv_bfloat16* w = p.wt + static_cast<size_t>(c) * p.taps;
+  for (int m = p.taps - 1; m >= 0; --m) {
+    float x = 0.f;
+    if (i - m >= 0) x = __bfloat162float(p.pre[static_cast<size_t>(q0 + i - m) * p.ldp + c]);
+    else if (past + i - m >= 0) x = __bfloat162float(cs[static_cast<size_t>((past + i - m) % p.taps) * C + c]);
+    y += x * __bfloat162float(w[p.taps - 1 - m]);
+  }
+  return df_silu(y);
+}
+
+// ================================================================ one row per sequence
+struct DeltaStepParams {
+  DeltaIn in;
+  float* state;                        // (slots, H, D, V)
+  const __nv_bfloat16 *gate, *norm_w;  // (T, ldg), (V)
+  __nv_bfloat16* out;                  // (T, ldo)
+  int ldg, ldo, silu;
+  float eps;
+};
+
+constexpr int kStepThreads = 256;
+
+// VG column groups of 4 (a power of two, 4 VG >= V); thread (rl, cg) holds rows rl, rl + RL, ... (NR of them)
+template <int NR>
+__global__ void __launch_bounds__(kStepThreads, 1) delta_step_kernel(DeltaStepParams p, int VG) {
+  __shared__ float sq[256], sk[256], sg[256], sv[256], su[256];
+  __shared__ float red[8 * 256], scal[4];
+  const DeltaIn& in = p.in;
+  const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int D = in.D, V = in.V, g = h / (in.H / in.G);
+  const int C = 2 * in.G * D + in.H * V;
+  const int RL = kStepThreads / VG, cg = tid % VG, rl = tid / VG, col = 4 * cg;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int slot = in.rows[t], past = in.past_lens[t];
+  float* st = p.state + (static_cast<size_t>(slot) * in.H + h) * D * V;
+  float4 S[NR];
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int d = rl + j * RL;
+    S[j] = (past > 0 && d < D && col < V) ? *reinterpret_cast<const float4*>(st + static_cast<size_t>(d) * V + col) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const __nv_bfloat16* cs = in.conv + static_cast<size_t>(slot) * in.taps * C;
+  for (int x = tid; x < 2 * D + V; x += kStepThreads) {
+    const int c = x < D ? g * D + x : x < 2 * D ? (in.G + g) * D + x - D : 2 * in.G * D + h * V + x - 2 * D;
+    const float y = conv_at(in, cs, C, t, past, 0, c);
+    if (x < D) sq[x] = y; else if (x < 2 * D) sk[x - D] = y; else sv[x - 2 * D] = y;
+  }
+  const float a = expf(__bfloat162float(in.A_log[h]));
+  if (in.channel) {
+    for (int d = tid; d < D; d += kStepThreads)
+      sg[d] = expf(-a * df_softplus(in.z[static_cast<size_t>(t) * in.ldz + h * D + d] + __bfloat162float(in.dt_bias[h * D + d])));
+  } else {
+    const float gs = expf(-a * df_softplus(in.z[static_cast<size_t>(t) * in.ldz + h] + __bfloat162float(in.dt_bias[h])));
+    for (int d = tid; d < D; d += kStepThreads) sg[d] = gs;
+  }
+  const float beta = df_sigmoid(in.b[static_cast<size_t>(t) * in.ldb + h]);
+  __syncthreads();
+  if (warp < 2) {                       // unit norms of q (with 1/sqrt(D)) and k
+    const float* src = warp == 0 ? sq : sk;
+    float ss = 0.f;
+    for (int d = lane; d < D; d += 32) ss += src[d] * src[d];
+    ss = warp_sum(ss);
+    if (lane == 0) scal[warp] = (warp == 0 ? 1.f / sqrtf(static_cast<float>(D)) : 1.f) / sqrtf(ss + 1e-6f);
+  }
+  // the ring entry of this position: no CTA of this launch reads it
+  if (in.taps > 1) {
+    __nv_bfloat16* dst = in.conv + (static_cast<size_t>(slot) * in.taps + past % in.taps) * C;
+    const __nv_bfloat16* src = in.pre + static_cast<size_t>(t) * in.ldp;
+    for (int c = tid; c < V; c += kStepThreads) dst[2 * in.G * D + h * V + c] = src[2 * in.G * D + h * V + c];
+    if (h % (in.H / in.G) == 0)
+      for (int c = tid; c < 2 * D; c += kStepThreads) {
+        const int ch = c < D ? g * D + c : (in.G + g) * D + c - D;
+        dst[ch] = src[ch];
+      }
+  }
+  __syncthreads();
+  const float nq = scal[0], nk = scal[1];
+  // sum over the rows of a per-thread partial, for every column; the result lands in dst[0 .. 4 VG)
+  auto column_sum = [&](float4 v, float* dst) {
+    for (int o = VG; o < 32; o <<= 1) {
+      v.x += __shfl_xor_sync(0xffffffffu, v.x, o);
+      v.y += __shfl_xor_sync(0xffffffffu, v.y, o);
+      v.z += __shfl_xor_sync(0xffffffffu, v.z, o);
+      v.w += __shfl_xor_sync(0xffffffffu, v.w, o);
+    }
+    const int sets = VG <= 32 ? 8 : kStepThreads / VG, set = VG <= 32 ? warp : rl;
+    if (VG > 32 || lane < VG) *reinterpret_cast<float4*>(red + set * 256 + col) = v;
+    __syncthreads();
+    for (int c = tid; c < 4 * VG; c += kStepThreads) {
+      float s = 0.f;
+      for (int i = 0; i < sets; ++i) s += red[i * 256 + c];
+      dst[c] = s;
+    }
+    __syncthreads();
+  };
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int d = rl + j * RL;
+    if (d < D) {
+      const float gd = sg[d], kd = sk[d] * nk;
+      S[j].x *= gd; S[j].y *= gd; S[j].z *= gd; S[j].w *= gd;
+      acc.x += S[j].x * kd; acc.y += S[j].y * kd; acc.z += S[j].z * kd; acc.w += S[j].w * kd;
+    }
+  }
+  column_sum(acc, su);
+  float4 u;
+  u.x = beta * ((col < V ? sv[col] : 0.f) - su[col]);
+  u.y = beta * ((col + 1 < V ? sv[col + 1] : 0.f) - su[col + 1]);
+  u.z = beta * ((col + 2 < V ? sv[col + 2] : 0.f) - su[col + 2]);
+  u.w = beta * ((col + 3 < V ? sv[col + 3] : 0.f) - su[col + 3]);
+  acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int j = 0; j < NR; ++j) {
+    const int d = rl + j * RL;
+    if (d < D) {
+      const float kd = sk[d] * nk, qd = sq[d] * nq;
+      S[j].x += kd * u.x; S[j].y += kd * u.y; S[j].z += kd * u.z; S[j].w += kd * u.w;
+      acc.x += S[j].x * qd; acc.y += S[j].y * qd; acc.z += S[j].z * qd; acc.w += S[j].w * qd;
+      if (col < V) *reinterpret_cast<float4*>(st + static_cast<size_t>(d) * V + col) = S[j];
+    }
+  }
+  __syncthreads();                      // su has been read by everyone
+  column_sum(acc, su);
+  if (warp == 0) {
+    float ss = 0.f;
+    for (int c = lane; c < V; c += 32) ss += su[c] * su[c];
+    ss = warp_sum(ss);
+    if (lane == 0) scal[2] = 1.f / sqrtf(ss / V + p.eps);
+  }
+  __syncthreads();
+  const float r = scal[2];
+  for (int c = tid; c < V; c += kStepThreads) {
+    const float zg = __bfloat162float(p.gate[static_cast<size_t>(t) * p.ldg + h * V + c]);
+    p.out[static_cast<size_t>(t) * p.ldo + h * V + c] =
+        __float2bfloat16_rn(su[c] * r * __bfloat162float(p.norm_w[c]) * (p.silu ? df_silu(zg) : df_sigmoid(zg)));
+  }
+}
+
+// ================================================================ blocks of 8 rows
+// Sequence s owns the blocks cu_q[s] / 8 + s, ...; padded row = 8 block + row of the block.  All arrays are per head.
+struct DeltaBlocks {
+  float *kt, *qt, *kh;                 // (H, R, DP): beta e^c k, e^c q, T^T e^(c_N - c) k
+  float *bv;                           // (H, R, V): beta v
+  float *pt;                           // (H, R, 8): P T
+  float *ge;                           // (H, R / 8, DP): e^(c_N)
+  int R;
+};
+
+// lane l ends with the sums over the warp of entries 2 l and 2 l + 1
+JS_DEVICE void warp_transpose_sum64(float (&v)[64]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int b = 16, half = 32; b > 0; b >>= 1, half >>= 1) {
+    const bool hi = (lane & b) != 0;
+#pragma unroll
+    for (int j = 0; j < half; ++j) {
+      const float send = hi ? v[j] : v[j + half];
+      const float keep = hi ? v[j + half] : v[j];
+      v[j] = keep + __shfl_xor_sync(0xffffffffu, send, b);
+    }
+  }
+}
+
+template <int DP, bool CH>
+__global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaBlocks o) {
+  constexpr int NW = DP / 32;
+  __shared__ float part[NW][64], G[64], Tm[64], nrm[NW][16], sbeta[kBlk], sgl[kBlk];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int h = blockIdx.y, tile = blockIdx.x, d = threadIdx.x, warp = d >> 5, lane = d & 31;
+  int lo = 0, hi = in.B - 1;
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (in.cu_q[mid] / kBlk + mid <= tile) lo = mid; else hi = mid - 1;
+  }
+  const int q0 = in.cu_q[lo], n = in.cu_q[lo + 1] - q0, r0 = (tile - (q0 / kBlk + lo)) * kBlk;
+  if (r0 >= n) return;
+  const int past = in.past_lens[lo], m_rows = min(kBlk, n - r0);
+  const int D = in.D, V = in.V, g = h / (in.H / in.G), C = 2 * in.G * D + in.H * V;
+  const __nv_bfloat16* cs = in.conv + static_cast<size_t>(in.rows[lo]) * in.taps * C;
+  const float a = expf(__bfloat162float(in.A_log[h]));
+  if (d < kBlk) {
+    const bool ok = d < m_rows;
+    const size_t t = q0 + r0 + (ok ? d : 0);
+    sbeta[d] = ok ? df_sigmoid(in.b[t * in.ldb + h]) : 0.f;
+    if (!CH) sgl[d] = ok ? -a * df_softplus(in.z[t * in.ldz + h] + __bfloat162float(in.dt_bias[h])) : 0.f;
+  }
+  float q[kBlk], k[kBlk], c[kBlk];
+#pragma unroll
+  for (int i = 0; i < kBlk; ++i) {
+    const bool ok = d < D && i < m_rows;
+    q[i] = ok ? conv_at(in, cs, C, q0, past, r0 + i, g * D + d) : 0.f;
+    k[i] = ok ? conv_at(in, cs, C, q0, past, r0 + i, (in.G + g) * D + d) : 0.f;
+    const float sq = warp_sum(q[i] * q[i]), sk = warp_sum(k[i] * k[i]);
+    if (lane == 0) { nrm[warp][i] = sq; nrm[warp][8 + i] = sk; }
+  }
+  __syncthreads();
+  float run = 0.f;
+#pragma unroll
+  for (int i = 0; i < kBlk; ++i) {
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) { sq += nrm[w][i]; sk += nrm[w][8 + i]; }
+    q[i] *= 1.f / (sqrtf(static_cast<float>(D)) * sqrtf(sq + 1e-6f));
+    k[i] *= 1.f / sqrtf(sk + 1e-6f);
+    if (CH) {
+      if (d < D && i < m_rows)
+        run += -a * df_softplus(in.z[static_cast<size_t>(q0 + r0 + i) * in.ldz + h * D + d] + __bfloat162float(in.dt_bias[h * D + d]));
+    } else {
+      run += sgl[i];
+    }
+    c[i] = run;
+  }
+  // pair sums: P_ij (j <= i) at [i][j], the strict K K^T part (j < i) at [j][i]
+  {
+    float v[64];
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i)
+#pragma unroll
+      for (int j = 0; j <= i; ++j) {
+        const float kj = (CH && j < i) ? k[j] * expf(c[i] - c[j]) : k[j];
+        v[i * 8 + j] = q[i] * kj;
+        if (j < i) v[j * 8 + i] = k[i] * kj;
+      }
+    warp_transpose_sum64(v);
+    part[warp][2 * lane] = v[0];
+    part[warp][2 * lane + 1] = v[1];
+  }
+  __syncthreads();
+  for (int x = d; x < 64; x += DP) {
+    float s = 0.f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) s += part[w][x];
+    if (!CH) {
+      const int i = max(x >> 3, x & 7), j = min(x >> 3, x & 7);
+      float e = 0.f;
+      for (int y = j + 1; y <= i; ++y) e += sgl[y];
+      s *= expf(e);
+    }
+    G[x] = s;
+  }
+  __syncthreads();
+  if (d < kBlk) {                       // column d of T = (1 + M)^-1
+    float col[kBlk];
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) {
+      float s = i == d ? 1.f : 0.f;
+#pragma unroll
+      for (int j = 0; j < i; ++j)
+        if (j >= d) s -= sbeta[i] * G[j * 8 + i] * col[j];
+      col[i] = i < d ? 0.f : s;
+      Tm[i * 8 + d] = col[i];
+    }
+  }
+  __syncthreads();
+  const size_t row = static_cast<size_t>(h) * o.R + static_cast<size_t>(tile) * kBlk;
+  for (int x = d; x < 64; x += DP) {
+    const int i = x >> 3, m = x & 7;
+    float s = 0.f;
+    for (int j = m; j <= i; ++j) s += G[i * 8 + j] * Tm[j * 8 + m];
+    o.pt[row * 8 + x] = s;
+  }
+  const float cn = c[kBlk - 1];
+  float e[kBlk];
+#pragma unroll
+  for (int i = 0; i < kBlk; ++i) {
+    const float ec = expf(c[i]);
+    o.kt[(row + i) * DP + d] = sbeta[i] * ec * k[i];
+    o.qt[(row + i) * DP + d] = ec * q[i];
+    e[i] = expf(cn - c[i]) * k[i];
+  }
+#pragma unroll
+  for (int m = 0; m < kBlk; ++m) {
+    float s = 0.f;
+#pragma unroll
+    for (int j = m; j < kBlk; ++j) s += Tm[j * 8 + m] * e[j];
+    o.kh[(row + m) * DP + d] = s;
+  }
+  o.ge[(static_cast<size_t>(h) * (o.R / kBlk) + tile) * DP + d] = expf(cn);
+  for (int x = d; x < kBlk * V; x += DP) {
+    const int i = x / V, vc = x % V;
+    o.bv[(row + i) * V + vc] = i < m_rows ? sbeta[i] * conv_at(in, cs, C, q0, past, r0 + i, 2 * in.G * D + h * V + vc) : 0.f;
+  }
+}
+
+JS_DEVICE void df_cp16(void* smem, const void* gmem) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem)), "l"(gmem) : "memory");
+}
+JS_DEVICE void df_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+JS_DEVICE void df_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+constexpr int kBlkStages = 3;
+
+// RL = DP / 8 lanes share two columns: lane r holds the rows 4 r .. + 3 and DP/2 + 4 r .. + 3
+template <int DP, int NCOL>
+__global__ void __launch_bounds__(DP / 8 * NCOL / 2)
+delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
+  constexpr int RL = DP / 8, NT = RL * NCOL / 2;
+  struct Stage {
+    float kt[kBlk][DP], qt[kBlk][DP], kh[kBlk][DP], ge[DP], bv[kBlk][NCOL], pt[64];
+  };
+  extern __shared__ __align__(16) uint8_t raw[];
+  Stage* sm = reinterpret_cast<Stage*>(raw);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int slice = blockIdx.x, h = blockIdx.y, sq = blockIdx.z, tid = threadIdx.x, lane = tid & 31;
+  const int q0 = in.cu_q[sq], n = in.cu_q[sq + 1] - q0;
+  if (n <= 0) return;
+  const int D = in.D, V = in.V, past = in.past_lens[sq], slot = in.rows[sq];
+  const int r = tid % RL, lc = tid / RL * 2, col = slice * NCOL + lc;
+  const int tile0 = q0 / kBlk + sq, nb = (n + kBlk - 1) / kBlk;
+  const size_t row0 = static_cast<size_t>(h) * o.R + static_cast<size_t>(tile0) * kBlk;
+  float* st = state + (static_cast<size_t>(slot) * in.H + h) * D * V;
+
+  auto stage_in = [&](int b) {
+    Stage& s = sm[b % kBlkStages];
+    const size_t row = row0 + static_cast<size_t>(b) * kBlk;
+    const float* src[3] = {o.kt + row * DP, o.qt + row * DP, o.kh + row * DP};
+    float* dst[3] = {&s.kt[0][0], &s.qt[0][0], &s.kh[0][0]};
+#pragma unroll
+    for (int a = 0; a < 3; ++a)
+      for (int x = tid; x < kBlk * DP / 4; x += NT) df_cp16(dst[a] + 4 * x, src[a] + 4 * x);
+    const float* ge = o.ge + (static_cast<size_t>(h) * (o.R / kBlk) + tile0 + b) * DP;
+    for (int x = tid; x < DP / 4; x += NT) df_cp16(s.ge + 4 * x, ge + 4 * x);
+    for (int x = tid; x < 16; x += NT) df_cp16(s.pt + 4 * x, o.pt + row * 8 + 4 * x);
+    for (int x = tid; x < kBlk * NCOL / 4; x += NT) {
+      const int i = x / (NCOL / 4), c = x % (NCOL / 4) * 4;
+      if (slice * NCOL + c < V) df_cp16(&s.bv[i][c], o.bv + (row + i) * V + slice * NCOL + c);
+    }
+  };
+  for (int b = 0; b < kBlkStages - 1; ++b) {
+    if (b < nb) stage_in(b);
+    df_commit();
+  }
+  const bool ok = col < V;              // V is a multiple of 4
+  float S[2][4][2];
+#pragma unroll
+  for (int ch = 0; ch < 2; ++ch)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = ch * (DP / 2) + 4 * r + e;
+      const float2 v = (past > 0 && ok && d < D) ? *reinterpret_cast<const float2*>(st + static_cast<size_t>(d) * V + col) : make_float2(0.f, 0.f);
+      S[ch][e][0] = v.x;
+      S[ch][e][1] = v.y;
+    }
+  const int i_own = r & 7;              // the row whose sums this lane ends up with
+  for (int b = 0; b < nb; ++b) {
+    df_wait<kBlkStages - 2>();
+    __syncthreads();
+    if (b + kBlkStages - 1 < nb) stage_in(b + kBlkStages - 1);
+    df_commit();
+    const Stage& s = sm[b % kBlkStages];
+    float acc[2][kBlk][2];              // [k or q][row][column]
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) {
+      acc[0][i][0] = acc[0][i][1] = acc[1][i][0] = acc[1][i][1] = 0.f;
+#pragma unroll
+      for (int ch = 0; ch < 2; ++ch) {
+        const float4 kv = *reinterpret_cast<const float4*>(&s.kt[i][ch * (DP / 2) + 4 * r]);
+        const float4 qv = *reinterpret_cast<const float4*>(&s.qt[i][ch * (DP / 2) + 4 * r]);
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          acc[0][i][c] += S[ch][0][c] * kv.x + S[ch][1][c] * kv.y + S[ch][2][c] * kv.z + S[ch][3][c] * kv.w;
+          acc[1][i][c] += S[ch][0][c] * qv.x + S[ch][1][c] * qv.y + S[ch][2][c] * qv.z + S[ch][3][c] * qv.w;
+        }
+      }
+    }
+    // sums over the RL lanes, halving what every lane keeps: the low three lane bits choose the row, the others sum
+#pragma unroll
+    for (int bit = 4, half = 4; bit > 0; bit >>= 1, half >>= 1) {
+      const bool hi = (r & bit) != 0;
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int j = 0; j < half; ++j)
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            const float send = hi ? acc[t][j][c] : acc[t][j + half][c];
+            const float keep = hi ? acc[t][j + half][c] : acc[t][j][c];
+            acc[t][j][c] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
+          }
+    }
+    float dk[2], dq[2];
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+      dk[c] = acc[0][0][c];
+      dq[c] = acc[1][0][c];
+#pragma unroll
+      for (int bit = 8; bit < RL; bit <<= 1) {
+        dk[c] += __shfl_xor_sync(0xffffffffu, dk[c], bit);
+        dq[c] += __shfl_xor_sync(0xffffffffu, dq[c], bit);
+      }
+    }
+    float W[kBlk][2];
+    const int base = lane & ~(RL - 1);
+#pragma unroll
+    for (int c = 0; c < 2; ++c) {
+      const float w = s.bv[i_own][lc + c] - dk[c];
+#pragma unroll
+      for (int m = 0; m < kBlk; ++m) W[m][c] = __shfl_sync(0xffffffffu, w, base + m);
+    }
+    if (r < kBlk && ok && b * kBlk + i_own < n) {
+#pragma unroll
+      for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int m = 0; m < kBlk; ++m) dq[c] += s.pt[i_own * 8 + m] * W[m][c];
+      *reinterpret_cast<float2*>(out + (static_cast<size_t>(q0 + b * kBlk + i_own) * in.H + h) * V + col) = make_float2(dq[0], dq[1]);
+    }
+#pragma unroll
+    for (int ch = 0; ch < 2; ++ch) {
+      const float4 gv = *reinterpret_cast<const float4*>(&s.ge[ch * (DP / 2) + 4 * r]);
+#pragma unroll
+      for (int c = 0; c < 2; ++c) { S[ch][0][c] *= gv.x; S[ch][1][c] *= gv.y; S[ch][2][c] *= gv.z; S[ch][3][c] *= gv.w; }
+#pragma unroll
+      for (int m = 0; m < kBlk; ++m) {
+        const float4 kv = *reinterpret_cast<const float4*>(&s.kh[m][ch * (DP / 2) + 4 * r]);
+#pragma unroll
+        for (int c = 0; c < 2; ++c) {
+          S[ch][0][c] += kv.x * W[m][c];
+          S[ch][1][c] += kv.y * W[m][c];
+          S[ch][2][c] += kv.z * W[m][c];
+          S[ch][3][c] += kv.w * W[m][c];
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int ch = 0; ch < 2; ++ch)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = ch * (DP / 2) + 4 * r + e;
+      if (ok && d < D) *reinterpret_cast<float2*>(st + static_cast<size_t>(d) * V + col) = make_float2(S[ch][e][0], S[ch][e][1]);
+    }
+  // the last rows' convolution inputs; every reader of the ring ran in the kernel before
+  if (in.taps > 1) {
+    const int C = 2 * in.G * D + in.H * V, g = h / (in.H / in.G);
+    const int qk = slice == 0 && h % (in.H / in.G) == 0 ? 2 * D : 0;
+    __nv_bfloat16* ring = in.conv + static_cast<size_t>(slot) * in.taps * C;
+    for (int x = tid; x < NCOL + qk; x += NT) {
+      if (x < NCOL && slice * NCOL + x >= V) continue;
+      const int y = x - NCOL;
+      const int c = x < NCOL ? 2 * in.G * D + h * V + slice * NCOL + x : y < D ? g * D + y : (in.G + g) * D + y - D;
+      for (int i = max(0, n - in.taps + 1); i < n; ++i)
+        ring[static_cast<size_t>((past + i) % in.taps) * C + c] = in.pre[static_cast<size_t>(q0 + i) * in.ldp + c];
+    }
+  }
+}
+
+struct FusedLaunch {
+  cudaLaunchConfig_t c = {};
+  cudaLaunchAttribute a;
+  FusedLaunch(dim3 grid, dim3 block, cudaStream_t stream, int pdl, size_t smem = 0) {
+    c.gridDim = grid;
+    c.blockDim = block;
+    c.stream = stream;
+    c.dynamicSmemBytes = smem;
+    a.id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    a.val.programmaticStreamSerializationAllowed = 1;
+    c.attrs = &a;
+    c.numAttrs = pdl ? 1 : 0;
+  }
+};
+
+template <int DP, int NCOL>
+static int launch_blocks(const DeltaIn& in, const DeltaBlocks& o, float* state, float* out, int pdl, cudaStream_t stream) {
+  constexpr int smem = kBlkStages * (3 * kBlk * DP + DP + kBlk * NCOL + 64) * 4;
+  static int configured[kMaxDevicesCached] = {};
+  auto kern = delta_block_kernel<DP, NCOL>;
+  if (ensure_dyn_smem(kern, smem, configured) != 0) return -3;
+  FusedLaunch l(dim3((in.V + NCOL - 1) / NCOL, in.H, in.B), dim3(DP / 8 * NCOL / 2), stream, pdl, smem);
+  return cudaLaunchKernelEx(&l.c, kern, in, o, state, out) == cudaSuccess ? 0 : -4;
+}
+
+template <int DP>
+static int launch_block_prep(const DeltaIn& in, const DeltaBlocks& o, int tiles, int pdl, cudaStream_t stream) {
+  FusedLaunch l(dim3(tiles, in.H), dim3(DP), stream, pdl);
+  return (in.channel ? cudaLaunchKernelEx(&l.c, delta_block_prep_kernel<DP, true>, in, o)
+                     : cudaLaunchKernelEx(&l.c, delta_block_prep_kernel<DP, false>, in, o)) == cudaSuccess ? 0 : -4;
+}
+
+static bool fused_shape_ok(int H, int G, int D, int V, int taps) {
+  return H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0 && V % 4 == 0 && taps >= 1 && taps <= kBlkMaxTaps;
+}
+
+}  // namespace js
+
+// One row per sequence, bf16: T = B rows.  Needs V % 4 == 0, V <= 256 and D * (V rounded up to a power of two) <= 16384 (D is
+// covered by at most 16 rows a thread).  gate (T, ldg), norm_w (V), out (T, ldo) bf16.
+extern "C" int js_delta_step(int H, int G, int D, int V, int ntaps, int channel, const void* pre, int ldp, const float* z, int ldz,
+                             const float* b, int ldb, const void* taps, const void* A_log, const void* dt_bias, void* conv, float* state,
+                             const int* rows, const int* cu_q, const int* past_lens, int B, const void* gate, int ldg, const void* norm_w,
+                             int silu, float eps, void* out, int ldo, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (B <= 0) return 0;
+  if (!fused_shape_ok(H, G, D, V, ntaps) || V > 256 || D > 256) return -10;
+  int VG = 1;
+  while (4 * VG < V) VG *= 2;
+  const int RL = kStepThreads / VG, NR = (D + RL - 1) / RL;
+  using bf = __nv_bfloat16;
+  DeltaStepParams p{};
+  p.in = DeltaIn{H, G, D, V, ntaps, channel, (const bf*)pre, z, b, ldp, ldz, ldb, (const bf*)taps, (const bf*)A_log, (const bf*)dt_bias,
+                 (bf*)conv, rows, cu_q, past_lens, B};
+  p.state = state; p.gate = (const bf*)gate; p.norm_w = (const bf*)norm_w; p.out = (bf*)out;
+  p.ldg = ldg; p.ldo = ldo; p.silu = silu; p.eps = eps;
+  FusedLaunch l(dim3(H, B), dim3(kStepThreads), stream, pdl);
+  if (NR > 16) return -10;
+  auto kern = NR <= 4 ? delta_step_kernel<4> : NR <= 8 ? delta_step_kernel<8> : delta_step_kernel<16>;
+  return cudaLaunchKernelEx(&l.c, kern, p, VG) == cudaSuccess ? 0 : -4;
+}
+
+// Prompt portions in blocks of 8 rows, bf16 inputs; D <= 128, V % 4 == 0.  R = 8 * (T / 8 + B) padded rows; kt, qt, kh (H, R, DP),
+// ge (H, R / 8, DP) with DP = 64 or 128; bv (H, R, V); pt (H, R, 8); out (T, H, V) fp32.
+extern "C" int js_delta_blocks(int H, int G, int D, int V, int ntaps, int channel, const void* pre, int ldp, const float* z, int ldz,
+                               const float* b, int ldb, const void* taps, const void* A_log, const void* dt_bias, void* conv, float* state,
+                               const int* rows, const int* cu_q, const int* past_lens, int B, int T, float* kt, float* qt, float* kh,
+                               float* bv, float* pt, float* ge, float* out, int ncol, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0 || B <= 0) return 0;
+  if (!fused_shape_ok(H, G, D, V, ntaps) || D > 128) return -10;
+  using bf = __nv_bfloat16;
+  const DeltaIn in{H, G, D, V, ntaps, channel, (const bf*)pre, z, b, ldp, ldz, ldb, (const bf*)taps, (const bf*)A_log, (const bf*)dt_bias,
+                   (bf*)conv, rows, cu_q, past_lens, B};
+  const int tiles = T / kBlk + B;
+  const DeltaBlocks o{kt, qt, kh, bv, pt, ge, tiles * kBlk};
+  if (D <= 64) {
+    if (int rc = launch_block_prep<64>(in, o, tiles, pdl, stream)) return rc;
+    return ncol == 16 ? launch_blocks<64, 16>(in, o, state, out, pdl, stream) : launch_blocks<64, 32>(in, o, state, out, pdl, stream);
+  }
+  if (int rc = launch_block_prep<128>(in, o, tiles, pdl, stream)) return rc;
+  return ncol == 16 ? launch_blocks<128, 16>(in, o, state, out, pdl, stream) : launch_blocks<128, 32>(in, o, state, out, pdl, stream);
+}

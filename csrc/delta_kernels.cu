@@ -8,8 +8,12 @@
 //           each root-to-leaf path is walked from the stored state;
 //   path    the stored state advances along chosen rows (the accepted nodes of a tree), nothing is read out.
 // A sequence whose committed length is 0 starts from zeros whatever its state slot holds.
+//
+// The convolutions' last inputs are a ring per state slot: the un-convolved row of position p is entry p % taps, so a
+// decode step writes an entry that no reader of the same step looks at.
 #include "common.cuh"
 
+#include <limits.h>
 #include <math.h>
 
 namespace js {
@@ -66,11 +70,10 @@ delta_prep_kernel(DeltaShape s, const E* pre, int ldp, const float* z, int ldz, 
     return;
   }
   const int sq = dl_find_seq(cu_q, B, t);
-  const int q0 = cu_q[sq], i = t - q0;
-  const bool fresh = past_lens[sq] == 0;
-  const int C = 2 * s.G * s.D + s.H * s.V, old = s.taps - 1;
-  const E* cs = conv + static_cast<size_t>(rows[sq]) * old * C;
-  // sources of the taps, newest first: rows of this batch (>= 0), stored inputs (-1 - slot), or nothing
+  const int q0 = cu_q[sq], i = t - q0, past = past_lens[sq];
+  const int C = 2 * s.G * s.D + s.H * s.V;
+  const E* cs = conv + static_cast<size_t>(rows[sq]) * s.taps * C;
+  // sources of the taps, newest first: rows of this batch (>= 0), ring entries (-1 - entry), or nothing (INT_MIN)
   int src[kMaxTaps];
   int have = 0;                         // rows of this batch found so far
   if (mask_bits == nullptr) {
@@ -89,7 +92,10 @@ delta_prep_kernel(DeltaShape s, const E* pre, int ldp, const float* z, int ldz, 
       }
     }
   }
-  for (int m = have; m < s.taps; ++m) src[m] = -1 - (old - 1 - (m - have));
+  for (int m = have; m < s.taps; ++m) {
+    const int pos = past - 1 - (m - have);
+    src[m] = pos >= 0 ? -1 - pos % s.taps : INT_MIN;
+  }
   const bool is_v = unit >= 2 * s.G;
   const int n = is_v ? s.V : s.D;
   const int c0 = is_v ? 2 * s.G * s.D + (unit - 2 * s.G) * s.V : unit * s.D;     // q heads, then k heads, then v heads
@@ -105,7 +111,7 @@ delta_prep_kernel(DeltaShape s, const E* pre, int ldp, const float* z, int ldz, 
       for (int m = s.taps - 1; m >= 0; --m) {
         float in = 0.f;
         if (src[m] >= 0) in = dl_ld(pre + static_cast<size_t>(src[m]) * ldp + c);
-        else if (!fresh) in = dl_ld(cs + static_cast<size_t>(-1 - src[m]) * C + c);
+        else if (src[m] != INT_MIN) in = dl_ld(cs + static_cast<size_t>(-1 - src[m]) * C + c);
         y += in * dl_ld(taps + static_cast<size_t>(c) * s.taps + s.taps - 1 - m);
       }
       y = dl_silu(y);
@@ -140,23 +146,36 @@ struct DeltaSeqParams {
   float* out;                   // (T, H, V); null in path mode
   const void* pre;              // un-convolved rows, for the stored convolution inputs
   int ldp, pre_bf16;
-  void* conv;                   // (slots, taps - 1, C)
+  void* conv;                   // (slots, taps, C) ring
 };
 
 enum : int { kDeltaCausal = 0, kDeltaTree = 1, kDeltaPath = 2 };
 constexpr int kDeltaCols = 32;      // value columns per CTA
 constexpr int kDeltaMaxPath = 256;
 
+// channel c of the ring: the inputs of the walk's last rows (path: their indices), the first of which has position `past`
 template <typename E>
-JS_DEVICE void delta_store_conv(const DeltaSeqParams& p, int q0, const int* path, int n, int slot, int c, bool fresh) {
-  const int old = p.s.taps - 1, C = 2 * p.s.G * p.s.D + p.s.H * p.s.V;
-  E* cs = static_cast<E*>(p.conv) + static_cast<size_t>(slot) * old * C + c;
-  const E* pre = static_cast<const E*>(p.pre) + c;
-  for (int j = 0; j < old; ++j) {          // ascending: entry j + n is read before it is overwritten
-    const int i = j + n - old;
-    if (i >= 0) cs[static_cast<size_t>(j) * C] = pre[static_cast<size_t>(q0 + (path != nullptr ? path[i] : i)) * p.ldp];
-    else if (fresh) dl_st(cs + static_cast<size_t>(j) * C, 0.f);
-    else cs[static_cast<size_t>(j) * C] = cs[static_cast<size_t>(j + n) * C];
+JS_DEVICE void delta_store_conv(const DeltaShape& s, void* conv, const void* pre, int ldp, int q0, const int* path, int n, int past,
+                                int slot, int c) {
+  const int C = 2 * s.G * s.D + s.H * s.V;
+  E* cs = static_cast<E*>(conv) + static_cast<size_t>(slot) * s.taps * C + c;
+  const E* src = static_cast<const E*>(pre) + c;
+  for (int i = max(0, n - s.taps + 1); i < n; ++i)
+    cs[static_cast<size_t>((past + i) % s.taps) * C] = src[static_cast<size_t>(q0 + (path != nullptr ? path[i] : i)) * ldp];
+}
+
+// ... for every channel that belongs to the value columns [v0, v0 + vn) of head h (and to its group's q and k, once)
+JS_DEVICE void delta_store_conv_head(const DeltaShape& s, void* conv, const void* pre, int ldp, int bf16, int q0, const int* path, int n,
+                                     int past, int slot, int h, int v0, int vn) {
+  if (s.taps < 2) return;
+  const int g = h / (s.H / s.G);
+  const int qk = v0 == 0 && h % (s.H / s.G) == 0 ? 2 * s.D : 0;
+  for (int c = threadIdx.x; c < vn + qk; c += blockDim.x) {
+    const int x = c - vn;
+    const int ch = c < vn ? 2 * s.G * s.D + h * s.V + v0 + c : x < s.D ? g * s.D + x : (s.G + g) * s.D + x - s.D;
+    if (c < vn && v0 + c >= s.V) continue;
+    if (bf16) delta_store_conv<__nv_bfloat16>(s, conv, pre, ldp, q0, path, n, past, slot, ch);
+    else delta_store_conv<float>(s, conv, pre, ldp, q0, path, n, past, slot, ch);
   }
 }
 
@@ -178,7 +197,7 @@ delta_seq_kernel(DeltaSeqParams p) {
   const int col = slice * kDeltaCols + tid / R, r = tid % R;
   const int g = h / (s.H / s.G), slot = p.rows[sqi];
   const int q0 = p.cu_q[sqi], n_rows = p.cu_q[sqi + 1] - q0;
-  const bool fresh = p.past_lens[sqi] == 0;
+  const bool fresh = MODE != kDeltaPath && p.past_lens[sqi] == 0;      // a tree always has a committed prefix
   if (n_rows <= 0) return;
   float* st = p.state + (static_cast<size_t>(slot) * s.H + h) * s.D * s.V;
   const bool cv = col < s.V;
@@ -326,22 +345,9 @@ delta_seq_kernel(DeltaSeqParams p) {
       const int d = 4 * (i * R + r) + e;
       if (cv && d < s.D) st[static_cast<size_t>(d) * s.V + col] = S[i][e];
     }
-  // the convolutions' last inputs: this CTA's value columns, and with slice 0 of a group's first head its q and k
-  if (s.taps > 1) {
-    const int* path = MODE == kDeltaPath ? spath : nullptr;
-    const int vc = 2 * s.G * s.D + h * s.V;
-    for (int c = tid; c < kDeltaCols; c += NT) {
-      if (slice * kDeltaCols + c >= s.V) break;
-      if (p.pre_bf16) delta_store_conv<__nv_bfloat16>(p, q0, path, n, slot, vc + slice * kDeltaCols + c, fresh);
-      else delta_store_conv<float>(p, q0, path, n, slot, vc + slice * kDeltaCols + c, fresh);
-    }
-    if (slice == 0 && h % (s.H / s.G) == 0)
-      for (int c = tid; c < 2 * s.D; c += NT) {
-        const int ch = c < s.D ? g * s.D + c : (s.G + g) * s.D + c - s.D;
-        if (p.pre_bf16) delta_store_conv<__nv_bfloat16>(p, q0, path, n, slot, ch, fresh);
-        else delta_store_conv<float>(p, q0, path, n, slot, ch, fresh);
-      }
-  }
+  // in path mode past_lens is the committed length behind the path
+  delta_store_conv_head(s, p.conv, p.pre, p.ldp, p.pre_bf16, q0, MODE == kDeltaPath ? spath : nullptr, n,
+                        p.past_lens[sqi] - (MODE == kDeltaPath ? n : 0), slot, h, slice * kDeltaCols, kDeltaCols);
 }
 
 template <int DP, int R, int TB>
@@ -412,7 +418,7 @@ static bool delta_shape_ok(int H, int G, int D, int V, int taps) {
 
 }  // namespace js
 
-// pre (T, ldp) un-convolved q | k | v rows, taps (C, n), conv (slots, n - 1, C), A_log (H), dt_bias (H or H*D): bf16 or fp32;
+// pre (T, ldp) un-convolved q | k | v rows, taps (C, n), conv (slots, n, C) ring, A_log (H), dt_bias (H or H*D): bf16 or fp32;
 // z (T, ldz), b (T, ldb) fp32.  Outputs fp32: q, k (T, G, D), v (T, H, V), gl (T, H or H*D), beta (T, H).  mask_bits (T, W)
 // for token trees, else null.
 extern "C" int js_delta_prep(int H, int G, int D, int V, int ntaps, int channel, const void* pre, int ldp, const float* z, int ldz,
@@ -435,7 +441,7 @@ extern "C" int js_delta_prep(int H, int G, int D, int V, int ntaps, int channel,
 }
 
 // The recurrence over prepared inputs.  mode 0 causal, 1 tree (W <= 8, at most 256 nodes), 2 path (B = 1; path_len on the
-// device, at most 256).  state (slots, H, D, V) fp32; out (T, H, V) fp32.
+// device, at most 256; past_lens is then the committed length behind the path).  state (slots, H, D, V) fp32; out (T, H, V) fp32.
 extern "C" int js_delta_seq(int mode, int H, int G, int D, int V, int ntaps, int channel, const float* q, const float* k, const float* v,
                             const float* gl, const float* beta, float* state, const int* rows, const int* cu_q, const int* past_lens,
                             int B, const int* mask_bits, int W, int leaf_groups, const int* path, const int* path_len, float* out,

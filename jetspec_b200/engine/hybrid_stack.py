@@ -8,8 +8,8 @@ Per layer, on the bf16 copy ``h`` of the fp32 residual stream ``x``:
    GEMM over both factors side by side;
 2. window attention: one kernel adds the biases, rotates and norms q and k and scatters K/V to the pool; the tcgen05
    attention kernel follows, with its key range cut to the window and the sink in its softmax;
-3. delta rule: one kernel convolves, normalises and forms the decays; the recurrence runs over the prepared rows and
-   the gated per-head norm follows;
+3. delta rule: a decode step is one kernel from the projections to the gated per-head norm; portions go in blocks of 8
+   rows (one kernel prepares all blocks, one walks them, the norm follows); token trees go row by row;
 4. output GEMMs, then ONE kernel for the residual step: the norms of the sublayers' outputs, the sum, the stream, the
    next bf16 input (and behind the last layer the model's final norm);
 5. experts: the permutation by expert depends on the token ids alone, so one launch at the start makes every layer's;
@@ -208,11 +208,13 @@ class HybridStack:
                           "ml": torch.zeros(splits, st.T, Hq, 2, dtype=torch.float32, device=self.device)}
         return st.ws.get(key)
 
-    def _delta_buf(self, st, L, hold: bool) -> dict:
-        """Prepared rows of a layer: one set for all layers, or one each when they have to outlive the forward."""
-        key = L.index if hold else (L.dc.heads, L.dc.kv_heads, L.dc.dim, L.dc.vdim, L.dc.decays)
+    def _delta_buf(self, st, L, hold: bool, kind: str = "rows", seqs: int = 0) -> dict:
+        """Workspace of a delta layer: one for all layers of a shape, or one each when it has to outlive the forward."""
+        c = L.dc
+        key = L.index if hold else (kind, seqs, c.heads, c.kv_heads, c.dim, c.vdim, c.decays)
         if key not in st.delta:
-            st.delta[key] = X.delta_buffers(st.T, L.dc, self.device)
+            st.delta[key] = (X.delta_block_buffers(st.T, seqs, c, self.device) if kind == "blocks"
+                             else X.delta_buffers(st.T, c, self.device))
         return st.delta[key]
 
     def _act(self, st, L, hold: bool) -> torch.Tensor:
@@ -320,13 +322,20 @@ class HybridStack:
     def _delta(self, st, L, pool, batch, pre, z, b, gate, y, hold, pdl) -> int:
         c = L.dc
         state, conv = pool.states.layer(L.index)
-        buf = self._delta_buf(st, L, hold)
-        X.delta_prep(buf, c, pre, z, b, L.taps, L.A_log, L.dt_bias, conv, batch.state_rows, batch.cu_q, batch.past, batch.mask, pdl=pdl)
-        X.delta_seq(buf, c, state, conv, pre, batch.state_rows, batch.cu_q, batch.past, batch.mask, pdl=pdl)
         o = st.get("do", L.o_cols, zero=L.o_cols != c.heads * c.vdim)
-        X.gated_head_norm(buf["o"], L.o_norm, gate[:, : c.heads * c.vdim], c.gate, L.eps, out=o, pdl=pdl)
+        gate = gate[:, : c.heads * c.vdim]
+        seqs = (batch.state_rows, batch.cu_q, batch.past)
+        if hold:
+            buf = self._delta_buf(st, L, True)
+            X.delta_prep(buf, c, pre, z, b, L.taps, L.A_log, L.dt_bias, conv, *seqs, batch.mask, pdl=pdl)
+            X.delta_seq(buf, c, state, conv, pre, *seqs, batch.mask, pdl=pdl)
+            X.gated_head_norm(buf["o"], L.o_norm, gate, c.gate, L.eps, out=o, pdl=pdl)
+            n = 3
+        else:
+            n = X.delta_forward(c, pre, z, b, L.taps, L.A_log, L.dt_bias, state, conv, *seqs, gate, L.o_norm, c.gate, L.eps, o,
+                                batch.max_rows, buffers=lambda kind: self._delta_buf(st, L, False, kind, batch.state_rows.numel()), pdl=pdl)
         X.gemm(o, L.w_o, out=y, pdl=pdl)
-        return 4
+        return n + 1
 
     def _experts(self, st, L, out, tap, pdl) -> int:
         m, T = L.moe, st.T
@@ -358,7 +367,8 @@ class HybridStack:
 
     # ------------------------------------------------------------------ token trees
     def commit(self, st, pool, state_rows, cu_q, past, path, path_len, pdl: bool = True) -> int:
-        """Advance one sequence's states along the rows ``path[:path_len]`` (device) of the tree forward run on ``st``."""
+        """Advance one sequence's states along the rows ``path[:path_len]`` (device) of the tree forward run on ``st``;
+        ``past`` is the committed length behind the path."""
         for L in self.layers:
             state, conv = pool.states.layer(L.index)
             pre = self._act(st, L, True)[:, L.at["q"]:L.at["q"] + L.dc.channels]
@@ -372,7 +382,7 @@ class HybridStack:
 
         def advance(row, past, start, path):
             end = min(start + nodes, st.T)
-            self.commit(st, pool, i32([row]), i32([start, end]), i32([past]), path.to(torch.int32), i32([path.numel()]))
+            self.commit(st, pool, i32([row]), i32([start, end]), i32([past + path.numel()]), path.to(torch.int32), i32([path.numel()]))
         pool.states.begin_trees(rows, starts, advance)
 
     # ------------------------------------------------------------------ batches
@@ -380,10 +390,11 @@ class HybridStack:
         """A batch of equal row counts (decode steps and token trees); one row a sequence is a plain decode step."""
         return types.SimpleNamespace(slot_map=slot_map, seq_rows=seq_rows, cu_q=cu_q, past=past, slots=slots,
                                      mask=None if causal or max_q == 1 else mask, positions=positions, max_keys=max_keys,
-                                     state_rows=seq_rows if state_rows is None else state_rows)
+                                     max_rows=max_q, state_rows=seq_rows if state_rows is None else state_rows)
 
     def ragged_batch(self, slot_map, meta, counts, past_lens):
         """Portions of prompts beside decoded tokens, or token trees."""
         return types.SimpleNamespace(slot_map=slot_map, seq_rows=meta.seq_rows, cu_q=meta.cu_q, past=meta.past_lens, slots=meta.slots,
                                      mask=None if meta.causal else meta.mask_bits, positions=meta.positions,
-                                     max_keys=max(a + b for a, b in zip(counts, past_lens)), state_rows=meta.seq_rows)
+                                     max_keys=max(a + b for a, b in zip(counts, past_lens)), max_rows=max(counts),
+                                     state_rows=meta.seq_rows)

@@ -966,12 +966,21 @@ def delta_buffers(T: int, cfg, device) -> dict:
             "beta": f(cfg.heads), "o": f(cfg.heads, cfg.vdim)}
 
 
+def _check_delta_pool(cfg, pre, z, b, conv, state=None) -> None:
+    """Shapes the kernels index by: the state pool's slots and the width of the rows."""
+    assert pre.shape[1] == cfg.channels and z.shape[1] >= cfg.decays and b.shape[1] >= cfg.heads and z.shape[0] == b.shape[0] == pre.shape[0]
+    assert conv.is_contiguous() and conv.shape[1:] == (cfg.taps, cfg.channels), conv.shape
+    if state is not None:
+        assert state.is_contiguous() and state.shape == (conv.shape[0], cfg.heads, cfg.dim, cfg.vdim), state.shape
+
+
 def delta_prep(buf: dict, cfg, pre, z, b, taps, A_log, dt_bias, conv, rows, cu_q, past_lens, mask_bits, pdl: bool = False) -> None:
     """Short convolutions, unit norms, decays and step sizes of every row into ``buf``."""
     lib = load()
     T = pre.shape[0]
     assert pre.stride(1) == 1 and z.stride(1) == 1 and b.stride(1) == 1 and z.dtype == b.dtype == torch.float32
     assert taps.dtype == pre.dtype == A_log.dtype == dt_bias.dtype == conv.dtype and taps.is_contiguous()
+    _check_delta_pool(cfg, pre, z, b, conv)
     _check(lib.js_delta_prep(
         cfg.heads, cfg.kv_heads, cfg.dim, cfg.vdim, cfg.taps, int(cfg.decay == "channel"), _p(pre), pre.stride(0), _p(z), z.stride(0),
         _p(b), b.stride(0), _p(taps), _p(A_log), _p(dt_bias), _p(conv), _p(rows), _p(cu_q), _p(past_lens), _p(mask_bits),
@@ -983,6 +992,8 @@ def delta_seq(buf: dict, cfg, state, conv, pre, rows, cu_q, past_lens, mask_bits
     """The recurrence over prepared rows: causal (states advance), over token trees (``mask_bits``: nothing is stored), or
     along the rows ``path[:path_len]`` of one sequence (states advance, nothing is read out)."""
     lib = load()
+    assert conv.shape[1:] == (cfg.taps, cfg.channels) and state.shape == (conv.shape[0], cfg.heads, cfg.dim, cfg.vdim)
+    assert conv.is_contiguous() and state.is_contiguous() and state.dtype == torch.float32 and conv.dtype == pre.dtype
     mode = 1 if mask_bits is not None else 2 if path is not None else 0
     B = rows.numel()
     W = mask_bits.shape[1] if mask_bits is not None else 0
@@ -1004,6 +1015,56 @@ def delta_mix(pre, z, b, taps, A_log, dt_bias, cfg, state, conv, rows, cu_q, pas
     delta_prep(buf, cfg, pre, z, b, taps, A_log, dt_bias, conv, rows, cu_q, past_lens, mask)
     delta_seq(buf, cfg, state, conv, pre, rows, cu_q, past_lens, mask)
     return buf["o"]
+
+
+def delta_step_ok(cfg) -> bool:
+    """Whether the one-kernel decode step takes this shape (a head's state fits one CTA's registers)."""
+    groups = 1
+    while 4 * groups < cfg.vdim:
+        groups *= 2
+    return cfg.vdim % 4 == 0 and cfg.vdim <= 256 and cfg.dim <= 256 and cfg.dim * groups <= 4096
+
+
+def delta_blocks_ok(cfg) -> bool:
+    return cfg.vdim % 4 == 0 and cfg.dim <= 128
+
+
+def delta_block_buffers(T: int, B: int, cfg, device) -> dict:
+    """Rows of the block form for ``T`` rows of ``B`` sequences, all fp32."""
+    R, DP, H = 8 * (T // 8 + B), 64 if cfg.dim <= 64 else 128, cfg.heads
+    f = lambda *n: torch.empty(H, *n, dtype=torch.float32, device=device)
+    return {"kt": f(R, DP), "qt": f(R, DP), "kh": f(R, DP), "bv": f(R, cfg.vdim), "pt": f(R, 8), "ge": f(R // 8, DP),
+            "o": torch.empty(T, H, cfg.vdim, dtype=torch.float32, device=device)}
+
+
+def delta_forward(cfg, pre, z, b, taps, A_log, dt_bias, state, conv, rows, cu_q, past_lens, gate, o_norm, kind: str, eps: float, out,
+                  max_rows: int, buffers=None, pdl: bool = False) -> int:
+    """Everything between a delta layer's projections, bf16, causal: one kernel for decode steps (one row a sequence), blocks
+    of 8 rows for portions, the row-by-row kernels for shapes neither takes.  ``buffers(kind)`` hands out the workspace of
+    ``"blocks"`` or ``"rows"``.  Returns the number of kernels launched."""
+    lib = load()
+    T, B = pre.shape[0], rows.numel()
+    get = buffers or (lambda k: delta_block_buffers(T, B, cfg, pre.device) if k == "blocks" else delta_buffers(T, cfg, pre.device))
+    assert pre.dtype == torch.bfloat16 and pre.stride(1) == 1 and z.stride(1) == 1 and b.stride(1) == 1 and gate.stride(1) == 1
+    assert conv.dtype == torch.bfloat16 and state.dtype == torch.float32
+    _check_delta_pool(cfg, pre, z, b, conv, state)
+    head = (cfg.heads, cfg.kv_heads, cfg.dim, cfg.vdim, cfg.taps, int(cfg.decay == "channel"), _p(pre), pre.stride(0), _p(z), z.stride(0),
+            _p(b), b.stride(0), _p(taps), _p(A_log), _p(dt_bias), _p(conv), _p(state), _p(rows), _p(cu_q), _p(past_lens), B)
+    if max_rows == 1 and T == B and delta_step_ok(cfg):
+        _check(lib.js_delta_step(*head, _p(gate), gate.stride(0), _p(o_norm), int(kind == "silu"), ctypes.c_float(eps), _p(out),
+                                 out.stride(0), int(pdl), _stream()), "js_delta_step")
+        return 1
+    if delta_blocks_ok(cfg):
+        w = get("blocks")
+        ncol = 16 if B * cfg.heads * ((cfg.vdim + 31) // 32) < SM_COUNT * 3 // 4 else 32
+        _check(lib.js_delta_blocks(*head, T, *(_p(w[n]) for n in ("kt", "qt", "kh", "bv", "pt", "ge", "o")), ncol, int(pdl), _stream()),
+               "js_delta_blocks")
+    else:
+        w = get("rows")
+        delta_prep(w, cfg, pre, z, b, taps, A_log, dt_bias, conv, rows, cu_q, past_lens, None, pdl=pdl)
+        delta_seq(w, cfg, state, conv, pre, rows, cu_q, past_lens, None, pdl=pdl)
+    gated_head_norm(w["o"], o_norm, gate, kind, eps, out=out, pdl=pdl)
+    return 3
 
 
 def gated_head_norm(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, kind: str, eps: float, out: Optional[torch.Tensor] = None,

@@ -409,8 +409,8 @@ def delta_mix(pre: torch.Tensor, z: torch.Tensor, b: torch.Tensor, taps: torch.T
     """Short convolutions and the gated delta rule over a ragged batch.
 
     ``pre (T, channels)`` are un-convolved q | k | v rows; sequence ``i`` owns rows ``cu_q[i]:cu_q[i+1]``, its state is
-    ``state[rows[i]] (H, D, V)`` and its last convolution inputs ``conv[rows[i]] (taps - 1, channels)``, oldest first.
-    A sequence whose ``past_lens`` is 0 starts from zeros whatever its slot holds.  Causal: tokens follow one another and
+    ``state[rows[i]] (H, D, V)`` and its last convolution inputs the ring ``conv[rows[i]] (taps, channels)``, the row of
+    position ``p`` in entry ``p % taps``.  A sequence whose ``past_lens`` is 0 starts from zeros whatever its slot holds.  Causal: tokens follow one another and
     the states advance.  With ``mask_bits`` (a token tree, parents before children) every node continues its parent's
     state and the stored states stay as they are.  Per head ``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q``.
     Returns the read-outs, fp32 ``(T, H, V)``."""
@@ -422,9 +422,12 @@ def delta_mix(pre: torch.Tensor, z: torch.Tensor, b: torch.Tensor, taps: torch.T
         n = e - s
         if n == 0:
             continue
-        S0, y0 = state[row].clone(), conv[row].to(pre.dtype)
-        if pl[i] == 0:
-            S0, y0 = torch.zeros_like(S0), torch.zeros_like(y0)
+        past, S0 = pl[i], state[row].clone()
+        if past == 0:
+            S0 = torch.zeros_like(S0)
+        y0 = torch.zeros(n_old, pre.shape[1], dtype=pre.dtype, device=pre.device)
+        for m in range(1, min(n_old, past) + 1):
+            y0[n_old - m] = conv[row, (past - m) % taps.shape[1]]
         anc = None if causal else unpack_ancestor_bits(mask_bits[s:e], n).cpu()
         kept = []                                       # per row: state behind it, un-convolved rows up to it
         for t in range(n):
@@ -444,7 +447,9 @@ def delta_mix(pre: torch.Tensor, z: torch.Tensor, b: torch.Tensor, taps: torch.T
             if causal and t:
                 kept[t - 1] = None
         if causal:
-            state[row], conv[row] = kept[-1][0], kept[-1][1].to(conv.dtype)
+            state[row] = kept[-1][0]
+            for t in range(max(0, n - n_old), n):
+                conv[row, (past + t) % taps.shape[1]] = pre[s + t].to(conv.dtype)
     return out
 
 

@@ -3,7 +3,7 @@
 Per recurrent layer::
 
     state : (slots + 1, heads, dim, vdim)      fp32
-    conv  : (slots + 1, taps - 1, channels)    the last inputs of the short convolutions, oldest first
+    conv  : (slots + 1, taps, channels)        ring of the short convolutions' last inputs: position p in entry p % taps
 
 A sequence's slot is its slot-map row in the paged pool.  Nothing is cleared when a slot changes hands: a forward whose
 committed length is 0 starts from zeros whatever the slot holds.  The last slot belongs to no sequence; warm-up launches
@@ -30,7 +30,7 @@ class StatePool:
         self.conv: list = []
         for c in self.shapes:
             self.state.append(None if c is None else torch.zeros(slots + 1, c.heads, c.dim, c.vdim, dtype=torch.float32, device=device))
-            self.conv.append(None if c is None else torch.zeros(slots + 1, c.taps - 1, c.channels, dtype=dtype, device=device))
+            self.conv.append(None if c is None else torch.zeros(slots + 1, c.taps, c.channels, dtype=dtype, device=device))
         self._at: dict = {}          # state slot -> first row of its tree among the held rows
         self._advance = None
         self._held: dict = {}        # layer -> (weights, pre, z, b) of every row of the last tree forward
