@@ -9,8 +9,9 @@
 //              o_i = (e^(c_i) q_i)^T S + sum_m (P T)_im w_m         the only chain left is one matrix product per block
 //              S  <- e^(c_N) S + sum_m (sum_j T_jm e^(c_N - c_j) k_j) w_m^T
 //
-//          A first kernel makes the bracketed rows of all blocks in parallel (with the convolutions and norms); a second one
-//          walks the blocks.  No exponent is ever positive.  All of it is fp32 on the CUDA cores, like the row-by-row kernel.
+//          A first kernel makes the bracketed rows of all blocks in parallel (with the convolutions and norms), in fp32; a
+//          second one walks the blocks with the state in registers.  Its products run on the tensor cores as three tf32
+//          products of split operands each, which keeps 32-bit accuracy; sums are fp32.  No exponent is ever positive.
 #include "common.cuh"
 
 #include <math.h>
@@ -38,16 +39,39 @@ struct DeltaIn {
 };
 
 // silu of the convolution of channel c at local row i of a sequence (rows q0 .., committed length past, ring cs)
+// un-convolved input of channel c at local row i of a sequence (rows q0 .., committed length past, ring cs)
+JS_DEVICE float conv_in(const DeltaIn& p, const __nv_bfloat16* cs, int C, int q0, int past, int i, int c) {
+  if (i >= 0) return __bfloat162float(p.pre[static_cast<size_t>(q0 + i) * p.ldp + c]);
+  return past + i >= 0 ? __bfloat162float(cs[static_cast<size_t>((past + i) % p.taps) * C + c]) : 0.f;
+}
+
+// silu of the convolution of channel c at local row i
 JS_DEVICE float conv_at(const DeltaIn& p, const __nv_bfloat16* cs, int C, int q0, int past, int i, int c) {
   float y = 0.f;
   const __nv_bfloat16* w = p.wt + static_cast<size_t>(c) * p.taps;
-  for (int m = p.taps - 1; m >= 0; --m) {
-    float x = 0.f;
-    if (i - m >= 0) x = __bfloat162float(p.pre[static_cast<size_t>(q0 + i - m) * p.ldp + c]);
-    else if (past + i - m >= 0) x = __bfloat162float(cs[static_cast<size_t>((past + i - m) % p.taps) * C + c]);
-    y += x * __bfloat162float(w[p.taps - 1 - m]);
-  }
+  for (int m = p.taps - 1; m >= 0; --m) y += conv_in(p, cs, C, q0, past, i - m, c) * __bfloat162float(w[p.taps - 1 - m]);
   return df_silu(y);
+}
+
+// the same for rows i0 .. i0 + n - 1 (n <= kBlk; the others give 0), every input loaded once; TP >= taps
+template <int TP>
+JS_DEVICE void conv_rows(const DeltaIn& p, const __nv_bfloat16* cs, int C, int q0, int past, int i0, int n, int c, float (&y)[kBlk]) {
+  float w[TP], x[kBlk + TP - 1];
+  const int skip = TP - p.taps;                 // leading taps of weight 0
+#pragma unroll
+  for (int j = 0; j < TP; ++j) w[j] = j >= skip ? __bfloat162float(p.wt[static_cast<size_t>(c) * p.taps + j - skip]) : 0.f;
+#pragma unroll
+  for (int j = 0; j < kBlk + TP - 1; ++j) {
+    const int i = i0 + j - (TP - 1);
+    x[j] = (j >= skip && i < i0 + n) ? conv_in(p, cs, C, q0, past, i, c) : 0.f;
+  }
+#pragma unroll
+  for (int i = 0; i < kBlk; ++i) {
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < TP; ++j) s += x[i + j] * w[j];
+    y[i] = i < n ? df_silu(s) : 0.f;
+  }
 }
 
 // ================================================================ one row per sequence
@@ -205,7 +229,7 @@ JS_DEVICE void warp_transpose_sum64(float (&v)[64]) {
   }
 }
 
-template <int DP, bool CH>
+template <int DP, bool CH, int TP>
 __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaBlocks o) {
   constexpr int NW = DP / 32;
   __shared__ float part[NW][64], G[64], Tm[64], nrm[NW][16], sbeta[kBlk], sgl[kBlk];
@@ -230,11 +254,11 @@ __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaB
     if (!CH) sgl[d] = ok ? -a * df_softplus(in.z[t * in.ldz + h] + __bfloat162float(in.dt_bias[h])) : 0.f;
   }
   float q[kBlk], k[kBlk], c[kBlk];
+  const int dc = min(d, D - 1), rows_d = d < D ? m_rows : 0;
+  conv_rows<TP>(in, cs, C, q0, past, r0, rows_d, g * D + dc, q);
+  conv_rows<TP>(in, cs, C, q0, past, r0, rows_d, (in.G + g) * D + dc, k);
 #pragma unroll
   for (int i = 0; i < kBlk; ++i) {
-    const bool ok = d < D && i < m_rows;
-    q[i] = ok ? conv_at(in, cs, C, q0, past, r0 + i, g * D + d) : 0.f;
-    k[i] = ok ? conv_at(in, cs, C, q0, past, r0 + i, (in.G + g) * D + d) : 0.f;
     const float sq = warp_sum(q[i] * q[i]), sk = warp_sum(k[i] * k[i]);
     if (lane == 0) { nrm[warp][i] = sq; nrm[warp][8 + i] = sk; }
   }
@@ -257,15 +281,21 @@ __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaB
   }
   // pair sums: P_ij (j <= i) at [i][j], the strict K K^T part (j < i) at [j][i]
   {
-    float v[64];
+    float v[64], kd[kBlk];              // kd[j] = k_j decayed from row j to row i
 #pragma unroll
-    for (int i = 0; i < kBlk; ++i)
+    for (int i = 0; i < kBlk; ++i) {
+      if (CH && i > 0) {
+        const float gi = expf(c[i] - c[i - 1]);
+#pragma unroll
+        for (int j = 0; j < i; ++j) kd[j] *= gi;
+      }
+      kd[i] = k[i];
 #pragma unroll
       for (int j = 0; j <= i; ++j) {
-        const float kj = (CH && j < i) ? k[j] * expf(c[i] - c[j]) : k[j];
-        v[i * 8 + j] = q[i] * kj;
-        if (j < i) v[j * 8 + i] = k[i] * kj;
+        v[i * 8 + j] = q[i] * kd[j];
+        if (j < i) v[j * 8 + i] = k[i] * kd[j];
       }
+    }
     warp_transpose_sum64(v);
     part[warp][2 * lane] = v[0];
     part[warp][2 * lane + 1] = v[1];
@@ -321,9 +351,11 @@ __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaB
     o.kh[(row + m) * DP + d] = s;
   }
   o.ge[(static_cast<size_t>(h) * (o.R / kBlk) + tile) * DP + d] = expf(cn);
-  for (int x = d; x < kBlk * V; x += DP) {
-    const int i = x / V, vc = x % V;
-    o.bv[(row + i) * V + vc] = i < m_rows ? sbeta[i] * conv_at(in, cs, C, q0, past, r0 + i, 2 * in.G * D + h * V + vc) : 0.f;
+  for (int vc = d; vc < V; vc += DP) {
+    float y[kBlk];
+    conv_rows<TP>(in, cs, C, q0, past, r0, m_rows, 2 * in.G * D + h * V + vc, y);
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) o.bv[(row + i) * V + vc] = sbeta[i] * y[i];
   }
 }
 
@@ -334,154 +366,187 @@ JS_DEVICE void df_commit() { asm volatile("cp.async.commit_group;" ::: "memory")
 template <int N>
 JS_DEVICE void df_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-constexpr int kBlkStages = 3;
+constexpr int kBlkStages = 4;
 
-// RL = DP / 8 lanes share two columns: lane r holds the rows 4 r .. + 3 and DP/2 + 4 r .. + 3
-template <int DP, int NCOL>
-__global__ void __launch_bounds__(DP / 8 * NCOL / 2)
+// x = hi + lo in two tf32 numbers (21 significant bits); three products of such halves make a 32-bit product on the
+// tensor cores: a b ~ ahi bhi + ahi blo + alo bhi
+JS_DEVICE void tf32_split(float x, uint32_t& hi, uint32_t& lo) {
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
+  const float rest = x - __uint_as_float(hi);
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(lo) : "f"(rest));
+}
+// d += a b, a 16 x 8 (row), b 8 x 8 (col), fp32 accumulators
+JS_DEVICE void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// The walk over the blocks of one (sequence, head): a CTA holds 16 NV value columns of the state, four warps a quarter of the
+// key dimension each.  A warp keeps its piece TRANSPOSED as the accumulators of 16 (values) x 8 (keys) tiles.  The column
+// order of an accumulator tile differs from the one an A operand wants, but as long as the B operand takes its rows in the
+// same order the sum over them is the same, so the state feeds the next product straight from the accumulators:
+//
+//   per block   [K part | Q part] (values x 8 rows) = S^T [kt | qt]^T   partial sums over the warp's keys, added across warps
+//               W^T = bv^T - K part;  O^T = Q part + W^T pt^T;  S^T = S^T ge + W^T kh
+template <int DP, int NV>
+__global__ void __launch_bounds__(128 * NV)
 delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
-  constexpr int RL = DP / 8, NT = RL * NCOL / 2;
-  struct Stage {
-    float kt[kBlk][DP], qt[kBlk][DP], kh[kBlk][DP], ge[DP], bv[kBlk][NCOL], pt[64];
+  constexpr int NT = DP / 32;                   // key tiles of 8 a warp holds
+  constexpr int LK = DP + 8, LH = DP + 4, LV = 16 * NV + 4;       // row strides without bank conflicts for their readers
+  constexpr int THREADS = 128 * NV;
+  struct __align__(16) Stage {
+    float kt[kBlk][LK], qt[kBlk][LK], kh[kBlk][LH], ge[DP], bv[kBlk][LV], pt[64];
   };
   extern __shared__ __align__(16) uint8_t raw[];
   Stage* sm = reinterpret_cast<Stage*>(raw);
+  float4* part = reinterpret_cast<float4*>(raw + sizeof(Stage) * kBlkStages);      // [2][NV][4 warps][2][32]
   pdl_launch_dependents();
   pdl_wait();
   const int slice = blockIdx.x, h = blockIdx.y, sq = blockIdx.z, tid = threadIdx.x, lane = tid & 31;
+  const int kw = (tid >> 5) & 3, vt = tid >> 7;
+  const int gr = lane >> 2, qd = lane & 3;
   const int q0 = in.cu_q[sq], n = in.cu_q[sq + 1] - q0;
   if (n <= 0) return;
   const int D = in.D, V = in.V, past = in.past_lens[sq], slot = in.rows[sq];
-  const int r = tid % RL, lc = tid / RL * 2, col = slice * NCOL + lc;
   const int tile0 = q0 / kBlk + sq, nb = (n + kBlk - 1) / kBlk;
   const size_t row0 = static_cast<size_t>(h) * o.R + static_cast<size_t>(tile0) * kBlk;
   float* st = state + (static_cast<size_t>(slot) * in.H + h) * D * V;
+  const int v0 = slice * 16 * NV + vt * 16 + gr;          // this lane's value columns: v0 and v0 + 8
+  const int dw = kw * (DP / 4);                           // first key of the warp
 
   auto stage_in = [&](int b) {
     Stage& s = sm[b % kBlkStages];
     const size_t row = row0 + static_cast<size_t>(b) * kBlk;
-    const float* src[3] = {o.kt + row * DP, o.qt + row * DP, o.kh + row * DP};
-    float* dst[3] = {&s.kt[0][0], &s.qt[0][0], &s.kh[0][0]};
-#pragma unroll
-    for (int a = 0; a < 3; ++a)
-      for (int x = tid; x < kBlk * DP / 4; x += NT) df_cp16(dst[a] + 4 * x, src[a] + 4 * x);
+    constexpr int CH = DP / 4;                            // 16-byte chunks of a row
+    for (int x = tid; x < kBlk * CH; x += THREADS) {
+      const int i = x / CH, c = x % CH * 4;
+      df_cp16(&s.kt[i][c], o.kt + (row + i) * DP + c);
+      df_cp16(&s.qt[i][c], o.qt + (row + i) * DP + c);
+      df_cp16(&s.kh[i][c], o.kh + (row + i) * DP + c);
+    }
     const float* ge = o.ge + (static_cast<size_t>(h) * (o.R / kBlk) + tile0 + b) * DP;
-    for (int x = tid; x < DP / 4; x += NT) df_cp16(s.ge + 4 * x, ge + 4 * x);
-    for (int x = tid; x < 16; x += NT) df_cp16(s.pt + 4 * x, o.pt + row * 8 + 4 * x);
-    for (int x = tid; x < kBlk * NCOL / 4; x += NT) {
-      const int i = x / (NCOL / 4), c = x % (NCOL / 4) * 4;
-      if (slice * NCOL + c < V) df_cp16(&s.bv[i][c], o.bv + (row + i) * V + slice * NCOL + c);
+    if (tid < CH) df_cp16(s.ge + 4 * tid, ge + 4 * tid);
+    else if (tid >= 64 && tid < 80) df_cp16(s.pt + 4 * (tid - 64), o.pt + row * 8 + 4 * (tid - 64));
+    else if (tid >= 96 && tid < 128) {
+      for (int x = tid - 96; x < kBlk * 4 * NV; x += 32) {
+        const int i = x / (4 * NV), c = x % (4 * NV) * 4;
+        if (slice * 16 * NV + c < V) df_cp16(&s.bv[i][c], o.bv + (row + i) * V + slice * 16 * NV + c);
+      }
     }
   };
   for (int b = 0; b < kBlkStages - 1; ++b) {
     if (b < nb) stage_in(b);
     df_commit();
   }
-  const bool ok = col < V;              // V is a multiple of 4
-  float S[2][4][2];
+  float S[NT][4];                       // (v0, d), (v0, d + 1), (v0 + 8, d), (v0 + 8, d + 1), d = dw + 8 nt + 2 qd
 #pragma unroll
-  for (int ch = 0; ch < 2; ++ch)
+  for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = ch * (DP / 2) + 4 * r + e;
-      const float2 v = (past > 0 && ok && d < D) ? *reinterpret_cast<const float2*>(st + static_cast<size_t>(d) * V + col) : make_float2(0.f, 0.f);
-      S[ch][e][0] = v.x;
-      S[ch][e][1] = v.y;
+      const int d = dw + 8 * nt + 2 * qd + (e & 1), v = v0 + (e >> 1) * 8;
+      S[nt][e] = (past > 0 && d < D && v < V) ? st[static_cast<size_t>(d) * V + v] : 0.f;
     }
-  const int i_own = r & 7;              // the row whose sums this lane ends up with
   for (int b = 0; b < nb; ++b) {
     df_wait<kBlkStages - 2>();
     __syncthreads();
     if (b + kBlkStages - 1 < nb) stage_in(b + kBlkStages - 1);
     df_commit();
     const Stage& s = sm[b % kBlkStages];
-    float acc[2][kBlk][2];              // [k or q][row][column]
+    float ak[3][4] = {}, aq[3][4] = {};
 #pragma unroll
-    for (int i = 0; i < kBlk; ++i) {
-      acc[0][i][0] = acc[0][i][1] = acc[1][i][0] = acc[1][i][1] = 0.f;
-#pragma unroll
-      for (int ch = 0; ch < 2; ++ch) {
-        const float4 kv = *reinterpret_cast<const float4*>(&s.kt[i][ch * (DP / 2) + 4 * r]);
-        const float4 qv = *reinterpret_cast<const float4*>(&s.qt[i][ch * (DP / 2) + 4 * r]);
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          acc[0][i][c] += S[ch][0][c] * kv.x + S[ch][1][c] * kv.y + S[ch][2][c] * kv.z + S[ch][3][c] * kv.w;
-          acc[1][i][c] += S[ch][0][c] * qv.x + S[ch][1][c] * qv.y + S[ch][2][c] * qv.z + S[ch][3][c] * qv.w;
-        }
-      }
+    for (int nt = 0; nt < NT; ++nt) {
+      const int d = dw + 8 * nt + 2 * qd;
+      const float2 kv = *reinterpret_cast<const float2*>(&s.kt[gr][d]);
+      const float2 qv = *reinterpret_cast<const float2*>(&s.qt[gr][d]);
+      uint32_t ah[4], al[4], kh0, kl0, kh1, kl1, qh0, ql0, qh1, ql1;
+      tf32_split(S[nt][0], ah[0], al[0]);
+      tf32_split(S[nt][2], ah[1], al[1]);
+      tf32_split(S[nt][1], ah[2], al[2]);
+      tf32_split(S[nt][3], ah[3], al[3]);
+      tf32_split(kv.x, kh0, kl0);
+      tf32_split(kv.y, kh1, kl1);
+      tf32_split(qv.x, qh0, ql0);
+      tf32_split(qv.y, qh1, ql1);
+      mma_tf32(ak[0], ah, kh0, kh1);
+      mma_tf32(ak[1], ah, kl0, kl1);
+      mma_tf32(ak[2], al, kh0, kh1);
+      mma_tf32(aq[0], ah, qh0, qh1);
+      mma_tf32(aq[1], ah, ql0, ql1);
+      mma_tf32(aq[2], al, qh0, qh1);
     }
-    // sums over the RL lanes, halving what every lane keeps: the low three lane bits choose the row, the others sum
-#pragma unroll
-    for (int bit = 4, half = 4; bit > 0; bit >>= 1, half >>= 1) {
-      const bool hi = (r & bit) != 0;
-#pragma unroll
-      for (int t = 0; t < 2; ++t)
-#pragma unroll
-        for (int j = 0; j < half; ++j)
-#pragma unroll
-          for (int c = 0; c < 2; ++c) {
-            const float send = hi ? acc[t][j][c] : acc[t][j + half][c];
-            const float keep = hi ? acc[t][j + half][c] : acc[t][j][c];
-            acc[t][j][c] = keep + __shfl_xor_sync(0xffffffffu, send, bit);
-          }
+    float4* pb = part + ((b & 1) * NV + vt) * 256;
+    pb[kw * 64 + lane] = make_float4(ak[0][0] + (ak[1][0] + ak[2][0]), ak[0][1] + (ak[1][1] + ak[2][1]),
+                                     ak[0][2] + (ak[1][2] + ak[2][2]), ak[0][3] + (ak[1][3] + ak[2][3]));
+    pb[kw * 64 + 32 + lane] = make_float4(aq[0][0] + (aq[1][0] + aq[2][0]), aq[0][1] + (aq[1][1] + aq[2][1]),
+                                          aq[0][2] + (aq[1][2] + aq[2][2]), aq[0][3] + (aq[1][3] + aq[2][3]));
+    __syncthreads();
+    float W[4];                         // (v0, m), (v0, m + 1), (v0 + 8, m), (v0 + 8, m + 1), m = 2 qd
+    {
+      const float4 p0 = pb[lane], p1 = pb[64 + lane], p2 = pb[128 + lane], p3 = pb[192 + lane];
+      const int c = vt * 16 + gr;
+      W[0] = s.bv[2 * qd][c] - ((p0.x + p1.x) + (p2.x + p3.x));
+      W[1] = s.bv[2 * qd + 1][c] - ((p0.y + p1.y) + (p2.y + p3.y));
+      W[2] = s.bv[2 * qd][c + 8] - ((p0.z + p1.z) + (p2.z + p3.z));
+      W[3] = s.bv[2 * qd + 1][c + 8] - ((p0.w + p1.w) + (p2.w + p3.w));
     }
-    float dk[2], dq[2];
+    uint32_t wh[4], wl[4];
+    tf32_split(W[0], wh[0], wl[0]);
+    tf32_split(W[2], wh[1], wl[1]);
+    tf32_split(W[1], wh[2], wl[2]);
+    tf32_split(W[3], wh[3], wl[3]);
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
-      dk[c] = acc[0][0][c];
-      dq[c] = acc[1][0][c];
+    for (int nt = 0; nt < NT; ++nt) {
+      const int d = dw + 8 * nt;
+      const float2 gv = *reinterpret_cast<const float2*>(&s.ge[d + 2 * qd]);
+      const float k0 = s.kh[2 * qd][d + gr], k1 = s.kh[2 * qd + 1][d + gr];
+      uint32_t h0, l0, h1, l1;
+      tf32_split(k0, h0, l0);
+      tf32_split(k1, h1, l1);
+      float low[4] = {};
+      S[nt][0] *= gv.x;
+      S[nt][1] *= gv.y;
+      S[nt][2] *= gv.x;
+      S[nt][3] *= gv.y;
+      mma_tf32(low, wh, l0, l1);
+      mma_tf32(low, wl, h0, h1);
+      mma_tf32(S[nt], wh, h0, h1);
 #pragma unroll
-      for (int bit = 8; bit < RL; bit <<= 1) {
-        dk[c] += __shfl_xor_sync(0xffffffffu, dk[c], bit);
-        dq[c] += __shfl_xor_sync(0xffffffffu, dq[c], bit);
-      }
+      for (int e = 0; e < 4; ++e) S[nt][e] += low[e];
     }
-    float W[kBlk][2];
-    const int base = lane & ~(RL - 1);
+    if (kw == (b & 3)) {                // the warps take turns with the read-outs
+      const float4 p0 = pb[32 + lane], p1 = pb[96 + lane], p2 = pb[160 + lane], p3 = pb[224 + lane];
+      float O[4] = {(p0.x + p1.x) + (p2.x + p3.x), (p0.y + p1.y) + (p2.y + p3.y), (p0.z + p1.z) + (p2.z + p3.z),
+                    (p0.w + p1.w) + (p2.w + p3.w)};
+      const float2 pv = *reinterpret_cast<const float2*>(&s.pt[gr * 8 + 2 * qd]);
+      uint32_t h0, l0, h1, l1;
+      tf32_split(pv.x, h0, l0);
+      tf32_split(pv.y, h1, l1);
+      float low[4] = {};
+      mma_tf32(low, wh, l0, l1);
+      mma_tf32(low, wl, h0, h1);
+      mma_tf32(O, wh, h0, h1);
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
-      const float w = s.bv[i_own][lc + c] - dk[c];
-#pragma unroll
-      for (int m = 0; m < kBlk; ++m) W[m][c] = __shfl_sync(0xffffffffu, w, base + m);
-    }
-    if (r < kBlk && ok && b * kBlk + i_own < n) {
-#pragma unroll
-      for (int c = 0; c < 2; ++c)
-#pragma unroll
-        for (int m = 0; m < kBlk; ++m) dq[c] += s.pt[i_own * 8 + m] * W[m][c];
-      *reinterpret_cast<float2*>(out + (static_cast<size_t>(q0 + b * kBlk + i_own) * in.H + h) * V + col) = make_float2(dq[0], dq[1]);
-    }
-#pragma unroll
-    for (int ch = 0; ch < 2; ++ch) {
-      const float4 gv = *reinterpret_cast<const float4*>(&s.ge[ch * (DP / 2) + 4 * r]);
-#pragma unroll
-      for (int c = 0; c < 2; ++c) { S[ch][0][c] *= gv.x; S[ch][1][c] *= gv.y; S[ch][2][c] *= gv.z; S[ch][3][c] *= gv.w; }
-#pragma unroll
-      for (int m = 0; m < kBlk; ++m) {
-        const float4 kv = *reinterpret_cast<const float4*>(&s.kh[m][ch * (DP / 2) + 4 * r]);
-#pragma unroll
-        for (int c = 0; c < 2; ++c) {
-          S[ch][0][c] += kv.x * W[m][c];
-          S[ch][1][c] += kv.y * W[m][c];
-          S[ch][2][c] += kv.z * W[m][c];
-          S[ch][3][c] += kv.w * W[m][c];
-        }
+      for (int e = 0; e < 4; ++e) {
+        const int i = b * kBlk + 2 * qd + (e & 1), v = v0 + (e >> 1) * 8;
+        if (i < n && v < V) out[(static_cast<size_t>(q0 + i) * in.H + h) * V + v] = O[e] + low[e];
       }
     }
   }
 #pragma unroll
-  for (int ch = 0; ch < 2; ++ch)
+  for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = ch * (DP / 2) + 4 * r + e;
-      if (ok && d < D) *reinterpret_cast<float2*>(st + static_cast<size_t>(d) * V + col) = make_float2(S[ch][e][0], S[ch][e][1]);
+      const int d = dw + 8 * nt + 2 * qd + (e & 1), v = v0 + (e >> 1) * 8;
+      if (d < D && v < V) st[static_cast<size_t>(d) * V + v] = S[nt][e];
     }
   // the last rows' convolution inputs; every reader of the ring ran in the kernel before
   if (in.taps > 1) {
+    constexpr int NCOL = 16 * NV;
     const int C = 2 * in.G * D + in.H * V, g = h / (in.H / in.G);
     const int qk = slice == 0 && h % (in.H / in.G) == 0 ? 2 * D : 0;
     __nv_bfloat16* ring = in.conv + static_cast<size_t>(slot) * in.taps * C;
-    for (int x = tid; x < NCOL + qk; x += NT) {
+    for (int x = tid; x < NCOL + qk; x += THREADS) {
       if (x < NCOL && slice * NCOL + x >= V) continue;
       const int y = x - NCOL;
       const int c = x < NCOL ? 2 * in.G * D + h * V + slice * NCOL + x : y < D ? g * D + y : (in.G + g) * D + y - D;
@@ -506,21 +571,22 @@ struct FusedLaunch {
   }
 };
 
-template <int DP, int NCOL>
+template <int DP, int NV>
 static int launch_blocks(const DeltaIn& in, const DeltaBlocks& o, float* state, float* out, int pdl, cudaStream_t stream) {
-  constexpr int smem = kBlkStages * (3 * kBlk * DP + DP + kBlk * NCOL + 64) * 4;
+  constexpr int smem = kBlkStages * (kBlk * (3 * DP + 20 + 16 * NV + 4) + DP + 64) * 4 + 2 * NV * 256 * 16;
   static int configured[kMaxDevicesCached] = {};
-  auto kern = delta_block_kernel<DP, NCOL>;
+  auto kern = delta_block_kernel<DP, NV>;
   if (ensure_dyn_smem(kern, smem, configured) != 0) return -3;
-  FusedLaunch l(dim3((in.V + NCOL - 1) / NCOL, in.H, in.B), dim3(DP / 8 * NCOL / 2), stream, pdl, smem);
+  FusedLaunch l(dim3((in.V + 16 * NV - 1) / (16 * NV), in.H, in.B), dim3(128 * NV), stream, pdl, smem);
   return cudaLaunchKernelEx(&l.c, kern, in, o, state, out) == cudaSuccess ? 0 : -4;
 }
 
 template <int DP>
 static int launch_block_prep(const DeltaIn& in, const DeltaBlocks& o, int tiles, int pdl, cudaStream_t stream) {
   FusedLaunch l(dim3(tiles, in.H), dim3(DP), stream, pdl);
-  return (in.channel ? cudaLaunchKernelEx(&l.c, delta_block_prep_kernel<DP, true>, in, o)
-                     : cudaLaunchKernelEx(&l.c, delta_block_prep_kernel<DP, false>, in, o)) == cudaSuccess ? 0 : -4;
+  auto kern = in.channel ? (in.taps <= 4 ? delta_block_prep_kernel<DP, true, 4> : delta_block_prep_kernel<DP, true, kBlkMaxTaps>)
+                         : (in.taps <= 4 ? delta_block_prep_kernel<DP, false, 4> : delta_block_prep_kernel<DP, false, kBlkMaxTaps>);
+  return cudaLaunchKernelEx(&l.c, kern, in, o) == cudaSuccess ? 0 : -4;
 }
 
 static bool fused_shape_ok(int H, int G, int D, int V, int taps) {
@@ -569,8 +635,8 @@ extern "C" int js_delta_blocks(int H, int G, int D, int V, int ntaps, int channe
   const DeltaBlocks o{kt, qt, kh, bv, pt, ge, tiles * kBlk};
   if (D <= 64) {
     if (int rc = launch_block_prep<64>(in, o, tiles, pdl, stream)) return rc;
-    return ncol == 16 ? launch_blocks<64, 16>(in, o, state, out, pdl, stream) : launch_blocks<64, 32>(in, o, state, out, pdl, stream);
+    return ncol == 16 ? launch_blocks<64, 1>(in, o, state, out, pdl, stream) : launch_blocks<64, 2>(in, o, state, out, pdl, stream);
   }
   if (int rc = launch_block_prep<128>(in, o, tiles, pdl, stream)) return rc;
-  return ncol == 16 ? launch_blocks<128, 16>(in, o, state, out, pdl, stream) : launch_blocks<128, 32>(in, o, state, out, pdl, stream);
+  return ncol == 16 ? launch_blocks<128, 1>(in, o, state, out, pdl, stream) : launch_blocks<128, 2>(in, o, state, out, pdl, stream);
 }

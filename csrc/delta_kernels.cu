@@ -398,6 +398,46 @@ gated_head_norm_kernel(const float* o, const E* w, const E* gate, int ldg, E* ou
   }
 }
 
+// the same for V a multiple of 4 up to 256 and Vp = V, four columns a lane and one pass over memory
+__global__ void __launch_bounds__(256)
+gated_head_norm_vec_kernel(const float* o, const __nv_bfloat16* w, const __nv_bfloat16* gate, int ldg, __nv_bfloat16* out, int ldo, int T, int H,
+                           int V, int silu, float eps) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int u = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (u >= T * H) return;
+  const int t = u / H, h = u % H;
+  const float4* src = reinterpret_cast<const float4*>(o + static_cast<size_t>(u) * V);
+  float4 y[2];
+  uint2 zr[2];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int d = 4 * (lane + 32 * j);
+    y[j] = d < V ? src[d / 4] : make_float4(0.f, 0.f, 0.f, 0.f);
+    zr[j] = d < V ? *reinterpret_cast<const uint2*>(gate + static_cast<size_t>(t) * ldg + h * V + d) : make_uint2(0u, 0u);
+  }
+#pragma unroll
+  for (int j = 0; j < 2; ++j) ss += y[j].x * y[j].x + y[j].y * y[j].y + y[j].z * y[j].z + y[j].w * y[j].w;
+  const float r = 1.f / sqrtf(warp_sum(ss) / V + eps);
+#pragma unroll
+  for (int j = 0; j < 2; ++j) {
+    const int d = 4 * (lane + 32 * j);
+    if (d >= V) continue;
+    const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&zr[j]);
+    const uint2 wr = *reinterpret_cast<const uint2*>(w + d);
+    const __nv_bfloat162* w2 = reinterpret_cast<const __nv_bfloat162*>(&wr);
+    const float2 za = __bfloat1622float2(z2[0]), zb = __bfloat1622float2(z2[1]);
+    const float2 wa = __bfloat1622float2(w2[0]), wb = __bfloat1622float2(w2[1]);
+    auto act = [&](float z) { return silu ? dl_silu(z) : dl_sigmoid(z); };
+    uint2 pk;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&pk);
+    o2[0] = __floats2bfloat162_rn(y[j].x * r * wa.x * act(za.x), y[j].y * r * wa.y * act(za.y));
+    o2[1] = __floats2bfloat162_rn(y[j].z * r * wb.x * act(zb.x), y[j].w * r * wb.y * act(zb.y));
+    *reinterpret_cast<uint2*>(out + static_cast<size_t>(t) * ldo + h * V + d) = pk;
+  }
+}
+
 struct DeltaLaunch {
   cudaLaunchConfig_t c = {};
   cudaLaunchAttribute a;
@@ -471,6 +511,10 @@ extern "C" int js_gated_head_norm(const float* o, const void* w, const void* gat
   if (T <= 0) return 0;
   DeltaLaunch l(dim3((T * H + 7) / 8), dim3(256), stream, pdl);
   using bf = __nv_bfloat16;
+  const bool aligned = !((reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(out)) & 7) &&
+                       !(reinterpret_cast<uintptr_t>(o) & 15);
+  if (bf16 && V == Vp && V % 4 == 0 && V <= 256 && ldg % 4 == 0 && ldo % 4 == 0 && aligned)
+    return cudaLaunchKernelEx(&l.c, gated_head_norm_vec_kernel, o, (const bf*)w, (const bf*)gate, ldg, (bf*)out, ldo, T, H, V, silu, eps) == cudaSuccess ? 0 : -4;
   const cudaError_t e =
       bf16 ? cudaLaunchKernelEx(&l.c, gated_head_norm_kernel<bf>, o, (const bf*)w, (const bf*)gate, ldg, (bf*)out, ldo, T, H, V, Vp, silu, eps)
            : cudaLaunchKernelEx(&l.c, gated_head_norm_kernel<float>, o, (const float*)w, (const float*)gate, ldg, (float*)out, ldo, T, H, V,

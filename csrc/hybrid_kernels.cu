@@ -249,7 +249,7 @@ struct ResidParams {
   int ld, ldt, W;
 };
 
-constexpr int kResidThreads = 512;
+constexpr int kResidThreads = 512;      // few rows (decode) want many threads a row
 
 __global__ void __launch_bounds__(kResidThreads) resid_norm_kernel(ResidParams p) {
   extern __shared__ float ry[];            // W
@@ -260,24 +260,22 @@ __global__ void __launch_bounds__(kResidThreads) resid_norm_kernel(ResidParams p
   float ss = 0.f;
   if (p.ya == nullptr) {
     const float wt = p.k > 0 ? 1.f / p.k : 0.f;
-    for (int c = tid * 2; c < W; c += kResidThreads * 2) {        // W even (padded): bf16 pairs
-      float2 acc = make_float2(0.f, 0.f);
-      for (int j = 0; j < p.k; ++j) {
-        const int r = p.inv[t * p.k + j];
-        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.ys + static_cast<size_t>(r) * p.ldy + c));
-        acc.x += f.x;
-        acc.y += f.y;
-      }
-      acc.x *= wt;
-      acc.y *= wt;
-      if (p.sh != nullptr) {
-        const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p.sh + static_cast<size_t>(t) * p.lds + c));
-        acc.x += f.x;
-        acc.y += f.y;
-      }
-      ry[c] = acc.x;
-      ss += acc.x * acc.x;
-      if (c + 1 < W) { ry[c + 1] = acc.y; ss += acc.y * acc.y; }
+    for (int c = tid * 4; c < W; c += kResidThreads * 4) {        // rows are padded to multiples of 4
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+      auto add = [&](const __nv_bfloat16* row) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(row + c);
+        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        acc[0] += lo.x; acc[1] += lo.y; acc[2] += hi.x; acc[3] += hi.y;
+      };
+#pragma unroll 4
+      for (int j = 0; j < p.k; ++j) add(p.ys + static_cast<size_t>(p.inv[t * p.k + j]) * p.ldy);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[e] *= wt;
+      if (p.sh != nullptr) add(p.sh + static_cast<size_t>(t) * p.lds);
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + e < W) { ry[c + e] = acc[e]; ss += acc[e] * acc[e]; }
     }
   } else {
     const __nv_bfloat16* a = p.ya + static_cast<size_t>(t) * p.lda;
@@ -359,63 +357,75 @@ struct TableLayer {
   int off_tok;           // where this layer's outputs start in `out`: per pass [tok | inv | group offsets]
 };
 
-constexpr int kTableThreads = 1024;
+constexpr int kTableWarps = 32;
 
-__global__ void __launch_bounds__(kTableThreads)
+__global__ void __launch_bounds__(32 * kTableWarps)
 table_sort_kernel(const TableLayer* layers, const int* ids, int T, int rows_per_pass, int V, int* out) {
   extern __shared__ int sh[];
+  __shared__ int warp_tot[kTableWarps];
   pdl_launch_dependents();
   pdl_wait();
   const TableLayer L = layers[blockIdx.x];
   const int t0 = blockIdx.y * rows_per_pass;
   const int n = min(rows_per_pass, T - t0);
   if (n <= 0) return;
-  const int P = n * L.top;
-  int* key = sh;                 // P
-  int* cnt = sh + P;             // E + 1
-  int* tok = out + L.off_tok + static_cast<size_t>(t0) * 2 * L.top + static_cast<size_t>(blockIdx.y) * (L.E + 1);
+  const int P = n * L.top, E = L.E, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  int* cnt = sh;                 // (warps, E): pairs of the warp's chunk per expert, then where the warp's next one goes
+  unsigned short* key = reinterpret_cast<unsigned short*>(sh + kTableWarps * E);      // P
+  int* tok = out + L.off_tok + static_cast<size_t>(t0) * 2 * L.top + static_cast<size_t>(blockIdx.y) * (E + 1);
   int* inv = tok + P;
   int* goff = inv + P;
-  for (int i = threadIdx.x; i <= L.E; i += blockDim.x) cnt[i] = 0;
+  for (int i = tid; i < kTableWarps * E; i += blockDim.x) cnt[i] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < P; p += blockDim.x) {
+  // every warp takes a consecutive chunk of the pairs, so that the order within an expert is the pairs' own
+  const int chunk = ((P + kTableWarps - 1) / kTableWarps + 31) / 32 * 32;
+  const int p0 = warp * chunk, p1 = min(P, p0 + chunk);
+  int* mine = cnt + warp * E;
+  for (int p = p0 + lane; p < p1; p += 32) {
     int id = ids[t0 + p / L.top];
     id = id < 0 ? 0 : (id >= V ? V - 1 : id);
     const int e = L.table[static_cast<size_t>(id) * L.top + p % L.top];
-    key[p] = e;
-    atomicAdd(&cnt[e], 1);
+    key[p] = static_cast<unsigned short>(e);
+    atomicAdd(&mine[e], 1);
   }
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if (warp == 0) {               // exclusive scan
-    int run = 0;
-    for (int i0 = 0; i0 <= L.E; i0 += 32) {
-      const int i = i0 + lane, c = i < L.E ? cnt[i] : 0;
-      int inc = c;
+  // exclusive scan over (expert, warp): thread e owns expert e (E <= 1024)
+  int total = 0;
+  if (tid < E)
+    for (int w = 0; w < kTableWarps; ++w) total += cnt[w * E + tid];
+  int inc = total;
 #pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const int v = __shfl_up_sync(0xffffffffu, inc, o);
-        if (lane >= o) inc += v;
-      }
-      if (i <= L.E) { cnt[i] = run + inc - c; goff[i] = run + inc - c; }
-      run += __shfl_sync(0xffffffffu, inc, 31);
+  for (int o = 1; o < 32; o <<= 1) {
+    const int v = __shfl_up_sync(0xffffffffu, inc, o);
+    if (lane >= o) inc += v;
+  }
+  if (lane == 31) warp_tot[warp] = inc;
+  __syncthreads();
+  int base = inc - total;
+  for (int w = 0; w < warp; ++w) base += warp_tot[w];
+  if (tid < E) {
+    goff[tid] = base;
+    for (int w = 0; w < kTableWarps; ++w) {
+      const int c = cnt[w * E + tid];
+      cnt[w * E + tid] = base;
+      base += c;
     }
   }
+  if (tid == 0) goff[E] = P;
   __syncthreads();
-  for (int e = warp; e < L.E; e += kTableThreads / 32) {
-    int base = cnt[e];
-    const int end = cnt[e + 1];
-    for (int p0 = 0; p0 < P && base < end; p0 += 32) {
-      const int p = p0 + lane;
-      const bool mine = p < P && key[p] == e;
-      const unsigned m = __ballot_sync(0xffffffffu, mine);
-      if (mine) {
-        const int pos = base + __popc(m & ((1u << lane) - 1u));
-        tok[pos] = t0 + p / L.top;
-        inv[p] = pos;
-      }
-      base += __popc(m);
+  for (int pb = p0; pb < p1; pb += 32) {
+    const int p = pb + lane;
+    const int e = p < p1 ? key[p] : -1;
+    const unsigned same = __match_any_sync(0xffffffffu, e);
+    const int rank = __popc(same & ((1u << lane) - 1u));
+    const int at = e >= 0 ? mine[e] + rank : 0;
+    __syncwarp();
+    if (e >= 0) {
+      tok[at] = t0 + p / L.top;
+      inv[p] = at;
+      if (rank == 0) mine[e] += __popc(same);
     }
+    __syncwarp();
   }
 }
 
@@ -468,14 +478,14 @@ extern "C" int js_window_attention_simt(const void* q, long long q_tok, const vo
                                           D, V, S, max_len, W, causal, scale, window, sink, status, pdl, stream);
 }
 
-// Either ya (with yb, wa, wb for a pair; bias optional) or ys / inv / k and sh, all bf16 rows of even
-// length >= W.  W at most 24576.
+// Either ya (with yb, wa, wb for a pair; bias optional) or ys / inv / k and sh, all bf16 rows whose
+// length is a multiple of 2 (ys, sh: 4) and >= W.  W at most 24576.
 extern "C" int js_resid_norm(const void* ya, int lda, const float* bias, const float* wa, const void* yb, int ldb, const float* wb,
                              const void* ys, int ldy, const int* inv, int k, const void* sh, int lds, const float* w, const float* fw,
                              float eps, float* x, void* h, int ld, void* tap, int ldt, int T, int W, int pdl, cudaStream_t stream) {
   using namespace js;
   if (T <= 0) return 0;
-  if (W < 1 || W > 24576 || ((lda | ldb | ldy | lds) & 1)) return -10;
+  if (W < 1 || W > 24576 || ((lda | ldb) & 1) || ((ldy | lds) & 3)) return -10;
   if (ya == nullptr && ys == nullptr && sh == nullptr) return -13;
   if (yb != nullptr && (wa == nullptr || wb == nullptr)) return -13;
   using bf = __nv_bfloat16;
@@ -503,9 +513,9 @@ extern "C" int js_table_sort(const void* layers, int n_layers, const int* ids, i
   if (T <= 0 || n_layers <= 0) return 0;
   if (rows_per_pass < 1 || max_top < 1 || rows_per_pass * max_top > 16384 || max_E < 1 || max_E > 1024) return -10;
   const int rows = T < rows_per_pass ? T : rows_per_pass;
-  const int smem = (rows * max_top + max_E + 1) * 4;
+  const int smem = kTableWarps * max_E * 4 + rows * max_top * 2;
   static int configured[kMaxDevicesCached] = {};
   if (ensure_dyn_smem(table_sort_kernel, smem, configured) != 0) return -3;
-  HybridLaunch l(dim3(n_layers, (T + rows_per_pass - 1) / rows_per_pass), dim3(kTableThreads), stream, pdl, smem);
+  HybridLaunch l(dim3(n_layers, (T + rows_per_pass - 1) / rows_per_pass), dim3(32 * kTableWarps), stream, pdl, smem);
   return cudaLaunchKernelEx(&l.c, table_sort_kernel, (const TableLayer*)layers, ids, T, rows_per_pass, V, out) == cudaSuccess ? 0 : -4;
 }
