@@ -22,6 +22,8 @@ JS_DEVICE float df_ld(const float* p) { return *p; }
 JS_DEVICE float df_ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
 JS_DEVICE float df_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 JS_DEVICE float df_silu(float z) { return z / (1.f + expf(-z)); }
+// the activation behind a convolution: its input is a bf16 projection, so the fast exponential's error does not show
+JS_DEVICE float df_silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 JS_DEVICE float df_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 
 constexpr int kBlk = 8;
@@ -50,7 +52,7 @@ JS_DEVICE float conv_at(const DeltaIn& p, const __nv_bfloat16* cs, int C, int q0
   float y = 0.f;
   const __nv_bfloat16* w = p.wt + static_cast<size_t>(c) * p.taps;
   for (int m = p.taps - 1; m >= 0; --m) y += conv_in(p, cs, C, q0, past, i - m, c) * __bfloat162float(w[p.taps - 1 - m]);
-  return df_silu(y);
+  return df_silu_fast(y);
 }
 
 // the same for rows i0 .. i0 + n - 1 (n <= kBlk; the others give 0), every input loaded once; TP >= taps
@@ -60,17 +62,25 @@ JS_DEVICE void conv_rows(const DeltaIn& p, const __nv_bfloat16* cs, int C, int q
   const int skip = TP - p.taps;                 // leading taps of weight 0
 #pragma unroll
   for (int j = 0; j < TP; ++j) w[j] = j >= skip ? __bfloat162float(p.wt[static_cast<size_t>(c) * p.taps + j - skip]) : 0.f;
+  if (i0 >= TP - 1) {
+    // all rows belong to this batch: plain loads that overlap (rows past the end repeat the last one and are dropped below)
+    const __nv_bfloat16* src = p.pre + static_cast<size_t>(q0 + i0 - (TP - 1)) * p.ldp + c;
+    const int last = TP - 2 + max(n, 1);
 #pragma unroll
-  for (int j = 0; j < kBlk + TP - 1; ++j) {
-    const int i = i0 + j - (TP - 1);
-    x[j] = (j >= skip && i < i0 + n) ? conv_in(p, cs, C, q0, past, i, c) : 0.f;
+    for (int j = 0; j < kBlk + TP - 1; ++j) x[j] = __bfloat162float(src[static_cast<size_t>(min(j, last)) * p.ldp]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < kBlk + TP - 1; ++j) {
+      const int i = i0 + j - (TP - 1);
+      x[j] = (j >= skip && i < i0 + n) ? conv_in(p, cs, C, q0, past, i, c) : 0.f;
+    }
   }
 #pragma unroll
   for (int i = 0; i < kBlk; ++i) {
     float s = 0.f;
 #pragma unroll
     for (int j = 0; j < TP; ++j) s += x[i + j] * w[j];
-    y[i] = i < n ? df_silu(s) : 0.f;
+    y[i] = i < n ? df_silu_fast(s) : 0.f;
   }
 }
 
@@ -214,17 +224,23 @@ struct DeltaBlocks {
   int R;
 };
 
-// lane l ends with the sums over the warp of entries 2 l and 2 l + 1
-JS_DEVICE void warp_transpose_sum64(float (&v)[64]) {
+// sums over the warp of N values, halving what every lane keeps: N = 64 leaves entries 2 l and 2 l + 1 in v[0], v[1] of lane l,
+// N = 16 entry l / 2 in v[0]
+template <int N>
+JS_DEVICE void warp_transpose_sum(float (&v)[N]) {
   const int lane = threadIdx.x & 31;
 #pragma unroll
-  for (int b = 16, half = 32; b > 0; b >>= 1, half >>= 1) {
+  for (int b = 16, half = N / 2; b > 0; b >>= 1, half >>= 1) {
     const bool hi = (lane & b) != 0;
+    if (half > 0) {
 #pragma unroll
-    for (int j = 0; j < half; ++j) {
-      const float send = hi ? v[j] : v[j + half];
-      const float keep = hi ? v[j + half] : v[j];
-      v[j] = keep + __shfl_xor_sync(0xffffffffu, send, b);
+      for (int j = 0; j < half; ++j) {
+        const float send = hi ? v[j] : v[j + half];
+        const float keep = hi ? v[j + half] : v[j];
+        v[j] = keep + __shfl_xor_sync(0xffffffffu, send, b);
+      }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], b);
     }
   }
 }
@@ -232,7 +248,7 @@ JS_DEVICE void warp_transpose_sum64(float (&v)[64]) {
 template <int DP, bool CH, int TP>
 __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaBlocks o) {
   constexpr int NW = DP / 32;
-  __shared__ float part[NW][64], G[64], Tm[64], nrm[NW][16], sbeta[kBlk], sgl[kBlk];
+  __shared__ float part[NW][64], G[64], Tm[64], nrm[NW][16], sbeta[kBlk], sg[kBlk];
   pdl_launch_dependents();
   pdl_wait();
   const int h = blockIdx.y, tile = blockIdx.x, d = threadIdx.x, warp = d >> 5, lane = d & 31;
@@ -251,66 +267,87 @@ __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaB
     const bool ok = d < m_rows;
     const size_t t = q0 + r0 + (ok ? d : 0);
     sbeta[d] = ok ? df_sigmoid(in.b[t * in.ldb + h]) : 0.f;
-    if (!CH) sgl[d] = ok ? -a * df_softplus(in.z[t * in.ldz + h] + __bfloat162float(in.dt_bias[h])) : 0.f;
+    if (!CH) sg[d] = ok ? expf(-a * df_softplus(in.z[t * in.ldz + h] + __bfloat162float(in.dt_bias[h]))) : 1.f;
   }
-  float q[kBlk], k[kBlk], c[kBlk];
+  float q[kBlk], k[kBlk], v[kBlk], gd[kBlk];
   const int dc = min(d, D - 1), rows_d = d < D ? m_rows : 0;
   conv_rows<TP>(in, cs, C, q0, past, r0, rows_d, g * D + dc, q);
   conv_rows<TP>(in, cs, C, q0, past, r0, rows_d, (in.G + g) * D + dc, k);
+  conv_rows<TP>(in, cs, C, q0, past, r0, d < V ? m_rows : 0, 2 * in.G * D + h * V + min(d, V - 1), v);
+  if (CH) {
 #pragma unroll
-  for (int i = 0; i < kBlk; ++i) {
-    const float sq = warp_sum(q[i] * q[i]), sk = warp_sum(k[i] * k[i]);
-    if (lane == 0) { nrm[warp][i] = sq; nrm[warp][8 + i] = sk; }
+    for (int i = 0; i < kBlk; ++i) gd[i] = in.z[static_cast<size_t>(q0 + r0 + min(i, m_rows - 1)) * in.ldz + h * D + dc];
+    const float dt = __bfloat162float(in.dt_bias[h * D + dc]);
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) gd[i] = (d < D && i < m_rows) ? expf(-a * df_softplus(gd[i] + dt)) : 1.f;
+  }
+  {
+    float ss[16];
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) { ss[i] = q[i] * q[i]; ss[8 + i] = k[i] * k[i]; }
+    warp_transpose_sum<16>(ss);         // lane l: sum l / 2
+    if ((lane & 1) == 0) nrm[warp][lane >> 1] = ss[0];
   }
   __syncthreads();
-  float run = 0.f;
 #pragma unroll
   for (int i = 0; i < kBlk; ++i) {
     float sq = 0.f, sk = 0.f;
 #pragma unroll
     for (int w = 0; w < NW; ++w) { sq += nrm[w][i]; sk += nrm[w][8 + i]; }
-    q[i] *= 1.f / (sqrtf(static_cast<float>(D)) * sqrtf(sq + 1e-6f));
+    q[i] *= 1.f / sqrtf(static_cast<float>(D) * (sq + 1e-6f));
     k[i] *= 1.f / sqrtf(sk + 1e-6f);
-    if (CH) {
-      if (d < D && i < m_rows)
-        run += -a * df_softplus(in.z[static_cast<size_t>(q0 + r0 + i) * in.ldz + h * D + d] + __bfloat162float(in.dt_bias[h * D + d]));
-    } else {
-      run += sgl[i];
-    }
-    c[i] = run;
+    if (!CH) gd[i] = sg[i];
   }
-  // pair sums: P_ij (j <= i) at [i][j], the strict K K^T part (j < i) at [j][i]
+  // pair sums: P_ij (j <= i) at [i][j], the strict K K^T part (j < i) at [j][i]; kd[j] = k_j decayed from row j to row i
   {
-    float v[64], kd[kBlk];              // kd[j] = k_j decayed from row j to row i
+    float s[64], kd[kBlk];
 #pragma unroll
     for (int i = 0; i < kBlk; ++i) {
-      if (CH && i > 0) {
-        const float gi = expf(c[i] - c[i - 1]);
+      if (i > 0) {
 #pragma unroll
-        for (int j = 0; j < i; ++j) kd[j] *= gi;
+        for (int j = 0; j < i; ++j) kd[j] *= gd[i];
       }
       kd[i] = k[i];
 #pragma unroll
       for (int j = 0; j <= i; ++j) {
-        v[i * 8 + j] = q[i] * kd[j];
-        if (j < i) v[j * 8 + i] = k[i] * kd[j];
+        s[i * 8 + j] = q[i] * kd[j];
+        if (j < i) s[j * 8 + i] = k[i] * kd[j];
       }
     }
-    warp_transpose_sum64(v);
-    part[warp][2 * lane] = v[0];
-    part[warp][2 * lane + 1] = v[1];
+    warp_transpose_sum<64>(s);          // lane l: sums 2 l and 2 l + 1
+    part[warp][2 * lane] = s[0];
+    part[warp][2 * lane + 1] = s[1];
+  }
+  // what does not need T: decayed q and k, beta v
+  const size_t row = static_cast<size_t>(h) * o.R + static_cast<size_t>(tile) * kBlk;
+  float e[kBlk], run = 1.f;
+#pragma unroll
+  for (int i = 0; i < kBlk; ++i) {
+    run *= gd[i];
+    o.kt[(row + i) * DP + d] = sbeta[i] * run * k[i];
+    o.qt[(row + i) * DP + d] = run * q[i];
+  }
+  o.ge[(static_cast<size_t>(h) * (o.R / kBlk) + tile) * DP + d] = run;
+  run = 1.f;
+#pragma unroll
+  for (int i = kBlk - 1; i >= 0; --i) {
+    e[i] = run * k[i];
+    run *= gd[i];
+  }
+  if (d < V) {
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) o.bv[(row + i) * V + d] = sbeta[i] * v[i];
+  }
+  for (int vc = d + DP; vc < V; vc += DP) {
+    conv_rows<TP>(in, cs, C, q0, past, r0, m_rows, 2 * in.G * D + h * V + vc, v);
+#pragma unroll
+    for (int i = 0; i < kBlk; ++i) o.bv[(row + i) * V + vc] = sbeta[i] * v[i];
   }
   __syncthreads();
   for (int x = d; x < 64; x += DP) {
     float s = 0.f;
 #pragma unroll
     for (int w = 0; w < NW; ++w) s += part[w][x];
-    if (!CH) {
-      const int i = max(x >> 3, x & 7), j = min(x >> 3, x & 7);
-      float e = 0.f;
-      for (int y = j + 1; y <= i; ++y) e += sgl[y];
-      s *= expf(e);
-    }
     G[x] = s;
   }
   __syncthreads();
@@ -327,21 +364,11 @@ __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaB
     }
   }
   __syncthreads();
-  const size_t row = static_cast<size_t>(h) * o.R + static_cast<size_t>(tile) * kBlk;
   for (int x = d; x < 64; x += DP) {
     const int i = x >> 3, m = x & 7;
     float s = 0.f;
     for (int j = m; j <= i; ++j) s += G[i * 8 + j] * Tm[j * 8 + m];
     o.pt[row * 8 + x] = s;
-  }
-  const float cn = c[kBlk - 1];
-  float e[kBlk];
-#pragma unroll
-  for (int i = 0; i < kBlk; ++i) {
-    const float ec = expf(c[i]);
-    o.kt[(row + i) * DP + d] = sbeta[i] * ec * k[i];
-    o.qt[(row + i) * DP + d] = ec * q[i];
-    e[i] = expf(cn - c[i]) * k[i];
   }
 #pragma unroll
   for (int m = 0; m < kBlk; ++m) {
@@ -349,13 +376,6 @@ __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaB
 #pragma unroll
     for (int j = m; j < kBlk; ++j) s += Tm[j * 8 + m] * e[j];
     o.kh[(row + m) * DP + d] = s;
-  }
-  o.ge[(static_cast<size_t>(h) * (o.R / kBlk) + tile) * DP + d] = expf(cn);
-  for (int vc = d; vc < V; vc += DP) {
-    float y[kBlk];
-    conv_rows<TP>(in, cs, C, q0, past, r0, m_rows, 2 * in.G * D + h * V + vc, y);
-#pragma unroll
-    for (int i = 0; i < kBlk; ++i) o.bv[(row + i) * V + vc] = sbeta[i] * y[i];
   }
 }
 
@@ -368,12 +388,12 @@ JS_DEVICE void df_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "me
 
 constexpr int kBlkStages = 4;
 
-// x = hi + lo in two tf32 numbers (21 significant bits); three products of such halves make a 32-bit product on the
-// tensor cores: a b ~ ahi bhi + ahi blo + alo bhi
+// x = hi + lo in two tf32 numbers (at least 20 significant bits); three products of such halves make a 32-bit product on
+// the tensor cores: a b ~ ahi bhi + ahi blo + alo bhi.  Cutting bits off runs at full rate, the rounding conversion
+// at a quarter of it or less (a block of the walk splits some 50 numbers a lane).
 JS_DEVICE void tf32_split(float x, uint32_t& hi, uint32_t& lo) {
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(hi) : "f"(x));
-  const float rest = x - __uint_as_float(hi);
-  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(lo) : "f"(rest));
+  hi = __float_as_uint(x) & 0xffffe000u;
+  lo = __float_as_uint(x - __uint_as_float(hi)) & 0xffffe000u;
 }
 // d += a b, a 16 x 8 (row), b 8 x 8 (col), fp32 accumulators
 JS_DEVICE void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -447,62 +467,94 @@ delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
       const int d = dw + 8 * nt + 2 * qd + (e & 1), v = v0 + (e >> 1) * 8;
       S[nt][e] = (past > 0 && d < D && v < V) ? st[static_cast<size_t>(d) * V + v] : 0.f;
     }
-  for (int b = 0; b < nb; ++b) {
-    df_wait<kBlkStages - 2>();
-    __syncthreads();
-    if (b + kBlkStages - 1 < nb) stage_in(b + kBlkStages - 1);
-    df_commit();
-    const Stage& s = sm[b % kBlkStages];
-    float ak[3][4] = {}, aq[3][4] = {};
+  auto fold = [](const float (&x)[3][4]) {
+    return make_float4(x[0][0] + (x[1][0] + x[2][0]), x[0][1] + (x[1][1] + x[2][1]), x[0][2] + (x[1][2] + x[2][2]),
+                       x[0][3] + (x[1][3] + x[2][3]));
+  };
+  // (P T) of block b as a B operand: read while the block's stage is still there, used one block later
+  float4* pmine = part + vt * 256 + kw * 64 + lane;
+  uint32_t wh[4] = {}, wl[4] = {};      // W^T of the block before, split, as an A operand
+  float2 pt_prev = make_float2(0.f, 0.f);
+  // the read-outs of a block: its Q parts were exchanged at the barrier behind it; the warps take turns
+  auto read_out = [&](int b) {
+    if (kw != (b & 3)) return;
+    const float4* pb = part + ((b + 1) & 1) * NV * 256 + vt * 256 + 32 + lane;
+    const float4 p0 = pb[0], p1 = pb[64], p2 = pb[128], p3 = pb[192];
+    float O[4] = {(p0.x + p1.x) + (p2.x + p3.x), (p0.y + p1.y) + (p2.y + p3.y), (p0.z + p1.z) + (p2.z + p3.z),
+                  (p0.w + p1.w) + (p2.w + p3.w)};
+    uint32_t h0, l0, h1, l1;
+    tf32_split(pt_prev.x, h0, l0);
+    tf32_split(pt_prev.y, h1, l1);
+    float low[4] = {};
+    mma_tf32(low, wh, l0, l1);
+    mma_tf32(low, wl, h0, h1);
+    mma_tf32(O, wh, h0, h1);
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      const int d = dw + 8 * nt + 2 * qd;
-      const float2 kv = *reinterpret_cast<const float2*>(&s.kt[gr][d]);
-      const float2 qv = *reinterpret_cast<const float2*>(&s.qt[gr][d]);
-      uint32_t ah[4], al[4], kh0, kl0, kh1, kl1, qh0, ql0, qh1, ql1;
-      tf32_split(S[nt][0], ah[0], al[0]);
-      tf32_split(S[nt][2], ah[1], al[1]);
-      tf32_split(S[nt][1], ah[2], al[2]);
-      tf32_split(S[nt][3], ah[3], al[3]);
-      tf32_split(kv.x, kh0, kl0);
-      tf32_split(kv.y, kh1, kl1);
-      tf32_split(qv.x, qh0, ql0);
-      tf32_split(qv.y, qh1, ql1);
-      mma_tf32(ak[0], ah, kh0, kh1);
-      mma_tf32(ak[1], ah, kl0, kl1);
-      mma_tf32(ak[2], al, kh0, kh1);
-      mma_tf32(aq[0], ah, qh0, qh1);
-      mma_tf32(aq[1], ah, ql0, ql1);
-      mma_tf32(aq[2], al, qh0, qh1);
+    for (int e = 0; e < 4; ++e) {
+      const int i = b * kBlk + 2 * qd + (e & 1), v = v0 + (e >> 1) * 8;
+      if (i < n && v < V) out[(static_cast<size_t>(q0 + i) * in.H + h) * V + v] = O[e] + low[e];
     }
-    float4* pb = part + ((b & 1) * NV + vt) * 256;
-    pb[kw * 64 + lane] = make_float4(ak[0][0] + (ak[1][0] + ak[2][0]), ak[0][1] + (ak[1][1] + ak[2][1]),
-                                     ak[0][2] + (ak[1][2] + ak[2][2]), ak[0][3] + (ak[1][3] + ak[2][3]));
-    pb[kw * 64 + 32 + lane] = make_float4(aq[0][0] + (aq[1][0] + aq[2][0]), aq[0][1] + (aq[1][1] + aq[2][1]),
-                                          aq[0][2] + (aq[1][2] + aq[2][2]), aq[0][3] + (aq[1][3] + aq[2][3]));
-    __syncthreads();
-    float W[4];                         // (v0, m), (v0, m + 1), (v0 + 8, m), (v0 + 8, m + 1), m = 2 qd
+  };
+  df_wait<kBlkStages - 2>();
+  __syncthreads();
+  for (int b = 0; b < nb; ++b) {
+    const Stage& s = sm[b % kBlkStages];
+    // ---- K part of block b, on the way to the barrier
+    uint32_t sh[NT][4], sl[NT][4];
     {
-      const float4 p0 = pb[lane], p1 = pb[64 + lane], p2 = pb[128 + lane], p3 = pb[192 + lane];
-      const int c = vt * 16 + gr;
-      W[0] = s.bv[2 * qd][c] - ((p0.x + p1.x) + (p2.x + p3.x));
-      W[1] = s.bv[2 * qd + 1][c] - ((p0.y + p1.y) + (p2.y + p3.y));
-      W[2] = s.bv[2 * qd][c + 8] - ((p0.z + p1.z) + (p2.z + p3.z));
-      W[3] = s.bv[2 * qd + 1][c + 8] - ((p0.w + p1.w) + (p2.w + p3.w));
+      float ak[3][4] = {};
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        const float2 kv = *reinterpret_cast<const float2*>(&s.kt[gr][dw + 8 * nt + 2 * qd]);
+        tf32_split(S[nt][0], sh[nt][0], sl[nt][0]);
+        tf32_split(S[nt][2], sh[nt][1], sl[nt][1]);
+        tf32_split(S[nt][1], sh[nt][2], sl[nt][2]);
+        tf32_split(S[nt][3], sh[nt][3], sl[nt][3]);
+        uint32_t h0, l0, h1, l1;
+        tf32_split(kv.x, h0, l0);
+        tf32_split(kv.y, h1, l1);
+        mma_tf32(ak[0], sh[nt], h0, h1);
+        mma_tf32(ak[1], sh[nt], l0, l1);
+        mma_tf32(ak[2], sl[nt], h0, h1);
+      }
+      pmine[(b & 1) * NV * 256] = fold(ak);
     }
-    uint32_t wh[4], wl[4];
-    tf32_split(W[0], wh[0], wl[0]);
-    tf32_split(W[2], wh[1], wl[1]);
-    tf32_split(W[1], wh[2], wl[2]);
-    tf32_split(W[3], wh[3], wl[3]);
+    df_wait<kBlkStages - 3>();          // block b + 1 is here too
+    __syncthreads();                    // ... for everyone, with all K parts of block b and all Q parts of block b - 1
+    const float4* pb = part + (b & 1) * NV * 256 + vt * 256 + lane;
+    const float4 p0 = pb[0], p1 = pb[64], p2 = pb[128], p3 = pb[192];
+    // ---- Q part of block b from the state before it; exchanged at the next barrier
+    {
+      float aq[3][4] = {};
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        const float2 qv = *reinterpret_cast<const float2*>(&s.qt[gr][dw + 8 * nt + 2 * qd]);
+        uint32_t h0, l0, h1, l1;
+        tf32_split(qv.x, h0, l0);
+        tf32_split(qv.y, h1, l1);
+        mma_tf32(aq[0], sh[nt], h0, h1);
+        mma_tf32(aq[1], sh[nt], l0, l1);
+        mma_tf32(aq[2], sl[nt], h0, h1);
+      }
+      if (b > 0) read_out(b - 1);       // reads the Q parts of block b - 1 from the other half of `part`
+      pmine[((b + 1) & 1) * NV * 256 + 32] = fold(aq);
+    }
+    // ---- W and the state's step
+    {
+      const int c = vt * 16 + gr;
+      tf32_split(s.bv[2 * qd][c] - ((p0.x + p1.x) + (p2.x + p3.x)), wh[0], wl[0]);
+      tf32_split(s.bv[2 * qd][c + 8] - ((p0.z + p1.z) + (p2.z + p3.z)), wh[1], wl[1]);
+      tf32_split(s.bv[2 * qd + 1][c] - ((p0.y + p1.y) + (p2.y + p3.y)), wh[2], wl[2]);
+      tf32_split(s.bv[2 * qd + 1][c + 8] - ((p0.w + p1.w) + (p2.w + p3.w)), wh[3], wl[3]);
+    }
+    pt_prev = *reinterpret_cast<const float2*>(&s.pt[gr * 8 + 2 * qd]);
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       const int d = dw + 8 * nt;
       const float2 gv = *reinterpret_cast<const float2*>(&s.ge[d + 2 * qd]);
-      const float k0 = s.kh[2 * qd][d + gr], k1 = s.kh[2 * qd + 1][d + gr];
       uint32_t h0, l0, h1, l1;
-      tf32_split(k0, h0, l0);
-      tf32_split(k1, h1, l1);
+      tf32_split(s.kh[2 * qd][d + gr], h0, l0);
+      tf32_split(s.kh[2 * qd + 1][d + gr], h1, l1);
       float low[4] = {};
       S[nt][0] *= gv.x;
       S[nt][1] *= gv.y;
@@ -514,25 +566,12 @@ delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) S[nt][e] += low[e];
     }
-    if (kw == (b & 3)) {                // the warps take turns with the read-outs
-      const float4 p0 = pb[32 + lane], p1 = pb[96 + lane], p2 = pb[160 + lane], p3 = pb[224 + lane];
-      float O[4] = {(p0.x + p1.x) + (p2.x + p3.x), (p0.y + p1.y) + (p2.y + p3.y), (p0.z + p1.z) + (p2.z + p3.z),
-                    (p0.w + p1.w) + (p2.w + p3.w)};
-      const float2 pv = *reinterpret_cast<const float2*>(&s.pt[gr * 8 + 2 * qd]);
-      uint32_t h0, l0, h1, l1;
-      tf32_split(pv.x, h0, l0);
-      tf32_split(pv.y, h1, l1);
-      float low[4] = {};
-      mma_tf32(low, wh, l0, l1);
-      mma_tf32(low, wl, h0, h1);
-      mma_tf32(O, wh, h0, h1);
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int i = b * kBlk + 2 * qd + (e & 1), v = v0 + (e >> 1) * 8;
-        if (i < n && v < V) out[(static_cast<size_t>(q0 + i) * in.H + h) * V + v] = O[e] + low[e];
-      }
-    }
+    // the buffer of block b - 1 is free: everyone passed this block's barrier
+    if (b + kBlkStages - 1 < nb) stage_in(b + kBlkStages - 1);
+    df_commit();
   }
+  __syncthreads();
+  read_out(nb - 1);
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
