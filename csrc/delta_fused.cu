@@ -246,10 +246,10 @@ JS_DEVICE void warp_transpose_sum(float (&v)[N]) {
 }
 
 template <int DP, bool CH, int TP>
-__global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaBlocks o) {
+__global__ void __launch_bounds__(DP, TP <= 4 ? 640 / DP : 1) delta_block_prep_kernel(DeltaIn in, DeltaBlocks o) {
   constexpr int NW = DP / 32;
-  __shared__ float part[NW][64], G[64], Tm[64], nrm[NW][16], sbeta[kBlk], sg[kBlk];
-  pdl_launch_dependents();
+  __shared__ float part[NW][64], G[64], Tm[64], nrm[NW][16], inv_norm[16], sbeta[kBlk], sg[kBlk];
+  // no early start of the walk behind: its few long CTAs would pile up on the SMs that empty first
   pdl_wait();
   const int h = blockIdx.y, tile = blockIdx.x, d = threadIdx.x, warp = d >> 5, lane = d & 31;
   int lo = 0, hi = in.B - 1;
@@ -289,13 +289,17 @@ __global__ void __launch_bounds__(DP) delta_block_prep_kernel(DeltaIn in, DeltaB
     if ((lane & 1) == 0) nrm[warp][lane >> 1] = ss[0];
   }
   __syncthreads();
+  if (d < 16) {                         // q's includes the 1/sqrt(D)
+    float s = 1e-6f;
+#pragma unroll
+    for (int w = 0; w < NW; ++w) s += nrm[w][d];
+    inv_norm[d] = 1.f / sqrtf(d < 8 ? static_cast<float>(D) * s : s);
+  }
+  __syncthreads();
 #pragma unroll
   for (int i = 0; i < kBlk; ++i) {
-    float sq = 0.f, sk = 0.f;
-#pragma unroll
-    for (int w = 0; w < NW; ++w) { sq += nrm[w][i]; sk += nrm[w][8 + i]; }
-    q[i] *= 1.f / sqrtf(static_cast<float>(D) * (sq + 1e-6f));
-    k[i] *= 1.f / sqrtf(sk + 1e-6f);
+    q[i] *= inv_norm[i];
+    k[i] *= inv_norm[8 + i];
     if (!CH) gd[i] = sg[i];
   }
   // pair sums: P_ij (j <= i) at [i][j], the strict K K^T part (j < i) at [j][i]; kd[j] = k_j decayed from row j to row i
@@ -386,14 +390,15 @@ JS_DEVICE void df_commit() { asm volatile("cp.async.commit_group;" ::: "memory")
 template <int N>
 JS_DEVICE void df_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-constexpr int kBlkStages = 4;
+constexpr int kBlkStages = 6;
 
-// x = hi + lo in two tf32 numbers (at least 20 significant bits); three products of such halves make a 32-bit product on
-// the tensor cores: a b ~ ahi bhi + ahi blo + alo bhi.  Cutting bits off runs at full rate, the rounding conversion
-// at a quarter of it or less (a block of the walk splits some 50 numbers a lane).
+// x = hi + lo as two tf32 operands (at least 20 significant bits together); three products of such halves make a 32-bit product
+// on the tensor cores: a b ~ ahi bhi + ahi blo + alo bhi.  The tensor cores read the upper 19 bits of a tf32 operand, so hi
+// is x itself and lo what those bits leave; the rounding conversion runs at a quarter of the rate of these two steps or
+// less, and a block of the walk splits some 50 numbers a lane.
 JS_DEVICE void tf32_split(float x, uint32_t& hi, uint32_t& lo) {
-  hi = __float_as_uint(x) & 0xffffe000u;
-  lo = __float_as_uint(x - __uint_as_float(hi)) & 0xffffe000u;
+  hi = __float_as_uint(x);
+  lo = __float_as_uint(x - __uint_as_float(hi & 0xffffe000u));
 }
 // d += a b, a 16 x 8 (row), b 8 x 8 (col), fp32 accumulators
 JS_DEVICE void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
@@ -401,30 +406,36 @@ JS_DEVICE void mma_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint
       : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// d = a b
+JS_DEVICE void mma_tf32_first(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%10, %10, %10, %10};"
+      : "=f"(d[0]), "=f"(d[1]), "=f"(d[2]), "=f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.f));
+}
 
-// The walk over the blocks of one (sequence, head): a CTA holds 16 NV value columns of the state, four warps a quarter of the
-// key dimension each.  A warp keeps its piece TRANSPOSED as the accumulators of 16 (values) x 8 (keys) tiles.  The column
+// The walk over the blocks of one (sequence, head): a CTA holds 16 NV value columns of the state, KW warps an equal part of
+// the key dimension each.  A warp keeps its piece TRANSPOSED as the accumulators of 16 (values) x 8 (keys) tiles.  The column
 // order of an accumulator tile differs from the one an A operand wants, but as long as the B operand takes its rows in the
 // same order the sum over them is the same, so the state feeds the next product straight from the accumulators:
 //
 //   per block   [K part | Q part] (values x 8 rows) = S^T [kt | qt]^T   partial sums over the warp's keys, added across warps
 //               W^T = bv^T - K part;  O^T = Q part + W^T pt^T;  S^T = S^T ge + W^T kh
-template <int DP, int NV>
-__global__ void __launch_bounds__(128 * NV)
+template <int DP, int NV, int KW>
+__global__ void __launch_bounds__(32 * KW * NV)
 delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
-  constexpr int NT = DP / 32;                   // key tiles of 8 a warp holds
+  constexpr int NT = DP / (8 * KW);             // key tiles of 8 a warp holds
   constexpr int LK = DP + 8, LH = DP + 4, LV = 16 * NV + 4;       // row strides without bank conflicts for their readers
-  constexpr int THREADS = 128 * NV;
+  constexpr int THREADS = 32 * KW * NV, HALF = NV * KW * 64;
   struct __align__(16) Stage {
     float kt[kBlk][LK], qt[kBlk][LK], kh[kBlk][LH], ge[DP], bv[kBlk][LV], pt[64];
   };
   extern __shared__ __align__(16) uint8_t raw[];
   Stage* sm = reinterpret_cast<Stage*>(raw);
-  float4* part = reinterpret_cast<float4*>(raw + sizeof(Stage) * kBlkStages);      // [2][NV][4 warps][2][32]
+  float4* part = reinterpret_cast<float4*>(raw + sizeof(Stage) * kBlkStages);      // [2][NV][KW][K, Q][32]
   pdl_launch_dependents();
   pdl_wait();
   const int slice = blockIdx.x, h = blockIdx.y, sq = blockIdx.z, tid = threadIdx.x, lane = tid & 31;
-  const int kw = (tid >> 5) & 3, vt = tid >> 7;
+  const int kw = (tid >> 5) % KW, vt = (tid >> 5) / KW;
   const int gr = lane >> 2, qd = lane & 3;
   const int q0 = in.cu_q[sq], n = in.cu_q[sq + 1] - q0;
   if (n <= 0) return;
@@ -433,7 +444,7 @@ delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
   const size_t row0 = static_cast<size_t>(h) * o.R + static_cast<size_t>(tile0) * kBlk;
   float* st = state + (static_cast<size_t>(slot) * in.H + h) * D * V;
   const int v0 = slice * 16 * NV + vt * 16 + gr;          // this lane's value columns: v0 and v0 + 8
-  const int dw = kw * (DP / 4);                           // first key of the warp
+  const int dw = kw * (DP / KW);                          // first key of the warp
 
   auto stage_in = [&](int b) {
     Stage& s = sm[b % kBlkStages];
@@ -467,26 +478,34 @@ delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
       const int d = dw + 8 * nt + 2 * qd + (e & 1), v = v0 + (e >> 1) * 8;
       S[nt][e] = (past > 0 && d < D && v < V) ? st[static_cast<size_t>(d) * V + v] : 0.f;
     }
+  // three accumulators, not one: the chain of dependent products is what a block waits for
   auto fold = [](const float (&x)[3][4]) {
     return make_float4(x[0][0] + (x[1][0] + x[2][0]), x[0][1] + (x[1][1] + x[2][1]), x[0][2] + (x[1][2] + x[2][2]),
                        x[0][3] + (x[1][3] + x[2][3]));
   };
   // (P T) of block b as a B operand: read while the block's stage is still there, used one block later
-  float4* pmine = part + vt * 256 + kw * 64 + lane;
+  float4* pmine = part + vt * KW * 64 + kw * 64 + lane;
+  auto gather = [&](const float4* pb) {         // sum of a part over the warps, in warp order
+    float4 t = pb[0];
+#pragma unroll
+    for (int w = 1; w < KW; ++w) {
+      const float4 x = pb[w * 64];
+      t = make_float4(t.x + x.x, t.y + x.y, t.z + x.z, t.w + x.w);
+    }
+    return t;
+  };
   uint32_t wh[4] = {}, wl[4] = {};      // W^T of the block before, split, as an A operand
   float2 pt_prev = make_float2(0.f, 0.f);
   // the read-outs of a block: its Q parts were exchanged at the barrier behind it; the warps take turns
   auto read_out = [&](int b) {
-    if (kw != (b & 3)) return;
-    const float4* pb = part + ((b + 1) & 1) * NV * 256 + vt * 256 + 32 + lane;
-    const float4 p0 = pb[0], p1 = pb[64], p2 = pb[128], p3 = pb[192];
-    float O[4] = {(p0.x + p1.x) + (p2.x + p3.x), (p0.y + p1.y) + (p2.y + p3.y), (p0.z + p1.z) + (p2.z + p3.z),
-                  (p0.w + p1.w) + (p2.w + p3.w)};
+    if (kw != (b & (KW - 1))) return;
+    const float4 q4 = gather(part + ((b + 1) & 1) * HALF + vt * KW * 64 + 32 + lane);
+    float O[4] = {q4.x, q4.y, q4.z, q4.w};
     uint32_t h0, l0, h1, l1;
     tf32_split(pt_prev.x, h0, l0);
     tf32_split(pt_prev.y, h1, l1);
-    float low[4] = {};
-    mma_tf32(low, wh, l0, l1);
+    float low[4];
+    mma_tf32_first(low, wh, l0, l1);
     mma_tf32(low, wl, h0, h1);
     mma_tf32(O, wh, h0, h1);
 #pragma unroll
@@ -502,7 +521,7 @@ delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
     // ---- K part of block b, on the way to the barrier
     uint32_t sh[NT][4], sl[NT][4];
     {
-      float ak[3][4] = {};
+      float ak[3][4];
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
         const float2 kv = *reinterpret_cast<const float2*>(&s.kt[gr][dw + 8 * nt + 2 * qd]);
@@ -513,39 +532,50 @@ delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
         uint32_t h0, l0, h1, l1;
         tf32_split(kv.x, h0, l0);
         tf32_split(kv.y, h1, l1);
-        mma_tf32(ak[0], sh[nt], h0, h1);
-        mma_tf32(ak[1], sh[nt], l0, l1);
-        mma_tf32(ak[2], sl[nt], h0, h1);
+        if (nt == 0) {
+          mma_tf32_first(ak[0], sh[nt], h0, h1);
+          mma_tf32_first(ak[1], sh[nt], l0, l1);
+          mma_tf32_first(ak[2], sl[nt], h0, h1);
+        } else {
+          mma_tf32(ak[0], sh[nt], h0, h1);
+          mma_tf32(ak[1], sh[nt], l0, l1);
+          mma_tf32(ak[2], sl[nt], h0, h1);
+        }
       }
-      pmine[(b & 1) * NV * 256] = fold(ak);
+      pmine[(b & 1) * HALF] = fold(ak);
     }
     df_wait<kBlkStages - 3>();          // block b + 1 is here too
     __syncthreads();                    // ... for everyone, with all K parts of block b and all Q parts of block b - 1
-    const float4* pb = part + (b & 1) * NV * 256 + vt * 256 + lane;
-    const float4 p0 = pb[0], p1 = pb[64], p2 = pb[128], p3 = pb[192];
+    const float4 k4 = gather(part + (b & 1) * HALF + vt * KW * 64 + lane);
     // ---- Q part of block b from the state before it; exchanged at the next barrier
     {
-      float aq[3][4] = {};
+      float aq[3][4];
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt) {
         const float2 qv = *reinterpret_cast<const float2*>(&s.qt[gr][dw + 8 * nt + 2 * qd]);
         uint32_t h0, l0, h1, l1;
         tf32_split(qv.x, h0, l0);
         tf32_split(qv.y, h1, l1);
-        mma_tf32(aq[0], sh[nt], h0, h1);
-        mma_tf32(aq[1], sh[nt], l0, l1);
-        mma_tf32(aq[2], sl[nt], h0, h1);
+        if (nt == 0) {
+          mma_tf32_first(aq[0], sh[nt], h0, h1);
+          mma_tf32_first(aq[1], sh[nt], l0, l1);
+          mma_tf32_first(aq[2], sl[nt], h0, h1);
+        } else {
+          mma_tf32(aq[0], sh[nt], h0, h1);
+          mma_tf32(aq[1], sh[nt], l0, l1);
+          mma_tf32(aq[2], sl[nt], h0, h1);
+        }
       }
       if (b > 0) read_out(b - 1);       // reads the Q parts of block b - 1 from the other half of `part`
-      pmine[((b + 1) & 1) * NV * 256 + 32] = fold(aq);
+      pmine[((b + 1) & 1) * HALF + 32] = fold(aq);
     }
     // ---- W and the state's step
     {
       const int c = vt * 16 + gr;
-      tf32_split(s.bv[2 * qd][c] - ((p0.x + p1.x) + (p2.x + p3.x)), wh[0], wl[0]);
-      tf32_split(s.bv[2 * qd][c + 8] - ((p0.z + p1.z) + (p2.z + p3.z)), wh[1], wl[1]);
-      tf32_split(s.bv[2 * qd + 1][c] - ((p0.y + p1.y) + (p2.y + p3.y)), wh[2], wl[2]);
-      tf32_split(s.bv[2 * qd + 1][c + 8] - ((p0.w + p1.w) + (p2.w + p3.w)), wh[3], wl[3]);
+      tf32_split(s.bv[2 * qd][c] - k4.x, wh[0], wl[0]);
+      tf32_split(s.bv[2 * qd][c + 8] - k4.z, wh[1], wl[1]);
+      tf32_split(s.bv[2 * qd + 1][c] - k4.y, wh[2], wl[2]);
+      tf32_split(s.bv[2 * qd + 1][c + 8] - k4.w, wh[3], wl[3]);
     }
     pt_prev = *reinterpret_cast<const float2*>(&s.pt[gr * 8 + 2 * qd]);
 #pragma unroll
@@ -555,16 +585,12 @@ delta_block_kernel(DeltaIn in, DeltaBlocks o, float* state, float* out) {
       uint32_t h0, l0, h1, l1;
       tf32_split(s.kh[2 * qd][d + gr], h0, l0);
       tf32_split(s.kh[2 * qd + 1][d + gr], h1, l1);
-      float low[4] = {};
-      S[nt][0] *= gv.x;
-      S[nt][1] *= gv.y;
-      S[nt][2] *= gv.x;
-      S[nt][3] *= gv.y;
-      mma_tf32(low, wh, l0, l1);
+      float low[4];
+      mma_tf32_first(low, wh, l0, l1);
       mma_tf32(low, wl, h0, h1);
-      mma_tf32(S[nt], wh, h0, h1);
 #pragma unroll
-      for (int e = 0; e < 4; ++e) S[nt][e] += low[e];
+      for (int e = 0; e < 4; ++e) S[nt][e] = fmaf(S[nt][e], (e & 1) ? gv.y : gv.x, low[e]);
+      mma_tf32(S[nt], wh, h0, h1);
     }
     // the buffer of block b - 1 is free: everyone passed this block's barrier
     if (b + kBlkStages - 1 < nb) stage_in(b + kBlkStages - 1);
@@ -610,13 +636,13 @@ struct FusedLaunch {
   }
 };
 
-template <int DP, int NV>
+template <int DP, int NV, int KW>
 static int launch_blocks(const DeltaIn& in, const DeltaBlocks& o, float* state, float* out, int pdl, cudaStream_t stream) {
-  constexpr int smem = kBlkStages * (kBlk * (3 * DP + 20 + 16 * NV + 4) + DP + 64) * 4 + 2 * NV * 256 * 16;
+  constexpr int smem = kBlkStages * (kBlk * (3 * DP + 20 + 16 * NV + 4) + DP + 64) * 4 + 2 * NV * KW * 64 * 16;
   static int configured[kMaxDevicesCached] = {};
-  auto kern = delta_block_kernel<DP, NV>;
+  auto kern = delta_block_kernel<DP, NV, KW>;
   if (ensure_dyn_smem(kern, smem, configured) != 0) return -3;
-  FusedLaunch l(dim3((in.V + 16 * NV - 1) / (16 * NV), in.H, in.B), dim3(128 * NV), stream, pdl, smem);
+  FusedLaunch l(dim3((in.V + 16 * NV - 1) / (16 * NV), in.H, in.B), dim3(32 * KW * NV), stream, pdl, smem);
   return cudaLaunchKernelEx(&l.c, kern, in, o, state, out) == cudaSuccess ? 0 : -4;
 }
 
@@ -659,11 +685,11 @@ extern "C" int js_delta_step(int H, int G, int D, int V, int ntaps, int channel,
 }
 
 // Prompt portions in blocks of 8 rows, bf16 inputs; D <= 128, V % 4 == 0.  R = 8 * (T / 8 + B) padded rows; kt, qt, kh (H, R, DP),
-// ge (H, R / 8, DP) with DP = 64 or 128; bv (H, R, V); pt (H, R, 8); out (T, H, V) fp32.
+// ge (H, R / 8, DP) with DP = 64 or 128; bv (H, R, V); pt (H, R, 8); out (T, H, V) fp32.  wide: 32 value columns a CTA, not 16.
 extern "C" int js_delta_blocks(int H, int G, int D, int V, int ntaps, int channel, const void* pre, int ldp, const float* z, int ldz,
                                const float* b, int ldb, const void* taps, const void* A_log, const void* dt_bias, void* conv, float* state,
                                const int* rows, const int* cu_q, const int* past_lens, int B, int T, float* kt, float* qt, float* kh,
-                               float* bv, float* pt, float* ge, float* out, int ncol, int pdl, cudaStream_t stream) {
+                               float* bv, float* pt, float* ge, float* out, int wide, int pdl, cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
   if (!fused_shape_ok(H, G, D, V, ntaps) || D > 128) return -10;
@@ -674,8 +700,8 @@ extern "C" int js_delta_blocks(int H, int G, int D, int V, int ntaps, int channe
   const DeltaBlocks o{kt, qt, kh, bv, pt, ge, tiles * kBlk};
   if (D <= 64) {
     if (int rc = launch_block_prep<64>(in, o, tiles, pdl, stream)) return rc;
-    return ncol == 16 ? launch_blocks<64, 1>(in, o, state, out, pdl, stream) : launch_blocks<64, 2>(in, o, state, out, pdl, stream);
+    return launch_blocks<64, 1, 4>(in, o, state, out, pdl, stream);
   }
   if (int rc = launch_block_prep<128>(in, o, tiles, pdl, stream)) return rc;
-  return ncol == 16 ? launch_blocks<128, 1>(in, o, state, out, pdl, stream) : launch_blocks<128, 2>(in, o, state, out, pdl, stream);
+  return wide ? launch_blocks<128, 2, 4>(in, o, state, out, pdl, stream) : launch_blocks<128, 1, 4>(in, o, state, out, pdl, stream);
 }

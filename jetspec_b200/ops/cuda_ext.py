@@ -1056,8 +1056,9 @@ def delta_forward(cfg, pre, z, b, taps, A_log, dt_bias, state, conv, rows, cu_q,
         return 1
     if delta_blocks_ok(cfg):
         w = get("blocks")
-        ncol = 16 if B * cfg.heads * ((cfg.vdim + 31) // 32) < SM_COUNT * 3 // 4 else 32
-        _check(lib.js_delta_blocks(*head, T, *(_p(w[n]) for n in ("kt", "qt", "kh", "bv", "pt", "ge", "o")), ncol, int(pdl), _stream()),
+        # 32 value columns a CTA share the loads, 16 fill the device: a lone sequence of few heads wants the latter
+        wide = B * cfg.heads * ((cfg.vdim + 31) // 32) >= SM_COUNT * 3 // 4
+        _check(lib.js_delta_blocks(*head, T, *(_p(w[n]) for n in ("kt", "qt", "kh", "bv", "pt", "ge", "o")), int(wide), int(pdl), _stream()),
                "js_delta_blocks")
     else:
         w = get("rows")
