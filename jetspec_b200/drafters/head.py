@@ -18,6 +18,7 @@ from typing import Optional
 import torch
 
 from .. import ops
+from ..utils.graphs import capture
 from .base import Drafter, TreeDrafter
 
 
@@ -221,7 +222,7 @@ class GraphedDraftHead(DraftHeadTreeDrafter):
             torch.cuda.synchronize()
             gs["stage_dev"].copy_(h, non_blocking=True)   # the warm-up consumed ST_NEW: stage again for the replay
             g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
+            with capture(g):
                 self._launch(gs, pdl=_PDL)
             gs["graphs"][key] = g
         r["no_topk"] = not want_topk

@@ -25,6 +25,7 @@ from ..drafters.base import TreeDrafter
 from ..drafters.head import DraftHeadTreeDrafter
 from ..ops import cuda_ext as X
 from ..ops import reference as ref
+from ..utils.graphs import capture
 
 ST_PAST, ST_CTX, ST_NEW, ST_DONE = 0, 1, 2, 3
 
@@ -113,7 +114,7 @@ class DraftWorker:
             steps = 1
             X.check_status("cuda")
             g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
+            with capture(g):
                 self._step(self._pdl)
             self.graph = g
             if int(done_view[ST_DONE]) != 0:

@@ -29,6 +29,7 @@ from ..ops import cuda_ext as X
 from ..ops import reference as ref
 from ..sampling import SamplingParams, sample
 from ..tree.builder import topk_rows
+from ..utils.graphs import capture
 
 ST_PAST, ST_CTX, ST_NEW, ST_DONE, ST_GEN, ST_NNODES, ST_ROUNDS = range(7)
 _PDL = os.environ.get("JETSPEC_PDL", "1") != "0"
@@ -532,13 +533,13 @@ class FastRound:
             r["ring_mod"] = par.ring_mod
         if ext is None:
             g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
+            with capture(g):
                 self._launch_round(r, pdl=_PDL)
             r["graph"] = g
         else:
             for part in ("a", "x", "b"):
                 g = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(g):
+                with capture(g):
                     self._launch_round(r, pdl=_PDL, part=part)
                 r["graph_" + part] = g
         pool.frozen = True
@@ -860,7 +861,7 @@ class FastRound:
                 self.tp.begin_sequence(self.tp._turn)     # cycle length that is safe across replays
                 r["ring_mod"] = self.tp.ring_mod
             g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
+            with capture(g):
                 self._launch_batch_verify(r, pdl=_PDL)
             r["graph"] = g
             pool.frozen = True

@@ -15,6 +15,9 @@ Per layer, on the bf16 copy ``h`` of the fp32 residual stream ``x``:
 5. experts: the permutation by expert depends on the token ids alone, so one launch at the start makes every layer's;
    two grouped GEMMs, the shared expert's two GEMMs, and the same residual kernel as the combine.
 
+Two branches of a layer do not depend on each other: window attention and delta rule, shared expert and routed experts.
+In captured graphs and on long portions they run on two streams: each alone leaves most of the device idle.
+
 Token trees leave the recurrent states alone and keep every layer's prepared rows; :meth:`HybridStack.commit` then
 advances the states along the accepted nodes.  Every size is padded to what the kernels want when the weights are
 prepared; padding is zero and stays zero.
@@ -29,6 +32,8 @@ import torch
 from ..ops import cuda_ext as X
 from ..runtime.kv_pool import window_row_width
 from .latent_stack import MAX_SORT_PAIRS, _pad, _up
+
+FORK_MIN_TOKENS = 512          # eager launches fork from this many rows on (below, the host is what a forward waits for)
 
 _TABLE_LAYER = np.dtype([("table", "<u8"), ("top", "<i4"), ("experts", "<i4"), ("off", "<i4"), ("pad", "<i4")])
 
@@ -168,6 +173,7 @@ class HybridStack:
         self.table, self.head = (w if self.wp == self.width else _pad(w, w.shape[0], self.wp) for w in (table, head))
         self.vocab = cfg.vocab_size
         self.routed = [L for L in self.layers if L.moe is not None]
+        self.side = torch.cuda.Stream(self.device) if self.device.type == "cuda" else None
         self.pass_rows = MAX_SORT_PAIRS // max([L.moe.top for L in self.routed], default=1)
 
     @staticmethod
@@ -219,6 +225,19 @@ class HybridStack:
 
     def _act(self, st, L, hold: bool) -> torch.Tensor:
         return st.get(f"act{L.index}" if hold else "act", L.act_cols)
+
+    def _beside(self, fork: bool, side, main) -> int:
+        """Launch ``side`` and ``main`` (functions of ``pdl for the first kernel``, returning launch counts), on two streams
+        when ``fork``; everything launched later waits for both."""
+        if not fork:
+            return side(True) + main(True)
+        cur = torch.cuda.current_stream()
+        self.side.wait_stream(cur)
+        with torch.cuda.stream(self.side):
+            n = side(False)               # a plain dependency across streams
+        n += main(True)
+        cur.wait_stream(self.side)
+        return n
 
     # ------------------------------------------------------------------ one forward
     def run(self, st, ids, pool, batch, xn, taps=None, tap_ids=None, pdl: bool = True) -> int:
@@ -277,17 +296,15 @@ class HybridStack:
             n += 1
         if not c.gate_rank:
             gate = act[:, L.at["gate"]:]
-        yl = None
-        if L.parallel:
-            yl = st.get("yl", self.wp)
-            n += self._window(st, L, pool, batch, act, yl, pdl)
-        yr = st.get("yr", self.wp)
+        yl, yr = st.get("yl", self.wp), st.get("yr", self.wp)
         pre = act[:, L.at["q"]:L.at["q"] + c.channels]
-        n += self._delta(st, L, pool, batch, pre, z, b, gate, yr, hold, pdl)
+        fork = L.parallel and self._forks(st)
+        window = lambda first: self._window(st, L, pool, batch, act, yl, pdl, pdl and first) if L.parallel else 0
+        n += self._beside(fork, window, lambda first: self._delta(st, L, pool, batch, pre, z, b, gate, yr, hold, pdl))
         mlp = L.moe is not None
         end = dict(out=None if mlp else out, tap=None if mlp else tap)
         if L.parallel:
-            self._resid(st, L.norm1, L.eps, ya=yl, bias=L.wo_bias, wa=L.left_norm, yb=yr, wb=L.right_norm, pdl=pdl, **end)
+            self._resid(st, L.norm1, L.eps, ya=yl, bias=L.wo_bias, wa=L.left_norm, yb=yr, wb=L.right_norm, pdl=pdl and not fork, **end)
         else:
             self._resid(st, L.norm1, L.eps, ya=yr, pdl=pdl, **end)
         n += 1
@@ -295,7 +312,10 @@ class HybridStack:
             n += self._experts(st, L, out, tap, pdl)
         return n
 
-    def _window(self, st, L, pool, batch, act, y, pdl) -> int:
+    def _forks(self, st) -> bool:
+        return st.T >= FORK_MIN_TOKENS or torch.cuda.is_current_stream_capturing()
+
+    def _window(self, st, L, pool, batch, act, y, pdl, first_pdl) -> int:
         c, T = L.wc, st.T
         lib, p = X.load(), X._p
         kp, vp = pool.layer(L.index)
@@ -304,7 +324,7 @@ class HybridStack:
         X._check(lib.js_window_post(
             p(proj), proj.stride(0), p(L.qkv_bias), c.heads, c.kv_heads, L.gp, c.dim, c.vdim, L.Dq, L.Dp, L.Vp, c.rot_dims, p(L.freq),
             int(c.qk_norm), X.ctypes.c_float(L.eps), p(batch.positions), p(batch.slots), kp.shape[1], T, p(q), p(kp), p(vp),
-            p(X.status_word(self.device)), int(pdl), X._stream()), "js_window_post")
+            p(X.status_word(self.device)), int(first_pdl), X._stream()), "js_window_post")
         o = st.get("wo", L.wo_cols, zero=True)
         Hq, n = c.kv_heads * L.gp, 3
         args = (batch.slot_map, batch.seq_rows, batch.cu_q, batch.past, batch.mask)
@@ -339,27 +359,35 @@ class HybridStack:
 
     def _experts(self, st, L, out, tap, pdl) -> int:
         m, T = L.moe, st.T
-        sh, n = None, 0
-        if m.shared is not None:
-            a, sh = st.get("sa", m.shared.ff), st.get("sh", self.wp)
-            X.gemm(st.h, m.shared.up, out=a, epi=X.EPI_SWIGLU, pdl=pdl)
-            X.gemm(a, m.shared.down, out=sh, pdl=pdl)
-            n += 2
-        at, j = st.sort_off[self.routed.index(L)], 0
+        fork = m.shared is not None and self._forks(st)
+        a, sh = (st.get("sa", m.shared.ff), st.get("sh", self.wp)) if m.shared is not None else (None, None)
         pending = []
-        for t0 in range(0, T, self.pass_rows):
-            rows = min(self.pass_rows, T - t0)
-            P = rows * m.top
-            tok, inv, off = st.sort[at:at + P], st.sort[at + P:at + 2 * P], st.sort[at + 2 * P:at + 2 * P + m.E + 1]
-            at += 2 * P + m.E + 1
-            g = lambda name, c: st.get(f"{name}{t0}", c, rows=P)
-            xs, hs, ys = g("xs", self.wp), g("hs", m.ff), g("ys", m.wd)
-            X.gather_rows(st.h, tok, xs, pdl=pdl)
-            cover = min(rows, ((4 * P // m.E + 128 + 127) // 128) * 128)
-            X.gemm_grouped(xs, m.up, hs, P, 2 * m.ff, m.E, off, cover, X.EPI_SWIGLU)
-            X.gemm_grouped(hs, m.down, ys, P, m.wd, m.E, off, cover, X.EPI_STORE)
-            pending.append((ys, inv, t0, rows))
-            n += 3
+
+        def shared(first):
+            if m.shared is None:
+                return 0
+            X.gemm(st.h, m.shared.up, out=a, epi=X.EPI_SWIGLU, pdl=pdl and first)
+            X.gemm(a, m.shared.down, out=sh, pdl=pdl)
+            return 2
+
+        def routed(first):
+            at = st.sort_off[self.routed.index(L)]
+            for t0 in range(0, T, self.pass_rows):
+                rows = min(self.pass_rows, T - t0)
+                P = rows * m.top
+                tok, inv, off = st.sort[at:at + P], st.sort[at + P:at + 2 * P], st.sort[at + 2 * P:at + 2 * P + m.E + 1]
+                at += 2 * P + m.E + 1
+                g = lambda name, c: st.get(f"{name}{t0}", c, rows=P)
+                xs, hs, ys = g("xs", self.wp), g("hs", m.ff), g("ys", m.wd)
+                X.gather_rows(st.h, tok, xs, pdl=pdl)
+                cover = min(rows, ((4 * P // m.E + 128 + 127) // 128) * 128)
+                X.gemm_grouped(xs, m.up, hs, P, 2 * m.ff, m.E, off, cover, X.EPI_SWIGLU)
+                X.gemm_grouped(hs, m.down, ys, P, m.wd, m.E, off, cover, X.EPI_STORE)
+                pending.append((ys, inv, t0, rows))
+            return 3 * len(pending)
+
+        n = self._beside(fork, shared, routed)
+        pdl = pdl and not fork
         for ys, inv, t0, rows in pending:          # h is rewritten here, so every pass has read it first
             self._resid(st, L.norm2, L.eps, out, tap, pdl, ys=ys, inv=inv, k=m.top, sh=sh, t0=t0, rows=rows)
             n += 1
