@@ -123,6 +123,20 @@ def case_parallel_block(reps: int = 3):
     torch.cuda.synchronize()
 
 
+def case_delta_rule(reps: int = 3):
+    """A prompt portion of 2048 rows through the block form of the delta rule, 16 heads of 128 with one decay a head."""
+    from jetspec_b200.models import DeltaConfig
+    T, D, c = 2048, 128, DeltaConfig(16, 8, 128, 128, 4)
+    i32 = dict(dtype=torch.int32, device="cuda")
+    pre, gate, z, b = bf(T, c.channels), bf(T, 16 * D), torch.randn(T, 16, device="cuda"), torch.randn(T, 16, device="cuda")
+    A = torch.linspace(-4, 0, 16, device="cuda").to(torch.bfloat16)
+    state, conv, out = torch.zeros(2, 16, D, D, device="cuda"), bf(2, 4, c.channels), bf(T, 16 * D)
+    rows, cu, past = torch.zeros(1, **i32), torch.tensor([0, T], **i32), torch.zeros(1, **i32)
+    for _ in range(reps):
+        X.delta_forward(c, pre, z, b, bf(c.channels, 4), A, bf(16), state, conv, rows, cu, past, gate, bf(D), c.gate, 1e-6, out, max_rows=T)
+    torch.cuda.synchronize()
+
+
 def case_round_small(reps: int = 2):
     """The small kernels of a decode round at Qwen3-8B sizes: RMSNorm, per-head norm + RoPE + KV scatter, the
     draft head's vocabulary top-k (GEMM epilogue + merge), device tree build, accept + commit, KV compaction."""
@@ -211,7 +225,7 @@ def case_collectives(reps: int = 3):
 if __name__ == "__main__":
     X.load()
     {"gemm": case_gemm, "gemm_rows2048": case_gemm_rows2048, "lm_head": case_lm_head, "attention": case_attention,
-     "latent_attention": case_latent_attention, "parallel_block": case_parallel_block, "nvfp4": case_nvfp4,
+     "latent_attention": case_latent_attention, "delta_rule": case_delta_rule, "parallel_block": case_parallel_block, "nvfp4": case_nvfp4,
      "round_small": case_round_small, "collectives": case_collectives}[sys.argv[1]]()
     X.check_status("cuda")
     print("ok")

@@ -1,9 +1,9 @@
 """Paged engine: AR vs batched decode, checking that a batch reproduces per-prompt outputs.
 
-    python examples/engine_generate.py [/path/to/model | karuzen]
+    python examples/engine_generate.py [/path/to/model | karuzen | zasipel]
 
-Any registered model family loads from its directory; ``karuzen`` is a tiny random model of that design, no argument a
-tiny random Qwen3.  The batch is run once more with its prompts fed in portions beside the others' decode steps.
+Any registered model family loads from its directory; ``karuzen`` and ``zasipel`` are tiny random models of those designs,
+no argument a tiny random Qwen3.  The batch is run once more with its prompts fed in portions beside the others' decode steps.
 
 Reference counterpart: ``examples/engine/jetspec_engine_generate.py:19-64``."""
 import os
@@ -14,13 +14,16 @@ import torch
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))   # run from a checkout
 
 from jetspec_b200 import JetSpecEngine, SamplingParams  # noqa: E402
-from jetspec_b200.models import KaruzenForCausalLM, Qwen3ForCausalLM, karuzen_tiny_config, tiny_config  # noqa: E402
+from jetspec_b200.models import (KaruzenForCausalLM, Qwen3ForCausalLM, ZasipelForCausalLM, karuzen_tiny_config, tiny_config,  # noqa: E402
+                                 zasipel_tiny_config)
 
 if __name__ == "__main__":
     dev = "cuda" if torch.cuda.is_available() else "cpu"
     dt = torch.bfloat16 if dev == "cuda" else torch.float32
     if len(sys.argv) > 1 and sys.argv[1] == "karuzen":
         model = KaruzenForCausalLM.random_init(karuzen_tiny_config(), seed=0, dtype=dt, init="stable")
+    elif len(sys.argv) > 1 and sys.argv[1] == "zasipel":
+        model = ZasipelForCausalLM.random_init(zasipel_tiny_config(), seed=0, dtype=dt, init="stable")
     else:
         model = sys.argv[1] if len(sys.argv) > 1 else Qwen3ForCausalLM.random_init(tiny_config(), seed=0, dtype=dt)
     eng = JetSpecEngine(model, device=dev, dtype=dt, block_size=16)

@@ -628,6 +628,23 @@ def test_draft_head_and_sampled_trees(arm):
 
 
 @pytest.mark.gpu
+@pytest.mark.parametrize("case", ["mixed", "wide"])
+def test_long_portions_run_their_branches_side_by_side(case):
+    """From 512 rows on a portion's independent branches use two streams; short portions and single tokens do not."""
+    from jetspec_b200.engine.hybrid_stack import FORK_MIN_TOKENS
+    cfg, w, n = CASES[case], WEIGHTS[case], FORK_MIN_TOKENS + 90
+    toks = prompt(n, cfg["vocab"])
+    eng = engine_from(cfg, w, ("cuda", torch.bfloat16))
+    got = {}
+    for name, sizes in (("whole", [n]), ("portions", [64, 1, 37]), ("both", [FORK_MIN_TOKENS, 1, 2])):
+        eng.reserve_pool(n + 16, 1)
+        got[name] = replay(eng, [[("a", c)] for c in portions(n, sizes)], {"a": toks})["a"]
+    assert_rows(got["whole"], got["portions"].double(), torch.bfloat16)
+    assert_rows(got["both"], got["portions"].double(), torch.bfloat16)
+    assert_rows(got["whole"][-60:], oracle_logits(case, cfg, w, toks)[-60:], torch.bfloat16)
+
+
+@pytest.mark.gpu
 def test_experts_in_several_passes():
     """More (token, expert) pairs than one permutation takes: the tokens go through the experts in passes."""
     from jetspec_b200.engine.fast_round import FastRound
