@@ -5,10 +5,10 @@
 // shared key/value matrix, and one gathered tile of latent rows serves as K (K-major operand) and as V (MN-major operand)
 // of both MMAs: a cached byte is read once per (128 query rows, column group).
 //
-//   * rows: a sequence's (token, head) pairs in row-major order, 128 per CTA, any number of heads;
+//   * rows: a sequence's (token, head) pairs in row-major order, 128 per CTA (64 for rows above 512 wide), any number of heads;
 //   * S = QA C^T and O += P C are tcgen05.mma with M = 128; S (two buffers) and O (up to 256 columns) live in tensor
-//     memory; latents wider than 256 are covered by two column groups (grid y), each computing all scores and its own half
-//     of the output columns;
+//     memory; outputs wider than 256 are covered by two column groups (grid y), each computing all scores and its own half
+//     of the output columns; columns behind the latent (a rotated key part) enter the scores only;
 //   * latent rows are gathered by slot with cp.async into 128-byte-swizzled tiles of 64 columns, TK keys each;
 //   * with few query rows (decode) only RQ = 32 or 64 rows of Q and P are kept in shared memory: an MMA's other rows then
 //     read whatever follows them, which only reaches accumulator rows nobody reads;
@@ -44,8 +44,13 @@ struct LatentAttnParams {
   int* status;
   int B, T, H, Rp, S, max_len, W, causal, splits;
   float scale_log2;
+  const float* sinks;          // (H) a valueless key's score (unscaled) per head, counted by the last split; may be null
+  const float* gate;           // (T, ldg) logits: head h's output is multiplied by sigmoid(gate[t, h]); may be null
+  int ldg;
   int nk;                      // 64-column chunks of a latent row
+  int nout;                    // leading chunks that are output
   int chunks0;                 // chunks of column group 0 (the rest belong to group 1)
+  int trows;                   // query rows per CTA: 128 or 64
   int rq;                      // query rows kept in shared memory: 32, 64 or 128
   int stages;
 };
@@ -119,21 +124,21 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int grp = blockIdx.y, split = blockIdx.z;
   const int v0 = grp == 0 ? 0 : p.chunks0;                       // first column chunk of this CTA's output
-  const int nv = grp == 0 ? p.chunks0 : nk - p.chunks0;          // and how many (at most 4)
+  const int nv = grp == 0 ? p.chunks0 : p.nout - p.chunks0;      // and how many (at most 4)
 
   pdl_launch_dependents();
   pdl_wait();
 
   int lo = 0, hi = p.B - 1;
   const int tile = blockIdx.x;
-  while (lo < hi) {      // sequence b starts at tile cu_q[b]*H/128 + b
+  while (lo < hi) {      // sequence b starts at tile cu_q[b]*H/trows + b
     const int mid = (lo + hi + 1) >> 1;
-    if (static_cast<int>(static_cast<long long>(p.cu_q[mid]) * p.H / LROWS) + mid <= tile) lo = mid; else hi = mid - 1;
+    if (static_cast<int>(static_cast<long long>(p.cu_q[mid]) * p.H / p.trows) + mid <= tile) lo = mid; else hi = mid - 1;
   }
   const int b = lo;
   const int q_begin = p.cu_q[b], n_b = p.cu_q[b + 1] - q_begin;
-  const int row0 = (tile - (static_cast<int>(static_cast<long long>(q_begin) * p.H / LROWS) + b)) * LROWS;
-  const int n_rows = min(LROWS, n_b * p.H - row0);
+  const int row0 = (tile - (static_cast<int>(static_cast<long long>(q_begin) * p.H / p.trows) + b)) * p.trows;
+  const int n_rows = min(p.trows, n_b * p.H - row0);
   if (n_rows <= 0) return;
   const int past = p.past_lens[b];
   const int* slots = p.slot_map + static_cast<size_t>(p.seq_rows[b]) * p.max_len;
@@ -306,6 +311,12 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
       mw[w] = (!p.causal && row_valid && w < p.W) ? p.mask_bits[static_cast<size_t>(q_begin + node) * p.W + w] : 0;
     constexpr unsigned long long kAll = TK == 64 ? ~0ull : (1ull << (TK & 63)) - 1ull;
     float m_run = -INFINITY, l_run = 0.f;
+    const int head = (row0 + (row_valid ? row : 0)) % p.H;
+    if (p.sinks != nullptr && split == p.splits - 1) {   // the last split always has a tile
+      const float s2 = p.sinks[head] * 1.4426950408889634f;
+      m_run = ceilf(s2);
+      l_run = exp2f(s2 - m_run);
+    }
     bool ok = true;
     for (int i = 0; i < nt && ok; ++i) {
       const int sb = i & 1;
@@ -409,7 +420,8 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
     if (ok) ok = lat_mbar_wait(o_done, 0, p.status, kTimeoutAccum);
     tc_fence_after();
     if (ok) {
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if (p.gate != nullptr) inv /= 1.f + expf(-p.gate[static_cast<size_t>(q_begin + node) * p.ldg + head]);
 #pragma unroll 1
       for (int c0 = 0; c0 < nv * 64; c0 += 32) {
         uint32_t orr[32];
@@ -451,7 +463,8 @@ __global__ void __launch_bounds__(LTHREADS, 1) latent_attn_tc_kernel(LatentAttnP
 // one CTA per (token, head) row: merge the key splits (at most 16; four columns per thread)
 constexpr int LMAX_SPLITS = 16;
 __global__ void __launch_bounds__(128)
-latent_attn_merge_kernel(const float* ws_o, const float* ws_ml, __nv_bfloat16* out, int rows, int Rp, int splits) {
+latent_attn_merge_kernel(const float* ws_o, const float* ws_ml, __nv_bfloat16* out, int rows, int H, int Rp, int cols, int splits,
+                         const float* gate, int ldg) {
   pdl_launch_dependents();
   pdl_wait();
   const int row = blockIdx.x, c = threadIdx.x * 4;
@@ -462,11 +475,12 @@ latent_attn_merge_kernel(const float* ws_o, const float* ws_ml, __nv_bfloat16* o
     if (s < splits) ml = *reinterpret_cast<const float2*>(ws_ml + (static_cast<size_t>(s) * rows + row) * 2);
     const float m = warp_max(ml.x);
     const float f = ml.x == -INFINITY ? 0.f : exp2f(ml.x - m);
-    const float l = warp_sum(ml.y * f);
+    float l = warp_sum(ml.y * f);
+    if (gate != nullptr) l *= 1.f + expf(-gate[static_cast<size_t>(row / H) * ldg + row % H]);
     if (s < LMAX_SPLITS) w[s] = l > 0.f ? f / l : 0.f;
   }
   __syncthreads();
-  if (c >= Rp) return;
+  if (c >= cols) return;
   float acc[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 4
   for (int s = 0; s < splits; ++s) {
@@ -500,21 +514,25 @@ static int launch_latent(const LatentAttnParams& p, int q_tiles, int groups, int
 
 }  // namespace js
 
-// q, out (T*H, Rp) bf16, pool (S, Rp) bf16, Rp a multiple of 64 up to 512; max_q = most query tokens of one sequence;
+// q, out (T*H, Rp) bf16, pool (S, Rp) bf16, Rp a multiple of 64 up to 768, of which the first out_cols (at most 512) are values;
+// sinks (H) and gate (T, ldg) fp32 or null; max_q = most query tokens of one sequence;
 // masks of up to 8 words per token; tk_want = keys per tile (32, or 64 where it fits; 0 picks).  splits > 1 needs ws_o (splits, T*H, Rp) fp32 and ws_ml (splits, T*H, 2) fp32.
 extern "C" int js_latent_attention_tc(const void* q, const void* pool, const int* slot_map, const int* seq_rows, const int* cu_q,
                                       const int* past_lens, const int* mask_bits, void* out, float* ws_o, float* ws_ml, int* status,
-                                      int B, int T, int H, int Rp, int S, int max_len, int W, int causal, int splits, int max_q,
-                                      float scale, int tk_want, int pdl, cudaStream_t stream) {
+                                      int B, int T, int H, int Rp, int out_cols, int S, int max_len, int W, int causal, int splits, int max_q,
+                                      float scale, const float* sinks, const float* gate, int ldg, int tk_want, int pdl,
+                                      cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
-  if (Rp % 64 || Rp < 64 || Rp > 512 || H < 1) return -10;
+  const int nout = (out_cols + 63) / 64;
+  if (Rp % 64 || Rp < 64 || Rp > 768 || nout < 1 || nout > 8 || nout > Rp / 64 || H < 1) return -10;
   if (splits < 1 || splits > LMAX_SPLITS) return -11;
   if (splits > 1 && (ws_o == nullptr || ws_ml == nullptr)) return -12;
   if (!causal && (mask_bits == nullptr || W < 1 || W > 8)) return -13;
   const int nk = Rp / 64;
   const long long rows = static_cast<long long>(max_q < 1 ? T : max_q) * H;
-  const int rq = rows <= 32 ? 32 : rows <= 64 ? 64 : 128;
+  const int trows = Rp > 512 ? 64 : LROWS;        // a wide row leaves shared memory for 64 queries only
+  const int rq = rows <= 32 ? 32 : rows <= 64 || trows == 64 ? 64 : 128;
   const int budget = kLatentSmemMax - 1024 - 256;
   int tk = 64, stages = (budget - nk * rq * 128 - lat_p_bytes(64, rq)) / lat_stage_bytes(64, nk);
   if (tk_want != 0 && tk_want != 32 && tk_want != 64) return -10;
@@ -524,16 +542,16 @@ extern "C" int js_latent_attention_tc(const void* q, const void* pool, const int
   }
   if (stages < 2) return -18;
   if (stages > LMAX_STAGES) stages = LMAX_STAGES;
-  const int chunks0 = nk <= 4 ? nk : (nk + 1) / 2;
+  const int chunks0 = nout <= 4 ? nout : (nout + 1) / 2;
   LatentAttnParams p{reinterpret_cast<const __nv_bfloat16*>(q), reinterpret_cast<const __nv_bfloat16*>(pool), slot_map, seq_rows, cu_q,
                      past_lens, mask_bits, reinterpret_cast<__nv_bfloat16*>(out), ws_o, ws_ml, status, B, T, H, Rp, S, max_len, W,
-                     causal, splits, scale * 1.4426950408889634f, nk, chunks0, rq, stages};
+                     causal, splits, scale * 1.4426950408889634f, sinks, gate, ldg, nk, nout, chunks0, trows, rq, stages};
   int smem = 1024 + nk * rq * 128 + lat_p_bytes(tk, rq) + stages * lat_stage_bytes(tk, nk) + 256;
   // an MMA reads 128 rows from every Q chunk and P buffer: what follows them must reach at least that far
   const int after_p = stages * lat_stage_bytes(tk, nk) + rq * 128;
   if (after_p < LROWS * 128) return -18;
-  const int q_tiles = static_cast<int>(static_cast<long long>(T) * H / LROWS) + B;
-  const int groups = chunks0 < nk ? 2 : 1;
+  const int q_tiles = static_cast<int>(static_cast<long long>(T) * H / trows) + B;
+  const int groups = chunks0 < nout ? 2 : 1;
   const int rc = tk == 64 ? launch_latent<64>(p, q_tiles, groups, smem, pdl != 0, stream)
                           : launch_latent<32>(p, q_tiles, groups, smem, pdl != 0, stream);
   if (rc != 0 || splits == 1) return rc;
@@ -547,5 +565,5 @@ extern "C" int js_latent_attention_tc(const void* q, const void* pool, const int
   c2.attrs = attr;
   c2.numAttrs = pdl ? 1 : 0;
   return cudaLaunchKernelEx(&c2, latent_attn_merge_kernel, static_cast<const float*>(ws_o), static_cast<const float*>(ws_ml),
-                            reinterpret_cast<__nv_bfloat16*>(out), T * H, Rp, splits) == cudaSuccess ? 0 : -5;
+                            reinterpret_cast<__nv_bfloat16*>(out), T * H, H, Rp, nout * 64, splits, gate, ldg) == cudaSuccess ? 0 : -5;
 }

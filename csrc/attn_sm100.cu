@@ -42,6 +42,8 @@ struct AttnParams {
   int B, T, Hq, Hkv, S, max_len, W, causal, splits;
   float scale_log2;            // softmax scale * log2(e)
   int ldo;                     // merge kernel: elements between tokens of `out`
+  const float* gate;           // merge kernel: (T, ldg) logits, a head's output is multiplied by their sigmoid; may be null
+  int ldg;
 };
 
 JS_DEVICE void cp_async16(void* smem, const void* gmem, bool valid) {
@@ -314,7 +316,8 @@ __global__ void attn_merge_kernel(AttnParams p) {
     const float4 v = *reinterpret_cast<const float4*>(p.ws_o + (s * stride + row) * AD + lane * 4);
     acc[0] += v.x * w; acc[1] += v.y * w; acc[2] += v.z * w; acc[3] += v.w * w;
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  if (p.gate != nullptr) inv /= 1.f + expf(-p.gate[static_cast<size_t>(row / p.Hq) * p.ldg + row % p.Hq]);
   __nv_bfloat16* dst = p.out + static_cast<size_t>(row / p.Hq) * p.ldo + (row % p.Hq) * AD + lane * 4;
   *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(acc[0] * inv, acc[1] * inv);
   *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(acc[2] * inv, acc[3] * inv);
@@ -381,12 +384,13 @@ extern "C" int js_paged_tree_attention(const void* q, const void* k_pool, const 
 }
 
 // Merge the key splits of a (splits, T, Hq, 128) fp32 workspace with its (max, sum) pairs into out (T, Hq*128), ldo elements
-// between tokens.
-extern "C" int js_attn_merge(float* ws_o, float* ws_ml, void* out, int ldo, int T, int Hq, int splits, int pdl, cudaStream_t stream) {
+// between tokens; gate (T, ldg) logits multiply a head's output by their sigmoid (null: none).
+extern "C" int js_attn_merge(float* ws_o, float* ws_ml, const float* gate, int ldg, void* out, int ldo, int T, int Hq, int splits, int pdl,
+                             cudaStream_t stream) {
   using namespace js;
   AttnParams p{};
   p.ws_o = ws_o; p.ws_ml = ws_ml; p.out = reinterpret_cast<__nv_bfloat16*>(out);
-  p.T = T; p.Hq = Hq; p.splits = splits; p.ldo = ldo;
+  p.T = T; p.Hq = Hq; p.splits = splits; p.ldo = ldo; p.gate = gate; p.ldg = ldg;
   cudaLaunchConfig_t c2 = {};
   c2.gridDim = dim3((T * Hq + 7) / 8);
   c2.blockDim = dim3(256);

@@ -59,7 +59,11 @@ struct AttnTcParams {
   long long kv_head, kv_slot;  // elements between heads / slots of the pools (S*128 and 128 for a (Hkv, S, 128) pool)
   int ldo;                     // elements between tokens of `out`
   int window;                  // > 0: a row sees the last `window` tokens of its own path only
-  int sink;                    // a valueless key of score 0 takes part in the softmax (counted by the last split)
+  int sink;                    // a valueless key takes part in the softmax (counted by the last split)
+  int keep;                    // positions below it stay visible behind the window
+  const float* sinks;          // (Hq) the valueless key's score (unscaled), null: 0
+  const float* gate;           // (T, ldg) logits: head h's output is multiplied by sigmoid(gate[t, h]); may be null
+  int ldg;
   int cluster_merge;           // the key splits of a tile form a cluster and merge through distributed shared memory
 };
 
@@ -166,10 +170,16 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   if (p.causal) L = min(L, past + node0 + NPT);
   // first key tile any row of this CTA can see (a tree's root sits at position `past`)
   const int t_first = p.window > 0 ? max(0, past + (p.causal ? node0 : 0) - p.window + 1) / TKEYS : 0;
-  const int n_tiles = (L + TKEYS - 1) / TKEYS - t_first;
-  const int t_begin = t_first + (n_tiles * split) / p.splits;
-  const int t_end = t_first + (n_tiles * (split + 1)) / p.splits;
+  // ... behind the tiles of kept first tokens: the CTA's tiles are 0 .. t_kept - 1 and t_first, t_first + 1, ...
+  const int t_kept = p.window > 0 ? min(t_first, (p.keep + TKEYS - 1) / TKEYS) : 0;
+  const int n_tiles = (L + TKEYS - 1) / TKEYS - t_first + t_kept;
+  const int t_begin = (n_tiles * split) / p.splits;
+  const int t_end = (n_tiles * (split + 1)) / p.splits;
   const int nt = t_end - t_begin;
+  auto tile_key = [&](int i) {          // first key of this split's tile i
+    const int t = t_begin + i;
+    return (t < t_kept ? t : t - t_kept + t_first) * TKEYS;
+  };
 
   // softmax thread's row
   const int row = (warp & 3) * 32 + lane;
@@ -180,7 +190,12 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 
   const bool cmerge = p.cluster_merge != 0;
   float m_run = -INFINITY, l_run = 0.f;     // softmax threads: running (integer) maximum and sum of their row
-  if (p.sink && split == p.splits - 1) { m_run = 0.f; l_run = 1.f; }     // the last split always has a tile
+  if (p.sink && split == p.splits - 1) {    // the last split always has a tile
+    const float s2 = p.sinks != nullptr && row_valid ? p.sinks[head] * 1.4426950408889634f : 0.f;
+    m_run = ceilf(s2);
+    l_run = exp2f(s2 - m_run);
+  }
+  const float gate = p.gate != nullptr && row_valid ? 1.f / (1.f + expf(-p.gate[static_cast<size_t>(q_begin + node) * p.ldg + head])) : 1.f;
   bool sm_ok = true;
   if (nt <= 0 && !cmerge) {   // more splits than key tiles: this split contributes nothing
     if (warp < 4 && row_valid && p.splits > 1) {
@@ -230,7 +245,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
     int slot_next[TKEYS / RSTEP];
 #pragma unroll
     for (int j = 0; j < TKEYS / RSTEP; ++j) {
-      const int kp = t_begin * TKEYS + r0 + RSTEP * j;
+      const int kp = tile_key(0) + r0 + RSTEP * j;
       slot_next[j] = kp < L ? __ldg(slots + kp) : 0;
     }
     bool ok = true;
@@ -255,13 +270,13 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         }
       }
       if (!ok) break;
-      const int k0 = (t_begin + i) * TKEYS;
+      const int k0 = tile_key(i), k0n = tile_key(i + 1);
       const uint32_t k_addr = smem_u32(sKV + s * kStageKV);
       int slot_cur[TKEYS / RSTEP];
 #pragma unroll
       for (int j = 0; j < TKEYS / RSTEP; ++j) {
         slot_cur[j] = slot_next[j];
-        const int kpn = k0 + TKEYS + r0 + RSTEP * j;
+        const int kpn = k0n + r0 + RSTEP * j;
         slot_next[j] = (i + 1 < nt && kpn < L) ? __ldg(slots + kpn) : 0;
       }
 #pragma unroll
@@ -348,10 +363,17 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 #pragma unroll
         for (int w = 0; w < 8; ++w) cnt += __popc(static_cast<unsigned>(mw[w]));
         cut = min(past, past + cnt - p.window);
-        int drop = cnt - p.window;     // ancestors out of the window are the lowest bits
+        // ancestors out of the window are the lowest bits (the d-th lowest is at position past + d); kept ones stay
+        int drop = cnt - p.window, spare = p.keep - past;
 #pragma unroll
-        for (int w = 0; w < 8; ++w)
-          for (; drop > 0 && mw[w] != 0; --drop) mw[w] &= mw[w] - 1;
+        for (int w = 0; w < 8; ++w) {
+          unsigned rest = static_cast<unsigned>(mw[w]);
+          for (; drop > 0 && rest != 0u; --drop, --spare) {
+            const unsigned low = rest & (0u - rest);
+            if (spare <= 0) mw[w] &= static_cast<int>(~low);
+            rest ^= low;
+          }
+        }
       }
     }
     bool ok = true;
@@ -366,7 +388,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
       tmem_ld_32x32(tmem_base + t_lane + sb * TKEYS + 32, sr + 32);
       tmem_ld_wait();
       // visibility of the tile's 64 keys for this row, as one 64-bit word (bit c = key k0 + c)
-      const int k0 = (t_begin + i) * TKEYS;
+      const int k0 = tile_key(i);
       const int jlo = k0 - past;                         // window index of the tile's first key (may be < 0)
       unsigned long long vm = 0ull;
       if (row_valid) {
@@ -390,7 +412,11 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         const int left = L - k0;                         // keys at or past L do not exist
         if (left < 64) vm &= (left <= 0) ? 0ull : ((1ull << left) - 1ull);
         const int hidden = cut - k0;                     // this many of the tile's keys lie before the window
-        if (hidden > 0) vm = hidden >= 64 ? 0ull : vm & (~0ull << hidden);
+        if (hidden > 0) {
+          const int kept = p.keep - k0;                  // ... of which the first `kept` are visible all the same
+          const unsigned long long stay = kept >= 64 ? ~0ull : kept > 0 ? (1ull << kept) - 1ull : 0ull;
+          vm &= (hidden >= 64 ? 0ull : ~0ull << hidden) | stay;
+        }
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // four chains instead of one 64-deep
       if (vm == ~0ull) {              // the common case: every key of the tile is visible to this row
@@ -464,7 +490,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
     if (tid == 0) attn_trace(3);    // output accumulator complete
     sm_ok = ok;
     if (ok && !cmerge) {
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      const float inv = l_run > 0.f ? gate / l_run : 0.f;
 #pragma unroll 1
       for (int c0 = 0; c0 < TD; c0 += 32) {
         uint32_t orr[32];
@@ -545,7 +571,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         wsrc[s2] = (ms == -INFINITY) ? 0.f : exp2f(ms - m);
         lsum += recv_ml[(s2 * TROWS + row) * 2 + 1] * wsrc[s2];
       }
-      const float inv = lsum > 0.f ? 1.f / lsum : 0.f;
+      const float inv = lsum > 0.f ? gate / lsum : 0.f;
       for (int c = split; c < 4; c += p.splits) {
         float acc[32];
 #pragma unroll
@@ -613,7 +639,8 @@ extern "C" int js_attn_tc_set_trace(unsigned long long* buf) {
   return cudaMemcpyToSymbol(js::g_attn_trace, &buf, sizeof(buf)) == cudaSuccess ? 0 : -1;
 }
 
-extern "C" int js_attn_merge(float* ws_o, float* ws_ml, void* out, int ldo, int T, int Hq, int splits, int pdl, cudaStream_t stream);
+extern "C" int js_attn_merge(float* ws_o, float* ws_ml, const float* gate, int ldg, void* out, int ldo, int T, int Hq, int splits, int pdl,
+                             cudaStream_t stream);
 
 // How many clusters of `splits` CTAs of the kernel for GQA group size G can be resident at once on the current
 // device (a cluster lives inside one GPC, so this is less than SMs / splits); 0 or negative = cannot say.  The host
@@ -650,14 +677,16 @@ extern "C" int js_attn_tc_max_active_clusters(int G, int splits) {
 // js_paged_tree_attention with the layout of the pools and the output spelled out: head h of slot s starts at
 // h * kv_head + s * kv_slot, token t of the output at t * ldo (all multiples of 8).  Needs 128 % (Hq / Hkv) == 0 and
 // W <= 8 (windows of up to 256 nodes).
-// window > 0 limits a row to the last `window` tokens of its own path; sink adds a valueless key of score 0.
+// window > 0 limits a row to the last `window` tokens of its own path and the positions below `keep`; sink adds a valueless
+// key of score sinks[head] (null: 0); gate (T, ldg) fp32 logits multiply a head's output by their sigmoid (null: none).
 extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
                                       const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
                                       float* ws_o, float* ws_ml, int* status, int B, int T, int Hq, int Hkv, int S, int max_len, int W,
-                                      int causal, int splits, float scale, int window, int sink, long long kv_head, long long kv_slot,
-                                      int ldo, int pdl, cudaStream_t stream) {
+                                      int causal, int splits, float scale, int window, int sink, int keep, const float* sinks,
+                                      const float* gate, int ldg, long long kv_head, long long kv_slot, int ldo, int pdl,
+                                      cudaStream_t stream) {
   using namespace js;
-  if (window < 0) return -10;
+  if (window < 0 || keep < 0) return -10;
   if (T <= 0 || B <= 0) return 0;
   if (Hq % Hkv) return -10;
   if ((kv_head % 8) || (kv_slot % 8) || (ldo % 8)) return -10;
@@ -686,7 +715,8 @@ extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const v
   AttnTcParams p{reinterpret_cast<const __nv_bfloat16*>(q), reinterpret_cast<const __nv_bfloat16*>(k_pool),
                  reinterpret_cast<const __nv_bfloat16*>(v_pool), slot_map, seq_rows, cu_q, past_lens, mask_bits,
                  reinterpret_cast<__nv_bfloat16*>(out), ws_o, ws_ml, status, B, T, Hq, Hkv, S, max_len, W, causal,
-                 splits, scale * 1.4426950408889634f, kv_head, kv_slot, ldo, window, sink, in_cluster ? 1 : 0};
+                 splits, scale * 1.4426950408889634f, kv_head, kv_slot, ldo, window, sink, keep, sinks, gate, ldg,
+                 in_cluster ? 1 : 0};
   int rc;
   switch (G) {
     case 1: rc = launch_attn_tc<1>(p, (T + 127) / 128 + B, pdl != 0, stream); break;
@@ -697,16 +727,19 @@ extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const v
     default: return -14;
   }
   if (rc != 0 || splits == 1 || p.cluster_merge) return rc;
-  return js_attn_merge(ws_o, ws_ml, out, ldo, T, Hq, splits, pdl, stream);
+  return js_attn_merge(ws_o, ws_ml, gate, ldg, out, ldo, T, Hq, splits, pdl, stream);
 }
 
+// The same without a window; sinks and gate may be null.
 extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
                                           const int* seq_rows, const int* cu_q, const int* past_lens,
                                           const int* mask_bits, void* out, float* ws_o, float* ws_ml, int* status, int B,
                                           int T, int Hq, int Hkv, int S, int max_len, int W, int causal, int splits,
-                                          float scale, long long kv_head, long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
+                                          float scale, const float* sinks, const float* gate, int ldg, long long kv_head,
+                                          long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
   return js_window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ws_o, ws_ml, status, B, T, Hq,
-                                Hkv, S, max_len, W, causal, splits, scale, 0, 0, kv_head, kv_slot, ldo, pdl, stream);
+                                Hkv, S, max_len, W, causal, splits, scale, 0, sinks != nullptr, 0, sinks, gate, ldg, kv_head, kv_slot, ldo,
+                                pdl, stream);
 }
 
 // Same arguments as js_paged_tree_attention.
@@ -716,6 +749,6 @@ extern "C" int js_paged_tree_attention_tc(const void* q, const void* k_pool, con
                                           int T, int Hq, int Hkv, int S, int max_len, int W, int causal, int splits,
                                           float scale, int pdl, cudaStream_t stream) {
   return js_paged_attention_tc_strided(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ws_o, ws_ml, status,
-                                       B, T, Hq, Hkv, S, max_len, W, causal, splits, scale,
+                                       B, T, Hq, Hkv, S, max_len, W, causal, splits, scale, nullptr, nullptr, 0,
                                        static_cast<long long>(S) * js::TD, js::TD, Hq * js::TD, pdl, stream);
 }

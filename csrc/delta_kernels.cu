@@ -9,6 +9,8 @@
 //   path    the stored state advances along chosen rows (the accepted nodes of a tree), nothing is read out.
 // A sequence whose committed length is 0 starts from zeros whatever its state slot holds.
 //
+// Retention is the same walk with u = v and one constant decay per head (js_retention_seq).
+//
 // The convolutions' last inputs are a ring per state slot: the un-convolved row of position p is entry p % taps, so a
 // decode step writes an entry that no reader of the same step looks at.
 #include "common.cuh"
@@ -40,6 +42,7 @@ constexpr int kMaxTaps = 17;
 struct DeltaShape {
   int H, G, D, V, taps;
   int channel;      // one decay per (head, key channel) instead of one per head
+  const float* decay;       // retention: the heads' constant decays (H)
 };
 
 // ---------------------------------------------------------------- inputs of the recurrence
@@ -179,11 +182,15 @@ JS_DEVICE void delta_store_conv_head(const DeltaShape& s, void* conv, const void
   }
 }
 
+// kinds of recurrence: delta rule with a decay per head or per key channel, retention
+enum : int { kRecHead = 0, kRecChannel = 1, kRecRetention = 2 };
+
 // R lanes share a column: lane r holds the rows 4 (i R + r) .. + 3.  DP: dim rounded up (32, 64, 128, 256).
-template <int DP, int R, int TB, bool CH, int MODE>
+template <int DP, int R, int TB, int REC, int MODE>
 __global__ void __launch_bounds__(kDeltaCols* R)
 delta_seq_kernel(DeltaSeqParams p) {
   constexpr int NT = kDeltaCols * R, NI = DP / (4 * R);
+  constexpr bool CH = REC == kRecChannel, RET = REC == kRecRetention;
   __shared__ __align__(16) float sq[2][TB][DP], sk[2][TB][DP], sg[2][TB][CH ? DP : 1];
   __shared__ float sv[2][TB][kDeltaCols], sb[2][TB];
   __shared__ int spath[kDeltaMaxPath];
@@ -235,8 +242,8 @@ delta_seq_kernel(DeltaSeqParams p) {
     for (int j = tid; j < TB; j += NT) {
       const bool ok = t0 + j < n;
       const size_t t = q0 + (ok ? (MODE == kDeltaCausal ? t0 + j : spath[t0 + j]) : 0);
-      sb[buf][j] = ok ? p.beta[t * s.H + h] : 0.f;
-      if (!CH) sg[buf][j][0] = ok ? expf(p.gl[t * s.H + h]) : 1.f;
+      sb[buf][j] = ok && !RET ? p.beta[t * s.H + h] : 0.f;
+      if (!CH) sg[buf][j][0] = !ok ? 1.f : RET ? s.decay[h] : expf(p.gl[t * s.H + h]);
     }
   };
   auto walk = [&](float (&S)[NI][4], int n) {
@@ -258,12 +265,16 @@ delta_seq_kernel(DeltaSeqParams p) {
           kk[i] = k4[i * R + r];
           const float4 gg = CH ? g4[i * R + r] : make_float4(gs, gs, gs, gs);
           S[i][0] *= gg.x; S[i][1] *= gg.y; S[i][2] *= gg.z; S[i][3] *= gg.w;
-          d0 += S[i][0] * kk[i].x; d1 += S[i][1] * kk[i].y; d2 += S[i][2] * kk[i].z; d3 += S[i][3] * kk[i].w;
+          if (!RET) {
+            d0 += S[i][0] * kk[i].x; d1 += S[i][1] * kk[i].y; d2 += S[i][2] * kk[i].z; d3 += S[i][3] * kk[i].w;
+          }
         }
-        float d = (d0 + d1) + (d2 + d3);
+        float d = (d0 + d1) + (d2 + d3), u = sv[buf][j][tid / R];
+        if (!RET) {
 #pragma unroll
-        for (int o = R / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
-        const float u = sb[buf][j] * (sv[buf][j][tid / R] - d);
+          for (int o = R / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xffffffffu, d, o);
+          u = sb[buf][j] * (u - d);
+        }
         d0 = d1 = d2 = d3 = 0.f;
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
@@ -362,16 +373,21 @@ static int launch_delta_seq(const DeltaSeqParams& p, int mode, int pdl, cudaStre
   a.val.programmaticStreamSerializationAllowed = 1;
   c.attrs = &a;
   c.numAttrs = pdl ? 1 : 0;
-  cudaError_t e;
-  if (p.s.channel)
-    e = mode == kDeltaCausal ? cudaLaunchKernelEx(&c, delta_seq_kernel<DP, R, TB, true, kDeltaCausal>, p)
-      : mode == kDeltaTree   ? cudaLaunchKernelEx(&c, delta_seq_kernel<DP, R, TB, true, kDeltaTree>, p)
-                             : cudaLaunchKernelEx(&c, delta_seq_kernel<DP, R, TB, true, kDeltaPath>, p);
-  else
-    e = mode == kDeltaCausal ? cudaLaunchKernelEx(&c, delta_seq_kernel<DP, R, TB, false, kDeltaCausal>, p)
-      : mode == kDeltaTree   ? cudaLaunchKernelEx(&c, delta_seq_kernel<DP, R, TB, false, kDeltaTree>, p)
-                             : cudaLaunchKernelEx(&c, delta_seq_kernel<DP, R, TB, false, kDeltaPath>, p);
+  auto pick = [&](auto causal, auto tree, auto path) {
+    return mode == kDeltaCausal ? cudaLaunchKernelEx(&c, causal, p) : mode == kDeltaTree ? cudaLaunchKernelEx(&c, tree, p) : cudaLaunchKernelEx(&c, path, p);
+  };
+#define JS_WALK(REC) \
+  pick(delta_seq_kernel<DP, R, TB, REC, kDeltaCausal>, delta_seq_kernel<DP, R, TB, REC, kDeltaTree>, delta_seq_kernel<DP, R, TB, REC, kDeltaPath>)
+  const cudaError_t e = p.s.decay != nullptr ? JS_WALK(kRecRetention) : p.s.channel ? JS_WALK(kRecChannel) : JS_WALK(kRecHead);
+#undef JS_WALK
   return e == cudaSuccess ? 0 : -4;
+}
+
+static int launch_walk(const DeltaSeqParams& p, int mode, int pdl, cudaStream_t stream) {
+  if (p.s.D <= 32) return launch_delta_seq<32, 4, 8>(p, mode, pdl, stream);
+  if (p.s.D <= 64) return launch_delta_seq<64, 4, 8>(p, mode, pdl, stream);
+  if (p.s.D <= 128) return launch_delta_seq<128, 4, 8>(p, mode, pdl, stream);
+  return launch_delta_seq<256, 8, 4>(p, mode, pdl, stream);
 }
 
 // ---------------------------------------------------------------- read-out
@@ -392,7 +408,7 @@ gated_head_norm_kernel(const float* o, const E* w, const E* gate, int ldg, E* ou
     float y = 0.f;
     if (d < V) {
       const float z = dl_ld(gate + static_cast<size_t>(t) * ldg + h * V + d);
-      y = src[d] * r * dl_ld(w + d) * (silu ? dl_silu(z) : dl_sigmoid(z));
+      y = src[d] * r * (w != nullptr ? dl_ld(w + d) : 1.f) * (silu ? dl_silu(z) : dl_sigmoid(z));
     }
     dl_st(out + static_cast<size_t>(t) * ldo + h * Vp + d, y);
   }
@@ -425,7 +441,7 @@ gated_head_norm_vec_kernel(const float* o, const __nv_bfloat16* w, const __nv_bf
     const int d = 4 * (lane + 32 * j);
     if (d >= V) continue;
     const __nv_bfloat162* z2 = reinterpret_cast<const __nv_bfloat162*>(&zr[j]);
-    const uint2 wr = *reinterpret_cast<const uint2*>(w + d);
+    const uint2 wr = w != nullptr ? *reinterpret_cast<const uint2*>(w + d) : make_uint2(0x3f803f80u, 0x3f803f80u);      // bf16 ones
     const __nv_bfloat162* w2 = reinterpret_cast<const __nv_bfloat162*>(&wr);
     const float2 za = __bfloat1622float2(z2[0]), zb = __bfloat1622float2(z2[1]);
     const float2 wa = __bfloat1622float2(w2[0]), wb = __bfloat1622float2(w2[1]);
@@ -468,7 +484,7 @@ extern "C" int js_delta_prep(int H, int G, int D, int V, int ntaps, int channel,
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
   if (!delta_shape_ok(H, G, D, V, ntaps)) return -10;
-  const DeltaShape s{H, G, D, V, ntaps, channel};
+  const DeltaShape s{H, G, D, V, ntaps, channel, nullptr};
   DeltaLaunch l(dim3(T, (2 * G + 2 * H + 7) / 8), dim3(256), stream, pdl);
   using bf = __nv_bfloat16;
   const cudaError_t e =
@@ -493,15 +509,31 @@ extern "C" int js_delta_seq(int mode, int H, int G, int D, int V, int ntaps, int
   if (mode == kDeltaPath && (path == nullptr || path_len == nullptr || B != 1)) return -13;
   if (mode != kDeltaPath && out == nullptr) return -13;
   DeltaSeqParams p{};
-  p.s = DeltaShape{H, G, D, V, ntaps, channel};
+  p.s = DeltaShape{H, G, D, V, ntaps, channel, nullptr};
   p.q = q; p.k = k; p.v = v; p.gl = gl; p.beta = beta; p.state = state;
   p.rows = rows; p.cu_q = cu_q; p.past_lens = past_lens; p.B = B;
   p.mask_bits = mask_bits; p.W = W; p.leaf_groups = leaf_groups; p.path = path; p.path_len = path_len;
   p.out = out; p.pre = pre; p.ldp = ldp; p.pre_bf16 = bf16; p.conv = conv;
-  if (D <= 32) return launch_delta_seq<32, 4, 8>(p, mode, pdl, stream);
-  if (D <= 64) return launch_delta_seq<64, 4, 8>(p, mode, pdl, stream);
-  if (D <= 128) return launch_delta_seq<128, 4, 8>(p, mode, pdl, stream);
-  return launch_delta_seq<256, 8, 4>(p, mode, pdl, stream);
+  return launch_walk(p, mode, pdl, stream);
+}
+
+// Retention over prepared fp32 rows q, k (T, H, D), v (T, H, V) with the heads' decays (H); modes and the rest as above.
+extern "C" int js_retention_seq(int mode, int H, int D, int V, const float* q, const float* k, const float* v, const float* decay,
+                                float* state, const int* rows, const int* cu_q, const int* past_lens, int B, const int* mask_bits, int W,
+                                int leaf_groups, const int* path, const int* path_len, float* out, int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (B <= 0) return 0;
+  if (!delta_shape_ok(H, H, D, V, 1) || mode < 0 || mode > 2 || decay == nullptr) return -10;
+  if (mode == kDeltaTree && (mask_bits == nullptr || W < 1 || W > 8 || leaf_groups < 1)) return -13;
+  if (mode == kDeltaPath && (path == nullptr || path_len == nullptr || B != 1)) return -13;
+  if (mode != kDeltaPath && out == nullptr) return -13;
+  DeltaSeqParams p{};
+  p.s = DeltaShape{H, H, D, V, 1, 0, decay};
+  p.q = q; p.k = k; p.v = v; p.state = state;
+  p.rows = rows; p.cu_q = cu_q; p.past_lens = past_lens; p.B = B;
+  p.mask_bits = mask_bits; p.W = W; p.leaf_groups = leaf_groups; p.path = path; p.path_len = path_len;
+  p.out = out;
+  return launch_walk(p, mode, pdl, stream);
 }
 
 // o (T, H, V) fp32 -> out (T, ldo) with head h at h * Vp (columns past V zero): o / rms * w * (silu or sigmoid)(gate (T, ldg)).

@@ -131,12 +131,14 @@ window_post_kernel(const __nv_bfloat16* proj, int ldp, const float* bias, int H,
 
 // ---------------------------------------------------------------- window attention on the plain cores
 // One CTA per (token, head); four warps take every fourth visible key each and merge at the end.  The row sees the last
-// `window` tokens of its own path; the sink is a key of score 0 without a value.
+// `window` tokens of its own path and the positions below `keep`; the sink is a key without a value whose score is sinks[h]
+// (or 0).  With `gate` (T, ldg) the head's output is multiplied by the sigmoid of its logit.
 template <typename E, int NPL>
 __global__ void __launch_bounds__(128)
 window_attn_simt_kernel(const E* q, long long q_tok, const E* kpool, const E* vpool, int Dp, int Vp, const int* slot_map, const int* seq_rows,
                         const int* cu_q, const int* past_lens, const int* mask_bits, E* out, int ldo, int B, int H, int G, int D, int V,
-                        int S, int max_len, int W, int causal, float scale, int window, int sink, int* status) {
+                        int S, int max_len, int W, int causal, float scale, int window, int sink, int keep, const float* sinks,
+                        const float* gate, int ldg, int* status) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y, g = h / (H / G);
@@ -165,17 +167,19 @@ window_attn_simt_kernel(const E* q, long long q_tok, const E* kpool, const E* vp
     acc[e] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  if (sink && warp == 0) { m = 0.f; l = 1.f; }
-  for (int j = (causal ? first : min(first, past)) + warp; j <= last; j += 4) {
+  if (sink && warp == 0) { m = sinks != nullptr ? sinks[h] : 0.f; l = 1.f; }
+  const int first_j = causal ? first : min(first, past), kept = min(keep, first_j);      // two ranges: [0, kept) and [first_j, last]
+  for (int x = warp; x < kept + last - first_j + 1; x += 4) {
+    const int j = x < kept ? x : first_j + x - kept;
     if (j < past) {
-      if (j < first) continue;
+      if (j < first && j >= keep) continue;
     } else if (!causal) {
       const int n = j - past;
       if (!((bits[n >> 5] >> (n & 31)) & 1)) continue;
       int depth = 0;                       // proper ancestors of node n, which are those of this row below n
       for (int w = 0; w < (n >> 5); ++w) depth += __popc(static_cast<unsigned>(bits[w]));
       depth += __popc(static_cast<unsigned>(bits[n >> 5]) & ((1u << (n & 31)) - 1u));
-      if (past + depth < first) continue;
+      if (past + depth < first && past + depth >= keep) continue;
     }
     int slot = slots[j];
     if (slot < 0 || slot >= S) { if (lane == 0) report(status, kBadSlot); slot = 0; }
@@ -211,7 +215,8 @@ window_attn_simt_kernel(const E* q, long long q_tok, const E* kpool, const E* vp
     f[w2] = sm[w2] == -INFINITY ? 0.f : expf(sm[w2] - mm);
     tot += sl[w2] * f[w2];
   }
-  const float inv = tot > 0.f ? 1.f / tot : 0.f;
+  float inv = tot > 0.f ? 1.f / tot : 0.f;
+  if (gate != nullptr) inv /= 1.f + expf(-gate[static_cast<size_t>(t) * ldg + h]);
   for (int c = threadIdx.x; c < V; c += blockDim.x)
     hk_st(out + static_cast<size_t>(t) * ldo + h * V + c, (so[c] * f[0] + so[V + c] * f[1] + so[2 * V + c] * f[2] + so[3 * V + c] * f[3]) * inv);
 }
@@ -220,13 +225,15 @@ template <typename E>
 static int launch_window_simt(const void* q, long long q_tok, const void* kp, const void* vp, int Dp, int Vp, const int* slot_map,
                               const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out, int ldo,
                               int B, int T, int H, int G, int D, int V, int S, int max_len, int W, int causal, float scale, int window,
-                              int sink, int* status, int pdl, cudaStream_t stream) {
+                              int sink, int keep, const float* sinks, const float* gate, int ldg, int* status, int pdl,
+                              cudaStream_t stream) {
   HybridLaunch l(dim3(T, H), dim3(128), stream, pdl, 4 * V * sizeof(float));
   const int n = D > V ? D : V;
   auto kern = n <= 64 ? window_attn_simt_kernel<E, 2> : n <= 128 ? window_attn_simt_kernel<E, 4>
             : n <= 256 ? window_attn_simt_kernel<E, 8> : window_attn_simt_kernel<E, 16>;
   return cudaLaunchKernelEx(&l.c, kern, (const E*)q, q_tok, (const E*)kp, (const E*)vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens,
-                            mask_bits, (E*)out, ldo, B, H, G, D, V, S, max_len, W, causal, scale, window, sink, status) == cudaSuccess ? 0 : -4;
+                            mask_bits, (E*)out, ldo, B, H, G, D, V, S, max_len, W, causal, scale, window, sink, keep, sinks, gate, ldg,
+                            status) == cudaSuccess ? 0 : -4;
 }
 
 // ---------------------------------------------------------------- the residual step behind a sublayer
@@ -464,18 +471,22 @@ extern "C" int js_window_post(const void* proj, int ldp, const float* bias, int 
 }
 
 // q: token t at t * q_tok, head h at h * D; pools (G, S, Dp) and (G, S, Vp); out (T, ldo), head h at h * V.  D, V at most 512.
+// sink: a valueless key of score sinks[h] (null: 0) takes part; keep: positions below it stay visible behind the window;
+// gate (T, ldg) fp32 logits or null.
 extern "C" int js_window_attention_simt(const void* q, long long q_tok, const void* kp, const void* vp, int Dp, int Vp, const int* slot_map,
                                         const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
                                         int ldo, int B, int T, int H, int G, int D, int V, int S, int max_len, int W, int causal,
-                                        float scale, int window, int sink, int bf16, int* status, int pdl, cudaStream_t stream) {
+                                        float scale, int window, int sink, int keep, const float* sinks, const float* gate, int ldg,
+                                        int bf16, int* status, int pdl, cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
-  if (H % G || D > 512 || V > 512 || D > Dp || V > Vp || window < 1) return -10;
+  if (H % G || D > 512 || V > 512 || D > Dp || V > Vp || window < 1 || keep < 0) return -10;
   if (!causal && (mask_bits == nullptr || W < 1)) return -13;
   return bf16 ? launch_window_simt<__nv_bfloat16>(q, q_tok, kp, vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ldo, B, T,
-                                                  H, G, D, V, S, max_len, W, causal, scale, window, sink, status, pdl, stream)
+                                                  H, G, D, V, S, max_len, W, causal, scale, window, sink, keep, sinks, gate, ldg,
+                                                  status, pdl, stream)
               : launch_window_simt<float>(q, q_tok, kp, vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ldo, B, T, H, G,
-                                          D, V, S, max_len, W, causal, scale, window, sink, status, pdl, stream);
+                                          D, V, S, max_len, W, causal, scale, window, sink, keep, sinks, gate, ldg, status, pdl, stream);
 }
 
 // Either ya (with yb, wa, wb for a pair; bias optional) or ys / inv / k and sh, all bf16 rows whose

@@ -237,12 +237,13 @@ __global__ void tap_rows_kernel(const float* x, int ld, __nv_bfloat16* dst, int 
 // ---------------------------------------------------------------- latent attention on the plain cores
 // One CTA per (token, head) row of absorbed queries: scores q . c over the sequence's cached latent rows, softmax, and
 // the weighted sum of the same rows.  Four warps take every fourth key each and merge at the end.  This is the 32-bit
-// path, and the bf16 path of latents wider than the tensor-core kernel's 512.
+// path, and the bf16 path of rows the tensor-core kernel does not take.  sinks (H): a valueless key's score (unscaled) per
+// head; gate (T, ldg): logits whose sigmoid multiplies a head's output; both may be null.
 template <typename E, int NPL>
 __global__ void __launch_bounds__(128)
 latent_attn_simt_kernel(const E* q, const E* pool, const int* slot_map, const int* seq_rows, const int* cu_q, const int* past_lens,
                         const int* mask_bits, E* out, int B, int H, int Rp, int S, int max_len, int W, int causal, float scale,
-                        int* status) {
+                        const float* sinks, const float* gate, int ldg, int* status) {
   const int row = blockIdx.x, t = row / H;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int lo = 0, hi = B - 1;
@@ -261,6 +262,7 @@ latent_attn_simt_kernel(const E* q, const E* pool, const int* slot_map, const in
     acc[e] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
+  if (sinks != nullptr && warp == 0) { m = sinks[row % H]; l = 1.f; }
   for (int j = warp; j < L; j += 4) {
     if (!causal && j >= past) {
       const int n = j - past;
@@ -297,7 +299,8 @@ latent_attn_simt_kernel(const E* q, const E* pool, const int* slot_map, const in
     f[w2] = sm[w2] == -INFINITY ? 0.f : expf(sm[w2] - mm);
     tot += sl[w2] * f[w2];
   }
-  const float inv = tot > 0.f ? 1.f / tot : 0.f;
+  float inv = tot > 0.f ? 1.f / tot : 0.f;
+  if (gate != nullptr) inv /= 1.f + expf(-gate[static_cast<size_t>(t) * ldg + row % H]);
   for (int c = threadIdx.x; c < Rp; c += blockDim.x)
     st_f(out + static_cast<size_t>(row) * Rp + c,
          (so[c] * f[0] + so[Rp + c] * f[1] + so[2 * Rp + c] * f[2] + so[3 * Rp + c] * f[3]) * inv);
@@ -306,12 +309,14 @@ latent_attn_simt_kernel(const E* q, const E* pool, const int* slot_map, const in
 template <typename E>
 static int launch_simt(const void* q, const void* pool, const int* slot_map, const int* seq_rows, const int* cu_q,
                        const int* past_lens, const int* mask_bits, void* out, int B, int T, int H, int Rp, int S, int max_len,
-                       int W, int causal, float scale, int* status, cudaStream_t stream) {
+                       int W, int causal, float scale, const float* sinks, const float* gate, int ldg, int* status,
+                       cudaStream_t stream) {
   const int smem = 4 * Rp * 4;
 #define JS_SIMT(N)                                                                                                        \
   if (Rp <= 32 * N) {                                                                                                     \
     latent_attn_simt_kernel<E, N><<<T * H, 128, smem, stream>>>(static_cast<const E*>(q), static_cast<const E*>(pool),    \
-        slot_map, seq_rows, cu_q, past_lens, mask_bits, static_cast<E*>(out), B, H, Rp, S, max_len, W, causal, scale, status); \
+        slot_map, seq_rows, cu_q, past_lens, mask_bits, static_cast<E*>(out), B, H, Rp, S, max_len, W, causal, scale, \
+        sinks, gate, ldg, status);                                                                                        \
     return cudaGetLastError() == cudaSuccess ? 0 : -4;                                                                    \
   }
   JS_SIMT(2) JS_SIMT(4) JS_SIMT(8) JS_SIMT(16) JS_SIMT(32) JS_SIMT(64)
@@ -394,12 +399,13 @@ extern "C" int js_latent_scatter(const void* c, int ldc, int R, void* pool, int 
 // q, out (T*H, Rp); pool (S, Rp); Rp at most 2048.
 extern "C" int js_latent_attention_simt(const void* q, const void* pool, const int* slot_map, const int* seq_rows, const int* cu_q,
                                         const int* past_lens, const int* mask_bits, void* out, int B, int T, int H, int Rp, int S,
-                                        int max_len, int W, int causal, float scale, int bf16, int* status, cudaStream_t stream) {
+                                        int max_len, int W, int causal, float scale, const float* sinks, const float* gate, int ldg,
+                                        int bf16, int* status, cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
   if (!causal && (mask_bits == nullptr || W < 1)) return -13;
-  return bf16 ? launch_simt<__nv_bfloat16>(q, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, B, T, H, Rp, S, max_len, W, causal, scale, status, stream)
-              : launch_simt<float>(q, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, B, T, H, Rp, S, max_len, W, causal, scale, status, stream);
+  return bf16 ? launch_simt<__nv_bfloat16>(q, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, B, T, H, Rp, S, max_len, W, causal, scale, sinks, gate, ldg, status, stream)
+              : launch_simt<float>(q, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, B, T, H, Rp, S, max_len, W, causal, scale, sinks, gate, ldg, status, stream);
 }
 
 // table (V, ldt) bf16; x fp32, emb (may be null) and h bf16 with leading dimension ld; w, b fp32 (W).

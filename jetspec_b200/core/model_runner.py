@@ -37,19 +37,19 @@ class DenseKVCache:
 
     def _grow(self, cap: int) -> None:
         widths, shapes = self.cfg.latent_widths(), self.cfg.kv_shapes()
-        if shapes is not None:
-            one = lambda i: [torch.zeros(s[0], cap, s[i], dtype=self.dtype, device=self.device) if s is not None else None for s in shapes]
-            nk, nv = one(1), one(2)
-        elif widths is not None:
-            nk, nv = [torch.zeros(1, cap, w, dtype=self.dtype, device=self.device) for w in widths], []
+        if shapes is not None or widths is not None:
+            rows = lambda heads, w: torch.zeros(heads, cap, w, dtype=self.dtype, device=self.device)
+            shapes, widths = shapes or [None] * len(widths), widths or [None] * len(shapes)
+            nk = [rows(s[0], s[1]) if s is not None else rows(1, w) if w is not None else None for s, w in zip(shapes, widths)]
+            nv = [rows(s[0], s[2]) if s is not None else None for s in shapes]
         else:
             L, Hkv, D = self.cfg.num_hidden_layers, self.cfg.num_key_value_heads, self.cfg.head_dim
             nk = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
             nv = [torch.zeros(Hkv, cap, D, dtype=self.dtype, device=self.device) for _ in range(L)]
         nr = []
-        if self.states is not None:     # (un-convolved rows, decay inputs, step-size inputs), each as one head
-            row = lambda w, dt: torch.zeros(1, cap, w, dtype=dt, device=self.device)
-            nr = [(row(c.channels, self.dtype), row(c.decays, torch.float32), row(c.heads, torch.float32)) for c in self.states.shapes]
+        if self.states is not None:     # the inputs of each layer's recurrence, each as one head
+            row = lambda w, f32: torch.zeros(1, cap, w, dtype=torch.float32 if f32 else self.dtype, device=self.device)
+            nr = [tuple(row(*h) for h in c.held) if c is not None else () for c in self.states.shapes]
         for new, old in ((nk, self.k), (nv, self.v), ([x for r in nr for x in r], [x for r in self.rec for x in r])):
             for n, o in zip(new, old):
                 if n is not None:
@@ -76,7 +76,7 @@ class DenseKVCache:
         (reference: ``_select_kv_cache``, ``jetspec/core/llm.py:86-112``).
         """
         n = len(keep_tree_indices)
-        if (n and n <= 64 and self.v and self.states is None and self.k[0].is_cuda and self.k[0].dtype == torch.bfloat16 and self.k[0].shape[-1] == 128
+        if (n and n <= 64 and self.v and self.cfg.kv_shapes() is None and self.cfg.latent_widths() is None and self.k[0].is_cuda and self.k[0].dtype == torch.bfloat16 and self.k[0].shape[-1] == 128
                 and self.k[0].is_contiguous()):
             from ..ops import cuda_ext as X                   # compaction kernel (rows staged in shared memory)
             keep = torch.as_tensor(keep_tree_indices, dtype=torch.int32).to(self.device)
@@ -90,22 +90,20 @@ class DenseKVCache:
                 t[:, past_len:past_len + n] = t[:, idx]
         self.length = past_len + n
 
-    def delta(self, layer: int, mixer, pre, z, b, mask_bits):
-        """Delta rule of ``len(pre)`` new rows behind the cached ones.  The committed rows the state lacks are folded in
+    def recur(self, layer: int, mixer, inputs, mask_bits):
+        """Recurrence of a layer over new rows behind the cached ones.  The committed rows the state lacks are folded in
         first; the new rows are read out from it without being stored, as a tree (``mask_bits``, ``None``: a chain)."""
-        from .. import ops
-        past, T = self.length, pre.shape[0]
+        past, T = self.length, inputs[0].shape[0]
         i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device=self.device)
-        weights, cfg = (mixer.conv(), mixer.A_log, mixer.dt_bias), mixer.cfg
         state, conv = self.states.layer(layer)
         if past > self.folded:
             rows = [x[0, self.folded:past] for x in self.rec[layer]]
-            ops.delta_mix(*rows, *weights, cfg, state, conv, i32(0), i32(0, past - self.folded), i32(self.folded), None, True)
-        for x, new in zip(self.rec[layer], (pre, z, b)):
+            mixer.mix(rows, state, conv, i32(0), i32(0, past - self.folded), i32(self.folded), None, True)
+        for x, new in zip(self.rec[layer], inputs):
             x[0, past:past + T] = new
         if mask_bits is None:                          # on copies: the rows may yet be cropped
-            state, conv = state[:1].clone(), conv[:1].clone()
-        return ops.delta_mix(pre, z, b, *weights, cfg, state, conv, i32(0), i32(0, T), i32(past), mask_bits, mask_bits is None)
+            state, conv = state[:1].clone(), conv[:1].clone() if conv is not None else None
+        return mixer.mix(inputs, state, conv, i32(0), i32(0, T), i32(past), mask_bits, mask_bits is None)
 
 
 class ModelRunner:
@@ -181,14 +179,28 @@ class ModelRunner:
             g = Hq // Hkv
             scale = 1.0 / math.sqrt(D)
 
+        def weights(s, seen, sink):
+            """Softmax over the visible keys; ``sink``: learned numbers per head, or whether a key of score 0 takes part."""
+            s = s.masked_fill(~seen, float("-inf"))
+            if isinstance(sink, torch.Tensor):
+                extra = sink.float().view(s.shape[:-2] + (1, 1)).expand(s.shape[:-1] + (1,))
+            elif sink:
+                extra = torch.zeros_like(s[..., :1])
+            else:
+                return torch.softmax(s, -1)
+            return torch.softmax(torch.cat((s, extra), -1), -1)[..., :-1]
+
         def latent(layer: int, mixer, q, c):
             """Latent attention as the plain formula over the contiguous cache: keys and values are expanded."""
             cache.k[layer][0, past:past + T] = c
-            C, m = cache.k[layer][0, :past + T].float(), mixer.cfg
+            rows, m = cache.k[layer][0, :past + T].float(), mixer.cfg
+            C = rows[:, : m.kv_rank]
             K = (C @ mixer.k_up.weight.float().t()).view(past + T, m.heads, m.dim)
             V = (C @ mixer.v_up.weight.float().t()).view(past + T, m.heads, m.vdim)
-            s = torch.einsum("nhd,lhd->hnl", q.float(), K) * m.scale
-            p = torch.softmax(s.masked_fill(~vis[None], float("-inf")), -1)
+            s = torch.einsum("nhd,lhd->hnl", q[..., : m.dim].float(), K)
+            if m.rot_dim:
+                s = s + torch.einsum("nhd,ld->hnl", q[..., m.dim:].float(), rows[:, m.kv_rank:])
+            p = weights(s * m.scale, vis[None], mixer.sink)
             return torch.einsum("hnl,lhv->nhv", p, V).reshape(T, m.heads * m.vdim).to(q.dtype)
 
         def attn(layer: int, q, k, v):
@@ -224,15 +236,13 @@ class ModelRunner:
             cache.v[layer][:, past:past + T] = v.transpose(0, 1)
             K, V = cache.k[layer][:, :past + T].float(), cache.v[layer][:, :past + T].float()
             s = torch.einsum("nhgd,hld->hgnl", q.float().view(T, m.kv_heads, m.heads // m.kv_heads, m.dim), K) * m.scale
-            seen = vis & (pos[:, None] - key_pos[None, :] < m.window)
-            s = s.masked_fill(~seen[None, None], float("-inf"))
-            if m.sink:
-                s = torch.cat((s, torch.zeros_like(s[..., :1])), -1)
-            p = torch.softmax(s, -1)[..., : past + T]
+            seen = vis & ((pos[:, None] - key_pos[None, :] < m.window) | (key_pos < m.keep_first)[None])
+            p = weights(s, seen[None, None], mixer.sink)
             return torch.einsum("hgnl,hlv->nhgv", p, V).reshape(T, m.heads * m.vdim).to(q.dtype)
 
         attn.latent, attn.window = latent, window
-        attn.delta = lambda layer, mixer, pre, z, b: cache.delta(layer, mixer, pre, z, b, bits)
+        attn.recur = lambda layer, mixer, *inputs: cache.recur(layer, mixer, inputs, bits)
+        attn.delta = attn.recur
         taps = list(target_layer_ids) if (output_hidden_states or target_layer_ids is not None) and target_layer_ids else None
         rows = slice(T - 1, T) if last_position_logits_only else None
         logits, hidden = self.model(ids, pos, attn, tap_layers=taps, logits_rows=rows)

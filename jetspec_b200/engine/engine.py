@@ -215,8 +215,7 @@ class JetSpecEngine:
     def ragged_kernels(self) -> bool:
         """Whether ragged forwards (portions of prompts beside decoded tokens) run on the fused kernel stack; K/V models
         run theirs through the module path's kernels."""
-        fused = self.cfg.latent_widths() is not None or self.cfg.kv_shapes() is not None
-        return self.use_kernels and fused and self.cfg.kernel_path_ok()
+        return self.use_kernels and self.cfg.kernel_stack() is not None and self.cfg.kernel_path_ok()
 
     @torch.inference_mode()
     def step(self, entries):

@@ -1,13 +1,15 @@
-"""Model configurations read from ``config.json``: Qwen3 (Hugging Face layout), Karuzen and Zasipel.
+"""Model configurations read from ``config.json``: Qwen3 (Hugging Face layout), Karuzen, Zasipel and Kizezen.
 
 Only the fields the decoder actually uses are kept.  The draft head adds
 ``block_size``, ``num_target_layers`` and ``dflash_config`` on top of the Qwen3
 fields (reference: ``jetspec/models/draft_head.py:317-337``).
 
 What the engines, the cache and the kernel path ask of a configuration, whatever the family: ``vocab_size``,
-``hidden_size``, ``num_hidden_layers`` (layer RUNS, i.e. cache layers), ``eos_token_id``, ``kernel_path_ok()`` and what a
-cache layer holds: ``latent_widths()`` (``None`` unless every layer caches one latent row a token), ``kv_shapes()``
-(``None`` when all layers hold the same K and V heads) and ``state_shapes()`` (``None`` without recurrent layers).
+``hidden_size``, ``num_hidden_layers`` (layer RUNS, i.e. cache layers), ``eos_token_id``, ``logit_scale``,
+``kernel_path_ok()``, ``kernel_stack()`` (which fused launch sequence runs the decoder, ``None`` for Qwen3's) and what a cache
+layer holds: ``latent_widths()`` (width of a latent row, ``None`` where a layer caches none, or ``None`` for a model without),
+``kv_shapes()`` (likewise; ``None`` when all layers hold the same K and V heads) and ``state_shapes()`` (``None`` without
+recurrent layers).
 """
 from __future__ import annotations
 
@@ -15,6 +17,8 @@ import json
 import os
 from dataclasses import dataclass, field, asdict
 from typing import Any, Optional
+
+from .rotary import BandScaling, RampScaling, RotaryConfig
 
 
 @dataclass
@@ -83,9 +87,15 @@ class Qwen3Config:
         """Per layer the :class:`DeltaConfig` whose state a sequence carries, or ``None``; ``None`` without any."""
         return None
 
+    logit_scale = 1.0
+
     def kernel_path_ok(self) -> bool:
         """Whether the graph-captured kernel path covers this geometry."""
         return self.head_dim == 128
+
+    def kernel_stack(self) -> Optional[str]:
+        """Name of the fused launch sequence of the decoder (see ``engine.fast_round``); ``None``: ``decoder_layers``."""
+        return None
 
     # -- io -------------------------------------------------------------------
     @classmethod
@@ -140,13 +150,26 @@ def _merge_eos(a, b) -> list:
 
 @dataclass
 class LatentAttentionConfig:
-    """Sizes of a latent attention: queries through a latent of ``q_rank``, keys and values from one of ``kv_rank``."""
+    """Sizes of a latent attention: queries through a latent of ``q_rank`` (0: one projection), keys and values from one of
+    ``kv_rank``; with ``rot`` every query head and the cached row carry ``rot.dims`` rotated entries more."""
     heads: int
     dim: int
     vdim: int
     q_rank: int
     kv_rank: int
     scale: float
+    rot: Optional[RotaryConfig] = None
+    sink_logits: bool = False        # a learned number per head in the softmax's denominator
+    gate: bool = False               # sigmoid gate per head on the output
+
+    @property
+    def rot_dim(self) -> int:
+        return self.rot.dims if self.rot is not None else 0
+
+    @property
+    def row(self) -> int:
+        """Entries of a cached row: the latent and the rotated key part all heads share."""
+        return self.kv_rank + self.rot_dim
 
 
 @dataclass
@@ -179,6 +202,7 @@ class KaruzenConfig:
     norm_eps: float = 1e-5
     eos_token_id: Any = None
     model_type: str = "karuzen"
+    logit_scale = 1.0                               # not a field: fixed by the design
 
     def layer_runs(self) -> list:
         """``[(layer index, add the embedding output before it), ...]`` in execution order.  Every run has its own
@@ -210,6 +234,9 @@ class KaruzenConfig:
 
     def kernel_path_ok(self) -> bool:
         return all(l.moe is None or (l.moe.experts <= 1024 and l.moe.top <= 32) for l in self.layers)
+
+    def kernel_stack(self) -> str:
+        return "latent"
 
     # -- io -------------------------------------------------------------------
     @classmethod
@@ -256,7 +283,9 @@ class KaruzenConfig:
                        "router": {"experts": l.moe.experts, "top": l.moe.top, "scale": l.moe.scale}}
                 if l.moe.shared_ff:
                     mlp["shared"] = {"ff": l.moe.shared_ff}
-            layers.append({"type": "latent_attention", "mixer": asdict(l.mixer), "mlp": mlp})
+            m = l.mixer
+            layers.append({"type": "latent_attention", "mlp": mlp, "mixer": {
+                "heads": m.heads, "dim": m.dim, "vdim": m.vdim, "q_rank": m.q_rank, "kv_rank": m.kv_rank, "scale": m.scale}})
         d = {"architecture": "Karuzen", "vocab": self.vocab_size, "width": self.hidden_size, "layers": layers,
              "norm": {"eps": self.norm_eps}}
         if self.loop_stop > self.loop_start:
@@ -275,7 +304,8 @@ class KaruzenConfig:
 @dataclass
 class WindowAttentionConfig:
     """Sizes and constants of a sliding-window attention over grouped K/V heads: a token sees itself and the
-    ``window - 1`` tokens before it; the first ``rot_dims`` dimensions are rotated in neighbouring pairs."""
+    ``window - 1`` tokens before it, and the sequence's first ``keep_first`` tokens; the first ``rot_dims`` dimensions are
+    rotated in neighbouring pairs, or as ``rot`` says."""
     heads: int
     kv_heads: int
     dim: int
@@ -287,6 +317,12 @@ class WindowAttentionConfig:
     sink: bool = True                # a valueless key of score 0 takes part in the softmax
     qk_norm: bool = True             # weightless RMS norm of q and k behind the rotation
     bias: bool = True                # biases on all four projections
+    keep_first: int = 0
+    sink_logits: bool = False        # a learned number per head in the softmax's denominator (instead of ``sink``)
+    proj_norm: bool = False          # weighted RMS norm over the whole q and k projections ahead of the rotation
+    o_bias: Optional[bool] = None    # bias on the output projection; None: as ``bias``
+    gate: bool = False               # sigmoid gate per head on the output
+    rot: Optional[RotaryConfig] = None
 
 
 @dataclass
@@ -302,6 +338,11 @@ class DeltaConfig:
     gate: str = "silu"
     decay_rank: int = 0
     gate_rank: int = 0
+
+    @property
+    def held(self) -> list:
+        """``(width, fp32?)`` of the rows that enter the recurrence (see ``GatedDelta.mix``)."""
+        return [(self.channels, False), (self.decays, True), (self.heads, True)]
 
     @property
     def channels(self) -> int:
@@ -344,6 +385,7 @@ class ZasipelConfig:
     norm_eps: float = 1e-6
     eos_token_id: Any = None
     model_type: str = "zasipel"
+    logit_scale = 1.0                               # not a field: fixed by the design
 
     @property
     def num_hidden_layers(self) -> int:
@@ -366,6 +408,9 @@ class ZasipelConfig:
         return all(l.delta.dim <= 256 and l.delta.vdim <= 256 and l.delta.taps <= 17
                    and (l.window is None or (l.window.dim <= 512 and l.window.vdim <= 512))
                    and (l.moe is None or l.moe.experts <= 1024) for l in self.layers)
+
+    def kernel_stack(self) -> str:
+        return "hybrid"
 
     # -- io -------------------------------------------------------------------
     @classmethod
@@ -443,6 +488,149 @@ class ZasipelConfig:
             json.dump(self.to_dict(), f, indent=1)
 
 
+@dataclass
+class RetentionConfig:
+    """Sizes of a retention: linear attention with one fixed decay per head and rotated queries and keys."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: list
+    rot: RotaryConfig
+    taps = channels = 0              # no short convolution: a sequence carries the state alone
+
+    @property
+    def held(self) -> list:
+        """``(width, fp32?)`` of the rows that enter the recurrence (see ``Retention.mix``)."""
+        return [(self.heads * self.dim, True), (self.heads * self.dim, True), (self.heads * self.vdim, False)]
+
+
+@dataclass
+class KizezenLayerConfig:
+    """``mixer``: a :class:`WindowAttentionConfig`, :class:`LatentAttentionConfig` or :class:`RetentionConfig`."""
+    mixer: Any
+    ff: int = 0                      # width of the feed-forward, 0 without one
+
+    @property
+    def mixer_type(self) -> str:
+        return {WindowAttentionConfig: "attention", LatentAttentionConfig: "latent_attention", RetentionConfig: "retention"}[type(self.mixer)]
+
+
+@dataclass
+class KizezenConfig:
+    """Kizezen: pre-norm blocks whose mixers are window attention, latent attention or retention, in any order; scaled
+    embeddings and logits; untied head."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float = 1e-5
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
+    eos_token_id: Any = None
+    model_type: str = "kizezen"
+    is_moe = False
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    def _per_layer(self, kind, of) -> Optional[list]:
+        out = [of(l.mixer) if isinstance(l.mixer, kind) else None for l in self.layers]
+        return out if any(x is not None for x in out) else None
+
+    def latent_widths(self) -> Optional[list]:
+        return self._per_layer(LatentAttentionConfig, lambda m: m.row)
+
+    def kv_shapes(self) -> list:
+        return self._per_layer(WindowAttentionConfig, lambda m: (m.kv_heads, m.dim, m.vdim)) or [None] * len(self.layers)
+
+    def state_shapes(self) -> Optional[list]:
+        return self._per_layer(RetentionConfig, lambda m: m)
+
+    def kernel_path_ok(self) -> bool:
+        """Sizes the fused kernels take, and a logit scale that keeps the order of the logits."""
+        def ok(m):
+            if isinstance(m, WindowAttentionConfig):
+                return m.dim <= 512 and m.vdim <= 512
+            return m.row <= 2048 if isinstance(m, LatentAttentionConfig) else m.dim <= 256
+        return self.logit_scale > 0 and all(ok(l.mixer) for l in self.layers)
+
+    def kernel_stack(self) -> str:
+        return "prenorm"
+
+    # -- io -------------------------------------------------------------------
+    @classmethod
+    def from_dict(cls, d: dict) -> "KizezenConfig":
+        def band(s):
+            return None if s is None else BandScaling(*(float(s[k]) for k in ("factor", "low", "high", "original")))
+
+        def ramp(s):
+            return None if s is None else RampScaling(*(float(s[k]) for k in ("factor", "original", "fast", "slow")))
+
+        def mixer(i, t, m):
+            r, size = m["rot"], {k: int(m[k]) for k in ("heads", "dim", "vdim")}
+            dims, base = int(r["dims"]), float(r["base"])
+            if t == "attention":
+                if size["heads"] % int(m["kv_heads"]):
+                    raise ValueError(f"layer {i}: {m['heads']} heads do not divide over {m['kv_heads']} key heads")
+                return WindowAttentionConfig(
+                    **size, kv_heads=int(m["kv_heads"]), window=int(m["mask"]["size"]), keep_first=int(m["mask"]["keep_first"]),
+                    rot_dims=dims, rot_base=base, rot=RotaryConfig(dims, base, "half", band(r.get("scaling"))), scale=float(m["scale"]),
+                    sink=False, sink_logits=True, qk_norm=False, proj_norm=True, bias=True, o_bias=False, gate=True)
+            if t == "latent_attention":
+                if dims != int(m["rot_dim"]):
+                    raise ValueError(f"layer {i}: {dims} rotated entries, but rot_dim {m['rot_dim']}")
+                return LatentAttentionConfig(**size, q_rank=0, kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
+                                             rot=RotaryConfig(dims, base, "next", ramp(r.get("scaling"))), sink_logits=True, gate=True)
+            if t == "retention":
+                decay = [float(x) for x in m["decay"]]
+                if len(decay) != size["heads"]:
+                    raise ValueError(f"layer {i}: {len(decay)} decays for {size['heads']} heads")
+                return RetentionConfig(**size, decay=decay, rot=RotaryConfig(dims, base, "half"))
+            raise ValueError(f"layer {i}: unknown mixer type {t!r}")
+
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            f = e.get("mlp")
+            if f is not None and f["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            lc = KizezenLayerConfig(mixer(i, e["type"], e["mixer"]), ff=int(f["ff"]) if f is not None else 0)
+            if lc.mixer_type != "latent_attention" and lc.mixer.rot.dims > lc.mixer.dim:
+                raise ValueError(f"layer {i}: {lc.mixer.rot.dims} rotated entries in heads of {lc.mixer.dim}")
+            layers.append(lc)
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers, norm_eps=float(d["norm"]["eps"]),
+                   embed_scale=float(d["embedding"]["scale"]), logit_scale=float(d["logit_scale"]), eos_token_id=d.get("eos_token_id"))
+
+    @classmethod
+    def from_pretrained(cls, path: str, subfolder: str = "") -> "KizezenConfig":
+        with open(os.path.join(path, subfolder, "config.json") if subfolder else os.path.join(path, "config.json")) as f:
+            return cls.from_dict(json.load(f))
+
+    def to_dict(self) -> dict:
+        layers = []
+        for l in self.layers:
+            m, r = l.mixer, l.mixer.rot
+            mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "rot": {"dims": r.dims, "base": r.base}}
+            if r.scaling is not None:
+                mixer["rot"]["scaling"] = asdict(r.scaling)
+            if isinstance(m, WindowAttentionConfig):
+                mixer.update(kv_heads=m.kv_heads, scale=m.scale, mask={"size": m.window, "keep_first": m.keep_first})
+            elif isinstance(m, LatentAttentionConfig):
+                mixer.update(kv_rank=m.kv_rank, rot_dim=m.rot_dim, scale=m.scale)
+            else:
+                mixer["decay"] = list(m.decay)
+            layers.append({"type": l.mixer_type, "mixer": mixer, "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None})
+        d = {"architecture": "Kizezen", "vocab": self.vocab_size, "width": self.hidden_size, "layers": layers,
+             "norm": {"eps": self.norm_eps}, "embedding": {"scale": self.embed_scale}, "logit_scale": self.logit_scale}
+        if self.eos_token_id is not None:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    def save_pretrained(self, path: str) -> None:
+        os.makedirs(path, exist_ok=True)
+        with open(os.path.join(path, "config.json"), "w") as f:
+            json.dump(self.to_dict(), f, indent=1)
+
+
 # Geometry presets used by the tests and the benchmarks (random-init weights).
 def tiny_config(**over) -> Qwen3Config:
     """2 layers, hidden 256, 4 q / 2 kv heads, head_dim 64, SwiGLU 512, vocab 1024."""
@@ -500,6 +688,22 @@ def zasipel_tiny_config(**over) -> ZasipelConfig:
               layers=[ZasipelLayerConfig(head, win, moe), ZasipelLayerConfig(chan, None, moe), ZasipelLayerConfig(head, win, None)])
     kw.update(over)
     return ZasipelConfig(**kw)
+
+
+def kizezen_tiny_config(**over) -> KizezenConfig:
+    """4 layers (retention, window attention, latent attention, window attention without a feed-forward); width 144."""
+    def win(window, keep, rot):
+        return WindowAttentionConfig(heads=6, kv_heads=2, dim=24, vdim=40, window=window, keep_first=keep, rot_dims=rot.dims, rot_base=rot.base,
+                                     rot=rot, scale=0.25, sink=False, sink_logits=True, qk_norm=False, proj_norm=True, bias=True,
+                                     o_bias=False, gate=True)
+    ret = RetentionConfig(heads=3, dim=20, vdim=28, decay=[0.9, 0.97, 0.995], rot=RotaryConfig(12, 1e4))
+    lat = LatentAttentionConfig(heads=5, dim=24, vdim=20, q_rank=0, kv_rank=56, scale=0.2, sink_logits=True, gate=True,
+                                rot=RotaryConfig(8, 1e4, "next", RampScaling(8.0, 256, 16.0, 2.0)))
+    kw = dict(vocab_size=320, hidden_size=144, norm_eps=1e-5, embed_scale=1.5, logit_scale=0.5, layers=[
+        KizezenLayerConfig(ret, 168), KizezenLayerConfig(win(21, 3, RotaryConfig(16, 1e4, "half", BandScaling(8.0, 1.0, 4.0, 128))), 200),
+        KizezenLayerConfig(lat, 120), KizezenLayerConfig(win(9, 0, RotaryConfig(24, 5e3)))])
+    kw.update(over)
+    return KizezenConfig(**kw)
 
 
 def draft_head_config(target: Qwen3Config, num_layers: int = 1, block_size: int = 16,

@@ -1,10 +1,11 @@
-"""Building blocks that are not Qwen3's: Dynamic Tanh, latent attention, tanh-GELU MLP, sigmoid-routed experts; window
-attention with a sink, gated delta rules, two mixers side by side, table-routed experts.
+"""Building blocks that are not Qwen3's: Dynamic Tanh, latent attention, GELU MLPs, sigmoid-routed experts; window
+attention with sinks, gated delta rules, retention, two mixers side by side, table-routed experts.
 
 Each takes its sizes and constants as arguments, so a design can combine them freely; the Qwen3 twins (RMSNorm, grouped
 query attention, SwiGLU MLP, softmax-routed experts) are in :mod:`jetspec_b200.models.qwen3`.  ``forward`` is the
 unfused form on :mod:`jetspec_b200.ops`, in any dtype and on any device; the fused kernel forms of whole decoders made
-of these blocks are :mod:`jetspec_b200.engine.latent_stack` and :mod:`jetspec_b200.engine.hybrid_stack`.
+of these blocks are :mod:`jetspec_b200.engine.latent_stack`, :mod:`jetspec_b200.engine.hybrid_stack` and
+:mod:`jetspec_b200.engine.prenorm_stack`.
 """
 from __future__ import annotations
 
@@ -12,7 +13,8 @@ import torch
 import torch.nn as nn
 
 from .. import ops
-from .config import DeltaConfig, LatentAttentionConfig, RoutedExpertsConfig, TableExpertsConfig, WindowAttentionConfig
+from .config import (DeltaConfig, LatentAttentionConfig, RetentionConfig, RoutedExpertsConfig, TableExpertsConfig,
+                     WindowAttentionConfig)
 
 
 class DynamicTanh(nn.Module):
@@ -29,27 +31,47 @@ class DynamicTanh(nn.Module):
 
 
 class LatentAttention(nn.Module):
-    """Attention whose queries and keys/values pass through RMS-normed latents; only the K/V latent is cached.
+    """Attention whose keys and values (and, with a ``q_rank``, queries) pass through RMS-normed latents; only the K/V latent
+    is cached, with the rotated key part all heads share where the design has one.
 
-    ``forward(h, attend)``: ``attend(q, c)`` stores the new latent rows ``c (T, kv_rank)`` and returns the attention of
-    ``q (T, heads, dim)`` over the cached latents, ``(T, heads * vdim)``."""
+    ``forward(h, attend, positions)``: ``attend(q, c)`` stores the new cache rows ``c (T, kv_rank + rot_dim)`` and returns the
+    attention of ``q (T, heads, dim + rot_dim)`` over the cached rows, ``(T, heads * vdim)``."""
 
     def __init__(self, cfg: LatentAttentionConfig, hidden: int, eps: float):
         super().__init__()
         self.cfg, self.eps = cfg, eps
         lin = lambda i, o: nn.Linear(i, o, bias=False)
-        self.q_down, self.q_up = lin(hidden, cfg.q_rank), lin(cfg.q_rank, cfg.heads * cfg.dim)
-        self.kv_down = lin(hidden, cfg.kv_rank)
+        qd = cfg.heads * (cfg.dim + cfg.rot_dim)
+        if cfg.q_rank:
+            self.q_down, self.q_up = lin(hidden, cfg.q_rank), lin(cfg.q_rank, qd)
+            self.q_norm = nn.Parameter(torch.ones(cfg.q_rank))
+        else:
+            self.q_proj = lin(hidden, qd)
+        self.kv_down = lin(hidden, cfg.row)
         self.k_up, self.v_up = lin(cfg.kv_rank, cfg.heads * cfg.dim), lin(cfg.kv_rank, cfg.heads * cfg.vdim)
         self.o_proj = lin(cfg.heads * cfg.vdim, hidden)
-        self.q_norm, self.kv_norm = nn.Parameter(torch.ones(cfg.q_rank)), nn.Parameter(torch.ones(cfg.kv_rank))
+        self.kv_norm = nn.Parameter(torch.ones(cfg.kv_rank))
+        self.sink = nn.Parameter(torch.zeros(cfg.heads)) if cfg.sink_logits else None
+        if cfg.gate:
+            self.gate_proj = lin(hidden, cfg.heads)
 
-    def forward(self, h, attend):
-        m = self.cfg
-        cq = ops.rmsnorm(ops.linear(h, self.q_down.weight), self.q_norm, self.eps)
-        c = ops.rmsnorm(ops.linear(h, self.kv_down.weight), self.kv_norm, self.eps)
-        q = ops.linear(cq, self.q_up.weight).view(h.shape[0], m.heads, m.dim)
-        return ops.linear(attend(q, c), self.o_proj.weight)
+    def forward(self, h, attend, positions=None):
+        m, T = self.cfg, h.shape[0]
+        if m.q_rank:
+            q = ops.linear(ops.rmsnorm(ops.linear(h, self.q_down.weight), self.q_norm, self.eps), self.q_up.weight)
+        else:
+            q = ops.linear(h, self.q_proj.weight)
+        q, c = q.view(T, m.heads, m.dim + m.rot_dim), ops.linear(h, self.kv_down.weight)
+        if m.rot is None:
+            c = ops.rmsnorm(c, self.kv_norm, self.eps)
+        else:
+            q = torch.cat((q[..., : m.dim], ops.rotate(q[..., m.dim:], positions, m.rot)), -1)
+            shared = ops.rotate(c[:, None, m.kv_rank:], positions, m.rot)[:, 0]
+            c = torch.cat((ops.rmsnorm(c[:, : m.kv_rank].contiguous(), self.kv_norm, self.eps), shared), -1)
+        y = attend(q, c)
+        if m.gate:
+            y = ops.head_gate(y, ops.linear_f32(h, self.gate_proj.weight))
+        return ops.linear(y, self.o_proj.weight)
 
 
 class GeluMLP(nn.Module):
@@ -64,6 +86,18 @@ class GeluMLP(nn.Module):
     def forward(self, h):
         a = ops.gelu_tanh_mul(ops.linear(h, self.gate_proj.weight), ops.linear(h, self.up_proj.weight))
         return ops.linear(a, self.down_proj.weight)
+
+
+class GeluErfMLP(nn.Module):
+    """``down(gelu(up(h)))`` with the exact (erf) gelu."""
+
+    def __init__(self, hidden: int, inter: int):
+        super().__init__()
+        self.up_proj = nn.Linear(hidden, inter, bias=False)
+        self.down_proj = nn.Linear(inter, hidden, bias=False)
+
+    def forward(self, h):
+        return ops.linear(ops.gelu_erf(ops.linear(h, self.up_proj.weight)), self.down_proj.weight)
 
 
 class SigmoidMoE(nn.Module):
@@ -105,8 +139,9 @@ class PlainRMSNorm(nn.Module):
 
 
 class WindowAttention(nn.Module):
-    """Sliding-window attention over grouped K/V heads: rotation of the first dimensions in neighbouring pairs, optional
-    weightless norm of q and k behind it, optional valueless sink of score 0, optional biases.
+    """Sliding-window attention over grouped K/V heads.  Options (see the configuration): rotation in neighbouring or half
+    pairs, norm of q and k per head behind it or over the whole projections ahead of it, kept first tokens, a valueless
+    sink of score 0 or a learned one per head, a sigmoid gate per head, biases.
 
     ``forward(h, positions, attend)``: ``attend(q, k, v)`` stores the new K/V rows and returns the attention,
     ``(T, heads * vdim)``."""
@@ -116,14 +151,33 @@ class WindowAttention(nn.Module):
         self.cfg, self.eps = cfg, eps
         lin = lambda i, o: nn.Linear(i, o, bias=cfg.bias)
         self.q_proj, self.k_proj = lin(hidden, cfg.heads * cfg.dim), lin(hidden, cfg.kv_heads * cfg.dim)
-        self.v_proj, self.o_proj = lin(hidden, cfg.kv_heads * cfg.vdim), lin(cfg.heads * cfg.vdim, hidden)
+        self.v_proj = lin(hidden, cfg.kv_heads * cfg.vdim)
+        self.o_proj = nn.Linear(cfg.heads * cfg.vdim, hidden, bias=cfg.bias if cfg.o_bias is None else cfg.o_bias)
+        if cfg.proj_norm:
+            self.q_norm, self.k_norm = nn.Parameter(torch.ones(cfg.heads * cfg.dim)), nn.Parameter(torch.ones(cfg.kv_heads * cfg.dim))
+        self.sink_logits = nn.Parameter(torch.zeros(cfg.heads)) if cfg.sink_logits else None
+        if cfg.gate:
+            self.gate_proj = nn.Linear(hidden, cfg.heads, bias=False)
+
+    @property
+    def sink(self):
+        """What the attention ops take: learned numbers per head, or whether a sink of score 0 takes part."""
+        return self.sink_logits if self.sink_logits is not None else self.cfg.sink
 
     def forward(self, h, positions, attend):
         c, T = self.cfg, h.shape[0]
         q, k, v = (ops.linear(h, p.weight, p.bias) for p in (self.q_proj, self.k_proj, self.v_proj))
-        q, k = (ops.rotate_norm(x.view(T, n, c.dim), positions, c.rot_dims, c.rot_base, self.eps if c.qk_norm else None)
-                for x, n in ((q, c.heads), (k, c.kv_heads)))
-        return ops.linear(attend(q, k, v.view(T, c.kv_heads, c.vdim)), self.o_proj.weight, self.o_proj.bias)
+        if c.proj_norm:
+            q, k = ops.rmsnorm(q, self.q_norm, self.eps), ops.rmsnorm(k, self.k_norm, self.eps)
+        q, k = q.view(T, c.heads, c.dim), k.view(T, c.kv_heads, c.dim)
+        if c.rot is not None:
+            q, k = ops.rotate(q, positions, c.rot), ops.rotate(k, positions, c.rot)
+        else:
+            q, k = (ops.rotate_norm(x, positions, c.rot_dims, c.rot_base, self.eps if c.qk_norm else None) for x in (q, k))
+        y = attend(q, k, v.view(T, c.kv_heads, c.vdim))
+        if c.gate:
+            y = ops.head_gate(y, ops.linear_f32(h, self.gate_proj.weight))
+        return ops.linear(y, self.o_proj.weight, self.o_proj.bias)
 
 
 class GatedDelta(nn.Module):
@@ -154,6 +208,10 @@ class GatedDelta(nn.Module):
         self.o_norm = nn.Parameter(torch.ones(cfg.vdim))
         self.o_proj = lin(vd, hidden)
 
+    def mix(self, inputs, state, conv, rows, cu_q, past_lens, mask_bits, causal):
+        """The recurrence over ``inputs = (pre, z, b)``; states advance when ``causal``."""
+        return ops.delta_mix(*inputs, self.conv(), self.A_log, self.dt_bias, self.cfg, state, conv, rows, cu_q, past_lens, mask_bits, causal)
+
     def conv(self) -> torch.Tensor:
         """Convolution taps of all channels, ``(channels, taps)``, in the order of ``pre``."""
         return torch.cat((self.q_conv, self.k_conv, self.v_conv), 0)
@@ -168,6 +226,34 @@ class GatedDelta(nn.Module):
         gate = lin(lin(h, self.gate_down.weight), self.gate_up.weight) if c.gate_rank else lin(h, self.gate_proj.weight)
         y = ops.gated_head_norm(recur(pre, z, b), self.o_norm, gate, c.gate, self.eps)
         return lin(y, self.o_proj.weight)
+
+
+class Retention(nn.Module):
+    """Linear attention with one fixed decay per head: rotated queries and keys, per-head norm of the read-outs without a
+    weight, silu gate over all columns.
+
+    ``forward(h, positions, recur)``: ``recur(q, k, v)`` advances the sequences' states by the rotated fp32 rows and returns
+    the read-outs, fp32 ``(T, heads, vdim)``."""
+
+    def __init__(self, cfg: RetentionConfig, hidden: int, eps: float):
+        super().__init__()
+        self.cfg, self.eps = cfg, eps
+        lin = lambda i, o: nn.Linear(i, o, bias=False)
+        self.q_proj, self.k_proj = lin(hidden, cfg.heads * cfg.dim), lin(hidden, cfg.heads * cfg.dim)
+        self.v_proj, self.gate_proj = lin(hidden, cfg.heads * cfg.vdim), lin(hidden, cfg.heads * cfg.vdim)
+        self.o_proj = lin(cfg.heads * cfg.vdim, hidden)
+
+    def mix(self, inputs, state, conv, rows, cu_q, past_lens, mask_bits, causal):
+        """The recurrence over ``inputs = (q, k, v)``; states advance when ``causal``."""
+        return ops.retention(*inputs, self.cfg, state, rows, cu_q, past_lens, mask_bits, causal)
+
+    def forward(self, h, positions, recur):
+        c, T = self.cfg, h.shape[0]
+        q, k = (ops.rotate(ops.linear(h, p.weight).view(T, c.heads, c.dim), positions, c.rot, torch.float32)
+                for p in (self.q_proj, self.k_proj))
+        o = recur(q.flatten(1), k.flatten(1) * c.dim ** -0.5, ops.linear(h, self.v_proj.weight))
+        y = ops.gated_head_norm(o, None, ops.linear(h, self.gate_proj.weight), "silu", self.eps)
+        return ops.linear(y, self.o_proj.weight)
 
 
 class SideBySide(nn.Module):

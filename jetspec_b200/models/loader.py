@@ -45,7 +45,9 @@ def tensor_shape(path: str, name: str) -> tuple:
 
 @torch.no_grad()
 def load_state_into(module: torch.nn.Module, path: str, remap: Optional[Callable] = None,
-                    strict: bool = True, prefix_strip: str = "") -> None:
+                    strict: bool = True, prefix_strip: str = "", optional: tuple = ("lm_head.weight",)) -> None:
+    """Copy the checkpoint under ``path`` into ``module``.  ``optional`` parameters may be absent from the file (by default a
+    head that is tied to the embedding)."""
     from safetensors import safe_open
     params = dict(module.named_parameters())
     params.update(dict(module.named_buffers()))
@@ -82,8 +84,7 @@ def load_state_into(module: torch.nn.Module, path: str, remap: Optional[Callable
                 raise KeyError(f"stacked parameter {name!r} is missing {len(want - got)} of {len(want)} slices "
                                f"(first: {lost})")
         missing = [n for n in module.state_dict() if n not in seen]
-        # a tied lm_head is legitimately absent from the file
-        missing = [n for n in missing if n != "lm_head.weight"]
+        missing = [n for n in missing if n not in optional]
         if missing:
             raise KeyError(f"parameters missing from checkpoint: {missing[:8]}{'…' if len(missing) > 8 else ''}")
 

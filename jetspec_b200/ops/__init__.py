@@ -92,11 +92,11 @@ def latent_scatter(c, pool, slots):
     return ref.latent_scatter(c, pool, slots)
 
 
-def latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal: bool = False):
-    if _kern_any(q):
+def latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal: bool = False, sink=None):
+    if _kern_any(q) and pool.shape[1] <= 2048:
         return _ext().latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits,
-                                       float(scale), bool(causal))
-    return ref.latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal)
+                                       float(scale), bool(causal), sink)
+    return ref.latent_attention(q, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal, sink)
 
 
 def sigmoid_moe(x, router_w, correction, w_up, w_down, top, scale):
@@ -131,12 +131,36 @@ def window_scatter(k, v, k_pool, v_pool, slots):
 
 
 def window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, window, sink,
-                     causal: bool = False):
+                     causal: bool = False, keep_first: int = 0):
     if _kern_any(q) and max(q.shape[-1], vdim) <= 512:
         return _ext().window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, float(scale),
-                                       int(window), bool(sink), bool(causal))
+                                       int(window), sink, bool(causal), keep_first=int(keep_first))
     return ref.window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, window, sink,
-                                causal)
+                                causal, keep_first)
+
+
+def gelu_erf(x):
+    if _kern_any(x):
+        return _ext().gelu_erf(x)
+    return ref.gelu_erf(x)
+
+
+def rotate(x, positions, rot, out_dtype=None):
+    if _kern_any(x) and x.shape[-1] <= 1024 and (out_dtype or x.dtype) in (torch.bfloat16, torch.float32):
+        return _ext().rotate(x, positions, rot, out_dtype or x.dtype)
+    return ref.rotate(x, positions, rot, out_dtype)
+
+
+def head_gate(y, logits):
+    if _kern_any(y):
+        return _ext().head_gate(y, logits)
+    return ref.head_gate(y, logits)
+
+
+def retention(q, k, v, cfg, state, rows, cu_q, past_lens, mask_bits, causal: bool = True):
+    if _kern_any(q) and cfg.dim <= 256 and (causal or mask_bits.shape[1] <= 8):
+        return _ext().retention(q, k, v, cfg, state, rows, cu_q, past_lens, mask_bits, bool(causal))
+    return ref.retention(q, k, v, cfg, state, rows, cu_q, past_lens, mask_bits, causal)
 
 
 def delta_mix(pre, z, b, taps, A_log, dt_bias, cfg, state, conv, rows, cu_q, past_lens, mask_bits, causal: bool = True):
@@ -211,6 +235,6 @@ __all__ = [
     "paged_tree_attention", "lm_head_argmax", "lm_head_topk_logprobs", "moe_forward",
     "dynamic_tanh", "gelu_tanh_mul", "relu_squared", "latent_scatter", "latent_attention", "sigmoid_moe",
     "rmsnorm_f32", "linear_f32", "rotate_norm", "window_scatter", "window_attention", "delta_mix", "gated_head_norm",
-    "experts_swiglu",
+    "experts_swiglu", "gelu_erf", "rotate", "head_gate", "retention",
     "pack_ancestor_bits", "unpack_ancestor_bits", "rope_cos_sin", "apply_rope", "moe_route", "sample",
 ]

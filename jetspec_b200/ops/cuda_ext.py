@@ -206,7 +206,7 @@ def inv_freq(head_dim: int, theta: float, device) -> torch.Tensor:
 # ------------------------------------------------------------------ GEMM
 EPI_STORE, EPI_SWIGLU, EPI_ARGMAX, EPI_TOPK, EPI_STORE_F32 = 0, 1, 2, 3, 4
 EPI_RELU2 = 8
-ACT_GELU_GLU, ACT_RELU2, ACT_NONE = 0, 1, 2
+ACT_GELU_GLU, ACT_RELU2, ACT_NONE, ACT_GELU_ERF = 0, 1, 2, 3
 SM_COUNT = 148
 _DEEP = os.environ.get("JETSPEC_GEMM_DEEP", "0") == "1"
 _SPLIT_DEEP = os.environ.get("JETSPEC_SPLIT_DEEP")      # force the split-K pipeline: 1 = 192 KB, 2 = 128 KB, 0 = 96 KB
@@ -616,10 +616,23 @@ def paged_tree_attention(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens,
     return out
 
 
+def _head_gate(gate: Optional[torch.Tensor]) -> tuple:
+    """Pointer and leading dimension of the fp32 gate logits ``(T, >= heads)`` of an attention kernel."""
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1)
+    return _p(gate), gate.stride(0) if gate is not None else 0
+
+
+def _sinks(sinks: Optional[torch.Tensor], heads: int):
+    """Pointer to the fp32 sink scores of an attention kernel's heads."""
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == heads)
+    return _p(sinks)
+
+
 def paged_attention_rows(q, k_rows, v_rows, slot_map, seq_rows, cu_q, past_lens, scale: float, max_q: int, out, max_keys: int,
-                         pdl: bool = False) -> torch.Tensor:
+                         pdl: bool = False, sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention over keys and values stored row-major, ``k_rows, v_rows (keys, Hkv*128)`` (views of one wider
-    matrix are fine), on the tcgen05 kernel; ``out (T, >= Hq*128)`` may be a column block of a wider matrix."""
+    matrix are fine), on the tcgen05 kernel; ``out (T, >= Hq*128)`` may be a column block of a wider matrix.  ``sinks (Hq,)``:
+    score of a valueless key per head; ``gate (T, >= Hq)``: logits whose sigmoid multiplies a head's output."""
     lib = load()
     T, Hq, D = q.shape
     Hkv = k_rows.shape[1] // 128
@@ -632,8 +645,8 @@ def paged_attention_rows(q, k_rows, v_rows, slot_map, seq_rows, cu_q, past_lens,
     _check(lib.js_paged_attention_tc_strided(
         _p(q), _p(k_rows), _p(v_rows), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), None, _p(out), _p(ws_o), _p(ws_ml),
         _p(status_word(q.device)), seq_rows.numel(), T, Hq, Hkv, k_rows.shape[0], slot_map.shape[1], 0, 1, splits,
-        ctypes.c_float(scale), ctypes.c_longlong(128), ctypes.c_longlong(k_rows.stride(0)), out.stride(0), int(pdl), _stream()),
-        "js_paged_attention_tc_strided")
+        ctypes.c_float(scale), _sinks(sinks, Hq), *_head_gate(gate), ctypes.c_longlong(128), ctypes.c_longlong(k_rows.stride(0)),
+        out.stride(0), int(pdl), _stream()), "js_paged_attention_tc_strided")
     return out
 
 
@@ -752,23 +765,33 @@ def latent_scatter(c: torch.Tensor, pool: torch.Tensor, slots: torch.Tensor) -> 
                                  _is_bf16(c), _p(status_word(c.device)), _stream()), "js_latent_scatter")
 
 
-LATENT_TC_MAX = 512        # widest latent row of the tensor-core kernel
+LATENT_TC_MAX = 512        # most value columns of the tensor-core kernel
+LATENT_TC_ROW = 768        # widest cached row of the tensor-core kernel
 
 
-def latent_attn_splits(T: int, heads: int, seqs: int, max_q: int, Rp: int, max_keys: int) -> int:
-    """Key splits of the tensor-core latent attention: one wave of CTAs (128 query rows of one sequence each, two column
-    groups for latents wider than 256), at least a couple of key tiles each."""
-    tiles = min(T * heads // 128 + seqs, seqs * ((max_q * heads + 127) // 128))
-    ctas = max(1, tiles * (2 if Rp > 256 else 1))
+def latent_tc_ok(Rp: int, out_cols: Optional[int] = None) -> bool:
+    """Whether the tensor-core kernel takes rows of ``Rp`` columns whose first ``out_cols`` are values."""
+    return Rp <= LATENT_TC_ROW and (Rp if out_cols is None else out_cols) <= LATENT_TC_MAX
+
+
+def latent_attn_splits(T: int, heads: int, seqs: int, max_q: int, Rp: int, max_keys: int, out_cols: Optional[int] = None) -> int:
+    """Key splits of the tensor-core latent attention: one wave of CTAs (128 query rows of one sequence each, 64 for rows
+    wider than 512; two column groups for more than 256 value columns), at least a couple of key tiles each."""
+    per = 64 if Rp > 512 else 128
+    tiles = min(T * heads // per + seqs, seqs * ((max_q * heads + per - 1) // per))
+    ctas = max(1, tiles * (2 if (Rp if out_cols is None else out_cols) > 256 else 1))
     return max(1, min(SM_COUNT // ctas, (max_keys + 127) // 128, 16))
 
 
 def latent_attention_rows(qa: torch.Tensor, pool: torch.Tensor, heads: int, slot_map, seq_rows, cu_q, past_lens, mask_bits,
                           scale: float, causal: bool, max_q: int, out: Optional[torch.Tensor] = None,
                           splits: Optional[int] = None, ws: Optional[dict] = None, max_keys: Optional[int] = None,
-                          pdl: bool = False, impl: Optional[str] = None, tile: int = 0) -> torch.Tensor:
+                          pdl: bool = False, impl: Optional[str] = None, tile: int = 0, out_cols: Optional[int] = None,
+                          sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention of absorbed query rows ``qa (T*heads, Rp)`` over the latent rows of ``pool (S, Rp)``; ``out`` has the
-    shape of ``qa``.  ``impl``: ``"tc"`` (bf16, Rp up to 512, masks up to 256 nodes) or ``"simt"``."""
+    shape of ``qa``, of which the first ``out_cols`` columns are wanted.  ``impl``: ``"tc"`` (bf16, see :func:`latent_tc_ok`,
+    masks up to 256 nodes) or ``"simt"``.  ``sinks (heads,)``: score of a valueless key per head; ``gate (T, >= heads)``: logits
+    whose sigmoid multiplies a head's output."""
     lib = load()
     rows, Rp = qa.shape
     T, B = rows // heads, seq_rows.numel()
@@ -777,36 +800,41 @@ def latent_attention_rows(qa: torch.Tensor, pool: torch.Tensor, heads: int, slot
         out = torch.empty_like(qa)
     W = mask_bits.shape[1] if mask_bits is not None else 0
     if impl is None:
-        impl = "tc" if qa.dtype == torch.bfloat16 and Rp <= LATENT_TC_MAX and W <= 8 else "simt"
+        impl = "tc" if qa.dtype == torch.bfloat16 and latent_tc_ok(Rp, out_cols) and W <= 8 else "simt"
     st = _p(status_word(qa.device))
     if impl == "simt":
         _check(lib.js_latent_attention_simt(_p(qa), _p(pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens),
                                             _p(mask_bits), _p(out), B, T, heads, Rp, pool.shape[0], slot_map.shape[1], W,
-                                            int(causal), ctypes.c_float(scale), _is_bf16(qa), st, _stream()),
+                                            int(causal), ctypes.c_float(scale), _sinks(sinks, heads), *_head_gate(gate),
+                                            _is_bf16(qa), st, _stream()),
                "js_latent_attention_simt")
         return out
     if splits is None:
-        splits = latent_attn_splits(T, heads, B, max_q, Rp, max_keys if max_keys is not None else slot_map.shape[1])
+        splits = latent_attn_splits(T, heads, B, max_q, Rp, max_keys if max_keys is not None else slot_map.shape[1], out_cols)
     if splits > 1 and ws is None:
         ws = {"o": torch.empty(splits, rows, Rp, dtype=torch.float32, device=qa.device),
               "ml": torch.empty(splits, rows, 2, dtype=torch.float32, device=qa.device)}
     _check(lib.js_latent_attention_tc(_p(qa), _p(pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), _p(mask_bits),
                                       _p(out), _p(ws["o"] if splits > 1 else None), _p(ws["ml"] if splits > 1 else None), st,
-                                      B, T, heads, Rp, pool.shape[0], slot_map.shape[1], W, int(causal), int(splits),
-                                      int(max_q), ctypes.c_float(scale), int(tile), int(pdl), _stream()), "js_latent_attention_tc")
+                                      B, T, heads, Rp, Rp if out_cols is None else int(out_cols), pool.shape[0], slot_map.shape[1], W,
+                                      int(causal), int(splits), int(max_q), ctypes.c_float(scale), _sinks(sinks, heads), *_head_gate(gate),
+                                      int(tile), int(pdl), _stream()), "js_latent_attention_tc")
     return out
 
 
 def latent_attention(q: torch.Tensor, w_uk, w_uv, pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float,
-                     causal: bool) -> torch.Tensor:
+                     causal: bool, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Unfused form (see :func:`jetspec_b200.ops.reference.latent_attention`): the key expansion is moved onto the
     query, the value expansion behind the attention, with library products around the attention kernel."""
-    T, H, D = q.shape
-    R, Rp = w_uk.shape[1], pool.shape[1]
-    V = w_uv.shape[0] // H
+    T, H, _ = q.shape
+    R, D, Rp = w_uk.shape[1], w_uk.shape[0] // H, pool.shape[1]
+    V, E = w_uv.shape[0] // H, q.shape[2] - D
     qa = torch.zeros(T, H, Rp, dtype=q.dtype, device=q.device)
-    qa[:, :, :R] = torch.bmm(q.transpose(0, 1), w_uk.view(H, D, R)).transpose(0, 1)
-    o = latent_attention_rows(qa.view(T * H, Rp), pool, H, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal, T)
+    qa[:, :, :R] = torch.bmm(q[..., :D].transpose(0, 1), w_uk.view(H, D, R)).transpose(0, 1)
+    qa[:, :, R:R + E] = q[..., D:]
+    sinks = sink.detach().float().contiguous() if sink is not None else None
+    o = latent_attention_rows(qa.view(T * H, Rp), pool, H, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, causal, T, sinks=sinks,
+                              out_cols=R)
     o = o.view(T, H, Rp)[:, :, :R].transpose(0, 1)
     return torch.bmm(o, w_uv.view(H, V, R).transpose(1, 2)).transpose(0, 1).reshape(T, H * V)
 
@@ -922,8 +950,11 @@ def rotate_norm(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float
 
 
 def window_attention(q, k_pool, v_pool, vdim: int, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int,
-                     sink: bool, causal: bool, out: Optional[torch.Tensor] = None, pdl: bool = False) -> torch.Tensor:
-    """Window attention on the plain cores (bf16 or fp32, heads of up to 512); see the reference op for the contract."""
+                     sink, causal: bool, out: Optional[torch.Tensor] = None, pdl: bool = False, keep_first: int = 0,
+                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Window attention on the plain cores (bf16 or fp32, heads of up to 512); see the reference op for the contract.  ``gate``:
+    logits whose sigmoid multiplies a head's output."""
+    sinks = sink.detach().float().contiguous() if isinstance(sink, torch.Tensor) else None
     lib = load()
     T, H, D = q.shape
     assert q.stride(2) == 1 and q.stride(1) == D
@@ -933,29 +964,34 @@ def window_attention(q, k_pool, v_pool, vdim: int, slot_map, seq_rows, cu_q, pas
     _check(lib.js_window_attention_simt(
         _p(q), ctypes.c_longlong(q.stride(0)), _p(k_pool), _p(v_pool), Dp, v_pool.shape[2], _p(slot_map), _p(seq_rows), _p(cu_q),
         _p(past_lens), _p(mask_bits), _p(out), out.stride(0), seq_rows.numel(), T, H, G, D, vdim, S, slot_map.shape[1],
-        mask_bits.shape[1] if mask_bits is not None else 0, int(causal), ctypes.c_float(scale), int(window), int(sink), _is_bf16(q),
-        _p(status_word(q.device)), int(pdl), _stream()), "js_window_attention_simt")
+        mask_bits.shape[1] if mask_bits is not None else 0, int(causal), ctypes.c_float(scale), int(window),
+        int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, H), *_head_gate(gate), _is_bf16(q), _p(status_word(q.device)),
+        int(pdl), _stream()), "js_window_attention_simt")
     return out
 
 
-def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int) -> int:
-    """Key splits of the tensor-core kernel: a CTA's rows span at most the window and their own tokens."""
-    return attn_splits_for(T, Hq, Hkv, min(max_keys, window + 128 // (Hq // Hkv)))
+def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int, keep_first: int = 0) -> int:
+    """Key splits of the tensor-core kernel: a CTA's rows span at most the window, their own tokens and the kept first ones."""
+    return attn_splits_for(T, Hq, Hkv, min(max_keys, window + 128 // (Hq // Hkv) + keep_first))
 
 
-def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int, sink: bool,
-                        causal: bool, out: torch.Tensor, splits: int = 1, ws: Optional[dict] = None, pdl: bool = False) -> torch.Tensor:
-    """Window attention on the tcgen05 kernel: bf16, heads padded to 128, groups of 1, 2, 4, 8 or 16 query heads."""
+def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int, sink,
+                        causal: bool, out: torch.Tensor, splits: int = 1, ws: Optional[dict] = None, pdl: bool = False,
+                        keep_first: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Window attention on the tcgen05 kernel: bf16, heads padded to 128, groups of 1, 2, 4, 8 or 16 query heads.  ``sink``:
+    whether a valueless key of score 0 takes part, or its score per head, fp32 ``(Hq,)``; ``gate (T, >= Hq)``: logits whose
+    sigmoid multiplies a head's output."""
     lib = load()
     T, Hq, D = q.shape
+    sinks = sink if isinstance(sink, torch.Tensor) else None
     G, S, _ = k_pool.shape
     assert D == 128 and q.is_contiguous() and k_pool.shape[2] == 128 and v_pool.shape[2] == 128
     _check(lib.js_window_attention_tc(
         _p(q), _p(k_pool), _p(v_pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), _p(mask_bits), _p(out),
         _p(ws["o"] if splits > 1 else None), _p(ws["ml"] if splits > 1 else None), _p(status_word(q.device)), seq_rows.numel(), T, Hq,
         G, S, slot_map.shape[1], mask_bits.shape[1] if mask_bits is not None else 0, int(causal), int(splits), ctypes.c_float(scale),
-        int(window), int(sink), ctypes.c_longlong(S * 128), ctypes.c_longlong(128), out.stride(0), int(pdl), _stream()),
-        "js_window_attention_tc")
+        int(window), int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, Hq), *_head_gate(gate),
+        ctypes.c_longlong(S * 128), ctypes.c_longlong(128), out.stride(0), int(pdl), _stream()), "js_window_attention_tc")
     return out
 
 
@@ -1076,10 +1112,86 @@ def gated_head_norm(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, kind: 
     vp = vp or V
     if out is None:
         out = torch.empty(T, H * vp, dtype=gate.dtype, device=gate.device)
-    assert w.dtype == gate.dtype == out.dtype and gate.stride(1) == 1
+    assert (w is None or w.dtype == gate.dtype) and gate.dtype == out.dtype and gate.stride(1) == 1
     _check(lib.js_gated_head_norm(_p(o), _p(w), _p(gate), gate.stride(0), _p(out), out.stride(0), T, H, V, vp, int(kind == "silu"),
                                   ctypes.c_float(eps), _is_bf16(gate), int(pdl), _stream()), "js_gated_head_norm")
     return out
+
+
+# ------------------------------------------------------------------ pre-norm steps, general rotations, retention
+_rot_freq: dict = {}
+
+
+def rot_freq(rot, device) -> torch.Tensor:
+    """fp32 frequencies of a ``RotaryConfig`` on the device."""
+    key = (rot, str(device))
+    if key not in _rot_freq:
+        _rot_freq[key] = torch.tensor(rot.frequencies(), dtype=torch.float32, device=device)
+    return _rot_freq[key]
+
+
+def gelu_erf(x: torch.Tensor) -> torch.Tensor:
+    lib = load()
+    x = x.contiguous()
+    out = torch.empty_like(x)
+    _check(lib.js_gelu_erf(_p(x), _p(out), ctypes.c_longlong(x.numel()), _is_bf16(x), _stream()), "js_gelu_erf")
+    return out
+
+
+def rotate(x: torch.Tensor, positions: torch.Tensor, rot, out_dtype) -> torch.Tensor:
+    lib = load()
+    T, heads, D = x.shape
+    x = x.contiguous()
+    out = torch.empty(T, heads, D, dtype=out_dtype, device=x.device)
+    pos, freq = positions.to(torch.int32), rot_freq(rot, x.device)      # named: they outlive the launch
+    _check(lib.js_rotate(_p(x), _is_bf16(x), _p(out), _is_bf16(out), _p(pos), T, heads, D, rot.dims, int(rot.pairing == "next"), _p(freq),
+                         ctypes.c_float(rot.amplitude()), _stream()), "js_rotate")
+    return out
+
+
+def head_gate(y: torch.Tensor, logits: torch.Tensor) -> torch.Tensor:
+    lib = load()
+    T, H = logits.shape
+    y, logits = y.contiguous(), logits.float()
+    assert logits.stride(1) == 1 and y.shape[0] == T and y.shape[1] % H == 0
+    out = torch.empty_like(y)
+    _check(lib.js_head_gate(_p(y), _p(logits), logits.stride(0), _p(out), T, H, y.shape[1] // H, _is_bf16(y), _stream()), "js_head_gate")
+    return out
+
+
+_decays: dict = {}
+
+
+def retention_decays(cfg, device) -> torch.Tensor:
+    """The heads' decays, fp32 on the device."""
+    key = (tuple(cfg.decay), str(device))
+    if key not in _decays:
+        _decays[key] = torch.tensor(cfg.decay, dtype=torch.float32, device=device)
+    return _decays[key]
+
+
+def retention_seq(q, k, v, cfg, state, rows, cu_q, past_lens, mask_bits=None, path=None, path_len=None, out=None, pdl: bool = False):
+    """Retention row by row over fp32 rows ``q, k (T, H*D)``, ``v (T, H*V)``: causal (states advance), over token trees
+    (``mask_bits``: nothing is stored), or along the rows ``path[:path_len]`` of one sequence (nothing is read out)."""
+    lib = load()
+    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (k, v, state))
+    assert k.shape[1] == cfg.heads * cfg.dim and v.shape[1] == cfg.heads * cfg.vdim and state.shape[1:] == (cfg.heads, cfg.dim, cfg.vdim)
+    mode = 1 if mask_bits is not None else 2 if path is not None else 0
+    assert mode == 2 or (q.dtype == torch.float32 and q.is_contiguous() and q.shape == k.shape)
+    B, W = rows.numel(), mask_bits.shape[1] if mask_bits is not None else 0
+    groups = max(1, min(32 * W // 4, 4 * SM_COUNT // max(1, B * cfg.heads * ((cfg.vdim + 31) // 32)))) if W else 1
+    if out is None and mode != 2:
+        out = torch.empty(k.shape[0], cfg.heads, cfg.vdim, dtype=torch.float32, device=k.device)
+    _check(lib.js_retention_seq(mode, cfg.heads, cfg.dim, cfg.vdim, _p(q), _p(k), _p(v), _p(retention_decays(cfg, k.device)), _p(state), _p(rows),
+                                _p(cu_q), _p(past_lens), B, _p(mask_bits), W, groups, _p(path), _p(path_len), _p(out), int(pdl), _stream()),
+           "js_retention_seq")
+    return out
+
+
+def retention(q, k, v, cfg, state, rows, cu_q, past_lens, mask_bits, causal: bool) -> torch.Tensor:
+    """Unfused form; see the reference op for the contract."""
+    q, k, v = (x.float().contiguous() for x in (q, k, v))
+    return retention_seq(q, k, v, cfg, state, rows, cu_q, past_lens, None if causal else mask_bits)
 
 
 # ------------------------------------------------------------------ MoE (grouped through the dense GEMM)

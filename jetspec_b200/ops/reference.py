@@ -173,15 +173,18 @@ def paged_tree_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Te
 
 def latent_attention(q: torch.Tensor, w_uk: torch.Tensor, w_uv: torch.Tensor, pool: torch.Tensor,
                      slot_map: torch.Tensor, seq_rows: torch.Tensor, cu_q: torch.Tensor, past_lens: torch.Tensor,
-                     mask_bits: Optional[torch.Tensor], scale: float, causal: bool = False) -> torch.Tensor:
+                     mask_bits: Optional[torch.Tensor], scale: float, causal: bool = False,
+                     sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Attention over slot-addressed latent rows, keys and values expanded from them.
 
-    ``q (T, H, D)``; ``pool (S, >= R)`` holds one latent row per slot; ``w_uk (H*D, R)`` and ``w_uv (H*V, R)`` give
-    head ``h`` of a cached row ``c`` the key ``w_uk[h] c`` and the value ``w_uv[h] c``.  Sequences, visibility and
-    masks as in :func:`paged_tree_attention`; softmax in fp32.  Returns ``(T, H*V)`` in ``q.dtype``.
+    ``q (T, H, D + E)``; ``pool (S, >= R + E)`` holds one row ``c | e`` per slot; ``w_uk (H*D, R)`` and ``w_uv (H*V, R)`` give
+    head ``h`` of a cached row the key ``w_uk[h] c | e`` and the value ``w_uv[h] c`` (``E`` may be 0).  Sequences, visibility
+    and masks as in :func:`paged_tree_attention`; softmax in fp32, with ``sink (H,)`` its denominator also holds
+    ``exp(sink)``.  Returns ``(T, H*V)`` in ``q.dtype``.
     """
-    T, H, D = q.shape
-    R, V = w_uk.shape[1], w_uv.shape[0] // H
+    T, H, _ = q.shape
+    R, D, V = w_uk.shape[1], w_uk.shape[0] // H, w_uv.shape[0] // H
+    E = q.shape[2] - D
     wk, wv = w_uk.float().view(H, D, R), w_uv.float().view(H, V, R)
     out = torch.empty(T, H * V, dtype=q.dtype, device=q.device)
     cu, pl, rows = cu_q.tolist(), past_lens.tolist(), seq_rows.tolist()
@@ -191,13 +194,19 @@ def latent_attention(q: torch.Tensor, w_uk: torch.Tensor, w_uv: torch.Tensor, po
         if n == 0:
             continue
         L = pl[b] + n
-        c = pool[slot_map[rows[b], :L].long(), :R].float()
+        row = pool[slot_map[rows[b], :L].long()].float()
+        c, e_part = row[:, :R], row[:, R:R + E]
         k, v = torch.einsum("lr,hdr->hld", c, wk), torch.einsum("lr,hvr->hlv", c, wv)
         vis = torch.ones(n, L, dtype=torch.bool, device=q.device)
         vis[:, pl[b]:] = (torch.tril(torch.ones(n, n, dtype=torch.bool, device=q.device)) if causal
                           else unpack_ancestor_bits(mask_bits[s:e], n))
-        sc = torch.einsum("nhd,hld->hnl", q[s:e].float(), k) * scale
-        p = torch.nan_to_num(torch.softmax(sc.masked_fill(~vis[None], float("-inf")), dim=-1), nan=0.0)
+        sc = torch.einsum("nhd,hld->hnl", q[s:e, :, :D].float(), k)
+        if E:
+            sc = sc + torch.einsum("nhd,ld->hnl", q[s:e, :, D:].float(), e_part)
+        sc = (sc * scale).masked_fill(~vis[None], float("-inf"))
+        if sink is not None:
+            sc = torch.cat((sc, sink.float().view(H, 1, 1).expand(H, n, 1)), -1)
+        p = torch.nan_to_num(torch.softmax(sc, dim=-1), nan=0.0)[..., :L]
         out[s:e] = torch.einsum("hnl,hlv->nhv", p, v).reshape(n, H * V).to(q.dtype)
     return out
 
@@ -360,10 +369,11 @@ def window_scatter(k: torch.Tensor, v: torch.Tensor, k_pool: torch.Tensor, v_poo
 
 def window_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, vdim: int, slot_map: torch.Tensor,
                      seq_rows: torch.Tensor, cu_q: torch.Tensor, past_lens: torch.Tensor, mask_bits: Optional[torch.Tensor],
-                     scale: float, window: int, sink: bool, causal: bool = False) -> torch.Tensor:
-    """:func:`paged_tree_attention` with a window, an optional valueless key of score 0, and heads narrower than the pools'
-    rows.  A row sees the last ``window`` tokens of its own path (itself included): in a tree a node's position is the
-    committed length plus its number of proper ancestors.  Returns ``(T, Hq*vdim)``."""
+                     scale: float, window: int, sink, causal: bool = False, keep_first: int = 0) -> torch.Tensor:
+    """:func:`paged_tree_attention` with a window, an optional sink, and heads narrower than the pools' rows.  ``sink``: whether
+    a valueless key of score 0 takes part in the softmax, or such a key's score per head ``(Hq,)``.  A row sees the last
+    ``window`` tokens of its own path (itself included) and those at positions below ``keep_first``: in a tree a node's
+    position is the committed length plus its number of proper ancestors.  Returns ``(T, Hq*vdim)``."""
     T, Hq, D = q.shape
     Hkv = k_pool.shape[0]
     g = Hq // Hkv
@@ -380,10 +390,12 @@ def window_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
         pos = past + anc.sum(-1) - 1
         key_pos = torch.cat((torch.arange(past, device=q.device), pos))
         vis = torch.cat((torch.ones(n, past, dtype=torch.bool, device=q.device), anc), -1)
-        vis &= pos[:, None] - key_pos[None] < window
+        vis &= (pos[:, None] - key_pos[None] < window) | (key_pos < keep_first)[None]
         sc = torch.einsum("nhgd,hld->hgnl", q[s:e].float().view(n, Hkv, g, D), k) * scale
         sc = sc.masked_fill(~vis[None, None], float("-inf"))
-        if sink:
+        if isinstance(sink, torch.Tensor):
+            sc = torch.cat((sc, sink.float().view(Hkv, g, 1, 1).expand(Hkv, g, n, 1)), -1)
+        elif sink:
             sc = torch.cat((sc, torch.zeros_like(sc[..., :1])), -1)
         p = torch.nan_to_num(torch.softmax(sc, dim=-1), nan=0.0)[..., : past + n]
         out[s:e] = torch.einsum("hgnl,hlv->nhgv", p, v).reshape(n, Hq * vdim).to(q.dtype)
@@ -453,10 +465,12 @@ def delta_mix(pre: torch.Tensor, z: torch.Tensor, b: torch.Tensor, taps: torch.T
     return out
 
 
-def gated_head_norm(o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, kind: str, eps: float) -> torch.Tensor:
-    """``o (T, H, V)`` divided by its root mean square per head, times ``weight (V,)``, times ``silu`` or ``sigmoid`` of
-    ``gate (T, H*V)``; fp32 math, result in ``gate.dtype``."""
-    y = o.float() / torch.sqrt(o.float().pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+def gated_head_norm(o: torch.Tensor, weight: Optional[torch.Tensor], gate: torch.Tensor, kind: str, eps: float) -> torch.Tensor:
+    """``o (T, H, V)`` divided by its root mean square per head, times ``weight (V,)`` if any, times ``silu`` or ``sigmoid``
+    of ``gate (T, H*V)``; fp32 math, result in ``gate.dtype``."""
+    y = o.float() / torch.sqrt(o.float().pow(2).mean(-1, keepdim=True) + eps)
+    if weight is not None:
+        y = y * weight.float()
     a = F.silu(gate.float()) if kind == "silu" else torch.sigmoid(gate.float())
     return (y.reshape(gate.shape) * a).to(gate.dtype)
 
@@ -469,3 +483,64 @@ def experts_swiglu(x, idx, w_gate, w_up, w_down) -> torch.Tensor:
         a = silu_mul(torch.cat((F.linear(x[tok], w_gate[e]), F.linear(x[tok], w_up[e])), -1))
         out.index_add_(0, tok, F.linear(a, w_down[e]).float())
     return out / idx.shape[1]
+
+
+# --------------------------------------------------------------------------
+# general rotations, gates per head, retention
+# --------------------------------------------------------------------------
+def gelu_erf(x: torch.Tensor) -> torch.Tensor:
+    """Exact gelu, fp32 inside."""
+    return F.gelu(x.float()).to(x.dtype)
+
+
+def rotate(x: torch.Tensor, positions: torch.Tensor, rot, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """Rotate the pairs ``rot`` (a ``RotaryConfig``) names in every head of ``x (T, heads, D)``; the entries behind
+    ``rot.dims`` pass unchanged.  fp32 math."""
+    y, n = x.float().clone(), rot.dims // 2
+    if n:
+        f = torch.tensor(rot.frequencies(), dtype=torch.float32, device=x.device)
+        a, amp = positions.to(torch.float32)[:, None] * f, rot.amplitude()
+        c, s = (amp * a.cos())[:, None], (amp * a.sin())[:, None]
+        first, second = (slice(0, n), slice(n, 2 * n)) if rot.pairing == "half" else (slice(0, 2 * n, 2), slice(1, 2 * n, 2))
+        u, v = y[..., first].clone(), y[..., second].clone()
+        y[..., first], y[..., second] = u * c - v * s, v * c + u * s
+    return y.to(out_dtype or x.dtype)
+
+
+def head_gate(y: torch.Tensor, logits: torch.Tensor) -> torch.Tensor:
+    """``y (T, H*V)`` with head ``h``'s columns times ``sigmoid(logits[:, h])``, ``logits (T, H)``."""
+    T, H = logits.shape
+    return (y.float().view(T, H, -1) * torch.sigmoid(logits.float())[..., None]).reshape(T, -1).to(y.dtype)
+
+
+def retention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cfg, state: torch.Tensor, rows: torch.Tensor, cu_q: torch.Tensor,
+              past_lens: torch.Tensor, mask_bits: Optional[torch.Tensor], causal: bool = True) -> torch.Tensor:
+    """Linear attention with one fixed decay per head over a ragged batch: ``S <- decay S + k v^T; o = S^T q``.
+
+    ``q, k (T, H*D)`` and ``v (T, H*V)`` rows, ``state (slots, H, D, V)`` fp32; sequences, fresh starts and trees as in
+    :func:`delta_mix`.  Returns the read-outs, fp32 ``(T, H, V)``."""
+    H, D, V = cfg.heads, cfg.dim, cfg.vdim
+    T = q.shape[0]
+    q, k, v = q.float().view(T, H, D), k.float().view(T, H, D), v.float().view(T, H, V)
+    decay = torch.tensor(cfg.decay, dtype=torch.float32, device=q.device)[:, None, None]
+    out = torch.empty(T, H, V, dtype=torch.float32, device=q.device)
+    cu, pl, rl = cu_q.tolist(), past_lens.tolist(), rows.tolist()
+    for i in range(len(cu) - 1):
+        s, e = cu[i], cu[i + 1]
+        S0 = state[rl[i]].clone() if pl[i] > 0 else torch.zeros_like(state[rl[i]])
+        anc = None if causal else unpack_ancestor_bits(mask_bits[s:e], e - s).cpu()
+        kept = []
+        for t in range(s, e):
+            if causal:
+                parent = len(kept) - 1
+            else:
+                up = [j for j in range(t - s) if bool(anc[t - s, j])]
+                parent = up[-1] if up else -1
+            S = decay * (kept[parent] if parent >= 0 else S0) + k[t][..., None] * v[t][:, None]
+            out[t] = torch.einsum("hdv,hd->hv", S, q[t])
+            if causal and kept:
+                kept[-1] = None
+            kept.append(S)
+        if causal and kept:
+            state[rl[i]] = kept[-1]
+    return out

@@ -3,8 +3,8 @@
 A decoder calls the backend once per layer run, ``backend(layer, q, k, v)`` for K/V attention,
 ``backend.latent(layer, mixer, q, c)`` for latent attention or ``backend.window(layer, mixer, q, k, v)`` for window
 attention; the backend writes the new rows into the pool at the step's slots and attends through the slot map.
-``backend.delta(layer, mixer, pre, z, b)`` advances the recurrent states of the batch's sequences (or, for token trees,
-reads them and holds the nodes' inputs until a path is committed).
+``backend.recur(layer, mixer, *inputs)`` advances the recurrent states of the batch's sequences by what ``mixer.mix`` makes of
+the inputs (or, for token trees, reads them and holds the nodes' inputs until a path is committed).
 """
 from __future__ import annotations
 
@@ -28,19 +28,20 @@ class PagedAttention:
         m, pool = self.meta, self.pool.latent(layer)
         ops.latent_scatter(c, pool, m.slots)
         return ops.latent_attention(q, mixer.k_up.weight, mixer.v_up.weight, pool, self.pool.slot_map, m.seq_rows,
-                                    m.cu_q, m.past_lens, m.mask_bits, mixer.cfg.scale, causal=m.causal)
+                                    m.cu_q, m.past_lens, m.mask_bits, mixer.cfg.scale, causal=m.causal, sink=mixer.sink)
 
     def window(self, layer, mixer, q, k, v):
         m, c = self.meta, mixer.cfg
         kp, vp = self.pool.layer(layer)
         ops.window_scatter(k, v, kp, vp, m.slots)
         return ops.window_attention(q, kp, vp, c.vdim, self.pool.slot_map, m.seq_rows, m.cu_q, m.past_lens, m.mask_bits, c.scale,
-                                    c.window, c.sink, causal=m.causal)
+                                    c.window, mixer.sink, causal=m.causal, keep_first=c.keep_first)
 
-    def delta(self, layer, mixer, pre, z, b):
+    def recur(self, layer, mixer, *inputs):
         m, states = self.meta, self.pool.states
-        weights = (mixer.conv(), mixer.A_log, mixer.dt_bias)
         if not m.causal:
-            states.hold(layer, weights, pre, z, b)
+            states.hold(layer, mixer, inputs)
         state, conv = states.layer(layer)
-        return ops.delta_mix(pre, z, b, *weights, mixer.cfg, state, conv, m.seq_rows, m.cu_q, m.past_lens, m.mask_bits, m.causal)
+        return mixer.mix(inputs, state, conv, m.seq_rows, m.cu_q, m.past_lens, m.mask_bits, m.causal)
+
+    delta = recur

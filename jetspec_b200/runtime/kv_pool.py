@@ -17,6 +17,9 @@ slot is its slot-map row, so it is granted, given back, evicted and used again t
     kv_layers : list of (k_pool, v_pool) or None
     states    : StatePool or None
 
+Kinds can differ from layer to layer: ``kv_layers`` and ``latent_pools`` then hold ``None`` where a layer caches the other kind
+or nothing.
+
 Everything below the buffers (pages, slot maps, admission, eviction, commit) is the same for all kinds.
 
 A *page* (``page_size`` consecutive slots) is the unit of allocation and is shared
@@ -91,9 +94,10 @@ class PagedKVPool:
             def pools(heads, dim, vdim):
                 return tuple(torch.zeros(heads, S, w, dtype=dtype, device=device) for w in window_row_width(dim, vdim, dtype))
             self.kv_layers = [pools(*shape) if shape is not None else None for shape in kv_shapes]
-        elif latent_widths is not None:
-            self.latent_pools = [torch.zeros(S, latent_row_width(w), dtype=dtype, device=device) for w in latent_widths]
-        else:
+        if latent_widths is not None:
+            self.latent_pools = [None if w is None else torch.zeros(S, latent_row_width(w), dtype=dtype, device=device)
+                                 for w in latent_widths]
+        if kv_shapes is None and latent_widths is None:
             self.k_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
             self.v_pool = torch.zeros(num_layers, num_kv_heads, S, head_dim, dtype=dtype, device=device)
         if state_shapes is not None:
@@ -110,11 +114,9 @@ class PagedKVPool:
     @classmethod
     def for_model(cls, cfg, num_pages: int, world: int = 1, **kw) -> "PagedKVPool":
         """A pool of the shape ``cfg``'s attention caches (``world``: ranks the K/V heads are sharded over)."""
-        widths = cfg.latent_widths()
-        if widths is not None:
-            return cls(len(widths), 0, 0, num_pages, latent_widths=widths, **kw)
-        if cfg.kv_shapes() is not None:
-            return cls(cfg.num_hidden_layers, 0, 0, num_pages, kv_shapes=cfg.kv_shapes(), state_shapes=cfg.state_shapes(), **kw)
+        widths, shapes = cfg.latent_widths(), cfg.kv_shapes()
+        if widths is not None or shapes is not None:
+            return cls(cfg.num_hidden_layers, 0, 0, num_pages, latent_widths=widths, kv_shapes=shapes, state_shapes=cfg.state_shapes(), **kw)
         return cls(cfg.num_hidden_layers, cfg.num_key_value_heads // world, cfg.head_dim, num_pages, **kw)
 
     @property

@@ -4,6 +4,7 @@ Per recurrent layer::
 
     state : (slots + 1, heads, dim, vdim)      fp32
     conv  : (slots + 1, taps, channels)        ring of the short convolutions' last inputs: position p in entry p % taps
+                                               (None for a recurrence without convolutions)
 
 A sequence's slot is its slot-map row in the paged pool.  Nothing is cleared when a slot changes hands: a forward whose
 committed length is 0 starts from zeros whatever the slot holds.  The last slot belongs to no sequence; warm-up launches
@@ -19,8 +20,6 @@ from typing import Callable, Optional
 
 import torch
 
-from .. import ops
-
 
 class StatePool:
     def __init__(self, shapes: list, slots: int, device="cpu", dtype=torch.float32):
@@ -30,10 +29,10 @@ class StatePool:
         self.conv: list = []
         for c in self.shapes:
             self.state.append(None if c is None else torch.zeros(slots + 1, c.heads, c.dim, c.vdim, dtype=torch.float32, device=device))
-            self.conv.append(None if c is None else torch.zeros(slots + 1, c.taps, c.channels, dtype=dtype, device=device))
+            self.conv.append(None if c is None or not c.channels else torch.zeros(slots + 1, c.taps, c.channels, dtype=dtype, device=device))
         self._at: dict = {}          # state slot -> first row of its tree among the held rows
         self._advance = None
-        self._held: dict = {}        # layer -> (weights, pre, z, b) of every row of the last tree forward
+        self._held: dict = {}        # layer -> (mixer, recurrence inputs of every row of the last tree forward)
 
     @property
     def scratch(self) -> int:
@@ -48,9 +47,9 @@ class StatePool:
         that holds the rows itself gives ``advance(row, past, start, path)``, which :meth:`commit` then calls."""
         self._at, self._held, self._advance = {int(r): int(s) for r, s in zip(rows, starts)}, {}, advance
 
-    def hold(self, layer: int, weights, pre, z, b) -> None:
-        """Keep a layer's recurrence inputs of a tree forward.  ``weights`` is ``(taps, A_log, dt_bias)``."""
-        self._held[layer] = (weights, pre, z, b)
+    def hold(self, layer: int, mixer, inputs) -> None:
+        """Keep a layer's recurrence inputs of a tree forward, the ones ``mixer.mix`` takes."""
+        self._held[layer] = (mixer, inputs)
 
     def commit(self, row: int, past: int, path: torch.Tensor) -> None:
         """Advance slot ``row`` (at committed length ``past``) along the accepted nodes ``path`` of its held tree."""
@@ -64,6 +63,5 @@ class StatePool:
         idx = path.to(self.device).long() + start
         i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=self.device)
         rows, cu_q, past_t = i32([row]), i32([0, n]), i32([past])
-        for i, ((taps, A_log, dt_bias), pre, z, b) in self._held.items():
-            ops.delta_mix(pre[idx], z[idx], b[idx], taps, A_log, dt_bias, self.shapes[i], self.state[i], self.conv[i], rows, cu_q,
-                          past_t, None, True)
+        for i, (mixer, inputs) in self._held.items():
+            mixer.mix([x[idx] for x in inputs], self.state[i], self.conv[i], rows, cu_q, past_t, None, True)
