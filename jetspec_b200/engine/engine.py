@@ -202,7 +202,8 @@ class JetSpecEngine:
                                    num_query_nodes=None if trees is not None else [int(t.numel()) for t in token_rows],
                                    device=self.device)
         ids = torch.cat([t.reshape(-1) for t in token_rows]).to(self.device)
-        if self.ragged_kernels:
+        # states advance over trees of up to 256 nodes on the kernel path
+        if self.ragged_kernels and (meta.causal or pool.states is None or meta.mask_bits.shape[1] <= 8):
             from .fast_round import FastRound
             logits, hidden = FastRound.get(self).ragged_forward(ids, meta, past_lens, taps, logits_rows)
             return logits, hidden, meta

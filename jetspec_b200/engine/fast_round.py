@@ -312,6 +312,20 @@ def decoder_layers(cfg, layers, st: _Stack, k_pools, v_pools, slot_map, seq_rows
     return n
 
 
+def _stack_class(name: str):
+    """Fused launch sequence of a decoder that :func:`decoder_layers` does not cover."""
+    if name == "latent":
+        from .latent_stack import LatentStack
+        return LatentStack
+    if name == "hybrid":
+        from .hybrid_stack import HybridStack
+        return HybridStack
+    if name == "prenorm":
+        from .prenorm_stack import PreNormStack
+        return PreNormStack
+    raise ValueError(f"unknown kernel stack {name!r}")
+
+
 class FastRound:
     """Graph-captured decode rounds for one engine (single sequence, greedy)."""
 
@@ -334,13 +348,10 @@ class FastRound:
         if self.tp is not None and self.ep is not None:
             raise NotImplementedError("tensor parallelism and expert parallelism are separate plans here")
         world = self.tp.world if self.tp is not None else 1
-        if self.cfg.latent_widths() is not None or self.cfg.kv_shapes() is not None:
+        if self.cfg.kernel_stack() is not None:
             if self.tp is not None or self.ep is not None:
                 raise NotImplementedError(f"{self.cfg.model_type} models run on one GPU")
-            if self.cfg.latent_widths() is not None:
-                from .latent_stack import LatentStack as Stack
-            else:
-                from .hybrid_stack import HybridStack as Stack
+            Stack = _stack_class(self.cfg.kernel_stack())
             self.stack = Stack(m, self.device)
             self.lm_head_w = self.stack.head
             self.lcfg, self.layers, self.freq = None, None, None
@@ -413,6 +424,8 @@ class FastRound:
         out = torch.empty(rows.shape[0], (V + 3) // 4 * 4, dtype=torch.float32, device=self.device)
         if rows.shape[0]:
             X.gemm(rows, self.lm_head_w, out=out, epi=X.EPI_STORE_F32)
+            if self.cfg.logit_scale != 1.0:
+                out *= self.cfg.logit_scale
         return out[:, :V]
 
     # ------------------------------------------------------------------ support matrix
@@ -748,7 +761,7 @@ class FastRound:
             r["uniform"].uniform_()
             lib.js_sample_temperature.restype = ctypes.c_int
             X._check(lib.js_sample_temperature(p(r["logits"]), 0, NB, self.lm_head_w.shape[0], r["logits"].stride(0),
-                                               ctypes.c_float(r["temperature"]), p(r["uniform"]), p(r["sampled"]), s()),
+                                               ctypes.c_float(r["temperature"] / self.cfg.logit_scale), p(r["uniform"]), p(r["sampled"]), s()),
                      "js_sample_temperature")
             r["greedy"].copy_(r["sampled"])
             n += 1

@@ -30,8 +30,8 @@ import numpy as np
 import torch
 
 from ..ops import cuda_ext as X
-from ..runtime.kv_pool import window_row_width
-from .latent_stack import MAX_SORT_PAIRS, _pad, _up
+from .latent_stack import MAX_SORT_PAIRS
+from .mixers import WindowMixer, pad, up
 
 FORK_MIN_TOKENS = 512          # eager launches fork from this many rows on (below, the host is what a forward waits for)
 
@@ -43,7 +43,7 @@ def _cols(parts, align: int = 8):
     offs, at = [], 0
     for n in parts:
         offs.append(at)
-        at = _up(at + n, align)
+        at = up(at + n, align)
     return offs, at
 
 
@@ -56,7 +56,7 @@ def _stack_rows(ws, offs, rows: int, cols: int) -> torch.Tensor:
 
 
 def _interleave(gate: torch.Tensor, up: torch.Tensor, ff: int, cols: int) -> torch.Tensor:
-    return X.interleave_gate_up(_pad(gate, ff, cols), _pad(up, ff, cols), 128)
+    return X.interleave_gate_up(pad(gate, ff, cols), pad(up, ff, cols), 128)
 
 
 class _LayerWeights:
@@ -75,9 +75,9 @@ class _LayerWeights:
             ws.append(w.detach())
 
         if self.parallel:
-            self._window(layer.mixer.left, l.window, wp, f32)
-            for n in "qkv":
-                add("w" + n, getattr(layer.mixer.left, n + "_proj").weight)
+            self.win = WindowMixer(layer.mixer.left, cfg.norm_eps, wp)
+            for n, w in zip("qkv", self.win.qkv):
+                add("w" + n, w)
             self.left_norm, self.right_norm = f32(layer.mixer.left_norm.weight), f32(layer.mixer.right_norm.weight)
         raw = [d.beta_proj.weight.detach()]
         if not c.decay_rank:
@@ -98,66 +98,49 @@ class _LayerWeights:
         sizes = dict(zip(names, (w.shape[0] for w in ws)))
         for n in names:
             if not any(n in g[1:] for g in groups):
-                at = _up(at, 8)
+                at = up(at, 8)
             self.at[n] = at
             at += sizes[n]
-        self.n_raw, self.act_cols = _up(sum(w.shape[0] for w in raw), 128), _up(at, 128)
-        self.w_in = torch.cat((_pad(torch.cat(raw, 0), self.n_raw, wp),
+        self.n_raw, self.act_cols = up(sum(w.shape[0] for w in raw), 128), up(at, 128)
+        self.w_in = torch.cat((pad(torch.cat(raw, 0), self.n_raw, wp),
                                _stack_rows(ws, [self.at[n] for n in names], self.act_cols, wp)), 0)
         # second factors: [decay logits (fp32) | gate (bf16)] over [a1 | g1]
         self.low = None
         if low:
             k0 = self.at[low[0][0]]
-            kc = _up(self.at[low[-1][0]] + low[-1][1].shape[0] - k0, 8)
+            kc = up(self.at[low[-1][0]] + low[-1][1].shape[0] - k0, 8)
             assert k0 + kc <= self.act_cols
-            nz = _up(c.decays, 128) if c.decay_rank else 0
-            ng = _up(c.heads * c.vdim, 128) if c.gate_rank else 0
+            nz = up(c.decays, 128) if c.decay_rank else 0
+            ng = up(c.heads * c.vdim, 128) if c.gate_rank else 0
             w2 = torch.zeros(nz + ng, kc, dtype=ws[0].dtype, device=ws[0].device)
-            for n, _, up in low:
+            for n, _, second in low:
                 r0, k = (0 if n == "a1" else nz), self.at[n] - k0
-                w2[r0:r0 + up.shape[0], k:k + up.shape[1]] = up.detach()
+                w2[r0:r0 + second.shape[0], k:k + second.shape[1]] = second.detach()
             self.low = types.SimpleNamespace(k0=k0, kc=kc, nz=nz, ng=ng, w=w2)
         self.taps, self.A_log, self.dt_bias = d.conv().detach().contiguous(), d.A_log.detach(), d.dt_bias.detach()
         self.o_norm, self.eps = d.o_norm.detach(), cfg.norm_eps
-        self.o_cols = _up(c.heads * c.vdim, 8)
-        self.w_o = _pad(d.o_proj.weight.detach(), wp, self.o_cols)
+        self.o_cols = up(c.heads * c.vdim, 8)
+        self.w_o = pad(d.o_proj.weight.detach(), wp, self.o_cols)
         self.norm1 = f32(layer.norm1.weight)
         self.moe = None
         if layer.mlp is not None:
             self._experts(layer.mlp, wp)
             self.norm2 = f32(layer.norm2.weight)
 
-    def _window(self, m, c, wp: int, f32) -> None:
-        self.wc, self.freq = c, None
-        g = c.heads // c.kv_heads
-        self.Dp, self.Vp = window_row_width(c.dim, c.vdim, torch.bfloat16)
-        gp = 1 << (g - 1).bit_length()
-        self.tc = self.Dp == 128 and self.Vp == 128 and gp <= 16        # what the tensor-core kernel takes
-        self.gp, self.Dq, vq = (gp, 128, 128) if self.tc else (g, c.dim, c.vdim)
-        self.wq_cols, self.wo_cols = c.kv_heads * self.gp * self.Dq, _up(c.kv_heads * self.gp * vq, 8)
-        o = torch.zeros(wp, c.kv_heads, self.gp, vq, dtype=m.o_proj.weight.dtype, device=m.o_proj.weight.device)
-        o[: m.o_proj.weight.shape[0], :, :g, : c.vdim] = m.o_proj.weight.detach().view(-1, c.kv_heads, g, c.vdim)
-        self.w_wo = _pad(o.view(wp, -1), wp, self.wo_cols)
-        self.qkv_bias = self.wo_bias = None
-        if c.bias:
-            self.qkv_bias = torch.cat([f32(p.bias) for p in (m.q_proj, m.k_proj, m.v_proj)])
-            self.wo_bias = f32(m.o_proj.bias)
-        self.freq = X.pair_freq(c.rot_dims, c.rot_base, m.q_proj.weight.device)
-
     def _experts(self, m, wp: int) -> None:
         c = m.cfg
-        ff, W = _up(c.ff, 64), m.w_down.shape[1]
-        wd = _up(W, 128)
+        ff, W = up(c.ff, 64), m.w_down.shape[1]
+        wd = up(W, 128)
         gu = torch.cat([_interleave(m.w_gate[e].detach(), m.w_up[e].detach(), ff, wp) for e in range(c.experts)], 0)
         dn = torch.zeros(c.experts, wd, ff, dtype=gu.dtype, device=gu.device)
         dn[:, :W, : c.ff] = m.w_down.detach()
         self.moe = types.SimpleNamespace(E=c.experts, top=c.top, ff=ff, wd=wd, up=gu, down=dn.view(c.experts * wd, ff),
                                          table=m.table.contiguous(), shared=None)
         if c.shared_ff:
-            sf = _up(c.shared_ff, 64)
+            sf = up(c.shared_ff, 64)
             self.moe.shared = types.SimpleNamespace(
                 ff=sf, up=_interleave(m.shared_gate.weight.detach(), m.shared_up.weight.detach(), sf, wp),
-                down=_pad(m.shared_down.weight.detach(), wp, sf))
+                down=pad(m.shared_down.weight.detach(), wp, sf))
 
 
 class HybridStack:
@@ -166,11 +149,11 @@ class HybridStack:
     def __init__(self, model, device):
         cfg = model.config
         self.cfg, self.device = cfg, torch.device(device)
-        self.width, self.wp = cfg.hidden_size, _up(cfg.hidden_size, 8)
+        self.width, self.wp = cfg.hidden_size, up(cfg.hidden_size, 8)
         self.layers = [_LayerWeights(l, cfg, i, self.wp) for i, l in enumerate(model.model.layers)]
         self.final_norm = model.model.norm.weight.detach().float().contiguous()
         table, head = model.model.embed_tokens.weight.detach(), model.lm_head.weight.detach()
-        self.table, self.head = (w if self.wp == self.width else _pad(w, w.shape[0], self.wp) for w in (table, head))
+        self.table, self.head = (w if self.wp == self.width else pad(w, w.shape[0], self.wp) for w in (table, head))
         self.vocab = cfg.vocab_size
         self.routed = [L for L in self.layers if L.moe is not None]
         self.side = torch.cuda.Stream(self.device) if self.device.type == "cuda" else None
@@ -206,13 +189,6 @@ class HybridStack:
             return cols[key]
         b.get = get
         return b
-
-    def _attn_ws(self, st, splits: int, Hq: int):
-        key = (splits, Hq)
-        if splits > 1 and key not in st.ws:
-            st.ws[key] = {"o": torch.zeros(splits, st.T, Hq, 128, dtype=torch.float32, device=self.device),
-                          "ml": torch.zeros(splits, st.T, Hq, 2, dtype=torch.float32, device=self.device)}
-        return st.ws.get(key)
 
     def _delta_buf(self, st, L, hold: bool, kind: str = "rows", seqs: int = 0) -> dict:
         """Workspace of a delta layer: one for all layers of a shape, or one each when it has to outlive the forward."""
@@ -304,7 +280,7 @@ class HybridStack:
         mlp = L.moe is not None
         end = dict(out=None if mlp else out, tap=None if mlp else tap)
         if L.parallel:
-            self._resid(st, L.norm1, L.eps, ya=yl, bias=L.wo_bias, wa=L.left_norm, yb=yr, wb=L.right_norm, pdl=pdl and not fork, **end)
+            self._resid(st, L.norm1, L.eps, ya=yl, bias=L.win.o_bias, wa=L.left_norm, yb=yr, wb=L.right_norm, pdl=pdl and not fork, **end)
         else:
             self._resid(st, L.norm1, L.eps, ya=yr, pdl=pdl, **end)
         n += 1
@@ -316,28 +292,9 @@ class HybridStack:
         return st.T >= FORK_MIN_TOKENS or torch.cuda.is_current_stream_capturing()
 
     def _window(self, st, L, pool, batch, act, y, pdl, first_pdl) -> int:
-        c, T = L.wc, st.T
-        lib, p = X.load(), X._p
-        kp, vp = pool.layer(L.index)
-        q = st.get("wq", L.wq_cols, zero=L.gp * c.kv_heads != c.heads)
-        proj = act[:, L.at["wq"]:]
-        X._check(lib.js_window_post(
-            p(proj), proj.stride(0), p(L.qkv_bias), c.heads, c.kv_heads, L.gp, c.dim, c.vdim, L.Dq, L.Dp, L.Vp, c.rot_dims, p(L.freq),
-            int(c.qk_norm), X.ctypes.c_float(L.eps), p(batch.positions), p(batch.slots), kp.shape[1], T, p(q), p(kp), p(vp),
-            p(X.status_word(self.device)), int(first_pdl), X._stream()), "js_window_post")
-        o = st.get("wo", L.wo_cols, zero=True)
-        Hq, n = c.kv_heads * L.gp, 3
-        args = (batch.slot_map, batch.seq_rows, batch.cu_q, batch.past, batch.mask)
-        if L.tc and (batch.mask is None or batch.mask.shape[1] <= 8):
-            splits = X.window_attn_splits(T, Hq, c.kv_heads, batch.max_keys, c.window)
-            X.window_attention_tc(q.view(T, Hq, 128), kp, vp, *args, c.scale, c.window, c.sink, batch.mask is None, o, splits=splits,
-                                  ws=self._attn_ws(st, splits, Hq), pdl=pdl)
-            n += int(splits > 1 and not X.attn_merges_in_cluster(T, Hq, c.kv_heads, splits))
-        else:
-            X.window_attention(q.view(T, c.heads, c.dim), kp, vp, c.vdim, *args, c.scale, c.window, c.sink, batch.mask is None, out=o,
-                               pdl=pdl)
-        X.gemm(o, L.w_wo, out=y, pdl=pdl)
-        return n
+        o, n = L.win.run(st, pool.layer(L.index), batch, act[:, L.at["wq"]:], None, None, pdl, first_pdl)
+        X.gemm(o, L.win.w_o, out=y, pdl=pdl)
+        return n + 1
 
     def _delta(self, st, L, pool, batch, pre, z, b, gate, y, hold, pdl) -> int:
         c = L.dc

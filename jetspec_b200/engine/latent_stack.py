@@ -6,11 +6,7 @@ Per layer run, with everything between the GEMMs folded into them or into one sm
    gate leave as fp32; gate/up (or the shared expert's up) leave as activated bf16, next to where the attention output
    will be (``cat``);
 2. latent RMS norms, the new row goes straight to its pool slot; sigmoid routing scales the shared activations;
-3. query up-projection, then one of two attention forms:
-   *absorbed* (decode, trees, short portions): ``W_uk`` is applied to the query and ``W_uv`` behind the attention, both as
-   batched GEMMs over heads, and the tcgen05 latent kernel attends over the cached rows themselves;
-   *expanded* (long prompt portions): keys and values are expanded from the gathered latents once and the tcgen05 K/V
-   kernel attends over them, which costs (dim + vdim) instead of 2 kv_rank per score;
+3. query up-projection, then one of the two attention forms of :class:`~jetspec_b200.engine.mixers.LatentMixer`;
 4. ONE output GEMM over ``cat``: attention output and feed-forward are both added to the fp32 residual stream, and the
    NEXT run's Dynamic Tanh is applied in the epilogue (with the embedding added first where a loop pass begins).
    Routed layers apply it in the experts' combine kernel instead.
@@ -24,30 +20,9 @@ import types
 import torch
 
 from ..ops import cuda_ext as X
-from ..runtime.kv_pool import latent_row_width
+from .mixers import EXPAND_MIN_TOKENS, LatentMixer, pad, pad_heads, up
 
 MAX_SORT_PAIRS = 16384        # (token, expert) pairs one launch of the permutation kernel takes
-EXPAND_MIN_TOKENS = 128       # a portion of at least this many tokens may take the expanded form
-
-
-def _up(n: int, m: int) -> int:
-    return (int(n) + m - 1) // m * m
-
-
-def _pad(w: torch.Tensor, rows: int, cols: int) -> torch.Tensor:
-    if w.shape == (rows, cols):
-        return w.contiguous()
-    out = torch.zeros(rows, cols, dtype=w.dtype, device=w.device)
-    out[: w.shape[0], : w.shape[1]] = w
-    return out
-
-
-def _pad_heads(w: torch.Tensor, heads: int, rows: int, cols: int) -> torch.Tensor:
-    """``(heads * r, c)`` -> ``(heads * rows, cols)``, every head padded on its own."""
-    r = w.shape[0] // heads
-    out = torch.zeros(heads, rows, cols, dtype=w.dtype, device=w.device)
-    out[:, :r, : w.shape[1]] = w.view(heads, r, w.shape[1])
-    return out.view(heads * rows, cols)
 
 
 class _LayerWeights:
@@ -55,11 +30,9 @@ class _LayerWeights:
 
     def __init__(self, layer, width: int, wp: int):
         m, mix, mlp = layer.mixer.cfg, layer.mixer, layer.mlp
-        self.heads, self.q_rank, self.kv_rank, self.scale, self.eps = m.heads, m.q_rank, m.kv_rank, m.scale, mix.eps
-        self.qp, self.rp = _up(m.q_rank, 8), latent_row_width(m.kv_rank)
-        # the K/V kernel has 128-wide heads; padding narrower ones up to it pays from 64 on
-        self.expand = 64 <= m.dim <= 128 and 64 <= m.vdim <= 128
-        self.dp, self.vp = (128, 128) if self.expand else (_up(m.dim, 8), _up(m.vdim, 8))
+        self.q_rank, self.kv_rank, self.eps = m.q_rank, m.kv_rank, mix.eps
+        self.mix = LatentMixer(mix)
+        self.qp = up(m.q_rank, 8)
         self.norm = (layer.norm.weight.float(), layer.norm.bias.float(), layer.norm.alpha.item())
         self.q_norm, self.kv_norm = mix.q_norm, mix.kv_norm
         raw = [mix.q_down.weight, mix.kv_down.weight]
@@ -68,13 +41,13 @@ class _LayerWeights:
         self.act_cols = 0
         self.gelu = True
         if mlp is not None and hasattr(mlp, "gate_proj"):
-            ff = _up(mlp.gate_proj.weight.shape[0], 64)
-            g, u = (_pad(w, ff, width).view(ff // 64, 64, width) for w in (mlp.gate_proj.weight, mlp.up_proj.weight))
+            ff = up(mlp.gate_proj.weight.shape[0], 64)
+            g, u = (pad(w, ff, width).view(ff // 64, 64, width) for w in (mlp.gate_proj.weight, mlp.up_proj.weight))
             act_w, self.act_cols, down = torch.cat((g, u), 1).reshape(2 * ff, width), ff, mlp.down_proj.weight
         elif mlp is not None:
             c = mlp.cfg
             raw.append(mlp.router.weight)
-            ffp, wd = _up(c.ff, 128), _up(width, 128)
+            ffp, wd = up(c.ff, 128), up(width, 128)
             self.moe = types.SimpleNamespace(
                 E=c.experts, top=c.top, scale=c.scale, ffp=ffp, wd=wd, corr=mlp.correction.float().contiguous(),
                 up=torch.zeros(c.experts * ffp, wp, dtype=mlp.w_up.dtype, device=mlp.w_up.device),
@@ -85,25 +58,18 @@ class _LayerWeights:
             if c.shared_ff:
                 raw.append(mlp.shared_gate.weight)
                 self.moe.gate_col = c.experts
-                self.gelu, self.act_cols = False, _up(c.shared_ff, 128)
-                act_w, down = _pad(mlp.shared_up.weight, self.act_cols, width), mlp.shared_down.weight
+                self.gelu, self.act_cols = False, up(c.shared_ff, 128)
+                act_w, down = pad(mlp.shared_up.weight, self.act_cols, width), mlp.shared_down.weight
         raw_w = torch.cat(raw, 0)
-        self.n_raw = _up(raw_w.shape[0], 128)
-        raw_w = _pad(raw_w, self.n_raw, width)
-        self.w_in = _pad(raw_w if act_w is None else torch.cat((raw_w, act_w), 0), self.n_raw + (0 if act_w is None else act_w.shape[0]), wp)
-        self.uq = _pad(_pad_heads(mix.q_up.weight, m.heads, self.dp, m.q_rank), m.heads * self.dp, self.qp)
-        uk, uv = mix.k_up.weight, mix.v_up.weight
-        self.uk_t = _pad_heads(uk.view(m.heads, m.dim, m.kv_rank).transpose(1, 2).reshape(m.heads * m.kv_rank, m.dim),
-                               m.heads, self.rp, self.dp)
-        self.uv = _pad_heads(uv, m.heads, self.vp, self.rp)
-        # keys and values of every head from a latent row, one product: [heads * 128 keys | heads * 128 values]
-        self.ukv = torch.cat((_pad_heads(uk, m.heads, self.dp, self.rp), self.uv), 0) if self.expand else None
-        attn_cols = m.heads * self.vp
+        self.n_raw = up(raw_w.shape[0], 128)
+        raw_w = pad(raw_w, self.n_raw, width)
+        self.w_in = pad(raw_w if act_w is None else torch.cat((raw_w, act_w), 0), self.n_raw + (0 if act_w is None else act_w.shape[0]), wp)
+        self.uq = pad(pad_heads(mix.q_up.weight, m.heads, self.mix.dp, m.q_rank), m.heads * self.mix.dp, self.qp)
+        attn_cols = self.mix.out_cols
         self.cat_cols = attn_cols + self.act_cols
-        self.w_out = torch.zeros(wp, self.cat_cols, dtype=uk.dtype, device=uk.device)
-        o = torch.zeros(width, m.heads, self.vp, dtype=uk.dtype, device=uk.device)
-        o[:, :, : m.vdim] = mix.o_proj.weight.view(width, m.heads, m.vdim)
-        self.w_out[:width, :attn_cols] = o.view(width, attn_cols)
+        self.w_out = torch.zeros(wp, self.cat_cols, dtype=mix.o_proj.weight.dtype, device=mix.o_proj.weight.device)
+        self.w_out[:width, :attn_cols] = self.mix.w_o
+        self.mix.w_o = None
         if self.act_cols:
             self.w_out[:width, attn_cols:attn_cols + down.shape[1]] = down
 
@@ -114,7 +80,7 @@ class LatentStack:
     def __init__(self, model, device):
         cfg = model.config
         self.cfg, self.device = cfg, torch.device(device)
-        self.width, self.wp = cfg.hidden_size, _up(cfg.hidden_size, 8)
+        self.width, self.wp = cfg.hidden_size, up(cfg.hidden_size, 8)
         self.layers = [_LayerWeights(l, self.width, self.wp) for l in model.model.layers]
         for L in self.layers:
             L.norm = self._pad_norm(*L.norm)
@@ -122,13 +88,13 @@ class LatentStack:
         self.final_norm = self._pad_norm(fn.weight.float(), fn.bias.float(), fn.alpha.item())
         self.runs = cfg.layer_runs()
         table = model.model.embed_tokens.weight
-        self.table = table if self.wp == self.width else _pad(table, table.shape[0], self.wp)
+        self.table = table if self.wp == self.width else pad(table, table.shape[0], self.wp)
         self.head = self.table
         self.vocab = cfg.vocab_size
         self.loops = any(again for _, again in self.runs)
 
     def _pad_norm(self, w, b, alpha):
-        p = lambda v: _pad(v.view(1, -1), 1, self.wp).view(-1)
+        p = lambda v: pad(v.view(1, -1), 1, self.wp).view(-1)
         return p(w), p(b), alpha
 
     @staticmethod
@@ -154,15 +120,6 @@ class LatentStack:
             return cols[key]
         b.get = get
         return b
-
-    def _attn_ws(self, st, splits: int, rows: int, rp: int):
-        if splits == 1:
-            return None
-        key = (splits, rows, rp)
-        if key not in st.ws:
-            st.ws[key] = {"o": torch.zeros(splits, rows, rp, dtype=torch.float32, device=self.device),
-                          "ml": torch.zeros(splits, rows, 2, dtype=torch.float32, device=self.device)}
-        return st.ws[key]
 
     # ------------------------------------------------------------------ one forward
     def run(self, st, ids, pools, batch, xn, taps=None, tap_ids=None, pdl: bool = True) -> int:
@@ -209,23 +166,21 @@ class LatentStack:
 
     def _layer(self, st, L, pool, batch, norm, h, emb, tapped, pdl) -> int:
         lib, p, s = X.load(), X._p, X._stream
-        T, H = st.T, L.heads
+        T, mix = st.T, L.mix
         raw, cat = st.get("raw", L.n_raw, torch.float32), st.get("cat", L.cat_cols)
-        act = cat[:, H * L.vp:] if L.act_cols else None
+        act = cat[:, mix.out_cols:] if L.act_cols else None
         X.gemm_inproj(st.h, L.w_in, raw, L.n_raw, act, L.gelu, pdl=pdl)
         n = 1
         pending = []
         if L.moe is not None:
             pending, launched = self._experts(st, L, raw, act, pdl)
             n += launched
-        cq, q = st.get("cq", L.qp), st.get("q", H * L.dp)
+        cq, q = st.get("cq", L.qp), st.get("q", mix.cfg.heads * mix.dp)
         X._check(lib.js_latent_post(p(raw), L.n_raw, L.q_rank, L.kv_rank, p(L.q_norm), p(L.kv_norm), X.ctypes.c_float(L.eps), p(cq),
-                                    L.qp, p(pool), L.rp, pool.shape[0], p(batch.slots), T, p(X.status_word(self.device)),
+                                    L.qp, p(pool), mix.rp, pool.shape[0], p(batch.slots), T, p(X.status_word(self.device)),
                                     int(pdl), s()), "js_latent_post")
         X.gemm(cq, L.uq, out=q, pdl=pdl)
-        n += 2
-        for part in batch.parts:
-            n += (self._expanded if part.expand and L.expand else self._absorbed)(st, L, pool, batch, part, q, cat, pdl)
+        n += 2 + mix.attend(st, pool, batch, q, cat, None, pdl)
         # the norm rides on the output GEMM unless a kernel still has to add to the stream (experts) or read it (taps)
         fused = not pending and not tapped
         X.gemm_resid32(cat, L.w_out, st.x, norm=norm if fused else None, h=h if fused else None, emb=emb if fused else None, pdl=pdl)
@@ -234,30 +189,6 @@ class LatentStack:
             self._combine(st, moe, None if tapped else emb, None if tapped else norm, h, pdl)
             n += 1
         return n
-
-    def _absorbed(self, st, L, pool, batch, part, q, cat, pdl) -> int:
-        r0, r1, H = part.r0, part.r1, L.heads
-        T = r1 - r0
-        qa, ol = st.get("qa", H * L.rp)[r0:r1], st.get("ol", H * L.rp)[r0:r1]
-        X.gemm_batched(q[r0:r1], L.uk_t, qa, H, L.rp, L.dp, L.dp, L.rp, H * L.rp, pdl=pdl)
-        rows = T * H
-        tc = L.rp <= X.LATENT_TC_MAX and (batch.mask is None or batch.mask.shape[1] <= 8)
-        splits = X.latent_attn_splits(T, H, part.seqs, part.max_q, L.rp, part.max_keys) if tc else 1
-        X.latent_attention_rows(qa.view(rows, L.rp), pool, H, batch.slot_map, part.seq_rows, part.cu_q, part.past,
-                                None if batch.mask is None else batch.mask[r0:r1], L.scale, batch.causal, part.max_q,
-                                out=ol.view(rows, L.rp), splits=splits, ws=self._attn_ws(st, splits, rows, L.rp), pdl=pdl,
-                                impl="tc" if tc else "simt")
-        X.gemm_batched(ol, L.uv, cat[r0:r1], H, L.vp, L.rp, L.rp, L.vp, cat.stride(0), pdl=pdl)
-        return 4 if splits > 1 else 3
-
-    def _expanded(self, st, L, pool, batch, part, q, cat, pdl) -> int:
-        r0, r1, H, keys = part.r0, part.r1, L.heads, part.keys
-        c, kv = st.get("c", L.rp, rows=keys), st.get("kv", H * 256, rows=keys)
-        X.gather_rows(pool, part.key_slots, c, pdl=pdl)
-        X.gemm(c, L.ukv, out=kv, pdl=pdl)
-        X.paged_attention_rows(q[r0:r1].view(r1 - r0, H, 128), kv[:, : H * 128], kv[:, H * 128:], part.key_map, part.key_base, part.cu_q,
-                               part.past, L.scale, part.max_q, cat[r0:r1], part.max_keys, pdl=pdl)
-        return 3
 
     def _experts(self, st, L, raw, act, pdl):
         """Route, sort by expert, run the two grouped GEMMs; the weighted rows stay behind for :meth:`_combine`."""
@@ -286,38 +217,44 @@ class LatentStack:
         return pending, n
 
     # ------------------------------------------------------------------ batches
-    @staticmethod
-    def part(r0, r1, seq_rows, cu_q, past, max_q, max_keys, expand=False, **kw):
-        """A group of consecutive sequences of a batch: rows ``[r0, r1)``, ``cu_q`` counted from ``r0``."""
-        return types.SimpleNamespace(r0=r0, r1=r1, seq_rows=seq_rows, cu_q=cu_q, past=past, max_q=max_q, max_keys=max_keys,
-                                     seqs=int(seq_rows.numel()), expand=expand, **kw)
-
     def uniform_batch(self, slot_map, seq_rows, cu_q, past, slots, mask, causal, rows, max_q, max_keys, positions=None,
                       state_rows=None):
         """A batch whose sequences all take the absorbed form (decode steps and token trees)."""
-        return types.SimpleNamespace(slot_map=slot_map, slots=slots, mask=mask, causal=causal,
-                                     parts=[self.part(0, rows, seq_rows, cu_q, past, max_q, max_keys)])
+        return types.SimpleNamespace(slot_map=slot_map, slots=slots, mask=None if causal else mask,
+                                     parts=[latent_part(0, rows, seq_rows, cu_q, past, max_q, max_keys)])
 
     def ragged_batch(self, slot_map, meta, counts, past_lens):
-        """Portions and decoded tokens: short ones absorbed, and (where every sequence behind the first long portion is
-        long too) the long ones expanded."""
-        dev, B = self.device, len(counts)
-        k = B
-        if meta.causal and any(L.expand for L in self.layers):
-            while k > 0 and counts[k - 1] >= EXPAND_MIN_TOKENS:
-                k -= 1
-        r_split = sum(counts[:k])
-        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
-        parts = []
-        if k > 0:
-            parts.append(self.part(0, r_split, meta.seq_rows[:k], meta.cu_q[: k + 1], meta.past_lens[:k], max(counts[:k]),
-                                   max(a + b for a, b in zip(counts[:k], past_lens[:k]))))
-        if k < B:
-            lens = [a + b for a, b in zip(counts[k:], past_lens[k:])]
-            base = [sum(lens[:j]) for j in range(len(lens))]
-            rows = meta.seq_rows[k:]
-            key_slots = torch.cat([slot_map[rows[j].long(), :n] for j, n in enumerate(lens)])
-            parts.append(self.part(r_split, sum(counts), rows, (meta.cu_q[k:] - meta.cu_q[k]).contiguous(), meta.past_lens[k:],
-                                   max(counts[k:]), max(lens), expand=True, keys=sum(lens), key_slots=key_slots,
-                                   key_base=i32(base), key_map=torch.arange(sum(lens), dtype=torch.int32, device=dev).view(-1, 1)))
-        return types.SimpleNamespace(slot_map=slot_map, slots=meta.slots, mask=meta.mask_bits, causal=meta.causal, parts=parts)
+        """Portions and decoded tokens, or token trees."""
+        return types.SimpleNamespace(slot_map=slot_map, slots=meta.slots, mask=None if meta.causal else meta.mask_bits,
+                                     parts=latent_parts(slot_map, meta, counts, past_lens, any(L.mix.expand for L in self.layers)))
+
+
+def latent_part(r0, r1, seq_rows, cu_q, past, max_q, max_keys, expand=False, **kw):
+    """A group of consecutive sequences of a batch: rows ``[r0, r1)``, ``cu_q`` counted from ``r0``."""
+    return types.SimpleNamespace(r0=r0, r1=r1, seq_rows=seq_rows, cu_q=cu_q, past=past, max_q=max_q, max_keys=max_keys,
+                                 seqs=int(seq_rows.numel()), expand=expand, **kw)
+
+
+def latent_parts(slot_map, meta, counts, past_lens, may_expand: bool) -> list:
+    """Sequence groups of a ragged batch in row order: short portions absorbed, and (where every sequence behind the first long
+    portion is long too) the long ones expanded."""
+    dev, B = slot_map.device, len(counts)
+    k = B
+    if meta.causal and may_expand:
+        while k > 0 and counts[k - 1] >= EXPAND_MIN_TOKENS:
+            k -= 1
+    r_split = sum(counts[:k])
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    parts = []
+    if k > 0:
+        parts.append(latent_part(0, r_split, meta.seq_rows[:k], meta.cu_q[: k + 1], meta.past_lens[:k], max(counts[:k]),
+                                 max(a + b for a, b in zip(counts[:k], past_lens[:k]))))
+    if k < B:
+        lens = [a + b for a, b in zip(counts[k:], past_lens[k:])]
+        base = [sum(lens[:j]) for j in range(len(lens))]
+        rows = meta.seq_rows[k:]
+        key_slots = torch.cat([slot_map[rows[j].long(), :n] for j, n in enumerate(lens)])
+        parts.append(latent_part(r_split, sum(counts), rows, (meta.cu_q[k:] - meta.cu_q[k]).contiguous(), meta.past_lens[k:],
+                                 max(counts[k:]), max(lens), expand=True, keys=sum(lens), key_slots=key_slots,
+                                 key_base=i32(base), key_map=torch.arange(sum(lens), dtype=torch.int32, device=dev).view(-1, 1)))
+    return parts

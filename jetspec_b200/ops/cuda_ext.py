@@ -1194,6 +1194,85 @@ def retention(q, k, v, cfg, state, rows, cu_q, past_lens, mask_bits, causal: boo
     return retention_seq(q, k, v, cfg, state, rows, cu_q, past_lens, None if causal else mask_bits)
 
 
+RETENTION_CHUNK = 128
+
+
+def retention_powers(cfg, device) -> torch.Tensor:
+    """Powers 0 .. 256 of the heads' decays ``(H, 257)``, evaluated in double and rounded to fp32 once."""
+    key = ("powers", tuple(cfg.decay), str(device))
+    if key not in _decays:
+        _decays[key] = torch.tensor([[d ** j for j in range(257)] for d in cfg.decay], dtype=torch.float64).float().to(device)
+    return _decays[key]
+
+
+def retention_fused_ok(cfg) -> bool:
+    """Whether the chunk and tree kernels take this shape (the step kernel and the row walk take dims up to 256)."""
+    return cfg.dim <= 128 and cfg.vdim <= 256
+
+
+def _retention_args(cfg, act, cols, rot, powers, state=None) -> tuple:
+    """The arguments all retention kernels start with.  ``cols``: where k, v and the gate start in ``act``; ``rot``: the layer's
+    columns ``(T, >= dims / 2, 2)`` of the rotary table."""
+    assert act.dtype == torch.bfloat16 and act.stride(1) == 1 and rot.dtype == torch.float32 and rot.stride(2) == 1 and rot.stride(1) == 2
+    assert act.shape[1] >= cols[2] + cfg.heads * cfg.vdim and rot.shape[0] >= act.shape[0] and rot.shape[1] >= cfg.rot.dims // 2
+    assert state is None or (state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (cfg.heads, cfg.dim, cfg.vdim))
+    return (cfg.heads, cfg.dim, cfg.vdim, cfg.rot.dims, _p(act), act.stride(0), *cols, _p(rot), rot.stride(0) // 2, _p(powers))
+
+
+def retention_rows_buffers(T: int, cfg, device) -> dict:
+    """Rotated fp32 rows and read-outs of the row-by-row walk."""
+    f = lambda n: torch.empty(T, cfg.heads * n, dtype=torch.float32, device=device)
+    return {"q": f(cfg.dim), "k": f(cfg.dim), "v": f(cfg.vdim), "o": torch.empty(T, cfg.heads, cfg.vdim, dtype=torch.float32, device=device)}
+
+
+def retention_chunk_buffer(T: int, B: int, cfg, device) -> torch.Tensor:
+    """States before every chunk of a portion's rows."""
+    return torch.empty(T // RETENTION_CHUNK + B, cfg.heads, cfg.dim, cfg.vdim, dtype=torch.float32, device=device)
+
+
+def retention_forward(cfg, act, cols, rot, state, rows, cu_q, past_lens, mask_bits, eps: float, out, max_rows: int, buffers=None,
+                      pdl: bool = False) -> int:
+    """Everything between a retention layer's projections ``act`` (bf16, q | k | v | gate) and its output product: rotations,
+    the recurrence, per-head norm and silu gate to ``out``.  One kernel for decode steps (one row a sequence) and for token
+    trees (``mask_bits``; nothing is stored), three for portions; row by row for shapes these do not take.
+    ``buffers(kind)`` hands out the workspace of ``"chunks"`` or ``"rows"``.  Returns the number of kernels launched."""
+    lib = load()
+    T, B = act.shape[0], rows.numel()
+    get = buffers or (lambda k: (retention_chunk_buffer if k == "chunks" else lambda t, b, c, d: retention_rows_buffers(t, c, d))(T, B, cfg, act.device))
+    assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and out.shape[1] >= cfg.heads * cfg.vdim
+    args = _retention_args(cfg, act, cols, rot, retention_powers(cfg, act.device), state)
+    seqs = (_p(rows), _p(cu_q), _p(past_lens), B)
+    if mask_bits is None and max_rows == 1 and T == B and cfg.vdim <= 1024:
+        cl = 1               # CTAs a head's value columns are dealt to: enough to fill the device, at least 32 columns each
+        while cl < 8 and (cfg.vdim > 256 * cl or (cfg.vdim >= 64 * cl and B * cfg.heads * cl < 2 * SM_COUNT)):
+            cl *= 2
+        _check(lib.js_retention_step(*args, *seqs, _p(state), ctypes.c_float(eps), _p(out), out.stride(0), cl, int(pdl), _stream()),
+               "js_retention_step")
+        return 1
+    if retention_fused_ok(cfg) and mask_bits is None:
+        U = get("chunks")
+        assert U.shape[0] >= T // RETENTION_CHUNK + B
+        _check(lib.js_retention_chunks(*args, *seqs, T, _p(state), _p(U), ctypes.c_float(eps), _p(out), out.stride(0), int(pdl), _stream()),
+               "js_retention_chunks")
+        return 3
+    if retention_fused_ok(cfg) and mask_bits.shape[1] <= 8:
+        _check(lib.js_retention_tree(*args, *seqs, T, _p(state), _p(mask_bits), mask_bits.shape[1], ctypes.c_float(eps), _p(out), out.stride(0),
+                                     int(pdl), _stream()), "js_retention_tree")
+        return 1
+    w = get("rows")
+    _check(lib.js_retention_prep(*args[:-1], T, _p(w["q"]), _p(w["k"]), _p(w["v"]), int(pdl), _stream()), "js_retention_prep")
+    retention_seq(w["q"], w["k"], w["v"], cfg, state, rows, cu_q, past_lens, mask_bits, out=w["o"], pdl=pdl)
+    gated_head_norm(w["o"], None, act[:, cols[2]:cols[2] + cfg.heads * cfg.vdim], "silu", eps, out=out, pdl=pdl)
+    return 3
+
+
+def retention_path(cfg, act, cols, rot, state, rows, cu_q, past_lens, path, path_len, pdl: bool = False) -> None:
+    """Advance one sequence's state along the rows ``path[:path_len]`` of a tree forward; ``past_lens`` is the committed length
+    behind the path."""
+    _check(load().js_retention_path(*_retention_args(cfg, act, cols, rot, retention_powers(cfg, act.device), state), _p(rows), _p(cu_q),
+                                    _p(past_lens), _p(state), _p(path), _p(path_len), int(pdl), _stream()), "js_retention_path")
+
+
 # ------------------------------------------------------------------ MoE (grouped through the dense GEMM)
 _moe_cache: dict = {}
 
