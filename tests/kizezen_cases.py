@@ -58,7 +58,7 @@ def cases():
                                   (latent(5, 12, 20, 40, rot(8, 1e3, **ramp(4, 64, 8, 1))), 88),
                                   (window(4, 4, 16, 16, 29, 0, rot(16, 500), scale=0.4), 0),
                                   (retention(20, 12, [1.0, 0.3, 0.75, 0.97], rot(20, 1e4)), 0),
-                                  (latent(3, 16, 12, 24, rot(6, 1e4), scale=0.5), 40)], eps=1e-3, embed=0.7, logit=1.7),
+                                  (latent(3, 16, 12, 24, rot(6, 1e4), scale=0.15), 40)], eps=1e-3, embed=0.7, logit=1.7),
         # a window of one token, one head, more kept tokens than the window holds
         "one": config(64, 90, [(window(1, 1, 8, 24, 1, 9, rot(2, 1e4)), 16), (latent(1, 8, 8, 8, rot(2, 1e4, **ramp(2, 32, 4, 1))), 24),
                                (retention(8, 8, [0.8], rot(2, 1e4)), 16)], embed=3.0, logit=0.3),

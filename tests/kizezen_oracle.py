@@ -213,8 +213,8 @@ def random_weights(cfg, seed=0, dtype=torch.float64):
             vec(p + ".mix.q.norm", H * D, 1.5, 0.3)
             vec(p + ".mix.k.norm", m["kv_heads"] * D, 1.5, 0.3)
         elif L["type"] == "latent_attention":
-            mat(p + ".mix.q", H * (D + m["rot_dim"]), W, std=1.5 / math.sqrt(W))
-            mat(p + ".mix.dkv", m["kv_rank"] + m["rot_dim"], W, std=1.5 / math.sqrt(W))
+            mat(p + ".mix.q", H * (D + m["rot_dim"]), W)
+            mat(p + ".mix.dkv", m["kv_rank"] + m["rot_dim"], W)
             vec(p + ".mix.dkv.norm", m["kv_rank"], 1.0, 0.2)
             mat(p + ".mix.uk", H * D, m["kv_rank"])
             mat(p + ".mix.uv", H * E, m["kv_rank"])
