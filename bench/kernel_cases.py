@@ -4,6 +4,8 @@
     python bench/kernel_cases.py gemm_rows2048   # the same shapes at 2048 rows (batched verify / prefill tiles)
     python bench/kernel_cases.py attention   # paged tree attention, 128 nodes over a 1.5k-token prefix
     python bench/kernel_cases.py latent_attention # latent attention: 16 requests, one token x 32 heads, 2k cached rows of 512
+    python bench/kernel_cases.py delta_rule  # a prompt portion through the block form of the gated delta rule
+    python bench/kernel_cases.py retention   # a prompt portion of 2048 rows through the chunk form of the retention, 16 heads of 128 x 256
     python bench/kernel_cases.py parallel_block   # input / output GEMMs of a parallel block at 128 rows (fused epilogues)
     python bench/kernel_cases.py lm_head     # vocabulary GEMM with the argmax epilogue
     python bench/kernel_cases.py nvfp4       # activation quantiser + block-scaled GEMM on the same four shapes
@@ -137,6 +139,18 @@ def case_delta_rule(reps: int = 3):
     torch.cuda.synchronize()
 
 
+def case_retention(reps: int = 3):
+    """A prompt portion of 2048 rows through the chunk form of the retention, 16 heads of 128 x 256."""
+    from jetspec_b200.models import RetentionConfig, RotaryConfig
+    T, c = 2048, RetentionConfig(16, 128, 256, [1.0 - 2.0 ** (-5 - i / 2) for i in range(16)], RotaryConfig(128, 1e4))
+    i32 = dict(dtype=torch.int32, device="cuda")
+    act, table, state, out = bf(T, 12288), torch.randn(T, 64, 2, device="cuda"), torch.zeros(2, 16, 128, 256, device="cuda"), bf(T, 4096)
+    rows, cu, past = torch.zeros(1, **i32), torch.tensor([0, T], **i32), torch.zeros(1, **i32)
+    for _ in range(reps):
+        X.retention_forward(c, act, (2048, 4096, 8192), table, state, rows, cu, past, None, 1e-5, out, T)
+    torch.cuda.synchronize()
+
+
 def case_round_small(reps: int = 2):
     """The small kernels of a decode round at Qwen3-8B sizes: RMSNorm, per-head norm + RoPE + KV scatter, the
     draft head's vocabulary top-k (GEMM epilogue + merge), device tree build, accept + commit, KV compaction."""
@@ -225,7 +239,7 @@ def case_collectives(reps: int = 3):
 if __name__ == "__main__":
     X.load()
     {"gemm": case_gemm, "gemm_rows2048": case_gemm_rows2048, "lm_head": case_lm_head, "attention": case_attention,
-     "latent_attention": case_latent_attention, "delta_rule": case_delta_rule, "parallel_block": case_parallel_block, "nvfp4": case_nvfp4,
+     "latent_attention": case_latent_attention, "delta_rule": case_delta_rule, "retention": case_retention, "parallel_block": case_parallel_block, "nvfp4": case_nvfp4,
      "round_small": case_round_small, "collectives": case_collectives}[sys.argv[1]]()
     X.check_status("cuda")
     print("ok")

@@ -80,10 +80,10 @@ def throughput(name, cfg, prompt=2048, context=2048, batches=(1, 16)):
     out = {"model": name, "family": cfg.model_type, "layer_runs": cfg.num_hidden_layers, "cache_bytes_per_token": 0}
     eng._ensure_pool((max(prompt, context) + 48) * max(batches), seqs=max(batches))
     pool, fast = eng.pool, FastRound.get(eng)
-    bufs = (pool.latent_pools if pool.latent_pools is not None else [b for kv in pool.kv_layers if kv is not None for b in kv]
-            if pool.kv_layers is not None else [pool.k_pool, pool.v_pool])
+    bufs = [b for b in pool.latent_pools or [] if b is not None] + [b for kv in pool.kv_layers or [] if kv is not None for b in kv]
+    bufs = bufs or [pool.k_pool, pool.v_pool]
     if pool.states is not None:
-        out["state_bytes_per_sequence"] = sum(t[0].numel() * t.element_size() for t in (*pool.states.state, *pool.states.conv))
+        out["state_bytes_per_sequence"] = sum(t[0].numel() * t.element_size() for t in (*pool.states.state, *pool.states.conv) if t is not None)
     out["cache_bytes_per_token"] = sum(b.numel() * b.element_size() for b in bufs) // pool.num_slots
     ids = torch.randint(0, cfg.vocab_size, (1, prompt), generator=torch.Generator().manual_seed(0)).cuda()
 
