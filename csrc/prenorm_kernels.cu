@@ -257,6 +257,132 @@ __global__ void __launch_bounds__(kPostThreads) attn_post_kernel(AttnPostParams 
   }
 }
 
+// The same with a token's q, k and v in one CTA and everything between load and store in registers.  An item is a group of
+// rotated entries ("half": 2 + 2 of them, "next": 2), 2 that pass, or 2 of padding.  Needs even D, V and widths, an even n
+// for "half", and at most kPostItems items of q and half as many of k a thread.
+constexpr int kPostItems = 4;
+
+struct PostItem {
+  float2 a, b;             // b: the partners of a rotated "half" group
+  float4 cs;               // (cos, sin) of one pair ("next") or two ("half")
+  int head, e, kind;       // first entry; 0 nothing, 1 rotated "half", 2 rotated "next", 3 passes, 4 padding
+};
+
+// quotient of small non-negative integers by a divisor whose reciprocal is given
+JS_DEVICE int small_div(int x, float inv) { return static_cast<int>((x + 0.5f) * inv); }
+
+JS_DEVICE PostItem post_load(const AttnPostParams& p, const __nv_bfloat16* row, const float2* rot, int c0, const float* w, int heads, int width,
+                             float inv_per, int idx, float& ss) {
+  PostItem it{};
+  const int n = p.n, groups = p.next ? n : n / 2, per = groups + (width - 2 * n) / 2;
+  if (idx >= heads * per) return it;
+  it.head = small_div(idx, inv_per);
+  const int g = idx - it.head * per;
+  it.kind = g < groups ? (p.next ? 2 : 1) : 2 * n + 2 * (g - groups) < p.D ? 3 : 4;
+  it.e = g < groups ? 2 * g : 2 * n + 2 * (g - groups);
+  if (it.kind == 4) return it;
+  auto load = [&](int c) {
+    float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + c0 + c));
+    if (p.bias != nullptr) {
+      const float2 b = *reinterpret_cast<const float2*>(p.bias + c0 + c);
+      v.x += b.x;
+      v.y += b.y;
+    }
+    ss += v.x * v.x + v.y * v.y;
+    if (w != nullptr) {
+      const float2 g2 = *reinterpret_cast<const float2*>(w + c);
+      v.x *= g2.x;
+      v.y *= g2.y;
+    }
+    return v;
+  };
+  if (it.kind == 1) it.cs = *reinterpret_cast<const float4*>(rot + it.e);
+  if (it.kind == 2) {
+    const float2 c = rot[it.e >> 1];
+    it.cs = make_float4(c.x, c.y, 0.f, 0.f);
+  }
+  it.a = load(it.head * p.D + it.e);
+  if (it.kind == 1) it.b = load(it.head * p.D + it.e + n);
+  return it;
+}
+
+JS_DEVICE void post_store(const AttnPostParams& p, const PostItem& it, float r, __nv_bfloat16* dst) {
+  if (it.kind == 0) return;
+  float2 a = it.a;
+  const float4 cs = it.cs;
+  if (it.kind == 1) {
+    a = make_float2(it.a.x * cs.x - it.b.x * cs.y, it.a.y * cs.z - it.b.y * cs.w);
+    const float2 b = make_float2(it.b.x * cs.x + it.a.x * cs.y, it.b.y * cs.z + it.a.y * cs.w);
+    *reinterpret_cast<__nv_bfloat162*>(dst + it.e + p.n) = __floats2bfloat162_rn(b.x * r, b.y * r);
+  } else if (it.kind == 2) {
+    a = make_float2(it.a.x * cs.x - it.a.y * cs.y, it.a.y * cs.x + it.a.x * cs.y);
+  }
+  *reinterpret_cast<__nv_bfloat162*>(dst + it.e) = __floats2bfloat162_rn(a.x * r, a.y * r);
+}
+
+template <int QI>
+__global__ void __launch_bounds__(kPostThreads, QI <= 2 ? 2 : 1)
+attn_post_vec_kernel(AttnPostParams p, float inv_q, float inv_k, float inv_v, float inv_group) {
+  constexpr int KI = QI > 1 ? QI / 2 : 1, NW = kPostThreads / 32;
+  __shared__ float red[2 * NW];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31;
+  const __nv_bfloat16* row = p.proj + static_cast<size_t>(t) * p.ldp;
+  const float2* rot = p.rot + static_cast<size_t>(t) * p.ldr;
+  const int slot = p.slots[t], kc = p.H * p.D, vc = kc + p.G * p.D;
+  PostItem q[QI], k[KI];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int j = 0; j < QI; ++j) q[j] = post_load(p, row, rot, 0, p.qw, p.H, p.Dq, inv_q, tid + j * kPostThreads, sq);
+#pragma unroll
+  for (int j = 0; j < KI; ++j) k[j] = post_load(p, row, rot, kc, p.kw, p.G, p.Dp, inv_k, tid + j * kPostThreads, sk);
+  const bool ok = slot >= 0 && slot < p.S;
+  if (!ok && tid == 0) report(p.status, kBadSlot);
+  if (ok) {
+    const int half = p.Vp / 2;
+    for (int i = tid; i < p.G * half; i += kPostThreads) {
+      const int g = small_div(i, inv_v), d = 2 * (i - g * half), c = vc + g * p.V + d;
+      float2 v = make_float2(0.f, 0.f);
+      if (d < p.V) {
+        v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + c));
+        if (p.bias != nullptr) {
+          const float2 b = *reinterpret_cast<const float2*>(p.bias + c);
+          v.x += b.x;
+          v.y += b.y;
+        }
+      }
+      *reinterpret_cast<__nv_bfloat162*>(p.vpool + (static_cast<size_t>(g) * p.S + slot) * p.Vp + d) = __floats2bfloat162_rn(v.x, v.y);
+    }
+  }
+  float rq = 1.f, rk = 1.f;
+  if (p.qw != nullptr) {
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { red[tid >> 5] = sq; red[NW + (tid >> 5)] = sk; }
+    __syncthreads();
+    static_assert(NW == 16, "one load a lane: q's sums in the lower half of the warp, k's in the upper");
+    float s = red[lane];
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+    rq = 1.f / sqrtf(__shfl_sync(0xffffffffu, s, 0) / (p.H * p.D) + p.eps);
+    rk = 1.f / sqrtf(__shfl_sync(0xffffffffu, s, 16) / (p.G * p.D) + p.eps);
+  }
+  const int group = p.H / p.G;
+#pragma unroll
+  for (int j = 0; j < QI; ++j) {
+    int hp = q[j].head;
+    if (p.Gp != group) {
+      const int g = small_div(hp, inv_group);
+      hp = g * p.Gp + hp - g * group;
+    }
+    post_store(p, q[j], rq, p.qout + (static_cast<size_t>(t) * p.G * p.Gp + hp) * p.Dq);
+  }
+  if (!ok) return;
+#pragma unroll
+  for (int j = 0; j < KI; ++j) post_store(p, k[j], rk, p.kpool + (static_cast<size_t>(k[j].head) * p.S + slot) * p.Dp);
+}
+
 // ---------------------------------------------------------------- behind the input projections of a latent attention
 // grid y: 0 = the cache row: raw (T, ldw) fp32 [latent | rotated key part] -> [latent / rms * w | rotated | zeros] at the token's pool
 // row; 1 = the rotated part of every query head, in place: q (T, ldq) with heads dq apart, entries [dim, dim + 2n).
@@ -382,6 +508,16 @@ extern "C" int js_attn_post(const void* proj, int ldp, const float* bias, const 
   if (H < 1 || G < 1 || H % G || Gp < H / G || D > Dq || D > Dp || V > Vp || dims > D || (dims & 1) || ldr < dims / 2 || H * D > 24576) return -10;
   AttnPostParams p{(const bf*)proj, bias, qw, kw, (const float2*)rot, slots, (bf*)qout, (bf*)kpool, (bf*)vpool, status,
                    ldp, H, G, Gp, D, V, Dq, Dp, Vp, dims / 2, next, ldr, S, eps};
+  const int n = dims / 2, rot_items = next ? n : n / 2;
+  const bool even = !((D | V | Dq | Dp | Vp | ldp | ldr) & 1) && (next || !(n & 1)) && !(reinterpret_cast<uintptr_t>(rot) & 15) && (qw == nullptr) == (kw == nullptr);
+  const int qi = H * (rot_items + (Dq - 2 * n) / 2), ki = G * (rot_items + (Dp - 2 * n) / 2);
+  auto fits = [&](int items) { return qi <= items * kPostThreads && ki <= (items > 1 ? items / 2 : 1) * kPostThreads; };
+  if (even && fits(kPostItems)) {
+    PrenormLaunch l(dim3(T), dim3(kPostThreads), stream, pdl);
+    auto kern = fits(1) ? attn_post_vec_kernel<1> : fits(2) ? attn_post_vec_kernel<2> : attn_post_vec_kernel<kPostItems>;
+    auto inv = [](int x) { return x > 0 ? 1.f / static_cast<float>(x) : 0.f; };
+    return cudaLaunchKernelEx(&l.c, kern, p, inv(qi / H), inv(ki / G), inv(Vp / 2), inv(H / G)) == cudaSuccess ? 0 : -4;
+  }
   const int smem = H * D * 4;
   static int configured[kMaxDevicesCached] = {};
   if (smem > 40 * 1024 && ensure_dyn_smem(attn_post_kernel, smem, configured) != 0) return -3;

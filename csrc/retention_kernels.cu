@@ -66,22 +66,83 @@ JS_DEVICE void ret_load_row(const RetIn& p, const __nv_bfloat16* src, const floa
   for (int e = 2 * n + lane; e < DP; e += 32) dst[e] = e < D ? __bfloat162float(src[e]) * scale : 0.f;
 }
 
-// 64 value rows of a head (columns [v0, v0 + VT)) to dst[row][LV], zeros where they do not exist
-template <int VT, int LV>
+JS_DEVICE void ret_cp16(void* dst, const void* src, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+JS_DEVICE void ret_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+JS_DEVICE void ret_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// The whole CTA: ROWS rows from token t0 on of the head whose columns start at col, rotated and times scale(row), to dst[row][LD];
+// rows from `rows` on are zero.  A warp takes every eighth row, four at a time, so that their loads overlap.
+template <int DP, int LD, int ROWS, typename F>
+JS_DEVICE void ret_load_rows(const RetIn& p, int col, size_t t0, int rows, F scale, float* dst) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = p.n, D = p.D, e = 2 * lane;
+  if (((n | D | p.ldp | p.ldr) & 1) != 0) {
+    for (int r = warp; r < ROWS; r += 8) {
+      const bool ok = r < rows;
+      const size_t t = t0 + (ok ? r : 0);
+      ret_load_row<DP>(p, p.act + t * p.ldp + col, p.rot + t * p.ldr, ok ? scale(r) : 0.f, ok, dst + r * LD);
+    }
+    return;
+  }
+  constexpr int BATCH = 4;
+  static_assert(DP <= 128 && ROWS % (8 * BATCH) == 0, "a lane covers a row's pairs at once");
+  for (int r0 = warp; r0 < ROWS; r0 += 8 * BATCH) {
+    uint32_t a[BATCH] = {}, b[BATCH] = {}, c[BATCH][2] = {};
+    float4 cs[BATCH];
+    float f[BATCH];
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) {
+      const int r = r0 + 8 * i;
+      const bool ok = r < rows;
+      const size_t t = t0 + (ok ? r : 0);
+      const __nv_bfloat16* src = p.act + t * p.ldp + col;
+      cs[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (ok && e < n) {
+        a[i] = *reinterpret_cast<const uint32_t*>(src + e);
+        b[i] = *reinterpret_cast<const uint32_t*>(src + e + n);
+        cs[i] = *reinterpret_cast<const float4*>(p.rot + t * p.ldr + e);
+      }
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (ok && 2 * n + e + 64 * j < D) c[i][j] = *reinterpret_cast<const uint32_t*>(src + 2 * n + e + 64 * j);
+      f[i] = ok ? scale(r) : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < BATCH; ++i) {
+      float* out = dst + (r0 + 8 * i) * LD;
+      if (e < n) {
+        const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[i])), v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&b[i]));
+        *reinterpret_cast<float2*>(out + e) = make_float2((u.x * cs[i].x - v.x * cs[i].y) * f[i], (u.y * cs[i].z - v.y * cs[i].w) * f[i]);
+        *reinterpret_cast<float2*>(out + e + n) = make_float2((v.x * cs[i].x + u.x * cs[i].y) * f[i], (v.y * cs[i].z + u.y * cs[i].w) * f[i]);
+      }
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (2 * n + e + 64 * j < DP) {       // entries past D are zero
+          const float2 u = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&c[i][j]));
+          *reinterpret_cast<float2*>(out + 2 * n + e + 64 * j) = make_float2(u.x * f[i], u.y * f[i]);
+        }
+    }
+  }
+}
+
+// ROWS value rows of a head (columns [v0, v0 + VT)) to dst[row][LV], zeros where they do not exist; the caller waits for the copies
+template <int VT, int LV, int ROWS>
 JS_DEVICE void ret_load_values(const RetIn& p, const __nv_bfloat16* src, int rows, int v0, __nv_bfloat16* dst) {
   if (((p.V | p.ldp | v0) & 7) == 0) {
-    for (int x = threadIdx.x; x < kRetTile * (VT / 8); x += kRetThreads) {
+    for (int x = threadIdx.x; x < ROWS * (VT / 8); x += kRetThreads) {
       const int r = x / (VT / 8), c = x % (VT / 8) * 8;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (r < rows && v0 + c < p.V) v = *reinterpret_cast<const uint4*>(src + static_cast<size_t>(r) * p.ldp + v0 + c);
-      *reinterpret_cast<uint4*>(dst + r * LV + c) = v;
+      const bool ok = r < rows && v0 + c < p.V;
+      ret_cp16(dst + r * LV + c, ok ? src + static_cast<size_t>(r) * p.ldp + v0 + c : src, ok);
     }
   } else {
-    for (int x = threadIdx.x; x < kRetTile * VT; x += kRetThreads) {
+    for (int x = threadIdx.x; x < ROWS * VT; x += kRetThreads) {
       const int r = x / VT, c = x % VT;
       dst[r * LV + c] = r < rows && v0 + c < p.V ? src[static_cast<size_t>(r) * p.ldp + v0 + c] : __float2bfloat16_rn(0.f);
     }
   }
+  ret_commit();
 }
 
 // sequence of a tile when sequence s starts at tile cu_q[s] / size + s
@@ -105,11 +166,11 @@ JS_DEVICE void ret_values(const __nv_bfloat16* base, uint32_t& even, uint32_t& o
 // ================================================================ U of every chunk
 // grid (chunks, H, ceil(V / VT)).  U (chunks, H, D, V) fp32.
 template <int DP, int VT>
-__global__ void __launch_bounds__(kRetThreads) retention_update_kernel(RetIn p, float* U) {
+__global__ void __launch_bounds__(kRetThreads, 2) retention_update_kernel(RetIn p, float* U) {
   constexpr int MW = DP / 16, NG = 8 / MW, NT = VT / NG / 8, LK = DP + 8, LV = VT + 16;
   extern __shared__ __align__(16) uint8_t raw[];
-  float* sK = reinterpret_cast<float*>(raw);                               // [64][LK]
-  __nv_bfloat16* sV = reinterpret_cast<__nv_bfloat16*>(sK + kRetTile * LK);    // [64][LV]
+  float* sK = reinterpret_cast<float*>(raw);                               // [128][LK]
+  __nv_bfloat16* sV = reinterpret_cast<__nv_bfloat16*>(sK + kRetChunk * LK);   // [128][LV]
   pdl_launch_dependents();
   pdl_wait();
   const int tile = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VT, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -125,34 +186,29 @@ __global__ void __launch_bounds__(kRetThreads) retention_update_kernel(RetIn p, 
   for (int t = 0; t < NT; ++t)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[t][e] = 0.f;
-  for (int k0 = 0; k0 < n; k0 += kRetTile) {
-    if (k0 > 0) __syncthreads();
-    const size_t t0 = q0 + r0 + k0;
-    for (int r = warp; r < kRetTile; r += 8) {
-      const bool ok = k0 + r < n;
-      const size_t t = t0 + (ok ? r : 0);
-      ret_load_row<DP>(p, p.act + t * p.ldp + p.kc + h * p.D, p.rot + t * p.ldr, ok ? p.k_scale * pw[n - 1 - k0 - r] : 0.f, ok, sK + r * LK);
-    }
-    ret_load_values<VT, LV>(p, p.act + t0 * p.ldp + p.vc + h * p.V, n - k0, v0, sV);
-    __syncthreads();
+  const size_t t0 = q0 + r0;
+  ret_load_values<VT, LV, kRetChunk>(p, p.act + t0 * p.ldp + p.vc + h * p.V, n, v0, sV);
+  ret_load_rows<DP, LK, kRetChunk>(p, p.kc + h * p.D, t0, n, [&](int r) { return p.k_scale * pw[n - 1 - r]; }, sK);
+  ret_wait<0>();
+  __syncthreads();
 #pragma unroll 2
-    for (int j = 0; j < kRetTile; j += 8) {
-      uint32_t ah[4], al[4];
-      tf32_split(sK[(j + qd) * LK + d0 + gr], ah[0], al[0]);
-      tf32_split(sK[(j + qd) * LK + d0 + gr + 8], ah[1], al[1]);
-      tf32_split(sK[(j + qd + 4) * LK + d0 + gr], ah[2], al[2]);
-      tf32_split(sK[(j + qd + 4) * LK + d0 + gr + 8], ah[3], al[3]);
+  for (int j = 0; j < kRetChunk; j += 8) {
+    if (j >= n) break;
+    uint32_t ah[4], al[4];
+    tf32_split(sK[(j + qd) * LK + d0 + gr], ah[0], al[0]);
+    tf32_split(sK[(j + qd) * LK + d0 + gr + 8], ah[1], al[1]);
+    tf32_split(sK[(j + qd + 4) * LK + d0 + gr], ah[2], al[2]);
+    tf32_split(sK[(j + qd + 4) * LK + d0 + gr + 8], ah[3], al[3]);
 #pragma unroll
-      for (int t = 0; t < NT; t += 2) {
-        uint32_t e0, o0, e1, o1;
-        const __nv_bfloat16* b = sV + (j + qd) * LV + c0 + 8 * t + 2 * gr;
-        ret_values(b, e0, o0);
-        ret_values(b + 4 * LV, e1, o1);
-        mma_tf32(acc[t], al, e0, e1);
-        mma_tf32(acc[t], ah, e0, e1);
-        mma_tf32(acc[t + 1], al, o0, o1);
-        mma_tf32(acc[t + 1], ah, o0, o1);
-      }
+    for (int t = 0; t < NT; t += 2) {
+      uint32_t e0, o0, e1, o1;
+      const __nv_bfloat16* b = sV + (j + qd) * LV + c0 + 8 * t + 2 * gr;
+      ret_values(b, e0, o0);
+      ret_values(b + 4 * LV, e1, o1);
+      mma_tf32(acc[t], al, e0, e1);
+      mma_tf32(acc[t], ah, e0, e1);
+      mma_tf32(acc[t + 1], al, o0, o1);
+      mma_tf32(acc[t + 1], ah, o0, o1);
     }
   }
   float* dst = U + (static_cast<size_t>(tile) * p.H + h) * p.D * p.V;
@@ -222,20 +278,20 @@ __global__ void __launch_bounds__(kRetThreads) retention_scan_kernel(RetIn p, fl
 // grid (tiles of 64 rows, H).  prefix: states before the chunks (chunks, H, D, V); with mask_bits (T, W) a token tree, whose prefix is
 // the sequence's own state (slots, H, D, V).  out (T, ldo) bf16, head h at column h * V.
 template <int DP, int VP>
-__global__ void __launch_bounds__(kRetThreads, VP >= 256 ? 2 : 3)
+__global__ void __launch_bounds__(kRetThreads, VP >= 128 ? 2 : 3)
 retention_rows_kernel(RetIn p, const float* prefix, const int* mask_bits, int W, float eps, __nv_bfloat16* out, int ldo) {
   constexpr int NT = VP / 16, LQ = DP + 4, LP = kRetTile + 4, LV = VP + 16, LS = VP + 8;
-  constexpr int SROWS = 32;              // state rows per slab
+  constexpr int SROWS = DP <= 64 && VP >= 256 ? 16 : 32;      // state rows per slab
   extern __shared__ __align__(16) uint8_t raw[];
   float* sQ = reinterpret_cast<float*>(raw);                               // [64][LQ]
   float* sK = sQ + kRetTile * LQ;                                          // [64][LQ], later the weights [64][LP]
   __nv_bfloat16* sV = reinterpret_cast<__nv_bfloat16*>(sK + kRetTile * LQ);    // [64][LV]
-  float* sS = sK;                                                          // [SROWS][LS], before the first key tile
+  float* sS = sK;                                                          // two slabs [SROWS][LS], before the first key tile
   __shared__ float spw[kRetPow], ssum[kRetTile][2];
   __shared__ unsigned smask[kRetTile][8];
   __shared__ int sdep[256];
   static_assert(LP <= LQ, "the weights fit the keys' place");
-  static_assert(SROWS * LS * 4 <= kRetTile * (LQ * 4 + LV * 2), "a slab fits the keys' and values' place");
+  static_assert(2 * SROWS * LS * 4 <= kRetTile * (LQ * 4 + LV * 2), "two slabs fit the keys' and values' place");
   pdl_launch_dependents();
   pdl_wait();
   const int tile = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -261,10 +317,23 @@ retention_rows_kernel(RetIn p, const float* prefix, const int* mask_bits, int W,
       smask[r][w] = r < n && w < W ? static_cast<unsigned>(mask_bits[static_cast<size_t>(q0 + r0 + r) * W + w]) : 0u;
     }
   }
-  for (int r = warp; r < kRetTile; r += 8) {
-    const size_t t = q0 + r0 + (r < n ? r : 0);
-    ret_load_row<DP>(p, p.act + t * p.ldp + h * D, p.rot + t * p.ldr, 1.f, r < n, sQ + r * LQ);
-  }
+  auto load_slab = [&](int d0, float* dst) {
+    if ((V & 3) == 0) {
+      for (int x = tid; x < SROWS * (VP / 4); x += kRetThreads) {
+        const int r = x / (VP / 4), c = x % (VP / 4) * 4;
+        const bool ok = d0 + r < D && c < V;
+        ret_cp16(dst + r * LS + c, ok ? S + static_cast<size_t>(d0 + r) * V + c : S, ok);
+      }
+    } else {
+      for (int x = tid; x < SROWS * VP; x += kRetThreads) {
+        const int r = x / VP, c = x % VP;
+        dst[r * LS + c] = d0 + r < D && c < V ? S[static_cast<size_t>(d0 + r) * V + c] : 0.f;
+      }
+    }
+    ret_commit();
+  };
+  if (has_state) load_slab(0, sS);
+  ret_load_rows<DP, LQ, kRetTile>(p, h * D, q0 + r0, n, [](int) { return 1.f; }, sQ);
   float acc[NT][4];
 #pragma unroll
   for (int t = 0; t < NT; ++t)
@@ -273,23 +342,16 @@ retention_rows_kernel(RetIn p, const float* prefix, const int* mask_bits, int W,
   const int cw = ch * (VP / 2);          // first value column of the warp
   // ---- the state before the chunk
   if (has_state) {
-    for (int d0 = 0; d0 < D; d0 += SROWS) {
-      __syncthreads();
-      if ((V & 3) == 0) {
-#pragma unroll 4
-        for (int x = tid; x < SROWS * (VP / 4); x += kRetThreads) {
-          const int r = x / (VP / 4), c = x % (VP / 4) * 4;
-          float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (d0 + r < D && c < V) v = *reinterpret_cast<const float4*>(S + static_cast<size_t>(d0 + r) * V + c);
-          *reinterpret_cast<float4*>(sS + r * LS + c) = v;
-        }
+    for (int d0 = 0, i = 0; d0 < D; d0 += SROWS, ++i) {
+      if (i > 0) __syncthreads();        // the slab before has been read: its place takes the next one
+      if (d0 + SROWS < D) {
+        load_slab(d0 + SROWS, sS + ((i + 1) & 1) * SROWS * LS);
+        ret_wait<1>();
       } else {
-        for (int x = tid; x < SROWS * VP; x += kRetThreads) {
-          const int r = x / VP, c = x % VP;
-          sS[r * LS + c] = d0 + r < D && c < V ? S[static_cast<size_t>(d0 + r) * V + c] : 0.f;
-        }
+        ret_wait<0>();
       }
       __syncthreads();
+      const float* slab = sS + (i & 1) * SROWS * LS;
 #pragma unroll
       for (int k = 0; k < SROWS; k += 8) {
         uint32_t ah[4], al[4];
@@ -299,8 +361,8 @@ retention_rows_kernel(RetIn p, const float* prefix, const int* mask_bits, int W,
         tf32_split(sQ[(rg + gr + 8) * LQ + d0 + k + qd + 4], ah[3], al[3]);
 #pragma unroll
         for (int t = 0; t < NT; t += 2) {
-          const float2 b0 = *reinterpret_cast<const float2*>(sS + (k + qd) * LS + cw + 8 * t + 2 * gr);
-          const float2 b1 = *reinterpret_cast<const float2*>(sS + (k + qd + 4) * LS + cw + 8 * t + 2 * gr);
+          const float2 b0 = *reinterpret_cast<const float2*>(slab + (k + qd) * LS + cw + 8 * t + 2 * gr);
+          const float2 b1 = *reinterpret_cast<const float2*>(slab + (k + qd + 4) * LS + cw + 8 * t + 2 * gr);
           uint32_t h0, l0, h1, l1;
           tf32_split(b0.x, h0, l0);
           tf32_split(b1.x, h1, l1);
@@ -327,11 +389,8 @@ retention_rows_kernel(RetIn p, const float* prefix, const int* mask_bits, int W,
   for (int k0 = first; k0 <= r0; k0 += kRetTile) {
     const int nk = min(kRetTile, n_seq - k0);
     __syncthreads();
-    for (int r = warp; r < kRetTile; r += 8) {
-      const size_t t = q0 + k0 + (r < nk ? r : 0);
-      ret_load_row<DP>(p, p.act + t * p.ldp + p.kc + h * D, p.rot + t * p.ldr, p.k_scale, r < nk, sK + r * LQ);
-    }
-    ret_load_values<VP, LV>(p, p.act + static_cast<size_t>(q0 + k0) * p.ldp + p.vc + h * V, nk, 0, sV);
+    ret_load_values<VP, LV, kRetTile>(p, p.act + static_cast<size_t>(q0 + k0) * p.ldp + p.vc + h * V, nk, 0, sV);
+    ret_load_rows<DP, LQ, kRetTile>(p, p.kc + h * D, q0 + k0, nk, [&](int) { return p.k_scale; }, sK);
     __syncthreads();
     float w[4][4];                       // the warp's 16 rows against 32 of the keys
 #pragma unroll
@@ -371,6 +430,7 @@ retention_rows_kernel(RetIn p, const float* prefix, const int* mask_bits, int W,
         }
         *reinterpret_cast<float2*>(sK + r * LP + c) = make_float2(w[t][2 * half] * f[0], w[t][2 * half + 1] * f[1]);
       }
+    ret_wait<0>();                       // the values
     __syncthreads();
 #pragma unroll 2
     for (int j = 0; j < kRetTile; j += 8) {
@@ -617,7 +677,7 @@ static bool ret_aligned(const void* act, const void* rot) { return !((reinterpre
 
 template <int DP, int VT>
 static int launch_update(const RetIn& p, float* U, int chunks, int pdl, cudaStream_t stream) {
-  constexpr int smem = kRetTile * ((DP + 8) * 4 + (VT + 16) * 2);
+  constexpr int smem = kRetChunk * ((DP + 8) * 4 + (VT + 16) * 2);
   static int configured[kMaxDevicesCached] = {};
   auto kern = retention_update_kernel<DP, VT>;
   if (ensure_dyn_smem(kern, smem, configured) != 0) return -3;
