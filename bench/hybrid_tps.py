@@ -95,7 +95,8 @@ def kernel_table(T, context, n_seq):
     lib, p = X.load(), X._p
     bias, wfreq, wq = torch.randn(win_cols, device=dev), X.pair_freq(64, 1e6, dev), bf(T, 16 * D)
     add("zasipel bias + rotation + norm + KV scatter", [lambda: X._check(lib.js_window_post(
-        p(act), n_act, p(bias), 16, 4, 4, D, D, D, D, D, 64, p(wfreq), 1, X.ctypes.c_float(1e-6), p(pos), p(pos), S, T, p(wq), p(kp), p(vp),
+        p(act), n_act, p(bias), 16, 4, 4, 1, D, D, D, D, D, 64, p(wfreq), 1, X.ctypes.c_float(1e-6), 0, X.ctypes.c_float(0.0), 20 * D, 1, p(pos),
+        p(pos), S, T, p(wq), p(kp), p(vp),
         p(X.status_word(dev)), 0, X._stream()), "post")], T * win_cols * 4, 0, 8, "qwen3 head norms + RoPE + KV scatter")
     seen_w = n_seq * sum(min(WIN, context + i + 1) for i in range(per))
     keys_w = n_seq * min(context + per, WIN + per - 1)

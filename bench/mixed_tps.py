@@ -182,7 +182,7 @@ def kernel_table(T, context, n_seq):
         p(x32), p(w1), X.ctypes.c_float(1e-5), p(hh), W, T, W, None, 0, 0, X._stream()), "norm")], T * W * 6, 0, 8, "qwen3 RMSNorm")
     ids, tab, fr = torch.arange(T, **i32), bf(32768, W), torch.rand(144, device=dev)
     add("kizezen embedding + norm + rotary tables", [lambda: X._check(lib.js_embed_rms(
-        p(ids), p(tab), 32768, W, X.ctypes.c_float(1.0), p(w1), X.ctypes.c_float(1e-5), p(x32), p(hh), W, T, W, p(pos), p(fr), p(fr), 144, p(table), 0,
+        p(ids), p(tab), 32768, W, X.ctypes.c_float(1.0), p(w1), X.ctypes.c_float(1e-5), p(x32), p(hh), W, T, W, p(pos), None, 0, p(fr), p(fr), 144, p(table), 0,
         X._stream()), "embed")], T * W * 8 + T * 144 * 8, 0, 8, "qwen3 RMSNorm")
     by = {r["kernel"]: r["fraction"] for r in rows}
     for r in rows:

@@ -43,7 +43,7 @@ constexpr int kTopK = 8;
 
 enum GemmEpi : int { EPI_STORE = 0, EPI_SWIGLU = 1, EPI_ARGMAX = 2, EPI_TOPK = 3, EPI_STORE_F32 = 4, EPI_ALLREDUCE = 5, EPI_EP_COMBINE = 6,
                     EPI_INPROJ = 7, EPI_RELU2 = 8, EPI_RESID32 = 9 };
-enum GemmAct : int { ACT_GELU_GLU = 0, ACT_RELU2 = 1, ACT_NONE = 2, ACT_GELU_ERF = 3 };
+enum GemmAct : int { ACT_GELU_GLU = 0, ACT_RELU2 = 1, ACT_NONE = 2, ACT_GELU_ERF = 3, ACT_XIELU = 4 };
 
 struct GemmParams {
   int M, N, K;
@@ -92,11 +92,12 @@ struct GemmParams {
   // EPI_INPROJ (fused input projections of a parallel block): columns below n_raw (a multiple of 128) are stored as
   // fp32 to C; the rest pass through `act` and go to C2 as bf16.  ACT_GELU_GLU: every 128 weight rows hold 64 gate rows
   // and the 64 up rows of the same outputs; ACT_RELU2: relu(.)^2 of each column; ACT_GELU_ERF: exact gelu of each
-  // column; ACT_NONE: as it is.
+  // column; ACT_XIELU: act_a z^2 + z / 2 for z > 0, act_b (e^z - 1 - z) + z / 2 below; ACT_NONE: as it is.
   __nv_bfloat16* C2;
   int ldc2;
   int n_raw;
   int act;
+  float act_a, act_b;
   // EPI_RESID32: C (fp32) = res32 + A W^T (+ emb); with norm_w, C2 = bf16(tanh(norm_alpha C) norm_w + norm_b), the
   // next layer's Dynamic Tanh.  res32 may be C.
   const float* res32;
@@ -700,6 +701,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             for (int j = 0; j < 32; ++j) {
               g[j] = 0.5f * g[j] * (1.f + erff(g[j] * 0.7071067811865476f));      // 1 / sqrt(2)
               u[j] = 0.5f * u[j] * (1.f + erff(u[j] * 0.7071067811865476f));
+            }
+          } else if (p.act == ACT_XIELU) {
+            auto xielu = [&](float z) { return 0.5f * z + (z > 0.f ? p.act_a * z * z : p.act_b * (__expf(z) - 1.f - z)); };
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              g[j] = xielu(g[j]);
+              u[j] = xielu(u[j]);
             }
           }
           store_bf16(out2 + nb - p.n_raw + cb, g);
@@ -1312,22 +1320,22 @@ extern "C" int js_gemm_nvfp4_allreduce(const void* Aq, const void* sfa, const fl
 }
 
 // Fused input projections of a parallel block: columns [0, n_raw) of A W^T as fp32 to C (T, ldc), the rest through `act`
-// (0: tanh-GELU gate * up, 64-row interleave; 1: relu^2; 2: none; 3: exact gelu) as bf16 to C2.  n_raw and N multiples of 128; bn 128 or 256.
+// (0: tanh-GELU gate * up, 64-row interleave; 1: relu^2; 2: none; 3: exact gelu; 4: xIELU with act_a, act_b) as bf16 to C2.  n_raw and N multiples of 128; bn 128 or 256.
 extern "C" int js_gemm_inproj(const void* A, const void* W, float* C, void* C2, int M, int N, int K, int lda, int ldw, int ldc,
-                              int ldc2, int n_raw, int act, int bn, int split, int deep, int* status, int pdl,
-                              cudaStream_t stream) {
+                              int ldc2, int n_raw, int act, float act_a, float act_b, int bn, int split, int deep, int* status,
+                              int pdl, cudaStream_t stream) {
   using namespace js;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((K % 8) || (lda % 8) || (ldw % 8)) return -10;
   if ((reinterpret_cast<uintptr_t>(A) | reinterpret_cast<uintptr_t>(W)) & 15) return -11;
   if (split < 1 || split > 4 || split > (K + BK - 1) / BK || (bn != 128 && split != 1)) return -12;
-  if ((N % 128) || (n_raw % 128) || n_raw < 0 || n_raw > N || (ldc % 4) || (ldc2 % 8) || act < 0 || act > 3) return -15;
+  if ((N % 128) || (n_raw % 128) || n_raw < 0 || n_raw > N || (ldc % 4) || (ldc2 % 8) || act < 0 || act > 4) return -15;
   if ((n_raw > 0 && (C == nullptr || ldc < n_raw)) || (n_raw < N && C2 == nullptr)) return -22;
   CUtensorMap ta, tw;
   if (make_map(&ta, A, M, K, lda, BM) || make_map(&tw, W, N, K, ldw, bn)) return -16;
   GemmParams p{};
   p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.C = C; p.status = status; p.world = 1;
-  p.C2 = reinterpret_cast<__nv_bfloat16*>(C2); p.ldc2 = ldc2; p.n_raw = n_raw; p.act = act;
+  p.C2 = reinterpret_cast<__nv_bfloat16*>(C2); p.ldc2 = ldc2; p.n_raw = n_raw; p.act = act; p.act_a = act_a; p.act_b = act_b;
   if (bn == 128)
     return deep == 1   ? launch_gemm<128, EPI_INPROJ, 192>(ta, tw, p, split, pdl != 0, stream)
            : deep == 2 ? launch_gemm<128, EPI_INPROJ, 128>(ta, tw, p, split, pdl != 0, stream)

@@ -56,7 +56,7 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(const float* x, int ld
 // square, store `width` entries (zeros past D).  Lane l holds the pairs l, l + 32, ...
 template <typename E, typename EB>
 JS_DEVICE void head_rotate_norm(const E* src, const EB* bias, E* dst, int D, int width, int dims, const float* freq, float pos,
-                                bool norm, float eps) {
+                                bool norm, float eps, float factor = 1.f) {
   constexpr int NP = 8;                // up to 512 entries
   const int lane = threadIdx.x & 31;
   float a[NP], b[NP], ss = 0.f;
@@ -75,7 +75,7 @@ JS_DEVICE void head_rotate_norm(const E* src, const EB* bias, E* dst, int D, int
     }
     ss += a[i] * a[i] + b[i] * b[i];
   }
-  const float r = norm ? 1.f / sqrtf(warp_sum(ss) / D + eps) : 1.f;
+  const float r = (norm ? 1.f / sqrtf(warp_sum(ss) / D + eps) : 1.f) * factor;
 #pragma unroll
   for (int i = 0; i < NP; ++i) {
     const int e = 2 * (lane + 32 * i);
@@ -93,147 +93,302 @@ rotate_norm_kernel(const E* x, E* out, const int* positions, int T, int heads, i
                          static_cast<float>(positions[u / heads]), norm != 0, eps);
 }
 
-// ---------------------------------------------------------------- fused: biases, rotation, norm, cache scatter
-// proj (T, ldp): [q heads | k heads | v heads]; q goes to qout (T, G, Gp, Dq) (each group of H/G heads padded to Gp heads,
-// which stay zero), k and v to their pool rows (G, S, Dp) and (G, S, Vp).
-__global__ void __launch_bounds__(256)
-window_post_kernel(const __nv_bfloat16* proj, int ldp, const float* bias, int H, int G, int Gp, int D, int V, int Dq, int Dp, int Vp, int dims,
-                   const float* freq, int norm, float eps, const int* positions, const int* slots, int S, __nv_bfloat16* qout,
-                   __nv_bfloat16* kpool, __nv_bfloat16* vpool, int* status) {
+// ---------------------------------------------------------------- fused: biases, rotation, norm, temperature, cache scatter
+// proj (T, ldp): [q heads | k heads | v heads]; q goes to qout (T, G, Gp, maps, Dq) (each group of H/G heads padded to Gp heads,
+// which stay zero), k and v to their pool rows (G, S, Dp) and (G, S, Vp), the keys of a head's maps side by side.  Values come
+// from column vcol of proj on (the keys' own column: they are the keys as projected).  Without kv there are queries only.
+struct WindowPostParams {
+  const __nv_bfloat16* proj;
+  const float *bias, *freq;
+  const int *positions, *slots;
+  __nv_bfloat16 *qout, *kpool, *vpool;
+  int* status;
+  int ldp, H, G, Gp, maps, D, V, Dq, Dp, Vp, dims, norm, S, vcol, kv, temp_every;
+  float eps, temp_coef;
+};
+
+__global__ void __launch_bounds__(256) window_post_kernel(WindowPostParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, lane = threadIdx.x & 31, u = blockIdx.y * 8 + (threadIdx.x >> 5);
-  if (u >= H + 2 * G) return;
-  const __nv_bfloat16* row = proj + static_cast<size_t>(t) * ldp;
-  const float pos = static_cast<float>(positions[t]);
-  if (u < H) {
-    const int hp = (u / (H / G)) * Gp + u % (H / G);
-    head_rotate_norm<__nv_bfloat16, float>(row + u * D, bias != nullptr ? bias + u * D : nullptr,
-                                           qout + (static_cast<size_t>(t) * G * Gp + hp) * Dq, D, Dq, dims, freq, pos, norm != 0, eps);
+  const int nq = p.H * p.maps, nk = p.kv ? p.G * p.maps : 0, nv = p.kv ? p.G : 0;
+  if (u >= nq + nk + nv) return;
+  const __nv_bfloat16* row = p.proj + static_cast<size_t>(t) * p.ldp;
+  const int ipos = p.positions[t];
+  const float pos = static_cast<float>(ipos);
+  if (u < nq) {
+    const int h = u / p.maps, group = p.H / p.G, hp = (h / group) * p.Gp + h % group;
+    const float f = p.temp_every > 0 ? 1.f + p.temp_coef * logf(static_cast<float>((ipos + 1) / p.temp_every + 1)) : 1.f;
+    head_rotate_norm<__nv_bfloat16, float>(row + u * p.D, p.bias != nullptr ? p.bias + u * p.D : nullptr,
+                                           p.qout + ((static_cast<size_t>(t) * p.G * p.Gp + hp) * p.maps + u % p.maps) * p.Dq, p.D, p.Dq, p.dims,
+                                           p.freq, pos, p.norm != 0, p.eps, f);
     return;
   }
-  const int slot = slots[t];
-  if (slot < 0 || slot >= S) {
-    if (lane == 0) report(status, kBadSlot);
+  const int slot = p.slots[t];
+  if (slot < 0 || slot >= p.S) {
+    if (lane == 0) report(p.status, kBadSlot);
     return;
   }
-  if (u < H + G) {
-    const int c = u * D;
-    head_rotate_norm<__nv_bfloat16, float>(row + c, bias != nullptr ? bias + c : nullptr,
-                                           kpool + (static_cast<size_t>(u - H) * S + slot) * Dp, D, Dp, dims, freq, pos, norm != 0, eps);
+  if (u < nq + nk) {
+    const int c = u * p.D, i = u - nq, share = p.Dp / p.maps;
+    head_rotate_norm<__nv_bfloat16, float>(row + c, p.bias != nullptr ? p.bias + c : nullptr,
+                                           p.kpool + (static_cast<size_t>(i / p.maps) * p.S + slot) * p.Dp + (i % p.maps) * share, p.D, share, p.dims,
+                                           p.freq, pos, p.norm != 0, p.eps);
     return;
   }
-  const int g = u - H - G, c = (H + G) * D + g * V;
-  __nv_bfloat16* dst = vpool + (static_cast<size_t>(g) * S + slot) * Vp;
-  for (int d = lane; d < Vp; d += 32)
-    dst[d] = __float2bfloat16_rn(d < V ? __bfloat162float(row[c + d]) + (bias != nullptr ? bias[c + d] : 0.f) : 0.f);
+  const int g = u - nq - nk, c = p.vcol + g * p.V;
+  __nv_bfloat16* dst = p.vpool + (static_cast<size_t>(g) * p.S + slot) * p.Vp;
+  for (int d = lane; d < p.Vp; d += 32)
+    dst[d] = __float2bfloat16_rn(d < p.V ? __bfloat162float(row[c + d]) + (p.bias != nullptr ? p.bias[c + d] : 0.f) : 0.f);
+}
+
+// ---------------------------------------------------------------- pooled blocks
+// Means of the cached keys and values of the blocks of P tokens whose last token is among the new ones.  One CTA per (block, head).
+// New tokens of sequence b: positions past .. past + n - 1 with n = cu[b + 1] - cu[b]; with counts instead n = counts[b] positions
+// that END at past (per_seq blocks are looked at then).
+template <typename E>
+__global__ void __launch_bounds__(128)
+pool_blocks_kernel(const E* kp, const E* vp, E* kb, E* vb, int S, int rows, int Kw, int Vw, const int* block_map, int max_blocks, int P,
+                   const int* slot_map, int max_len, const int* seq_rows, const int* cu_q, const int* past_lens, const int* counts,
+                   int per_seq, int B, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x, g = blockIdx.y;
+  int b, j, past, n;
+  if (counts != nullptr) {
+    b = c / per_seq;
+    j = c % per_seq;
+    n = counts[b];
+    past = past_lens[b] - n;
+  } else {
+    int lo = 0, hi = B - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (cu_q[mid] / P + mid <= c) lo = mid; else hi = mid - 1;
+    }
+    b = lo;
+    j = c - (cu_q[b] / P + b);
+    n = cu_q[b + 1] - cu_q[b];
+    past = past_lens[b];
+  }
+  const int blk = past / P + j;
+  if (blk >= (past + n) / P) return;
+  const int row = seq_rows[b];
+  const int dst = blk < max_blocks ? block_map[static_cast<size_t>(row) * max_blocks + blk] : -1;
+  if (dst < 0 || dst >= rows) {
+    if (threadIdx.x == 0) report(status, kBadSlot);
+    return;
+  }
+  const int* slots = slot_map + static_cast<size_t>(row) * max_len + static_cast<size_t>(blk) * P;
+  const float inv = 1.f / P;
+  for (int e = threadIdx.x; e < Kw + Vw; e += blockDim.x) {
+    const bool k = e < Kw;
+    const int w = k ? Kw : Vw, col = k ? e : e - Kw;
+    const E* src = (k ? kp : vp) + static_cast<size_t>(g) * S * w + col;
+    float acc = 0.f;
+#pragma unroll 4
+    for (int i = 0; i < P; ++i) {
+      const int slot = slots[i];
+      if (slot >= 0 && slot < S) acc += hk_ld(src + static_cast<size_t>(slot) * w);
+      else report(status, kBadSlot);
+    }
+    hk_st((k ? kb : vb) + (static_cast<size_t>(g) * rows + dst) * w + col, acc * inv);
+  }
 }
 
 // ---------------------------------------------------------------- window attention on the plain cores
 // One CTA per (token, head); four warps take every fourth visible key each and merge at the end.  The row sees the last
-// `window` tokens of its own path and the positions below `keep`; the sink is a key without a value whose score is sinks[h]
-// (or 0).  With `gate` (T, ldg) the head's output is multiplied by the sigmoid of its logit.
-template <typename E, int NPL>
-__global__ void __launch_bounds__(128)
-window_attn_simt_kernel(const E* q, long long q_tok, const E* kpool, const E* vpool, int Dp, int Vp, const int* slot_map, const int* seq_rows,
-                        const int* cu_q, const int* past_lens, const int* mask_bits, E* out, int ldo, int B, int H, int G, int D, int V,
-                        int S, int max_len, int W, int causal, float scale, int window, int sink, int keep, const float* sinks,
-                        const float* gate, int ldg, int* status) {
+// `window` tokens of its own path (0: all) and the positions below `keep`; the sink is a key without a value whose score is sinks[h]
+// (or 0).  With `gate` (T, ldg) the head's output is multiplied by the sigmoid of its logit.  softcap > 0 caps the scores.
+// Pooled blocks of P positions that end before the window are keys too, read from their rows or, where they reach into a token
+// tree, averaged over the row's path.  MAPS = 2: two queries a head against the two halves of a key row, outputs combined to
+// share * (o1 - lam o2) / rms.
+struct WindowSimt {
+  const void *q, *kpool, *vpool, *kblocks, *vblocks;
+  void* out;
+  const int *slot_map, *seq_rows, *cu_q, *past_lens, *mask_bits, *block_map;
+  const float *sinks, *gate, *lam;
+  int* status;
+  long long q_tok;
+  int Dp, Vp, ldo, B, H, G, D, V, S, max_len, W, causal, window, sink, keep, ldg, P, block_rows, max_blocks;
+  float scale, softcap, share, eps;
+};
+
+template <typename E, int NPL, int MAPS>
+__global__ void __launch_bounds__(128) window_attn_simt_kernel(WindowSimt p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int t = blockIdx.x, h = blockIdx.y, g = h / (H / G);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  int lo = 0, hi = B - 1;
+  const E *kpool = reinterpret_cast<const E*>(p.kpool), *vpool = reinterpret_cast<const E*>(p.vpool);
+  const int t = blockIdx.x, h = blockIdx.y, g = h / (p.H / p.G), D = p.D, V = p.V, W = p.W;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, kmap = p.Dp / MAPS;
+  int lo = 0, hi = p.B - 1;
   while (lo < hi) {
     const int mid = (lo + hi + 1) >> 1;
-    if (cu_q[mid] <= t) lo = mid; else hi = mid - 1;
+    if (p.cu_q[mid] <= t) lo = mid; else hi = mid - 1;
   }
-  const int i = t - cu_q[lo], past = past_lens[lo], n_b = cu_q[lo + 1] - cu_q[lo];
-  const int* slots = slot_map + static_cast<size_t>(seq_rows[lo]) * max_len;
-  const int* bits = causal ? nullptr : mask_bits + static_cast<size_t>(t) * W;
+  const bool causal = p.causal != 0;
+  const int i = t - p.cu_q[lo], past = p.past_lens[lo], n_b = p.cu_q[lo + 1] - p.cu_q[lo];
+  const int* slots = p.slot_map + static_cast<size_t>(p.seq_rows[lo]) * p.max_len;
+  const int* bits = causal ? nullptr : p.mask_bits + static_cast<size_t>(t) * W;
   int pos = past + i;
   if (!causal) {
     int cnt = 0;
     for (int w = 0; w < W; ++w) cnt += __popc(static_cast<unsigned>(bits[w]));
     pos = past + cnt - 1;
   }
-  const int first = max(0, pos - window + 1);
+  const int first = p.window > 0 ? max(0, pos - p.window + 1) : 0;
   const int last = causal ? past + i : past + n_b - 1;
-  float qv[NPL], acc[NPL];
+  float qv[MAPS][NPL], acc[MAPS][NPL], m[MAPS], l[MAPS];
 #pragma unroll
-  for (int e = 0; e < NPL; ++e) {
-    const int c = lane + 32 * e;
-    qv[e] = c < D ? hk_ld(q + t * q_tok + static_cast<size_t>(h) * D + c) * scale : 0.f;
-    acc[e] = 0.f;
+  for (int u = 0; u < MAPS; ++u) {
+#pragma unroll
+    for (int e = 0; e < NPL; ++e) {
+      const int c = lane + 32 * e;
+      qv[u][e] = c < D ? hk_ld(reinterpret_cast<const E*>(p.q) + t * p.q_tok + static_cast<size_t>(h * MAPS + u) * D + c) * p.scale : 0.f;
+      acc[u][e] = 0.f;
+    }
+    m[u] = -INFINITY;
+    l[u] = 0.f;
+    if (p.sink && warp == 0) { m[u] = p.sinks != nullptr ? p.sinks[h] : 0.f; l[u] = 1.f; }
   }
-  float m = -INFINITY, l = 0.f;
-  if (sink && warp == 0) { m = sinks != nullptr ? sinks[h] : 0.f; l = 1.f; }
-  const int first_j = causal ? first : min(first, past), kept = min(keep, first_j);      // two ranges: [0, kept) and [first_j, last]
+  auto dot = [&](const E* kr, int u) {
+    float d = 0.f;
+#pragma unroll
+    for (int e = 0; e < NPL; ++e) {
+      const int c = lane + 32 * e;
+      if (c < D) d += qv[u][e] * hk_ld(kr + u * kmap + c);
+    }
+    return warp_sum(d);
+  };
+  // one more key of score d (map u) and value v(c)
+  auto add = [&](float d, int u, auto v) {
+    if (p.softcap > 0.f) d = p.softcap * tanhf(d / p.softcap);
+    const float mn = fmaxf(m[u], d), a = expf(m[u] - mn), w = expf(d - mn);
+    l[u] = l[u] * a + w;
+#pragma unroll
+    for (int e = 0; e < NPL; ++e) {
+      const int c = lane + 32 * e;
+      acc[u][e] = acc[u][e] * a + (c < V ? w * v(c) : 0.f);
+    }
+    m[u] = mn;
+  };
+  auto slot_of = [&](int j) {
+    int slot = slots[j];
+    if (slot < 0 || slot >= p.S) { if (lane == 0) report(p.status, kBadSlot); slot = 0; }
+    return static_cast<size_t>(slot);
+  };
+  const int first_j = causal ? first : min(first, past), kept = min(p.keep, first_j);      // two ranges: [0, kept) and [first_j, last]
   for (int x = warp; x < kept + last - first_j + 1; x += 4) {
     const int j = x < kept ? x : first_j + x - kept;
     if (j < past) {
-      if (j < first && j >= keep) continue;
+      if (j < first && j >= p.keep) continue;
     } else if (!causal) {
       const int n = j - past;
       if (!((bits[n >> 5] >> (n & 31)) & 1)) continue;
       int depth = 0;                       // proper ancestors of node n, which are those of this row below n
       for (int w = 0; w < (n >> 5); ++w) depth += __popc(static_cast<unsigned>(bits[w]));
       depth += __popc(static_cast<unsigned>(bits[n >> 5]) & ((1u << (n & 31)) - 1u));
-      if (past + depth < first && past + depth >= keep) continue;
+      if (past + depth < first && past + depth >= p.keep) continue;
     }
-    int slot = slots[j];
-    if (slot < 0 || slot >= S) { if (lane == 0) report(status, kBadSlot); slot = 0; }
-    const E* kr = kpool + (static_cast<size_t>(g) * S + slot) * Dp;
-    const E* vr = vpool + (static_cast<size_t>(g) * S + slot) * Vp;
-    float d = 0.f;
+    const size_t slot = slot_of(j);
+    const E* kr = kpool + (static_cast<size_t>(g) * p.S + slot) * p.Dp;
+    const E* vr = vpool + (static_cast<size_t>(g) * p.S + slot) * p.Vp;
 #pragma unroll
-    for (int e = 0; e < NPL; ++e) {
-      const int c = lane + 32 * e;
-      if (c < D) d += qv[e] * hk_ld(kr + c);
-    }
-    d = warp_sum(d);
-    const float mn = fmaxf(m, d), a = expf(m - mn), p = expf(d - mn);
-    l = l * a + p;
-#pragma unroll
-    for (int e = 0; e < NPL; ++e) {
-      const int c = lane + 32 * e;
-      acc[e] = acc[e] * a + (c < V ? p * hk_ld(vr + c) : 0.f);
-    }
-    m = mn;
+    for (int u = 0; u < MAPS; ++u) add(dot(kr, u), u, [&](int c) { return hk_ld(vr + c); });
   }
-  __shared__ float sm[4], sl[4];
-  extern __shared__ float so[];            // 4 x V
-  if (lane == 0) { sm[warp] = m; sl[warp] = l; }
+  if (p.P > 0) {
+    const int blocks = pos - p.window >= 0 ? (pos - p.window + 1) / p.P : 0, stored = causal ? blocks : past / p.P;
+    // slot of position j of this row's own path
+    auto path_slot = [&](int j) {
+      if (j < past) return slot_of(j);
+      int left = j - past, w = 0;
+      while (w < W && left >= __popc(static_cast<unsigned>(bits[w]))) left -= __popc(static_cast<unsigned>(bits[w++]));
+      if (w >= W) { if (lane == 0) report(p.status, kBadNode); return slot_of(past); }
+      unsigned word = static_cast<unsigned>(bits[w]);
+      for (; left > 0; --left) word &= word - 1u;
+      return slot_of(past + 32 * w + __ffs(static_cast<int>(word)) - 1);
+    };
+    for (int b = warp; b < blocks; b += 4) {
+      if (b < stored) {
+        int r = b < p.max_blocks ? p.block_map[static_cast<size_t>(p.seq_rows[lo]) * p.max_blocks + b] : -1;
+        if (r < 0 || r >= p.block_rows) { if (lane == 0) report(p.status, kBadSlot); r = 0; }
+        const E* kr = reinterpret_cast<const E*>(p.kblocks) + (static_cast<size_t>(g) * p.block_rows + r) * p.Dp;
+        const E* vr = reinterpret_cast<const E*>(p.vblocks) + (static_cast<size_t>(g) * p.block_rows + r) * p.Vp;
 #pragma unroll
-  for (int e = 0; e < NPL; ++e)
-    if (lane + 32 * e < V) so[warp * V + lane + 32 * e] = acc[e];
+        for (int u = 0; u < MAPS; ++u) add(dot(kr, u), u, [&](int c) { return hk_ld(vr + c); });
+        continue;
+      }
+      const float inv = 1.f / p.P;
+      float d[MAPS] = {}, mean[NPL] = {};
+      for (int j = b * p.P; j < (b + 1) * p.P; ++j) {
+        const size_t slot = path_slot(j);
+#pragma unroll
+        for (int u = 0; u < MAPS; ++u) d[u] += dot(kpool + (static_cast<size_t>(g) * p.S + slot) * p.Dp, u);
+#pragma unroll
+        for (int e = 0; e < NPL; ++e)
+          if (lane + 32 * e < V) mean[e] += hk_ld(vpool + (static_cast<size_t>(g) * p.S + slot) * p.Vp + lane + 32 * e);
+      }
+#pragma unroll
+      for (int u = 0; u < MAPS; ++u) add(d[u] * inv, u, [&](int c) { return mean[(c - lane) / 32] * inv; });
+    }
+  }
+  __shared__ float sm[MAPS][4], sl[MAPS][4], red[4];
+  extern __shared__ float so[];            // MAPS x 4 x V
+#pragma unroll
+  for (int u = 0; u < MAPS; ++u) {
+    if (lane == 0) { sm[u][warp] = m[u]; sl[u][warp] = l[u]; }
+#pragma unroll
+    for (int e = 0; e < NPL; ++e)
+      if (lane + 32 * e < V) so[(u * 4 + warp) * V + lane + 32 * e] = acc[u][e];
+  }
   __syncthreads();
-  const float mm = fmaxf(fmaxf(sm[0], sm[1]), fmaxf(sm[2], sm[3]));
-  float f[4], tot = 0.f;
+  float f[MAPS][4];
 #pragma unroll
-  for (int w2 = 0; w2 < 4; ++w2) {
-    f[w2] = sm[w2] == -INFINITY ? 0.f : expf(sm[w2] - mm);
-    tot += sl[w2] * f[w2];
+  for (int u = 0; u < MAPS; ++u) {
+    const float mm = fmaxf(fmaxf(sm[u][0], sm[u][1]), fmaxf(sm[u][2], sm[u][3]));
+    float tot = 0.f;
+#pragma unroll
+    for (int w2 = 0; w2 < 4; ++w2) {
+      f[u][w2] = sm[u][w2] == -INFINITY ? 0.f : expf(sm[u][w2] - mm);
+      tot += sl[u][w2] * f[u][w2];
+    }
+    const float inv = tot > 0.f ? 1.f / tot : 0.f;
+#pragma unroll
+    for (int w2 = 0; w2 < 4; ++w2) f[u][w2] *= inv;
   }
-  float inv = tot > 0.f ? 1.f / tot : 0.f;
-  if (gate != nullptr) inv /= 1.f + expf(-gate[static_cast<size_t>(t) * ldg + h]);
-  for (int c = threadIdx.x; c < V; c += blockDim.x)
-    hk_st(out + static_cast<size_t>(t) * ldo + h * V + c, (so[c] * f[0] + so[V + c] * f[1] + so[2 * V + c] * f[2] + so[3 * V + c] * f[3]) * inv);
+  auto read = [&](int u, int c) {
+    const float* o = so + u * 4 * V + c;
+    return o[0] * f[u][0] + o[V] * f[u][1] + o[2 * V] * f[u][2] + o[3 * V] * f[u][3];
+  };
+  E* out = reinterpret_cast<E*>(p.out) + static_cast<size_t>(t) * p.ldo + h * V;
+  if constexpr (MAPS == 1) {
+    const float gate = p.gate != nullptr ? 1.f / (1.f + expf(-p.gate[static_cast<size_t>(t) * p.ldg + h])) : 1.f;
+    for (int c = threadIdx.x; c < V; c += blockDim.x) hk_st(out + c, read(0, c) * gate);
+  } else {
+    const float lam = *p.lam;
+    float o[(NPL + 3) / 4], ss = 0.f;      // a thread's columns: threadIdx.x, + 128, ...
+#pragma unroll
+    for (int e = 0; e < (NPL + 3) / 4; ++e) {
+      const int c = threadIdx.x + 128 * e;
+      o[e] = c < V ? read(0, c) - lam * read(1, c) : 0.f;
+      ss += o[e] * o[e];
+    }
+    const float r = p.share / sqrtf(cta_sum<128>(ss, red) / V + p.eps);
+#pragma unroll
+    for (int e = 0; e < (NPL + 3) / 4; ++e) {
+      const int c = threadIdx.x + 128 * e;
+      if (c < V) hk_st(out + c, o[e] * r);
+    }
+  }
 }
 
-template <typename E>
-static int launch_window_simt(const void* q, long long q_tok, const void* kp, const void* vp, int Dp, int Vp, const int* slot_map,
-                              const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out, int ldo,
-                              int B, int T, int H, int G, int D, int V, int S, int max_len, int W, int causal, float scale, int window,
-                              int sink, int keep, const float* sinks, const float* gate, int ldg, int* status, int pdl,
-                              cudaStream_t stream) {
-  HybridLaunch l(dim3(T, H), dim3(128), stream, pdl, 4 * V * sizeof(float));
-  const int n = D > V ? D : V;
-  auto kern = n <= 64 ? window_attn_simt_kernel<E, 2> : n <= 128 ? window_attn_simt_kernel<E, 4>
-            : n <= 256 ? window_attn_simt_kernel<E, 8> : window_attn_simt_kernel<E, 16>;
-  return cudaLaunchKernelEx(&l.c, kern, (const E*)q, q_tok, (const E*)kp, (const E*)vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens,
-                            mask_bits, (E*)out, ldo, B, H, G, D, V, S, max_len, W, causal, scale, window, sink, keep, sinks, gate, ldg,
-                            status) == cudaSuccess ? 0 : -4;
+template <typename E, int MAPS>
+static int launch_window_simt(const WindowSimt& p, int T, int pdl, cudaStream_t stream) {
+  HybridLaunch l(dim3(T, p.H), dim3(128), stream, pdl, MAPS * 4 * p.V * sizeof(float));
+  const int n = p.D > p.V ? p.D : p.V;
+  auto kern = n <= 64 ? window_attn_simt_kernel<E, 2, MAPS> : n <= 128 ? window_attn_simt_kernel<E, 4, MAPS>
+            : n <= 256 ? window_attn_simt_kernel<E, 8, MAPS> : window_attn_simt_kernel<E, 16, MAPS>;
+  return cudaLaunchKernelEx(&l.c, kern, p) == cudaSuccess ? 0 : -4;
 }
 
 // ---------------------------------------------------------------- the residual step behind a sublayer
@@ -458,35 +613,60 @@ extern "C" int js_rotate_norm(const void* x, void* out, const int* positions, in
   return cudaGetLastError() == cudaSuccess ? 0 : -4;
 }
 
-extern "C" int js_window_post(const void* proj, int ldp, const float* bias, int H, int G, int Gp, int D, int V, int Dq, int Dp, int Vp, int dims,
-                              const float* freq, int norm, float eps, const int* positions, const int* slots, int S, int T, void* qout,
-                              void* kpool, void* vpool, int* status, int pdl, cudaStream_t stream) {
+// See window_post_kernel.
+extern "C" int js_window_post(const void* proj, int ldp, const float* bias, int H, int G, int Gp, int maps, int D, int V, int Dq, int Dp, int Vp,
+                              int dims, const float* freq, int norm, float eps, int temp_every, float temp_coef, int vcol, int kv,
+                              const int* positions, const int* slots, int S, int T, void* qout, void* kpool, void* vpool, int* status,
+                              int pdl, cudaStream_t stream) {
   using namespace js;
   if (T <= 0) return 0;
-  if (H % G || Dp > 512 || Dq > 512 || D > Dq || D > Dp || V > Vp || dims > D || (dims & 1) || Gp < H / G) return -10;
-  HybridLaunch l(dim3(T, (H + 2 * G + 7) / 8), dim3(256), stream, pdl);
+  if (maps < 1 || H % G || Dp > 512 * maps || Dp % maps || Dq > 512 || D > Dq || D > Dp / maps || V > Vp || dims > D || (dims & 1) || Gp < H / G) return -10;
+  HybridLaunch l(dim3(T, (H * maps + (kv ? G * (maps + 1) : 0) + 7) / 8), dim3(256), stream, pdl);
   using bf = __nv_bfloat16;
-  return cudaLaunchKernelEx(&l.c, window_post_kernel, (const bf*)proj, ldp, bias, H, G, Gp, D, V, Dq, Dp, Vp, dims, freq, norm, eps, positions,
-                            slots, S, (bf*)qout, (bf*)kpool, (bf*)vpool, status) == cudaSuccess ? 0 : -4;
+  WindowPostParams p{(const bf*)proj, bias, freq, positions, slots, (bf*)qout, (bf*)kpool, (bf*)vpool, status,
+                     ldp, H, G, Gp, maps, D, V, Dq, Dp, Vp, dims, norm, S, vcol, kv, temp_every, eps, temp_coef};
+  return cudaLaunchKernelEx(&l.c, window_post_kernel, p) == cudaSuccess ? 0 : -4;
 }
 
-// q: token t at t * q_tok, head h at h * D; pools (G, S, Dp) and (G, S, Vp); out (T, ldo), head h at h * V.  D, V at most 512.
-// sink: a valueless key of score sinks[h] (null: 0) takes part; keep: positions below it stay visible behind the window;
-// gate (T, ldg) fp32 logits or null.
+// Pools (G, S, Kw) and (G, S, Vw), block rows (G, rows, Kw) and (G, rows, Vw); see pool_blocks_kernel.  T bounds the new tokens of
+// all sequences; with counts, per_seq bounds a sequence's blocks.
+extern "C" int js_pool_blocks(const void* kp, const void* vp, void* kb, void* vb, int G, int S, int rows, int Kw, int Vw, const int* block_map,
+                              int max_blocks, int P, const int* slot_map, int max_len, const int* seq_rows, const int* cu_q,
+                              const int* past_lens, const int* counts, int per_seq, int B, int T, int bf16, int* status, int pdl,
+                              cudaStream_t stream) {
+  using namespace js;
+  if (B <= 0 || (counts == nullptr && T <= 0)) return 0;
+  if (P < 1 || G < 1 || (counts == nullptr ? cu_q == nullptr : per_seq < 1)) return -10;
+  HybridLaunch l(dim3(counts != nullptr ? B * per_seq : T / P + B, G), dim3(128), stream, pdl);
+  using bf = __nv_bfloat16;
+  if (bf16)
+    return cudaLaunchKernelEx(&l.c, pool_blocks_kernel<bf>, (const bf*)kp, (const bf*)vp, (bf*)kb, (bf*)vb, S, rows, Kw, Vw, block_map, max_blocks, P,
+                              slot_map, max_len, seq_rows, cu_q, past_lens, counts, per_seq, B, status) == cudaSuccess ? 0 : -4;
+  return cudaLaunchKernelEx(&l.c, pool_blocks_kernel<float>, (const float*)kp, (const float*)vp, (float*)kb, (float*)vb, S, rows, Kw, Vw, block_map,
+                            max_blocks, P, slot_map, max_len, seq_rows, cu_q, past_lens, counts, per_seq, B, status) == cudaSuccess ? 0 : -4;
+}
+
+// q: token t at t * q_tok, head h (map m) at (h * maps + m) * D; pools (G, S, Dp) and (G, S, Vp); out (T, ldo), head h at h * V.
+// D, V at most 512.  sink: a valueless key of score sinks[h] (null: 0) takes part; keep: positions below it stay visible behind the
+// window (0: no window); gate (T, ldg) fp32 logits or null; softcap 0: none; P > 0: pooled blocks in kb (G, block_rows, Dp), vb
+// (G, block_rows, Vp) through block_map (rows, max_blocks); maps 2 combines with lam (device), share and eps.
 extern "C" int js_window_attention_simt(const void* q, long long q_tok, const void* kp, const void* vp, int Dp, int Vp, const int* slot_map,
                                         const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
                                         int ldo, int B, int T, int H, int G, int D, int V, int S, int max_len, int W, int causal,
                                         float scale, int window, int sink, int keep, const float* sinks, const float* gate, int ldg,
-                                        int bf16, int* status, int pdl, cudaStream_t stream) {
+                                        float softcap, int P, const void* kb, const void* vb, int block_rows, const int* block_map,
+                                        int max_blocks, int maps, const float* lam, float share, float eps, int bf16, int* status, int pdl,
+                                        cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
-  if (H % G || D > 512 || V > 512 || D > Dp || V > Vp || window < 1 || keep < 0) return -10;
+  if (maps < 1 || maps > 2 || H % G || D > 512 || V > 512 || Dp % maps || D > Dp / maps || V > Vp || window < 0 || keep < 0 || P < 0) return -10;
   if (!causal && (mask_bits == nullptr || W < 1)) return -13;
-  return bf16 ? launch_window_simt<__nv_bfloat16>(q, q_tok, kp, vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ldo, B, T,
-                                                  H, G, D, V, S, max_len, W, causal, scale, window, sink, keep, sinks, gate, ldg,
-                                                  status, pdl, stream)
-              : launch_window_simt<float>(q, q_tok, kp, vp, Dp, Vp, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ldo, B, T, H, G,
-                                          D, V, S, max_len, W, causal, scale, window, sink, keep, sinks, gate, ldg, status, pdl, stream);
+  if ((P > 0 && (window < 1 || kb == nullptr || vb == nullptr || block_map == nullptr)) || (maps == 2 && lam == nullptr)) return -13;
+  WindowSimt p{q, kp, vp, kb, vb, out, slot_map, seq_rows, cu_q, past_lens, mask_bits, block_map, sinks, gate, lam, status, q_tok,
+               Dp, Vp, ldo, B, H, G, D, V, S, max_len, W, causal, window, sink, keep, ldg, P, block_rows, max_blocks,
+               scale, softcap, share, eps};
+  if (bf16) return maps == 2 ? launch_window_simt<__nv_bfloat16, 2>(p, T, pdl, stream) : launch_window_simt<__nv_bfloat16, 1>(p, T, pdl, stream);
+  return maps == 2 ? launch_window_simt<float, 2>(p, T, pdl, stream) : launch_window_simt<float, 1>(p, T, pdl, stream);
 }
 
 // Either ya (with yb, wa, wb for a pair; bias optional) or ys / inv / k and sh, all bf16 rows whose

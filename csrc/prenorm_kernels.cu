@@ -1,5 +1,6 @@
-// Steps between the GEMMs of pre-norm decoders with mixed mixers: scaled embedding with the first norm and the step's rotary
-// tables, RMS norm of the fp32 residual stream, what follows an attention's input projections (biases, norms over whole
+// Steps between the GEMMs of pre-norm decoders with mixed mixers: scaled embedding (with learned positions) with the first norm
+// and the step's rotary tables, RMS norm of the fp32 residual stream, the residual step of sublayers whose output is normed
+// (with a weighted average over the depth), what follows an attention's input projections (biases, norms over whole
 // projections, general rotations, cache scatter), and the unfused forms.  Math is fp32; the residual stream is fp32.
 //
 // Rotations: entry pairs (i, i + n) ("half") or (2i, 2i + 1) ("next") of a head's first 2n entries.  The fused steps read
@@ -57,6 +58,27 @@ __global__ void gelu_erf_kernel(const E* x, E* out, size_t n) {
   }
 }
 
+template <typename E>
+__global__ void xielu_kernel(const E* x, E* out, size_t n, float up, float down) {
+  for (size_t i = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x; i < n; i += static_cast<size_t>(gridDim.x) * blockDim.x) {
+    const float z = pn_ld(x + i);
+    pn_st(out + i, 0.5f * z + (z > 0.f ? up * z * z : down * (expm1f(z) - z)));
+  }
+}
+
+// out = sum_j w[j] hist_j, the terms given by address
+constexpr int kDepthTerms = 64;
+struct DepthTerms {
+  const float* x[kDepthTerms];
+};
+__global__ void depth_average_kernel(DepthTerms h, int terms, const float* w, int first, float* out, size_t n) {
+  for (size_t i = blockIdx.x * static_cast<size_t>(blockDim.x) + threadIdx.x; i < n; i += static_cast<size_t>(gridDim.x) * blockDim.x) {
+    float acc = first ? 0.f : out[i];
+    for (int j = 0; j < terms; ++j) acc += w[j] * h.x[j][i];
+    out[i] = acc;
+  }
+}
+
 // out (T, H, V) = y * sigmoid(logits[t, h])
 template <typename E>
 __global__ void head_gate_kernel(const E* y, const float* logits, int ldz, E* out, size_t n, int H, int V) {
@@ -95,11 +117,12 @@ __global__ void rotate_kernel(const E* x, O* out, const int* positions, size_t u
 constexpr int kRowThreads = 256;
 constexpr int kRowKeep = 8;              // float4s a thread holds on to (rows up to 8192 wide); the rest is read twice
 
-// x[t] = scale * table[ids[t]], h[t] = bf16(x / rms(x) * w), rot[t] = (amp cos, amp sin) of the nf concatenated frequencies.
+// x[t] = scale * table[ids[t]] (+ pos_table[positions[t]], its last row past the end), h[t] = bf16(x / rms(x) * w), rot[t] = (amp cos, amp sin) of the nf concatenated frequencies.
 // Rows are ld long (a multiple of 4), zero past W; w too.
 __global__ void __launch_bounds__(kRowThreads)
 embed_rms_kernel(const int* ids, const __nv_bfloat16* table, int V, int ldt, float scale, const float* w, float eps, float* x,
-                 __nv_bfloat16* h, int ld, int W, const int* positions, const float* freq, const float* amp, int nf, float2* rot) {
+                 __nv_bfloat16* h, int ld, int W, const int* positions, const __nv_bfloat16* pos_table, int n_pos, const float* freq,
+                 const float* amp, int nf, float2* rot) {
   __shared__ float red[kRowThreads / 32];
   pdl_launch_dependents();
   pdl_wait();
@@ -108,11 +131,26 @@ embed_rms_kernel(const int* ids, const __nv_bfloat16* table, int V, int ldt, flo
   id = id < 0 ? 0 : (id >= V ? V - 1 : id);
   const uint2* src = reinterpret_cast<const uint2*>(table + static_cast<size_t>(id) * ldt);
   float4* xr = reinterpret_cast<float4*>(x + static_cast<size_t>(t) * ld);
+  const uint2* add = nullptr;
+  if (pos_table != nullptr) {
+    const int at = positions[t];
+    add = reinterpret_cast<const uint2*>(pos_table + static_cast<size_t>(at < 0 ? 0 : (at >= n_pos ? n_pos - 1 : at)) * ldt);
+  }
   auto load = [&](int c) {
     const uint2 raw = src[c];
     const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
     const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-    return make_float4(lo.x * scale, lo.y * scale, hi.x * scale, hi.y * scale);
+    float4 v = make_float4(lo.x * scale, lo.y * scale, hi.x * scale, hi.y * scale);
+    if (add != nullptr) {
+      const uint2 more = add[c];
+      const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&more.x));
+      const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&more.y));
+      v.x += a.x;
+      v.y += a.y;
+      v.z += b.x;
+      v.w += b.y;
+    }
+    return v;
   };
   float ss = 0.f;
   for (int c = tid; c < W4; c += kRowThreads) {
@@ -180,6 +218,96 @@ rms_rows_kernel(const float* x, const float* w, float eps, __nv_bfloat16* h, int
     if (c < W4) put(c, v[j], g[j]);
   }
   for (int c = tid + kRowKeep * kRowThreads; c < W4; c += kRowThreads) put(c, xr[c], w4[c]);
+}
+
+// ---------------------------------------------------------------- the residual step of a sublayer whose output is normed
+// v = src + y / rms(y) * w.  Within a layer x = v.  At a layer's end (d set) v is the layer's result: it goes to hist slot `terms`
+// and x = sum_{j < terms} d[j] hist[j] + d[terms] v.  h = bf16(x / rms(x) * fw), tap = bf16(x).  Rows are ld long (a multiple of
+// 4) and zero past W, weights too.
+struct SandwichParams {
+  const __nv_bfloat16* y;
+  const float *src, *w, *fw, *d;
+  float *hist, *x;
+  __nv_bfloat16 *h, *tap;
+  size_t hist_stride;
+  int ldy, ld, ldt, W, terms;
+  float eps;
+};
+
+template <int NT, int KEEP>
+__global__ void __launch_bounds__(NT) sandwich_kernel(SandwichParams p) {
+  __shared__ float red[NT / 32];
+  pdl_launch_dependents();
+  const int t = blockIdx.x, tid = threadIdx.x, W4 = p.ld / 4;
+  const size_t row = static_cast<size_t>(t) * p.ld;
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  pdl_wait();
+  float4 v[KEEP], s[KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = tid + j * NT;
+    v[j] = s[j] = zero;
+    if (c < W4) {
+      const uint2 raw = *reinterpret_cast<const uint2*>(p.y + static_cast<size_t>(t) * p.ldy + 4 * c);
+      const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+      const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+      v[j] = make_float4(a.x, a.y, b.x, b.y);
+      s[j] = reinterpret_cast<const float4*>(p.src + row)[c];
+    }
+    ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+  }
+  // the history is on its way while the sum is made
+  float4 acc[KEEP];
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) acc[j] = zero;
+  for (int i = 0; i < p.terms; ++i) {
+    const float di = __ldg(p.d + i);
+    const float4* hr = reinterpret_cast<const float4*>(p.hist + i * p.hist_stride + row);
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j) {
+      const int c = tid + j * NT;
+      if (c < W4) {
+        const float4 u = hr[c];
+        acc[j].x += di * u.x;
+        acc[j].y += di * u.y;
+        acc[j].z += di * u.z;
+        acc[j].w += di * u.w;
+      }
+    }
+  }
+  const float r = 1.f / sqrtf(pn_sum<NT>(ss, red) / p.W + p.eps);
+  const float dl = p.d != nullptr ? __ldg(p.d + p.terms) : 1.f;
+  ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = tid + j * NT;
+    if (c >= W4) continue;
+    const float4 g = reinterpret_cast<const float4*>(p.w)[c];
+    float4 u = make_float4(s[j].x + v[j].x * r * g.x, s[j].y + v[j].y * r * g.y, s[j].z + v[j].z * r * g.z, s[j].w + v[j].w * r * g.w);
+    if (p.d != nullptr) {
+      reinterpret_cast<float4*>(p.hist + p.terms * p.hist_stride + row)[c] = u;
+      u = make_float4(acc[j].x + dl * u.x, acc[j].y + dl * u.y, acc[j].z + dl * u.z, acc[j].w + dl * u.w);
+    }
+    reinterpret_cast<float4*>(p.x + row)[c] = u;
+    if (p.tap != nullptr) {
+      const float e[4] = {u.x, u.y, u.z, u.w};
+      for (int i = 0; i < 4; ++i)
+        if (4 * c + i < p.W) p.tap[static_cast<size_t>(t) * p.ldt + 4 * c + i] = __float2bfloat16_rn(e[i]);
+    }
+    v[j] = u;
+    ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
+  }
+  const float rf = 1.f / sqrtf(pn_sum<NT>(ss, red) / p.W + p.eps);
+#pragma unroll
+  for (int j = 0; j < KEEP; ++j) {
+    const int c = tid + j * NT;
+    if (c >= W4) continue;
+    const float4 g = reinterpret_cast<const float4*>(p.fw)[c];
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v[j].x * rf * g.x, v[j].y * rf * g.y);
+    const __nv_bfloat162 b = __floats2bfloat162_rn(v[j].z * rf * g.z, v[j].w * rf * g.w);
+    reinterpret_cast<uint2*>(p.h + row)[c] = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  }
 }
 
 // ---------------------------------------------------------------- behind the input projections of a K/V attention
@@ -477,15 +605,65 @@ extern "C" int js_rotate(const void* x, int x_bf16, void* out, int o_bf16, const
 }
 
 // table (V, ldt) bf16, x (T, ld) fp32, h (T, ld) bf16, w (ld) fp32; ld and ldt multiples of 4, at least W; rot (T, nf) float2.
+// pos_table (n_pos, ldt) bf16 or null.
 extern "C" int js_embed_rms(const int* ids, const void* table, int V, int ldt, float scale, const float* w, float eps, float* x, void* h, int ld,
-                            int T, int W, const int* positions, const float* freq, const float* amp, int nf, void* rot, int pdl,
-                            cudaStream_t stream) {
+                            int T, int W, const int* positions, const void* pos_table, int n_pos, const float* freq, const float* amp, int nf,
+                            void* rot, int pdl, cudaStream_t stream) {
   using namespace js;
   if (T <= 0) return 0;
   if ((ld % 4) || (ldt % 4) || ldt < ld || W < 1 || W > ld) return -10;
   PrenormLaunch l(dim3(T), dim3(kRowThreads), stream, pdl);
   return cudaLaunchKernelEx(&l.c, embed_rms_kernel, ids, (const __nv_bfloat16*)table, V, ldt, scale, w, eps, x, (__nv_bfloat16*)h, ld, W, positions,
-                            freq, amp, nf, (float2*)rot) == cudaSuccess ? 0 : -4;
+                            (const __nv_bfloat16*)pos_table, n_pos, freq, amp, nf, (float2*)rot) == cudaSuccess ? 0 : -4;
+}
+
+extern "C" int js_xielu(const void* x, void* out, long long n, float up, float down, int bf16, cudaStream_t stream) {
+  using namespace js;
+  using bf = __nv_bfloat16;
+  if (n <= 0) return 0;
+  if (bf16) xielu_kernel<bf><<<pn_grid(n), 256, 0, stream>>>((const bf*)x, (bf*)out, n, up, down);
+  else xielu_kernel<float><<<pn_grid(n), 256, 0, stream>>>((const float*)x, (float*)out, n, up, down);
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// out (n) = sum over `terms` of w[j] times the n floats at addr[j] (host array of device addresses)
+extern "C" int js_depth_average(const unsigned long long* addr, int terms, const float* w, float* out, long long n, cudaStream_t stream) {
+  using namespace js;
+  if (n <= 0 || terms <= 0) return 0;
+  for (int j0 = 0; j0 < terms; j0 += kDepthTerms) {
+    DepthTerms h{};
+    const int m = terms - j0 < kDepthTerms ? terms - j0 : kDepthTerms;
+    for (int j = 0; j < m; ++j) h.x[j] = reinterpret_cast<const float*>(addr[j0 + j]);
+    depth_average_kernel<<<pn_grid(n), 256, 0, stream>>>(h, m, w + j0, j0 == 0, out, n);
+  }
+  return cudaGetLastError() == cudaSuccess ? 0 : -4;
+}
+
+// See sandwich_kernel.  d: null within a layer, else terms + 1 weights on the device; hist (layers + 1, T, ld) with hist_stride
+// elements between layers.  ld a multiple of 4, at most 32768; ldy a multiple of 4, at least ld.
+extern "C" int js_sandwich(const void* y, int ldy, const float* src, const float* w, const float* d, int terms, float* hist,
+                           long long hist_stride, float* x, const float* fw, float eps, void* h, int ld, void* tap, int ldt, int T, int W,
+                           int pdl, cudaStream_t stream) {
+  using namespace js;
+  if (T <= 0) return 0;
+  if ((ld % 4) || (ldy % 4) || ldy < ld || W < 1 || W > ld || ld > 32768 || terms < 0 || (d != nullptr) != (hist != nullptr) || (d == nullptr && terms)) return -10;
+  SandwichParams p{(const __nv_bfloat16*)y, src, w, fw, d, hist, x, (__nv_bfloat16*)h, (__nv_bfloat16*)tap, (size_t)hist_stride,
+                   ldy, ld, ldt, W, terms, eps};
+  const int w4 = ld / 4;
+  // few rows (decode) want many threads a row, many rows several float4 a thread
+  const bool few = T <= 296;
+  int nt = 256;
+  auto kern = sandwich_kernel<256, 1>;
+  if (w4 <= 256) {}
+  else if (w4 <= 512 && !few) kern = sandwich_kernel<256, 2>;
+  else if (w4 <= 512) { kern = sandwich_kernel<512, 1>; nt = 512; }
+  else if (w4 <= 1024 && !few) kern = sandwich_kernel<256, 4>;
+  else if (w4 <= 1024) { kern = sandwich_kernel<1024, 1>; nt = 1024; }
+  else if (w4 <= 2048) { kern = sandwich_kernel<512, 4>; nt = 512; }
+  else if (w4 <= 4096) { kern = sandwich_kernel<1024, 4>; nt = 1024; }
+  else { kern = sandwich_kernel<1024, 8>; nt = 1024; }
+  PrenormLaunch l(dim3(T), dim3(nt), stream, pdl);
+  return cudaLaunchKernelEx(&l.c, kern, p) == cudaSuccess ? 0 : -4;
 }
 
 // x (T, ld) fp32 -> h (T, ld) bf16, w (ld) fp32, ld a multiple of 4; tap (T, ldt) bf16 gets the first W columns of x, or is null.

@@ -36,6 +36,13 @@ def resolve_eos(model, tokenizer) -> set:
     return ids
 
 
+def check_positions(cfg, tokens: int) -> None:
+    """Refuse sequences a learned position table has no rows for."""
+    most = getattr(cfg, "max_positions", None)
+    if most is not None and tokens > most:
+        raise ValueError(f"{tokens} tokens, but the model has {most} positions")
+
+
 def decode_text(tokenizer, ids) -> str:
     return tokenizer.decode(ids, skip_special_tokens=True) if tokenizer is not None else ""
 
@@ -79,6 +86,7 @@ class LLM:
         """Plain decode.  Returns ``{"token_ids", "text", "decode_time"}``."""
         sp = sampling_params or SamplingParams()
         ids = self._ids(prompt)
+        check_positions(self.model.config, ids.shape[1] + sp.max_new_tokens - 1)
         cache = self.runner.new_cache(ids.shape[1] + sp.max_new_tokens + 1)
         logits, cache, _ = self.runner.forward(ids, cache, last_position_logits_only=True)
         out = [self._pick(logits, sp.temperature)]
@@ -98,6 +106,7 @@ class LLM:
         committed and the rejected drafts' KV cropped.  Returns ``{"token_ids","text","tpf"}``."""
         sp = sampling_params or SamplingParams()
         committed = self._ids(prompt)
+        check_positions(self.model.config, committed.shape[1] + sp.max_new_tokens - 1)
         if hasattr(drafter, "reset_cache"):
             drafter.reset_cache()
         k = max(1, block_size - 1)
@@ -160,6 +169,7 @@ class LLM:
         """
         sp = sampling_params or SamplingParams()
         committed = self._ids(prompt)
+        check_positions(self.model.config, committed.shape[1] + sp.max_new_tokens - 1)
         if hasattr(tree_drafter, "reset_cache"):
             tree_drafter.reset_cache()
         algo_obj = get_algorithm(algo, **(algo_kwargs or {}))

@@ -12,6 +12,8 @@ from typing import Optional, Sequence
 
 import torch
 
+from ..ops import reference as ref
+
 
 class DenseKVCache:
     """Contiguous ``(Hkv, capacity, D)`` K and V per layer with a shared length; a latent-attention model's latent rows
@@ -40,7 +42,8 @@ class DenseKVCache:
         if shapes is not None or widths is not None:
             rows = lambda heads, w: torch.zeros(heads, cap, w, dtype=self.dtype, device=self.device)
             shapes, widths = shapes or [None] * len(widths), widths or [None] * len(shapes)
-            nk = [rows(s[0], s[1]) if s is not None else rows(1, w) if w is not None else None for s, w in zip(shapes, widths)]
+            keys = lambda heads, dim, vdim, maps=1: rows(heads, dim * maps)
+            nk = [keys(*s) if s is not None else rows(1, w) if w is not None else None for s, w in zip(shapes, widths)]
             nv = [rows(s[0], s[2]) if s is not None else None for s in shapes]
         else:
             L, Hkv, D = self.cfg.num_hidden_layers, self.cfg.num_key_value_heads, self.cfg.head_dim
@@ -229,16 +232,35 @@ class ModelRunner:
             from ..tree.ancestor import pack_ancestor_bits
             bits = pack_ancestor_bits(ancestor.to(ids.device))
 
+        sources = cfg.kv_sources() if hasattr(cfg, "kv_sources") else None
+
         def window(layer: int, mixer, q, k, v):
-            """Window attention as the plain formula over the contiguous cache."""
+            """Attention in a window, with pooled blocks or differential, as the plain formula over the contiguous cache.  A
+            block's score is the mean of its tokens' scores, and its weight is shared out over their values."""
             m = mixer.cfg
-            cache.k[layer][:, past:past + T] = k.transpose(0, 1)
-            cache.v[layer][:, past:past + T] = v.transpose(0, 1)
-            K, V = cache.k[layer][:, :past + T].float(), cache.v[layer][:, :past + T].float()
-            s = torch.einsum("nhgd,hld->hgnl", q.float().view(T, m.kv_heads, m.heads // m.kv_heads, m.dim), K) * m.scale
-            seen = vis & ((pos[:, None] - key_pos[None, :] < m.window) | (key_pos < m.keep_first)[None])
-            p = weights(s, seen[None, None], mixer.sink)
-            return torch.einsum("hgnl,hlv->nhgv", p, V).reshape(T, m.heads * m.vdim).to(q.dtype)
+            at = layer if sources is None else sources[layer]
+            if k is not None:
+                cache.k[at][:, past:past + T] = k.transpose(0, 1)
+                cache.v[at][:, past:past + T] = v.transpose(0, 1)
+            K, V = cache.k[at][:, :past + T].float(), cache.v[at][:, :past + T].float()
+            seen = vis & ((pos[:, None] - key_pos[None, :] < m.window) | (key_pos < m.keep_first)[None]) if m.window else vis
+            if m.pool:
+                ends = (torch.arange(int(pos.max()) // m.pool + 1, device=ids.device) + 1) * m.pool - 1
+                far = ends[None] <= pos[:, None] - m.window
+                share = (key_pos[:, None] // m.pool == (ends // m.pool)[None]).float() / m.pool
+            acc = []
+            for i in range(m.maps):
+                qi = q[:, i::m.maps].float().reshape(T, m.kv_heads, m.heads // m.kv_heads, m.dim)
+                s = torch.einsum("nhgd,hld->hgnl", qi, K[..., i * m.dim:(i + 1) * m.dim]) * m.scale
+                if m.pool:
+                    all_s, both = torch.cat((s, (s * vis) @ share), -1), torch.cat((seen, far), -1)
+                    p = weights(ref.softcapped(all_s, m.softcap), both[None, None], mixer.sink)
+                    p = p[..., : past + T] + (p[..., past + T:] @ share.t()) * vis
+                else:
+                    p = weights(ref.softcapped(s, m.softcap), seen[None, None], mixer.sink)
+                acc.append(torch.einsum("hgnl,hlv->nhgv", p, V).reshape(T, m.heads, m.vdim))
+            o = acc[0] if m.diff is None else ref.differential(torch.stack(acc, 2), *mixer.differential())
+            return o.reshape(T, m.heads * m.vdim).to(q.dtype)
 
         attn.latent, attn.window = latent, window
         attn.recur = lambda layer, mixer, *inputs: cache.recur(layer, mixer, inputs, bits)

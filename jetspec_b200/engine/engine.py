@@ -29,7 +29,7 @@ from typing import Optional, Sequence
 import torch
 
 from .. import ops
-from ..core.llm import decode_text, resolve_eos
+from ..core.llm import check_positions, decode_text, resolve_eos
 from ..models import is_model, load_target
 from ..runtime import PagedAttention, PagedKVPool, Scheduler, SequenceRequest, build_attn_metadata
 from ..sampling import SamplingParams, sample
@@ -232,6 +232,7 @@ class JetSpecEngine:
         for i in order:
             sid, toks, _ = entries[i]
             have = pool.state(sid).length if pool.has(sid) else 0
+            check_positions(self.cfg, have + len(toks))
             pool.reserve(sid, have + len(toks))
             seqs.append(sid)
             rows.append(torch.tensor(toks, dtype=torch.long, device=self.device))
@@ -281,6 +282,7 @@ class JetSpecEngine:
         sp = sampling_params or SamplingParams()
         ids = self._ids(prompt)
         T = ids.shape[1]
+        check_positions(self.cfg, T + sp.max_new_tokens - 1)
         self._ensure_pool(T + sp.max_new_tokens + 1)
         sid = self._new_seq_id()
         try:
@@ -361,6 +363,7 @@ class JetSpecEngine:
         if max_depth < 0:
             raise ValueError(f"max_tree_depth must be >= 0; got {max_depth}")
         prompt_len = committed.shape[1]
+        check_positions(self.cfg, prompt_len + sp.max_new_tokens - 1)
         D = max(1, block_size - 1)
         ext_budget = int((extend_kwargs or {}).get("ext_budget", D)) if extend_kwargs else 0
         n_max = bucket_for_n(budget + ext_budget)
@@ -510,6 +513,7 @@ class JetSpecEngine:
         """
         sp = sampling_params or SamplingParams()
         id_rows = [self._ids(p)[0] for p in prompts]
+        check_positions(self.cfg, max(int(r.numel()) for r in id_rows) + sp.max_new_tokens - 1)
         longest = max(int(r.numel()) for r in id_rows) + sp.max_new_tokens + 1
         if self.pool is None or self._num_pages is None:
             self._ensure_pool(sum(int(r.numel()) + sp.max_new_tokens + 1 for r in id_rows), seqs=len(prompts))
@@ -614,6 +618,7 @@ class JetSpecEngine:
         """
         sp = sampling_params or SamplingParams()
         id_rows = [self._ids(p)[0] for p in prompts]
+        check_positions(self.cfg, max(int(r.numel()) for r in id_rows) + sp.max_new_tokens - 1)
         D = max(1, block_size - 1)
         n_max = bucket_for_n(budget)
         taps = list(target_layer_ids) if (target_layer_ids is not None and block_size > 1) else None

@@ -775,7 +775,8 @@ class FastRound:
                                            p(r["committed"]), r["committed"].numel(), p(r["eos"]), r["n_eos"],
                                            r["max_new"], p(r["path_idx"]), p(r["result"]), p(status), int(pdl), s()),
                  "js_tree_accept_commit")
-        if pool.states is not None and NB > 1:         # one row is a plain decode step: its states advanced in the forward
+        # one row is a plain decode step: its states advanced, its blocks were pooled in the forward
+        if (pool.states is not None or pool.kv_blocks is not None) and NB > 1:
             n += self.stack.commit(st, pool, r["seq_rows"], r["cu_q"], r["state"][ST_PAST:ST_PAST + 1], r["path_idx"],
                                    r["state"][ST_NEW:ST_NEW + 1], pdl=pdl)
         if remote is not None:

@@ -47,28 +47,33 @@ def split_ws(st, splits: int, rows: int, cols: int):
 
 
 class WindowMixer:
-    """Window attention over K/V pools: one kernel behind the input projections (biases, norms, rotation, cache scatter), then
-    the tcgen05 attention (heads up to 128, groups of up to 16) or the plain-core one; sinks and gates ride in its softmax
-    and epilogue.  ``proj`` are the unpadded q | k | v columns, ``gate`` one fp32 logit per (padded) head."""
+    """Attention over K/V pools, in a window or over the whole past: one kernel behind the input projections (biases, norms,
+    rotation, temperature, cache scatter), the means of blocks that are whole by then where the layer pools blocks, then the
+    tcgen05 attention (heads up to 128, groups of up to 16) or the plain-core one; sinks, gates, capped scores, pooled blocks and
+    the difference of two maps ride in its softmax and epilogue.  ``proj`` are the unpadded q | k | v columns (q | k where the
+    values are the keys, q alone over another layer's), ``gate`` one fp32 logit per (padded) head."""
 
     def __init__(self, m, eps: float, wp: int):
         c = self.cfg = m.cfg
         f32 = lambda p: p.detach().float().contiguous()
         g = c.heads // c.kv_heads
         self.eps = eps
-        self.Dp, self.Vp = window_row_width(c.dim, c.vdim, torch.bfloat16)
+        self.Dp, self.Vp = window_row_width(c.dim, c.vdim, torch.bfloat16, c.maps)
         gp = 1 << (g - 1).bit_length()
-        self.tc = self.Dp == 128 and self.Vp == 128 and gp <= 16        # what the tensor-core kernel takes
-        self.gp, self.Dq, self.vq = (gp, 128, 128) if self.tc else (g, c.dim, c.vdim)
+        # what the tensor-core kernel takes
+        self.tc = self.Dp == 128 and self.Vp == 128 and gp <= 16 and X.window_tc_ok(c.maps, c.pool, c.softcap)
+        self.gp, self.Dq, self.vq = (gp, 128 // c.maps, 128) if self.tc else (g, c.dim, c.vdim)
         self.heads = c.kv_heads * self.gp
-        self.q_cols, self.o_cols = self.heads * self.Dq, up(self.heads * self.vq, 8)
+        self.q_cols, self.o_cols = self.heads * c.maps * self.Dq, up(self.heads * self.vq, 8)
         w = m.o_proj.weight.detach()
         o = torch.zeros(wp, c.kv_heads, self.gp, self.vq, dtype=w.dtype, device=w.device)
         o[: w.shape[0], :, :g, : c.vdim] = w.view(-1, c.kv_heads, g, c.vdim)
         self.w_o = pad(o.view(wp, -1), wp, self.o_cols)
-        self.qkv_bias = torch.cat([f32(p.bias) for p in (m.q_proj, m.k_proj, m.v_proj)]) if c.bias else None
+        projs = [p for p in (m.q_proj, m.k_proj, m.v_proj) if p is not None]
+        self.qkv_bias = torch.cat([f32(p.bias) for p in projs]) if c.bias else None
         self.o_bias = f32(m.o_proj.bias) if m.o_proj.bias is not None else None
-        self.qkv = [p.weight.detach() for p in (m.q_proj, m.k_proj, m.v_proj)]
+        self.qkv = [p.weight.detach() for p in projs]
+        self.v_col = (c.heads + (0 if c.tie_values else c.kv_heads)) * c.maps * c.dim
         self.q_norm, self.k_norm = (f32(m.q_norm), f32(m.k_norm)) if c.proj_norm else (None, None)
         self.freq = X.pair_freq(c.rot_dims, c.rot_base, w.device) if c.rot is None else None
         self.sink, self.gate = c.sink, None
@@ -76,8 +81,11 @@ class WindowMixer:
             self.sink = pad_heads(f32(m.sink_logits).view(-1, 1), c.kv_heads, self.gp, 1).view(-1).contiguous()
         if c.gate:
             self.gate = pad_heads(m.gate_proj.weight.detach(), c.kv_heads, self.gp, m.gate_proj.weight.shape[1])
+        self.diff = m.differential()
+        if self.diff is not None:
+            self.diff = (self.diff[0].detach().reshape(1).contiguous(), *self.diff[1:])
 
-    def run(self, st, pool, batch, proj, gate, rot, pdl: bool, first_pdl: bool):
+    def run(self, st, pool, batch, proj, gate, rot, pdl: bool, first_pdl: bool, blocks=None):
         """Returns the attention output ``(T, o_cols)`` and the number of kernels launched."""
         c, T = self.cfg, st.T
         lib, p = X.load(), X._p
@@ -86,9 +94,10 @@ class WindowMixer:
         status = p(X.status_word(kp.device))
         if c.rot is None:
             X._check(lib.js_window_post(
-                p(proj), proj.stride(0), p(self.qkv_bias), c.heads, c.kv_heads, self.gp, c.dim, c.vdim, self.Dq, self.Dp, self.Vp, c.rot_dims,
-                p(self.freq), int(c.qk_norm), X.ctypes.c_float(self.eps), p(batch.positions), p(batch.slots), kp.shape[1], T, p(q), p(kp),
-                p(vp), status, int(first_pdl), X._stream()), "js_window_post")
+                p(proj), proj.stride(0), p(self.qkv_bias), c.heads, c.kv_heads, self.gp, c.maps, c.dim, c.vdim, self.Dq, self.Dp, self.Vp,
+                c.rot_dims, p(self.freq), int(c.qk_norm), X.ctypes.c_float(self.eps), c.temp_every, X.ctypes.c_float(c.temp_coef), self.v_col,
+                int(c.kv_from is None), p(batch.positions), p(batch.slots), kp.shape[1], T, p(q), p(kp), p(vp), status, int(first_pdl),
+                X._stream()), "js_window_post")
         else:
             X._check(lib.js_attn_post(
                 p(proj), proj.stride(0), p(self.qkv_bias), p(self.q_norm), p(self.k_norm), c.heads, c.kv_heads, self.gp, c.dim, c.vdim, self.Dq,
@@ -96,15 +105,23 @@ class WindowMixer:
                 p(batch.slots), kp.shape[1], T, p(q), p(kp), p(vp), status, int(first_pdl), X._stream()), "js_attn_post")
         o = st.get("wo", self.o_cols, zero=True)
         Hq, n = self.heads, 2
+        if blocks is not None and batch.mask is None:        # rows of a token tree are not committed yet
+            X.pool_blocks(kp, vp, *blocks, batch.slot_map, batch.seq_rows, batch.cu_q, batch.past, rows=T, pdl=pdl)
+            n += 1
         args = (batch.slot_map, batch.seq_rows, batch.cu_q, batch.past, batch.mask)
-        if self.tc and (batch.mask is None or batch.mask.shape[1] <= 8):
-            splits = X.window_attn_splits(T, Hq, c.kv_heads, batch.max_keys, c.window, c.keep_first)
+        more = dict(keep_first=c.keep_first, gate=gate)
+        if c.softcap or blocks is not None or self.diff is not None:
+            more.update(softcap=c.softcap, blocks=blocks, diff=self.diff)
+        # a token tree deeper than the window would see blocks of its own nodes, which only the plain-core kernel makes
+        shallow = batch.mask is None or (batch.mask.shape[1] <= 8 and (blocks is None or c.window >= batch.max_rows))
+        if self.tc and shallow:
+            splits = X.window_attn_splits(T, Hq, c.kv_heads, batch.max_keys, c.window, c.keep_first, c.pool)
             X.window_attention_tc(q.view(T, Hq, 128), kp, vp, *args, c.scale, c.window, self.sink, batch.mask is None, o, splits=splits,
-                                  ws=split_ws(st, splits, T * Hq, 128), pdl=pdl, keep_first=c.keep_first, gate=gate)
+                                  ws=split_ws(st, splits, T * Hq * c.maps, 128), pdl=pdl, **more)
             n += int(splits > 1 and not X.attn_merges_in_cluster(T, Hq, c.kv_heads, splits))
         else:
-            X.window_attention(q.view(T, Hq, self.Dq), kp, vp, self.vq, *args, c.scale, c.window, self.sink, batch.mask is None, out=o,
-                               pdl=pdl, keep_first=c.keep_first, gate=gate)
+            X.window_attention(q.view(T, Hq * c.maps, self.Dq), kp, vp, self.vq, *args, c.scale, c.window, self.sink, batch.mask is None, out=o,
+                               pdl=pdl, **more)
         return o, n
 
 

@@ -1,5 +1,5 @@
-"""Fused kernel form of a pre-norm decoder whose layers hold window attention, latent attention or retention in any order
-(Kizezen) for the engine's kernel path.
+"""Fused kernel form of a pre-norm decoder whose layers hold attention over K/V heads, latent attention or retention in any
+order (Kizezen, Sogidra) for the engine's kernel path.
 
 Per layer, on ``h``, the bf16 norm of the fp32 residual stream ``x``:
 
@@ -7,13 +7,17 @@ Per layer, on ``h``, the bf16 norm of the fp32 residual stream ``x``:
 2. the mixer (:mod:`~jetspec_b200.engine.mixers`): one kernel behind the projections and the attention with sinks and gates
    folded in, or the retention kernels;
 3. the output GEMM adds to the stream, one kernel norms it;
-4. feed-forward: up GEMM with the exact gelu in its epilogue, down GEMM that adds to the stream, the next norm (behind the
-   last layer the model's final one).
+4. feed-forward: up GEMM with the activation (exact gelu, xIELU) in its epilogue, down GEMM that adds to the stream, the next
+   norm (behind the last layer the model's final one).
 
-The embedding kernel norms its rows for the first layer and makes the (cos, sin) tables of all layers' rotations.
+Where sublayers have a norm on their output too, the output GEMM leaves bf16 rows and ONE kernel norms them, adds them to the
+stream and norms the sum; at a layer's end it also keeps the layer's result and makes the weighted sum over the depth.
 
-Token trees leave the recurrent states alone and keep every retention layer's projections; :meth:`PreNormStack.commit` then
-advances the states along the accepted nodes.
+The embedding kernel adds learned positions, norms its rows for the first layer and makes the (cos, sin) tables of all layers'
+rotations.
+
+Token trees leave the recurrent states alone and keep every retention layer's projections, and pool no blocks;
+:meth:`PreNormStack.commit` then advances the states along the accepted nodes and pools the blocks they complete.
 """
 from __future__ import annotations
 
@@ -22,6 +26,7 @@ import types
 import torch
 
 from ..models.config import LatentAttentionConfig, WindowAttentionConfig
+from ..models.layers import XieluMLP
 from ..ops import cuda_ext as X
 from .latent_stack import latent_part, latent_parts
 from .mixers import LatentMixer, RetentionMixer, WindowMixer, pad, pad_heads, up
@@ -35,7 +40,9 @@ class _LayerWeights:
         f32 = lambda p: p.detach().float().contiguous()
         self.index, self.eps, self.rot_at = i, eps, 0
         self.kind, raw = cfg.layers[i].mixer_type, []
+        row = lambda n: pad(n.scale().detach().view(1, -1), 1, wp).view(-1)
         if isinstance(c, WindowAttentionConfig):
+            self.kind = "attention"
             self.mix = WindowMixer(mix, eps, wp)
             act = torch.cat(self.mix.qkv, 0)                   # read as unpadded rows
             raw = [self.mix.gate] if c.gate else []
@@ -57,13 +64,16 @@ class _LayerWeights:
         self.act_cols = up(act.shape[0], 128)
         blocks = [pad(torch.cat(raw, 0), self.n_raw, wp)] if raw else []
         self.w_in = torch.cat(blocks + [pad(act, self.act_cols, wp)], 0)
-        self.norm1 = pad(f32(layer.norm1.weight).view(1, -1), 1, wp).view(-1)
-        self.ff = 0
+        self.norm1, self.ff = row(layer.norm1), 0
+        self.out1 = row(layer.norm1b) if hasattr(layer, "norm1b") else None      # norms on the sublayers' outputs
+        self.depth = f32(layer.dwa) if hasattr(layer, "dwa") else None
         if layer.mlp is not None:
             self.ff = up(layer.mlp.up_proj.weight.shape[0], 128)
             self.w_up = pad(layer.mlp.up_proj.weight.detach(), self.ff, wp)
             self.w_down = pad(layer.mlp.down_proj.weight.detach(), wp, self.ff)
-            self.norm2 = pad(f32(layer.norm2.weight).view(1, -1), 1, wp).view(-1)
+            self.norm2 = row(layer.norm2)
+            self.out2 = row(layer.norm2b) if self.out1 is not None else None
+            self.act = dict(act=X.ACT_XIELU, act_args=layer.mlp.coefficients()) if isinstance(layer.mlp, XieluMLP) else dict(act=X.ACT_GELU_ERF)
 
 
 class PreNormStack:
@@ -74,10 +84,14 @@ class PreNormStack:
         self.cfg, self.device = cfg, torch.device(device)
         self.width, self.wp = cfg.hidden_size, up(cfg.hidden_size, 8)
         self.layers = [_LayerWeights(l, cfg, i, self.wp) for i, l in enumerate(model.model.layers)]
-        self.final_norm = pad(model.model.norm.weight.detach().float().view(1, -1), 1, self.wp).view(-1)
+        self.final_norm = pad(model.model.norm.scale().detach().view(1, -1), 1, self.wp).view(-1)
         table, head = model.model.embed_tokens.weight.detach(), model.lm_head.weight.detach()
         self.table, self.head = (w if self.wp == self.width else pad(w, w.shape[0], self.wp) for w in (table, head))
+        pos = getattr(model.model, "pos_embed", None)
+        self.pos_table = pad(pos.weight.detach(), pos.weight.shape[0], self.wp) if pos is not None else None
         self.vocab, self.embed_scale = cfg.vocab_size, float(cfg.embed_scale)
+        self.depth = self.layers[0].depth is not None
+        self.pooled = [L for L in self.layers if getattr(L.mix.cfg, "pool", 0)]
         self._rotations()
         self.recurrent = [L for L in self.layers if L.kind == "retention"]
         self.may_expand = any(L.kind == "latent_attention" and L.mix.expand for L in self.layers)
@@ -114,6 +128,8 @@ class PreNormStack:
         b = types.SimpleNamespace(T=T, max_keys=max_keys, cols=cols, ws={})
         b.x = torch.zeros(T, self.wp, dtype=torch.float32, device=dev)
         b.h = torch.zeros(T, self.wp, dtype=torch.bfloat16, device=dev)
+        # embedding output and every layer's result
+        b.hist = torch.empty(len(self.layers) + 1, T, self.wp, dtype=torch.float32, device=dev) if self.depth else None
         b.rot = torch.zeros(T, self.n_freq, 2, dtype=torch.float32, device=dev)
 
         def get(name, c, dtype=torch.bfloat16, rows=T, zero=False):
@@ -138,8 +154,9 @@ class PreNormStack:
         lib, p = X.load(), X._p
         T, n, last = st.T, 1, len(self.layers) - 1
         X._check(lib.js_embed_rms(p(ids), p(self.table), self.vocab, self.table.stride(0), X.ctypes.c_float(self.embed_scale),
-                                  p(self.layers[0].norm1), X.ctypes.c_float(self.layers[0].eps), p(st.x), p(st.h), self.wp, T, self.width,
-                                  p(batch.positions), p(self.freq), p(self.amp), self.n_freq, p(st.rot), int(pdl), X._stream()),
+                                  p(self.layers[0].norm1), X.ctypes.c_float(self.layers[0].eps), p(st.x if not self.depth else st.hist[0]), p(st.h),
+                                  self.wp, T, self.width, p(batch.positions), p(self.pos_table),
+                                  self.pos_table.shape[0] if self.pos_table is not None else 0, p(self.freq), p(self.amp), self.n_freq, p(st.rot), int(pdl), X._stream()),
                  "js_embed_rms")
         tap_ids = list(tap_ids) if taps is not None else []
         for i, L in enumerate(self.layers):
@@ -171,11 +188,13 @@ class PreNormStack:
         gate = raw[:, L.gate_at:] if L.gated else None
         rot = self._rot(st, L)
         if L.kind == "attention":
-            o, n = L.mix.run(st, pool.layer(L.index), batch, act, gate, rot, pdl, pdl)
+            o, n = L.mix.run(st, pool.layer(L.index), batch, act, gate, rot, pdl, pdl, blocks=pool.blocks(L.index))
         elif L.kind == "latent_attention":
             o, n = self._latent(st, L, pool.latent(L.index), batch, raw, act, gate, rot, pdl)
         else:
             o, n = L.mix.run(st, pool.states.layer(L.index)[0], batch, act, rot, pdl)
+        if L.out1 is not None:
+            return n + self._normed(st, L, o, norm, h, tap, pdl)
         X.gemm_resid32(o, L.w_o, st.x, pdl=pdl)
         n += 3
         if not L.ff:
@@ -183,10 +202,26 @@ class PreNormStack:
             return n
         self._norm(st, L.norm2, L.eps, st.h, None, pdl)
         a = st.get("ff", L.ff)
-        X.gemm_inproj(st.h, L.w_up, None, 0, a, False, pdl=pdl, act=X.ACT_GELU_ERF)
+        X.gemm_inproj(st.h, L.w_up, None, 0, a, False, pdl=pdl, **L.act)
         X.gemm_resid32(a, L.w_down, st.x, pdl=pdl)
         self._norm(st, norm, L.eps, h, tap, pdl)
         return n + 3
+
+    def _normed(self, st, L, o, norm, h, tap, pdl) -> int:
+        """What follows the mixer where sublayers have norms on their outputs.  Returns the launches, the input GEMM's included."""
+        y = st.get("y", self.wp)
+        X.gemm(o, L.w_o, out=y, pdl=pdl)
+        x = st.hist[0] if self.depth and L.index == 0 else st.x        # the embedding output stays as it is
+        end = dict(hist=st.hist, d=L.depth, tap=tap, pdl=pdl)
+        if not L.ff:
+            X.sandwich(y, x, L.out1, st.x, norm, L.eps, h, self.width, **end)
+            return 3
+        X.sandwich(y, x, L.out1, st.x, L.norm2, L.eps, st.h, self.width, pdl=pdl)
+        a = st.get("ff", L.ff)
+        X.gemm_inproj(st.h, L.w_up, None, 0, a, False, pdl=pdl, **L.act)
+        X.gemm(a, L.w_down, out=y, pdl=pdl)
+        X.sandwich(y, st.x, L.out2, st.x, norm, L.eps, h, self.width, **end)
+        return 6
 
     def _latent(self, st, L, pool, batch, raw, act, gate, rot, pdl):
         m, c, p = L.mix, L.mix.cfg, X._p
@@ -200,11 +235,14 @@ class PreNormStack:
 
     # ------------------------------------------------------------------ token trees
     def commit(self, st, pool, state_rows, cu_q, past, path, path_len, pdl: bool = True) -> int:
-        """Advance one sequence's states along the rows ``path[:path_len]`` (device) of the tree forward run on ``st``;
-        ``past`` is the committed length behind the path."""
+        """Advance one sequence's states along the rows ``path[:path_len]`` (device) of the tree forward run on ``st`` and pool the
+        blocks they complete; ``past`` is the committed length behind the path."""
+        for L in self.pooled:
+            X.pool_blocks(*pool.layer(L.index), *pool.blocks(L.index), pool.slot_map, state_rows, None, past, counts=path_len,
+                          most=path.numel(), pdl=pdl)
         for L in self.recurrent:
             L.mix.advance(self._act(st, L, True), self._rot(st, L), pool.states.layer(L.index)[0], state_rows, cu_q, past, path, path_len, pdl)
-        return len(self.recurrent)
+        return len(self.recurrent) + len(self.pooled)
 
     def hold_trees(self, st, pool, rows, starts, nodes: int) -> None:
         """Register the tree forward on ``st`` with the state pool: the tree of state slot ``rows[j]`` begins at row

@@ -1,4 +1,4 @@
-"""Model configurations read from ``config.json``: Qwen3 (Hugging Face layout), Karuzen, Zasipel and Kizezen.
+"""Model configurations read from ``config.json``: Qwen3 (Hugging Face layout), Karuzen, Zasipel, Kizezen and Sogidra.
 
 Only the fields the decoder actually uses are kept.  The draft head adds
 ``block_size``, ``num_target_layers`` and ``dflash_config`` on top of the Qwen3
@@ -9,7 +9,9 @@ What the engines, the cache and the kernel path ask of a configuration, whatever
 ``kernel_path_ok()``, ``kernel_stack()`` (which fused launch sequence runs the decoder, ``None`` for Qwen3's) and what a cache
 layer holds: ``latent_widths()`` (width of a latent row, ``None`` where a layer caches none, or ``None`` for a model without),
 ``kv_shapes()`` (likewise; ``None`` when all layers hold the same K and V heads) and ``state_shapes()`` (``None`` without
-recurrent layers).
+recurrent layers).  Optional, for caches of K and V heads: ``kv_sources()`` (per layer, the layer whose keys and values it
+reads) and ``kv_pools()`` (per layer, tokens to a pooled block, 0 without).  A model whose positions are a learned table has
+``max_positions``.
 """
 from __future__ import annotations
 
@@ -303,9 +305,10 @@ class KaruzenConfig:
 
 @dataclass
 class WindowAttentionConfig:
-    """Sizes and constants of a sliding-window attention over grouped K/V heads: a token sees itself and the
-    ``window - 1`` tokens before it, and the sequence's first ``keep_first`` tokens; the first ``rot_dims`` dimensions are
-    rotated in neighbouring pairs, or as ``rot`` says."""
+    """Sizes and constants of an attention over grouped K/V heads, in a sliding window or over the whole past: a token sees
+    itself and the ``window - 1`` tokens before it (``window`` 0: all of them), the sequence's first ``keep_first`` tokens, and
+    with ``pool`` one key and value for each whole block of that many tokens behind the window, the means over the block.
+    The first ``rot_dims`` dimensions are rotated in neighbouring pairs, or as ``rot`` says."""
     heads: int
     kv_heads: int
     dim: int
@@ -323,6 +326,18 @@ class WindowAttentionConfig:
     o_bias: Optional[bool] = None    # bias on the output projection; None: as ``bias``
     gate: bool = False               # sigmoid gate per head on the output
     rot: Optional[RotaryConfig] = None
+    pool: int = 0
+    softcap: float = 0.0             # > 0: scores pass through softcap * tanh(score / softcap)
+    tie_values: bool = False         # the values are the keys as projected, ahead of norm and rotation
+    diff: Optional[float] = None     # differential attention: two maps a head over the same values, a1 - lambda a2 normed
+    temp_every: int = 0              # > 0: q is multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
+    temp_coef: float = 0.0
+    kv_from: Optional[int] = None    # no keys and values of its own: those of this layer
+
+    @property
+    def maps(self) -> int:
+        """Attention maps of a head; q and k carry one vector for each."""
+        return 2 if self.diff is not None else 1
 
 
 @dataclass
@@ -631,6 +646,125 @@ class KizezenConfig:
             json.dump(self.to_dict(), f, indent=1)
 
 
+@dataclass
+class SogidraLayerConfig:
+    mixer: WindowAttentionConfig
+    ff: int = 0                      # width of the feed-forward, 0 without one
+
+    @property
+    def mixer_type(self) -> str:
+        return "attention" if self.mixer.diff is not None else "attention_2"
+
+
+@dataclass
+class SogidraConfig:
+    """Sogidra: differential attention over the whole past and window attention with pooled blocks, in any order, keys and
+    values shared between layers; norms before and after every sublayer; a weighted average over the depth behind every layer;
+    learned positions; tied head."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    max_positions: int
+    norm_eps: float = 1e-6
+    eos_token_id: Any = None
+    model_type: str = "sogidra"
+    logit_scale = embed_scale = 1.0                 # not fields: fixed by the design
+    is_moe = False
+
+    @property
+    def num_hidden_layers(self) -> int:
+        return len(self.layers)
+
+    def latent_widths(self) -> None:
+        return None
+
+    def kv_shapes(self) -> list:
+        return [(m.kv_heads, m.dim, m.vdim, m.maps) if m.kv_from is None else None for m in (l.mixer for l in self.layers)]
+
+    def kv_sources(self) -> list:
+        return [i if l.mixer.kv_from is None else l.mixer.kv_from for i, l in enumerate(self.layers)]
+
+    def kv_pools(self) -> list:
+        return [l.mixer.pool for l in self.layers]
+
+    def state_shapes(self) -> None:
+        return None
+
+    def kernel_path_ok(self) -> bool:
+        return self.hidden_size <= 32768 and all(l.mixer.dim <= 512 and l.mixer.vdim <= 512 for l in self.layers)
+
+    def kernel_stack(self) -> str:
+        return "prenorm"
+
+    # -- io -------------------------------------------------------------------
+    @classmethod
+    def from_dict(cls, d: dict) -> "SogidraConfig":
+        def mixer(i, t, m):
+            size = {k: int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim")}
+            if size["heads"] % size["kv_heads"]:
+                raise ValueError(f"layer {i}: {m['heads']} heads do not divide over {m['kv_heads']} key heads")
+            common = dict(**size, scale=float(m["scale"]), rot_dims=0, rot_base=1.0, sink=False, o_bias=False)
+            if t == "attention":
+                temp, src = m.get("q_temp") or {}, m.get("kv_from")
+                return WindowAttentionConfig(**common, window=0, qk_norm=False, bias=True, diff=float(m["diff"]),
+                                             temp_every=int(temp.get("every", 0)), temp_coef=float(temp.get("coef", 0.0)),
+                                             kv_from=int(src) if src is not None else None)
+            if t == "attention_2":
+                if size["dim"] != size["vdim"]:
+                    raise ValueError(f"layer {i}: values are keys, but heads have {m['dim']} and {m['vdim']} entries")
+                if int(m["mask"]["size"]) < 1 or int(m["mask"]["pool"]) < 1:
+                    raise ValueError(f"layer {i}: mask {m['mask']}")
+                return WindowAttentionConfig(**common, window=int(m["mask"]["size"]), pool=int(m["mask"]["pool"]), qk_norm=True, bias=False,
+                                             tie_values=True, softcap=float(m["softcap"]))
+            raise ValueError(f"layer {i}: unknown mixer type {t!r}")
+
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            f = e.get("mlp")
+            if f is not None and f["kind"] != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {f['kind']!r}")
+            layers.append(SogidraLayerConfig(mixer(i, e["type"], e["mixer"]), ff=int(f["ff"]) if f is not None else 0))
+        for i, l in enumerate(layers):
+            m = l.mixer
+            if m.kv_from is None:
+                continue
+            src = layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
+            if src is None or src.diff is None or src.kv_from is not None or (src.kv_heads, src.dim, src.vdim) != (m.kv_heads, m.dim, m.vdim):
+                raise ValueError(f"layer {i} cannot use the keys and values of layer {m.kv_from}")
+        return cls(vocab_size=int(d["vocab"]), hidden_size=int(d["width"]), layers=layers, max_positions=int(d["max_positions"]),
+                   norm_eps=float(d["norm"]["eps"]), eos_token_id=d.get("eos_token_id"))
+
+    @classmethod
+    def from_pretrained(cls, path: str, subfolder: str = "") -> "SogidraConfig":
+        with open(os.path.join(path, subfolder, "config.json") if subfolder else os.path.join(path, "config.json")) as f:
+            return cls.from_dict(json.load(f))
+
+    def to_dict(self) -> dict:
+        layers = []
+        for l in self.layers:
+            m = l.mixer
+            mixer = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale}
+            if m.diff is not None:
+                mixer["diff"] = m.diff
+                if m.temp_every:
+                    mixer["q_temp"] = {"every": m.temp_every, "coef": m.temp_coef}
+                if m.kv_from is not None:
+                    mixer["kv_from"] = m.kv_from
+            else:
+                mixer.update(softcap=m.softcap, mask={"size": m.window, "pool": m.pool})
+            layers.append({"type": l.mixer_type, "mixer": mixer, "mlp": {"kind": "dense", "ff": l.ff} if l.ff else None})
+        d = {"architecture": "Sogidra", "vocab": self.vocab_size, "width": self.hidden_size, "layers": layers,
+             "norm": {"eps": self.norm_eps}, "max_positions": self.max_positions}
+        if self.eos_token_id is not None:
+            d["eos_token_id"] = self.eos_token_id
+        return d
+
+    def save_pretrained(self, path: str) -> None:
+        os.makedirs(path, exist_ok=True)
+        with open(os.path.join(path, "config.json"), "w") as f:
+            json.dump(self.to_dict(), f, indent=1)
+
+
 # Geometry presets used by the tests and the benchmarks (random-init weights).
 def tiny_config(**over) -> Qwen3Config:
     """2 layers, hidden 256, 4 q / 2 kv heads, head_dim 64, SwiGLU 512, vocab 1024."""
@@ -704,6 +838,23 @@ def kizezen_tiny_config(**over) -> KizezenConfig:
         KizezenLayerConfig(lat, 120), KizezenLayerConfig(win(9, 0, RotaryConfig(24, 5e3)))])
     kw.update(over)
     return KizezenConfig(**kw)
+
+
+def sogidra_tiny_config(**over) -> SogidraConfig:
+    """4 layers (pooled window, differential, pooled window without a feed-forward, differential on the second layer's keys);
+    width 136."""
+    def diff(**kw):
+        return WindowAttentionConfig(heads=4, kv_heads=2, dim=20, vdim=36, window=0, rot_dims=0, rot_base=1.0, scale=0.25, sink=False,
+                                     qk_norm=False, bias=True, o_bias=False, diff=0.4, temp_every=16, temp_coef=0.3, **kw)
+
+    def pooled(window, pool):
+        return WindowAttentionConfig(heads=6, kv_heads=2, dim=28, vdim=28, window=window, rot_dims=0, rot_base=1.0, scale=0.4, sink=False,
+                                     qk_norm=True, bias=False, o_bias=False, tie_values=True, softcap=20.0, pool=pool)
+    kw = dict(vocab_size=320, hidden_size=136, max_positions=512, norm_eps=1e-5, layers=[
+        SogidraLayerConfig(pooled(21, 5), 168), SogidraLayerConfig(diff(), 200), SogidraLayerConfig(pooled(9, 8)),
+        SogidraLayerConfig(diff(kv_from=1), 120)])
+    kw.update(over)
+    return SogidraConfig(**kw)
 
 
 def draft_head_config(target: Qwen3Config, num_layers: int = 1, block_size: int = 16,

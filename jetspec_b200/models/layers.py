@@ -1,5 +1,6 @@
-"""Building blocks that are not Qwen3's: Dynamic Tanh, latent attention, GELU MLPs, sigmoid-routed experts; window
-attention with sinks, gated delta rules, retention, two mixers side by side, table-routed experts.
+"""Building blocks that are not Qwen3's: Dynamic Tanh, latent attention, GELU and xIELU MLPs, sigmoid-routed experts; attention
+in a window, with sinks, with pooled blocks or differential, gated delta rules, retention, two mixers side by side, table-routed
+experts.
 
 Each takes its sizes and constants as arguments, so a design can combine them freely; the Qwen3 twins (RMSNorm, grouped
 query attention, SwiGLU MLP, softmax-routed experts) are in :mod:`jetspec_b200.models.qwen3`.  ``forward`` is the
@@ -100,6 +101,28 @@ class GeluErfMLP(nn.Module):
         return ops.linear(ops.gelu_erf(ops.linear(h, self.up_proj.weight)), self.down_proj.weight)
 
 
+class XieluMLP(nn.Module):
+    """``down(xielu(up(h)))``; the activation's two learned numbers ``act`` pass through a softplus."""
+
+    def __init__(self, hidden: int, inter: int):
+        super().__init__()
+        self.up_proj = nn.Linear(hidden, inter, bias=False)
+        self.down_proj = nn.Linear(inter, hidden, bias=False)
+        self.act = nn.Parameter(torch.zeros(2))
+        self._coef = None
+
+    def coefficients(self) -> tuple:
+        """Factors of the quadratic and of the exponential part, as host numbers (read once per parameter value)."""
+        key = (self.act.data_ptr(), self.act._version)
+        if self._coef is None or self._coef[0] != key:
+            up, down = torch.nn.functional.softplus(self.act.detach().double().cpu()).tolist()
+            self._coef = (key, (up, 0.5 + down))
+        return self._coef[1]
+
+    def forward(self, h):
+        return ops.linear(ops.xielu(ops.linear(h, self.up_proj.weight), *self.coefficients()), self.down_proj.weight)
+
+
 class SigmoidMoE(nn.Module):
     """Experts chosen by ``sigmoid(router(h)) + correction`` and weighted by the normalised sigmoid without it; expert =
     ``down(relu(up(h))^2)``.  A shared expert of the same form, gated by ``sigmoid(shared_gate(h))``, is added."""
@@ -134,30 +157,60 @@ class PlainRMSNorm(nn.Module):
         self.eps = eps
         self.weight = nn.Parameter(torch.ones(dim))
 
+    def scale(self):
+        """What the normed rows are multiplied by, fp32."""
+        return self.weight.float()
+
     def forward(self, x):
         return ops.rmsnorm_f32(x, self.weight, self.eps)
 
 
-class WindowAttention(nn.Module):
-    """Sliding-window attention over grouped K/V heads.  Options (see the configuration): rotation in neighbouring or half
-    pairs, norm of q and k per head behind it or over the whole projections ahead of it, kept first tokens, a valueless
-    sink of score 0 or a learned one per head, a sigmoid gate per head, biases.
+class OffsetRMSNorm(PlainRMSNorm):
+    """:class:`PlainRMSNorm` whose weight is stored as its distance from one."""
 
-    ``forward(h, positions, attend)``: ``attend(q, k, v)`` stores the new K/V rows and returns the attention,
-    ``(T, heads * vdim)``."""
+    def __init__(self, dim: int, eps: float):
+        super().__init__(dim, eps)
+        nn.init.zeros_(self.weight)
+
+    def scale(self):
+        return self.weight.float() + 1.0
+
+    def forward(self, x):
+        return ops.rmsnorm_f32(x, self.scale(), self.eps)
+
+
+class WindowAttention(nn.Module):
+    """Attention over grouped K/V heads, in a sliding window or over the whole past.  Options (see the configuration): rotation
+    in neighbouring or half pairs, norm of q and k per head behind it or over the whole projections ahead of it, kept first
+    tokens, pooled blocks behind the window, a valueless sink of score 0 or a learned one per head, capped scores, two
+    attention maps a head whose difference counts, a temperature that grows with the position, values that are the keys,
+    keys and values of another layer, a sigmoid gate per head, biases.
+
+    ``forward(h, positions, attend)``: ``attend(q, k, v)`` stores the new K/V rows (``None`` for both: there are none) and
+    returns the attention, ``(T, heads * vdim)``."""
 
     def __init__(self, cfg: WindowAttentionConfig, hidden: int, eps: float):
         super().__init__()
         self.cfg, self.eps = cfg, eps
         lin = lambda i, o: nn.Linear(i, o, bias=cfg.bias)
-        self.q_proj, self.k_proj = lin(hidden, cfg.heads * cfg.dim), lin(hidden, cfg.kv_heads * cfg.dim)
-        self.v_proj = lin(hidden, cfg.kv_heads * cfg.vdim)
+        self.q_proj = lin(hidden, cfg.heads * cfg.maps * cfg.dim)
+        self.k_proj = lin(hidden, cfg.kv_heads * cfg.maps * cfg.dim) if cfg.kv_from is None else None
+        self.v_proj = lin(hidden, cfg.kv_heads * cfg.vdim) if cfg.kv_from is None and not cfg.tie_values else None
         self.o_proj = nn.Linear(cfg.heads * cfg.vdim, hidden, bias=cfg.bias if cfg.o_bias is None else cfg.o_bias)
         if cfg.proj_norm:
             self.q_norm, self.k_norm = nn.Parameter(torch.ones(cfg.heads * cfg.dim)), nn.Parameter(torch.ones(cfg.kv_heads * cfg.dim))
         self.sink_logits = nn.Parameter(torch.zeros(cfg.heads)) if cfg.sink_logits else None
         if cfg.gate:
             self.gate_proj = nn.Linear(hidden, cfg.heads, bias=False)
+        if cfg.diff is not None:
+            self.lq1, self.lk1, self.lq2, self.lk2 = (nn.Parameter(torch.zeros(cfg.dim)) for _ in range(4))
+
+    def differential(self):
+        """``(lambda, share, eps)`` of :func:`ops.reference.differential`; ``None`` with one map a head."""
+        if self.cfg.diff is None:
+            return None
+        dot = lambda a, b: torch.exp((a.float() * b.float()).sum())
+        return dot(self.lq1, self.lk1) - dot(self.lq2, self.lk2) + self.cfg.diff, 1.0 - self.cfg.diff, self.eps
 
     @property
     def sink(self):
@@ -166,15 +219,23 @@ class WindowAttention(nn.Module):
 
     def forward(self, h, positions, attend):
         c, T = self.cfg, h.shape[0]
-        q, k, v = (ops.linear(h, p.weight, p.bias) for p in (self.q_proj, self.k_proj, self.v_proj))
+        q, k, v = (ops.linear(h, p.weight, p.bias) if p is not None else None for p in (self.q_proj, self.k_proj, self.v_proj))
+        if c.tie_values:
+            v = k
         if c.proj_norm:
             q, k = ops.rmsnorm(q, self.q_norm, self.eps), ops.rmsnorm(k, self.k_norm, self.eps)
-        q, k = q.view(T, c.heads, c.dim), k.view(T, c.kv_heads, c.dim)
-        if c.rot is not None:
-            q, k = ops.rotate(q, positions, c.rot), ops.rotate(k, positions, c.rot)
-        else:
-            q, k = (ops.rotate_norm(x, positions, c.rot_dims, c.rot_base, self.eps if c.qk_norm else None) for x in (q, k))
-        y = attend(q, k, v.view(T, c.kv_heads, c.vdim))
+
+        def turn(x, heads):
+            x = x.view(T, heads, c.dim)
+            if c.rot is not None:
+                return ops.rotate(x, positions, c.rot)
+            return ops.rotate_norm(x, positions, c.rot_dims, c.rot_base, self.eps if c.qk_norm else None)
+        q = turn(q, c.heads * c.maps)
+        if c.temp_every:
+            q = ops.query_temperature(q, positions, c.temp_every, c.temp_coef)
+        if k is not None:
+            k, v = turn(k, c.kv_heads * c.maps).reshape(T, c.kv_heads, c.maps * c.dim), v.view(T, c.kv_heads, c.vdim)
+        y = attend(q, k, v)
         if c.gate:
             y = ops.head_gate(y, ops.linear_f32(h, self.gate_proj.weight))
         return ops.linear(y, self.o_proj.weight, self.o_proj.bias)

@@ -126,17 +126,40 @@ def rotate_norm(x, positions, dims, base, eps):
     return ref.rotate_norm(x, positions, dims, base, eps)
 
 
-def window_scatter(k, v, k_pool, v_pool, slots):
-    return ref.window_scatter(k, v, k_pool, v_pool, slots)
+def window_scatter(k, v, k_pool, v_pool, slots, maps: int = 1):
+    return ref.window_scatter(k, v, k_pool, v_pool, slots, maps)
+
+
+def pool_blocks(k_pool, v_pool, kb_pool, vb_pool, block_map, P, slot_map, seq_rows, cu_q, past_lens):
+    if _kern_any(k_pool):
+        return _ext().pool_blocks(k_pool, v_pool, kb_pool, vb_pool, block_map, int(P), slot_map, seq_rows, cu_q, past_lens)
+    return ref.pool_blocks(k_pool, v_pool, kb_pool, vb_pool, block_map, P, slot_map, seq_rows, cu_q, past_lens)
 
 
 def window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, window, sink,
-                     causal: bool = False, keep_first: int = 0):
+                     causal: bool = False, keep_first: int = 0, softcap: float = 0.0, blocks=None, diff=None):
     if _kern_any(q) and max(q.shape[-1], vdim) <= 512:
         return _ext().window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, float(scale),
-                                       int(window), sink, bool(causal), keep_first=int(keep_first))
+                                       int(window), sink, bool(causal), keep_first=int(keep_first), softcap=float(softcap),
+                                       blocks=blocks, diff=diff)
     return ref.window_attention(q, k_pool, v_pool, vdim, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale, window, sink,
-                                causal, keep_first)
+                                causal, keep_first, softcap, blocks, diff)
+
+
+def query_temperature(x, positions, every, coef):
+    return ref.query_temperature(x, positions, every, coef)
+
+
+def depth_average(history, weights):
+    if history[0].is_cuda and history[0].dtype == torch.float32:
+        return _ext().depth_average(history, weights)
+    return ref.depth_average(history, weights)
+
+
+def xielu(x, up: float, down: float):
+    if _kern_any(x):
+        return _ext().xielu(x, up, down)
+    return ref.xielu(x, up, down)
 
 
 def gelu_erf(x):
@@ -235,6 +258,6 @@ __all__ = [
     "paged_tree_attention", "lm_head_argmax", "lm_head_topk_logprobs", "moe_forward",
     "dynamic_tanh", "gelu_tanh_mul", "relu_squared", "latent_scatter", "latent_attention", "sigmoid_moe",
     "rmsnorm_f32", "linear_f32", "rotate_norm", "window_scatter", "window_attention", "delta_mix", "gated_head_norm",
-    "experts_swiglu", "gelu_erf", "rotate", "head_gate", "retention",
+    "experts_swiglu", "pool_blocks", "query_temperature", "depth_average", "xielu", "gelu_erf", "rotate", "head_gate", "retention",
     "pack_ancestor_bits", "unpack_ancestor_bits", "rope_cos_sin", "apply_rope", "moe_route", "sample",
 ]

@@ -206,7 +206,7 @@ def inv_freq(head_dim: int, theta: float, device) -> torch.Tensor:
 # ------------------------------------------------------------------ GEMM
 EPI_STORE, EPI_SWIGLU, EPI_ARGMAX, EPI_TOPK, EPI_STORE_F32 = 0, 1, 2, 3, 4
 EPI_RELU2 = 8
-ACT_GELU_GLU, ACT_RELU2, ACT_NONE, ACT_GELU_ERF = 0, 1, 2, 3
+ACT_GELU_GLU, ACT_RELU2, ACT_NONE, ACT_GELU_ERF, ACT_XIELU = 0, 1, 2, 3, 4
 SM_COUNT = 148
 _DEEP = os.environ.get("JETSPEC_GEMM_DEEP", "0") == "1"
 _SPLIT_DEEP = os.environ.get("JETSPEC_SPLIT_DEEP")      # force the split-K pipeline: 1 = 192 KB, 2 = 128 KB, 0 = 96 KB
@@ -860,10 +860,10 @@ def sigmoid_route(logits: torch.Tensor, correction: torch.Tensor, top: int, scal
 
 def gemm_inproj(x, w, raw: Optional[torch.Tensor], n_raw: int, act_out: Optional[torch.Tensor], gelu: bool, pdl: bool = False,
                 bn: Optional[int] = None, split: Optional[int] = None, deep: Optional[int] = None,
-                act: Optional[int] = None) -> None:
+                act: Optional[int] = None, act_args: tuple = (0.0, 0.0)) -> None:
     """Fused input projections: ``x @ w.T`` whose first ``n_raw`` columns go to ``raw`` as fp32 and the rest through the
     activation (``gelu``: tanh-GELU gate * up on 64-row interleaved weights, else relu^2; ``act`` names any ``ACT_*``
-    instead) to ``act_out`` as bf16."""
+    instead, with its constants ``act_args``) to ``act_out`` as bf16."""
     act = act if act is not None else ACT_GELU_GLU if gelu else ACT_RELU2
     lib = load()
     M, K = x.shape
@@ -876,7 +876,7 @@ def gemm_inproj(x, w, raw: Optional[torch.Tensor], n_raw: int, act_out: Optional
             bn, split, deep = pick_gemm_config(M, N, K, EPI_SWIGLU, 128)
     _check(lib.js_gemm_inproj(_p(x), _p(w), _p(raw), _p(act_out), M, N, K, x.stride(0), w.stride(0),
                               raw.stride(0) if raw is not None else 0, act_out.stride(0) if act_out is not None else 0,
-                              int(n_raw), int(act), bn, split, int(deep), _p(status_word(x.device)), int(pdl),
+                              int(n_raw), int(act), *map(ctypes.c_float, act_args), bn, split, int(deep), _p(status_word(x.device)), int(pdl),
                               _stream()), f"js_gemm_inproj(M={M},N={N},K={K},bn={bn},split={split})")
 
 
@@ -951,13 +951,17 @@ def rotate_norm(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float
 
 def window_attention(q, k_pool, v_pool, vdim: int, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int,
                      sink, causal: bool, out: Optional[torch.Tensor] = None, pdl: bool = False, keep_first: int = 0,
-                     gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Window attention on the plain cores (bf16 or fp32, heads of up to 512); see the reference op for the contract.  ``gate``:
-    logits whose sigmoid multiplies a head's output."""
+                     gate: Optional[torch.Tensor] = None, softcap: float = 0.0, blocks=None, diff=None) -> torch.Tensor:
+    """Window attention on the plain cores (bf16 or fp32, heads of up to 512); see the reference op for the arguments.  ``gate``:
+    logits whose sigmoid multiplies a head's output (one map a head)."""
     sinks = sink.detach().float().contiguous() if isinstance(sink, torch.Tensor) else None
     lib = load()
     T, H, D = q.shape
     assert q.stride(2) == 1 and q.stride(1) == D
+    maps, (lam, share, eps) = (1, (None, 0.0, 0.0)) if diff is None else (2, diff)
+    H //= maps
+    lam = lam.detach().float().contiguous() if lam is not None else None
+    kb, vb, block_map, P = blocks if blocks is not None else (None, None, None, 0)
     G, S, Dp = k_pool.shape
     if out is None:
         out = torch.empty(T, H * vdim, dtype=q.dtype, device=q.device)
@@ -965,14 +969,68 @@ def window_attention(q, k_pool, v_pool, vdim: int, slot_map, seq_rows, cu_q, pas
         _p(q), ctypes.c_longlong(q.stride(0)), _p(k_pool), _p(v_pool), Dp, v_pool.shape[2], _p(slot_map), _p(seq_rows), _p(cu_q),
         _p(past_lens), _p(mask_bits), _p(out), out.stride(0), seq_rows.numel(), T, H, G, D, vdim, S, slot_map.shape[1],
         mask_bits.shape[1] if mask_bits is not None else 0, int(causal), ctypes.c_float(scale), int(window),
-        int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, H), *_head_gate(gate), _is_bf16(q), _p(status_word(q.device)),
-        int(pdl), _stream()), "js_window_attention_simt")
+        int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, H), *_head_gate(gate), ctypes.c_float(softcap), int(P), _p(kb),
+        _p(vb), kb.shape[1] if P else 0, _p(block_map), block_map.shape[1] if P else 0, maps, _p(lam), ctypes.c_float(share), ctypes.c_float(eps),
+        _is_bf16(q), _p(status_word(q.device)), int(pdl), _stream()), "js_window_attention_simt")
     return out
 
 
-def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int, keep_first: int = 0) -> int:
-    """Key splits of the tensor-core kernel: a CTA's rows span at most the window, their own tokens and the kept first ones."""
-    return attn_splits_for(T, Hq, Hkv, min(max_keys, window + 128 // (Hq // Hkv) + keep_first))
+def pool_blocks(k_pool, v_pool, kb_pool, vb_pool, block_map, P: int, slot_map, seq_rows, cu_q, past_lens, rows: Optional[int] = None,
+                counts=None, most: int = 0, pdl: bool = False) -> None:
+    """Pool the blocks whose last token is among the sequences' new rows (see the reference op).  ``rows`` bounds the new rows
+    where ``cu_q`` must not be read.  With ``counts`` (device) instead of ``cu_q`` the new tokens of a sequence are the last
+    ``counts`` ones ahead of ``past_lens``, at most ``most``."""
+    lib = load()
+    G, S, Kw = k_pool.shape
+    rows = int(cu_q[-1]) if rows is None and counts is None else rows or 0
+    _check(lib.js_pool_blocks(_p(k_pool), _p(v_pool), _p(kb_pool), _p(vb_pool), G, S, kb_pool.shape[1], Kw, v_pool.shape[2], _p(block_map),
+                              block_map.shape[1], P, _p(slot_map), slot_map.shape[1], _p(seq_rows), _p(cu_q), _p(past_lens), _p(counts),
+                              most // P + 1, seq_rows.numel(), rows, _is_bf16(k_pool), _p(status_word(k_pool.device)), int(pdl), _stream()),
+           "js_pool_blocks")
+
+
+def xielu(x: torch.Tensor, up: float, down: float) -> torch.Tensor:
+    lib = load()
+    x = x.contiguous()
+    out = torch.empty_like(x)
+    _check(lib.js_xielu(_p(x), _p(out), ctypes.c_longlong(x.numel()), ctypes.c_float(up), ctypes.c_float(down), _is_bf16(x), _stream()), "js_xielu")
+    return out
+
+
+def depth_average(history: list, weights: torch.Tensor) -> torch.Tensor:
+    lib = load()
+    history, w = [x.contiguous() for x in history], weights.detach().float().contiguous()
+    out = torch.empty_like(history[0])
+    addr = (ctypes.c_ulonglong * len(history))(*[x.data_ptr() for x in history])
+    _check(lib.js_depth_average(addr, len(history), _p(w), _p(out), ctypes.c_longlong(out.numel()), _stream()), "js_depth_average")
+    return out
+
+
+def sandwich(y, src, w, x, next_norm, eps: float, h, width: int, hist: Optional[torch.Tensor] = None, d: Optional[torch.Tensor] = None,
+             tap: Optional[torch.Tensor] = None, pdl: bool = False) -> None:
+    """Residual step of a sublayer whose output is normed: ``x = src + rms(y) w`` and ``h`` its norm with ``next_norm``.  At the
+    end of a layer, ``hist (layers + 1, T, ld)`` and ``d`` (the layer's depth weights): the sum is the layer's result, kept as
+    the next entry of ``hist``, and ``x`` the weighted sum over the entries so far."""
+    lib = load()
+    T, ld = x.shape
+    assert src.stride(0) == ld and h.stride(0) == ld
+    terms = d.numel() - 1 if d is not None else 0
+    assert d is None or (hist.shape[1:] == x.shape and hist.shape[0] > terms)
+    _check(lib.js_sandwich(_p(y), y.stride(0), _p(src), _p(w), _p(d), terms, _p(hist if d is not None else None), ctypes.c_longlong(T * ld),
+                           _p(x), _p(next_norm), ctypes.c_float(eps), _p(h), ld, _p(tap), tap.stride(0) if tap is not None else 0, T, width,
+                           int(pdl), _stream()), "js_sandwich")
+
+
+def window_tc_ok(maps: int, pool: int, softcap: float) -> bool:
+    """Whether the tensor-core kernel has a form for these options."""
+    return maps == 1 and pool == 0 and softcap == 0.0
+
+
+def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int, keep_first: int = 0, pool: int = 0) -> int:
+    """Key splits of the tensor-core kernel: a CTA's rows span at most the window, their own tokens, the kept first ones and the
+    pooled blocks."""
+    keys = min(max_keys, window + 128 // (Hq // Hkv) + keep_first) if window else max_keys
+    return attn_splits_for(T, Hq, Hkv, keys + (max_keys // pool if pool else 0))
 
 
 def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int, sink,

@@ -362,21 +362,58 @@ def rotate_norm(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float
     return y.to(x.dtype)
 
 
-def window_scatter(k: torch.Tensor, v: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, slots: torch.Tensor) -> None:
-    """:func:`kv_scatter` into pools whose rows may be wider than the heads."""
+def window_scatter(k: torch.Tensor, v: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, slots: torch.Tensor, maps: int = 1) -> None:
+    """:func:`kv_scatter` into pools whose rows may be wider than the heads; a key of several ``maps`` has an equal share of the
+    row for each."""
+    if maps > 1:
+        wide = k.new_zeros(*k.shape[:2], maps, k_pool.shape[-1] // maps)
+        wide[..., : k.shape[-1] // maps] = k.view(*k.shape[:2], maps, -1)
+        k = wide.flatten(2)
     kv_scatter(k, v, k_pool[..., : k.shape[-1]], v_pool[..., : v.shape[-1]], slots)
+
+
+def pool_blocks(k_pool: torch.Tensor, v_pool: torch.Tensor, kb_pool: torch.Tensor, vb_pool: torch.Tensor, block_map: torch.Tensor, P: int,
+                slot_map: torch.Tensor, seq_rows: torch.Tensor, cu_q: torch.Tensor, past_lens: torch.Tensor) -> None:
+    """Pool the blocks of ``P`` tokens whose last token is among the sequences' new rows: their rows ``block_map[row, b]`` of
+    ``kb_pool`` and ``vb_pool`` get the means of the cached keys and values."""
+    cu, pl, rows = cu_q.tolist(), past_lens.tolist(), seq_rows.tolist()
+    for i in range(len(cu) - 1):
+        first, stop = pl[i] // P, (pl[i] + cu[i + 1] - cu[i]) // P
+        if stop > first:
+            slots, at = slot_map[rows[i], first * P:stop * P].long(), block_map[rows[i], first:stop].long()
+            for src, dst in ((k_pool, kb_pool), (v_pool, vb_pool)):
+                dst[:, at] = src[:, slots].float().view(src.shape[0], stop - first, P, -1).mean(2).to(dst.dtype)
+
+
+def softcapped(s: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(s / cap) if cap > 0 else s
+
+
+def differential(a: torch.Tensor, lam: torch.Tensor, share: float, eps: float) -> torch.Tensor:
+    """Outputs ``a (T, H, 2, V)`` of a head's two maps to ``share * rms_norm(a1 - lam a2)``, fp32 ``(T, H, V)``."""
+    o = a[:, :, 0].float() - lam.float() * a[:, :, 1].float()
+    return share * o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps)
 
 
 def window_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, vdim: int, slot_map: torch.Tensor,
                      seq_rows: torch.Tensor, cu_q: torch.Tensor, past_lens: torch.Tensor, mask_bits: Optional[torch.Tensor],
-                     scale: float, window: int, sink, causal: bool = False, keep_first: int = 0) -> torch.Tensor:
+                     scale: float, window: int, sink, causal: bool = False, keep_first: int = 0, softcap: float = 0.0,
+                     blocks=None, diff=None) -> torch.Tensor:
     """:func:`paged_tree_attention` with a window, an optional sink, and heads narrower than the pools' rows.  ``sink``: whether
     a valueless key of score 0 takes part in the softmax, or such a key's score per head ``(Hq,)``.  A row sees the last
-    ``window`` tokens of its own path (itself included) and those at positions below ``keep_first``: in a tree a node's
-    position is the committed length plus its number of proper ancestors.  Returns ``(T, Hq*vdim)``."""
+    ``window`` tokens of its own path (itself included; 0: all of them) and those at positions below ``keep_first``: in a tree a
+    node's position is the committed length plus its number of proper ancestors.  ``softcap``: see :func:`softcapped`.
+
+    ``blocks = (kb_pool, vb_pool, block_map, P)``: a row also sees, in the same softmax, one pooled key and value for each block
+    of ``P`` positions that ends before its window.  Blocks that end in committed tokens or in a portion are read from their
+    rows; those that reach into a token tree are the means over the row's own path.
+
+    ``diff = (lam, share, eps)``: ``q (T, 2 Hq, D)`` holds two vectors a head and the pools' rows two keys, whose attentions over
+    the same values are combined by :func:`differential`.  Returns ``(T, Hq*vdim)``."""
     T, Hq, D = q.shape
-    Hkv = k_pool.shape[0]
-    g = Hq // Hkv
+    Hkv, maps = k_pool.shape[0], 1 if diff is None else 2
+    Hq //= maps
+    g, km = Hq // Hkv, k_pool.shape[2] // maps
     out = torch.empty(T, Hq * vdim, dtype=q.dtype, device=q.device)
     cu, pl, rows = cu_q.tolist(), past_lens.tolist(), seq_rows.tolist()
     for b in range(len(cu) - 1):
@@ -385,20 +422,48 @@ def window_attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
         if n == 0:
             continue
         slots = slot_map[rows[b], :past + n].long()
-        k, v = k_pool[:, slots, :D].float(), v_pool[:, slots, :vdim].float()
         anc = (torch.tril(torch.ones(n, n, dtype=torch.bool, device=q.device)) if causal else unpack_ancestor_bits(mask_bits[s:e], n))
         pos = past + anc.sum(-1) - 1
         key_pos = torch.cat((torch.arange(past, device=q.device), pos))
-        vis = torch.cat((torch.ones(n, past, dtype=torch.bool, device=q.device), anc), -1)
-        vis &= (pos[:, None] - key_pos[None] < window) | (key_pos < keep_first)[None]
-        sc = torch.einsum("nhgd,hld->hgnl", q[s:e].float().view(n, Hkv, g, D), k) * scale
-        sc = sc.masked_fill(~vis[None, None], float("-inf"))
-        if isinstance(sink, torch.Tensor):
-            sc = torch.cat((sc, sink.float().view(Hkv, g, 1, 1).expand(Hkv, g, n, 1)), -1)
-        elif sink:
-            sc = torch.cat((sc, torch.zeros_like(sc[..., :1])), -1)
-        p = torch.nan_to_num(torch.softmax(sc, dim=-1), nan=0.0)[..., : past + n]
-        out[s:e] = torch.einsum("hgnl,hlv->nhgv", p, v).reshape(n, Hq * vdim).to(q.dtype)
+        path = torch.cat((torch.ones(n, past, dtype=torch.bool, device=q.device), anc), -1)
+        vis = path
+        if window > 0:
+            vis = path & ((pos[:, None] - key_pos[None] < window) | (key_pos < keep_first)[None])
+        stored = 0
+        if blocks is not None:
+            kb_pool, vb_pool, block_map, P = blocks
+            stored = (past + n if causal else past) // P
+            at = block_map[rows[b], :stored].long()
+            ends = (torch.arange(max(stored, int(pos.max()) // P + 1), device=q.device) + 1) * P - 1
+            far = ends[None] <= pos[:, None] - window
+            # blocks that reach into the tree: shares of the row's path tokens
+            share = torch.zeros(past + n, far.shape[1], device=q.device)
+            share[torch.arange(past + n, device=q.device), (key_pos // P).clamp(max=far.shape[1] - 1)] = 1.0 / P
+        acc = []
+        for m in range(maps):
+            k, v = k_pool[:, slots, m * km:m * km + D].float(), v_pool[:, slots, :vdim].float()
+            qm = q[s:e, m::maps].float().reshape(n, Hkv, g, D)
+            raw = torch.einsum("nhgd,hld->hgnl", qm, k) * scale
+            sc = softcapped(raw, softcap).masked_fill(~vis, float("-inf"))
+            if blocks is not None:
+                kb, vb = kb_pool[:, at, :D].float(), vb_pool[:, at, :vdim].float()
+                sb = torch.cat((torch.einsum("nhgd,hld->hgnl", qm, kb) * scale, (raw * path) @ share[:, stored:]), -1)
+                sc = torch.cat((sc, softcapped(sb, softcap).masked_fill(~far, float("-inf"))), -1)
+            if isinstance(sink, torch.Tensor):
+                sc = torch.cat((sc, sink.float().view(Hkv, g, 1, 1).expand(Hkv, g, n, 1)), -1)
+            elif sink:
+                sc = torch.cat((sc, torch.zeros_like(sc[..., :1])), -1)
+            p = torch.nan_to_num(torch.softmax(sc, dim=-1), nan=0.0)
+            w = p[..., : past + n]
+            if blocks is not None:
+                pb = p[..., past + n:past + n + far.shape[1]]
+                w = w + (pb[..., stored:] @ share[:, stored:].t()) * path
+            o = torch.einsum("hgnl,hlv->nhgv", w, v)
+            if blocks is not None:
+                o = o + torch.einsum("hgnl,hlv->nhgv", pb[..., :stored], vb)
+            acc.append(o.reshape(n, Hq, vdim))
+        o = acc[0] if diff is None else differential(torch.stack(acc, 2), *diff)
+        out[s:e] = o.reshape(n, Hq * vdim).to(q.dtype)
     return out
 
 
@@ -488,6 +553,27 @@ def experts_swiglu(x, idx, w_gate, w_up, w_down) -> torch.Tensor:
 # --------------------------------------------------------------------------
 # general rotations, gates per head, retention
 # --------------------------------------------------------------------------
+def xielu(x: torch.Tensor, up: float, down: float) -> torch.Tensor:
+    """``up x^2 + x / 2`` for positive ``x``, ``down (e^x - 1 - x) + x / 2`` below; 32-bit math."""
+    z = x.float()
+    return (torch.where(z > 0, up * z * z, down * (torch.expm1(z.clamp(max=0.0)) - z)) + 0.5 * z).to(x.dtype)
+
+
+def query_temperature(x: torch.Tensor, positions: torch.Tensor, every: int, coef: float) -> torch.Tensor:
+    """``x (T, ...)`` times ``1 + coef ln(floor((p + 1) / every) + 1)`` of each row's position ``p``."""
+    f = 1.0 + coef * torch.log(((positions + 1) // every + 1).float())
+    return (x.float() * f.view(-1, *[1] * (x.dim() - 1))).to(x.dtype)
+
+
+def depth_average(history: list, weights: torch.Tensor) -> torch.Tensor:
+    """``sum_j weights[j] history[j]`` of fp32 rows."""
+    w = weights.float()
+    out = history[0] * w[0]
+    for j in range(1, len(history)):
+        out = out + history[j] * w[j]
+    return out
+
+
 def gelu_erf(x: torch.Tensor) -> torch.Tensor:
     """Exact gelu, fp32 inside."""
     return F.gelu(x.float()).to(x.dtype)

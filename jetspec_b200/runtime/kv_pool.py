@@ -18,7 +18,17 @@ slot is its slot-map row, so it is granted, given back, evicted and used again t
     states    : StatePool or None
 
 Kinds can differ from layer to layer: ``kv_layers`` and ``latent_pools`` then hold ``None`` where a layer caches the other kind
-or nothing.
+or nothing.  A layer that uses another layer's keys and values has that layer's pools in ``kv_layers``.
+
+A layer whose attention sees whole blocks of ``P`` tokens through one pooled key and value keeps these beside its K and V::
+
+    kv_blocks  : list of (k_pool, v_pool) or None    (Hkv, num_pages * ceil(page_size / P), width)
+    block_maps : {P: (max_seqs, max_len // P)}       row of every block of a sequence
+
+A block's row belongs to the logical page its last token lies in, so blocks are granted, given back and used again with the
+pages.  Tokens may trade slots inside a sequence (below); blocks never do.  A block is pooled when its last token is
+committed: in the forward of a prompt portion or decoded token, or when a path of a token tree is committed
+(:meth:`PagedKVPool.pool_committed`).
 
 Everything below the buffers (pages, slot maps, admission, eviction, commit) is the same for all kinds.
 
@@ -64,9 +74,10 @@ def latent_row_width(width: int) -> int:
     return (int(width) + 63) // 64 * 64
 
 
-def window_row_width(dim: int, vdim: int, dtype: torch.dtype) -> tuple:
-    """Elements a K and a V row take: bf16 heads of up to 128 are padded to the tensor-core attention's 128."""
-    return (128, 128) if dtype == torch.bfloat16 and max(dim, vdim) <= 128 else (int(dim), int(vdim))
+def window_row_width(dim: int, vdim: int, dtype: torch.dtype, maps: int = 1) -> tuple:
+    """Elements a K and a V row take: bf16 heads of up to 128 are padded to the tensor-core attention's 128.  The keys of a
+    head's ``maps`` lie side by side in its row, an equal share of it each."""
+    return (128, 128) if dtype == torch.bfloat16 and max(dim * maps, vdim) <= 128 else (int(dim) * maps, int(vdim))
 
 
 @dataclass
@@ -83,17 +94,26 @@ class PagedKVPool:
     def __init__(self, num_layers: int, num_kv_heads: int, head_dim: int, num_pages: int,
                  page_size: int = 16, max_seqs: int = 64, max_seq_len: int = 4096,
                  device="cpu", dtype=torch.float32, latent_widths: Optional[list] = None,
-                 kv_shapes: Optional[list] = None, state_shapes: Optional[list] = None):
+                 kv_shapes: Optional[list] = None, state_shapes: Optional[list] = None,
+                 kv_sources: Optional[list] = None, kv_pools: Optional[list] = None):
         self.num_layers, self.num_kv_heads, self.head_dim = num_layers, num_kv_heads, head_dim
         self.page_size, self.num_pages = int(page_size), int(num_pages)
         self.max_seqs, self.max_seq_len = int(max_seqs), int(max_seq_len)
         self.device, self.dtype = torch.device(device), dtype
         S = self.num_pages * self.page_size
-        self.k_pool = self.v_pool = self.latent_pools = self.kv_layers = self.states = None
+        self.k_pool = self.v_pool = self.latent_pools = self.kv_layers = self.states = self.kv_blocks = None
+        self.block_maps: dict = {}
         if kv_shapes is not None:
-            def pools(heads, dim, vdim):
-                return tuple(torch.zeros(heads, S, w, dtype=dtype, device=device) for w in window_row_width(dim, vdim, dtype))
-            self.kv_layers = [pools(*shape) if shape is not None else None for shape in kv_shapes]
+            def pools(rows, heads, dim, vdim, maps=1):
+                return tuple(torch.zeros(heads, rows, w, dtype=dtype, device=device) for w in window_row_width(dim, vdim, dtype, maps))
+            self.kv_layers = [pools(S, *shape) if shape is not None else None for shape in kv_shapes]
+            if kv_sources is not None:
+                self.kv_layers = [self.kv_layers[j] for j in kv_sources]
+            if kv_pools is not None and any(kv_pools):
+                self.block_sizes = list(kv_pools)
+                self.kv_blocks = [pools(self.num_pages * self._blocks_per_page(P), *shape) if P else None for P, shape in zip(kv_pools, kv_shapes)]
+                self.block_maps = {P: torch.zeros(self.max_seqs, max(1, self.max_seq_len // P), dtype=torch.int32, device=device)
+                                   for P in set(kv_pools) if P}
         if latent_widths is not None:
             self.latent_pools = [None if w is None else torch.zeros(S, latent_row_width(w), dtype=dtype, device=device)
                                  for w in latent_widths]
@@ -116,7 +136,9 @@ class PagedKVPool:
         """A pool of the shape ``cfg``'s attention caches (``world``: ranks the K/V heads are sharded over)."""
         widths, shapes = cfg.latent_widths(), cfg.kv_shapes()
         if widths is not None or shapes is not None:
-            return cls(cfg.num_hidden_layers, 0, 0, num_pages, latent_widths=widths, kv_shapes=shapes, state_shapes=cfg.state_shapes(), **kw)
+            optional = {k: getattr(cfg, k)() for k in ("kv_sources", "kv_pools") if hasattr(cfg, k)}
+            return cls(cfg.num_hidden_layers, 0, 0, num_pages, latent_widths=widths, kv_shapes=shapes, state_shapes=cfg.state_shapes(),
+                       **optional, **kw)
         return cls(cfg.num_hidden_layers, cfg.num_key_value_heads // world, cfg.head_dim, num_pages, **kw)
 
     @property
@@ -138,6 +160,38 @@ class PagedKVPool:
 
     def latent(self, li: int) -> torch.Tensor:
         return self.latent_pools[li]
+
+    def _blocks_per_page(self, P: int) -> int:
+        """Most blocks of ``P`` tokens that end in one page."""
+        return (self.page_size + P - 1) // P
+
+    def blocks(self, li: int):
+        """``(k rows, v rows, block map, P)`` of a layer's pooled blocks, or ``None``."""
+        if self.kv_blocks is None or self.kv_blocks[li] is None:
+            return None
+        P = self.block_sizes[li]
+        return (*self.kv_blocks[li], self.block_maps[P], P)
+
+    def _map_blocks(self, st: "SeqState", base: int) -> None:
+        """Rows of the blocks that end at position ``base`` or later in the pages of ``st``."""
+        for P, table in self.block_maps.items():
+            first, stop = base // P, min(len(st.pages) * self.page_size // P, table.shape[1])
+            if stop > first:
+                b = torch.arange(first, stop)
+                page = ((b + 1) * P - 1) // self.page_size
+                rows = torch.tensor(st.pages)[page] * self._blocks_per_page(P) + b - page * self.page_size // P
+                table[st.row, first:stop] = rows.to(torch.int32).to(self.device, non_blocking=True)
+
+    def pool_committed(self, row: int, past: int, n: int) -> None:
+        """Pool the blocks whose last token is among the positions ``[past, past + n)`` of slot-map row ``row``."""
+        if self.kv_blocks is None or n <= 0:
+            return
+        from .. import ops
+        i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device=self.device)
+        rows, cu_q, past_t = i32(row), i32(0, n), i32(past)
+        for li, (kv, kb) in enumerate(zip(self.kv_layers, self.kv_blocks)):
+            if kb is not None and (past + n) // self.block_sizes[li] > past // self.block_sizes[li]:
+                ops.pool_blocks(*kv, *self.blocks(li), self.slot_map, rows, cu_q, past_t)
 
     # -- sequences ------------------------------------------------------------
     def has(self, seq_id: int) -> bool:
@@ -198,6 +252,8 @@ class PagedKVPool:
                    + torch.arange(self.page_size, dtype=torch.int32).repeat(len(new_pages)))
             end = min(base + ids.numel(), self.max_seq_len)
             self.slot_map[st.row, base:end] = ids[: end - base].to(self.device, non_blocking=True)
+            if self.block_maps:
+                self._map_blocks(st, base)
         st.capacity = min(len(st.pages) * self.page_size, self.max_seq_len)
         st.last_used = next(self._clock)
         return True
@@ -256,7 +312,8 @@ class PagedKVPool:
         ``path`` lists accepted node indices (root first).  The window
         ``slot_map[row, past:past+num_nodes]`` is permuted to ``path`` followed by the
         remaining nodes in index order, and the committed length becomes
-        ``past + len(path)``.  No KV bytes move; recurrent states advance along the path.
+        ``past + len(path)``.  No KV bytes move; recurrent states advance along the path, and
+        blocks it completes are pooled.
         """
         st = self._seqs[seq_id]
         if isinstance(path, (list, tuple)):      # host path: the permutation is built without a device read
@@ -274,5 +331,6 @@ class PagedKVPool:
             self.states.commit(st.row, past, order[:n_path])
         win = self.slot_map[st.row, past:past + num_nodes]
         self.slot_map[st.row, past:past + num_nodes] = win[order]
+        self.pool_committed(st.row, past, n_path)
         st.length = past + n_path
         st.last_used = next(self._clock)
