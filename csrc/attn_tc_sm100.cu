@@ -18,9 +18,18 @@
 //
 // Roles (416 threads): warps 0-3 softmax + epilogue (tensor-memory lane quadrant = warp id),
 // warp 4 MMA issuer / TMEM owner, warps 5-12 loaders.  Every wait is bounded (status word).
+//
+// Forms (template parameter MODE):
+//   * kPlain: the above, with an optional window, kept first tokens, sinks and gates;
+//   * kPooled: scores may be capped, and tiles of pooled blocks (one key and value per P tokens, read through a block map)
+//     stand ahead of the window's tiles;
+//   * kDiff: two attention maps a head over the same values.  Query and key rows hold 64 columns for each map, so a tile's K
+//     and V are gathered once and give two score tiles and two outputs (warps 0-3 and 4-7 own one map each, warp 8
+//     issues, four loader warps); the epilogue (or the merge of the key splits) norms o1 - lam o2.
 #include "common.cuh"
 
 #include <math.h>
+#include <type_traits>
 
 namespace js {
 
@@ -28,12 +37,15 @@ constexpr int TD = 128;          // head dim
 constexpr int TROWS = 128;       // query rows per CTA
 constexpr int TKEYS = 64;        // keys per tile
 constexpr int TSTAGES = 3;
-constexpr int TLOADERS = 256;       // loader threads (gather throughput grows with the copies in flight)
-constexpr int TTHREADS = 160 + TLOADERS;
+constexpr int TTHREADS = 416;       // softmax threads of every map, one issuing warp, loaders
+enum AttnMode : int { kPlain = 0, kPooled = 1, kDiff = 2 };
+// loader threads (gather throughput grows with the copies in flight)
+__host__ __device__ constexpr int loader_threads(int mode) { return TTHREADS - 32 - (mode == kDiff ? 256 : 128); }
+__host__ __device__ constexpr int attn_maps(int mode) { return mode == kDiff ? 2 : 1; }
 constexpr int kStageKV = 2 * TKEYS * 256;      // K then V, each 2 halves x 64 keys x 128 B
 constexpr int kSmemQ = TROWS * 256;            // 2 halves x 128 rows x 128 B
 constexpr int kSmemP = TROWS * 128;            // 128 rows x 64 keys bf16
-constexpr int kAttnTcSmem = kSmemQ + TSTAGES * kStageKV + 2 * kSmemP + 256 + 1024;
+constexpr int attn_tc_smem(int mode) { return kSmemQ + TSTAGES * kStageKV + 2 * attn_maps(mode) * kSmemP + 256 + 1024; }
 // Key splits that merge inside a cluster (portable cluster size); the chunk receive area must fit the dead
 // K/V stages + P buffers, the (max, sum) pairs the dead Q tile.
 constexpr int kMaxClusterSplits = 8;
@@ -65,7 +77,30 @@ struct AttnTcParams {
   const float* gate;           // (T, ldg) logits: head h's output is multiplied by sigmoid(gate[t, h]); may be null
   int ldg;
   int cluster_merge;           // the key splits of a tile form a cluster and merge through distributed shared memory
+  // kPooled
+  float cap_log2, inv_cap;     // score cap in the log2 domain (0: none), scale / cap
+  int cap_poly;                // |score / cap| is small enough for the polynomial
+  int P;                       // tokens to a block, 0 without blocks
+  const __nv_bfloat16 *kb_pool, *vb_pool;      // (Hkv, block_rows, 128)
+  const int* block_map;        // (max_seqs, max_blocks)
+  int block_rows, max_blocks;
+  // kDiff
+  const float* lam;
+  float share, eps;
+  int V;                       // true width of a head's values
 };
+
+// cap tanh(s / cap) in the log2 domain for x = s / cap; the polynomial is for |x| up to 0.35 (error below 1e-7)
+JS_DEVICE float capped_poly(float x, float cap_log2) {
+  const float u = x * x;       // Taylor series of tanh(x) / x
+  return cap_log2 * x * (1.f + u * (-1.f / 3.f + u * (2.f / 15.f + u * (-17.f / 315.f + u * (62.f / 2835.f)))));
+}
+JS_DEVICE float capped_any(float x, float cap_log2) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));      // e^(2x)
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return cap_log2 - 2.f * cap_log2 * r;
+}
 
 JS_DEVICE void cp_async16_tc(uint32_t smem_addr, const void* gmem, bool valid) {
   const int n = valid ? 16 : 0;   // src-size 0 -> zero fill
@@ -128,22 +163,23 @@ JS_DEVICE void attn_trace(int slot) {
   }
 }
 
-template <int G>
+template <int G, int MODE>
 __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcParams p) {
   constexpr int NPT = TROWS / G;   // nodes per q tile
+  constexpr int MAPS = attn_maps(MODE), TLOADERS = loader_threads(MODE), MMA_WARP = 4 * MAPS;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
   uint8_t* sKV = sQ + kSmemQ;
   uint8_t* sP = sKV + TSTAGES * kStageKV;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 2 * kSmemP);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 2 * MAPS * kSmemP);
   uint64_t* q_full = bars;                 // 1
   uint64_t* kv_full = bars + 1;            // TSTAGES
   uint64_t* kv_empty = kv_full + TSTAGES;  // TSTAGES
-  uint64_t* s_full = kv_empty + TSTAGES;   // 2
-  uint64_t* p_full = s_full + 2;           // 2
-  uint64_t* pv_done = p_full + 2;          // 2
-  uint64_t* o_done = pv_done + 2;          // 1
+  uint64_t* s_full = kv_empty + TSTAGES;   // 2 a map
+  uint64_t* p_full = s_full + 2 * MAPS;    // 2 a map
+  uint64_t* pv_done = p_full + 2 * MAPS;   // 2 a map
+  uint64_t* o_done = pv_done + 2 * MAPS;   // 1
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(o_done + 1);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -172,14 +208,29 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   const int t_first = p.window > 0 ? max(0, past + (p.causal ? node0 : 0) - p.window + 1) / TKEYS : 0;
   // ... behind the tiles of kept first tokens: the CTA's tiles are 0 .. t_kept - 1 and t_first, t_first + 1, ...
   const int t_kept = p.window > 0 ? min(t_first, (p.keep + TKEYS - 1) / TKEYS) : 0;
-  const int n_tiles = (L + TKEYS - 1) / TKEYS - t_first + t_kept;
+  // tiles of pooled blocks come first: the blocks the CTA's last row sees (those of committed tokens, over a token tree)
+  int nb_max = 0, t_pool = 0;
+  if constexpr (MODE == kPooled) {
+    if (p.P > 0) {
+      const int behind = past + (p.causal ? min(node0 + NPT, n_b) : n_b) - p.window;      // positions behind the last row's window
+      nb_max = behind > 0 ? behind / p.P : 0;
+      if (!p.causal) nb_max = min(nb_max, past / p.P);
+      t_pool = (nb_max + TKEYS - 1) / TKEYS;
+    }
+  }
+  const int n_tiles = (L + TKEYS - 1) / TKEYS - t_first + t_kept + t_pool;
   const int t_begin = (n_tiles * split) / p.splits;
   const int t_end = (n_tiles * (split + 1)) / p.splits;
   const int nt = t_end - t_begin;
   auto tile_key = [&](int i) {          // first key of this split's tile i
-    const int t = t_begin + i;
+    int t = t_begin + i;
+    if constexpr (MODE == kPooled) {
+      if (t < t_pool) return t * TKEYS;
+      t -= t_pool;
+    }
     return (t < t_kept ? t : t - t_kept + t_first) * TKEYS;
   };
+  auto pooled_tile = [&](int i) { return MODE == kPooled && t_begin + i < t_pool; };      // its keys are blocks
 
   // softmax thread's row
   const int row = (warp & 3) * 32 + lane;
@@ -188,7 +239,9 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   const size_t out_row = static_cast<size_t>(q_begin + (row_valid ? node : 0)) * p.Hq + head;
   __nv_bfloat16* out_ptr = p.out + static_cast<size_t>(q_begin + (row_valid ? node : 0)) * p.ldo + head * TD;
 
-  const bool cmerge = p.cluster_merge != 0;
+  const bool cmerge = MODE != kDiff && p.cluster_merge != 0;
+  const int map = MODE == kDiff ? warp >> 2 : 0;      // softmax threads: the map they own
+  const bool softmax_warp = warp < 4 * MAPS;
   float m_run = -INFINITY, l_run = 0.f;     // softmax threads: running (integer) maximum and sum of their row
   if (p.sink && split == p.splits - 1) {    // the last split always has a tile
     const float s2 = p.sinks != nullptr && row_valid ? p.sinks[head] * 1.4426950408889634f : 0.f;
@@ -198,8 +251,8 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   const float gate = p.gate != nullptr && row_valid ? 1.f / (1.f + expf(-p.gate[static_cast<size_t>(q_begin + node) * p.ldg + head])) : 1.f;
   bool sm_ok = true;
   if (nt <= 0 && !cmerge) {   // more splits than key tiles: this split contributes nothing
-    if (warp < 4 && row_valid && p.splits > 1) {
-      float* ml = p.ws_ml + (static_cast<size_t>(split) * p.T * p.Hq + out_row) * 2;
+    if (softmax_warp && row_valid && p.splits > 1) {
+      float* ml = p.ws_ml + ((static_cast<size_t>(split) * p.T * p.Hq + out_row) * MAPS + map) * 2;
       ml[0] = -INFINITY;
       ml[1] = 0.f;
     }
@@ -209,12 +262,12 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   if (tid == 0 && nt > 0) {
     mbar_init(q_full, TLOADERS);
     for (int s = 0; s < TSTAGES; ++s) { mbar_init(&kv_full[s], TLOADERS); mbar_init(&kv_empty[s], 1); }
-    for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], 128); mbar_init(&pv_done[i], 1); }
+    for (int i = 0; i < 2 * MAPS; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], 128); mbar_init(&pv_done[i], 1); }
     mbar_init(o_done, 1);
     fence_barrier_init();
   }
-  if (warp == 4 && nt > 0) {
-    tmem_alloc(tmem_slot, 256);
+  if (warp == MMA_WARP && nt > 0) {
+    tmem_alloc(tmem_slot, 256 * MAPS);
     tmem_relinquish();
   }
   tc_fence_before();
@@ -222,14 +275,14 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   tc_fence_after();
   const uint32_t tmem_base = nt > 0 ? *tmem_slot : 0u;
   if (tid == 0) attn_trace(1);      // setup done
-  const uint32_t tmem_o = tmem_base + 128;      // S buffers at columns [0,64) and [64,128)
+  const uint32_t tmem_o = tmem_base + 128 * MAPS;      // map m: S buffers at columns 128 m and 128 m + 64, O behind all of them
 
   const uint32_t t_lane = static_cast<uint32_t>((warp & 3) * 32) << 16;
   if (nt <= 0) {
     // (cluster merge) nothing to compute: this CTA only takes part in the exchange below
-  } else if (warp >= 5) {
+  } else if (warp > MMA_WARP) {
     // ================================================================ loaders
-    const int lt = tid - 160;
+    const int lt = tid - (MMA_WARP + 1) * 32;
     const uint32_t q_addr = smem_u32(sQ);
     for (int c = lt; c < TROWS * 16; c += TLOADERS) {
       const int r = c >> 4, ch = c & 15;
@@ -243,11 +296,17 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
     const int ch = lt & 15, r0 = lt >> 4;       // this thread copies chunk `ch` of keys r0, r0+RSTEP, ...
     // slots of the first tile; the next tile's are fetched while the current tile's copies are issued
     int slot_next[TKEYS / RSTEP];
+    const int* blocks = nullptr;
+    if constexpr (MODE == kPooled) blocks = p.block_map + static_cast<size_t>(p.seq_rows[b]) * p.max_blocks;
+    // slot of key kp of tile i, 0 past the end
+    auto slot_at = [&](int i, int kp) {
+      if constexpr (MODE == kPooled) {
+        if (pooled_tile(i)) return kp < nb_max ? (kp < p.max_blocks ? __ldg(blocks + kp) : -1) : 0;
+      }
+      return kp < L ? __ldg(slots + kp) : 0;
+    };
 #pragma unroll
-    for (int j = 0; j < TKEYS / RSTEP; ++j) {
-      const int kp = tile_key(0) + r0 + RSTEP * j;
-      slot_next[j] = kp < L ? __ldg(slots + kp) : 0;
-    }
+    for (int j = 0; j < TKEYS / RSTEP; ++j) slot_next[j] = slot_at(0, tile_key(0) + r0 + RSTEP * j);
     bool ok = true;
     // copies complete in issue order (Q, tile 0, tile 1, ...); `next_sig` is the next one to publish (-1 = Q)
     int next_sig = -1;
@@ -276,20 +335,31 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 #pragma unroll
       for (int j = 0; j < TKEYS / RSTEP; ++j) {
         slot_cur[j] = slot_next[j];
-        const int kpn = k0n + r0 + RSTEP * j;
-        slot_next[j] = (i + 1 < nt && kpn < L) ? __ldg(slots + kpn) : 0;
+        slot_next[j] = i + 1 < nt ? slot_at(i + 1, k0n + r0 + RSTEP * j) : 0;
+      }
+      const bool is_pool = pooled_tile(i);
+      const int limit = is_pool ? nb_max : L, n_slots = is_pool ? p.block_rows : p.S;
+      const __nv_bfloat16 *k_src = p.k_pool, *v_src = p.v_pool;
+      long long head_stride = p.kv_head, slot_stride = p.kv_slot;
+      if constexpr (MODE == kPooled) {
+        if (is_pool) {
+          k_src = p.kb_pool;
+          v_src = p.vb_pool;
+          head_stride = static_cast<long long>(p.block_rows) * TD;
+          slot_stride = TD;
+        }
       }
 #pragma unroll
       for (int j = 0; j < TKEYS / RSTEP; ++j) {
         const int r = r0 + RSTEP * j;
         const int kp = k0 + r;
-        const bool valid = kp < L;
+        const bool valid = kp < limit;
         int slot = slot_cur[j];
-        if (slot < 0 || slot >= p.S) { report(p.status, kBadSlot); slot = 0; }
-        const size_t off = static_cast<size_t>(h) * p.kv_head + static_cast<size_t>(slot) * p.kv_slot + ch * 8;
+        if (slot < 0 || slot >= n_slots) { report(p.status, kBadSlot); slot = 0; }
+        const size_t off = static_cast<size_t>(h) * head_stride + static_cast<size_t>(slot) * slot_stride + ch * 8;
         const uint32_t dst = (ch >> 3) * (TKEYS * 128) + r * 128 + (((ch & 7) ^ (r & 7)) << 4);
-        cp_async16_tc(k_addr + dst, p.k_pool + off, valid);
-        cp_async16_tc(k_addr + TKEYS * 256 + dst, p.v_pool + off, valid);
+        cp_async16_tc(k_addr + dst, k_src + off, valid);
+        cp_async16_tc(k_addr + TKEYS * 256 + dst, v_src + off, valid);
       }
       cp_async_commit_tc();
       if (lt == 0 && i < 8) attn_trace(32 + i);    // copies of tile i issued
@@ -300,22 +370,29 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
       cp_async_wait_tc<0>();
       publish_before(nt);
     }
-  } else if (warp == 4) {
+  } else if (warp == MMA_WARP) {
     // ================================================================ MMA issuer
     if (lane == 0) {
       constexpr uint32_t idesc_qk = umma_idesc_bf16(TROWS, TKEYS);
       constexpr uint32_t idesc_pv = umma_idesc_bf16_bmn(TROWS, TD);
       bool ok = mbar_wait_backoff(q_full, 0, p.status, kTimeoutFull);
       attn_trace(2);                // Q landed
+      // O += P V of tile j for every map, each as soon as its P is there
       auto issue_pv = [&](int j) {
         const int s = j % TSTAGES, pb = j & 1;
         const uint32_t v_addr = smem_u32(sKV + s * kStageKV + TKEYS * 256);
-        const uint64_t a_desc = umma_desc_sw128(smem_u32(sP + pb * kSmemP));
 #pragma unroll
-        for (int k = 0; k < TKEYS / 16; ++k)
-          umma_f16(tmem_o, a_desc + 2 * k, umma_desc_sw128_mn(v_addr + k * 2048, TKEYS * 128), idesc_pv, (j | k) != 0 ? 1u : 0u);
-        umma_commit(&kv_empty[s]);
-        umma_commit(&pv_done[pb]);
+        for (int m = 0; m < MAPS; ++m) {
+          if (!mbar_wait_backoff(&p_full[2 * m + pb], (j >> 1) & 1, p.status, kTimeoutAccum)) return false;
+          tc_fence_after();
+          const uint64_t a_desc = umma_desc_sw128(smem_u32(sP + (2 * m + pb) * kSmemP));
+#pragma unroll
+          for (int k = 0; k < TKEYS / 16; ++k)
+            umma_f16(tmem_o + m * TD, a_desc + 2 * k, umma_desc_sw128_mn(v_addr + k * 2048, TKEYS * 128), idesc_pv, (j | k) != 0 ? 1u : 0u);
+          if (m == MAPS - 1) umma_commit(&kv_empty[s]);
+          umma_commit(&pv_done[2 * m + pb]);
+        }
+        return true;
       };
       for (int i = 0; i < nt && ok; ++i) {
         const int s = i % TSTAGES, sb = i & 1;
@@ -327,25 +404,18 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         const uint32_t k_addr = smem_u32(sKV + s * kStageKV);
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
-          const uint32_t hoff = (k >> 2), kk = k & 3;
-          umma_f16(tmem_base + sb * TKEYS, umma_desc_sw128(smem_u32(sQ) + hoff * (TROWS * 128)) + 2 * kk,
-                   umma_desc_sw128(k_addr + hoff * (TKEYS * 128)) + 2 * kk, idesc_qk, k != 0 ? 1u : 0u);
+          const uint32_t hoff = (k >> 2), kk = k & 3;          // each half of the columns is a map of its own in kDiff
+          umma_f16(tmem_base + (MAPS == 2 ? hoff * 2 * TKEYS : 0) + sb * TKEYS, umma_desc_sw128(smem_u32(sQ) + hoff * (TROWS * 128)) + 2 * kk,
+                   umma_desc_sw128(k_addr + hoff * (TKEYS * 128)) + 2 * kk, idesc_qk, (MAPS == 2 ? kk : k) != 0 ? 1u : 0u);
+          if (MAPS == 2 && k == 3) umma_commit(&s_full[sb]);
         }
-        umma_commit(&s_full[sb]);
+        umma_commit(&s_full[2 * (MAPS - 1) + sb]);
         if (i >= 1) {
-          ok = mbar_wait_backoff(&p_full[(i - 1) & 1], ((i - 1) >> 1) & 1, p.status, kTimeoutAccum);
+          ok = issue_pv(i - 1);
           if (!ok) break;
-          tc_fence_after();
-          issue_pv(i - 1);
         }
       }
-      if (ok) {
-        ok = mbar_wait_backoff(&p_full[(nt - 1) & 1], ((nt - 1) >> 1) & 1, p.status, kTimeoutAccum);
-        if (ok) {
-          tc_fence_after();
-          issue_pv(nt - 1);
-        }
-      }
+      if (ok) ok = issue_pv(nt - 1);
       umma_commit(o_done);     // also releases the epilogue on an error path
     }
   } else {
@@ -355,13 +425,16 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
     for (int w = 0; w < 8; ++w)
       mw[w] = (!p.causal && row_valid && w < p.W) ? p.mask_bits[static_cast<size_t>(q_begin + node) * p.W + w] : 0;
     int cut = 0;                       // committed keys below it are out of the row's window
+    int nb_row = 0;                    // blocks the row sees
     if (p.window > 0) {
       if (p.causal) {
         cut = past + node - p.window + 1;
+        if constexpr (MODE == kPooled) nb_row = p.P > 0 && cut > 0 ? cut / p.P : 0;
       } else {                         // a node's position is its number of proper ancestors behind the committed length
         int cnt = 0;
 #pragma unroll
         for (int w = 0; w < 8; ++w) cnt += __popc(static_cast<unsigned>(mw[w]));
+        if constexpr (MODE == kPooled) nb_row = p.P > 0 && past + cnt > p.window ? min(past + cnt - p.window, past) / p.P : 0;
         cut = min(past, past + cnt - p.window);
         // ancestors out of the window are the lowest bits (the d-th lowest is at position past + d); kept ones stay
         int drop = cnt - p.window, spare = p.keep - past;
@@ -379,19 +452,22 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
     bool ok = true;
     for (int i = 0; i < nt && ok; ++i) {
       const int sb = i & 1;
-      ok = mbar_wait_backoff(&s_full[sb], (i >> 1) & 1, p.status, kTimeoutAccum);
+      ok = mbar_wait_backoff(&s_full[2 * map + sb], (i >> 1) & 1, p.status, kTimeoutAccum);
       if (!ok) break;
       tc_fence_after();
       if (tid == 0 && i < 8) attn_trace(16 + i);   // scores of tile i ready
       uint32_t sr[64];
-      tmem_ld_32x32(tmem_base + t_lane + sb * TKEYS, sr);
-      tmem_ld_32x32(tmem_base + t_lane + sb * TKEYS + 32, sr + 32);
+      tmem_ld_32x32(tmem_base + t_lane + (2 * map + sb) * TKEYS, sr);
+      tmem_ld_32x32(tmem_base + t_lane + (2 * map + sb) * TKEYS + 32, sr + 32);
       tmem_ld_wait();
       // visibility of the tile's 64 keys for this row, as one 64-bit word (bit c = key k0 + c)
       const int k0 = tile_key(i);
       const int jlo = k0 - past;                         // window index of the tile's first key (may be < 0)
       unsigned long long vm = 0ull;
-      if (row_valid) {
+      if (pooled_tile(i)) {
+        const int seen = nb_row - k0;
+        if (row_valid && seen > 0) vm = seen >= TKEYS ? ~0ull : (1ull << seen) - 1ull;
+      } else if (row_valid) {
         if (jlo <= -TKEYS) {
           vm = ~0ull;                                    // the whole tile is prefix
         } else {
@@ -419,10 +495,23 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         }
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};   // four chains instead of one 64-deep
+      float to_log2 = p.scale_log2;
+      if constexpr (MODE == kPooled) {
+        if (p.cap_log2 > 0.f) {
+          if (p.cap_poly) {
+#pragma unroll
+            for (int c = 0; c < 64; ++c) sr[c] = __float_as_uint(capped_poly(__uint_as_float(sr[c]) * p.inv_cap, p.cap_log2));
+          } else {
+#pragma unroll
+            for (int c = 0; c < 64; ++c) sr[c] = __float_as_uint(capped_any(__uint_as_float(sr[c]) * p.inv_cap, p.cap_log2));
+          }
+          to_log2 = 1.f;
+        }
+      }
       if (vm == ~0ull) {              // the common case: every key of the tile is visible to this row
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
-          const float x = __uint_as_float(sr[c]) * p.scale_log2;
+          const float x = __uint_as_float(sr[c]) * to_log2;
           sr[c] = __float_as_uint(x);
           mx4[c & 3] = fmaxf(mx4[c & 3], x);
         }
@@ -430,7 +519,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
           const bool vis = (vm >> c) & 1ull;
-          const float x = vis ? __uint_as_float(sr[c]) * p.scale_log2 : -INFINITY;
+          const float x = vis ? __uint_as_float(sr[c]) * to_log2 : -INFINITY;
           sr[c] = __float_as_uint(x);
           mx4[c & 3] = fmaxf(mx4[c & 3], x);
         }
@@ -443,10 +532,10 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
       const float alpha = exp2f(m_run - m_safe);          // 0 when nothing was visible before
       m_run = m_new;
       // P buffer sb is free once PV of tile i-2 has completed
-      if (i >= 2) ok = mbar_wait_backoff(&pv_done[sb], ((i - 2) >> 1) & 1, p.status, kTimeoutAccum);
+      if (i >= 2) ok = mbar_wait_backoff(&pv_done[2 * map + sb], ((i - 2) >> 1) & 1, p.status, kTimeoutAccum);
       if (!ok) break;
       float rs4[4] = {0.f, 0.f, 0.f, 0.f};
-      const uint32_t p_row = smem_u32(sP + sb * kSmemP) + row * 128;
+      const uint32_t p_row = smem_u32(sP + (2 * map + sb) * kSmemP) + row * 128;
 #pragma unroll
       for (int c8 = 0; c8 < 8; ++c8) {
         uint32_t w4[4];
@@ -465,23 +554,23 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
       // rescale O when some row of this warp raised its maximum (tcgen05.ld/st are warp-wide)
       const bool need = i > 0 && alpha != 1.f;
       if (__any_sync(0xffffffffu, need)) {
-        ok = mbar_wait_backoff(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1, p.status, kTimeoutAccum);   // every earlier PV is in O
+        ok = mbar_wait_backoff(&pv_done[2 * map + ((i - 1) & 1)], ((i - 1) >> 1) & 1, p.status, kTimeoutAccum);   // every earlier PV is in O
         if (!ok) break;
         tc_fence_after();
 #pragma unroll 1
         for (int c0 = 0; c0 < TD; c0 += 32) {
           uint32_t orr[32];
-          tmem_ld_32x32(tmem_o + t_lane + c0, orr);
+          tmem_ld_32x32(tmem_o + map * TD + t_lane + c0, orr);
           tmem_ld_wait();
 #pragma unroll
           for (int j = 0; j < 32; ++j) orr[j] = __float_as_uint(__uint_as_float(orr[j]) * alpha);
-          tmem_st_32x32(tmem_o + t_lane + c0, orr);
+          tmem_st_32x32(tmem_o + map * TD + t_lane + c0, orr);
         }
         tmem_st_wait();
       }
       fence_proxy_async();          // P (generic-proxy stores) -> visible to the MMA's async-proxy reads
       tc_fence_before();
-      mbar_arrive(&p_full[sb]);
+      mbar_arrive(&p_full[2 * map + sb]);
       if (tid == 0 && i < 8) attn_trace(24 + i);   // P of tile i published
     }
     // ---- epilogue
@@ -489,12 +578,46 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
     tc_fence_after();
     if (tid == 0) attn_trace(3);    // output accumulator complete
     sm_ok = ok;
-    if (ok && !cmerge) {
+    if (MODE == kDiff && p.splits == 1) {
+      // both maps' threads of a row finish half of its columns each; sums and denominators pass through the dead Q tile
+      float* den = reinterpret_cast<float*>(sQ);
+      float* sq = den + 2 * TROWS;
+      auto both_maps = [] { asm volatile("bar.sync 1, 256;" ::: "memory"); };
+      den[map * TROWS + row] = l_run > 0.f ? 1.f / l_run : 0.f;
+      both_maps();
+      const float i1 = den[row], i2 = den[TROWS + row] * *p.lam;
+      float v[64], ss = 0.f;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t a[32], c[32];
+        const uint32_t at = tmem_o + t_lane + map * 64 + half * 32;
+        tmem_ld_32x32(at, a);
+        tmem_ld_32x32(at + TD, c);
+        tmem_ld_wait();
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+          v[half * 32 + j] = __uint_as_float(a[j]) * i1 - __uint_as_float(c[j]) * i2;
+          ss += v[half * 32 + j] * v[half * 32 + j];
+        }
+      }
+      sq[map * TROWS + row] = ss;
+      both_maps();
+      const float r = p.share / sqrtf((sq[row] + sq[TROWS + row]) / p.V + p.eps);
+      if (ok && row_valid) {
+        uint4 pk[8];
+        __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(pk);
+#pragma unroll
+        for (int j = 0; j < 32; ++j) o2[j] = __floats2bfloat162_rn(v[2 * j] * r, v[2 * j + 1] * r);
+        uint4* dst = reinterpret_cast<uint4*>(out_ptr + map * 64);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) dst[j] = pk[j];
+      }
+    } else if (ok && !cmerge) {
       const float inv = l_run > 0.f ? gate / l_run : 0.f;
 #pragma unroll 1
       for (int c0 = 0; c0 < TD; c0 += 32) {
         uint32_t orr[32];
-        tmem_ld_32x32(tmem_o + t_lane + c0, orr);
+        tmem_ld_32x32(tmem_o + map * TD + t_lane + c0, orr);
         tmem_ld_wait();
         if (!row_valid) continue;
         if (p.splits == 1) {
@@ -507,7 +630,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
 #pragma unroll
           for (int j = 0; j < 4; ++j) dst[j] = pk[j];
         } else {
-          float4* dst = reinterpret_cast<float4*>(p.ws_o + (static_cast<size_t>(split) * p.T * p.Hq + out_row) * TD + c0);
+          float4* dst = reinterpret_cast<float4*>(p.ws_o + ((static_cast<size_t>(split) * p.T * p.Hq + out_row) * MAPS + map) * TD + c0);
 #pragma unroll
           for (int j = 0; j < 8; ++j)
             dst[j] = make_float4(__uint_as_float(orr[4 * j]), __uint_as_float(orr[4 * j + 1]),
@@ -515,7 +638,7 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
         }
       }
       if (p.splits > 1 && row_valid) {
-        float* ml = p.ws_ml + (static_cast<size_t>(split) * p.T * p.Hq + out_row) * 2;
+        float* ml = p.ws_ml + ((static_cast<size_t>(split) * p.T * p.Hq + out_row) * MAPS + map) * 2;
         ml[0] = m_run;
         ml[1] = l_run;
       }
@@ -597,16 +720,52 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
   if (tid == 0) attn_trace(4);      // epilogue stores issued
   tc_fence_before();
   __syncthreads();
-  if (warp == 4 && nt > 0) {
+  if (warp == MMA_WARP && nt > 0) {
     tc_fence_after();
-    tmem_dealloc(tmem_base, 256);
+    tmem_dealloc(tmem_base, 256 * MAPS);
   }
 }
 
-template <int G>
+// merge of the key splits of a differential attention: one warp per (token, head) norms the difference of the merged maps
+__global__ void __launch_bounds__(256) diff_merge_kernel(AttnTcParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int rows = p.T * p.Hq;
+  if (row >= rows) return;
+  const float lam = *p.lam;
+  float o[4] = {}, ss = 0.f;
+#pragma unroll
+  for (int m = 0; m < 2; ++m) {
+    const size_t at = static_cast<size_t>(row) * 2 + m, stride = static_cast<size_t>(rows) * 2;
+    float top = -INFINITY;
+    for (int s = 0; s < p.splits; ++s) top = fmaxf(top, p.ws_ml[(s * stride + at) * 2]);
+    float acc[4] = {}, l = 0.f;
+    for (int s = 0; s < p.splits; ++s) {
+      const float ms = p.ws_ml[(s * stride + at) * 2], ls = p.ws_ml[(s * stride + at) * 2 + 1];
+      if (ms == -INFINITY) continue;   // this split saw no visible key (its O may be unwritten)
+      const float w = exp2f(ms - top);
+      l += ls * w;
+      const float4 v = *reinterpret_cast<const float4*>(p.ws_o + (s * stride + at) * TD + lane * 4);
+      acc[0] += v.x * w; acc[1] += v.y * w; acc[2] += v.z * w; acc[3] += v.w * w;
+    }
+    const float f = (l > 0.f ? 1.f / l : 0.f) * (m == 0 ? 1.f : -lam);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[j] += acc[j] * f;
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) ss += o[j] * o[j];
+  const float r = p.share / sqrtf(warp_sum(ss) / p.V + p.eps);
+  __nv_bfloat16* dst = p.out + static_cast<size_t>(row / p.Hq) * p.ldo + (row % p.Hq) * TD + lane * 4;
+  *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(o[0] * r, o[1] * r);
+  *reinterpret_cast<__nv_bfloat162*>(dst + 2) = __floats2bfloat162_rn(o[2] * r, o[3] * r);
+}
+
+template <int G, int MODE>
 static int launch_attn_tc(const AttnTcParams& p, int q_tiles, bool pdl, cudaStream_t stream) {
   static int configured[kMaxDevicesCached] = {};
-  auto kern = paged_tree_attn_tc_kernel<G>;
+  constexpr int kAttnTcSmem = attn_tc_smem(MODE);
+  auto kern = paged_tree_attn_tc_kernel<G, MODE>;
   if (ensure_dyn_smem(kern, kAttnTcSmem, configured) != 0) return -3;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(q_tiles, p.Hkv, p.splits);
@@ -649,12 +808,13 @@ extern "C" int js_attn_tc_max_active_clusters(int G, int splits) {
   using namespace js;
   if (splits < 1 || splits > kMaxClusterSplits) return -1;
   const void* kern = nullptr;
+  constexpr int kAttnTcSmem = attn_tc_smem(kPlain);      // what kPooled takes as well
   switch (G) {
-    case 1: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<1>); break;
-    case 2: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<2>); break;
-    case 4: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<4>); break;
-    case 8: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<8>); break;
-    case 16: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<16>); break;
+    case 1: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<1, kPlain>); break;
+    case 2: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<2, kPlain>); break;
+    case 4: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<4, kPlain>); break;
+    case 8: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<8, kPlain>); break;
+    case 16: kern = reinterpret_cast<const void*>(paged_tree_attn_tc_kernel<16, kPlain>); break;
     default: return -2;
   }
   if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, kAttnTcSmem) != cudaSuccess) return -3;
@@ -679,14 +839,21 @@ extern "C" int js_attn_tc_max_active_clusters(int G, int splits) {
 // W <= 8 (windows of up to 256 nodes).
 // window > 0 limits a row to the last `window` tokens of its own path and the positions below `keep`; sink adds a valueless
 // key of score sinks[head] (null: 0); gate (T, ldg) fp32 logits multiply a head's output by their sigmoid (null: none).
+// softcap > 0 caps the scores, cap_poly says that no score exceeds 0.35 softcap; P > 0 adds the pooled blocks of P tokens
+// that end before a row's window (kb, vb (Hkv, block_rows, 128) through block_map (max_seqs, max_blocks)); over a token tree the
+// window must reach past the tree.  maps 2: differential attention with lam (device), share, eps and V value columns, q and pool
+// rows 64 columns a map, ws_o and ws_ml twice as many rows; without a window, sinks or gates.
 extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const void* v_pool, const int* slot_map,
                                       const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
                                       float* ws_o, float* ws_ml, int* status, int B, int T, int Hq, int Hkv, int S, int max_len, int W,
                                       int causal, int splits, float scale, int window, int sink, int keep, const float* sinks,
-                                      const float* gate, int ldg, long long kv_head, long long kv_slot, int ldo, int pdl,
-                                      cudaStream_t stream) {
+                                      const float* gate, int ldg, float softcap, int cap_poly, int P, const void* kb, const void* vb,
+                                      int block_rows, const int* block_map, int max_blocks, int maps, const float* lam, float share,
+                                      float eps, int V, long long kv_head, long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
   using namespace js;
-  if (window < 0 || keep < 0) return -10;
+  if (window < 0 || keep < 0 || softcap < 0.f || P < 0 || maps < 1 || maps > 2) return -10;
+  if (P > 0 && (window < 1 || kb == nullptr || vb == nullptr || block_map == nullptr)) return -13;
+  if (maps == 2 && (window || sink || gate != nullptr || P || softcap > 0.f || lam == nullptr || V < 1 || V > TD)) return -13;
   if (T <= 0 || B <= 0) return 0;
   if (Hq % Hkv) return -10;
   if ((kv_head % 8) || (kv_slot % 8) || (ldo % 8)) return -10;
@@ -696,7 +863,7 @@ extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const v
   if (!causal && (mask_bits == nullptr || W < 1 || W > 8)) return -13;
   // The key splits merge inside a cluster only while every cluster of the launch is resident at once (a second
   // wave would double the kernel's time); otherwise partials go through the workspace and the merge kernel.
-  bool in_cluster = splits >= 2 && splits <= kMaxClusterSplits;
+  bool in_cluster = maps == 1 && splits >= 2 && splits <= kMaxClusterSplits;
   if (in_cluster) {
     static int room[kMaxDevicesCached][5][kMaxClusterSplits + 1] = {};     // 0 = not asked yet
     int dev = 0;
@@ -716,18 +883,34 @@ extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const v
                  reinterpret_cast<const __nv_bfloat16*>(v_pool), slot_map, seq_rows, cu_q, past_lens, mask_bits,
                  reinterpret_cast<__nv_bfloat16*>(out), ws_o, ws_ml, status, B, T, Hq, Hkv, S, max_len, W, causal,
                  splits, scale * 1.4426950408889634f, kv_head, kv_slot, ldo, window, sink, keep, sinks, gate, ldg,
-                 in_cluster ? 1 : 0};
-  int rc;
-  switch (G) {
-    case 1: rc = launch_attn_tc<1>(p, (T + 127) / 128 + B, pdl != 0, stream); break;
-    case 2: rc = launch_attn_tc<2>(p, (T + 63) / 64 + B, pdl != 0, stream); break;
-    case 4: rc = launch_attn_tc<4>(p, (T + 31) / 32 + B, pdl != 0, stream); break;
-    case 8: rc = launch_attn_tc<8>(p, (T + 15) / 16 + B, pdl != 0, stream); break;
-    case 16: rc = launch_attn_tc<16>(p, (T + 7) / 8 + B, pdl != 0, stream); break;
-    default: return -14;
-  }
+                 in_cluster ? 1 : 0, softcap * 1.4426950408889634f, softcap > 0.f ? scale / softcap : 0.f, cap_poly, P,
+                 reinterpret_cast<const __nv_bfloat16*>(kb), reinterpret_cast<const __nv_bfloat16*>(vb), block_map, block_rows, max_blocks,
+                 lam, share, eps, V};
+  auto launch = [&](auto mode) {
+    constexpr int M = decltype(mode)::value;
+    switch (G) {
+      case 1: return launch_attn_tc<1, M>(p, (T + 127) / 128 + B, pdl != 0, stream);
+      case 2: return launch_attn_tc<2, M>(p, (T + 63) / 64 + B, pdl != 0, stream);
+      case 4: return launch_attn_tc<4, M>(p, (T + 31) / 32 + B, pdl != 0, stream);
+      case 8: return launch_attn_tc<8, M>(p, (T + 15) / 16 + B, pdl != 0, stream);
+      case 16: return launch_attn_tc<16, M>(p, (T + 7) / 8 + B, pdl != 0, stream);
+      default: return -14;
+    }
+  };
+  const int rc = maps == 2 ? launch(std::integral_constant<int, kDiff>{})
+               : P > 0 || softcap > 0.f ? launch(std::integral_constant<int, kPooled>{}) : launch(std::integral_constant<int, kPlain>{});
   if (rc != 0 || splits == 1 || p.cluster_merge) return rc;
-  return js_attn_merge(ws_o, ws_ml, gate, ldg, out, ldo, T, Hq, splits, pdl, stream);
+  if (maps == 1) return js_attn_merge(ws_o, ws_ml, gate, ldg, out, ldo, T, Hq, splits, pdl, stream);
+  cudaLaunchConfig_t c2 = {};
+  c2.gridDim = dim3((T * Hq + 7) / 8);
+  c2.blockDim = dim3(256);
+  c2.stream = stream;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  c2.attrs = attr;
+  c2.numAttrs = pdl ? 1 : 0;
+  return cudaLaunchKernelEx(&c2, diff_merge_kernel, p) == cudaSuccess ? 0 : -5;
 }
 
 // The same without a window; sinks and gate may be null.
@@ -738,8 +921,8 @@ extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, 
                                           float scale, const float* sinks, const float* gate, int ldg, long long kv_head,
                                           long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
   return js_window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ws_o, ws_ml, status, B, T, Hq,
-                                Hkv, S, max_len, W, causal, splits, scale, 0, sinks != nullptr, 0, sinks, gate, ldg, kv_head, kv_slot, ldo,
-                                pdl, stream);
+                                Hkv, S, max_len, W, causal, splits, scale, 0, sinks != nullptr, 0, sinks, gate, ldg, 0.f, 0, 0, nullptr, nullptr, 0,
+                                nullptr, 0, 1, nullptr, 0.f, 0.f, js::TD, kv_head, kv_slot, ldo, pdl, stream);
 }
 
 // Same arguments as js_paged_tree_attention.

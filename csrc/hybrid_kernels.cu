@@ -202,7 +202,7 @@ pool_blocks_kernel(const E* kp, const E* vp, E* kb, E* vb, int S, int rows, int 
 // (or 0).  With `gate` (T, ldg) the head's output is multiplied by the sigmoid of its logit.  softcap > 0 caps the scores.
 // Pooled blocks of P positions that end before the window are keys too, read from their rows or, where they reach into a token
 // tree, averaged over the row's path.  MAPS = 2: two queries a head against the two halves of a key row, outputs combined to
-// share * (o1 - lam o2) / rms.
+// share * (o1 - lam o2) / rms over Vn columns (the rest of V is padding).
 struct WindowSimt {
   const void *q, *kpool, *vpool, *kblocks, *vblocks;
   void* out;
@@ -210,7 +210,7 @@ struct WindowSimt {
   const float *sinks, *gate, *lam;
   int* status;
   long long q_tok;
-  int Dp, Vp, ldo, B, H, G, D, V, S, max_len, W, causal, window, sink, keep, ldg, P, block_rows, max_blocks;
+  int Dp, Vp, ldo, B, H, G, D, V, S, max_len, W, causal, window, sink, keep, ldg, P, block_rows, max_blocks, Vn;
   float scale, softcap, share, eps;
 };
 
@@ -373,7 +373,7 @@ __global__ void __launch_bounds__(128) window_attn_simt_kernel(WindowSimt p) {
       o[e] = c < V ? read(0, c) - lam * read(1, c) : 0.f;
       ss += o[e] * o[e];
     }
-    const float r = p.share / sqrtf(cta_sum<128>(ss, red) / V + p.eps);
+    const float r = p.share / sqrtf(cta_sum<128>(ss, red) / p.Vn + p.eps);
 #pragma unroll
     for (int e = 0; e < (NPL + 3) / 4; ++e) {
       const int c = threadIdx.x + 128 * e;
@@ -649,21 +649,21 @@ extern "C" int js_pool_blocks(const void* kp, const void* vp, void* kb, void* vb
 // q: token t at t * q_tok, head h (map m) at (h * maps + m) * D; pools (G, S, Dp) and (G, S, Vp); out (T, ldo), head h at h * V.
 // D, V at most 512.  sink: a valueless key of score sinks[h] (null: 0) takes part; keep: positions below it stay visible behind the
 // window (0: no window); gate (T, ldg) fp32 logits or null; softcap 0: none; P > 0: pooled blocks in kb (G, block_rows, Dp), vb
-// (G, block_rows, Vp) through block_map (rows, max_blocks); maps 2 combines with lam (device), share and eps.
+// (G, block_rows, Vp) through block_map (rows, max_blocks); maps 2 combines with lam (device), share and eps, normed over the first Vn of V columns (the rest being zero).
 extern "C" int js_window_attention_simt(const void* q, long long q_tok, const void* kp, const void* vp, int Dp, int Vp, const int* slot_map,
                                         const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
                                         int ldo, int B, int T, int H, int G, int D, int V, int S, int max_len, int W, int causal,
                                         float scale, int window, int sink, int keep, const float* sinks, const float* gate, int ldg,
                                         float softcap, int P, const void* kb, const void* vb, int block_rows, const int* block_map,
-                                        int max_blocks, int maps, const float* lam, float share, float eps, int bf16, int* status, int pdl,
+                                        int max_blocks, int maps, const float* lam, float share, float eps, int Vn, int bf16, int* status, int pdl,
                                         cudaStream_t stream) {
   using namespace js;
   if (T <= 0 || B <= 0) return 0;
   if (maps < 1 || maps > 2 || H % G || D > 512 || V > 512 || Dp % maps || D > Dp / maps || V > Vp || window < 0 || keep < 0 || P < 0) return -10;
   if (!causal && (mask_bits == nullptr || W < 1)) return -13;
-  if ((P > 0 && (window < 1 || kb == nullptr || vb == nullptr || block_map == nullptr)) || (maps == 2 && lam == nullptr)) return -13;
+  if ((P > 0 && (window < 1 || kb == nullptr || vb == nullptr || block_map == nullptr)) || (maps == 2 && (lam == nullptr || Vn < 1 || Vn > V))) return -13;
   WindowSimt p{q, kp, vp, kb, vb, out, slot_map, seq_rows, cu_q, past_lens, mask_bits, block_map, sinks, gate, lam, status, q_tok,
-               Dp, Vp, ldo, B, H, G, D, V, S, max_len, W, causal, window, sink, keep, ldg, P, block_rows, max_blocks,
+               Dp, Vp, ldo, B, H, G, D, V, S, max_len, W, causal, window, sink, keep, ldg, P, block_rows, max_blocks, Vn,
                scale, softcap, share, eps};
   if (bf16) return maps == 2 ? launch_window_simt<__nv_bfloat16, 2>(p, T, pdl, stream) : launch_window_simt<__nv_bfloat16, 1>(p, T, pdl, stream);
   return maps == 2 ? launch_window_simt<float, 2>(p, T, pdl, stream) : launch_window_simt<float, 1>(p, T, pdl, stream);

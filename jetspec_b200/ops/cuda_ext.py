@@ -951,9 +951,10 @@ def rotate_norm(x: torch.Tensor, positions: torch.Tensor, dims: int, base: float
 
 def window_attention(q, k_pool, v_pool, vdim: int, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int,
                      sink, causal: bool, out: Optional[torch.Tensor] = None, pdl: bool = False, keep_first: int = 0,
-                     gate: Optional[torch.Tensor] = None, softcap: float = 0.0, blocks=None, diff=None) -> torch.Tensor:
+                     gate: Optional[torch.Tensor] = None, softcap: float = 0.0, blocks=None, diff=None,
+                     norm_dim: Optional[int] = None) -> torch.Tensor:
     """Window attention on the plain cores (bf16 or fp32, heads of up to 512); see the reference op for the arguments.  ``gate``:
-    logits whose sigmoid multiplies a head's output (one map a head)."""
+    logits whose sigmoid multiplies a head's output (one map a head).  ``norm_dim``: columns of ``vdim`` that are not padding."""
     sinks = sink.detach().float().contiguous() if isinstance(sink, torch.Tensor) else None
     lib = load()
     T, H, D = q.shape
@@ -971,7 +972,7 @@ def window_attention(q, k_pool, v_pool, vdim: int, slot_map, seq_rows, cu_q, pas
         mask_bits.shape[1] if mask_bits is not None else 0, int(causal), ctypes.c_float(scale), int(window),
         int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, H), *_head_gate(gate), ctypes.c_float(softcap), int(P), _p(kb),
         _p(vb), kb.shape[1] if P else 0, _p(block_map), block_map.shape[1] if P else 0, maps, _p(lam), ctypes.c_float(share), ctypes.c_float(eps),
-        _is_bf16(q), _p(status_word(q.device)), int(pdl), _stream()), "js_window_attention_simt")
+        int(norm_dim or vdim), _is_bf16(q), _p(status_word(q.device)), int(pdl), _stream()), "js_window_attention_simt")
     return out
 
 
@@ -1023,7 +1024,10 @@ def sandwich(y, src, w, x, next_norm, eps: float, h, width: int, hist: Optional[
 
 def window_tc_ok(maps: int, pool: int, softcap: float) -> bool:
     """Whether the tensor-core kernel has a form for these options."""
-    return maps == 1 and pool == 0 and softcap == 0.0
+    return maps == 1 or (maps == 2 and pool == 0 and softcap == 0.0)
+
+
+TANH_SMALL = 0.35        # |score / cap| up to which the tensor-core kernel caps with a polynomial
 
 
 def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int, keep_first: int = 0, pool: int = 0) -> int:
@@ -1035,11 +1039,17 @@ def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int, ke
 
 def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int, sink,
                         causal: bool, out: torch.Tensor, splits: int = 1, ws: Optional[dict] = None, pdl: bool = False,
-                        keep_first: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        keep_first: int = 0, gate: Optional[torch.Tensor] = None, softcap: float = 0.0, score_bound: Optional[float] = None,
+                        blocks=None, diff=None, vdim: int = 128) -> torch.Tensor:
     """Window attention on the tcgen05 kernel: bf16, heads padded to 128, groups of 1, 2, 4, 8 or 16 query heads.  ``sink``:
     whether a valueless key of score 0 takes part, or its score per head, fp32 ``(Hq,)``; ``gate (T, >= Hq)``: logits whose
-    sigmoid multiplies a head's output."""
+    sigmoid multiplies a head's output.  ``softcap``, ``blocks``: see the reference op (trees must not be deeper than the window);
+    ``score_bound``: what no scaled score can exceed, where that is known.  ``diff = (lam, share, eps)``: ``q (T, Hq, 128)`` and the
+    pools' keys hold 64 columns for each of two maps, ``vdim`` is the true width of the values."""
     lib = load()
+    maps, (lam, share, eps) = (1, (None, 0.0, 0.0)) if diff is None else (2, diff)
+    kb, vb, block_map, P = blocks if blocks is not None else (None, None, None, 0)
+    poly = softcap > 0.0 and score_bound is not None and score_bound <= TANH_SMALL * softcap
     T, Hq, D = q.shape
     sinks = sink if isinstance(sink, torch.Tensor) else None
     G, S, _ = k_pool.shape
@@ -1048,8 +1058,9 @@ def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, 
         _p(q), _p(k_pool), _p(v_pool), _p(slot_map), _p(seq_rows), _p(cu_q), _p(past_lens), _p(mask_bits), _p(out),
         _p(ws["o"] if splits > 1 else None), _p(ws["ml"] if splits > 1 else None), _p(status_word(q.device)), seq_rows.numel(), T, Hq,
         G, S, slot_map.shape[1], mask_bits.shape[1] if mask_bits is not None else 0, int(causal), int(splits), ctypes.c_float(scale),
-        int(window), int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, Hq), *_head_gate(gate),
-        ctypes.c_longlong(S * 128), ctypes.c_longlong(128), out.stride(0), int(pdl), _stream()), "js_window_attention_tc")
+        int(window), int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, Hq), *_head_gate(gate), ctypes.c_float(softcap),
+        int(poly), int(P), _p(kb), _p(vb), kb.shape[1] if P else 0, _p(block_map), block_map.shape[1] if P else 0, maps, _p(lam),
+        ctypes.c_float(share), ctypes.c_float(eps), int(vdim), ctypes.c_longlong(S * 128), ctypes.c_longlong(128), out.stride(0), int(pdl), _stream()), "js_window_attention_tc")
     return out
 
 

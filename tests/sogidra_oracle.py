@@ -184,11 +184,11 @@ def random_weights(cfg, seed=0, dtype=torch.float64):
         p, m, f = f"l{i}", L["mixer"], L["mlp"]
         H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         for n in ("norm1", "norm1b") + (("norm2", "norm2b") if f is not None else ()):
-            vec(f"{p}.{n}", W, 0.0, 0.2)
+            vec(f"{p}.{n}", W, -0.3 if n.endswith("b") else 0.0, 0.2)
         if L["type"] == "attention":
             for n, c in (("q", 2 * H * D), ("k", 2 * G * D), ("v", G * E)):
                 if n == "q" or m.get("kv_from") is None:
-                    mat(f"{p}.mix.{n}", c, W, std=1.5 / math.sqrt(W))
+                    mat(f"{p}.mix.{n}", c, W)
                     vec(f"{p}.mix.{n}.b", c, 0.0, 0.5)
             for n in ("lq1", "lk1", "lq2", "lk2"):
                 vec(f"{p}.mix.{n}", D, 0.3 if n == "lq1" else 0.0, 0.8 / math.sqrt(D) ** 0.5)
