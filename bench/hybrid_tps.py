@@ -100,7 +100,7 @@ def kernel_table(T, context, n_seq):
         p(X.status_word(dev)), 0, X._stream()), "post")], T * win_cols * 4, 0, 8, "qwen3 head norms + RoPE + KV scatter")
     seen_w = n_seq * sum(min(WIN, context + i + 1) for i in range(per))
     keys_w = n_seq * min(context + per, WIN + per - 1)
-    sp = X.window_attn_splits(T, 16, 4, context + per, WIN)
+    sp = X.window_attn_splits(T, 16, 4, context + per, WIN, seqs=n_seq)
     ws = {"o": torch.zeros(sp, T, 16, D, device=dev), "ml": torch.zeros(sp, T, 16, 2, device=dev)}
     wo = bf(T, 16 * D)
     add("zasipel window attention", [lambda k=k, v=v: X.window_attention_tc(wq.view(T, 16, D), k, v, smap, srow, cu, past, None, D ** -0.5, WIN, True,

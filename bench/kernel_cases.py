@@ -6,6 +6,7 @@
     python bench/kernel_cases.py latent_attention # latent attention: 16 requests, one token x 32 heads, 2k cached rows of 512
     python bench/kernel_cases.py delta_rule  # a prompt portion through the block form of the gated delta rule
     python bench/kernel_cases.py retention   # a prompt portion of 2048 rows through the chunk form of the retention, 16 heads of 128 x 256
+    python bench/kernel_cases.py depth       # a prompt of 2048 rows: pooled and differential attention, the step at a layer's end (9 terms)
     python bench/kernel_cases.py parallel_block   # input / output GEMMs of a parallel block at 128 rows (fused epilogues)
     python bench/kernel_cases.py lm_head     # vocabulary GEMM with the argmax epilogue
     python bench/kernel_cases.py nvfp4       # activation quantiser + block-scaled GEMM on the same four shapes
@@ -151,6 +152,24 @@ def case_retention(reps: int = 3):
     torch.cuda.synchronize()
 
 
+def case_depth(reps: int = 3):
+    """A prompt portion of 2048 rows: window attention with pooled blocks and capped scores, differential attention (32 heads over
+    8), and the residual step with a depth average over 9 terms at width 4096."""
+    T, H, G, D, W = 2048, 32, 8, 128, 4096
+    i32 = dict(dtype=torch.int32, device="cuda")
+    q, kp, vp, out = bf(T, H, D), bf(G, T + 64, D), bf(G, T + 64, D), bf(T, H * D)
+    kb, vb, bmap = bf(G, 128, D), bf(G, 128, D), torch.randperm(128, device="cuda").to(torch.int32).view(1, 128)
+    smap, rows = torch.randperm(T + 64, device="cuda")[:T].to(torch.int32).view(1, T), torch.zeros(1, **i32)
+    cu, past, lam = torch.tensor([0, T], **i32), torch.zeros(1, **i32), torch.tensor([0.5], device="cuda")
+    hist, x, y, h = torch.randn(9, T, W, device="cuda"), torch.randn(T, W, device="cuda"), bf(T, W), bf(T, W)
+    one, d = torch.ones(W, device="cuda"), torch.rand(9, device="cuda")
+    for _ in range(reps):
+        X.window_attention_tc(q, kp, vp, smap, rows, cu, past, None, D ** -0.5, 1024, False, True, out, softcap=50.0, blocks=(kb, vb, bmap, 16))
+        X.window_attention_tc(q, kp, vp, smap, rows, cu, past, None, 0.125, 0, False, True, out, diff=(lam, 0.6, 1e-5))
+        X.sandwich(y, x, one, x, one, 1e-5, h, W, hist=hist, d=d)
+    torch.cuda.synchronize()
+
+
 def case_round_small(reps: int = 2):
     """The small kernels of a decode round at Qwen3-8B sizes: RMSNorm, per-head norm + RoPE + KV scatter, the
     draft head's vocabulary top-k (GEMM epilogue + merge), device tree build, accept + commit, KV compaction."""
@@ -239,7 +258,7 @@ def case_collectives(reps: int = 3):
 if __name__ == "__main__":
     X.load()
     {"gemm": case_gemm, "gemm_rows2048": case_gemm_rows2048, "lm_head": case_lm_head, "attention": case_attention,
-     "latent_attention": case_latent_attention, "delta_rule": case_delta_rule, "retention": case_retention, "parallel_block": case_parallel_block, "nvfp4": case_nvfp4,
+     "latent_attention": case_latent_attention, "delta_rule": case_delta_rule, "retention": case_retention, "depth": case_depth, "parallel_block": case_parallel_block, "nvfp4": case_nvfp4,
      "round_small": case_round_small, "collectives": case_collectives}[sys.argv[1]]()
     X.check_status("cuda")
     print("ok")

@@ -80,7 +80,8 @@ def throughput(name, cfg, prompt=2048, context=2048, batches=(1, 16)):
     out = {"model": name, "family": cfg.model_type, "layer_runs": cfg.num_hidden_layers, "cache_bytes_per_token": 0}
     eng._ensure_pool((max(prompt, context) + 48) * max(batches), seqs=max(batches))
     pool, fast = eng.pool, FastRound.get(eng)
-    bufs = [b for b in pool.latent_pools or [] if b is not None] + [b for kv in pool.kv_layers or [] if kv is not None for b in kv]
+    held = {id(kv): kv for kv in (*(pool.kv_layers or []), *(pool.kv_blocks or [])) if kv is not None}        # shared pools once
+    bufs = [b for b in pool.latent_pools or [] if b is not None] + [b for kv in held.values() for b in kv]
     bufs = bufs or [pool.k_pool, pool.v_pool]
     if pool.states is not None:
         out["state_bytes_per_sequence"] = sum(t[0].numel() * t.element_size() for t in (*pool.states.state, *pool.states.conv) if t is not None)

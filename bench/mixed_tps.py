@@ -108,7 +108,7 @@ def kernel_table(T, context, n_seq):
         status, 0, X._stream()), "post")], T * 6144 * 4, 0, 8, "qwen3 head norms + RoPE + KV scatter")
     seen_w = n_seq * sum(min(WIN + KEEP, context + i + 1) for i in range(per))
     keys_w = n_seq * min(context + per, WIN + KEEP + per - 1)
-    sp = X.window_attn_splits(T, H, KV, context + per, WIN, KEEP)
+    sp = X.window_attn_splits(T, H, KV, context + per, WIN, KEEP, seqs=n_seq)
     ws = {"o": torch.zeros(sp, T, H, D, device=dev), "ml": torch.zeros(sp, T, H, 2, device=dev)}
     sinks, gate = torch.randn(H, device=dev), torch.randn(T, 128, device=dev)
     add(f"kizezen window attention, sinks, gate ({sp} splits)", [lambda k=k, v=v: X.window_attention_tc(

@@ -78,8 +78,7 @@ struct AttnTcParams {
   int ldg;
   int cluster_merge;           // the key splits of a tile form a cluster and merge through distributed shared memory
   // kPooled
-  float cap_log2, inv_cap;     // score cap in the log2 domain (0: none), scale / cap
-  int cap_poly;                // |score / cap| is small enough for the polynomial
+  float cap_log2, cap_in;      // score cap in the log2 domain (0: none), 2 log2(e) scale / cap
   int P;                       // tokens to a block, 0 without blocks
   const __nv_bfloat16 *kb_pool, *vb_pool;      // (Hkv, block_rows, 128)
   const int* block_map;        // (max_seqs, max_blocks)
@@ -90,16 +89,12 @@ struct AttnTcParams {
   int V;                       // true width of a head's values
 };
 
-// cap tanh(s / cap) in the log2 domain for x = s / cap; the polynomial is for |x| up to 0.35 (error below 1e-7)
-JS_DEVICE float capped_poly(float x, float cap_log2) {
-  const float u = x * x;       // Taylor series of tanh(x) / x
-  return cap_log2 * x * (1.f + u * (-1.f / 3.f + u * (2.f / 15.f + u * (-17.f / 315.f + u * (62.f / 2835.f)))));
-}
-JS_DEVICE float capped_any(float x, float cap_log2) {
+// cap tanh(s / cap) in the log2 domain, x = 2 log2(e) s / cap: absolute error below 1e-5 for caps up to 100
+JS_DEVICE float capped(float x, float cap_log2) {
   float e, r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * 2.8853900817779268f));      // e^(2x)
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x));
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
-  return cap_log2 - 2.f * cap_log2 * r;
+  return fmaf(-2.f * cap_log2, r, cap_log2);
 }
 
 JS_DEVICE void cp_async16_tc(uint32_t smem_addr, const void* gmem, bool valid) {
@@ -498,13 +493,8 @@ __global__ void __launch_bounds__(TTHREADS, 1) paged_tree_attn_tc_kernel(AttnTcP
       float to_log2 = p.scale_log2;
       if constexpr (MODE == kPooled) {
         if (p.cap_log2 > 0.f) {
-          if (p.cap_poly) {
 #pragma unroll
-            for (int c = 0; c < 64; ++c) sr[c] = __float_as_uint(capped_poly(__uint_as_float(sr[c]) * p.inv_cap, p.cap_log2));
-          } else {
-#pragma unroll
-            for (int c = 0; c < 64; ++c) sr[c] = __float_as_uint(capped_any(__uint_as_float(sr[c]) * p.inv_cap, p.cap_log2));
-          }
+          for (int c = 0; c < 64; ++c) sr[c] = __float_as_uint(capped(__uint_as_float(sr[c]) * p.cap_in, p.cap_log2));
           to_log2 = 1.f;
         }
       }
@@ -839,7 +829,7 @@ extern "C" int js_attn_tc_max_active_clusters(int G, int splits) {
 // W <= 8 (windows of up to 256 nodes).
 // window > 0 limits a row to the last `window` tokens of its own path and the positions below `keep`; sink adds a valueless
 // key of score sinks[head] (null: 0); gate (T, ldg) fp32 logits multiply a head's output by their sigmoid (null: none).
-// softcap > 0 caps the scores, cap_poly says that no score exceeds 0.35 softcap; P > 0 adds the pooled blocks of P tokens
+// softcap > 0 caps the scores; P > 0 adds the pooled blocks of P tokens
 // that end before a row's window (kb, vb (Hkv, block_rows, 128) through block_map (max_seqs, max_blocks)); over a token tree the
 // window must reach past the tree.  maps 2: differential attention with lam (device), share, eps and V value columns, q and pool
 // rows 64 columns a map, ws_o and ws_ml twice as many rows; without a window, sinks or gates.
@@ -847,7 +837,7 @@ extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const v
                                       const int* seq_rows, const int* cu_q, const int* past_lens, const int* mask_bits, void* out,
                                       float* ws_o, float* ws_ml, int* status, int B, int T, int Hq, int Hkv, int S, int max_len, int W,
                                       int causal, int splits, float scale, int window, int sink, int keep, const float* sinks,
-                                      const float* gate, int ldg, float softcap, int cap_poly, int P, const void* kb, const void* vb,
+                                      const float* gate, int ldg, float softcap, int P, const void* kb, const void* vb,
                                       int block_rows, const int* block_map, int max_blocks, int maps, const float* lam, float share,
                                       float eps, int V, long long kv_head, long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
   using namespace js;
@@ -883,7 +873,7 @@ extern "C" int js_window_attention_tc(const void* q, const void* k_pool, const v
                  reinterpret_cast<const __nv_bfloat16*>(v_pool), slot_map, seq_rows, cu_q, past_lens, mask_bits,
                  reinterpret_cast<__nv_bfloat16*>(out), ws_o, ws_ml, status, B, T, Hq, Hkv, S, max_len, W, causal,
                  splits, scale * 1.4426950408889634f, kv_head, kv_slot, ldo, window, sink, keep, sinks, gate, ldg,
-                 in_cluster ? 1 : 0, softcap * 1.4426950408889634f, softcap > 0.f ? scale / softcap : 0.f, cap_poly, P,
+                 in_cluster ? 1 : 0, softcap * 1.4426950408889634f, softcap > 0.f ? 2.8853900817779268f * scale / softcap : 0.f, P,
                  reinterpret_cast<const __nv_bfloat16*>(kb), reinterpret_cast<const __nv_bfloat16*>(vb), block_map, block_rows, max_blocks,
                  lam, share, eps, V};
   auto launch = [&](auto mode) {
@@ -921,7 +911,7 @@ extern "C" int js_paged_attention_tc_strided(const void* q, const void* k_pool, 
                                           float scale, const float* sinks, const float* gate, int ldg, long long kv_head,
                                           long long kv_slot, int ldo, int pdl, cudaStream_t stream) {
   return js_window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, out, ws_o, ws_ml, status, B, T, Hq,
-                                Hkv, S, max_len, W, causal, splits, scale, 0, sinks != nullptr, 0, sinks, gate, ldg, 0.f, 0, 0, nullptr, nullptr, 0,
+                                Hkv, S, max_len, W, causal, splits, scale, 0, sinks != nullptr, 0, sinks, gate, ldg, 0.f, 0, nullptr, nullptr, 0,
                                 nullptr, 0, 1, nullptr, 0.f, 0.f, js::TD, kv_head, kv_slot, ldo, pdl, stream);
 }
 

@@ -142,58 +142,178 @@ __global__ void __launch_bounds__(256) window_post_kernel(WindowPostParams p) {
     dst[d] = __float2bfloat16_rn(d < p.V ? __bfloat162float(row[c + d]) + (p.bias != nullptr ? p.bias[c + d] : 0.f) : 0.f);
 }
 
+// The same without rotation, 8 entries a thread: 2^lp neighbouring lanes make a head vector, 2^lpv a value row.  With tied values
+// the key's lanes store the value row too.  D, V, the widths, ldp and vcol multiples of 8.
+__global__ void __launch_bounds__(256) window_post_vec_kernel(WindowPostParams p, int lp, int lpv, int tied) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, idx = blockIdx.y * 256 + threadIdx.x;
+  const int nq = p.H * p.maps, nk = p.kv ? p.G * p.maps : 0, nv = p.kv && !tied ? p.G : 0;
+  const int vectors = (nq + nk) << lp, share = p.Dp / p.maps;
+  const __nv_bfloat16* row = p.proj + static_cast<size_t>(t) * p.ldp;
+  const bool head = idx < vectors, value = !head && idx - vectors < nv << lpv;
+  const int u = head ? idx >> lp : (idx - vectors) >> lpv;
+  const int e = 8 * (head ? idx & ((1 << lp) - 1) : (idx - vectors) & ((1 << lpv) - 1));
+  const int col = (head ? u * p.D : p.vcol + u * p.V) + e;
+  float v[8] = {}, ss = 0.f;
+  if ((head || value) && e < (head ? p.D : p.V)) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(row + col);
+    const __nv_bfloat162* r2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 f = __bfloat1622float2(r2[j]);
+      v[2 * j] = f.x;
+      v[2 * j + 1] = f.y;
+    }
+    if (p.bias != nullptr) {
+      const float4 a = *reinterpret_cast<const float4*>(p.bias + col), b = *reinterpret_cast<const float4*>(p.bias + col + 4);
+      v[0] += a.x; v[1] += a.y; v[2] += a.z; v[3] += a.w;
+      v[4] += b.x; v[5] += b.y; v[6] += b.z; v[7] += b.w;
+    }
+  }
+  auto store = [&](__nv_bfloat16* dst, float f) {
+    uint4 out;
+    __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o2[j] = __floats2bfloat162_rn(v[2 * j] * f, v[2 * j + 1] * f);
+    *reinterpret_cast<uint4*>(dst) = out;
+  };
+  float f = 1.f;
+  if (p.norm) {                              // every lane takes part
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+    for (int o = 1; o < 1 << lp; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    f = 1.f / sqrtf(ss / p.D + p.eps);
+  }
+  if (!head && !value) return;
+  if (head && u < nq) {
+    if (e >= p.Dq) return;
+    if (p.temp_every > 0) f *= 1.f + p.temp_coef * logf(static_cast<float>((p.positions[t] + 1) / p.temp_every + 1));
+    const int h = u / p.maps, group = p.H / p.G, hp = (h / group) * p.Gp + h % group;
+    store(p.qout + ((static_cast<size_t>(t) * p.G * p.Gp + hp) * p.maps + u % p.maps) * p.Dq + e, f);
+    return;
+  }
+  const int slot = p.slots[t];
+  if (slot < 0 || slot >= p.S) {
+    if (e == 0) report(p.status, kBadSlot);
+    return;
+  }
+  if (head) {
+    const int i = u - nq;
+    if (e < share) store(p.kpool + (static_cast<size_t>(i / p.maps) * p.S + slot) * p.Dp + (i % p.maps) * share + e, f);
+    if (tied && e < p.Vp) store(p.vpool + (static_cast<size_t>(i) * p.S + slot) * p.Vp + e, 1.f);
+  } else if (e < p.Vp) {
+    store(p.vpool + (static_cast<size_t>(u) * p.S + slot) * p.Vp + e, 1.f);
+  }
+}
+
 // ---------------------------------------------------------------- pooled blocks
 // Means of the cached keys and values of the blocks of P tokens whose last token is among the new ones.  One CTA per (block, head).
 // New tokens of sequence b: positions past .. past + n - 1 with n = cu[b + 1] - cu[b]; with counts instead n = counts[b] positions
 // that END at past (per_seq blocks are looked at then).
-template <typename E>
-__global__ void __launch_bounds__(128)
-pool_blocks_kernel(const E* kp, const E* vp, E* kb, E* vb, int S, int rows, int Kw, int Vw, const int* block_map, int max_blocks, int P,
-                   const int* slot_map, int max_len, const int* seq_rows, const int* cu_q, const int* past_lens, const int* counts,
-                   int per_seq, int B, int* status) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int c = blockIdx.x, g = blockIdx.y;
+struct PoolBlocks {
+  const void *kp, *vp;
+  void *kb, *vb;
+  const int *block_map, *slot_map, *seq_rows, *cu_q, *past_lens, *counts;
+  int* status;
+  int S, rows, Kw, Vw, max_blocks, P, max_len, per_seq, B;
+};
+
+// Row of the block candidate c stands for, and where its tokens' slots are; false: no such block.
+JS_DEVICE bool block_of(const PoolBlocks& p, int c, int& dst, const int*& slots) {
   int b, j, past, n;
-  if (counts != nullptr) {
-    b = c / per_seq;
-    j = c % per_seq;
-    n = counts[b];
-    past = past_lens[b] - n;
+  if (p.counts != nullptr) {
+    b = c / p.per_seq;
+    j = c % p.per_seq;
+    n = p.counts[b];
+    past = p.past_lens[b] - n;
   } else {
-    int lo = 0, hi = B - 1;
+    int lo = 0, hi = p.B - 1;
     while (lo < hi) {
       const int mid = (lo + hi + 1) >> 1;
-      if (cu_q[mid] / P + mid <= c) lo = mid; else hi = mid - 1;
+      if (p.cu_q[mid] / p.P + mid <= c) lo = mid; else hi = mid - 1;
     }
     b = lo;
-    j = c - (cu_q[b] / P + b);
-    n = cu_q[b + 1] - cu_q[b];
-    past = past_lens[b];
+    j = c - (p.cu_q[b] / p.P + b);
+    n = p.cu_q[b + 1] - p.cu_q[b];
+    past = p.past_lens[b];
   }
-  const int blk = past / P + j;
-  if (blk >= (past + n) / P) return;
-  const int row = seq_rows[b];
-  const int dst = blk < max_blocks ? block_map[static_cast<size_t>(row) * max_blocks + blk] : -1;
-  if (dst < 0 || dst >= rows) {
-    if (threadIdx.x == 0) report(status, kBadSlot);
-    return;
+  const int blk = past / p.P + j;
+  if (blk >= (past + n) / p.P) return false;
+  const int row = p.seq_rows[b];
+  dst = blk < p.max_blocks ? p.block_map[static_cast<size_t>(row) * p.max_blocks + blk] : -1;
+  if (dst < 0 || dst >= p.rows) {
+    if (threadIdx.x == 0) report(p.status, kBadSlot);
+    return false;
   }
-  const int* slots = slot_map + static_cast<size_t>(row) * max_len + static_cast<size_t>(blk) * P;
-  const float inv = 1.f / P;
-  for (int e = threadIdx.x; e < Kw + Vw; e += blockDim.x) {
-    const bool k = e < Kw;
-    const int w = k ? Kw : Vw, col = k ? e : e - Kw;
-    const E* src = (k ? kp : vp) + static_cast<size_t>(g) * S * w + col;
+  slots = p.slot_map + static_cast<size_t>(row) * p.max_len + static_cast<size_t>(blk) * p.P;
+  return true;
+}
+
+template <typename E>
+__global__ void __launch_bounds__(128) pool_blocks_kernel(PoolBlocks p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int g = blockIdx.y;
+  int dst;
+  const int* slots;
+  if (!block_of(p, blockIdx.x, dst, slots)) return;
+  const float inv = 1.f / p.P;
+  for (int e = threadIdx.x; e < p.Kw + p.Vw; e += blockDim.x) {
+    const bool k = e < p.Kw;
+    const int w = k ? p.Kw : p.Vw, col = k ? e : e - p.Kw;
+    const E* src = reinterpret_cast<const E*>(k ? p.kp : p.vp) + static_cast<size_t>(g) * p.S * w + col;
     float acc = 0.f;
 #pragma unroll 4
-    for (int i = 0; i < P; ++i) {
+    for (int i = 0; i < p.P; ++i) {
       const int slot = slots[i];
-      if (slot >= 0 && slot < S) acc += hk_ld(src + static_cast<size_t>(slot) * w);
-      else report(status, kBadSlot);
+      if (slot >= 0 && slot < p.S) acc += hk_ld(src + static_cast<size_t>(slot) * w);
+      else report(p.status, kBadSlot);
     }
-    hk_st((k ? kb : vb) + (static_cast<size_t>(g) * rows + dst) * w + col, acc * inv);
+    hk_st(reinterpret_cast<E*>(k ? p.kb : p.vb) + (static_cast<size_t>(g) * p.rows + dst) * w + col, acc * inv);
   }
+}
+
+// bf16 rows of Kw + Vw <= 256 columns, multiples of 8: 8 warps take every eighth token each, a lane 8 columns
+__global__ void __launch_bounds__(256) pool_blocks_vec_kernel(PoolBlocks p) {
+  __shared__ float part[8][256];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int g = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int dst;
+  const int* slots;
+  if (!block_of(p, blockIdx.x, dst, slots)) return;
+  const int e = lane * 8, all = p.Kw + p.Vw;
+  const bool k = e < p.Kw;
+  const int w = k ? p.Kw : p.Vw, col = k ? e : e - p.Kw;
+  const __nv_bfloat16* src = reinterpret_cast<const __nv_bfloat16*>(k ? p.kp : p.vp) + static_cast<size_t>(g) * p.S * w + col;
+  float acc[8] = {};
+  if (e < all) {
+#pragma unroll 4
+    for (int i = warp; i < p.P; i += 8) {
+      int slot = slots[i];
+      if (slot < 0 || slot >= p.S) { report(p.status, kBadSlot); slot = 0; }
+      const uint4 raw = *reinterpret_cast<const uint4*>(src + static_cast<size_t>(slot) * w);
+      const __nv_bfloat162* r2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(r2[j]);
+        acc[2 * j] += f.x;
+        acc[2 * j + 1] += f.y;
+      }
+    }
+    *reinterpret_cast<float4*>(&part[warp][e]) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+    *reinterpret_cast<float4*>(&part[warp][e + 4]) = make_float4(acc[4], acc[5], acc[6], acc[7]);
+  }
+  __syncthreads();
+  const int c = threadIdx.x;
+  if (c >= all) return;
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) sum += part[i][c];
+  const bool ck = c < p.Kw;
+  reinterpret_cast<__nv_bfloat16*>(ck ? p.kb : p.vb)[(static_cast<size_t>(g) * p.rows + dst) * (ck ? p.Kw : p.Vw) + (ck ? c : c - p.Kw)] =
+      __float2bfloat16_rn(sum / p.P);
 }
 
 // ---------------------------------------------------------------- window attention on the plain cores
@@ -621,10 +741,21 @@ extern "C" int js_window_post(const void* proj, int ldp, const float* bias, int 
   using namespace js;
   if (T <= 0) return 0;
   if (maps < 1 || H % G || Dp > 512 * maps || Dp % maps || Dq > 512 || D > Dq || D > Dp / maps || V > Vp || dims > D || (dims & 1) || Gp < H / G) return -10;
-  HybridLaunch l(dim3(T, (H * maps + (kv ? G * (maps + 1) : 0) + 7) / 8), dim3(256), stream, pdl);
   using bf = __nv_bfloat16;
   WindowPostParams p{(const bf*)proj, bias, freq, positions, slots, (bf*)qout, (bf*)kpool, (bf*)vpool, status,
                      ldp, H, G, Gp, maps, D, V, Dq, Dp, Vp, dims, norm, S, vcol, kv, temp_every, eps, temp_coef};
+  const int share = Dp / maps, wide = Dq > share ? Dq : share;
+  const bool tied = kv && maps == 1 && vcol == H * D && V == D && Vp <= wide;
+  if (dims == 0 && ((D | V | Dq | share | Vp | ldp | vcol) & 7) == 0 && wide <= 256 && Vp <= 256 && (reinterpret_cast<uintptr_t>(proj) & 15) == 0 &&
+      (reinterpret_cast<uintptr_t>(bias) & 15) == 0) {
+    int lp = 0, lpv = 0;
+    while (8 << lp < wide) ++lp;
+    while (8 << lpv < Vp) ++lpv;
+    const int n = ((H * maps + (kv ? G * maps : 0)) << lp) + (kv && !tied ? G << lpv : 0);
+    HybridLaunch l(dim3(T, (n + 255) / 256), dim3(256), stream, pdl);
+    return cudaLaunchKernelEx(&l.c, window_post_vec_kernel, p, lp, lpv, static_cast<int>(tied)) == cudaSuccess ? 0 : -4;
+  }
+  HybridLaunch l(dim3(T, (H * maps + (kv ? G * (maps + 1) : 0) + 7) / 8), dim3(256), stream, pdl);
   return cudaLaunchKernelEx(&l.c, window_post_kernel, p) == cudaSuccess ? 0 : -4;
 }
 
@@ -637,13 +768,11 @@ extern "C" int js_pool_blocks(const void* kp, const void* vp, void* kb, void* vb
   using namespace js;
   if (B <= 0 || (counts == nullptr && T <= 0)) return 0;
   if (P < 1 || G < 1 || (counts == nullptr ? cu_q == nullptr : per_seq < 1)) return -10;
-  HybridLaunch l(dim3(counts != nullptr ? B * per_seq : T / P + B, G), dim3(128), stream, pdl);
-  using bf = __nv_bfloat16;
-  if (bf16)
-    return cudaLaunchKernelEx(&l.c, pool_blocks_kernel<bf>, (const bf*)kp, (const bf*)vp, (bf*)kb, (bf*)vb, S, rows, Kw, Vw, block_map, max_blocks, P,
-                              slot_map, max_len, seq_rows, cu_q, past_lens, counts, per_seq, B, status) == cudaSuccess ? 0 : -4;
-  return cudaLaunchKernelEx(&l.c, pool_blocks_kernel<float>, (const float*)kp, (const float*)vp, (float*)kb, (float*)vb, S, rows, Kw, Vw, block_map,
-                            max_blocks, P, slot_map, max_len, seq_rows, cu_q, past_lens, counts, per_seq, B, status) == cudaSuccess ? 0 : -4;
+  PoolBlocks p{kp, vp, kb, vb, block_map, slot_map, seq_rows, cu_q, past_lens, counts, status, S, rows, Kw, Vw, max_blocks, P, max_len, per_seq, B};
+  const bool vec = bf16 && Kw % 8 == 0 && Vw % 8 == 0 && Kw + Vw <= 256;
+  HybridLaunch l(dim3(counts != nullptr ? B * per_seq : T / P + B, G), dim3(vec ? 256 : 128), stream, pdl);
+  auto kern = vec ? pool_blocks_vec_kernel : bf16 ? pool_blocks_kernel<__nv_bfloat16> : pool_blocks_kernel<float>;
+  return cudaLaunchKernelEx(&l.c, kern, p) == cudaSuccess ? 0 : -4;
 }
 
 // q: token t at t * q_tok, head h (map m) at (h * maps + m) * D; pools (G, S, Dp) and (G, S, Vp); out (T, ldo), head h at h * V.

@@ -115,11 +115,9 @@ class WindowMixer:
         # a token tree deeper than the window would see blocks of its own nodes, which only the plain-core kernel makes
         shallow = batch.mask is None or (batch.mask.shape[1] <= 8 and (blocks is None or c.window >= batch.max_rows))
         if self.tc and shallow:
-            if c.softcap and c.qk_norm:                          # normed q and k: their product is bounded (and a little rounding)
-                more.update(score_bound=1.02 * abs(c.scale) * c.dim)
             if self.diff is not None:
                 more.update(vdim=c.vdim)
-            splits = X.window_attn_splits(T, Hq, c.kv_heads, batch.max_keys, c.window, c.keep_first, c.pool)
+            splits = X.window_attn_splits(T, Hq, c.kv_heads, batch.max_keys, c.window, c.keep_first, c.pool, batch.seq_rows.numel())
             X.window_attention_tc(q.view(T, Hq, 128), kp, vp, *args, c.scale, c.window, self.sink, batch.mask is None, o, splits=splits,
                                   ws=split_ws(st, splits, T * Hq * c.maps, 128), pdl=pdl, **more)
             n += int(splits > 1 and (self.diff is not None or not X.attn_merges_in_cluster(T, Hq, c.kv_heads, splits)))

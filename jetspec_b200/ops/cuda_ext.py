@@ -567,15 +567,16 @@ def attn_merges_in_cluster(T: int, Hq: int, Hkv: int, splits: int) -> bool:
     return ((T + npt - 1) // npt) * Hkv <= _attn_cluster_room(G, splits)
 
 
-def attn_splits_for(T: int, Hq: int, Hkv: int, max_keys: int) -> int:
-    """Key splits for ``T`` query tokens: fill the SMs with ONE wave of CTAs, a couple of key tiles per split."""
+def attn_splits_for(T: int, Hq: int, Hkv: int, max_keys: int, seqs: int = 1) -> int:
+    """Key splits for ``T`` query tokens of ``seqs`` sequences: fill the SMs with ONE wave of CTAs, a couple of key tiles per
+    split."""
     G = Hq // Hkv
     if attn_impl(Hq, Hkv) == "tc":                      # 128 rows per CTA, one CTA per SM
         # one wave of CTAs, a couple of key tiles per split.  Measured on the decode round (prefix ~2.5 k keys): more,
         # shorter splits win even when they need the separate merge launch (TP=2: 9 splits + merge 4.60 ms per round,
         # 6 splits merged inside a cluster 4.71 ms), because the kernel's time is the chain of key tiles of one CTA.
         npt = 128 // G
-        ctas = max(1, ((T + npt - 1) // npt) * Hkv)
+        ctas = max(1, max((T + npt - 1) // npt, seqs) * Hkv)             # a tile's rows are one sequence's
         return max(1, min(SM_COUNT // ctas, (max_keys + 127) // 128, 16))
     npt = max(1, 64 // G)
     return attn_splits((T + npt - 1) // npt, Hkv, max_keys)
@@ -1027,29 +1028,26 @@ def window_tc_ok(maps: int, pool: int, softcap: float) -> bool:
     return maps == 1 or (maps == 2 and pool == 0 and softcap == 0.0)
 
 
-TANH_SMALL = 0.35        # |score / cap| up to which the tensor-core kernel caps with a polynomial
-
-
-def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int, keep_first: int = 0, pool: int = 0) -> int:
+def window_attn_splits(T: int, Hq: int, Hkv: int, max_keys: int, window: int, keep_first: int = 0, pool: int = 0,
+                       seqs: int = 1) -> int:
     """Key splits of the tensor-core kernel: a CTA's rows span at most the window, their own tokens, the kept first ones and the
     pooled blocks."""
     keys = min(max_keys, window + 128 // (Hq // Hkv) + keep_first) if window else max_keys
-    return attn_splits_for(T, Hq, Hkv, keys + (max_keys // pool if pool else 0))
+    return attn_splits_for(T, Hq, Hkv, keys + (max_keys // pool if pool else 0), seqs)
 
 
 def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, mask_bits, scale: float, window: int, sink,
                         causal: bool, out: torch.Tensor, splits: int = 1, ws: Optional[dict] = None, pdl: bool = False,
-                        keep_first: int = 0, gate: Optional[torch.Tensor] = None, softcap: float = 0.0, score_bound: Optional[float] = None,
+                        keep_first: int = 0, gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
                         blocks=None, diff=None, vdim: int = 128) -> torch.Tensor:
     """Window attention on the tcgen05 kernel: bf16, heads padded to 128, groups of 1, 2, 4, 8 or 16 query heads.  ``sink``:
     whether a valueless key of score 0 takes part, or its score per head, fp32 ``(Hq,)``; ``gate (T, >= Hq)``: logits whose
-    sigmoid multiplies a head's output.  ``softcap``, ``blocks``: see the reference op (trees must not be deeper than the window);
-    ``score_bound``: what no scaled score can exceed, where that is known.  ``diff = (lam, share, eps)``: ``q (T, Hq, 128)`` and the
+    sigmoid multiplies a head's output.  ``softcap``, ``blocks``: see the reference op (trees must not be deeper than the window).
+    ``diff = (lam, share, eps)``: ``q (T, Hq, 128)`` and the
     pools' keys hold 64 columns for each of two maps, ``vdim`` is the true width of the values."""
     lib = load()
     maps, (lam, share, eps) = (1, (None, 0.0, 0.0)) if diff is None else (2, diff)
     kb, vb, block_map, P = blocks if blocks is not None else (None, None, None, 0)
-    poly = softcap > 0.0 and score_bound is not None and score_bound <= TANH_SMALL * softcap
     T, Hq, D = q.shape
     sinks = sink if isinstance(sink, torch.Tensor) else None
     G, S, _ = k_pool.shape
@@ -1059,7 +1057,7 @@ def window_attention_tc(q, k_pool, v_pool, slot_map, seq_rows, cu_q, past_lens, 
         _p(ws["o"] if splits > 1 else None), _p(ws["ml"] if splits > 1 else None), _p(status_word(q.device)), seq_rows.numel(), T, Hq,
         G, S, slot_map.shape[1], mask_bits.shape[1] if mask_bits is not None else 0, int(causal), int(splits), ctypes.c_float(scale),
         int(window), int(sinks is not None or bool(sink)), int(keep_first), _sinks(sinks, Hq), *_head_gate(gate), ctypes.c_float(softcap),
-        int(poly), int(P), _p(kb), _p(vb), kb.shape[1] if P else 0, _p(block_map), block_map.shape[1] if P else 0, maps, _p(lam),
+        int(P), _p(kb), _p(vb), kb.shape[1] if P else 0, _p(block_map), block_map.shape[1] if P else 0, maps, _p(lam),
         ctypes.c_float(share), ctypes.c_float(eps), int(vdim), ctypes.c_longlong(S * 128), ctypes.c_longlong(128), out.stride(0), int(pdl), _stream()), "js_window_attention_tc")
     return out
 
