@@ -1,9 +1,9 @@
 """Paged engine: AR vs batched decode, checking that a batch reproduces per-prompt outputs.
 
-    python examples/engine_generate.py [/path/to/model | karuzen | zasipel | kizezen]
+    python examples/engine_generate.py [/path/to/model | karuzen | zasipel | kizezen | sogidra]
 
-Any registered model family loads from its directory; ``karuzen``, ``zasipel`` and ``kizezen`` are tiny random models of those
-designs, no argument a tiny random Qwen3.  The batch is run once more with its prompts fed in portions beside the others' decode steps.
+Any registered model family loads from its directory; ``karuzen``, ``zasipel``, ``kizezen`` and ``sogidra`` are tiny random
+models of those designs, no argument a tiny random Qwen3.  The batch is run once more with its prompts fed in portions beside the others' decode steps.
 
 Reference counterpart: ``examples/engine/jetspec_engine_generate.py:19-64``."""
 import os
@@ -14,11 +14,12 @@ import torch
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))   # run from a checkout
 
 from jetspec_b200 import JetSpecEngine, SamplingParams  # noqa: E402
-from jetspec_b200.models import (KaruzenForCausalLM, KizezenForCausalLM, Qwen3ForCausalLM, ZasipelForCausalLM,  # noqa: E402
-                                 karuzen_tiny_config, kizezen_tiny_config, tiny_config, zasipel_tiny_config)
+from jetspec_b200.models import (KaruzenForCausalLM, KizezenForCausalLM, Qwen3ForCausalLM, SogidraForCausalLM,  # noqa: E402
+                                 ZasipelForCausalLM, karuzen_tiny_config, kizezen_tiny_config, sogidra_tiny_config, tiny_config,
+                                 zasipel_tiny_config)
 
 TINY = {"karuzen": (KaruzenForCausalLM, karuzen_tiny_config), "zasipel": (ZasipelForCausalLM, zasipel_tiny_config),
-        "kizezen": (KizezenForCausalLM, kizezen_tiny_config)}
+        "kizezen": (KizezenForCausalLM, kizezen_tiny_config), "sogidra": (SogidraForCausalLM, sogidra_tiny_config)}
 
 if __name__ == "__main__":
     dev = "cuda" if torch.cuda.is_available() else "cpu"
