@@ -121,7 +121,7 @@ def linear_f32(x, w):
 
 
 def rotate_norm(x, positions, dims, base, eps):
-    if _kern_any(x):
+    if _kern_any(x) and x.shape[-1] <= 512:
         return _ext().rotate_norm(x, positions, dims, base, eps)
     return ref.rotate_norm(x, positions, dims, base, eps)
 

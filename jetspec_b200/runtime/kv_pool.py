@@ -186,12 +186,14 @@ class PagedKVPool:
         """Pool the blocks whose last token is among the positions ``[past, past + n)`` of slot-map row ``row``."""
         if self.kv_blocks is None or n <= 0:
             return
+        done = [li for li, P in enumerate(self.block_sizes) if P and (past + n) // P > past // P]
+        if not done:
+            return
         from .. import ops
         i32 = lambda *v: torch.tensor(v, dtype=torch.int32, device=self.device)
         rows, cu_q, past_t = i32(row), i32(0, n), i32(past)
-        for li, (kv, kb) in enumerate(zip(self.kv_layers, self.kv_blocks)):
-            if kb is not None and (past + n) // self.block_sizes[li] > past // self.block_sizes[li]:
-                ops.pool_blocks(*kv, *self.blocks(li), self.slot_map, rows, cu_q, past_t)
+        for li in done:
+            ops.pool_blocks(*self.kv_layers[li], *self.blocks(li), self.slot_map, rows, cu_q, past_t)
 
     # -- sequences ------------------------------------------------------------
     def has(self, seq_id: int) -> bool:

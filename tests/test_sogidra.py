@@ -55,7 +55,7 @@ def test_xielu(arm):
 
 
 @pytest.mark.parametrize("arm", ARMS)
-@pytest.mark.parametrize("every,coef", [(1, 0.3), (7, 0.6), (128, 1.5)])
+@pytest.mark.parametrize("every,coef", [(1, 0.3), (7, 0.6), (100, 1.5)])
 def test_query_temperature_steps_where_it_should(arm, every, coef):
     from jetspec_b200 import ops
     pos = torch.tensor([0, 1, every - 2, every - 1, every, 2 * every - 2, 2 * every - 1, 5000]).clamp(min=0)
@@ -189,7 +189,7 @@ def _pooled_case(arm, H, G, D, size, P, cap, scale, past, n, parents=None, mask=
     return got.float().cpu().view(n, H, D), formula
 
 
-SHAPES = [(4, 2, 16, 5, 3, 8.0), (3, 1, 20, 1, 1, 30.0), (6, 3, 128, 40, 12, 50.0), (20, 1, 24, 9, 2, 3.0), (2, 1, 160, 33, 5, 20.0), (5, 5, 10, 100, 64, 0.0)]
+SHAPES = [(4, 2, 16, 5, 3, 8.0), (3, 1, 20, 1, 1, 30.0), (6, 2, 128, 44, 10, 45.0), (20, 1, 24, 9, 2, 3.0), (2, 1, 160, 33, 5, 20.0), (5, 5, 10, 100, 64, 0.0)]
 
 
 @pytest.mark.parametrize("arm", ARMS)
@@ -262,7 +262,7 @@ def _diff_case(arm, H, G, D, V, scale, past, n, parents=None, mask=None, big=Non
     return got.float().cpu().view(n, H, V), formula
 
 
-DIFFS = [(4, 2, 16, 24), (3, 1, 20, 8), (6, 3, 64, 128), (20, 1, 12, 16), (2, 1, 80, 136), (5, 5, 9, 11), (8, 1, 48, 96), (32, 2, 64, 100)]
+DIFFS = [(4, 2, 16, 24), (3, 1, 20, 8), (6, 2, 64, 128), (20, 1, 12, 16), (2, 1, 80, 136), (5, 5, 9, 11), (8, 1, 40, 88), (32, 2, 64, 100)]
 
 
 @pytest.mark.parametrize("arm", ARMS)
